@@ -150,7 +150,9 @@ enum {
      * gate_up projection followed by silu_and_mul (src/models/utils.cc:41-57). */
     B200_EPILOGUE_SWIGLU = 1,
     B200_EPILOGUE_GEGLU = 2,     /* tanh-approximated GELU, as gelu_and_mul (src/layers/activation.cu:11-13) */
-    B200_EPILOGUE_GEGLU_ERF = 3  /* exact GELU, as torch::gelu in MoELayer::forward (src/moe/moe.cc:80) */
+    B200_EPILOGUE_GEGLU_ERF = 3, /* exact GELU, as torch::gelu in MoELayer::forward (src/moe/moe.cc:80) */
+    /* y[m, n] = max(acc[m, n], 0)^2, not gated: N outputs (no counterpart in the reference). */
+    B200_EPILOGUE_RELU2 = 4
 };
 
 /* LinearBase::forward (src/layers/linear.cc:24-26): y = x W^T (+ bias), bf16 in,
@@ -303,6 +305,54 @@ B200_API int b200_sample_from_probs(int32_t* out, const float* probs, int rows, 
                                     const int32_t* top_k, int top_k_value, const float* top_p,
                                     float top_p_value, const float* uniform, b200_stream_t stream);
 
+/* ---- latent attention, table routing, fp32 residual (no counterparts in the reference) --------- */
+
+/* Attention in the latent space: every query row attends over one shared latent per token that serves
+ * as key and value of all heads (the per-head up-projections are absorbed into the query before and
+ * applied to the result after).  Row i sees keys [0, row_len[i]) of page-table row row_table[i]:
+ *   out[i, h, :] = softmax_j(scale * q[i, h] . c_j) c_j.
+ * q, out [rows, heads, width] contiguous; cache [num_slots, width]; width a multiple of 128.
+ * dtype B200_DTYPE_*.  bf16 with width <= 512 runs split-KV on the tcgen05 tensor cores; everything else
+ * on a plain kernel (as it does with plain != 0).  workspace: b200_latent_attention_workspace_bytes. */
+B200_API int64_t b200_latent_attention_workspace_bytes(int rows, int heads, int width);
+B200_API int b200_latent_attention(void* out, const void* q, const void* cache, int64_t num_slots,
+                                   const int32_t* page_table, int64_t page_table_stride,
+                                   const int32_t* row_table, const int32_t* row_len, int rows, int heads,
+                                   int width, int page_size, float scale, int dtype, int plain,
+                                   void* workspace, int64_t workspace_bytes, b200_stream_t stream);
+
+/* residual[t, :] += sum_k src_scale * src[src_rows[t * src_top + k], :]   (src NULL: nothing added;
+ * src_rows NULL: row t; init != 0: the sum replaces the residual instead, e.g. an embedding lookup), then
+ *   out = out_scale * residual / sqrt(mean(residual^2) + eps) * (weight + weight_offset)
+ * to row t, or to the rows out_rows[t * out_top + k].  residual fp32 [tokens, padded]; src, weight, out of
+ * `dtype`; the mean is over `width`, columns [width, padded) are zero and stay so.  padded % 64 == 0.
+ * A src row outside [0, src_count) adds nothing and is reported in the device status word. */
+B200_API int b200_residual_norm(void* out, const int32_t* out_rows, int out_top, float* residual,
+                                const void* src, const int32_t* src_rows, int src_top, int64_t src_count,
+                                float src_scale, int init, const void* weight, float weight_offset,
+                                float out_scale, int tokens, int width, int padded, float eps, int dtype,
+                                b200_stream_t stream);
+
+/* Expert placement for a table of token id -> experts ([vocab, top] int32): counts[e] rows of expert e,
+ * offsets[e] their first row (offsets[experts] = the total) and rows[t * top + k], the row of token t's
+ * k-th expert in the expert-sorted order. */
+B200_API int b200_table_route(int32_t* rows, int32_t* counts, int32_t* offsets, const int32_t* table,
+                              const int32_t* token_ids, int tokens, int vocab, int top, int experts,
+                              b200_stream_t stream);
+
+/* One projection per head in one launch: y[m, h*N + n] = sum_k x[m, h*K + k] w[h*N + n, k] for
+ * h < heads.  x [M, heads*K], y [M, heads*N] contiguous, w [heads*N, K]. */
+B200_API int b200_linear_heads(void* y, const void* x, const void* w, int M, int heads, int N, int K,
+                               b200_stream_t stream);
+
+/* The fp32 counterparts of b200_linear / the grouped expert GEMM / b200_linear_heads, in true fp32 (no
+ * tensor cores): y[m, n] over `groups` problems.  counts/offsets (device, [groups]) non-NULL: group g
+ * multiplies rows [offsets[g], offsets[g] + counts[g]) of x; NULL and groups > 1: per-head columns as in
+ * b200_linear_heads.  max_rows bounds M or any count. */
+B200_API int b200_linear_f32(float* y, const float* x, const float* w, int max_rows, int N, int K,
+                             int groups, const int32_t* counts, const int32_t* offsets, int epilogue,
+                             b200_stream_t stream);
+
 /* ---- tensor-parallel all-reduce (include/sglang/distributed/distributed.h:24) --- */
 
 /* One process per GPU.  A communicator owns this rank's two exchange buffers (call parity 0 / 1)
@@ -420,18 +470,66 @@ typedef struct b200_step {
 
 typedef struct b200_engine b200_engine;
 
+/* Models whose layers are listed one by one (no counterpart in the reference, whose models repeat one
+ * layer): every layer names its mixer and its feed-forward with their own sizes.  The residual stream
+ * of such a model is fp32.  All matrices are stored [out, in] with both sides padded with zeros to a
+ * multiple of 64 (b200_pad_width; head and value dimensions up to 128 are padded to 128, latent widths
+ * to a multiple of 128), vectors likewise; norms divide by the true width. */
+enum { B200_DTYPE_BF16 = 0, B200_DTYPE_F32 = 1 };
+enum { B200_MIXER_LATENT_ATTENTION = 0 };
+enum { B200_MLP_NONE = 0, B200_MLP_DENSE = 1, B200_MLP_TABLE_MOE = 2 };
+
+typedef struct b200_layer_config {
+    int32_t mixer;         /* B200_MIXER_* */
+    int32_t heads;
+    int32_t head_dim;      /* query / key dimensions per head */
+    int32_t value_dim;
+    int32_t q_rank;        /* width of the query latent */
+    int32_t kv_rank;       /* width of the key / value latent: what the cache holds per token */
+    float score_scale;
+    int32_t mlp;           /* B200_MLP_* */
+    int32_t intermediate;  /* of the dense layer, or of each expert */
+    int32_t epilogue;      /* B200_EPILOGUE_*: what is between the up and the down projection; a gated one
+                              has gate and up stacked in "mlp_up" */
+    int32_t num_experts;
+    int32_t experts_per_tok; /* width of the token-id -> experts table; each chosen expert weighs 1 / that */
+} b200_layer_config;
+
+typedef struct b200_stack_config {
+    int32_t num_layers;
+    const b200_layer_config* layers;
+    int32_t dtype;       /* B200_DTYPE_*: bf16 matrices and activations, or everything in fp32 */
+    float norm_offset;   /* added to the stored weights of the layer norms and the final norm (0 or 1) */
+    float logit_scale;
+} b200_stack_config;
+
+/* The padded size of a width / of a per-head dimension / of a latent width (see above). */
+B200_API int b200_pad_width(int n);
+B200_API int b200_pad_head_dim(int n);
+B200_API int b200_pad_latent(int n);
+
 /* Engine::Engine (src/engine/engine.cc:412-489): allocates weights (uninitialised), the KV
  * pool [2, L, (num_pages+1)*page_size, kv_heads/tp, head_dim], the page table and token pool
  * [max_running_req+1, align32(max_seq_len)] (dummy row filled with slot num_pages*page_size),
  * RoPE tables and activation buffers on the current device. */
 B200_API int b200_engine_create(const b200_model_config* model, const b200_engine_config* config,
                                 b200_engine** out);
+/* The same for a model whose layers are listed one by one; of `model` only num_layers, hidden_size,
+ * vocab_size, rms_norm_eps and tie_word_embeddings are read.  One latent pool per layer
+ * [(num_pages+1)*page_size, pad(kv_rank)] stands where the K/V pools are.  tp_size must be 1. */
+B200_API int b200_engine_create_stack(const b200_model_config* model, const b200_stack_config* stack,
+                                      const b200_engine_config* config, b200_engine** out);
 B200_API int b200_engine_destroy(b200_engine* engine);
 
 /* Device address and size of a named tensor: "embed", "lm_head", "final_norm", "rope_cos",
  * "rope_sin", "page_table", "token_pool", "kv_cache", "logits", "next_tokens", and per layer
  * "qkv", "qkv_bias", "o", "gate_up", "down", "input_norm", "post_norm", "q_norm", "k_norm",
- * "router", "experts_gate_up", "experts_down" (layouts: src/models/weight_loader.cc:27-33,455,497). */
+ * "router", "experts_gate_up", "experts_down" (layouts: src/models/weight_loader.cc:27-33,455,497).
+ * Layer stacks: per layer "norm1", "norm2", "down_qkv" [q latent + kv latent, hidden], "q_latent_norm",
+ * "kv_latent_norm", "uq" [heads*dim, q latent], "uk" [heads*dim, kv latent], "uk_absorb" (per head the
+ * transpose of its rows of uk: [heads, kv latent, dim]), "uv" [heads*vdim, kv latent], "o"
+ * [hidden, heads*vdim], "mlp_up", "mlp_down" (experts stacked), "expert_table" int32 [vocab, experts
+ * per token], "latent_cache". */
 B200_API int b200_engine_tensor(b200_engine* engine, const char* name, int layer, void** device_ptr,
                                 int64_t* nbytes);
 /* Synchronous host-to-device copy into a named tensor (nbytes must equal its size). */
@@ -479,8 +577,19 @@ B200_API int b200_engine_step_async(b200_engine* engine, const b200_step* step, 
 B200_API int b200_engine_wait(b200_engine* engine, int64_t ticket, const int32_t** tokens,
                               const uint8_t** finished);
 
-/* Copies the bf16 logits [rows, vocab] of the last step to host memory (synchronous). */
+/* Copies the logits [rows, vocab] of the last step to host memory (synchronous): bf16, or fp32 for a
+ * layer stack that runs in fp32. */
 B200_API int b200_engine_read_logits(b200_engine* engine, void* host, int rows);
+
+/* Logits at any tokens of the last step, not only each request's last one (scoring a prompt): the final
+ * hidden states stay on the device until the next step, and this applies the output head to the rows
+ * `tokens` (HOST int32, places in the step's flattened token order) in slabs and copies fp32 logits
+ * [count, vocab] to host memory.  Synchronous.  No counterpart in the reference. */
+B200_API int b200_engine_token_logits(b200_engine* engine, const int32_t* tokens, int count, float* host);
+
+/* Tests: from the next step on, layer stacks copy the fp32 residual stream after every layer to host
+ * memory [num_layers, tokens of the step, hidden] (prefill steps only); NULL turns it off. */
+B200_API int b200_engine_trace_residual(b200_engine* engine, float* host);
 
 /* Tensor parallelism (engine created with tp_size > 1): export this rank's IPC handle
  * (b200_comm_handle_bytes bytes) and connect to all ranks' handles before the first step. */

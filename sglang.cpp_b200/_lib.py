@@ -27,6 +27,11 @@ ERROR_NAMES = {
 EPILOGUE_NONE = 0
 EPILOGUE_SWIGLU = 1
 EPILOGUE_GEGLU = 2
+EPILOGUE_RELU2 = 4
+
+DTYPE_BF16, DTYPE_F32 = 0, 1
+MIXER_LATENT_ATTENTION = 0
+MLP_NONE, MLP_DENSE, MLP_TABLE_MOE = 0, 1, 2
 
 
 class B200Error(RuntimeError):
@@ -92,6 +97,18 @@ PROTOTYPES: dict[str, tuple] = {
     "b200_engine_comm_attach": (_I, [_P, _P, _P, _P]),
     "b200_engine_comm_export": (_I, [_P, _P]),
     "b200_engine_comm_connect": (_I, [_P, _P]),
+    "b200_latent_attention_workspace_bytes": (_L, [_I, _I, _I]),
+    "b200_latent_attention": (_I, [_P, _P, _P, _L, _P, _L, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _L, _P]),
+    "b200_residual_norm": (_I, [_P, _P, _I, _P, _P, _P, _I, _L, _F, _I, _P, _F, _F, _I, _I, _I, _F, _I, _P]),
+    "b200_table_route": (_I, [_P, _P, _P, _P, _P, _I, _I, _I, _I, _P]),
+    "b200_linear_heads": (_I, [_P, _P, _P, _I, _I, _I, _I, _P]),
+    "b200_linear_f32": (_I, [_P, _P, _P, _I, _I, _I, _I, _P, _P, _I, _P]),
+    "b200_pad_width": (_I, [_I]),
+    "b200_pad_head_dim": (_I, [_I]),
+    "b200_pad_latent": (_I, [_I]),
+    "b200_engine_create_stack": (_I, [_P, _P, _P, POINTER(c_void_p)]),
+    "b200_engine_token_logits": (_I, [_P, _P, _I, _P]),
+    "b200_engine_trace_residual": (_I, [_P, _P]),
     "b200_engine_create": (_I, [_P, _P, POINTER(c_void_p)]),
     "b200_engine_destroy": (_I, [_P]),
     "b200_engine_tensor": (_I, [_P, c_char_p, _I, POINTER(c_void_p), POINTER(c_int64)]),
@@ -123,6 +140,24 @@ class ModelConfigStruct(ctypes.Structure):
         ("fused_residual", c_int32), ("attention_bias", c_int32), ("hidden_act", c_int32),
         ("num_experts", c_int32), ("num_experts_per_tok", c_int32),
         ("moe_intermediate_size", c_int32), ("norm_topk_prob", c_int32),
+    ]
+
+
+class LayerConfigStruct(ctypes.Structure):
+    """b200_layer_config."""
+    _fields_ = [
+        ("mixer", c_int32), ("heads", c_int32), ("head_dim", c_int32), ("value_dim", c_int32),
+        ("q_rank", c_int32), ("kv_rank", c_int32), ("score_scale", c_float), ("mlp", c_int32),
+        ("intermediate", c_int32), ("epilogue", c_int32), ("num_experts", c_int32),
+        ("experts_per_tok", c_int32),
+    ]
+
+
+class StackConfigStruct(ctypes.Structure):
+    """b200_stack_config."""
+    _fields_ = [
+        ("num_layers", c_int32), ("layers", POINTER(LayerConfigStruct)), ("dtype", c_int32),
+        ("norm_offset", c_float), ("logit_scale", c_float),
     ]
 
 

@@ -94,6 +94,24 @@ def build(verbose: bool = False, ptxas_v: bool = False, force: bool = False) -> 
     return LIB_PATH
 
 
+def ensure_built() -> Path:
+    """Build unless the library is there and newer than every source; processes that start together
+    wait for one another."""
+    import fcntl
+
+    deps = _sources() + sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h")) + [PKG_DIR.parent / "include" / "b200_token_loop.h"]
+
+    def fresh() -> bool:
+        return LIB_PATH.exists() and all(LIB_PATH.stat().st_mtime >= d.stat().st_mtime for d in deps)
+
+    if fresh():
+        return LIB_PATH
+    LIB_DIR.mkdir(exist_ok=True)
+    with open(LIB_DIR / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return LIB_PATH if fresh() else build()
+
+
 if __name__ == "__main__":
     path = build(verbose="-v" in sys.argv, ptxas_v="--ptxas" in sys.argv, force="-f" in sys.argv)
     print(path)

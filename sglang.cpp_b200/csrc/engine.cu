@@ -16,6 +16,7 @@
 #include <vector>
 
 #include "common.cuh"
+#include "engine_state.h"
 #include "kernels.h"
 
 namespace b200 {
@@ -33,7 +34,8 @@ __global__ void prepare_tokens_kernel(const int32_t* __restrict__ meta, int Bp, 
                                       const int32_t* __restrict__ token_pool, int64_t pt_stride,
                                       int pt_rows, int pt_cols, int32_t* __restrict__ positions,
                                       int32_t* __restrict__ out_loc, int32_t* __restrict__ input_ids,
-                                      int32_t* __restrict__ seq_lens) {
+                                      int32_t* __restrict__ seq_lens, int32_t* __restrict__ token_row,
+                                      int32_t* __restrict__ token_len) {
     pdl_launch_dependents();
     pdl_wait_prior();
     const int32_t* table_idx = meta;
@@ -51,6 +53,10 @@ __global__ void prepare_tokens_kernel(const int32_t* __restrict__ meta, int Bp, 
     const int row = table_idx[lo];
     const bool ok = row >= 0 && row < pt_rows && pos >= 0 && pos < pt_cols;
     positions[i] = pos;
+    if (token_row != nullptr) {   // layer stacks: what every token attends over
+        token_row[i] = ok ? row : 0;
+        token_len[i] = pos + 1;
+    }
     out_loc[i] = ok ? page_table[row * pt_stride + pos] : 0;
     input_ids[i] = ok ? token_pool[row * pt_stride + pos] : 0;
 }
@@ -64,6 +70,22 @@ __global__ void select_last_rows_kernel(uint4* __restrict__ dst, const uint4* __
     const int64_t row = qo[b + 1] - 1;
     for (int v = threadIdx.x; v < vec_per_row; v += blockDim.x)
         dst[static_cast<int64_t>(b) * vec_per_row + v] = src[row * vec_per_row + v];
+}
+
+// dst[i] = src[tokens[i]] for rows of vec_per_row 16-byte vectors.
+__global__ void take_rows_kernel(uint4* __restrict__ dst, const uint4* __restrict__ src,
+                                 const int32_t* __restrict__ tokens, int vec_per_row) {
+    const int64_t i = blockIdx.x, row = tokens[i];
+    for (int v = threadIdx.x; v < vec_per_row; v += blockDim.x) dst[i * vec_per_row + v] = src[row * vec_per_row + v];
+}
+
+// fp32 logits for the sampler, whose keys are bf16.
+__global__ void round_logits_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict__ in, int64_t n) {
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < n;
+         i += static_cast<int64_t>(gridDim.x) * blockDim.x)
+        out[i] = __float2bfloat16_rn(in[i]);
 }
 
 __global__ void scatter_int32_kernel(int32_t* __restrict__ table, int64_t rows, int64_t stride,
@@ -110,21 +132,6 @@ __global__ void fill_int32_kernel(int32_t* p, int32_t v, int64_t n) {
     if (i < n) p[i] = v;
 }
 
-struct LayerWeights {
-    __nv_bfloat16 *qkv = nullptr, *qkv_bias = nullptr, *o = nullptr, *gate_up = nullptr, *down = nullptr;
-    __nv_bfloat16 *input_norm = nullptr, *post_norm = nullptr, *q_norm = nullptr, *k_norm = nullptr;
-    __nv_bfloat16 *router = nullptr, *experts_gate_up = nullptr, *experts_down = nullptr;
-    // qkv and gate_up with the norm weight in front of them folded into their columns (decode steps
-    // whose GEMMs carry the add + norm in their epilogues)
-    __nv_bfloat16 *qkv_folded = nullptr, *gate_up_folded = nullptr;
-    CUtensorMap tmap_k, tmap_v;
-};
-
-struct Tensor {
-    void* ptr;
-    int64_t bytes;
-};
-
 }  // namespace
 }  // namespace b200
 
@@ -146,131 +153,7 @@ int launch_allreduce(b200_comm* c, int parity, int mode, void* out, void* residu
                      int rows, int hidden, float eps, bool round_first, int* status, cudaStream_t stream);
 }
 
-struct b200_engine {
-    b200_model_config m;
-    b200_engine_config c;
-    int device = 0;
-    int hq = 0, hkv = 0, inter = 0, qkv_dim = 0;  // per-rank sizes
-    int moe_inter = 0, experts_local = 0, expert_begin = 0;  // per-rank expert layout
-    int64_t num_slots = 0;
-    int pt_rows = 0, pt_cols = 0;
-    int max_tokens = 0, max_batch = 0;
-    float sm_scale = 0.f;
-
-    std::vector<void*> allocs;
-    std::map<std::string, Tensor> named;  // "name" or "name.<layer>"
-    std::vector<LayerWeights> layers;
-
-    __nv_bfloat16 *embed = nullptr, *lm_head = nullptr, *final_norm = nullptr;
-    float *rope_cos = nullptr, *rope_sin = nullptr;
-    __nv_bfloat16* kv_cache = nullptr;
-    int32_t *page_table = nullptr, *token_pool = nullptr;
-
-    // activations
-    __nv_bfloat16 *x = nullptr, *residual = nullptr, *qkv = nullptr, *attn_out = nullptr, *h = nullptr,
-                  *sel = nullptr, *logits = nullptr;
-    int32_t *positions = nullptr, *out_loc = nullptr, *input_ids = nullptr, *seq_lens = nullptr,
-            *next_tokens = nullptr;
-    void* attn_ws = nullptr;
-    int64_t attn_ws_bytes = 0;
-    __nv_bfloat16* router_logits = nullptr;
-    void* moe_ws = nullptr;
-
-    // per-step metadata: pinned staging + device mirror
-    int32_t* meta_host = nullptr;
-    int32_t* meta_dev = nullptr;
-    int meta_ints = 0;
-    int32_t *scatter_host = nullptr, *scatter_dev = nullptr;
-    int64_t scatter_cap = 0;
-
-    cudaStream_t stream = nullptr;
-    cudaEvent_t ev_meta_done = nullptr, ev_step_begin = nullptr, ev_step_end = nullptr,
-                ev_scatter_done = nullptr;
-    bool meta_in_flight = false, scatter_in_flight = false;
-    int* status = nullptr;
-
-    std::map<int, cudaGraphExec_t> graphs;          // padded decode batch size -> graph ending in argmax
-    std::map<int, cudaGraphExec_t> graphs_sampled;  // ... ending in the sampling kernel
-    std::map<int, int> graph_launches;              // kernels inside each captured graph
-
-    // Optional per-kernel timing of the attention launches of eager steps.
-    bool profile_attention = false;
-    bool capturing = false;
-    std::vector<cudaEvent_t> prof_events;   // 2 per layer
-    std::vector<cudaEvent_t> prof_events_ar;  // 2 per all-reduce call
-    int prof_ar_recorded = 0;
-    int prof_pairs_recorded = 0;
-    int launches_last_step = 0;
-    b200_comm* comm = nullptr;  // tensor parallelism: exchange buffers for the fused all-reduce
-    int64_t comm_buffer_bytes = 0;
-
-    // Results of the steps in flight: a ring of pinned, device-mapped slots the last kernel of a step
-    // writes straight into (tokens, finish flags, the device status words, the ticket), one event each.
-    struct ResultSlot {
-        int32_t* tokens = nullptr;         // [max_batch]
-        uint8_t* finished = nullptr;       // [max_batch]
-        uint8_t* ignore_eos = nullptr;     // [max_batch], written by the host before the launch
-        int32_t* status = nullptr;         // [2] + 64-bit ticket behind them
-        cudaEvent_t done = nullptr;
-        int64_t ticket = -1;
-        int num_reqs = 0;
-    };
-    static constexpr int kResultSlots = 4;
-    ResultSlot ring[kResultSlots];
-    uint8_t* ring_host = nullptr;
-    int64_t next_ticket = 0;
-    int32_t eos_token_id = -1;
-    void* chain_scratch = nullptr;  // fp32 sums, partial sums of squares and barrier words of the decode layer chain
-    // B200_DECODE_CHAIN=1: decode steps run everything between two attention launches as one
-    // persistent kernel (decode_chain.cu).  Off by default: measured on B200 it is the slower of the
-    // two paths (each of its phases pays several ~1 us round trips to L2 that separate launches hide
-    // behind one another under programmatic dependent launch).
-    bool use_chain = false;
-    // Decode steps of a dense, unsharded model of at most 256 tokens: no add + norm kernels.  o_proj and
-    // down_proj add the residual in their split-K epilogue and accumulate each row's sum of squares;
-    // qkv_proj and gate_up_proj read the un-normalised residual against weights with the norm weight
-    // folded in, and scale their accumulator by the row's 1 / rms.  B200_FOLD_NORM=0 turns it off.
-    bool use_fold = true;
-    bool use_fold_heads = true;         // B200_FOLD_HEADS=0: QK-norm + RoPE + K/V store stay a kernel of their own
-    bool folded_valid = false;          // the folded copies match qkv / gate_up / the norm weights
-    unsigned long long* ssq = nullptr;  // [2 * layers + 1, kSsqStride] sums of squares of the residual rows
-    static constexpr int kSsqStride = 256;
-    bool use_pdl = true;  // B200_PDL=0 turns programmatic dependent launches off
-    bool kv_evict_first = true;  // B200_KV_EVICT_FIRST=0: K/V loads with the default L2 policy
-    // Seeds are 64-bit: keep them 8-byte aligned inside the int32 staging block.  The 64-bit step
-    // index follows them, so a captured graph reads a fresh one on every replay.
-    static int seed_offset(int Bp) { return (7 * Bp + 1 + 1) & ~1; }
-    static int step_index_offset(int Bp) { return seed_offset(Bp) + 2 * Bp; }
-};
-
 namespace {
-
-int dev_alloc(b200_engine* e, void** out, int64_t bytes, bool zero) {
-    void* p = nullptr;
-    if (bytes <= 0) bytes = 16;
-    B200_CHECK_CUDA(cudaMalloc(&p, static_cast<size_t>(bytes)));
-    e->allocs.push_back(p);
-    if (zero) B200_CHECK_CUDA(cudaMemset(p, 0, static_cast<size_t>(bytes)));
-    *out = p;
-    return B200_OK;
-}
-
-template <typename T>
-int named_alloc(b200_engine* e, T** out, const std::string& name, int64_t elems, bool zero = false) {
-    void* p = nullptr;
-    const int64_t bytes = elems * static_cast<int64_t>(sizeof(T));
-    int err = dev_alloc(e, &p, bytes, zero);
-    if (err != B200_OK) return err;
-    *out = static_cast<T*>(p);
-    e->named[name] = Tensor{p, bytes};
-    return B200_OK;
-}
-
-#define B200_TRY(expr)                  \
-    do {                                \
-        int err__ = (expr);             \
-        if (err__ != B200_OK) return err__; \
-    } while (0)
 
 int build_rope_tables(b200_engine* e) {
     // cos/sin [max_position, head_dim / 2] in fp32, with the reference's sequence of fp32
@@ -325,16 +208,99 @@ int ensure_folded(b200_engine* e) {
     return B200_OK;
 }
 
+// First kernel of every step: per-token quantities from the staged per-request ones.
+int enqueue_prepare(b200_engine* e, int Bp, int T) {
+    const int n = T > Bp ? T : Bp;
+    B200_CHECK_CUDA(launch_kernel(prepare_tokens_kernel, dim3(div_ceil(n, 256)), dim3(256), 0, e->stream,
+                                  dim3(1, 1, 1), static_cast<const int32_t*>(e->meta_dev), Bp, T,
+                                  static_cast<const int32_t*>(e->page_table),
+                                  static_cast<const int32_t*>(e->token_pool), static_cast<int64_t>(e->pt_cols),
+                                  e->pt_rows, e->pt_cols, e->positions, e->out_loc, e->input_ids, e->seq_lens,
+                                  e->stack ? stack_token_row(e) : nullptr, e->stack ? stack_token_len(e) : nullptr));
+    return B200_OK;
+}
+
+// What is the same for every model: the final hidden states, their row size, the output head.
+const void* hidden_states(const b200_engine* e) { return e->stack ? stack_hidden(e) : e->x; }
+int hidden_row_bytes(const b200_engine* e) { return e->stack ? stack_row_bytes(e) : e->m.hidden_size * 2; }
+int logits_ld(const b200_engine* e) { return e->stack ? stack_logits_ld(e) : e->m.vocab_size; }
+bool logits_f32(const b200_engine* e) { return e->stack && stack_dtype(e) == B200_DTYPE_F32; }
+int output_head(b200_engine* e, const void* rows, int count) {
+    if (e->stack) return layer_stack_head(e, e->logits, rows, count);
+    return launch_linear(e->logits, rows, e->lm_head, nullptr, count, e->m.vocab_size, e->m.hidden_size,
+                         e->m.hidden_size, B200_EPILOGUE_NONE, e->status, e->stream);
+}
+
+// Last part of every step: each request's last row, the head, token selection and write-back.
+int enqueue_output(b200_engine* e, int phase, int B, int Bp, bool sampling, uint64_t step_index) {
+    const b200_model_config& m = e->m;
+    cudaStream_t s = e->stream;
+    const int32_t* meta_table_idx = e->meta_dev;
+    const int32_t* meta_qo = e->meta_dev + 2 * Bp;
+    const void* head_in = hidden_states(e);
+    if (phase == B200_PHASE_PREFILL) {
+        B200_CHECK_CUDA(launch_kernel(select_last_rows_kernel, dim3(Bp), dim3(128), 0, s, dim3(1, 1, 1),
+                                      reinterpret_cast<uint4*>(e->sel), static_cast<const uint4*>(head_in),
+                                      meta_qo, hidden_row_bytes(e) / 16));
+        head_in = e->sel;
+    }
+    B200_TRY(output_head(e, head_in, Bp));
+    const int ld = logits_ld(e);
+    // Token write-back, token_pool[table_idx[i], write_pos[i]] = next_tokens[i], by the kernel that picks the token.
+    TokenWriteBack wb;
+    wb.pool = e->token_pool;
+    wb.rows = e->pt_rows;
+    wb.stride = e->pt_cols;
+    wb.cols = e->pt_cols;
+    wb.table_idx = meta_table_idx;
+    wb.write_pos = e->meta_dev + 3 * Bp + 1;
+    wb.count = B;
+    if (sampling) {
+        const void* logits = e->logits;
+        if (logits_f32(e)) {
+            const int64_t n = static_cast<int64_t>(Bp) * ld;
+            B200_CHECK_CUDA(launch_kernel(round_logits_kernel, dim3(static_cast<unsigned>((n + 1023) / 1024)), dim3(256), 0, s,
+                                          dim3(1, 1, 1), static_cast<__nv_bfloat16*>(e->logits_bf16),
+                                          reinterpret_cast<const float*>(e->logits), n));
+            logits = e->logits_bf16;
+        }
+        // meta layout after write_pos[Bp]: temperatures | top_k | top_p | seeds (2 ints each)
+        const int32_t* sp = e->meta_dev + 4 * Bp + 1;
+        return launch_sample(e->next_tokens, logits, B, m.vocab_size, ld, reinterpret_cast<const float*>(sp), sp + Bp,
+                             reinterpret_cast<const float*>(sp + 2 * Bp),
+                             reinterpret_cast<const uint64_t*>(e->meta_dev + e->seed_offset(Bp)), step_index, nullptr, s,
+                             reinterpret_cast<const uint64_t*>(e->meta_dev + e->step_index_offset(Bp)), &wb);
+    }
+    if (logits_f32(e))
+        return launch_argmax_f32(e->next_tokens, reinterpret_cast<const float*>(e->logits), B, m.vocab_size, ld, s, &wb);
+    return launch_argmax(e->next_tokens, e->logits, B, m.vocab_size, ld, s, &wb);
+}
+
+// A step of a model whose layers are listed one by one.
+int enqueue_stack_forward(b200_engine* e, int phase, int B, int Bp, int T, bool sampling, uint64_t step_index) {
+    const uint64_t launches_before = kernel_launch_count();
+    struct PdlScope {
+        ~PdlScope() { set_pdl_launches(false); }
+    } pdl_scope;
+    set_pdl_launches(false);   // the first kernel follows a copy
+    B200_TRY(enqueue_prepare(e, Bp, T));
+    set_pdl_launches(e->use_pdl && !e->trace_residual && !(e->profile_attention && !e->capturing));
+    B200_TRY(layer_stack_enqueue(e, phase, Bp, T));
+    B200_TRY(enqueue_output(e, phase, B, Bp, sampling, step_index));
+    e->launches_last_step = static_cast<int>(kernel_launch_count() - launches_before);
+    return B200_OK;
+}
+
 // The layer stack on `T` tokens of `Bp` requests; everything is enqueued on e->stream.
 int enqueue_forward(b200_engine* e, int phase, int B, int Bp, int T, int max_extend,
                     bool sampling = false, uint64_t step_index = 0) {
+    if (e->stack) return enqueue_stack_forward(e, phase, B, Bp, T, sampling, step_index);
     const b200_model_config& m = e->m;
     cudaStream_t s = e->stream;
     const int hidden = m.hidden_size, d = m.head_dim;
     const uint64_t launches_before = kernel_launch_count();
     const int32_t* meta_table_idx = e->meta_dev;
     const int32_t* meta_qo = e->meta_dev + 2 * Bp;
-
     const bool fold = fold_supported(e, phase, T);
     // The residual stream starts at zero, so the first fused add+norm leaves residual = embedding
     // (what the reference's layer 0 does with `residual = x`).  With the norms folded into the GEMMs
@@ -348,15 +314,7 @@ int enqueue_forward(b200_engine* e, int phase, int B, int Bp, int T, int max_ext
         ~PdlScope() { set_pdl_launches(false); }
     } pdl_scope;
     set_pdl_launches(false);  // the first kernel follows a memset / copy: ordinary dependency
-    {
-        const int n = T > Bp ? T : Bp;
-        B200_CHECK_CUDA(launch_kernel(prepare_tokens_kernel, dim3(div_ceil(n, 256)), dim3(256), 0, s,
-                                      dim3(1, 1, 1), static_cast<const int32_t*>(e->meta_dev), Bp, T,
-                                      static_cast<const int32_t*>(e->page_table),
-                                      static_cast<const int32_t*>(e->token_pool),
-                                      static_cast<int64_t>(e->pt_cols), e->pt_rows, e->pt_cols, e->positions,
-                                      e->out_loc, e->input_ids, e->seq_lens));
-    }
+    B200_TRY(enqueue_prepare(e, Bp, T));
     // (Per-kernel event timing wants each kernel to start after its predecessor ends.)
     // The embedding is launched as an ordinary dependent of the prepare kernel: every later kernel
     // of the step can then rely on seq_lens / positions / out_loc being complete even in code it
@@ -633,36 +591,7 @@ int enqueue_forward(b200_engine* e, int phase, int B, int Bp, int T, int max_ext
         B200_TRY(launch_rmsnorm(e->x, e->residual, e->final_norm, T, hidden, m.rms_norm_eps, s));
     else
         B200_TRY(add_norm(e->final_norm));
-    const __nv_bfloat16* head_in = e->x;
-    if (phase == B200_PHASE_PREFILL) {
-        B200_CHECK_CUDA(launch_kernel(select_last_rows_kernel, dim3(Bp), dim3(128), 0, s, dim3(1, 1, 1),
-                                      reinterpret_cast<uint4*>(e->sel), reinterpret_cast<const uint4*>(e->x),
-                                      meta_qo, hidden / 8));
-        head_in = e->sel;
-    }
-    B200_TRY(launch_linear(e->logits, head_in, e->lm_head, nullptr, Bp, m.vocab_size, hidden, hidden,
-                           B200_EPILOGUE_NONE, e->status, s));
-    // Token write-back, token_pool[table_idx[i], write_pos[i]] = next_tokens[i], by the kernel that picks the token.
-    TokenWriteBack wb;
-    wb.pool = e->token_pool;
-    wb.rows = e->pt_rows;
-    wb.stride = e->pt_cols;
-    wb.cols = e->pt_cols;
-    wb.table_idx = meta_table_idx;
-    wb.write_pos = e->meta_dev + 3 * Bp + 1;
-    wb.count = B;
-    if (sampling) {
-        // meta layout after write_pos[Bp]: temperatures | top_k | top_p | seeds (2 ints each)
-        const int32_t* sp = e->meta_dev + 4 * Bp + 1;
-        B200_TRY(launch_sample(e->next_tokens, e->logits, B, m.vocab_size, m.vocab_size,
-                               reinterpret_cast<const float*>(sp), sp + Bp,
-                               reinterpret_cast<const float*>(sp + 2 * Bp),
-                               reinterpret_cast<const uint64_t*>(e->meta_dev + e->seed_offset(Bp)), step_index,
-                               nullptr, s,
-                               reinterpret_cast<const uint64_t*>(e->meta_dev + e->step_index_offset(Bp)), &wb));
-    } else {
-        B200_TRY(launch_argmax(e->next_tokens, e->logits, B, m.vocab_size, m.vocab_size, s, &wb));
-    }
+    B200_TRY(enqueue_output(e, phase, B, Bp, sampling, step_index));
     e->launches_last_step = static_cast<int>(kernel_launch_count() - launches_before);
     return B200_OK;
 }
@@ -722,56 +651,145 @@ int stage_step(b200_engine* e, const b200_step* st, int Bp, int* T_out, int* max
 
 extern "C" {
 
-int b200_engine_create(const b200_model_config* model, const b200_engine_config* config,
-                       b200_engine** out) {
+// Weights, K/V pools and activations of the grouped-query models.
+static int alloc_gqa_model(b200_engine* e) {
+    const b200_model_config& m = e->m;
+    const b200_engine_config& c = e->c;
+    const int64_t Tm = e->max_tokens;
+    const int64_t H = m.hidden_size, D = m.head_dim;
+    B200_TRY(named_alloc(e, &e->embed, "embed", static_cast<int64_t>(m.vocab_size) * H));
+    if (m.tie_word_embeddings) {
+        e->lm_head = e->embed;
+        e->named["lm_head"] = e->named["embed"];
+    } else {
+        B200_TRY(named_alloc(e, &e->lm_head, "lm_head", static_cast<int64_t>(m.vocab_size) * H));
+    }
+    B200_TRY(named_alloc(e, &e->final_norm, "final_norm", H));
+    B200_TRY(named_alloc(e, &e->rope_cos, "rope_cos", static_cast<int64_t>(m.max_position) * (D / 2)));
+    B200_TRY(named_alloc(e, &e->rope_sin, "rope_sin", static_cast<int64_t>(m.max_position) * (D / 2)));
+    B200_TRY(build_rope_tables(e));
+    B200_TRY(named_alloc(e, &e->kv_cache, "kv_cache", 2 * static_cast<int64_t>(m.num_layers) * e->num_slots * e->hkv * D, true));
+    e->layers.resize(m.num_layers);
+    for (int l = 0; l < m.num_layers; ++l) {
+        LayerWeights& L = e->layers[l];
+        const std::string sfx = "." + std::to_string(l);
+        B200_TRY(named_alloc(e, &L.qkv, "qkv" + sfx, static_cast<int64_t>(e->qkv_dim) * H));
+        if (m.attention_bias) B200_TRY(named_alloc(e, &L.qkv_bias, "qkv_bias" + sfx, e->qkv_dim));
+        B200_TRY(named_alloc(e, &L.o, "o" + sfx, H * e->hq * D));
+        B200_TRY(named_alloc(e, &L.input_norm, "input_norm" + sfx, H));
+        B200_TRY(named_alloc(e, &L.post_norm, "post_norm" + sfx, H));
+        if (m.qk_norm) {
+            B200_TRY(named_alloc(e, &L.q_norm, "q_norm" + sfx, D));
+            B200_TRY(named_alloc(e, &L.k_norm, "k_norm" + sfx, D));
+        }
+        if (m.num_experts > 0) {
+            const int64_t ie = e->moe_inter, el = e->experts_local;
+            B200_TRY(named_alloc(e, &L.router, "router" + sfx, static_cast<int64_t>(m.num_experts) * H));
+            B200_TRY(named_alloc(e, &L.experts_gate_up, "experts_gate_up" + sfx, el * 2 * ie * H));
+            B200_TRY(named_alloc(e, &L.experts_down, "experts_down" + sfx, el * H * ie));
+        } else {
+            B200_TRY(named_alloc(e, &L.gate_up, "gate_up" + sfx, 2 * static_cast<int64_t>(e->inter) * H));
+            B200_TRY(named_alloc(e, &L.down, "down" + sfx, H * e->inter));
+        }
+        const __nv_bfloat16* kc = e->kv_cache + static_cast<int64_t>(l) * e->num_slots * e->hkv * D;
+        const __nv_bfloat16* vc = kc + static_cast<int64_t>(m.num_layers) * e->num_slots * e->hkv * D;
+        B200_TRY(make_kv_tmap(&L.tmap_k, kc, e->num_slots, e->hkv, c.page_size));
+        B200_TRY(make_kv_tmap(&L.tmap_v, vc, e->num_slots, e->hkv, c.page_size));
+    }
+    const int64_t inter_buf = m.num_experts > 0 ? m.moe_intermediate_size : e->inter;
+    B200_TRY(named_alloc(e, &e->x, "x", Tm * H));
+    B200_TRY(named_alloc(e, &e->residual, "residual", Tm * H));
+    B200_TRY(named_alloc(e, &e->qkv, "qkv_act", Tm * e->qkv_dim));
+    B200_TRY(named_alloc(e, &e->attn_out, "attn_out", Tm * e->hq * D));
+    B200_TRY(named_alloc(e, &e->h, "mlp_act", Tm * inter_buf));
+    B200_TRY(named_alloc(e, &e->sel, "sel", static_cast<int64_t>(e->max_batch) * H));
+    B200_TRY(named_alloc(e, &e->logits, "logits", static_cast<int64_t>(e->max_batch) * m.vocab_size));
+    e->comm_buffer_bytes = Tm * H * 2;
+    if (c.tp_size > 1) B200_TRY(b200_comm_create(c.tp_rank, c.tp_size, e->comm_buffer_bytes, &e->comm));
+    if (m.num_experts > 0) {
+        B200_TRY(named_alloc(e, &e->router_logits, "router_logits", Tm * m.num_experts));
+        B200_TRY(dev_alloc(e, &e->moe_ws,
+                        moe_workspace_bytes(static_cast<int>(Tm), m.num_experts, m.num_experts_per_tok, m.hidden_size,
+                                            e->moe_inter),
+                        false));
+    }
+    if (const char* v = getenv("B200_FOLD_NORM")) e->use_fold = atoi(v) != 0;
+    if (const char* v = getenv("B200_FOLD_HEADS")) e->use_fold_heads = atoi(v) != 0;
+    if (e->use_fold && c.tp_size == 1 && m.num_experts == 0 && fold_shapes_ok(e)) {
+        for (LayerWeights& L : e->layers) {
+            void* p = nullptr;
+            B200_TRY(dev_alloc(e, &p, static_cast<int64_t>(e->qkv_dim) * H * 2, false));
+            L.qkv_folded = static_cast<__nv_bfloat16*>(p);
+            B200_TRY(dev_alloc(e, &p, 2 * static_cast<int64_t>(e->inter) * H * 2, false));
+            L.gate_up_folded = static_cast<__nv_bfloat16*>(p);
+        }
+        void* p = nullptr;
+        B200_TRY(dev_alloc(e, &p, static_cast<int64_t>(2 * m.num_layers + 1) * b200_engine::kSsqStride * 8, true));
+        e->ssq = static_cast<unsigned long long*>(p);
+    }
+    B200_TRY(dev_alloc(e, &e->chain_scratch, decode_chain_scratch_bytes(m.hidden_size), true));
+    e->attn_ws_bytes = decode_workspace_bytes(e->max_batch, e->hq, e->hkv);
+    B200_TRY(dev_alloc(e, &e->attn_ws, e->attn_ws_bytes, true));
+
+    return B200_OK;
+}
+
+static int create_engine(const b200_model_config* model, const b200_stack_config* stack,
+                         const b200_engine_config* config, b200_engine** out) {
     B200_CHECK_ARG(model && config && out, "engine_create: NULL argument");
     const b200_model_config& m = *model;
     const b200_engine_config& c = *config;
     B200_CHECK_ARG(m.num_layers > 0 && m.hidden_size > 0 && m.vocab_size > 0, "engine_create: bad model size");
-    B200_CHECK_ARG(m.head_dim == 128, "engine_create: head_dim must be 128 (as the reference's attention is)");
-    B200_CHECK_ARG(m.hidden_size % 64 == 0 && m.intermediate_size % 64 == 0,
-                   "engine_create: hidden and intermediate sizes must be multiples of 64");
     B200_CHECK_ARG(c.tp_size >= 1 && c.tp_rank >= 0 && c.tp_rank < c.tp_size, "engine_create: bad TP rank/size");
-    B200_CHECK_ARG(m.num_qo_heads % c.tp_size == 0, "num_qo_heads must be divisible by tp_size");
-    // Fewer KV heads than ranks: each KV head is replicated on tp_size / num_kv_heads ranks.
-    B200_CHECK_ARG(m.num_kv_heads % c.tp_size == 0 || c.tp_size % m.num_kv_heads == 0,
-                   "num_kv_heads must divide, or be divisible by, tp_size");
-    if (m.num_experts > 0 && c.expert_parallel) {
-        B200_CHECK_ARG(m.num_experts % c.tp_size == 0, "num_experts must be divisible by tp_size");
-        B200_CHECK_ARG(m.moe_intermediate_size % 64 == 0, "MoELayer intermediate size must be a multiple of 64");
-    } else if (m.num_experts > 0) {
-        B200_CHECK_ARG(m.moe_intermediate_size % (64 * c.tp_size) == 0,
-                       "MoELayer intermediate size / tp_size must be a multiple of 64");
-    }
-    B200_CHECK_ARG(m.intermediate_size % (64 * c.tp_size) == 0 || m.num_experts > 0,
-                   "intermediate_size / tp_size must be a multiple of 64");
     B200_CHECK_ARG(c.page_size >= 1 && (c.page_size & (c.page_size - 1)) == 0,
                    "engine_create: page_size must be a power of two");
     B200_CHECK_ARG(c.num_pages >= 1 && c.max_running_req >= 1 && c.max_seq_len >= 1 && c.max_extend_tokens >= 1,
                    "engine_create: bad engine sizes");
+    if (stack) {
+        B200_CHECK_ARG(c.tp_size == 1, "engine_create: layer stacks are not sharded (tp_size must be 1)");
+    } else {
+        B200_CHECK_ARG(m.head_dim == 128, "engine_create: head_dim must be 128 (as the reference's attention is)");
+        B200_CHECK_ARG(m.hidden_size % 64 == 0 && m.intermediate_size % 64 == 0,
+                       "engine_create: hidden and intermediate sizes must be multiples of 64");
+        B200_CHECK_ARG(m.num_qo_heads % c.tp_size == 0, "num_qo_heads must be divisible by tp_size");
+        // Fewer KV heads than ranks: each KV head is replicated on tp_size / num_kv_heads ranks.
+        B200_CHECK_ARG(m.num_kv_heads % c.tp_size == 0 || c.tp_size % m.num_kv_heads == 0,
+                       "num_kv_heads must divide, or be divisible by, tp_size");
+        if (m.num_experts > 0 && c.expert_parallel) {
+            B200_CHECK_ARG(m.num_experts % c.tp_size == 0, "num_experts must be divisible by tp_size");
+            B200_CHECK_ARG(m.moe_intermediate_size % 64 == 0, "MoELayer intermediate size must be a multiple of 64");
+        } else if (m.num_experts > 0) {
+            B200_CHECK_ARG(m.moe_intermediate_size % (64 * c.tp_size) == 0,
+                           "MoELayer intermediate size / tp_size must be a multiple of 64");
+    }
+    B200_CHECK_ARG(m.intermediate_size % (64 * c.tp_size) == 0 || m.num_experts > 0,
+                   "intermediate_size / tp_size must be a multiple of 64");
     const int hkv = m.num_kv_heads >= c.tp_size ? m.num_kv_heads / c.tp_size : 1;
     B200_CHECK_ARG(hkv <= 8 && 8 % hkv == 0, "engine_create: kv heads per rank must be 1, 2, 4 or 8");
+    }
 
     b200_engine* e = new b200_engine();
     e->m = m;
     e->c = c;
     B200_CHECK_CUDA(cudaGetDevice(&e->device));
-    e->hq = m.num_qo_heads / c.tp_size;
-    e->hkv = hkv;
-    if (m.num_experts > 0) {
-        const bool ep = c.expert_parallel != 0;
-        e->moe_inter = ep ? m.moe_intermediate_size : m.moe_intermediate_size / c.tp_size;
-        e->experts_local = ep ? m.num_experts / c.tp_size : m.num_experts;
-        e->expert_begin = ep ? c.tp_rank * e->experts_local : 0;
-    }
-    e->inter = m.intermediate_size / c.tp_size;
-    e->qkv_dim = (e->hq + 2 * e->hkv) * m.head_dim;
     e->num_slots = static_cast<int64_t>(c.num_pages + 1) * c.page_size;
+    if (!stack) {
+        e->hq = m.num_qo_heads / c.tp_size;
+        e->hkv = m.num_kv_heads >= c.tp_size ? m.num_kv_heads / c.tp_size : 1;
+        if (m.num_experts > 0) {
+            const bool ep = c.expert_parallel != 0;
+            e->moe_inter = ep ? m.moe_intermediate_size : m.moe_intermediate_size / c.tp_size;
+            e->experts_local = ep ? m.num_experts / c.tp_size : m.num_experts;
+            e->expert_begin = ep ? c.tp_rank * e->experts_local : 0;
+        }
+        e->inter = m.intermediate_size / c.tp_size;
+        e->qkv_dim = (e->hq + 2 * e->hkv) * m.head_dim;
+        e->sm_scale = 1.0f / sqrtf(static_cast<float>(m.head_dim));
+    }
     e->pt_rows = c.max_running_req + 1;
     e->pt_cols = align_ceil(c.max_seq_len, 32);
     e->max_batch = c.max_running_req + 1;
     e->max_tokens = c.max_extend_tokens > e->max_batch ? c.max_extend_tokens : e->max_batch;
-    e->sm_scale = 1.0f / sqrtf(static_cast<float>(m.head_dim));
     int err = B200_OK;
     e->status = device_status_words(&err);
     if (err != B200_OK) { delete e; return err; }
@@ -782,19 +800,7 @@ int b200_engine_create(const b200_model_config* model, const b200_engine_config*
     auto fail = [&](int code) { b200_engine_destroy(e); return code; };
 #define E_TRY(expr) do { int c__ = (expr); if (c__ != B200_OK) return fail(c__); } while (0)
 
-    const int64_t H = m.hidden_size, D = m.head_dim;
-    E_TRY(named_alloc(e, &e->embed, "embed", static_cast<int64_t>(m.vocab_size) * H));
-    if (m.tie_word_embeddings) {
-        e->lm_head = e->embed;
-        e->named["lm_head"] = e->named["embed"];
-    } else {
-        E_TRY(named_alloc(e, &e->lm_head, "lm_head", static_cast<int64_t>(m.vocab_size) * H));
-    }
-    E_TRY(named_alloc(e, &e->final_norm, "final_norm", H));
-    E_TRY(named_alloc(e, &e->rope_cos, "rope_cos", static_cast<int64_t>(m.max_position) * (D / 2)));
-    E_TRY(named_alloc(e, &e->rope_sin, "rope_sin", static_cast<int64_t>(m.max_position) * (D / 2)));
-    E_TRY(build_rope_tables(e));
-    E_TRY(named_alloc(e, &e->kv_cache, "kv_cache", 2 * static_cast<int64_t>(m.num_layers) * e->num_slots * e->hkv * D, true));
+    const int64_t Tm = e->max_tokens;
     E_TRY(named_alloc(e, &e->page_table, "page_table", static_cast<int64_t>(e->pt_rows) * e->pt_cols, true));
     E_TRY(named_alloc(e, &e->token_pool, "token_pool", static_cast<int64_t>(e->pt_rows) * e->pt_cols, true));
     {
@@ -806,73 +812,23 @@ int b200_engine_create(const b200_model_config* model, const b200_engine_config*
             return fail(B200_ERR_CUDA);
         }
     }
-    e->layers.resize(m.num_layers);
-    for (int l = 0; l < m.num_layers; ++l) {
-        LayerWeights& L = e->layers[l];
-        const std::string sfx = "." + std::to_string(l);
-        E_TRY(named_alloc(e, &L.qkv, "qkv" + sfx, static_cast<int64_t>(e->qkv_dim) * H));
-        if (m.attention_bias) E_TRY(named_alloc(e, &L.qkv_bias, "qkv_bias" + sfx, e->qkv_dim));
-        E_TRY(named_alloc(e, &L.o, "o" + sfx, H * e->hq * D));
-        E_TRY(named_alloc(e, &L.input_norm, "input_norm" + sfx, H));
-        E_TRY(named_alloc(e, &L.post_norm, "post_norm" + sfx, H));
-        if (m.qk_norm) {
-            E_TRY(named_alloc(e, &L.q_norm, "q_norm" + sfx, D));
-            E_TRY(named_alloc(e, &L.k_norm, "k_norm" + sfx, D));
-        }
-        if (m.num_experts > 0) {
-            const int64_t ie = e->moe_inter, el = e->experts_local;
-            E_TRY(named_alloc(e, &L.router, "router" + sfx, static_cast<int64_t>(m.num_experts) * H));
-            E_TRY(named_alloc(e, &L.experts_gate_up, "experts_gate_up" + sfx, el * 2 * ie * H));
-            E_TRY(named_alloc(e, &L.experts_down, "experts_down" + sfx, el * H * ie));
-        } else {
-            E_TRY(named_alloc(e, &L.gate_up, "gate_up" + sfx, 2 * static_cast<int64_t>(e->inter) * H));
-            E_TRY(named_alloc(e, &L.down, "down" + sfx, H * e->inter));
-        }
-        const __nv_bfloat16* kc = e->kv_cache + static_cast<int64_t>(l) * e->num_slots * e->hkv * D;
-        const __nv_bfloat16* vc = kc + static_cast<int64_t>(m.num_layers) * e->num_slots * e->hkv * D;
-        E_TRY(make_kv_tmap(&L.tmap_k, kc, e->num_slots, e->hkv, c.page_size));
-        E_TRY(make_kv_tmap(&L.tmap_v, vc, e->num_slots, e->hkv, c.page_size));
-    }
-    const int64_t Tm = e->max_tokens;
-    const int64_t inter_buf = m.num_experts > 0 ? m.moe_intermediate_size : e->inter;
-    E_TRY(named_alloc(e, &e->x, "x", Tm * H));
-    E_TRY(named_alloc(e, &e->residual, "residual", Tm * H));
-    E_TRY(named_alloc(e, &e->qkv, "qkv_act", Tm * e->qkv_dim));
-    E_TRY(named_alloc(e, &e->attn_out, "attn_out", Tm * e->hq * D));
-    E_TRY(named_alloc(e, &e->h, "mlp_act", Tm * inter_buf));
-    E_TRY(named_alloc(e, &e->sel, "sel", static_cast<int64_t>(e->max_batch) * H));
-    E_TRY(named_alloc(e, &e->logits, "logits", static_cast<int64_t>(e->max_batch) * m.vocab_size));
     E_TRY(named_alloc(e, &e->positions, "positions", Tm));
     E_TRY(named_alloc(e, &e->out_loc, "out_loc", Tm));
     E_TRY(named_alloc(e, &e->input_ids, "input_ids", Tm));
     E_TRY(named_alloc(e, &e->seq_lens, "seq_lens", e->max_batch));
     E_TRY(named_alloc(e, &e->next_tokens, "next_tokens", e->max_batch, true));
-    e->comm_buffer_bytes = Tm * H * 2;
-    if (c.tp_size > 1) E_TRY(b200_comm_create(c.tp_rank, c.tp_size, e->comm_buffer_bytes, &e->comm));
-    if (m.num_experts > 0) {
-        E_TRY(named_alloc(e, &e->router_logits, "router_logits", Tm * m.num_experts));
-        E_TRY(dev_alloc(e, &e->moe_ws,
-                        moe_workspace_bytes(static_cast<int>(Tm), m.num_experts, m.num_experts_per_tok, m.hidden_size,
-                                            e->moe_inter),
-                        false));
-    }
-    if (const char* v = getenv("B200_FOLD_NORM")) e->use_fold = atoi(v) != 0;
-    if (const char* v = getenv("B200_FOLD_HEADS")) e->use_fold_heads = atoi(v) != 0;
-    if (e->use_fold && c.tp_size == 1 && m.num_experts == 0 && fold_shapes_ok(e)) {
-        for (LayerWeights& L : e->layers) {
-            void* p = nullptr;
-            E_TRY(dev_alloc(e, &p, static_cast<int64_t>(e->qkv_dim) * H * 2, false));
-            L.qkv_folded = static_cast<__nv_bfloat16*>(p);
-            E_TRY(dev_alloc(e, &p, 2 * static_cast<int64_t>(e->inter) * H * 2, false));
-            L.gate_up_folded = static_cast<__nv_bfloat16*>(p);
-        }
+    E_TRY(stack ? layer_stack_create(e, stack) : alloc_gqa_model(e));
+    if (stack) {
+        const int64_t z = stack_dtype(e) == B200_DTYPE_F32 ? 4 : 2;
         void* p = nullptr;
-        E_TRY(dev_alloc(e, &p, static_cast<int64_t>(2 * m.num_layers + 1) * b200_engine::kSsqStride * 8, true));
-        e->ssq = static_cast<unsigned long long*>(p);
+        E_TRY(dev_alloc(e, &p, static_cast<int64_t>(e->max_batch) * stack_row_bytes(e), true));
+        e->sel = static_cast<__nv_bfloat16*>(p);
+        E_TRY(dev_alloc(e, &p, static_cast<int64_t>(e->max_batch) * stack_logits_ld(e) * z, true));
+        e->logits = static_cast<__nv_bfloat16*>(p);
+        e->named["logits"] = Tensor{p, static_cast<int64_t>(e->max_batch) * stack_logits_ld(e) * z};
+        if (z == 4) E_TRY(dev_alloc(e, &e->logits_bf16, static_cast<int64_t>(e->max_batch) * stack_logits_ld(e) * 2, true));
     }
-    E_TRY(dev_alloc(e, &e->chain_scratch, decode_chain_scratch_bytes(m.hidden_size), true));
-    e->attn_ws_bytes = decode_workspace_bytes(e->max_batch, e->hq, e->hkv);
-    E_TRY(dev_alloc(e, &e->attn_ws, e->attn_ws_bytes, true));
+    E_TRY(dev_alloc(e, reinterpret_cast<void**>(&e->row_ids_dev), e->max_batch * 4, true));
 
     e->meta_ints = 9 * e->max_batch + 16;
     if (cudaMallocHost(&e->meta_host, e->meta_ints * sizeof(int32_t)) != cudaSuccess) {
@@ -918,6 +874,16 @@ int b200_engine_create(const b200_model_config* model, const b200_engine_config*
     return B200_OK;
 }
 
+int b200_engine_create(const b200_model_config* model, const b200_engine_config* config, b200_engine** out) {
+    return create_engine(model, nullptr, config, out);
+}
+
+int b200_engine_create_stack(const b200_model_config* model, const b200_stack_config* stack,
+                             const b200_engine_config* config, b200_engine** out) {
+    B200_CHECK_ARG(stack, "engine_create_stack: NULL argument");
+    return create_engine(model, stack, config, out);
+}
+
 int b200_engine_destroy(b200_engine* e) {
     if (!e) return B200_OK;
     if (e->stream) cudaStreamSynchronize(e->stream);
@@ -926,6 +892,7 @@ int b200_engine_destroy(b200_engine* e) {
     for (cudaEvent_t ev : e->prof_events) cudaEventDestroy(ev);
     for (cudaEvent_t ev : e->prof_events_ar) cudaEventDestroy(ev);
     if (e->comm) b200_comm_destroy(e->comm);
+    layer_stack_destroy(e);
     for (void* p : e->allocs) cudaFree(p);
     if (e->meta_host) cudaFreeHost(e->meta_host);
     if (e->scatter_host) cudaFreeHost(e->scatter_host);
@@ -1037,6 +1004,7 @@ int b200_engine_capture_graphs(b200_engine* e, const int32_t* batch_sizes, int c
             st.temperatures = variant ? &one : nullptr;   // non-NULL only switches the staging of sampling fields on
             int T = 0, max_ext = 0;
             B200_TRY(stage_step(e, &st, Bp, &T, &max_ext));
+            if (e->stack) B200_TRY(layer_stack_plan(e, &st, st.phase, Bp, T));
             const size_t bytes = (variant ? b200_engine::step_index_offset(Bp) + 2 : 4 * Bp + 1) * sizeof(int32_t);
             B200_CHECK_CUDA(cudaMemcpyAsync(e->meta_dev, e->meta_host, bytes, cudaMemcpyHostToDevice, e->stream));
             B200_TRY(ensure_folded(e));
@@ -1093,10 +1061,12 @@ static int run_step(b200_engine* e, const b200_step* st, int32_t* next_tokens_ho
 
     cudaStream_t s = e->stream;
     B200_TRY(ensure_folded(e));
+    e->tokens_last_step = T;
     B200_CHECK_CUDA(cudaEventRecord(e->ev_step_begin, s));
     const size_t meta_bytes =
         (sampling ? b200_engine::step_index_offset(Bg) + 2 : 4 * Bg + 1) * sizeof(int32_t);
     B200_CHECK_CUDA(cudaMemcpyAsync(e->meta_dev, e->meta_host, meta_bytes, cudaMemcpyHostToDevice, s));
+    if (e->stack) B200_TRY(layer_stack_plan(e, st, st->phase, Bg, T));
     B200_CHECK_CUDA(cudaEventRecord(e->ev_meta_done, s));
     e->meta_in_flight = true;
     // A captured graph covers all Bg rows; padded rows carry write_pos = -1 so nothing of
@@ -1203,8 +1173,49 @@ int b200_engine_read_logits(b200_engine* e, void* host, int rows) {
     B200_CHECK_ARG(e && host, "engine_read_logits: NULL argument");
     B200_CHECK_ARG(rows >= 0 && rows <= e->max_batch, "engine_read_logits: rows out of range");
     B200_CHECK_CUDA(cudaStreamSynchronize(e->stream));
-    B200_CHECK_CUDA(cudaMemcpy(host, e->logits, static_cast<size_t>(rows) * e->m.vocab_size * 2,
-                               cudaMemcpyDeviceToHost));
+    const size_t z = logits_f32(e) ? 4 : 2;
+    B200_CHECK_CUDA(cudaMemcpy2D(host, e->m.vocab_size * z, e->logits, logits_ld(e) * z, e->m.vocab_size * z, rows,
+                                 cudaMemcpyDeviceToHost));
+    return B200_OK;
+}
+
+int b200_engine_token_logits(b200_engine* e, const int32_t* tokens, int count, float* host) {
+    B200_CHECK_ARG(e && count >= 0 && (count == 0 || (tokens && host)), "engine_token_logits: NULL argument");
+    for (int i = 0; i < count; ++i)
+        B200_CHECK_ARG(tokens[i] >= 0 && tokens[i] < e->tokens_last_step,
+                       "engine_token_logits: token %d is not one of the last step's %d", tokens[i], e->tokens_last_step);
+    const int row_bytes = hidden_row_bytes(e), vocab = e->m.vocab_size, ld = logits_ld(e);
+    const size_t z = logits_f32(e) ? 4 : 2;
+    std::vector<uint16_t> narrow;
+    for (int i0 = 0; i0 < count; i0 += e->max_batch) {
+        const int n = count - i0 < e->max_batch ? count - i0 : e->max_batch;
+        B200_CHECK_CUDA(cudaStreamSynchronize(e->stream));
+        B200_CHECK_CUDA(cudaMemcpy(e->row_ids_dev, tokens + i0, n * sizeof(int32_t), cudaMemcpyHostToDevice));
+        take_rows_kernel<<<n, 128, 0, e->stream>>>(reinterpret_cast<uint4*>(e->sel), static_cast<const uint4*>(hidden_states(e)),
+                                                   e->row_ids_dev, row_bytes / 16);
+        B200_CHECK_LAUNCH();
+        B200_TRY(output_head(e, e->sel, n));
+        B200_CHECK_CUDA(cudaStreamSynchronize(e->stream));
+        float* dst = host + static_cast<int64_t>(i0) * vocab;
+        if (z == 4) {
+            B200_CHECK_CUDA(cudaMemcpy2D(dst, vocab * z, e->logits, ld * z, vocab * z, n, cudaMemcpyDeviceToHost));
+            continue;
+        }
+        narrow.resize(static_cast<size_t>(n) * vocab);
+        B200_CHECK_CUDA(cudaMemcpy2D(narrow.data(), vocab * z, e->logits, ld * z, vocab * z, n, cudaMemcpyDeviceToHost));
+        for (size_t j = 0; j < narrow.size(); ++j) {
+            const uint32_t bits = static_cast<uint32_t>(narrow[j]) << 16;
+            memcpy(dst + j, &bits, 4);
+        }
+    }
+    return B200_OK;
+}
+
+int b200_engine_trace_residual(b200_engine* e, float* host) {
+    B200_CHECK_ARG(e && e->stack, "engine_trace_residual: only layer stacks keep an fp32 residual stream");
+    B200_CHECK_CUDA(cudaStreamSynchronize(e->stream));
+    stack_set_trace(e, host);
+    e->trace_residual = host != nullptr;
     return B200_OK;
 }
 

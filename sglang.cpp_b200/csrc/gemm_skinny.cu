@@ -104,6 +104,10 @@ struct SkinnyParams {
     const int32_t* group_counts;
     const int32_t* group_offsets;
     int w_rows_per_group;
+    // Per-head mode: blockIdx.z = head; it reads columns [z * head_k, ...) of x and writes columns
+    // [z * n_out, ...) of y with the weights of its own w_rows_per_group rows.
+    int head_k;          // 0 = off
+    int64_t y_pitch;     // row pitch of y (n_out, or heads * n_out)
     // Fusions with the residual stream (split-K launches of the decode step; see SkinnyFusion in kernels.h).
     const unsigned long long* ssq_in;   // "normalised input": accumulator x rsqrt(ssq_in[m] / 2^24 / norm_width + eps)
     float norm_eps;
@@ -137,7 +141,7 @@ skinny_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w,
                    const __grid_constant__ CUtensorMap tmap_x64,
                    const __grid_constant__ CUtensorMap tmap_x128,
                    const __grid_constant__ CUtensorMap tmap_x256, const SkinnyParams p) {
-    constexpr int NUM_A = EPI == B200_EPILOGUE_NONE ? 1 : 2;
+    constexpr int NUM_A = epilogue_is_gated(EPI) ? 2 : 1;
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t full_bar[kMaxStages];
     __shared__ __align__(8) uint64_t empty_bar[kMaxStages];
@@ -154,6 +158,13 @@ skinny_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w,
     int rows = p.M;         // valid rows of x / y handled by this CTA
     int x_row0 = 0;         // first row of x and of y
     int w_row0 = 0;         // first row of this group's weights
+    int x_col0 = 0;         // per-head mode: first column of x / of y
+    int y_col0 = 0;
+    if (p.head_k > 0) {
+        w_row0 = static_cast<int>(blockIdx.z) * p.w_rows_per_group;
+        x_col0 = static_cast<int>(blockIdx.z) * p.head_k;
+        y_col0 = static_cast<int>(blockIdx.z) * p.n_out;
+    }
     const CUtensorMap* tx = &tmap_x;
     if (p.group_counts != nullptr) {
         pdl_wait_prior();   // the group table comes from the kernel before this one
@@ -252,7 +263,7 @@ skinny_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w,
                     load_w(dst, kc, w_row0 + n0, bar);
                     if (NUM_A == 2) load_w(dst + a_bytes, kc, w_row0 + p.up_row_offset + n0, bar);
                 }
-                tma_load_2d(dst + NUM_A * a_bytes, tx, kc, x_row0, bar);
+                tma_load_2d(dst + NUM_A * a_bytes, tx, x_col0 + kc, x_row0, bar);
             }
         }
     } else if (warp == 1) {
@@ -390,8 +401,9 @@ skinny_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w,
                                     v = gated_act<EPI>(gv) * uv;
                                 } else {
                                     v = __uint_as_float(g[j]) + bias;
+                                    if (EPI == B200_EPILOGUE_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
                                 }
-                                p.y[static_cast<int64_t>(x_row0 + m) * p.n_out + n] = __float2bfloat16_rn(v);
+                                p.y[static_cast<int64_t>(x_row0 + m) * p.y_pitch + y_col0 + n] = __float2bfloat16_rn(v);
                             }
                         }
                     }
@@ -585,9 +597,10 @@ skinny_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w,
                         } else if (p.bias) {
                             v[e] += __bfloat162float(p.bias[n + e]);
                         }
+                        if (EPI == B200_EPILOGUE_RELU2) v[e] = fmaxf(v[e], 0.f) * fmaxf(v[e], 0.f);
                     }
                     uint2 packed = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
-                    *reinterpret_cast<uint2*>(p.y + static_cast<int64_t>(x_row0 + m) * p.n_out + n) = packed;
+                    *reinterpret_cast<uint2*>(p.y + static_cast<int64_t>(x_row0 + m) * p.y_pitch + y_col0 + n) = packed;
                 }
             }
         }
@@ -605,6 +618,7 @@ SkinnyKernel skinny_kernel_for(int epilogue, bool heads = false) {
         case B200_EPILOGUE_SWIGLU: return skinny_gemm_kernel<B200_EPILOGUE_SWIGLU>;
         case B200_EPILOGUE_GEGLU: return skinny_gemm_kernel<B200_EPILOGUE_GEGLU>;
         case B200_EPILOGUE_GEGLU_ERF: return skinny_gemm_kernel<B200_EPILOGUE_GEGLU_ERF>;
+        case B200_EPILOGUE_RELU2: return skinny_gemm_kernel<B200_EPILOGUE_RELU2>;
         default: return skinny_gemm_kernel<B200_EPILOGUE_NONE>;
     }
 }
@@ -673,7 +687,7 @@ static int env_int(const char* name, int dflt) {
 // K split of a slab: up to one CTA per SM in total, at most 8 ranks (portable cluster size).
 int skinny_gemm_split(int M, int N, int K, int epilogue) {
     (void)M;
-    const int n_out = epilogue != B200_EPILOGUE_NONE ? N / 2 : N;
+    const int n_out = epilogue_is_gated(epilogue) ? N / 2 : N;
     const int kb_total = K / kBlockK;
     const int n_tiles = div_ceil(n_out, kTileN);
     const int forced = env_int("B200_GEMM_SPLIT", 0);
@@ -690,7 +704,7 @@ int skinny_gemm_split(int M, int N, int K, int epilogue) {
 int launch_skinny_gemm(void* y, const void* x, const void* w, const void* bias, int M, int N,
                        int K, int64_t ldx, int epilogue, int* status, cudaStream_t stream,
                        const SkinnyFusion* fuse = nullptr) {
-    const bool gated = epilogue != B200_EPILOGUE_NONE;
+    const bool gated = epilogue_is_gated(epilogue);
     const int n_out = gated ? N / 2 : N;
     // accumulator columns: 32, or a multiple of the 64-column exchange round (the epilogue walks whole rounds)
     const int nt = M <= 32 ? 32 : div_ceil(M, kRoundCols) * kRoundCols;
@@ -757,6 +771,8 @@ int launch_skinny_gemm(void* y, const void* x, const void* w, const void* bias, 
     p.group_counts = nullptr;
     p.group_offsets = nullptr;
     p.w_rows_per_group = 0;
+    p.head_k = 0;
+    p.y_pitch = n_out;
     set_fusion(&p, fuse);
 
     auto kernel = skinny_kernel_for(epilogue, p.head_mode != 0);
@@ -774,7 +790,7 @@ int launch_grouped_gemm(void* y, const void* x, const void* w, const int32_t* co
                         const int32_t* offsets, int num_groups, int max_rows_per_group,
                         int64_t total_rows, int N, int K, int epilogue, int* status,
                         cudaStream_t stream) {
-    const bool gated = epilogue != B200_EPILOGUE_NONE;
+    const bool gated = epilogue_is_gated(epilogue);
     const int n_out = gated ? N / 2 : N;
     const int num_a = gated ? 2 : 1;
     const int kb_total = K / kBlockK;
@@ -822,12 +838,60 @@ int launch_grouped_gemm(void* y, const void* x, const void* w, const int32_t* co
     p.group_counts = counts;
     p.group_offsets = offsets;
     p.w_rows_per_group = N;
+    p.head_k = 0;
+    p.y_pitch = n_out;
     set_fusion(&p, nullptr);
     auto kernel = skinny_kernel_for(epilogue);
     B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(smem_bytes)));
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(n_tiles, slabs, num_groups), dim3(kThreads), smem_bytes, stream,
                                   dim3(1, 1, 1), tmap_w, tx[0], tx[1], tx[2], tx[3], p));
+    return B200_OK;
+}
+
+// y[m, h*N + n] = sum_k x[m, h*K + k] w[h*N + n, k]: one projection per head, slabs of 256 rows.
+int launch_linear_heads(void* y, const void* x, const void* w, int M, int heads, int N, int K, int* status,
+                        cudaStream_t stream) {
+    const int kb_total = K / kBlockK;
+    const int n_tiles = div_ceil(N, kTileN);
+    for (int m0 = 0; m0 < M; m0 += 256) {
+        const int rows = M - m0 < 256 ? M - m0 : 256;
+        const int nt = rows <= 32 ? 32 : div_ceil(rows, kRoundCols) * kRoundCols;
+        const uint32_t stage_bytes = kTileN * kBlockK * 2 + nt * kBlockK * 2;
+        int stages = kb_total < kMaxStages ? kb_total : kMaxStages;
+        while (stages > 2 && stages * stage_bytes > 100 * 1024) --stages;   // two CTAs per SM
+        const uint32_t smem_bytes = stages * stage_bytes + 1024;
+        const __nv_bfloat16* xs = static_cast<const __nv_bfloat16*>(x) + static_cast<int64_t>(m0) * heads * K;
+        CUtensorMap tmap_w, tmap_x;
+        int err = cached_tmap(&tmap_w, w, static_cast<uint64_t>(K), static_cast<uint64_t>(heads) * N,
+                              static_cast<uint64_t>(K) * 2, kBlockK, kTileN);
+        if (err != B200_OK) return err;
+        err = cached_tmap(&tmap_x, xs, static_cast<uint64_t>(heads) * K, static_cast<uint64_t>(rows),
+                          static_cast<uint64_t>(heads) * K * 2, kBlockK, static_cast<uint32_t>(nt));
+        if (err != B200_OK) return err;
+        SkinnyParams p;
+        p.y = static_cast<__nv_bfloat16*>(y) + static_cast<int64_t>(m0) * heads * N;
+        p.bias = nullptr;
+        p.M = rows;
+        p.n_out = N;
+        p.up_row_offset = 0;
+        p.kb_total = kb_total;
+        p.nt = nt;
+        p.stages = stages;
+        p.epilogue = B200_EPILOGUE_NONE;
+        p.status = status;
+        p.group_counts = nullptr;
+        p.group_offsets = nullptr;
+        p.w_rows_per_group = N;
+        p.head_k = K;
+        p.y_pitch = static_cast<int64_t>(heads) * N;
+        set_fusion(&p, nullptr);
+        auto kernel = skinny_kernel_for(B200_EPILOGUE_NONE);
+        B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                             static_cast<int>(smem_bytes)));
+        B200_CHECK_CUDA(launch_kernel(kernel, dim3(n_tiles, 1, heads), dim3(kThreads), smem_bytes, stream,
+                                      dim3(1, 1, 1), tmap_w, tmap_x, tmap_x, tmap_x, tmap_x, p));
+    }
     return B200_OK;
 }
 
@@ -841,7 +905,7 @@ int launch_linear(void* y, const void* x, const void* w, const void* bias, int M
         }
         return launch_tile_gemm(y, x, w, bias, M, N, K, ldx, epilogue, status, stream);
     }
-    const int n_out = epilogue != B200_EPILOGUE_NONE ? N / 2 : N;
+    const int n_out = epilogue_is_gated(epilogue) ? N / 2 : N;
     const __nv_bfloat16* xp = static_cast<const __nv_bfloat16*>(x);
     __nv_bfloat16* yp = static_cast<__nv_bfloat16*>(y);
     for (int m0 = 0; m0 < M; m0 += 256) {
@@ -858,15 +922,27 @@ int launch_linear(void* y, const void* x, const void* w, const void* bias, int M
 
 extern "C" {
 
+int b200_linear_heads(void* y, const void* x, const void* w, int M, int heads, int N, int K, b200_stream_t stream) {
+    B200_CHECK_ARG(M >= 0 && heads > 0 && N > 0 && K > 0, "linear_heads: bad shape");
+    B200_CHECK_ARG(M == 0 || (y && x && w), "linear_heads: NULL tensor");
+    B200_CHECK_ARG(K % 64 == 0 && N % 8 == 0, "linear_heads: K must be a multiple of 64, N of 8");
+    B200_CHECK_ARG(heads <= 65535, "linear_heads: too many heads");
+    if (M == 0) return B200_OK;
+    int err = B200_OK;
+    int* status = b200::device_status_words(&err);
+    if (err != B200_OK) return err;
+    return b200::launch_linear_heads(y, x, w, M, heads, N, K, status, static_cast<cudaStream_t>(stream));
+}
+
 int b200_linear(void* y, const void* x, const void* w, const void* bias, int M, int N, int K,
                 int64_t ldx, int epilogue, b200_stream_t stream) {
     B200_CHECK_ARG(M >= 0 && N > 0 && K > 0, "linear: bad shape");
     B200_CHECK_ARG(M == 0 || (y && x && w), "linear: NULL tensor");
     B200_CHECK_ARG(K % 64 == 0, "linear: K must be a multiple of 64");
     B200_CHECK_ARG(ldx >= K && ldx % 8 == 0, "linear: ldx must be >= K and a multiple of 8");
-    B200_CHECK_ARG(epilogue >= B200_EPILOGUE_NONE && epilogue <= B200_EPILOGUE_GEGLU_ERF,
+    B200_CHECK_ARG(epilogue >= B200_EPILOGUE_NONE && epilogue <= B200_EPILOGUE_RELU2,
                    "linear: unknown epilogue");
-    const bool gated = epilogue != B200_EPILOGUE_NONE;
+    const bool gated = b200::epilogue_is_gated(epilogue);
     B200_CHECK_ARG(!gated || (N % 2 == 0), "linear: a gated epilogue needs an even N");
     B200_CHECK_ARG(!gated || bias == nullptr, "linear: bias is not supported with a gated epilogue");
     B200_CHECK_ARG((gated ? N / 2 : N) % 8 == 0, "linear: output width must be a multiple of 8");

@@ -77,7 +77,7 @@ template <int EPI>
 __global__ void __launch_bounds__(kThreads, 1)
 tile_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
                  const TileParams p) {
-    constexpr bool GATED = EPI != B200_EPILOGUE_NONE;
+    constexpr bool GATED = epilogue_is_gated(EPI);
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t full_bar[kStages];
     __shared__ __align__(8) uint64_t empty_bar[kStages];
@@ -270,6 +270,10 @@ tile_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
                         for (int j = 0; j < 32; ++j)
                             if (n + j < p.n_out) v[j] += __bfloat162float(p.bias[n + j]);
                     }
+                    if (EPI == B200_EPILOGUE_RELU2) {
+#pragma unroll
+                        for (int j = 0; j < 32; ++j) v[j] = fmaxf(v[j], 0.f) * fmaxf(v[j], 0.f);
+                    }
 #pragma unroll
                     for (int j = 0; j < 32; j += 8) {
                         if (n + j < p.n_out) {  // n_out is a multiple of 8: whole 16-byte groups
@@ -298,7 +302,7 @@ tile_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
 
 int launch_tile_gemm(void* y, const void* x, const void* w, const void* bias, int M, int N, int K,
                      int64_t ldx, int epilogue, int* status, cudaStream_t stream) {
-    const bool gated = epilogue != B200_EPILOGUE_NONE;
+    const bool gated = epilogue_is_gated(epilogue);
     const int n_out = gated ? N / 2 : N;
     TileParams p;
     p.y = static_cast<__nv_bfloat16*>(y);
@@ -331,6 +335,7 @@ int launch_tile_gemm(void* y, const void* x, const void* w, const void* bias, in
     if (epilogue == B200_EPILOGUE_SWIGLU) kernel = tile_gemm_kernel<B200_EPILOGUE_SWIGLU>;
     if (epilogue == B200_EPILOGUE_GEGLU) kernel = tile_gemm_kernel<B200_EPILOGUE_GEGLU>;
     if (epilogue == B200_EPILOGUE_GEGLU_ERF) kernel = tile_gemm_kernel<B200_EPILOGUE_GEGLU_ERF>;
+    if (epilogue == B200_EPILOGUE_RELU2) kernel = tile_gemm_kernel<B200_EPILOGUE_RELU2>;
     B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(smem_bytes)));
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(grid), dim3(kThreads), smem_bytes, stream, dim3(1, 1, 1),
@@ -347,7 +352,7 @@ int launch_grouped_tile_gemm(void* y, const void* x, const void* w, const int32_
         set_last_error("grouped GEMM: %d groups exceed %d", num_groups, kMaxGroups);
         return B200_ERR_UNSUPPORTED;
     }
-    const bool gated = epilogue != B200_EPILOGUE_NONE;
+    const bool gated = epilogue_is_gated(epilogue);
     const int n_out = gated ? N / 2 : N;
     TileParams p;
     p.y = static_cast<__nv_bfloat16*>(y);
@@ -376,6 +381,7 @@ int launch_grouped_tile_gemm(void* y, const void* x, const void* w, const int32_
     if (epilogue == B200_EPILOGUE_SWIGLU) kernel = tile_gemm_kernel<B200_EPILOGUE_SWIGLU>;
     if (epilogue == B200_EPILOGUE_GEGLU) kernel = tile_gemm_kernel<B200_EPILOGUE_GEGLU>;
     if (epilogue == B200_EPILOGUE_GEGLU_ERF) kernel = tile_gemm_kernel<B200_EPILOGUE_GEGLU_ERF>;
+    if (epilogue == B200_EPILOGUE_RELU2) kernel = tile_gemm_kernel<B200_EPILOGUE_RELU2>;
     B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(smem_bytes)));
     // the number of tiles is only known on the device: one persistent CTA per SM

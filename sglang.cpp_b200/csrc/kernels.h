@@ -6,7 +6,14 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include "../../include/b200_token_loop.h"
+
 namespace b200 {
+
+// Gated epilogues take two stacked halves of W (gate, up); the others one.
+constexpr bool epilogue_is_gated(int epilogue) {
+    return epilogue != B200_EPILOGUE_NONE && epilogue != B200_EPILOGUE_RELU2;
+}
 
 int launch_rmsnorm(void* out, const void* x, const void* weight, int rows, int hidden, float eps,
                    cudaStream_t stream);
@@ -44,6 +51,8 @@ int launch_sample(int32_t* out, const void* logits, int rows, int vocab, int64_t
                   const float* temperatures, const int32_t* top_k, const float* top_p,
                   const uint64_t* seeds, uint64_t step_index, uint8_t* mask, cudaStream_t stream,
                   const uint64_t* step_index_dev = nullptr, const TokenWriteBack* write_back = nullptr);
+int launch_argmax_f32(int32_t* out, const float* logits, int rows, int vocab, int64_t ld, cudaStream_t stream,
+                      const TokenWriteBack* write_back = nullptr);
 int launch_argmax(int32_t* out, const void* logits, int rows, int vocab, int64_t ld,
                   cudaStream_t stream, const TokenWriteBack* write_back = nullptr);
 
@@ -104,6 +113,75 @@ int launch_grouped_gemm(void* y, const void* x, const void* w, const int32_t* co
                         const int32_t* offsets, int num_groups, int max_rows_per_group,
                         int64_t total_rows, int N, int K, int epilogue, int* status,
                         cudaStream_t stream);
+
+int launch_linear_heads(void* y, const void* x, const void* w, int M, int heads, int N, int K, int* status,
+                        cudaStream_t stream);
+// fp32 GEMMs of every form the layer stack uses (linear_f32.cu); see b200_linear_f32.
+int launch_linear_f32(float* y, const float* x, const float* w, int max_rows, int N, int K, int groups,
+                      const int32_t* counts, const int32_t* offsets, int epilogue, cudaStream_t stream);
+
+// fp32 residual stream: add, norm, and the gather / scatter around them (residual.cu).
+struct ResidualNorm {
+    void* out = nullptr;
+    const int32_t* out_rows = nullptr;
+    int out_top = 1;
+    float* residual = nullptr;
+    const void* src = nullptr;
+    const int32_t* src_rows = nullptr;
+    int src_top = 1;
+    int64_t src_count = 0;
+    float src_scale = 1.f;
+    bool init = false;
+    const void* weight = nullptr;
+    float weight_offset = 0.f, out_scale = 1.f;
+    int tokens = 0, width = 0, padded = 0;
+    float eps = 0.f;
+};
+int launch_residual_norm(const ResidualNorm& a, int dtype, int* status, cudaStream_t stream);
+
+// Expert placement of every table-routed layer of a step in one launch (moe.cu): one CTA per layer.
+struct TableRouteLayer {
+    const int32_t* table;     // [vocab, top]
+    int32_t *rows, *counts, *offsets;
+    int top, experts;
+};
+constexpr int kMaxTableExperts = 4096;
+int launch_table_route(const TableRouteLayer* layers_dev, int num_layers, int max_experts, const int32_t* token_ids,
+                       int tokens, int vocab, int* status, cudaStream_t stream);
+
+// Latent attention (latent_attention.cu, latent_attention_tc.cu).
+// The output of the joint down-projection [tokens, qp + rp] -> RMS-normalised query latent [tokens, qp]
+// and RMS-normalised key/value latent straight into the pool.
+int launch_latent_norm_store(void* q_latent, void* cache, const void* joint, const void* q_weight,
+                             const void* kv_weight, const int32_t* out_loc, int tokens, int q_rank, int qp,
+                             int kv_rank, int rp, int64_t num_slots, float eps, int dtype, int* status,
+                             cudaStream_t stream);
+struct LatentAttention {
+    void* out = nullptr;              // [rows, heads, width]
+    const void* q = nullptr;          // [rows, heads, width]
+    const void* cache = nullptr;      // [num_slots, width]
+    int64_t num_slots = 0;
+    const int32_t* page_table = nullptr;
+    int64_t pt_stride = 0;
+    const int32_t* row_table = nullptr;   // page-table row of every query row
+    const int32_t* row_len = nullptr;     // keys it sees
+    int rows = 0, heads = 0, width = 0, page_size = 1;
+    float scale = 1.f;
+    void* workspace = nullptr;
+    int64_t workspace_bytes = 0;
+};
+int64_t latent_attention_workspace_bytes(int rows, int heads, int width);
+bool latent_attention_tc_supported(const LatentAttention& a);
+int launch_latent_attention_tc(const LatentAttention& a, int* status, cudaStream_t stream);
+int launch_latent_attention_plain(const LatentAttention& a, int dtype, int* status, cudaStream_t stream);
+// Rows of a paged latent pool gathered into consecutive rows: request b's positions [0, seq_lens[b]) to
+// rows base[b] + position (base[b] < 0: skipped).
+int launch_gather_latents(void* out, const void* cache, int64_t num_slots, const int32_t* page_table,
+                          int64_t pt_stride, const int32_t* table_idx, const int32_t* seq_lens,
+                          const int32_t* base, int batch, int max_len, int rp, int* status, cudaStream_t stream);
+// out[i] = in[rows[i]] (gather) or out[rows[i]] = in[i] (scatter) for rows of vec_per_row 16-byte vectors.
+int launch_move_rows(void* out, const void* in, const int32_t* rows, int count, int vec_per_row, bool scatter,
+                     cudaStream_t stream);
 
 int64_t moe_workspace_bytes(int tokens, int E, int top_k, int H, int I);
 int launch_moe_forward(void* out, const void* hidden, const void* router_logits, const void* gate_up,

@@ -1,0 +1,285 @@
+// Attention over a shared low-rank latent: the paged latent pool, the plain attention kernel, and the
+// gathers that feed the expanded form.
+//
+// One row of `width` numbers per token is key and value of every head at once.  With the per-head
+// up-projections moved to the other side of the products (k_h = U_h c  =>  q_h . k_h = (U_h^T q_h) . c,
+// and sum_j p_j (V_h c_j) = V_h sum_j p_j c_j) attention runs in the latent space and reads one latent per
+// token whatever the number of heads: that is the form decode steps and short extensions take.  Long
+// extensions expand keys and values once per step instead (layer_stack.cu), which costs fewer
+// multiplications per query.
+#include <math.h>
+
+#include "common.cuh"
+#include "kernels.h"
+
+namespace b200 {
+namespace {
+
+template <typename T>
+__device__ __forceinline__ float as_float(T v);
+template <>
+__device__ __forceinline__ float as_float<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ float as_float<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+// Columns [0, qp) of a token's joint row are its query latent, [qp, qp + rp) its key/value latent; each is
+// divided by its own root mean square (over the true widths) and scaled by its own weight.
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_norm_store_kernel(T* __restrict__ q_latent, T* __restrict__ cache, const T* __restrict__ joint,
+                         const T* __restrict__ q_weight, const T* __restrict__ kv_weight,
+                         const int32_t* __restrict__ out_loc, int q_rank, int qp, int kv_rank, int rp,
+                         int64_t num_slots, float eps, int* status) {
+    __shared__ float red[2][8];
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int64_t t = blockIdx.x;
+    const T* row = joint + t * (qp + rp);
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x; i < qp; i += blockDim.x) {
+        const float v = as_float(row[i]);
+        sq += v * v;
+    }
+    for (int i = threadIdx.x; i < rp; i += blockDim.x) {
+        const float v = as_float(row[qp + i]);
+        sk += v * v;
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (lane == 0) {
+        red[0][warp] = sq;
+        red[1][warp] = sk;
+    }
+    __syncthreads();
+    const int nw = blockDim.x >> 5;
+    sq = warp_sum(lane < nw ? red[0][lane] : 0.f);
+    sk = warp_sum(lane < nw ? red[1][lane] : 0.f);
+    const float rq = rsqrtf(sq / static_cast<float>(q_rank) + eps);
+    const float rk = rsqrtf(sk / static_cast<float>(kv_rank) + eps);
+    for (int i = threadIdx.x; i < qp; i += blockDim.x)
+        put(q_latent + t * qp + i, as_float(row[i]) * rq * as_float(q_weight[i]));
+    const int64_t slot = out_loc[t];
+    if (slot < 0 || slot >= num_slots) {
+        if (threadIdx.x == 0) atomicExch(&status[kStatusBadIndex], static_cast<int>(slot) + 1);
+        return;
+    }
+    for (int i = threadIdx.x; i < rp; i += blockDim.x)
+        put(cache + slot * rp + i, as_float(row[qp + i]) * rk * as_float(kv_weight[i]));
+}
+
+// One CTA per (query row, head); its warps take every fourth key each with an online softmax whose
+// output row is in shared memory, and merge at the end.  Any width, either dtype; not built for speed.
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_attention_plain_kernel(T* __restrict__ out, const T* __restrict__ q, const T* __restrict__ cache,
+                              int64_t num_slots, const int32_t* __restrict__ page_table, int64_t pt_stride,
+                              const int32_t* __restrict__ row_table, const int32_t* __restrict__ row_len, int heads,
+                              int width, float scale, int* status) {
+    extern __shared__ float smem[];   // q [width], then o [4][width]
+    __shared__ float s_m[4], s_l[4];
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int64_t row = blockIdx.x;
+    const int h = blockIdx.y;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    float* sq = smem;
+    float* so = smem + (1 + warp) * width;
+    const T* qr = q + (row * heads + h) * width;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) sq[i] = as_float(qr[i]);
+    for (int i = lane; i < width; i += 32) so[i] = 0.f;
+    __syncthreads();
+    const int32_t* pt = page_table + static_cast<int64_t>(row_table[row]) * pt_stride;
+    const int len = row_len[row];
+    float m = -INFINITY, l = 0.f;
+    for (int j = warp; j < len; j += 4) {
+        int64_t slot = pt[j];
+        if (slot < 0 || slot >= num_slots) {
+            if (lane == 0) atomicExch(&status[kStatusBadIndex], static_cast<int>(slot) + 1);
+            slot = 0;
+        }
+        const T* c = cache + slot * width;
+        float s = 0.f;
+        for (int i = lane; i < width; i += 32) s = fmaf(sq[i], as_float(c[i]), s);
+        s = warp_sum(s) * scale;
+        const float m_new = fmaxf(m, s);
+        const float alpha = expf(m - m_new), p = expf(s - m_new);
+        l = l * alpha + p;
+        m = m_new;
+        for (int i = lane; i < width; i += 32) so[i] = so[i] * alpha + p * as_float(c[i]);
+    }
+    if (lane == 0) {
+        s_m[warp] = m;
+        s_l[warp] = l;
+    }
+    __syncthreads();
+    float mx = -INFINITY, tot = 0.f, f[4];
+#pragma unroll
+    for (int w = 0; w < 4; ++w) mx = fmaxf(mx, s_m[w]);
+#pragma unroll
+    for (int w = 0; w < 4; ++w) {
+        f[w] = s_m[w] == -INFINITY ? 0.f : expf(s_m[w] - mx);
+        tot += f[w] * s_l[w];
+    }
+    const float inv = tot > 0.f ? 1.f / tot : 0.f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        float v = 0.f;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) v += f[w] * smem[(1 + w) * width + i];
+        put(out + (row * heads + h) * width + i, v * inv);
+    }
+}
+
+__global__ void __launch_bounds__(256)
+gather_latents_kernel(uint4* __restrict__ out, const uint4* __restrict__ cache, int64_t num_slots,
+                      const int32_t* __restrict__ page_table, int64_t pt_stride,
+                      const int32_t* __restrict__ table_idx, const int32_t* __restrict__ seq_lens,
+                      const int32_t* __restrict__ base, int vec_per_row, int* status) {
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int b = blockIdx.y;
+    const int at = base[b];
+    const int len = seq_lens[b];
+    if (at < 0) return;
+    const int32_t* pt = page_table + static_cast<int64_t>(table_idx[b]) * pt_stride;
+    const int64_t total = static_cast<int64_t>(len) * vec_per_row;
+    for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
+         i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+        const int64_t pos = i / vec_per_row;
+        const int v = static_cast<int>(i - pos * vec_per_row);
+        int64_t slot = pt[pos];
+        if (slot < 0 || slot >= num_slots) {
+            if (v == 0) atomicExch(&status[kStatusBadIndex], static_cast<int>(slot) + 1);
+            slot = 0;
+        }
+        out[(at + pos) * vec_per_row + v] = cache[slot * vec_per_row + v];
+    }
+}
+
+template <bool SCATTER>
+__global__ void __launch_bounds__(128)
+move_rows_kernel(uint4* __restrict__ out, const uint4* __restrict__ in, const int32_t* __restrict__ rows,
+                 int vec_per_row) {
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int64_t i = blockIdx.x, r = rows[i];
+    const uint4* src = in + (SCATTER ? i : r) * vec_per_row;
+    uint4* dst = out + (SCATTER ? r : i) * vec_per_row;
+    for (int v = threadIdx.x; v < vec_per_row; v += blockDim.x) dst[v] = src[v];
+}
+
+}  // namespace
+
+int launch_latent_norm_store(void* q_latent, void* cache, const void* joint, const void* q_weight,
+                             const void* kv_weight, const int32_t* out_loc, int tokens, int q_rank, int qp,
+                             int kv_rank, int rp, int64_t num_slots, float eps, int dtype, int* status,
+                             cudaStream_t stream) {
+    if (tokens == 0) return B200_OK;
+    if (dtype == B200_DTYPE_F32) {
+        B200_CHECK_CUDA(launch_kernel(latent_norm_store_kernel<float>, dim3(tokens), dim3(256), 0, stream, dim3(1, 1, 1),
+                                      static_cast<float*>(q_latent), static_cast<float*>(cache),
+                                      static_cast<const float*>(joint), static_cast<const float*>(q_weight),
+                                      static_cast<const float*>(kv_weight), out_loc, q_rank, qp, kv_rank, rp, num_slots,
+                                      eps, status));
+    } else {
+        using B = __nv_bfloat16;
+        B200_CHECK_CUDA(launch_kernel(latent_norm_store_kernel<B>, dim3(tokens), dim3(256), 0, stream, dim3(1, 1, 1),
+                                      static_cast<B*>(q_latent), static_cast<B*>(cache), static_cast<const B*>(joint),
+                                      static_cast<const B*>(q_weight), static_cast<const B*>(kv_weight), out_loc, q_rank,
+                                      qp, kv_rank, rp, num_slots, eps, status));
+    }
+    return B200_OK;
+}
+
+int launch_latent_attention_plain(const LatentAttention& a, int dtype, int* status, cudaStream_t stream) {
+    if (a.rows == 0) return B200_OK;
+    const int smem = 5 * a.width * static_cast<int>(sizeof(float));
+    if (smem > 200 * 1024 || a.heads > 65535) {
+        set_last_error("latent attention: width %d or %d heads exceed the plain kernel", a.width, a.heads);
+        return B200_ERR_UNSUPPORTED;
+    }
+    auto run = [&](auto* tag) -> int {
+        using T = typename std::remove_pointer<decltype(tag)>::type;
+        auto kernel = latent_attention_plain_kernel<T>;
+        B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+        B200_CHECK_CUDA(launch_kernel(kernel, dim3(a.rows, a.heads), dim3(128), smem, stream, dim3(1, 1, 1),
+                                      static_cast<T*>(a.out), static_cast<const T*>(a.q),
+                                      static_cast<const T*>(a.cache), a.num_slots, a.page_table, a.pt_stride,
+                                      a.row_table, a.row_len, a.heads, a.width, a.scale, status));
+        return B200_OK;
+    };
+    return dtype == B200_DTYPE_F32 ? run(static_cast<float*>(nullptr)) : run(static_cast<__nv_bfloat16*>(nullptr));
+}
+
+int launch_gather_latents(void* out, const void* cache, int64_t num_slots, const int32_t* page_table,
+                          int64_t pt_stride, const int32_t* table_idx, const int32_t* seq_lens,
+                          const int32_t* base, int batch, int max_len, int rp, int* status, cudaStream_t stream) {
+    if (batch == 0 || max_len == 0) return B200_OK;
+    const int vec = rp / 8;
+    const int64_t blocks = div_ceil64(static_cast<int64_t>(max_len) * vec, 256);
+    B200_CHECK_CUDA(launch_kernel(gather_latents_kernel, dim3(static_cast<unsigned>(blocks < 592 ? blocks : 592), batch),
+                                  dim3(256), 0, stream, dim3(1, 1, 1), static_cast<uint4*>(out),
+                                  static_cast<const uint4*>(cache), num_slots, page_table, pt_stride, table_idx,
+                                  seq_lens, base, vec, status));
+    return B200_OK;
+}
+
+int launch_move_rows(void* out, const void* in, const int32_t* rows, int count, int vec_per_row, bool scatter,
+                     cudaStream_t stream) {
+    if (count == 0) return B200_OK;
+    B200_CHECK_CUDA(launch_kernel(scatter ? move_rows_kernel<true> : move_rows_kernel<false>, dim3(count), dim3(128), 0,
+                                  stream, dim3(1, 1, 1), static_cast<uint4*>(out), static_cast<const uint4*>(in), rows,
+                                  vec_per_row));
+    return B200_OK;
+}
+
+}  // namespace b200
+
+extern "C" {
+
+int64_t b200_latent_attention_workspace_bytes(int rows, int heads, int width) {
+    if (rows < 0 || heads <= 0 || width <= 0) return -1;
+    return b200::latent_attention_workspace_bytes(rows, heads, width);
+}
+
+int b200_latent_attention(void* out, const void* q, const void* cache, int64_t num_slots, const int32_t* page_table,
+                          int64_t page_table_stride, const int32_t* row_table, const int32_t* row_len, int rows,
+                          int heads, int width, int page_size, float scale, int dtype, int plain, void* workspace,
+                          int64_t workspace_bytes, b200_stream_t stream) {
+    B200_CHECK_ARG(rows >= 0 && heads > 0 && width > 0 && width % 128 == 0 && num_slots > 0,
+                   "latent_attention: bad shape");
+    B200_CHECK_ARG(page_size >= 1 && (page_size & (page_size - 1)) == 0, "latent_attention: page_size must be a power of two");
+    B200_CHECK_ARG(dtype == B200_DTYPE_BF16 || dtype == B200_DTYPE_F32, "latent_attention: unknown dtype");
+    if (rows == 0) return B200_OK;
+    B200_CHECK_ARG(out && q && cache && page_table && row_table && row_len, "latent_attention: NULL tensor");
+    int err = B200_OK;
+    int* status = b200::device_status_words(&err);
+    if (err != B200_OK) return err;
+    b200::LatentAttention a;
+    a.out = out;
+    a.q = q;
+    a.cache = cache;
+    a.num_slots = num_slots;
+    a.page_table = page_table;
+    a.pt_stride = page_table_stride;
+    a.row_table = row_table;
+    a.row_len = row_len;
+    a.rows = rows;
+    a.heads = heads;
+    a.width = width;
+    a.page_size = page_size;
+    a.scale = scale;
+    a.workspace = workspace;
+    a.workspace_bytes = workspace_bytes;
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    if (dtype == B200_DTYPE_BF16 && !plain && b200::latent_attention_tc_supported(a)) {
+        B200_CHECK_ARG(workspace && workspace_bytes >= b200::latent_attention_workspace_bytes(rows, heads, width),
+                       "latent_attention: workspace too small");
+        return b200::launch_latent_attention_tc(a, status, s);
+    }
+    return b200::launch_latent_attention_plain(a, dtype, status, s);
+}
+
+}  // extern "C"

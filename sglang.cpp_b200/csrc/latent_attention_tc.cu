@@ -1,0 +1,676 @@
+// Split-KV attention in the latent space on the tcgen05 tensor cores (decode steps, short extensions).
+//
+// Every query row (one token) has H heads that all read the same latents, so one latent tile is loaded
+// once for all heads.  The products are turned around so that the long dimension, not the few heads, fills
+// the 128 rows of the MMA:
+//     S^T = C Q^T      128 keys x N heads, K = latent width: A is the latent tile as TMA delivers it
+//     O^T += C^T P^T   128 latent elements x N heads, K = 128 keys: A is the SAME tile read MN-major, so it
+//                      is fetched from HBM once and never moved again
+// with N = 16, 32 or 64 heads per block (more heads run as further blocks of the same row) and S^T, O^T
+// accumulating in TMEM.
+//
+// A tile is 128 keys; it lives in shared memory as width / 128 units of 128 keys x 128 elements (32 KB), a
+// ring of which the producer keeps full; a unit is free again as soon as its O^T product has read it.
+// Softmax: one thread per key (= TMEM lane), all heads of the block in its registers.  The reference
+// maximum of a head only moves when some score exceeds it by more than 2^8, which a single block-wide vote
+// finds out; the running sum stays per thread until a row is finished.  Everything about scores and weights
+// is fp32; the weights are rounded to bf16 only as the operand of the second product.
+//
+// Work split: the tiles of all (row, head block) items form one sequence that is cut into equal contiguous
+// runs, one per CTA (one CTA per SM).  An item that spans CTAs leaves fp32 partials, combined by the merge
+// kernel.  No host plan: lengths are read from device memory, so a captured graph replays at any lengths.
+//
+// Roles: warp 0 producer, warp 1 one thread issues every MMA, warps 2-5 softmax and output.
+#include <math.h>
+
+#include "common.cuh"
+#include "kernels.h"
+#include "tcgen05.cuh"
+#include "tensormap.cuh"
+
+namespace b200 {
+namespace {
+
+constexpr int kTileKeys = 128;
+constexpr int kUnitElems = 128;                            // latent elements per unit
+constexpr uint32_t kAtomBytes = kTileKeys * 128;           // 128 keys x 64 elements, 128-byte rows
+constexpr uint32_t kUnitBytes = 2 * kAtomBytes;
+constexpr int kMaxUnits = 6;                               // units in the ring
+constexpr int kThreads = 192;
+constexpr int kMaxWidth = 512;
+constexpr uint32_t kColO = 0, kColS = 256;                 // TMEM columns: O^T (4 x 64), S^T (2 x 64)
+constexpr float kLazyLog2 = 8.0f;
+
+struct LatentParams {
+    __nv_bfloat16* out;         // [rows, heads, width]
+    float* part_o;              // [2 * grid][N][width] un-normalised
+    float* part_m;              // [2 * grid][N]
+    float* part_l;
+    int32_t* item_cta;          // [2 * items]: first and last CTA of an item
+    const int32_t* page_table;
+    int64_t pt_stride;
+    const int32_t* row_table;
+    const int32_t* row_len;
+    int rows, heads, width;
+    int blocks, per_block;      // head blocks per row, heads per block (<= N)
+    int nb;                     // units per tile
+    int ring;                   // units in the ring (>= nb)
+    int kpc;                    // keys per TMA copy
+    int64_t num_slots;
+    float scale_log2;
+    int* status;
+};
+
+// MN-major operand under the 128-byte swizzle (rows are keys, 64 latent elements per 128-byte row): the
+// next 64 elements one atom further, the next 8 keys 1024 bytes further.
+__device__ __forceinline__ uint64_t mnmajor_desc(uint32_t smem_addr) {
+    uint64_t d = 0;
+    d |= static_cast<uint64_t>((smem_addr >> 4) & 0x3FFFu);
+    d |= static_cast<uint64_t>(kAtomBytes >> 4) << 16;
+    d |= static_cast<uint64_t>(1024 >> 4) << 32;
+    d |= static_cast<uint64_t>(1) << 46;
+    d |= static_cast<uint64_t>(2) << 61;
+    return d;
+}
+
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+__device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+__device__ __forceinline__ bool softmax_any(bool v) {
+    uint32_t r;
+    asm volatile(
+        "{\n\t"
+        ".reg .pred p, q;\n\t"
+        "setp.ne.u32 p, %1, 0;\n\t"
+        "bar.red.or.pred q, 2, 128, p;\n\t"
+        "selp.u32 %0, 1, 0, q;\n\t"
+        "}\n"
+        : "=r"(r)
+        : "r"(v ? 1u : 0u)
+        : "memory");
+    return r != 0;
+}
+
+// Sums N per-lane vectors over the 32 lanes of a warp: each halving step swaps half of what is left with
+// the lane `off` away.  Afterwards v[j] holds the total of column `col0 + j`, j < max(N / 32, 1).
+template <int N>
+__device__ __forceinline__ int warp_transpose_sum(float (&v)[N]) {
+    const int lane = threadIdx.x & 31;
+    int n = N, col0 = 0;
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) {
+        if (n > 1) {
+            const int half = n / 2;
+            const bool upper = (lane & off) != 0;
+#pragma unroll
+            for (int j = 0; j < N / 2; ++j) {
+                if (j < half) {
+                    const float send = upper ? v[j] : v[j + half];
+                    const float keep = upper ? v[j + half] : v[j];
+                    v[j] = keep + __shfl_xor_sync(0xffffffffu, send, off);
+                }
+            }
+            if (upper) col0 += half;
+            n = half;
+        } else {
+            v[0] += __shfl_xor_sync(0xffffffffu, v[0], off);
+        }
+    }
+    return col0;
+}
+
+// The run of tiles a CTA owns, walked item by item by every role in the same order.
+struct Walk {
+    int row, block, tile;   // current item and first tile of it that belongs to this CTA
+    int left;               // tiles this CTA still has to do
+};
+struct Segment {
+    int row, block, t0, t1, len;   // tiles [t0, t1) of an item whose row has len keys
+    bool starts, ends;             // the item starts / ends inside this segment
+};
+__device__ __forceinline__ bool next_segment(Walk& w, const LatentParams& p, Segment& s) {
+    if (w.left <= 0) return false;
+    int len = p.row_len[w.row];
+    while (len <= 0) {   // rows without keys own no tile
+        ++w.row;
+        w.block = 0;
+        if (w.row >= p.rows) return false;
+        len = p.row_len[w.row];
+    }
+    const int nt = (len + kTileKeys - 1) / kTileKeys;
+    s.row = w.row;
+    s.block = w.block;
+    s.len = len;
+    s.t0 = w.tile;
+    s.t1 = min(nt, w.tile + w.left);
+    s.starts = s.t0 == 0;
+    s.ends = s.t1 == nt;
+    w.left -= s.t1 - s.t0;
+    w.tile = 0;
+    if (++w.block == p.blocks) {
+        w.block = 0;
+        if (++w.row >= p.rows) w.left = 0;
+    }
+    return true;
+}
+
+template <int N>
+__global__ void __launch_bounds__(kThreads, 1)
+latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid_constant__ CUtensorMap tmap_q,
+                           const LatentParams p) {
+    extern __shared__ uint8_t smem_raw[];
+    __shared__ __align__(8) uint64_t unit_full[kMaxUnits];
+    __shared__ __align__(8) uint64_t unit_empty[kMaxUnits];
+    __shared__ __align__(8) uint64_t q_full, q_empty, s_full[2], p_full, pv_done, o_free;
+    __shared__ uint32_t tmem_base_slot;
+    __shared__ int s_scan[kThreads / 32 + 1];
+    __shared__ int s_total, s_row, s_block, s_tile;
+    __shared__ __align__(16) float s_ref[N];     // reference maximum per head, log2 units
+    __shared__ __align__(16) float s_alpha[N];
+    __shared__ float s_warp[4][N];
+    __shared__ volatile int s_failed[2];
+
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t smem_base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+    const uint32_t q_base = smem_base + static_cast<uint32_t>(p.ring) * kUnitBytes;
+    const uint32_t p_base = q_base + static_cast<uint32_t>(N) * static_cast<uint32_t>(p.width) * 2u;
+
+    pdl_launch_dependents();
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < p.ring; ++i) {
+            mbar_init(smem_u32(&unit_full[i]), 1);
+            mbar_init(smem_u32(&unit_empty[i]), 1);
+        }
+        mbar_init(smem_u32(&q_full), 1);
+        mbar_init(smem_u32(&q_empty), 1);
+        mbar_init(smem_u32(&s_full[0]), 1);
+        mbar_init(smem_u32(&s_full[1]), 1);
+        mbar_init(smem_u32(&p_full), 4);
+        mbar_init(smem_u32(&pv_done), 1);
+        mbar_init(smem_u32(&o_free), 4);
+        fence_mbar_init();
+        tma_prefetch_desc(&tmap_c);
+        tma_prefetch_desc(&tmap_q);
+        s_row = p.rows;
+        s_failed[0] = s_failed[1] = 0;
+    }
+    if (warp == 1) {
+        tmem_alloc(smem_u32(&tmem_base_slot), 512);
+        tmem_relinquish();
+    }
+    pdl_wait_prior();
+
+    // ---- where this CTA's run starts: a scan of the rows' tile counts ----
+    {
+        const int per = (p.rows + kThreads - 1) / kThreads;
+        const int r0 = min(static_cast<int>(threadIdx.x) * per, p.rows), r1 = min(r0 + per, p.rows);
+        int mine = 0;
+        for (int r = r0; r < r1; ++r) mine += (max(p.row_len[r], 0) + kTileKeys - 1) / kTileKeys * p.blocks;
+        int incl = mine;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int up = __shfl_up_sync(0xffffffffu, incl, o);
+            if (lane >= o) incl += up;
+        }
+        if (lane == 31) s_scan[warp] = incl;
+        __syncthreads();
+        int before = 0, total = 0;
+        for (int w = 0; w < kThreads / 32; ++w) {
+            if (w < warp) before += s_scan[w];
+            total += s_scan[w];
+        }
+        const int begin = before + incl - mine;
+        const int run = (total + static_cast<int>(gridDim.x) - 1) / static_cast<int>(gridDim.x);
+        const int g0 = static_cast<int>(blockIdx.x) * run;
+        if (g0 >= begin && g0 < begin + mine) {
+            int at = begin;
+            for (int r = r0; r < r1; ++r) {
+                const int nt = (max(p.row_len[r], 0) + kTileKeys - 1) / kTileKeys;
+                if (g0 < at + nt * p.blocks) {
+                    s_row = r;
+                    s_block = (g0 - at) / nt;
+                    s_tile = (g0 - at) % nt;
+                    break;
+                }
+                at += nt * p.blocks;
+            }
+        }
+        if (threadIdx.x == 0) s_total = total;
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem_base = tmem_base_slot;
+    const int run = (s_total + static_cast<int>(gridDim.x) - 1) / static_cast<int>(gridDim.x);
+    const int g0 = static_cast<int>(blockIdx.x) * run;
+    Walk walk;
+    walk.row = s_row;
+    walk.block = s_block;
+    walk.tile = s_tile;
+    walk.left = s_row < p.rows ? min(run, s_total - g0) : 0;
+    bool failed = false;
+    Segment seg;
+
+    if (warp == 0) {
+        // ================= producer =================
+        const int copies = kTileKeys / p.kpc;
+        int unit = 0, nseg = 0;
+        while (!failed && next_segment(walk, p, seg)) {
+            const int32_t* pt = p.page_table + static_cast<int64_t>(p.row_table[seg.row]) * p.pt_stride;
+            for (int t = seg.t0; t < seg.t1 && !failed; ++t) {
+                // the slots of this tile's pages; a copy past the last key reads a row outside the tensor,
+                // which the copy engine fills with zeros
+                int sl[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int copy = i * 32 + lane, key = t * kTileKeys + copy * p.kpc;
+                    sl[i] = static_cast<int>(p.num_slots);
+                    if (copy < copies && key < seg.len) {
+                        const int64_t v = pt[key];
+                        if (v < 0 || v + p.kpc > p.num_slots)
+                            atomicExch(&p.status[kStatusBadIndex], static_cast<int>(v) + 1);
+                        else
+                            sl[i] = static_cast<int>(v);
+                    }
+                }
+                for (int u = 0; u < p.nb && !failed; ++u, ++unit) {
+                    const int s = unit % p.ring;
+                    const bool ok = unit < p.ring || mbar_wait_bounded(smem_u32(&unit_empty[s]),
+                                                                       static_cast<uint32_t>(unit / p.ring - 1) & 1u, p.status, 601);
+                    if (!__all_sync(0xffffffffu, ok)) {
+                        failed = true;
+                        break;
+                    }
+                    const uint32_t bar = smem_u32(&unit_full[s]);
+                    const uint32_t dst = smem_base + static_cast<uint32_t>(s) * kUnitBytes;
+                    if (lane == 0) mbar_arrive_expect_tx(bar, kUnitBytes);
+                    __syncwarp();
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const int copy = i * 32 + lane;
+                        if (copy < copies) {
+                            const uint32_t to = dst + static_cast<uint32_t>(copy * p.kpc) * 128u;
+                            tma_load_2d(to, &tmap_c, u * kUnitElems, sl[i], bar);
+                            tma_load_2d(to + kAtomBytes, &tmap_c, u * kUnitElems + 64, sl[i], bar);
+                        }
+                    }
+                }
+                if (t == seg.t0 && !failed) {
+                    // the queries of this item, behind the first tile's latents
+                    const bool ok = nseg == 0 || mbar_wait_bounded(smem_u32(&q_empty), static_cast<uint32_t>(nseg - 1) & 1u,
+                                                                   p.status, 602);
+                    if (!__all_sync(0xffffffffu, ok)) {
+                        failed = true;
+                        break;
+                    }
+                    const uint32_t bar = smem_u32(&q_full);
+                    if (lane == 0) mbar_arrive_expect_tx(bar, static_cast<uint32_t>(N) * p.width * 2u);
+                    __syncwarp();
+                    for (int a = lane; a < p.width / 64; a += 32)
+                        tma_load_2d(q_base + static_cast<uint32_t>(a) * N * 128u, &tmap_q, a * 64,
+                                    seg.row * p.heads + seg.block * p.per_block, bar);
+                }
+            }
+            ++nseg;
+        }
+    } else if (warp == 1) {
+        // ================= MMA issuer =================
+        if (lane == 0) {
+            const uint32_t idesc_s = idesc_bf16_m128(N);
+            const uint32_t idesc_o = idesc_bf16_m128(N) | (1u << 15);   // A is MN-major
+            int unit = 0;    // first unit of the tile whose S^T is being issued
+            int tiles = 0;   // tiles whose P has been consumed
+            int nseg = 0;
+            // units [u0, u1) of S^T for the tile that starts at unit `first`, into buffer `buf`
+            auto issue_s = [&](int first, int u0, int u1, int buf) {
+                for (int u = u0; u < u1; ++u) {
+                    const int n = first + u, s = n % p.ring;
+                    if (!mbar_wait_bounded(smem_u32(&unit_full[s]), static_cast<uint32_t>(n / p.ring) & 1u, p.status, 603)) {
+                        failed = true;
+                        return;
+                    }
+                    tc_fence_after();
+                    const uint32_t a = smem_base + static_cast<uint32_t>(s) * kUnitBytes;
+                    const uint32_t b = q_base + static_cast<uint32_t>(2 * u) * N * 128u;
+                    const uint32_t d = tmem_base + kColS + static_cast<uint32_t>(buf) * 64u;
+#pragma unroll
+                    for (int ks = 0; ks < 8; ++ks)
+                        tc_mma_bf16(d, kmajor_sw128_desc(a + (ks >> 2) * kAtomBytes + (ks & 3) * 32),
+                                    kmajor_sw128_desc(b + (ks >> 2) * N * 128u + (ks & 3) * 32), idesc_s,
+                                    (u > 0 || ks > 0) ? 1u : 0u);
+                }
+                if (u1 == p.nb) tc_commit(smem_u32(&s_full[buf]));
+            };
+            while (!failed && next_segment(walk, p, seg)) {
+                if (!mbar_wait_bounded(smem_u32(&q_full), static_cast<uint32_t>(nseg) & 1u, p.status, 604)) {
+                    failed = true;
+                    break;
+                }
+                tc_fence_after();
+                issue_s(unit, 0, p.nb, tiles & 1);
+                for (int t = seg.t0; t < seg.t1 && !failed; ++t) {
+                    const int cur = unit;
+                    unit += p.nb;
+                    const bool more = t + 1 < seg.t1;
+                    // as much of the next tile's S^T as the ring can hold beside the current tile
+                    const int ahead = min(p.nb, p.ring - p.nb);
+                    if (more && ahead > 0) issue_s(unit, 0, ahead, (tiles + 1) & 1);
+                    if (!more) tc_commit(smem_u32(&q_empty));   // every S^T of this item has been issued
+                    if (failed || !mbar_wait_bounded(smem_u32(&p_full), static_cast<uint32_t>(tiles) & 1u, p.status, 605)) {
+                        failed = true;
+                        break;
+                    }
+                    if (t == seg.t0 && nseg > 0 &&
+                        !mbar_wait_bounded(smem_u32(&o_free), static_cast<uint32_t>(nseg - 1) & 1u, p.status, 606)) {
+                        failed = true;
+                        break;
+                    }
+                    tc_fence_after();
+                    for (int u = 0; u < p.nb; ++u) {
+                        const int s = (cur + u) % p.ring;
+                        const uint32_t a = smem_base + static_cast<uint32_t>(s) * kUnitBytes;
+                        const uint32_t d = tmem_base + kColO + static_cast<uint32_t>(u * N);
+#pragma unroll
+                        for (int ks = 0; ks < 8; ++ks)
+                            tc_mma_bf16(d, mnmajor_desc(a + ks * 2048),
+                                        kmajor_sw128_desc(p_base + (ks >> 2) * N * 128u + (ks & 3) * 32), idesc_o,
+                                        (t > seg.t0 || ks > 0) ? 1u : 0u);
+                        tc_commit(smem_u32(&unit_empty[s]));
+                    }
+                    tc_commit(smem_u32(&pv_done));
+                    if (more && ahead < p.nb) issue_s(unit, ahead, p.nb, (tiles + 1) & 1);
+                    ++tiles;
+                }
+                ++nseg;
+            }
+        }
+    } else {
+        // ================= softmax and output =================
+        const int q = warp & 3;                 // TMEM lane quarter this warp may read
+        const int key = q * 32 + lane;          // key inside the tile = latent element inside a unit
+        const int st = static_cast<int>(threadIdx.x) - 64;   // 0..127
+        const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(q * 32) << 16);
+        const uint32_t p_key = p_base + static_cast<uint32_t>(key >> 6) * N * 128u + static_cast<uint32_t>(key & 7) * 2u;
+        const uint32_t p_chunk = static_cast<uint32_t>((key & 63) >> 3);
+        int tiles = 0;
+        float l[N];
+        while (!failed && next_segment(walk, p, seg)) {
+#pragma unroll
+            for (int h = 0; h < N; ++h) l[h] = 0.f;
+            if (st < N) s_ref[st] = -INFINITY;
+            softmax_sync();
+            for (int t = seg.t0; t < seg.t1; ++t, ++tiles) {
+                const int buf = tiles & 1;
+                if (!mbar_wait_bounded(smem_u32(&s_full[buf]), static_cast<uint32_t>(tiles >> 1) & 1u, p.status, 607)) failed = true;
+                tc_fence_after();
+                const uint32_t s_addr = lane_addr + kColS + static_cast<uint32_t>(buf) * 64u;
+                const bool valid = t * kTileKeys + key < seg.len;
+                // does any score outgrow its head's reference?
+                bool over = false;
+#pragma unroll
+                for (int c = 0; c < N / 16; ++c) {
+                    uint32_t sv[16];
+                    tmem_ld_32x32b_x16(s_addr + c * 16, sv);
+                    tmem_ld_wait();
+#pragma unroll
+                    for (int j = 0; j < 16; ++j)
+                        over |= __uint_as_float(sv[j]) * p.scale_log2 > s_ref[c * 16 + j] + kLazyLog2;
+                }
+                // the previous product has read P and written O before either is touched again
+                if (t > seg.t0 && !failed &&
+                    !mbar_wait_bounded(smem_u32(&pv_done), static_cast<uint32_t>(tiles - 1) & 1u, p.status, 608))
+                    failed = true;
+                // a wait that ran out in one warp ends all four at the same place (two flags in turn: a
+                // warp may be one tile behind the one that sets the next)
+                if (failed) s_failed[tiles & 1] = 1;
+                const bool moved = softmax_any(over && valid);
+                if (s_failed[tiles & 1] != 0) {
+                    failed = true;
+                    break;
+                }
+                tc_fence_after();
+                if (moved) {
+#pragma unroll
+                    for (int c = 0; c < N / 16; ++c) {
+                        uint32_t sv[16];
+                        tmem_ld_32x32b_x16(s_addr + c * 16, sv);
+                        tmem_ld_wait();
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) {
+                            const float mx = warp_max(valid ? __uint_as_float(sv[j]) * p.scale_log2 : -INFINITY);
+                            if (lane == 0) s_warp[q][c * 16 + j] = mx;
+                        }
+                    }
+                    softmax_sync();
+                    if (st < N) {
+                        const float old = s_ref[st];
+                        const float mx = fmaxf(fmaxf(fmaxf(s_warp[0][st], s_warp[1][st]), fmaxf(s_warp[2][st], s_warp[3][st])), old);
+                        s_alpha[st] = old == -INFINITY ? 1.f : ex2(old - mx);
+                        s_ref[st] = mx;
+                    }
+                    softmax_sync();
+                    if (t > seg.t0) {
+#pragma unroll
+                        for (int h = 0; h < N; ++h) l[h] *= s_alpha[h];
+                        for (int u = 0; u < p.nb; ++u)
+#pragma unroll
+                            for (int c = 0; c < N / 16; ++c) {
+                                const uint32_t o_addr = lane_addr + kColO + static_cast<uint32_t>(u * N + c * 16);
+                                uint32_t ov[16];
+                                tmem_ld_32x32b_x16(o_addr, ov);
+                                tmem_ld_wait();
+#pragma unroll
+                                for (int j = 0; j < 16; ++j)
+                                    ov[j] = __float_as_uint(__uint_as_float(ov[j]) * s_alpha[c * 16 + j]);
+                                tmem_st_32x32b_x16(o_addr, ov);
+                            }
+                        tmem_st_wait();
+                    }
+                }
+#pragma unroll
+                for (int c = 0; c < N / 16; ++c) {
+                    uint32_t sv[16];
+                    tmem_ld_32x32b_x16(s_addr + c * 16, sv);
+                    tmem_ld_wait();
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) {
+                        const int h = c * 16 + j;
+                        const float w = valid ? ex2(fmaf(__uint_as_float(sv[j]), p.scale_log2, -s_ref[h])) : 0.f;
+                        l[h] += w;
+                        const __nv_bfloat16 b = __float2bfloat16_rn(w);
+                        const uint32_t addr = p_key + static_cast<uint32_t>(h) * 128u + ((p_chunk ^ (h & 7)) << 4);
+                        asm volatile("st.shared.b16 [%0], %1;" ::"r"(addr), "h"(*reinterpret_cast<const uint16_t*>(&b))
+                                     : "memory");
+                    }
+                }
+                fence_proxy_async_smem();
+                tc_fence_before();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(smem_u32(&p_full));
+            }
+            if (failed) break;
+            if (!mbar_wait_bounded(smem_u32(&pv_done), static_cast<uint32_t>(tiles - 1) & 1u, p.status, 609)) failed = true;
+            tc_fence_after();
+            {
+                const int col = warp_transpose_sum<N>(l);
+                constexpr int kCols = N >= 32 ? N / 32 : 1;
+#pragma unroll
+                for (int j = 0; j < kCols; ++j) s_warp[q][col + j] = l[j];
+            }
+            if (softmax_any(failed)) {
+                failed = true;
+                break;
+            }
+            const int item = seg.row * p.blocks + seg.block;
+            const int cut = seg.starts ? 1 : 0;      // partial slot: 1 = goes on in the next CTA, 0 = came from the one before
+            const bool whole = seg.starts && seg.ends;
+            const int64_t slot = static_cast<int64_t>(blockIdx.x) * 2 + cut;
+            if (st < N) {
+                const float tot = s_warp[0][st] + s_warp[1][st] + s_warp[2][st] + s_warp[3][st];
+                s_alpha[st] = whole ? 1.f / tot : 1.f;
+                if (!whole) {
+                    p.part_m[slot * N + st] = s_ref[st];
+                    p.part_l[slot * N + st] = tot;
+                }
+            }
+            if (st == 0 && seg.starts) {
+                // the CTAs that share this item follow from its first tile's place in the sequence
+                const int nt = (seg.len + kTileKeys - 1) / kTileKeys;
+                const int first = g0 + tiles - (seg.t1 - seg.t0);
+                p.item_cta[2 * item] = static_cast<int>(blockIdx.x);
+                p.item_cta[2 * item + 1] = (first + nt - 1) / run;
+            }
+            softmax_sync();
+            const int h0 = seg.block * p.per_block;
+            const int nh = min(p.per_block, p.heads - h0);
+            for (int u = 0; u < p.nb; ++u) {
+                const int e = u * kUnitElems + key;
+#pragma unroll
+                for (int c = 0; c < N / 16; ++c) {
+                    uint32_t ov[16];
+                    tmem_ld_32x32b_x16(lane_addr + kColO + static_cast<uint32_t>(u * N + c * 16), ov);
+                    tmem_ld_wait();
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) {
+                        const int h = c * 16 + j;
+                        if (h < nh) {
+                            const float v = __uint_as_float(ov[j]);
+                            if (whole)
+                                p.out[(static_cast<int64_t>(seg.row) * p.heads + h0 + h) * p.width + e] =
+                                    __float2bfloat16_rn(v * s_alpha[h]);
+                            else
+                                p.part_o[(slot * N + h) * p.width + e] = v;
+                        }
+                    }
+                }
+            }
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(smem_u32(&o_free));
+        }
+    }
+    __syncwarp();
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 1) tmem_dealloc(tmem_base, 512);
+}
+
+// One CTA per (item, head): weighs the partials of an item that was cut over several CTAs.
+__global__ void __launch_bounds__(128)
+latent_merge_kernel(const LatentParams p, int N) {
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int row = blockIdx.x / p.heads, head = blockIdx.x - row * p.heads;
+    const int block = head / p.per_block, h = head - block * p.per_block;
+    const int item = row * p.blocks + block;
+    __nv_bfloat16* out = p.out + (static_cast<int64_t>(row) * p.heads + head) * p.width;
+    if (p.row_len[row] <= 0) {   // no keys: zeros
+        for (int i = threadIdx.x; i < p.width; i += blockDim.x) out[i] = __float2bfloat16_rn(0.f);
+        return;
+    }
+    const int c0 = p.item_cta[2 * item], c1 = p.item_cta[2 * item + 1];
+    if (c0 == c1) return;   // written whole
+    auto slot_of = [&](int c) { return (static_cast<int64_t>(c) * 2 + (c == c0 ? 1 : 0)) * N + h; };
+    float mx = -INFINITY;
+    for (int c = c0; c <= c1; ++c) mx = fmaxf(mx, p.part_m[slot_of(c)]);
+    float tot = 0.f;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    const int e = static_cast<int>(threadIdx.x) * 4;
+    for (int c = c0; c <= c1; ++c) {
+        const int64_t s = slot_of(c);
+        const float f = ex2(p.part_m[s] - mx);
+        tot += f * p.part_l[s];
+        if (e < p.width) {
+            const float4 v = *reinterpret_cast<const float4*>(p.part_o + s * p.width + e);
+            acc.x += f * v.x;
+            acc.y += f * v.y;
+            acc.z += f * v.z;
+            acc.w += f * v.w;
+        }
+    }
+    const float inv = tot > 0.f ? 1.f / tot : 0.f;
+    if (e < p.width)
+        *reinterpret_cast<uint2*>(out + e) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
+}
+
+struct Shape {
+    int n, blocks, per_block;
+};
+Shape shape_of(int heads) {
+    Shape s;
+    s.blocks = div_ceil(heads, 64);
+    s.per_block = div_ceil(heads, s.blocks);
+    s.n = s.per_block <= 16 ? 16 : s.per_block <= 32 ? 32 : 64;
+    return s;
+}
+
+int64_t align256(int64_t x) { return (x + 255) / 256 * 256; }
+
+}  // namespace
+
+int64_t latent_attention_workspace_bytes(int rows, int heads, int width) {
+    const Shape s = shape_of(heads);
+    const int64_t slots = 2ll * 160;   // two per CTA, at most one CTA per SM (148)
+    return align256(slots * s.n * width * 4) + 2 * align256(slots * s.n * 4) + align256(static_cast<int64_t>(rows) * s.blocks * 8);
+}
+
+bool latent_attention_tc_supported(const LatentAttention& a) {
+    return a.width % kUnitElems == 0 && a.width <= kMaxWidth && a.scale > 0.f && sm_count() <= 160 &&
+           (reinterpret_cast<uintptr_t>(a.cache) & 15u) == 0 && (reinterpret_cast<uintptr_t>(a.q) & 15u) == 0;
+}
+
+int launch_latent_attention_tc(const LatentAttention& a, int* status, cudaStream_t stream) {
+    if (a.rows == 0) return B200_OK;
+    const Shape sh = shape_of(a.heads);
+    const int grid = sm_count();
+    LatentParams p;
+    p.out = static_cast<__nv_bfloat16*>(a.out);
+    uint8_t* ws = static_cast<uint8_t*>(a.workspace);
+    const int64_t slots = 2ll * 160;
+    p.part_o = reinterpret_cast<float*>(ws);
+    ws += align256(slots * sh.n * a.width * 4);
+    p.part_m = reinterpret_cast<float*>(ws);
+    ws += align256(slots * sh.n * 4);
+    p.part_l = reinterpret_cast<float*>(ws);
+    ws += align256(slots * sh.n * 4);
+    p.item_cta = reinterpret_cast<int32_t*>(ws);
+    p.page_table = a.page_table;
+    p.pt_stride = a.pt_stride;
+    p.row_table = a.row_table;
+    p.row_len = a.row_len;
+    p.rows = a.rows;
+    p.heads = a.heads;
+    p.width = a.width;
+    p.blocks = sh.blocks;
+    p.per_block = sh.per_block;
+    p.nb = a.width / kUnitElems;
+    p.kpc = a.page_size < kTileKeys ? a.page_size : kTileKeys;
+    p.num_slots = a.num_slots;
+    p.scale_log2 = a.scale * 1.4426950408889634f;
+    p.status = status;
+    const uint32_t fixed = static_cast<uint32_t>(sh.n) * a.width * 2u + 2u * sh.n * 128u + 1024u;
+    int ring = kMaxUnits;
+    while (ring > p.nb && static_cast<uint32_t>(ring) * kUnitBytes + fixed > 220u * 1024u) --ring;
+    p.ring = ring;
+    const uint32_t smem = static_cast<uint32_t>(ring) * kUnitBytes + fixed;
+
+    CUtensorMap tc, tq;
+    int err = cached_tmap(&tc, a.cache, static_cast<uint64_t>(a.width), static_cast<uint64_t>(a.num_slots),
+                          static_cast<uint64_t>(a.width) * 2, 64, static_cast<uint32_t>(p.kpc));
+    if (err != B200_OK) return err;
+    err = cached_tmap(&tq, a.q, static_cast<uint64_t>(a.width), static_cast<uint64_t>(a.rows) * a.heads,
+                      static_cast<uint64_t>(a.width) * 2, 64, static_cast<uint32_t>(sh.n));
+    if (err != B200_OK) return err;
+    auto kernel = sh.n == 16 ? latent_attention_tc_kernel<16> : sh.n == 32 ? latent_attention_tc_kernel<32>
+                                                                         : latent_attention_tc_kernel<64>;
+    B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+    B200_CHECK_CUDA(launch_kernel(kernel, dim3(grid), dim3(kThreads), smem, stream, dim3(1, 1, 1), tc, tq, p));
+    B200_CHECK_CUDA(launch_kernel(latent_merge_kernel, dim3(a.rows * a.heads), dim3(128), 0, stream, dim3(1, 1, 1), p, sh.n));
+    return B200_OK;
+}
+
+}  // namespace b200

@@ -157,6 +157,69 @@ moe_combine_kernel(uint4* __restrict__ out, const uint4* __restrict__ y, const i
     }
 }
 
+// Table routing (experts by token id): the placement does not depend on the activations, so one launch at
+// the start of a step lays out every table-routed layer of the model, one CTA per layer: histogram in
+// shared memory, scan, then a row for every (token, choice) pair.
+__global__ void __launch_bounds__(1024)
+table_route_kernel(const TableRouteLayer* __restrict__ layers, const int32_t* __restrict__ token_ids, int tokens,
+                   int vocab, int* status) {
+    extern __shared__ int s_cnt[];
+    __shared__ int s_warp[32];
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const TableRouteLayer L = layers[blockIdx.x];
+    const int E = L.experts;
+    auto expert_of = [&](int pair) {
+        const int id = token_ids[pair / L.top];
+        const int e = id >= 0 && id < vocab ? L.table[static_cast<int64_t>(id) * L.top + pair % L.top] : 0;
+        if (e < 0 || e >= E) {
+            atomicExch(&status[kStatusBadIndex], e + 1);
+            return 0;
+        }
+        return e;
+    };
+    for (int e = threadIdx.x; e < E; e += blockDim.x) s_cnt[e] = 0;
+    __syncthreads();
+    const int pairs = tokens * L.top;
+    for (int i = threadIdx.x; i < pairs; i += blockDim.x) atomicAdd(&s_cnt[expert_of(i)], 1);
+    __syncthreads();
+    // exclusive scan of the counts, each thread a contiguous piece; the counts become running cursors
+    const int per = (E + static_cast<int>(blockDim.x) - 1) / static_cast<int>(blockDim.x);
+    const int e0 = min(static_cast<int>(threadIdx.x) * per, E), e1 = min(e0 + per, E);
+    int mine = 0;
+    for (int e = e0; e < e1; ++e) mine += s_cnt[e];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    int incl = mine;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const int up = __shfl_up_sync(0xffffffffu, incl, o);
+        if (lane >= o) incl += up;
+    }
+    if (lane == 31) s_warp[warp] = incl;
+    __syncthreads();
+    if (warp == 0) {
+        int v = lane < static_cast<int>(blockDim.x >> 5) ? s_warp[lane] : 0;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int up = __shfl_up_sync(0xffffffffu, v, o);
+            if (lane >= o) v += up;
+        }
+        s_warp[lane] = v;
+    }
+    __syncthreads();
+    int run = incl - mine + (warp > 0 ? s_warp[warp - 1] : 0);
+    for (int e = e0; e < e1; ++e) {
+        const int c = s_cnt[e];
+        L.counts[e] = c;
+        L.offsets[e] = run;
+        s_cnt[e] = run;
+        run += c;
+    }
+    if (threadIdx.x == 0) L.offsets[E] = pairs;
+    __syncthreads();
+    for (int i = threadIdx.x; i < pairs; i += blockDim.x) L.rows[i] = atomicAdd(&s_cnt[expert_of(i)], 1);
+}
+
 struct MoeWorkspace {
     int32_t *ids, *counts, *offsets, *cursor, *pos;
     float* weights;
@@ -190,6 +253,14 @@ int64_t carve(MoeWorkspace* w, uint8_t* base, int tokens, int E, int top_k, int 
 int64_t moe_workspace_bytes(int tokens, int E, int top_k, int H, int I) {
     MoeWorkspace w;
     return carve(&w, nullptr, tokens, E, top_k, H, I);
+}
+
+int launch_table_route(const TableRouteLayer* layers_dev, int num_layers, int max_experts, const int32_t* token_ids,
+                       int tokens, int vocab, int* status, cudaStream_t stream) {
+    if (tokens == 0 || num_layers == 0) return B200_OK;
+    B200_CHECK_CUDA(launch_kernel(table_route_kernel, dim3(num_layers), dim3(1024), max_experts * sizeof(int), stream,
+                                  dim3(1, 1, 1), layers_dev, token_ids, tokens, vocab, status));
+    return B200_OK;
 }
 
 int launch_moe_route(int32_t* ids, float* weights, int32_t* counts, const void* logits, int tokens, int E,
@@ -259,6 +330,31 @@ int b200_moe_route(int32_t* topk_ids, float* topk_weights, int32_t* expert_count
     B200_CHECK_ARG(topk_ids && topk_weights && expert_counts && router_logits, "moe_route: NULL tensor");
     return b200::launch_moe_route(topk_ids, topk_weights, expert_counts, router_logits, tokens, num_experts,
                                   top_k, renormalize, static_cast<cudaStream_t>(stream));
+}
+
+int b200_table_route(int32_t* rows, int32_t* counts, int32_t* offsets, const int32_t* table,
+                     const int32_t* token_ids, int tokens, int vocab, int top, int experts, b200_stream_t stream) {
+    B200_CHECK_ARG(tokens >= 0 && vocab > 0 && top > 0 && experts >= top, "table_route: bad shape");
+    B200_CHECK_ARG(experts <= b200::kMaxTableExperts, "table_route: at most %d experts", b200::kMaxTableExperts);
+    if (tokens == 0) return B200_OK;
+    B200_CHECK_ARG(rows && counts && offsets && table && token_ids, "table_route: NULL tensor");
+    int err = B200_OK;
+    int* status = b200::device_status_words(&err);
+    if (err != B200_OK) return err;
+    // the kernel reads its layer descriptions from device memory; a caller of the single-layer form pays
+    // for a small allocation
+    const b200::TableRouteLayer layer{table, rows, counts, offsets, top, experts};
+    void* dev = nullptr;
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    B200_CHECK_CUDA(cudaMalloc(&dev, sizeof(layer)));
+    cudaError_t ce = cudaMemcpyAsync(dev, &layer, sizeof(layer), cudaMemcpyHostToDevice, s);
+    if (ce == cudaSuccess)
+        err = b200::launch_table_route(static_cast<const b200::TableRouteLayer*>(dev), 1, experts, token_ids, tokens, vocab,
+                                       status, s);
+    if (ce == cudaSuccess) ce = cudaStreamSynchronize(s);
+    cudaFree(dev);
+    B200_CHECK_CUDA(ce);
+    return err;
 }
 
 int b200_moe_forward_local(void* out, const void* hidden_states, const void* router_logits,

@@ -99,7 +99,45 @@ argmax_bf16_kernel(int32_t* __restrict__ out, const __nv_bfloat16* __restrict__ 
     }
 }
 
+// fp32 logits (models that run in fp32): one CTA per row, same ordering rules.
+__global__ void __launch_bounds__(512)
+argmax_f32_kernel(int32_t* __restrict__ out, const float* __restrict__ logits, int vocab, int64_t ld,
+                  const TokenWriteBack wb) {
+    __shared__ float s_v[16];
+    __shared__ int s_i[16];
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const float* row = logits + static_cast<int64_t>(blockIdx.x) * ld;
+    MaxIdx best{-INFINITY, 0x7fffffff};
+    for (int i = threadIdx.x; i < vocab; i += blockDim.x) best = better(best, MaxIdx{row[i], i});
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int pass = 0; pass < 2; ++pass) {
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            MaxIdx other{__shfl_xor_sync(0xffffffffu, best.v, o), __shfl_xor_sync(0xffffffffu, best.i, o)};
+            best = better(best, other);
+        }
+        if (pass == 1) break;
+        if (lane == 0) {
+            s_v[warp] = best.v;
+            s_i[warp] = best.i;
+        }
+        __syncthreads();
+        if (warp != 0) return;
+        best = lane < static_cast<int>(blockDim.x >> 5) ? MaxIdx{s_v[lane], s_i[lane]} : MaxIdx{-INFINITY, 0x7fffffff};
+    }
+    if (lane == 0) emit_token(out, wb, static_cast<int>(blockIdx.x), best.i == 0x7fffffff ? 0 : best.i);
+}
+
 }  // namespace
+
+int launch_argmax_f32(int32_t* out, const float* logits, int rows, int vocab, int64_t ld, cudaStream_t stream,
+                      const TokenWriteBack* write_back) {
+    if (rows == 0) return B200_OK;
+    B200_CHECK_CUDA(launch_kernel(argmax_f32_kernel, dim3(rows), dim3(512), 0, stream, dim3(1, 1, 1), out, logits,
+                                  vocab, ld, write_back ? *write_back : TokenWriteBack{}));
+    return B200_OK;
+}
 
 int launch_argmax(int32_t* out, const void* logits, int rows, int vocab, int64_t ld,
                   cudaStream_t stream, const TokenWriteBack* write_back) {

@@ -66,20 +66,16 @@ class Engine:
         (include/sglang/models/config.h:15-42), named as b200_model_config names them."""
         self.model_config = model_config
         self.config = config
-        m = ModelConfigStruct(
-            model_config.num_layers, model_config.hidden_size, model_config.num_qo_heads,
-            model_config.num_kv_heads, model_config.head_dim, model_config.intermediate_size,
-            model_config.vocab_size, model_config.rms_norm_eps, model_config.rope_theta,
-            model_config.max_position, int(model_config.tie_word_embeddings), int(model_config.qk_norm),
-            int(model_config.fused_residual), int(model_config.attention_bias),
-            1 if model_config.hidden_act == "gelu" else 0, model_config.num_experts,
-            model_config.num_experts_per_tok, model_config.moe_intermediate_size,
-            int(model_config.norm_topk_prob))
+        self._h = ctypes.c_void_p()
+        self.stack = getattr(model_config, "layers", None) is not None   # layers listed one by one
+        self.dtype = torch.bfloat16
         c = EngineConfigStruct(config.page_size, config.num_pages, config.max_running_req,
                                config.max_seq_len, config.max_extend_tokens, config.tp_rank,
                                config.tp_size, int(config.expert_parallel))
-        self._h = ctypes.c_void_p()
-        call("b200_engine_create", ctypes.byref(m), ctypes.byref(c), ctypes.byref(self._h))
+        if self.stack:
+            self._create_stack(model_config, c)
+        else:
+            self._create_uniform(model_config, c)
         # A small ring of pinned token buffers, one per step in flight: a step enqueued before the
         # previous step's tokens were read must not overwrite them (the reference allocates a
         # pinned tensor per ForwardOutput, src/engine/engine.cc:526-531).
@@ -89,6 +85,30 @@ class Engine:
         self.dummy_table_idx = config.max_running_req
         self.pt_cols = (config.max_seq_len + 31) // 32 * 32   # page-table row length (src/engine/engine.cc:452-459)
         self._step_index = 0
+
+    def _create_uniform(self, model_config, c) -> None:
+        m = ModelConfigStruct(
+            model_config.num_layers, model_config.hidden_size, model_config.num_qo_heads,
+            model_config.num_kv_heads, model_config.head_dim, model_config.intermediate_size,
+            model_config.vocab_size, model_config.rms_norm_eps, model_config.rope_theta,
+            model_config.max_position, int(model_config.tie_word_embeddings), int(model_config.qk_norm),
+            int(model_config.fused_residual), int(model_config.attention_bias),
+            1 if model_config.hidden_act == "gelu" else 0, model_config.num_experts,
+            model_config.num_experts_per_tok, model_config.moe_intermediate_size,
+            int(model_config.norm_topk_prob))
+        call("b200_engine_create", ctypes.byref(m), ctypes.byref(c), ctypes.byref(self._h))
+
+    def _create_stack(self, model_config, c) -> None:
+        self.dtype = model_config.torch_dtype
+        layers = (_lib.LayerConfigStruct * len(model_config.layers))(
+            *[_lib.LayerConfigStruct(*spec.as_tuple()) for spec in model_config.layers])
+        m = ModelConfigStruct(num_layers=len(model_config.layers), hidden_size=model_config.hidden_size,
+                              vocab_size=model_config.vocab_size, rms_norm_eps=model_config.rms_norm_eps,
+                              tie_word_embeddings=int(model_config.tie_word_embeddings))
+        st = _lib.StackConfigStruct(len(model_config.layers), layers,
+                                    _lib.DTYPE_F32 if self.dtype == torch.float32 else _lib.DTYPE_BF16,
+                                    model_config.norm_offset, model_config.logit_scale)
+        call("b200_engine_create_stack", ctypes.byref(m), ctypes.byref(st), ctypes.byref(c), ctypes.byref(self._h))
 
     def close(self) -> None:
         if self._h:
@@ -115,7 +135,16 @@ class Engine:
     def load_weights(self, w: dict, tp_rank: int = 0, tp_size: int = 1) -> None:
         """Upload weights given in the reference's packed layouts (full, unsharded tensors: a dict
         with "embed", "final_norm", optional "lm_head" and a list "layers" of per-layer dicts),
-        cut with the reference's TP shard rules for this rank (sglang_cpp_b200.tp.shard_layer)."""
+        cut with the reference's TP shard rules for this rank (sglang_cpp_b200.tp.shard_layer).  Models
+        whose layers are listed one by one upload what weights.pack_layer_stack made, as it is."""
+        if self.stack:
+            for name, t in w.items():
+                if name != "layers":
+                    self.load(name, 0, t)
+            for l, L in enumerate(w["layers"]):
+                for name, t in L.items():
+                    self.load(name, l, t)
+            return
         from .tp import shard_layer
 
         cfg = self.model_config
@@ -197,6 +226,22 @@ class Engine:
                 m = min(chunk, view.numel() - off)
                 view[off:off + m] = (torch.randn(m, generator=g, device=dev, dtype=torch.float32) * std).to(torch.bfloat16)
 
+        if self.stack:
+            fill("embed", 0, seed * 1000 + 1)
+            fill("lm_head", 0, seed * 1000 + 2)
+            for l, spec in enumerate(cfg.layers):
+                for i, name in enumerate(("down_qkv", "uq", "uk", "uk_absorb", "uv", "o", "mlp_up", "mlp_down")):
+                    fill(name, l, seed * 1000 + 100 + l * 16 + i)
+                for name in ("q_latent_norm", "kv_latent_norm"):   # (norm1 / norm2 hold gain - 1: zero as allocated)
+                    fill(name, l, 0, ones=True)
+                if spec.num_experts:
+                    ptr, n = self.tensor_info("expert_table", l)
+                    g = torch.Generator(device=dev).manual_seed(seed * 1000 + 99 + l * 16)
+                    rank_of = torch.rand(cfg.vocab_size, spec.num_experts, generator=g, device=dev)
+                    table = rank_of.topk(spec.experts_per_tok, dim=1).indices.to(torch.int32)
+                    _as_cuda_tensor(ptr, n).view(torch.int32).copy_(table.flatten())
+            torch.cuda.synchronize()
+            return
         fill("embed", 0, seed * 1000 + 1)
         if not cfg.tie_word_embeddings:
             fill("lm_head", 0, seed * 1000 + 2)
@@ -317,8 +362,25 @@ class Engine:
         call("b200_engine_synchronize", self._h)
 
     def logits(self, rows: int) -> torch.Tensor:
-        out = torch.empty(rows, self.model_config.vocab_size, dtype=torch.bfloat16)
+        out = torch.empty(rows, self.model_config.vocab_size, dtype=self.dtype)
         call("b200_engine_read_logits", self._h, out.data_ptr(), rows)
+        return out
+
+    def token_logits(self, tokens) -> torch.Tensor:
+        """fp32 logits at any tokens of the last step (places in its flattened token order)."""
+        t = _i32(tokens)
+        out = torch.empty(len(t), self.model_config.vocab_size, dtype=torch.float32)
+        call("b200_engine_token_logits", self._h, t.ctypes.data, len(t), out.data_ptr())
+        return out
+
+    def trace_residual(self, tokens: Optional[int]) -> Optional[torch.Tensor]:
+        """Debugging: the fp32 residual stream [layers, tokens, hidden] that prefill steps of ``tokens``
+        tokens write from now on (read it after ``synchronize()``); None turns it off."""
+        out = None
+        if tokens is not None:
+            out = torch.zeros(len(self.model_config.layers), tokens, self.model_config.hidden_size)
+        call("b200_engine_trace_residual", self._h, out.data_ptr() if out is not None else None)
+        self._trace = out
         return out
 
     def set_profiling(self, on: bool) -> None:

@@ -586,6 +586,42 @@ class HostBatcher:
     def pages_held(self, req: Req) -> int:
         return self._held.get(req.table_idx, 0)
 
+    # ---- requests fed token by token ------------------------------------------
+    def open_request(self, max_len: int) -> Req:
+        """A request whose tokens arrive later, in portions (``extend``), up to ``max_len`` of them."""
+        row = self.table_manager.allocate()
+        self._next_uid += 1
+        self._held[row] = 0
+        return Req(np.zeros(0, np.int32), row, 0, 0, max_len, self._next_uid, False,
+                   CacheHandle(0, self.cache_manager.prefix_cache.root))
+
+    def extend(self, reqs, portions):
+        """One step that runs ``portions[i]`` as the next tokens of ``reqs[i]``: portions of prompts and
+        single tokens in one batch.  (A step of single tokens only runs as a decode step.)  Nothing is
+        written back; read the logits with ``Engine.token_logits`` or ``Engine.logits``."""
+        decode = all(len(t) == 1 and r.cached_len > 0 for r, t in zip(reqs, portions))
+        for r, toks in zip(reqs, portions):
+            if not 0 < len(toks) <= r.max_device_len - r.cached_len:
+                raise ValueError(f"extend: {len(toks)} tokens for a request that can take "
+                                 f"{r.max_device_len - r.cached_len} more")
+            toks = np.asarray(toks, dtype=np.int32)
+            at = np.arange(r.cached_len, r.cached_len + len(toks), dtype=np.int32)
+            self.tables.write_tokens(np.full(len(toks), r.table_idx, np.int32), at, toks)
+            r.input_ids = np.concatenate([r.input_ids, toks])
+            r.device_len = r.cached_len + len(toks)
+        self.allocate(reqs)
+        out = self.engine.forward_batch(1 if decode else 0, [r.table_idx for r in reqs], [r.cached_len for r in reqs],
+                                        [r.extend_len() for r in reqs], write_pos=[-1] * len(reqs))
+        for r in reqs:
+            r.cached_len = r.device_len
+        return out
+
+    def release(self, req: Req) -> None:
+        """Give back what a finished request holds (its table row; its pages, or to the prefix cache)."""
+        self.cache_manager.cache_req(req, finished=True)
+        self.table_manager.free(req.table_idx)
+        self._held.pop(req.table_idx, None)
+
     # ---- steps --------------------------------------------------------------
     def prefill(self, reqs, chunk_tokens: Optional[int] = None, sampling: Optional[dict] = None):
         """One prefill step over `reqs` (each runs positions [cached_len, device_len)).

@@ -7,7 +7,10 @@ of gate/up into ``gate_up_proj`` (:27-41, 62-120) and the stacking of per-expert
 ``tp.shard_layer`` when the engine uploads (``Engine.load_weights``).  Pure torch / numpy, no CUDA.
 
 Not restated: the FP8 block-quantised checkpoints the reference dequantises at load (:213-234);
-only BF16 / F16 / F32 tensors are accepted.
+only BF16 / F16 / F32 and I32 (index tables) tensors are accepted.
+
+Models whose layers are listed one by one (``models.StackConfig``) have a packing of their own,
+``pack_layer_stack``: the layouts of ``b200_engine_create_stack``, zero-padded.
 """
 from __future__ import annotations
 
@@ -19,7 +22,7 @@ from pathlib import Path
 import numpy as np
 import torch
 
-_DTYPES = {"BF16": (torch.bfloat16, 2), "F16": (torch.float16, 2), "F32": (torch.float32, 4)}
+_DTYPES = {"BF16": (torch.bfloat16, 2), "F16": (torch.float16, 2), "F32": (torch.float32, 4), "I32": (torch.int32, 4)}
 _EXPERT = re.compile(r"^(.*\.experts)\.(\d+)\.(.+)$")
 
 
@@ -50,7 +53,7 @@ def read_safetensors(path) -> dict:
 
 
 def write_safetensors(path, tensors: dict) -> None:
-    """The inverse of read_safetensors (tests and tools; BF16 / F16 / F32 only)."""
+    """The inverse of read_safetensors (tests and tools; the same dtypes)."""
     names = {v[0]: k for k, v in _DTYPES.items()}
     header, blobs, off = {}, [], 0
     for name, t in tensors.items():
@@ -153,13 +156,75 @@ def unpack_checkpoint(cfg, w: dict) -> dict:
     return out
 
 
+def pack_layer_stack(cfg, tensors: dict) -> dict:
+    """Rapizen parameter names -> the padded layouts of ``b200_engine_create_stack``, in the dtype the
+    model runs in.  Every tensor is checked against the shape its layer's description asks for."""
+    from ._lib import MLP_DENSE, MLP_NONE, load
+
+    lib = load()
+    width, head, latent = lib.b200_pad_width, lib.b200_pad_head_dim, lib.b200_pad_latent
+    D, V = cfg.hidden_size, cfg.vocab_size
+    hp = width(D)
+
+    def need(name, *shape, dtype=None):
+        if name not in tensors:
+            raise KeyError(f"checkpoint has no tensor {name}")
+        t = tensors[name]
+        if tuple(t.shape) != shape:
+            raise ValueError(f"{name} has shape {tuple(t.shape)}, expected {shape}")
+        return t.to(dtype or cfg.torch_dtype)
+
+    def pad(t, *shape):
+        out = torch.zeros(shape, dtype=t.dtype)
+        out[tuple(slice(0, n) for n in t.shape)] = t
+        return out
+
+    w = {"embed": pad(need("embed", V, D), width(V), hp), "final_norm": pad(need("final.norm", D), hp), "layers": []}
+    if not cfg.tie_word_embeddings:
+        w["lm_head"] = pad(need("head", V, D), width(V), hp)
+    for i, c in enumerate(cfg.layers):
+        p, m = f"l{i}.", f"l{i}.mix."
+        H, d, dv, qr, kr = c.heads, c.head_dim, c.value_dim, c.q_rank, c.kv_rank
+        dp, vp, qp, rp = head(d), head(dv), width(qr), latent(kr)
+        uk = pad(need(m + "uk", H * d, kr).view(H, d, kr), H, dp, rp)
+        L = {"norm1": pad(need(p + "norm1", D), hp),
+             "down_qkv": torch.cat([pad(need(m + "dq", qr, D), qp, hp), pad(need(m + "dkv", kr, D), rp, hp)]),
+             "q_latent_norm": pad(need(m + "dq.norm", qr), qp),
+             "kv_latent_norm": pad(need(m + "dkv.norm", kr), rp),
+             "uq": pad(need(m + "uq", H * d, qr).view(H, d, qr), H, dp, qp),
+             "uk_absorb": uk.transpose(1, 2).contiguous(),
+             "uv": pad(need(m + "uv", H * dv, kr).view(H, dv, kr), H, vp, rp),
+             "o": pad(need(m + "o", D, H * dv).view(D, H, dv), hp, H, vp)}
+        if cfg.expands_keys(c):
+            L["uk"] = uk
+        if c.mlp != MLP_NONE:
+            f, I = p + "mlp.", c.intermediate
+            ip = width(I)
+            L["norm2"] = pad(need(p + "norm2", D), hp)
+            if c.mlp == MLP_DENSE:
+                L["mlp_up"] = torch.cat([pad(need(f + "gate", I, D), ip, hp), pad(need(f + "up", I, D), ip, hp)])
+                L["mlp_down"] = pad(need(f + "down", D, I), hp, ip)
+            else:
+                experts = [f"{f}e{e}." for e in range(c.num_experts)]
+                L["mlp_up"] = torch.stack([pad(need(e + "up", I, D), ip, hp) for e in experts])
+                L["mlp_down"] = torch.stack([pad(need(e + "down", D, I), hp, ip) for e in experts])
+                table = need(f + "table", V, c.experts_per_tok, dtype=torch.int32)
+                if int(table.min()) < 0 or int(table.max()) >= c.num_experts:
+                    raise ValueError(f"{f}table names an expert outside [0, {c.num_experts})")
+                L["expert_table"] = table.contiguous()
+        w["layers"].append(L)
+    return w
+
+
 def load_checkpoint(cfg, directory) -> dict:
-    """All ``*.safetensors`` shards of a directory, packed."""
+    """All ``*.safetensors`` shards of a directory, packed for the kind of model ``cfg`` describes."""
     tensors = {}
     for f in sorted(Path(directory).glob("*.safetensors")):
         tensors.update(read_safetensors(f))
     if not tensors:
         raise FileNotFoundError(f"no .safetensors files under {directory}")
+    if getattr(cfg, "layers", None) is not None:
+        return pack_layer_stack(cfg, tensors)
     return pack_checkpoint(cfg, tensors)
 
 
