@@ -284,8 +284,7 @@ int enqueue_stack_forward(b200_engine* e, int phase, int B, int Bp, int T, bool 
     } pdl_scope;
     set_pdl_launches(false);   // the first kernel follows a copy
     B200_TRY(enqueue_prepare(e, Bp, T));
-    set_pdl_launches(e->use_pdl && !e->trace_residual && !(e->profile_attention && !e->capturing));
-    B200_TRY(layer_stack_enqueue(e, phase, Bp, T));
+    B200_TRY(layer_stack_enqueue(e, phase, Bp, T, e->use_pdl && !e->trace_residual && !(e->profile_attention && !e->capturing)));
     B200_TRY(enqueue_output(e, phase, B, Bp, sampling, step_index));
     e->launches_last_step = static_cast<int>(kernel_launch_count() - launches_before);
     return B200_OK;

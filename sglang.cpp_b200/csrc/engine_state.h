@@ -172,8 +172,9 @@ void layer_stack_destroy(b200_engine* e);
 // Decides, on the host, which requests of a prefill step attend in the latent space and which through
 // expanded keys and values, and stages that plan behind the step's metadata copy.
 int layer_stack_plan(b200_engine* e, const b200_step* st, int phase, int Bp, int T);
-// The layers on `T` tokens; leaves the final-norm output in stack_hidden().
-int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T);
+// The layers on `T` tokens, as programmatic dependent launches if `pdl`; leaves the final-norm output in
+// stack_hidden().
+int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl);
 // `count` rows of hidden states -> logits [count, stack_logits_ld].
 int layer_stack_head(b200_engine* e, void* logits, const void* rows, int count);
 int stack_dtype(const b200_engine* e);

@@ -167,6 +167,9 @@ struct LatentAttention {
     const int32_t* row_len = nullptr;     // keys it sees
     int rows = 0, heads = 0, width = 0, page_size = 1;
     float scale = 1.f;
+    // Only key row_len[i] - 1 of row i was written by kernels that may still be running when this one
+    // starts (a decode step), and the tables and lengths are complete: the rest is read ahead of them.
+    bool only_last_key_new = false;
     void* workspace = nullptr;
     int64_t workspace_bytes = 0;
 };

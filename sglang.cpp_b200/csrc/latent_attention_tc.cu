@@ -58,6 +58,8 @@ struct LatentParams {
     int kpc;                    // keys per TMA copy
     int64_t num_slots;
     float scale_log2;
+    int early;                  // only the last key of a row is new in this step: everything else may be read
+                                // ahead of the previous kernel's completion
     int* status;
 };
 
@@ -178,6 +180,10 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
     const uint32_t smem_base = (smem_u32(smem_raw) + 1023u) & ~1023u;
     const uint32_t q_base = smem_base + static_cast<uint32_t>(p.ring) * kUnitBytes;
     const uint32_t p_base = q_base + static_cast<uint32_t>(N) * static_cast<uint32_t>(p.width) * 2u;
+    const uint32_t stage_off = p_base + 2u * N * 128u - smem_u32(smem_raw);   // output staging [16][128] fp32
+    // The weights are the B operand of the second product: keys contiguous (one 2-byte store per head), or for
+    // a full 64 heads heads contiguous, so that a thread stores its key's row in 16-byte pieces.
+    constexpr bool kHeadsContiguous = N == 64;
 
     pdl_launch_dependents();
     if (threadIdx.x == 0) {
@@ -202,7 +208,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
         tmem_alloc(smem_u32(&tmem_base_slot), 512);
         tmem_relinquish();
     }
-    pdl_wait_prior();
+    if (!p.early) pdl_wait_prior();
 
     // ---- where this CTA's run starts: a scan of the rows' tile counts ----
     {
@@ -258,29 +264,49 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
     if (warp == 0) {
         // ================= producer =================
         const int copies = kTileKeys / p.kpc;
-        int unit = 0, nseg = 0;
-        while (!failed && next_segment(walk, p, seg)) {
-            const int32_t* pt = p.page_table + static_cast<int64_t>(p.row_table[seg.row]) * p.pt_stride;
-            for (int t = seg.t0; t < seg.t1 && !failed; ++t) {
-                // the slots of this tile's pages; a copy past the last key reads a row outside the tensor,
-                // which the copy engine fills with zeros
-                int sl[4];
+        int ring_at = 0, unit = 0, nseg = 0;
+        uint32_t ring_parity = 1;          // of the slot's previous use
+        bool waited = !p.early;
+        // The slots of a tile's pages; a copy past the last key reads a row outside the tensor, which the
+        // copy engine fills with zeros.
+        auto slots_of = [&](const Segment& g, int t, int (&sl)[4]) {
+            const int32_t* pt = p.page_table + static_cast<int64_t>(p.row_table[g.row]) * p.pt_stride;
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    const int copy = i * 32 + lane, key = t * kTileKeys + copy * p.kpc;
-                    sl[i] = static_cast<int>(p.num_slots);
-                    if (copy < copies && key < seg.len) {
-                        const int64_t v = pt[key];
-                        if (v < 0 || v + p.kpc > p.num_slots)
-                            atomicExch(&p.status[kStatusBadIndex], static_cast<int>(v) + 1);
-                        else
-                            sl[i] = static_cast<int>(v);
-                    }
+            for (int i = 0; i < 4; ++i) {
+                const int copy = i * 32 + lane, key = t * kTileKeys + copy * p.kpc;
+                sl[i] = static_cast<int>(p.num_slots);
+                if (copy < copies && key < g.len) {
+                    const int64_t v = pt[key];
+                    if (v < 0 || v + p.kpc > p.num_slots)
+                        atomicExch(&p.status[kStatusBadIndex], static_cast<int>(v) + 1);
+                    else
+                        sl[i] = static_cast<int>(v);
                 }
-                for (int u = 0; u < p.nb && !failed; ++u, ++unit) {
-                    const int s = unit % p.ring;
-                    const bool ok = unit < p.ring || mbar_wait_bounded(smem_u32(&unit_empty[s]),
-                                                                       static_cast<uint32_t>(unit / p.ring - 1) & 1u, p.status, 601);
+            }
+        };
+        // one tile ahead: the slots of the next tile are looked up before this one waits for the ring
+        int sl[4], sl_next[4];
+        bool have = next_segment(walk, p, seg);
+        if (have) slots_of(seg, seg.t0, sl_next);
+        while (have && !failed) {
+            Segment upcoming = seg;
+            bool more = false;
+            for (int t = seg.t0; t < seg.t1 && !failed; ++t) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) sl[i] = sl_next[i];
+                if (t + 1 < seg.t1) {
+                    slots_of(seg, t + 1, sl_next);
+                } else {
+                    more = next_segment(walk, p, upcoming);
+                    if (more) slots_of(upcoming, upcoming.t0, sl_next);
+                }
+                if (!waited && (t + 1) * kTileKeys >= seg.len) {   // this tile holds the newest key
+                    pdl_wait_prior();
+                    waited = true;
+                }
+                for (int u = 0; u < p.nb; ++u, ++unit) {
+                    const int s = ring_at;
+                    const bool ok = unit < p.ring || mbar_wait_bounded(smem_u32(&unit_empty[s]), ring_parity, p.status, 601);
                     if (!__all_sync(0xffffffffu, ok)) {
                         failed = true;
                         break;
@@ -298,9 +324,17 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                             tma_load_2d(to + kAtomBytes, &tmap_c, u * kUnitElems + 64, sl[i], bar);
                         }
                     }
+                    if (++ring_at == p.ring) {
+                        ring_at = 0;
+                        ring_parity ^= 1u;
+                    }
                 }
                 if (t == seg.t0 && !failed) {
                     // the queries of this item, behind the first tile's latents
+                    if (!waited) {
+                        pdl_wait_prior();
+                        waited = true;
+                    }
                     const bool ok = nseg == 0 || mbar_wait_bounded(smem_u32(&q_empty), static_cast<uint32_t>(nseg - 1) & 1u,
                                                                    p.status, 602);
                     if (!__all_sync(0xffffffffu, ok)) {
@@ -316,22 +350,33 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                 }
             }
             ++nseg;
+            have = more;
+            seg = upcoming;
         }
+        if (!waited) pdl_wait_prior();
     } else if (warp == 1) {
         // ================= MMA issuer =================
+        pdl_wait_prior();
         if (lane == 0) {
             const uint32_t idesc_s = idesc_bf16_m128(N);
-            const uint32_t idesc_o = idesc_bf16_m128(N) | (1u << 15);   // A is MN-major
+            // A is MN-major; B is too where the heads of a key are contiguous
+            const uint32_t idesc_o = idesc_bf16_m128(N) | (1u << 15) | (kHeadsContiguous ? 1u << 16 : 0u);
             int unit = 0;    // first unit of the tile whose S^T is being issued
             int tiles = 0;   // tiles whose P has been consumed
             int nseg = 0;
-            // units [u0, u1) of S^T for the tile that starts at unit `first`, into buffer `buf`
-            auto issue_s = [&](int first, int u0, int u1, int buf) {
-                for (int u = u0; u < u1; ++u) {
+            // Units [u0, u1) of S^T for the tile that starts at unit `first`, into buffer `buf`.  Without
+            // `block` it stops at the first unit that has not arrived.  Returns how far it got.
+            auto issue_s = [&](int first, int u0, int u1, int buf, bool block) -> int {
+                int u = u0;
+                for (; u < u1; ++u) {
                     const int n = first + u, s = n % p.ring;
-                    if (!mbar_wait_bounded(smem_u32(&unit_full[s]), static_cast<uint32_t>(n / p.ring) & 1u, p.status, 603)) {
-                        failed = true;
-                        return;
+                    const uint32_t bar = smem_u32(&unit_full[s]), parity = static_cast<uint32_t>(n / p.ring) & 1u;
+                    if (!mbar_try_wait(bar, parity)) {
+                        if (!block) break;
+                        if (!mbar_wait_bounded(bar, parity, p.status, 603)) {
+                            failed = true;
+                            return u;
+                        }
                     }
                     tc_fence_after();
                     const uint32_t a = smem_base + static_cast<uint32_t>(s) * kUnitBytes;
@@ -343,7 +388,8 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                                     kmajor_sw128_desc(b + (ks >> 2) * N * 128u + (ks & 3) * 32), idesc_s,
                                     (u > 0 || ks > 0) ? 1u : 0u);
                 }
-                if (u1 == p.nb) tc_commit(smem_u32(&s_full[buf]));
+                if (u == p.nb && u > u0) tc_commit(smem_u32(&s_full[buf]));
+                return u;
             };
             while (!failed && next_segment(walk, p, seg)) {
                 if (!mbar_wait_bounded(smem_u32(&q_full), static_cast<uint32_t>(nseg) & 1u, p.status, 604)) {
@@ -351,14 +397,13 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                     break;
                 }
                 tc_fence_after();
-                issue_s(unit, 0, p.nb, tiles & 1);
+                issue_s(unit, 0, p.nb, tiles & 1, true);
                 for (int t = seg.t0; t < seg.t1 && !failed; ++t) {
                     const int cur = unit;
                     unit += p.nb;
                     const bool more = t + 1 < seg.t1;
-                    // as much of the next tile's S^T as the ring can hold beside the current tile
-                    const int ahead = min(p.nb, p.ring - p.nb);
-                    if (more && ahead > 0) issue_s(unit, 0, ahead, (tiles + 1) & 1);
+                    // as much of the next tile's S^T as has already arrived
+                    const int ahead = more ? issue_s(unit, 0, min(p.nb, p.ring - p.nb), (tiles + 1) & 1, false) : 0;
                     if (!more) tc_commit(smem_u32(&q_empty));   // every S^T of this item has been issued
                     if (failed || !mbar_wait_bounded(smem_u32(&p_full), static_cast<uint32_t>(tiles) & 1u, p.status, 605)) {
                         failed = true;
@@ -377,12 +422,14 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
 #pragma unroll
                         for (int ks = 0; ks < 8; ++ks)
                             tc_mma_bf16(d, mnmajor_desc(a + ks * 2048),
-                                        kmajor_sw128_desc(p_base + (ks >> 2) * N * 128u + (ks & 3) * 32), idesc_o,
+                                        kHeadsContiguous ? mnmajor_desc(p_base + ks * 2048)
+                                                         : kmajor_sw128_desc(p_base + (ks >> 2) * N * 128u + (ks & 3) * 32),
+                                        idesc_o,
                                         (t > seg.t0 || ks > 0) ? 1u : 0u);
                         tc_commit(smem_u32(&unit_empty[s]));
                     }
                     tc_commit(smem_u32(&pv_done));
-                    if (more && ahead < p.nb) issue_s(unit, ahead, p.nb, (tiles + 1) & 1);
+                    if (more && ahead < p.nb) issue_s(unit, ahead, p.nb, (tiles + 1) & 1, true);
                     ++tiles;
                 }
                 ++nseg;
@@ -396,8 +443,10 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
         const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(q * 32) << 16);
         const uint32_t p_key = p_base + static_cast<uint32_t>(key >> 6) * N * 128u + static_cast<uint32_t>(key & 7) * 2u;
         const uint32_t p_chunk = static_cast<uint32_t>((key & 63) >> 3);
+        float* stage = reinterpret_cast<float*>(smem_raw + stage_off);
         int tiles = 0;
         float l[N];
+        pdl_wait_prior();
         while (!failed && next_segment(walk, p, seg)) {
 #pragma unroll
             for (int h = 0; h < N; ++h) l[h] = 0.f;
@@ -417,8 +466,13 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                     tmem_ld_32x32b_x16(s_addr + c * 16, sv);
                     tmem_ld_wait();
 #pragma unroll
-                    for (int j = 0; j < 16; ++j)
-                        over |= __uint_as_float(sv[j]) * p.scale_log2 > s_ref[c * 16 + j] + kLazyLog2;
+                    for (int j = 0; j < 16; j += 4) {
+                        const float4 ref = *reinterpret_cast<const float4*>(&s_ref[c * 16 + j]);
+                        over |= __uint_as_float(sv[j]) * p.scale_log2 > ref.x + kLazyLog2;
+                        over |= __uint_as_float(sv[j + 1]) * p.scale_log2 > ref.y + kLazyLog2;
+                        over |= __uint_as_float(sv[j + 2]) * p.scale_log2 > ref.z + kLazyLog2;
+                        over |= __uint_as_float(sv[j + 3]) * p.scale_log2 > ref.w + kLazyLog2;
+                    }
                 }
                 // the previous product has read P and written O before either is touched again
                 if (t > seg.t0 && !failed &&
@@ -476,15 +530,39 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                     uint32_t sv[16];
                     tmem_ld_32x32b_x16(s_addr + c * 16, sv);
                     tmem_ld_wait();
+                    float w[16];
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) {
-                        const int h = c * 16 + j;
-                        const float w = valid ? ex2(fmaf(__uint_as_float(sv[j]), p.scale_log2, -s_ref[h])) : 0.f;
-                        l[h] += w;
-                        const __nv_bfloat16 b = __float2bfloat16_rn(w);
-                        const uint32_t addr = p_key + static_cast<uint32_t>(h) * 128u + ((p_chunk ^ (h & 7)) << 4);
-                        asm volatile("st.shared.b16 [%0], %1;" ::"r"(addr), "h"(*reinterpret_cast<const uint16_t*>(&b))
-                                     : "memory");
+                    for (int j = 0; j < 16; j += 4) {
+                        const float4 ref = *reinterpret_cast<const float4*>(&s_ref[c * 16 + j]);
+                        w[j] = ex2(fmaf(__uint_as_float(sv[j]), p.scale_log2, -ref.x));
+                        w[j + 1] = ex2(fmaf(__uint_as_float(sv[j + 1]), p.scale_log2, -ref.y));
+                        w[j + 2] = ex2(fmaf(__uint_as_float(sv[j + 2]), p.scale_log2, -ref.z));
+                        w[j + 3] = ex2(fmaf(__uint_as_float(sv[j + 3]), p.scale_log2, -ref.w));
+                    }
+                    if (!valid) {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) w[j] = 0.f;
+                    }
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) l[c * 16 + j] += w[j];
+                    if (kHeadsContiguous) {
+#pragma unroll
+                        for (int j = 0; j < 16; j += 8) {
+                            const uint32_t addr = swz128(p_base + static_cast<uint32_t>(key) * 128u, c * 2 + j / 8);
+                            asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(addr), "r"(pack_bf16(w[j], w[j + 1])),
+                                         "r"(pack_bf16(w[j + 2], w[j + 3])), "r"(pack_bf16(w[j + 4], w[j + 5])),
+                                         "r"(pack_bf16(w[j + 6], w[j + 7]))
+                                         : "memory");
+                        }
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) {
+                            const int h = c * 16 + j;
+                            const __nv_bfloat16 b = __float2bfloat16_rn(w[j]);
+                            const uint32_t addr = p_key + static_cast<uint32_t>(h) * 128u + ((p_chunk ^ (h & 7)) << 4);
+                            asm volatile("st.shared.b16 [%0], %1;" ::"r"(addr), "h"(*reinterpret_cast<const uint16_t*>(&b))
+                                         : "memory");
+                        }
                     }
                 }
                 fence_proxy_async_smem();
@@ -528,24 +606,38 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
             const int h0 = seg.block * p.per_block;
             const int nh = min(p.per_block, p.heads - h0);
             for (int u = 0; u < p.nb; ++u) {
-                const int e = u * kUnitElems + key;
 #pragma unroll
                 for (int c = 0; c < N / 16; ++c) {
+                    if (c * 16 >= nh) break;
                     uint32_t ov[16];
                     tmem_ld_32x32b_x16(lane_addr + kColO + static_cast<uint32_t>(u * N + c * 16), ov);
                     tmem_ld_wait();
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) {
-                        const int h = c * 16 + j;
-                        if (h < nh) {
-                            const float v = __uint_as_float(ov[j]);
-                            if (whole)
-                                p.out[(static_cast<int64_t>(seg.row) * p.heads + h0 + h) * p.width + e] =
-                                    __float2bfloat16_rn(v * s_alpha[h]);
-                            else
-                                p.part_o[(slot * N + h) * p.width + e] = v;
+                    for (int j = 0; j < 16; ++j) stage[j * kUnitElems + key] = __uint_as_float(ov[j]) * s_alpha[c * 16 + j];
+                    softmax_sync();
+                    // 16 heads x 128 elements, whole rows of a head at a time
+                    if (whole) {
+#pragma unroll
+                        for (int i = st; i < 16 * kUnitElems / 8; i += 128) {
+                            const int h = c * 16 + i / (kUnitElems / 8), e = i % (kUnitElems / 8) * 8;
+                            if (h < nh) {
+                                const float* v = stage + (i / (kUnitElems / 8)) * kUnitElems + e;
+                                const float4 a = *reinterpret_cast<const float4*>(v), b = *reinterpret_cast<const float4*>(v + 4);
+                                *reinterpret_cast<uint4*>(p.out + (static_cast<int64_t>(seg.row) * p.heads + h0 + h) * p.width +
+                                                          u * kUnitElems + e) =
+                                    make_uint4(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w), pack_bf16(b.x, b.y), pack_bf16(b.z, b.w));
+                            }
+                        }
+                    } else {
+#pragma unroll
+                        for (int i = st; i < 16 * kUnitElems / 4; i += 128) {
+                            const int h = c * 16 + i / (kUnitElems / 4), e = i % (kUnitElems / 4) * 4;
+                            if (h < nh)
+                                *reinterpret_cast<float4*>(p.part_o + (slot * N + h) * p.width + u * kUnitElems + e) =
+                                    *reinterpret_cast<const float4*>(stage + (i / (kUnitElems / 4)) * kUnitElems + e);
                         }
                     }
+                    softmax_sync();
                 }
             }
             tc_fence_before();
@@ -580,6 +672,7 @@ latent_merge_kernel(const LatentParams p, int N) {
     float tot = 0.f;
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
     const int e = static_cast<int>(threadIdx.x) * 4;
+#pragma unroll 4
     for (int c = c0; c <= c1; ++c) {
         const int64_t s = slot_of(c);
         const float f = ex2(p.part_m[s] - mx);
@@ -651,10 +744,11 @@ int launch_latent_attention_tc(const LatentAttention& a, int* status, cudaStream
     p.kpc = a.page_size < kTileKeys ? a.page_size : kTileKeys;
     p.num_slots = a.num_slots;
     p.scale_log2 = a.scale * 1.4426950408889634f;
+    p.early = a.only_last_key_new && pdl_launches_enabled() ? 1 : 0;
     p.status = status;
-    const uint32_t fixed = static_cast<uint32_t>(sh.n) * a.width * 2u + 2u * sh.n * 128u + 1024u;
+    const uint32_t fixed = static_cast<uint32_t>(sh.n) * a.width * 2u + 2u * sh.n * 128u + 16u * kUnitElems * 4u + 1024u;
     int ring = kMaxUnits;
-    while (ring > p.nb && static_cast<uint32_t>(ring) * kUnitBytes + fixed > 220u * 1024u) --ring;
+    while (ring > p.nb && static_cast<uint32_t>(ring) * kUnitBytes + fixed > 224u * 1024u) --ring;
     p.ring = ring;
     const uint32_t smem = static_cast<uint32_t>(ring) * kUnitBytes + fixed;
 

@@ -346,7 +346,7 @@ int project_experts(b200_engine* e, void* y, const void* x, const void* w, const
 
 // Latent-space attention of `rows` query rows (q and out [rows, heads * dim], tables per row).
 int attend_latent(b200_engine* e, const StackLayer& L, void* out, const void* q, const int32_t* row_table,
-                  const int32_t* row_len, int rows) {
+                  const int32_t* row_len, int rows, bool decode) {
     LayerStack* S = e->stack;
     const int H = L.c.heads;
     for (int r0 = 0; r0 < rows; r0 += S->latent_rows) {
@@ -368,6 +368,7 @@ int attend_latent(b200_engine* e, const StackLayer& L, void* out, const void* q,
         a.width = L.rp;
         a.page_size = e->c.page_size;
         a.scale = L.c.score_scale;
+        a.only_last_key_new = decode;
         a.workspace = S->ws;
         a.workspace_bytes = S->ws_bytes;
         if (S->dtype == B200_DTYPE_BF16 && latent_attention_tc_supported(a))
@@ -382,7 +383,7 @@ int attend_latent(b200_engine* e, const StackLayer& L, void* out, const void* q,
 int attend(b200_engine* e, const StackLayer& L, int phase, int Bp, int T) {
     LayerStack* S = e->stack;
     if (phase == B200_PHASE_DECODE || S->plan_expanded == 0 || !L.can_expand)
-        return attend_latent(e, L, S->attn, S->q, S->token_row, S->token_len, T);
+        return attend_latent(e, L, S->attn, S->q, S->token_row, S->token_len, T, phase == B200_PHASE_DECODE);
     const int H = L.c.heads;
     const int32_t* x_len = S->plan_dev;
     const int32_t* x_base = x_len + Bp;
@@ -403,14 +404,14 @@ int attend(b200_engine* e, const StackLayer& L, int phase, int Bp, int T) {
     const int n = S->plan_latent;
     if (n == 0) return B200_OK;
     S_TRY(launch_move_rows(S->qc, S->q, tokens, n, H * L.dp / 8, false, e->stream));
-    S_TRY(attend_latent(e, L, S->ac, S->qc, S->compact_row, S->compact_len, n));
+    S_TRY(attend_latent(e, L, S->ac, S->qc, S->compact_row, S->compact_len, n, false));
     return launch_move_rows(S->attn, S->ac, tokens, n, H * L.vp / 8, true, e->stream);
     (void)T;
 }
 
 }  // namespace
 
-int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T) {
+int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
     LayerStack* S = e->stack;
     cudaStream_t s = e->stream;
     const int hp = S->hp, width = e->m.hidden_size;
@@ -462,7 +463,10 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T) {
     for (int l = 0; l < num_layers; ++l) {
         const StackLayer& L = S->layers[l];
         const b200_layer_config& c = L.c;
+        // The first norm is launched as an ordinary dependent of what prepares the step, so that every
+        // kernel after it finds positions, slots and lengths complete even ahead of its own wait.
         S_TRY(norm_to(L.norm1, S->x, nullptr, 1, 1.f));
+        if (l == 0) set_pdl_launches(pdl);
         S_TRY(traced(l));
         S_TRY(project(e, S->joint, S->x, L.down_qkv, T, L.qp + L.rp, hp, B200_EPILOGUE_NONE));
         S_TRY(launch_latent_norm_store(S->cq, L.cache, S->joint, L.q_norm, L.kv_norm, e->out_loc, T, c.q_rank, L.qp,
