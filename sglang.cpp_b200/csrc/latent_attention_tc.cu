@@ -20,7 +20,9 @@
 // runs, one per CTA (one CTA per SM).  An item that spans CTAs leaves fp32 partials, combined by the merge
 // kernel.  No host plan: lengths are read from device memory, so a captured graph replays at any lengths.
 //
-// Roles: warp 0 producer, warp 1 one thread issues every MMA, warps 2-5 softmax and output.
+// Roles: warp 0 producer, warp 1 issues S^T, warps 2-5 softmax and output, warp 6 issues O^T.  S^T and (where
+// shared memory allows) P are double-buffered, so the two products and the softmax of neighbouring tiles
+// overlap.
 #include <math.h>
 
 #include "common.cuh"
@@ -36,10 +38,11 @@ constexpr int kUnitElems = 128;                            // latent elements pe
 constexpr uint32_t kAtomBytes = kTileKeys * 128;           // 128 keys x 64 elements, 128-byte rows
 constexpr uint32_t kUnitBytes = 2 * kAtomBytes;
 constexpr int kMaxUnits = 6;                               // units in the ring
-constexpr int kThreads = 192;
+constexpr int kThreads = 224;
 constexpr int kMaxWidth = 512;
 constexpr uint32_t kColO = 0, kColS = 256;                 // TMEM columns: O^T (4 x 64), S^T (2 x 64)
 constexpr float kLazyLog2 = 8.0f;
+constexpr int kLens = 64;
 
 struct LatentParams {
     __nv_bfloat16* out;         // [rows, heads, width]
@@ -55,6 +58,7 @@ struct LatentParams {
     int blocks, per_block;      // head blocks per row, heads per block (<= N)
     int nb;                     // units per tile
     int ring;                   // units in the ring (>= nb)
+    int p_bufs;                 // buffers of P, 1 or 2
     int kpc;                    // keys per TMA copy
     int64_t num_slots;
     float scale_log2;
@@ -129,6 +133,8 @@ __device__ __forceinline__ int warp_transpose_sum(float (&v)[N]) {
 struct Walk {
     int row, block, tile;   // current item and first tile of it that belongs to this CTA
     int left;               // tiles this CTA still has to do
+    int row0;               // first row of the run: the lengths of the next kLens rows are in shared memory
+    const int* lens;
 };
 struct Segment {
     int row, block, t0, t1, len;   // tiles [t0, t1) of an item whose row has len keys
@@ -136,12 +142,13 @@ struct Segment {
 };
 __device__ __forceinline__ bool next_segment(Walk& w, const LatentParams& p, Segment& s) {
     if (w.left <= 0) return false;
-    int len = p.row_len[w.row];
+    auto len_of = [&](int row) { return row - w.row0 < kLens ? w.lens[row - w.row0] : p.row_len[row]; };
+    int len = len_of(w.row);
     while (len <= 0) {   // rows without keys own no tile
         ++w.row;
         w.block = 0;
         if (w.row >= p.rows) return false;
-        len = p.row_len[w.row];
+        len = len_of(w.row);
     }
     const int nt = (len + kTileKeys - 1) / kTileKeys;
     s.row = w.row;
@@ -167,7 +174,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t unit_full[kMaxUnits];
     __shared__ __align__(8) uint64_t unit_empty[kMaxUnits];
-    __shared__ __align__(8) uint64_t q_full, q_empty, s_full[2], p_full, pv_done, o_free;
+    __shared__ __align__(8) uint64_t q_full, q_empty, s_full[2], s_empty[2], p_full[2], pv_done[2], o_free;
     __shared__ uint32_t tmem_base_slot;
     __shared__ int s_scan[kThreads / 32 + 1];
     __shared__ int s_total, s_row, s_block, s_tile;
@@ -175,12 +182,14 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
     __shared__ __align__(16) float s_alpha[N];
     __shared__ float s_warp[4][N];
     __shared__ volatile int s_failed[2];
+    __shared__ int s_len[kLens];
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t smem_base = (smem_u32(smem_raw) + 1023u) & ~1023u;
     const uint32_t q_base = smem_base + static_cast<uint32_t>(p.ring) * kUnitBytes;
     const uint32_t p_base = q_base + static_cast<uint32_t>(N) * static_cast<uint32_t>(p.width) * 2u;
-    const uint32_t stage_off = p_base + 2u * N * 128u - smem_u32(smem_raw);   // output staging [16][128] fp32
+    constexpr uint32_t kPBytes = 2u * N * 128u;
+    const uint32_t stage_off = p_base + static_cast<uint32_t>(p.p_bufs) * kPBytes - smem_u32(smem_raw);   // output staging [16][128] fp32
     // The weights are the B operand of the second product: keys contiguous (one 2-byte store per head), or for
     // a full 64 heads heads contiguous, so that a thread stores its key's row in 16-byte pieces.
     constexpr bool kHeadsContiguous = N == 64;
@@ -193,10 +202,12 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
         }
         mbar_init(smem_u32(&q_full), 1);
         mbar_init(smem_u32(&q_empty), 1);
-        mbar_init(smem_u32(&s_full[0]), 1);
-        mbar_init(smem_u32(&s_full[1]), 1);
-        mbar_init(smem_u32(&p_full), 4);
-        mbar_init(smem_u32(&pv_done), 1);
+        for (int i = 0; i < 2; ++i) {
+            mbar_init(smem_u32(&s_full[i]), 1);
+            mbar_init(smem_u32(&s_empty[i]), 4);
+            mbar_init(smem_u32(&p_full[i]), 4);
+            mbar_init(smem_u32(&pv_done[i]), 1);
+        }
         mbar_init(smem_u32(&o_free), 4);
         fence_mbar_init();
         tma_prefetch_desc(&tmap_c);
@@ -247,6 +258,9 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
         }
         if (threadIdx.x == 0) s_total = total;
     }
+    __syncthreads();
+    if (threadIdx.x < kLens && s_row + static_cast<int>(threadIdx.x) < p.rows)
+        s_len[threadIdx.x] = p.row_len[s_row + threadIdx.x];
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
@@ -257,6 +271,8 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
     walk.row = s_row;
     walk.block = s_block;
     walk.tile = s_tile;
+    walk.row0 = s_row;
+    walk.lens = s_len;
     walk.left = s_row < p.rows ? min(run, s_total - g0) : 0;
     bool failed = false;
     Segment seg;
@@ -267,15 +283,16 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
         int ring_at = 0, unit = 0, nseg = 0;
         uint32_t ring_parity = 1;          // of the slot's previous use
         bool waited = !p.early;
-        // The slots of a tile's pages; a copy past the last key reads a row outside the tensor, which the
-        // copy engine fills with zeros.
-        auto slots_of = [&](const Segment& g, int t, int (&sl)[4]) {
+        // Page-table look-ups run a group of 128 copies (kpc tiles) ahead of the loads: copy i of a group is
+        // held, and issued, by lane i % 32.  A copy past the last key reads a row outside the tensor, which
+        // the copy engine fills with zeros.
+        auto slots_of = [&](const Segment& g, int t0, int (&sl)[4]) {
             const int32_t* pt = p.page_table + static_cast<int64_t>(p.row_table[g.row]) * p.pt_stride;
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-                const int copy = i * 32 + lane, key = t * kTileKeys + copy * p.kpc;
+                const int key = t0 * kTileKeys + (i * 32 + lane) * p.kpc;
                 sl[i] = static_cast<int>(p.num_slots);
-                if (copy < copies && key < g.len) {
+                if (key < min(g.len, g.t1 * kTileKeys)) {
                     const int64_t v = pt[key];
                     if (v < 0 || v + p.kpc > p.num_slots)
                         atomicExch(&p.status[kStatusBadIndex], static_cast<int>(v) + 1);
@@ -284,7 +301,6 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                 }
             }
         };
-        // one tile ahead: the slots of the next tile are looked up before this one waits for the ring
         int sl[4], sl_next[4];
         bool have = next_segment(walk, p, seg);
         if (have) slots_of(seg, seg.t0, sl_next);
@@ -292,13 +308,16 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
             Segment upcoming = seg;
             bool more = false;
             for (int t = seg.t0; t < seg.t1 && !failed; ++t) {
+                const int in_group = (t - seg.t0) & (p.kpc - 1);
+                if (in_group == 0) {
 #pragma unroll
-                for (int i = 0; i < 4; ++i) sl[i] = sl_next[i];
-                if (t + 1 < seg.t1) {
-                    slots_of(seg, t + 1, sl_next);
-                } else {
-                    more = next_segment(walk, p, upcoming);
-                    if (more) slots_of(upcoming, upcoming.t0, sl_next);
+                    for (int i = 0; i < 4; ++i) sl[i] = sl_next[i];
+                    if (t + p.kpc < seg.t1) {
+                        slots_of(seg, t + p.kpc, sl_next);
+                    } else {
+                        more = next_segment(walk, p, upcoming);
+                        if (more) slots_of(upcoming, upcoming.t0, sl_next);
+                    }
                 }
                 if (!waited && (t + 1) * kTileKeys >= seg.len) {   // this tile holds the newest key
                     pdl_wait_prior();
@@ -317,8 +336,8 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                     __syncwarp();
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
-                        const int copy = i * 32 + lane;
-                        if (copy < copies) {
+                        const int copy = i * 32 + lane - in_group * copies;
+                        if (copy >= 0 && copy < copies) {
                             const uint32_t to = dst + static_cast<uint32_t>(copy * p.kpc) * 128u;
                             tma_load_2d(to, &tmap_c, u * kUnitElems, sl[i], bar);
                             tma_load_2d(to + kAtomBytes, &tmap_c, u * kUnitElems + 64, sl[i], bar);
@@ -355,82 +374,77 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
         }
         if (!waited) pdl_wait_prior();
     } else if (warp == 1) {
-        // ================= MMA issuer =================
+        // ================= S^T = C Q^T =================
         pdl_wait_prior();
-        if (lane == 0) {
-            const uint32_t idesc_s = idesc_bf16_m128(N);
-            // A is MN-major; B is too where the heads of a key are contiguous
-            const uint32_t idesc_o = idesc_bf16_m128(N) | (1u << 15) | (kHeadsContiguous ? 1u << 16 : 0u);
-            int unit = 0;    // first unit of the tile whose S^T is being issued
-            int tiles = 0;   // tiles whose P has been consumed
-            int nseg = 0;
-            // Units [u0, u1) of S^T for the tile that starts at unit `first`, into buffer `buf`.  Without
-            // `block` it stops at the first unit that has not arrived.  Returns how far it got.
-            auto issue_s = [&](int first, int u0, int u1, int buf, bool block) -> int {
-                int u = u0;
-                for (; u < u1; ++u) {
-                    const int n = first + u, s = n % p.ring;
-                    const uint32_t bar = smem_u32(&unit_full[s]), parity = static_cast<uint32_t>(n / p.ring) & 1u;
-                    if (!mbar_try_wait(bar, parity)) {
-                        if (!block) break;
-                        if (!mbar_wait_bounded(bar, parity, p.status, 603)) {
-                            failed = true;
-                            return u;
-                        }
-                    }
-                    tc_fence_after();
-                    const uint32_t a = smem_base + static_cast<uint32_t>(s) * kUnitBytes;
-                    const uint32_t b = q_base + static_cast<uint32_t>(2 * u) * N * 128u;
-                    const uint32_t d = tmem_base + kColS + static_cast<uint32_t>(buf) * 64u;
-#pragma unroll
-                    for (int ks = 0; ks < 8; ++ks)
-                        tc_mma_bf16(d, kmajor_sw128_desc(a + (ks >> 2) * kAtomBytes + (ks & 3) * 32),
-                                    kmajor_sw128_desc(b + (ks >> 2) * N * 128u + (ks & 3) * 32), idesc_s,
-                                    (u > 0 || ks > 0) ? 1u : 0u);
-                }
-                if (u == p.nb && u > u0) tc_commit(smem_u32(&s_full[buf]));
-                return u;
-            };
+        if (elect_one()) {
+            const uint32_t idesc = idesc_bf16_m128(N);
+            int slot = 0, tiles = 0, nseg = 0;
+            uint32_t parity = 0;
             while (!failed && next_segment(walk, p, seg)) {
-                if (!mbar_wait_bounded(smem_u32(&q_full), static_cast<uint32_t>(nseg) & 1u, p.status, 604)) {
-                    failed = true;
-                    break;
-                }
-                tc_fence_after();
-                issue_s(unit, 0, p.nb, tiles & 1, true);
-                for (int t = seg.t0; t < seg.t1 && !failed; ++t) {
-                    const int cur = unit;
-                    unit += p.nb;
-                    const bool more = t + 1 < seg.t1;
-                    // as much of the next tile's S^T as has already arrived
-                    const int ahead = more ? issue_s(unit, 0, min(p.nb, p.ring - p.nb), (tiles + 1) & 1, false) : 0;
-                    if (!more) tc_commit(smem_u32(&q_empty));   // every S^T of this item has been issued
-                    if (failed || !mbar_wait_bounded(smem_u32(&p_full), static_cast<uint32_t>(tiles) & 1u, p.status, 605)) {
+                if (!mbar_wait_bounded(smem_u32(&q_full), static_cast<uint32_t>(nseg) & 1u, p.status, 603)) break;
+                for (int t = seg.t0; t < seg.t1 && !failed; ++t, ++tiles) {
+                    const int buf = tiles & 1;
+                    if (tiles >= 2 && !mbar_wait_bounded(smem_u32(&s_empty[buf]), static_cast<uint32_t>((tiles >> 1) - 1) & 1u,
+                                                         p.status, 604)) {
                         failed = true;
                         break;
                     }
-                    if (t == seg.t0 && nseg > 0 &&
-                        !mbar_wait_bounded(smem_u32(&o_free), static_cast<uint32_t>(nseg - 1) & 1u, p.status, 606)) {
-                        failed = true;
-                        break;
-                    }
-                    tc_fence_after();
+                    const uint32_t d = tmem_base + kColS + static_cast<uint32_t>(buf) * 64u;
+                    uint64_t b = kmajor_sw128_desc(q_base);
                     for (int u = 0; u < p.nb; ++u) {
-                        const int s = (cur + u) % p.ring;
-                        const uint32_t a = smem_base + static_cast<uint32_t>(s) * kUnitBytes;
-                        const uint32_t d = tmem_base + kColO + static_cast<uint32_t>(u * N);
+                        if (!mbar_wait_bounded(smem_u32(&unit_full[slot]), parity, p.status, 605)) {
+                            failed = true;
+                            break;
+                        }
+                        tc_fence_after();
+                        const uint64_t a = kmajor_sw128_desc(smem_base + static_cast<uint32_t>(slot) * kUnitBytes);
 #pragma unroll
                         for (int ks = 0; ks < 8; ++ks)
-                            tc_mma_bf16(d, mnmajor_desc(a + ks * 2048),
-                                        kHeadsContiguous ? mnmajor_desc(p_base + ks * 2048)
-                                                         : kmajor_sw128_desc(p_base + (ks >> 2) * N * 128u + (ks & 3) * 32),
-                                        idesc_o,
-                                        (t > seg.t0 || ks > 0) ? 1u : 0u);
-                        tc_commit(smem_u32(&unit_empty[s]));
+                            tc_mma_bf16(d, a + ((ks >> 2) * kAtomBytes + (ks & 3) * 32) / 16,
+                                        b + ((ks >> 2) * N * 128 + (ks & 3) * 32) / 16, idesc, (u > 0 || ks > 0) ? 1u : 0u);
+                        b += 2 * N * 128 / 16;
+                        if (++slot == p.ring) {
+                            slot = 0;
+                            parity ^= 1u;
+                        }
                     }
-                    tc_commit(smem_u32(&pv_done));
-                    if (more && ahead < p.nb) issue_s(unit, ahead, p.nb, (tiles + 1) & 1, true);
-                    ++tiles;
+                    if (failed) break;
+                    tc_commit(smem_u32(&s_full[buf]));
+                }
+                tc_commit(smem_u32(&q_empty));
+                ++nseg;
+            }
+        }
+    } else if (warp == 6) {
+        // ================= O^T += C^T P^T =================
+        pdl_wait_prior();
+        if (elect_one()) {
+            // A is MN-major; B is too where the heads of a key are contiguous
+            const uint32_t idesc = idesc_bf16_m128(N) | (1u << 15) | (kHeadsContiguous ? 1u << 16 : 0u);
+            int slot = 0, tiles = 0, nseg = 0;
+            while (!failed && next_segment(walk, p, seg)) {
+                for (int t = seg.t0; t < seg.t1; ++t, ++tiles) {
+                    if (!mbar_wait_bounded(smem_u32(&p_full[tiles & 1]), static_cast<uint32_t>(tiles >> 1) & 1u, p.status, 606) ||
+                        (t == seg.t0 && nseg > 0 &&
+                         !mbar_wait_bounded(smem_u32(&o_free), static_cast<uint32_t>(nseg - 1) & 1u, p.status, 610))) {
+                        failed = true;
+                        break;
+                    }
+                    tc_fence_after();
+                    const uint32_t pb = p_base + (p.p_bufs == 2 ? static_cast<uint32_t>(tiles & 1) * kPBytes : 0u);
+                    const uint64_t b = kHeadsContiguous ? mnmajor_desc(pb) : kmajor_sw128_desc(pb);
+                    uint32_t d = tmem_base + kColO;
+                    for (int u = 0; u < p.nb; ++u, d += N) {
+                        const uint64_t a = mnmajor_desc(smem_base + static_cast<uint32_t>(slot) * kUnitBytes);
+#pragma unroll
+                        for (int ks = 0; ks < 8; ++ks)
+                            tc_mma_bf16(d, a + ks * 2048 / 16,
+                                        b + (kHeadsContiguous ? ks * 2048 : (ks >> 2) * N * 128 + (ks & 3) * 32) / 16, idesc,
+                                        (t > seg.t0 || ks > 0) ? 1u : 0u);
+                        tc_commit(smem_u32(&unit_empty[slot]));
+                        if (++slot == p.ring) slot = 0;
+                    }
+                    tc_commit(smem_u32(&pv_done[tiles & 1]));
                 }
                 ++nseg;
             }
@@ -457,6 +471,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                 if (!mbar_wait_bounded(smem_u32(&s_full[buf]), static_cast<uint32_t>(tiles >> 1) & 1u, p.status, 607)) failed = true;
                 tc_fence_after();
                 const uint32_t s_addr = lane_addr + kColS + static_cast<uint32_t>(buf) * 64u;
+                const uint32_t p_buf = p.p_bufs == 2 ? static_cast<uint32_t>(buf) * kPBytes : 0u;
                 const bool valid = t * kTileKeys + key < seg.len;
                 // does any score outgrow its head's reference?
                 bool over = false;
@@ -474,9 +489,10 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                         over |= __uint_as_float(sv[j + 3]) * p.scale_log2 > ref.w + kLazyLog2;
                     }
                 }
-                // the previous product has read P and written O before either is touched again
-                if (t > seg.t0 && !failed &&
-                    !mbar_wait_bounded(smem_u32(&pv_done), static_cast<uint32_t>(tiles - 1) & 1u, p.status, 608))
+                // the product that last read this buffer of P is done
+                const int read_by = tiles - p.p_bufs;
+                if (t - seg.t0 >= p.p_bufs && !failed &&
+                    !mbar_wait_bounded(smem_u32(&pv_done[read_by & 1]), static_cast<uint32_t>(read_by >> 1) & 1u, p.status, 608))
                     failed = true;
                 // a wait that ran out in one warp ends all four at the same place (two flags in turn: a
                 // warp may be one tile behind the one that sets the next)
@@ -508,6 +524,11 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                     }
                     softmax_sync();
                     if (t > seg.t0) {
+                        // every product so far has added to O
+                        if (!mbar_wait_bounded(smem_u32(&pv_done[(tiles - 1) & 1]), static_cast<uint32_t>((tiles - 1) >> 1) & 1u,
+                                               p.status, 611))
+                            failed = true;
+                        tc_fence_after();
 #pragma unroll
                         for (int h = 0; h < N; ++h) l[h] *= s_alpha[h];
                         for (int u = 0; u < p.nb; ++u)
@@ -548,7 +569,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                     if (kHeadsContiguous) {
 #pragma unroll
                         for (int j = 0; j < 16; j += 8) {
-                            const uint32_t addr = swz128(p_base + static_cast<uint32_t>(key) * 128u, c * 2 + j / 8);
+                            const uint32_t addr = swz128(p_base + p_buf + static_cast<uint32_t>(key) * 128u, c * 2 + j / 8);
                             asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(addr), "r"(pack_bf16(w[j], w[j + 1])),
                                          "r"(pack_bf16(w[j + 2], w[j + 3])), "r"(pack_bf16(w[j + 4], w[j + 5])),
                                          "r"(pack_bf16(w[j + 6], w[j + 7]))
@@ -559,7 +580,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                         for (int j = 0; j < 16; ++j) {
                             const int h = c * 16 + j;
                             const __nv_bfloat16 b = __float2bfloat16_rn(w[j]);
-                            const uint32_t addr = p_key + static_cast<uint32_t>(h) * 128u + ((p_chunk ^ (h & 7)) << 4);
+                            const uint32_t addr = p_key + p_buf + static_cast<uint32_t>(h) * 128u + ((p_chunk ^ (h & 7)) << 4);
                             asm volatile("st.shared.b16 [%0], %1;" ::"r"(addr), "h"(*reinterpret_cast<const uint16_t*>(&b))
                                          : "memory");
                         }
@@ -568,10 +589,13 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                 fence_proxy_async_smem();
                 tc_fence_before();
                 __syncwarp();
-                if (lane == 0) mbar_arrive(smem_u32(&p_full));
+                if (lane == 0) {
+                    mbar_arrive(smem_u32(&s_empty[buf]));
+                    mbar_arrive(smem_u32(&p_full[buf]));
+                }
             }
             if (failed) break;
-            if (!mbar_wait_bounded(smem_u32(&pv_done), static_cast<uint32_t>(tiles - 1) & 1u, p.status, 609)) failed = true;
+            if (!mbar_wait_bounded(smem_u32(&pv_done[(tiles - 1) & 1]), static_cast<uint32_t>((tiles - 1) >> 1) & 1u, p.status, 609)) failed = true;
             tc_fence_after();
             {
                 const int col = warp_transpose_sum<N>(l);
@@ -746,11 +770,15 @@ int launch_latent_attention_tc(const LatentAttention& a, int* status, cudaStream
     p.scale_log2 = a.scale * 1.4426950408889634f;
     p.early = a.only_last_key_new && pdl_launches_enabled() ? 1 : 0;
     p.status = status;
-    const uint32_t fixed = static_cast<uint32_t>(sh.n) * a.width * 2u + 2u * sh.n * 128u + 16u * kUnitElems * 4u + 1024u;
+    const uint32_t p_bytes = 2u * sh.n * 128u;
+    const uint32_t fixed = static_cast<uint32_t>(sh.n) * a.width * 2u + p_bytes + 16u * kUnitElems * 4u + 1024u;
+    constexpr uint32_t kBudget = 224u * 1024u;
     int ring = kMaxUnits;
-    while (ring > p.nb && static_cast<uint32_t>(ring) * kUnitBytes + fixed > 224u * 1024u) --ring;
+    while (ring > p.nb && static_cast<uint32_t>(ring) * kUnitBytes + fixed > kBudget) --ring;
     p.ring = ring;
-    const uint32_t smem = static_cast<uint32_t>(ring) * kUnitBytes + fixed;
+    uint32_t smem = static_cast<uint32_t>(ring) * kUnitBytes + fixed;
+    p.p_bufs = smem + p_bytes <= kBudget ? 2 : 1;
+    if (p.p_bufs == 2) smem += p_bytes;
 
     CUtensorMap tc, tq;
     int err = cached_tmap(&tc, a.cache, static_cast<uint64_t>(a.width), static_cast<uint64_t>(a.num_slots),
