@@ -748,6 +748,152 @@ def run_gpu_tp(args, dist_ready=False, as_record=False):
 
 
 # ------------------------------------------------------------------------------- CPU side
+# ------------------------------------------------------------------------------- layer stacks
+# name -> (width, layers, heads, query latent, kv latent, experts, experts per token, expert ff, batch, context)
+RAPIZEN_SIZES = {
+    "1k": (1024, 12, 8, 384, 256, 32, 2, 1024, 64, 2048),
+    "2k": (2048, 12, 16, 768, 512, 64, 4, 1024, 64, 2048),
+    "4k": (4096, 8, 32, 1536, 512, 32, 2, 2048, 64, 2048),
+}
+RAPIZEN_VOCAB = 32768
+
+
+def rapizen_pair(size: str):
+    """A Rapizen model whose first layer is dense, and a Qwen3-MoE model of the same width, depth, heads and
+    experts (four query heads per KV head)."""
+    from oracle import token_loop_oracle as O
+    from sglang_cpp_b200 import _lib
+    from sglang_cpp_b200.models import LayerSpec, StackConfig
+
+    D, L, H, qr, kr, E, top, ff, _, _ = RAPIZEN_SIZES[size]
+
+    def layer(dense):
+        s = LayerSpec(H, 128, 128, qr, kr, 128 ** -0.5)
+        if dense:
+            s.mlp, s.intermediate, s.epilogue = _lib.MLP_DENSE, 4 * D, _lib.EPILOGUE_GEGLU
+        else:
+            s.mlp, s.intermediate, s.epilogue = _lib.MLP_TABLE_MOE, ff, _lib.EPILOGUE_RELU2
+            s.num_experts, s.experts_per_tok = E, top
+        return s
+
+    new = StackConfig(D, RAPIZEN_VOCAB, 1e-6, [layer(i == 0) for i in range(L)], norm_offset=1.0, logit_scale=0.5)
+    like = O.ModelConfig(L, D, H, max(H // 4, 2), 128, 4 * D, RAPIZEN_VOCAB, 1e-6, 1e6, 8192, False, True, True, "silu",
+                         E, top, ff, True)
+    return new, like
+
+
+def stack_arm(pkg, cfg, size: str, K: int, W: int) -> dict:
+    """Decode and prefill throughput of one model on one GPU (weights drawn on the device)."""
+    from sglang_cpp_b200.engine import Engine, EngineConfig
+    from sglang_cpp_b200.host_batch import HostBatcher
+
+    D, L, H, qr, kr, E, top, ff, B, ctx = RAPIZEN_SIZES[size]
+    stack = getattr(cfg, "layers", None) is not None
+    new_tokens, chunk, page = K + W + 24, MAX_EXTEND_TOKENS, 64
+    num_pages = B * math.ceil((ctx + new_tokens + 1) / page) + 8
+    engine = Engine(cfg, EngineConfig(page, num_pages, B, ctx + new_tokens + 1, chunk))
+    engine.fill_random(seed=0)
+    hb = HostBatcher(engine, num_pages, page, B, enable_prefix_cache=False)
+    rng = np.random.default_rng(4)
+    reqs = [hb.add_request(rng.integers(0, RAPIZEN_VOCAB, size=ctx).astype(np.int32), new_tokens) for _ in range(B)]
+    per = max(chunk // ctx, 1)
+    prefill_ms = []
+    for i in range(0, B, per):
+        hb.prefill(reqs[i:i + per]).synchronize()
+        prefill_ms.append(engine.last_step_ms())
+    # the same prefill steps once more, attention launches timed one by one
+    engine.set_profiling(True)
+    for r in reqs[:per]:
+        r.cached_len, r.device_len = 0, ctx
+    hb.prefill(reqs[:per]).synchronize()
+    attn_prefill_ms, n_attn, _ = engine.read_profile()
+    engine.set_profiling(False)
+    engine.capture_graphs([B])
+    stream = torch.cuda.ExternalStream(pkg.load_library().b200_engine_stream(engine._h))
+    for _ in range(W):
+        hb.decode(reqs)
+    engine.synchronize()
+    torch.cuda.synchronize()
+    ctx0 = reqs[0].device_len
+    ev0, ev1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    wall = time.perf_counter()
+    ev0.record(stream)
+    for _ in range(K):
+        hb.decode(reqs)
+    ev1.record(stream)
+    engine.synchronize()
+    torch.cuda.synchronize()
+    wall = time.perf_counter() - wall
+    ms = ev0.elapsed_time(ev1) / K
+    launches = engine.read_profile()[2]
+    engine.set_profiling(True)
+    attn = []
+    for _ in range(4):
+        hb.decode(reqs).synchronize()
+        attn.append(engine.read_profile()[0] / L)
+    engine.set_profiling(False)
+    peak, _ = measured_peaks()
+    tf = json.loads((ROOT / "MEASURED_PEAKS.json").read_text())["bf16_tflops_sustained"] \
+        if (ROOT / "MEASURED_PEAKS.json").exists() else 1400.0
+    mean_ctx = ctx0 + (K - 1) / 2
+    if stack:
+        attn_w = D * (qr + kr) + H * 128 * (qr + 2 * kr) + H * 128 * D
+        kv_tok = kr * 2
+        dense, exp_mats = 1, 2
+    else:
+        kvh = cfg.num_kv_heads
+        attn_w = D * (H + 2 * kvh) * 128 + H * 128 * D
+        kv_tok = 2 * kvh * 128 * 2
+        dense, exp_mats = 0, 3
+    hit = E * (1 - (1 - top / E) ** B)   # experts a decode step of B uniform tokens reads
+    weights = 2 * (L * attn_w + dense * 3 * 4 * D * D + (L - dense) * hit * exp_mats * ff * D + RAPIZEN_VOCAB * D)
+    step_bytes = weights + L * B * mean_ctx * kv_tok
+    flops_tok = 2 * (L * attn_w + dense * 3 * 4 * D * D + (L - dense) * top * exp_mats * ff * D) + \
+        L * 4 * H * 128 * ctx / 2
+    pf = statistics.median(prefill_ms)
+    pf_attn_flops = per * 4 * H * 128 * ctx * ctx / 2
+    out = {"decode_ms": round(ms, 4), "decode_tokens_s": round(B / ms * 1e3), "e2e_decode_tokens_s": round(B * K / wall),
+           "decode_frac_hbm": round(step_bytes / (ms * 1e-3) / (peak * 1e9), 3), "kernels_per_step": launches,
+           "attention_us": round(statistics.median(attn) * 1e3, 1),
+           "attention_frac_hbm": round(B * (mean_ctx + 4) * kv_tok / (statistics.median(attn) * 1e-3) / (peak * 1e9), 3),
+           "prefill_tokens_s": round(per * ctx / pf * 1e3),
+           "prefill_frac_tensor": round(per * ctx * flops_tok / (pf * 1e-3) / (tf * 1e12), 3),
+           "prefill_attention_us": round(attn_prefill_ms / max(n_attn, 1) * 1e3, 1),
+           "prefill_attention_frac_tensor": round(pf_attn_flops / (attn_prefill_ms / max(n_attn, 1) * 1e-3) / (tf * 1e12), 3)}
+    engine.close()
+    return out
+
+
+def run_gpu_rapizen(args):
+    """Workload "rapizen": prefill and decode of the layer-stack design at sizes that resemble a real
+    model's layers, beside Qwen3-MoE of the same size.  (attention_us of the new design covers the
+    absorbed projections, the attention kernel and its merge; fractions are of the measured copy
+    bandwidth and the sustained cuBLAS rate.)"""
+    import __graft_entry__ as entry
+
+    torch.cuda.set_device(0)
+    pkg = entry.load_package()
+    pkg.load_library()
+    sampler = ClockSampler(0)
+    sampler.start()
+    sizes = {}
+    for size in (args.size.split(",") if args.size else RAPIZEN_SIZES):
+        new, like = rapizen_pair(size)
+        sizes[size] = {"rapizen": stack_arm(pkg, new, size, args.steps, args.warmup),
+                       "qwen3_moe": stack_arm(pkg, like, size, args.steps, args.warmup)}
+    clocks = sampler.stop()
+    first = next(iter(sizes))
+    print(json.dumps({
+        "metric": "decode tokens/s (Rapizen layer stack, %s)" % first, "value": sizes[first]["rapizen"]["decode_tokens_s"],
+        "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+        "ms_per_step": sizes[first]["rapizen"]["decode_ms"], "higher_is_better": True, "scaling": "strong",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "clocks": clocks,
+        "config": {"workload": "rapizen: batch 64, context 2048, page 64; weights and caches larger than L2",
+                   "sizes": {k: dict(zip(("width", "layers", "heads", "q_rank", "kv_rank", "experts", "top", "ff", "batch",
+                                          "context"), RAPIZEN_SIZES[k])) for k in sizes}},
+        "sizes": sizes}))
+
+
 def cpu_decode_sample(steps: int, warmup: int, seconds_budget: float = 0.0, num_reqs: int = BATCH):
     """Times the CPU oracle (a port: the reference has no CPU forward) on decode steps of the
     workload's batch: `num_reqs` requests (all 64 unless host memory is short) at their real context
@@ -837,13 +983,14 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--chunk-tokens", type=int, default=2048, help="c3: tokens a prompt advances per prefill batch")
-    ap.add_argument("--workload", default="c2", choices=["c2", "c3", "c4", "c5"],
+    ap.add_argument("--workload", default="c2", choices=["c2", "c3", "c4", "c5", "rapizen"],
                     help="c2 (default, the headline metric): Qwen3-0.6B decode, replicas when N > 1; "
                          "c3: Qwen3-0.6B chunked prefill alternating with sampled decode, one GPU; "
                          "c4: Llama-3-8B decode, tensor parallel over the N ranks; "
                          "c5: Qwen3-30B-A3B decode, experts and attention heads split over the N ranks")
     ap.add_argument("--context", type=int, default=0,
                     help="c2 only: give every prompt this length instead of U[512,2048]")
+    ap.add_argument("--size", default="", help="rapizen only: sizes to run, with commas between them (default: all)")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-tp-record", action="store_true",
                     help="c2 only: do not run the tensor-parallel workload after the headline")
@@ -863,6 +1010,10 @@ def main():
         run_reference(args)
     elif args.workload in ("c4", "c5"):
         run_gpu_tp(args)
+    elif args.workload == "rapizen":
+        if args.gpus != 1:
+            raise SystemExit("workload rapizen runs on one GPU")
+        run_gpu_rapizen(args)
     elif args.workload == "c3":
         if args.gpus != 1:
             raise SystemExit("workload c3 runs on one GPU")
