@@ -108,6 +108,28 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&p);
 }
 
+// Eight neighbouring elements of an fp32 or bf16 row (16-byte accesses).
+struct Vec8 {
+    float v[8];
+};
+__device__ __forceinline__ Vec8 load8(const float* p) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    return Vec8{{a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w}};
+}
+__device__ __forceinline__ Vec8 load8(const __nv_bfloat16* p) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    return Vec8{{bf16_lo(u.x), bf16_hi(u.x), bf16_lo(u.y), bf16_hi(u.y), bf16_lo(u.z), bf16_hi(u.z), bf16_lo(u.w),
+                 bf16_hi(u.w)}};
+}
+__device__ __forceinline__ void store8(float* p, const Vec8& x) {
+    *reinterpret_cast<float4*>(p) = make_float4(x.v[0], x.v[1], x.v[2], x.v[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(x.v[4], x.v[5], x.v[6], x.v[7]);
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const Vec8& x) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(x.v[0], x.v[1]), pack_bf16(x.v[2], x.v[3]),
+                                              pack_bf16(x.v[4], x.v[5]), pack_bf16(x.v[6], x.v[7]));
+}
+
 __device__ __forceinline__ float round_bf16(float x) {
     return __bfloat162float(__float2bfloat16_rn(x));
 }

@@ -854,13 +854,21 @@ int launch_linear_heads(void* y, const void* x, const void* w, int M, int heads,
                         cudaStream_t stream) {
     const int kb_total = K / kBlockK;
     const int n_tiles = div_ceil(N, kTileN);
+    // the K split of the plain form, over all heads' tiles
+    int split = 1;
+    while (split < 8 && n_tiles * heads * split * 2 <= sm_count() && split * 2 <= kb_total) split *= 2;
+    const int kbp = div_ceil(kb_total, split);
     for (int m0 = 0; m0 < M; m0 += 256) {
         const int rows = M - m0 < 256 ? M - m0 : 256;
         const int nt = rows <= 32 ? 32 : div_ceil(rows, kRoundCols) * kRoundCols;
         const uint32_t stage_bytes = kTileN * kBlockK * 2 + nt * kBlockK * 2;
-        int stages = kb_total < kMaxStages ? kb_total : kMaxStages;
-        while (stages > 2 && stages * stage_bytes > 100 * 1024) --stages;   // two CTAs per SM
-        const uint32_t smem_bytes = stages * stage_bytes + 1024;
+        const int cpr = nt < kRoundCols ? nt : kRoundCols;
+        const uint32_t exch_bytes = split > 1 ? (nt > cpr ? 2u : 1u) * cpr * kTileN * 4u : 0u;
+        int stages = kbp < kMaxStages ? kbp : kMaxStages;
+        // more CTAs than SMs: small rings, two CTAs per SM
+        const uint32_t limit = n_tiles * heads * split > sm_count() ? 100 * 1024 : 200 * 1024;
+        while (stages > 1 && stages * stage_bytes + exch_bytes > limit) --stages;
+        const uint32_t smem_bytes = stages * stage_bytes + exch_bytes + 1024;
         const __nv_bfloat16* xs = static_cast<const __nv_bfloat16*>(x) + static_cast<int64_t>(m0) * heads * K;
         CUtensorMap tmap_w, tmap_x;
         int err = cached_tmap(&tmap_w, w, static_cast<uint64_t>(K), static_cast<uint64_t>(heads) * N,
@@ -889,8 +897,8 @@ int launch_linear_heads(void* y, const void* x, const void* w, int M, int heads,
         auto kernel = skinny_kernel_for(B200_EPILOGUE_NONE);
         B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                              static_cast<int>(smem_bytes)));
-        B200_CHECK_CUDA(launch_kernel(kernel, dim3(n_tiles, 1, heads), dim3(kThreads), smem_bytes, stream,
-                                      dim3(1, 1, 1), tmap_w, tmap_x, tmap_x, tmap_x, tmap_x, p));
+        B200_CHECK_CUDA(launch_kernel(kernel, dim3(n_tiles, split, heads), dim3(kThreads), smem_bytes, stream,
+                                      dim3(1, split, 1), tmap_w, tmap_x, tmap_x, tmap_x, tmap_x, p));
     }
     return B200_OK;
 }

@@ -25,49 +25,63 @@ __device__ __forceinline__ void put(float* p, float v) { *p = v; }
 __device__ __forceinline__ void put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 
 // Columns [0, qp) of a token's joint row are its query latent, [qp, qp + rp) its key/value latent; each is
-// divided by its own root mean square (over the true widths) and scaled by its own weight.
+// divided by its own root mean square (over the true widths) and scaled by its own weight.  One warp per
+// latent: warps 0 and 1 of a pair take the two latents of one token, four tokens per CTA, the row in
+// registers (latents of up to 8 x 256 elements; wider ones are read again).
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_norm_store_kernel(T* __restrict__ q_latent, T* __restrict__ cache, const T* __restrict__ joint,
                          const T* __restrict__ q_weight, const T* __restrict__ kv_weight,
-                         const int32_t* __restrict__ out_loc, int q_rank, int qp, int kv_rank, int rp,
+                         const int32_t* __restrict__ out_loc, int tokens, int q_rank, int qp, int kv_rank, int rp,
                          int64_t num_slots, float eps, int* status) {
-    __shared__ float red[2][8];
+    constexpr int kKeep = 8;
     pdl_launch_dependents();
     pdl_wait_prior();
-    const int64_t t = blockIdx.x;
-    const T* row = joint + t * (qp + rp);
-    float sq = 0.f, sk = 0.f;
-    for (int i = threadIdx.x; i < qp; i += blockDim.x) {
-        const float v = as_float(row[i]);
-        sq += v * v;
-    }
-    for (int i = threadIdx.x; i < rp; i += blockDim.x) {
-        const float v = as_float(row[qp + i]);
-        sk += v * v;
-    }
-    sq = warp_sum(sq);
-    sk = warp_sum(sk);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    if (lane == 0) {
-        red[0][warp] = sq;
-        red[1][warp] = sk;
+    const int64_t t = static_cast<int64_t>(blockIdx.x) * (blockDim.x >> 6) + (warp >> 1);
+    if (t >= tokens) return;
+    const bool kv = (warp & 1) != 0;
+    const T* src = joint + t * (qp + rp) + (kv ? qp : 0);
+    const T* weight = kv ? kv_weight : q_weight;
+    const int nvec = (kv ? rp : qp) >> 3;
+    int64_t slot = 0;
+    if (kv) slot = out_loc[t];
+    Vec8 x[kKeep];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+        const int v = lane + i * 32;
+        if (v < nvec) {
+            x[i] = load8(src + v * 8);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) ss += x[i].v[j] * x[i].v[j];
+        }
     }
-    __syncthreads();
-    const int nw = blockDim.x >> 5;
-    sq = warp_sum(lane < nw ? red[0][lane] : 0.f);
-    sk = warp_sum(lane < nw ? red[1][lane] : 0.f);
-    const float rq = rsqrtf(sq / static_cast<float>(q_rank) + eps);
-    const float rk = rsqrtf(sk / static_cast<float>(kv_rank) + eps);
-    for (int i = threadIdx.x; i < qp; i += blockDim.x)
-        put(q_latent + t * qp + i, as_float(row[i]) * rq * as_float(q_weight[i]));
-    const int64_t slot = out_loc[t];
-    if (slot < 0 || slot >= num_slots) {
-        if (threadIdx.x == 0) atomicExch(&status[kStatusBadIndex], static_cast<int>(slot) + 1);
-        return;
+    for (int v = lane + kKeep * 32; v < nvec; v += 32) {
+        const Vec8 y = load8(src + v * 8);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ss += y.v[j] * y.v[j];
     }
-    for (int i = threadIdx.x; i < rp; i += blockDim.x)
-        put(cache + slot * rp + i, as_float(row[qp + i]) * rk * as_float(kv_weight[i]));
+    const float r = rsqrtf(warp_sum(ss) / static_cast<float>(kv ? kv_rank : q_rank) + eps);
+    T* dst = q_latent + t * qp;
+    if (kv) {
+        if (slot < 0 || slot >= num_slots) {
+            if (lane == 0) atomicExch(&status[kStatusBadIndex], static_cast<int>(slot) + 1);
+            return;
+        }
+        dst = cache + slot * rp;
+    }
+    auto emit = [&](int v, const Vec8& y) {
+        const Vec8 g = load8(weight + v * 8);
+        Vec8 o;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) o.v[j] = y.v[j] * r * g.v[j];
+        store8(dst + v * 8, o);
+    };
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i)
+        if (lane + i * 32 < nvec) emit(lane + i * 32, x[i]);
+    for (int v = lane + kKeep * 32; v < nvec; v += 32) emit(v, load8(src + v * 8));
 }
 
 // One CTA per (query row, head); its warps take every fourth key each with an online softmax whose
@@ -177,17 +191,20 @@ int launch_latent_norm_store(void* q_latent, void* cache, const void* joint, con
                              int kv_rank, int rp, int64_t num_slots, float eps, int dtype, int* status,
                              cudaStream_t stream) {
     if (tokens == 0) return B200_OK;
+    // few tokens: a CTA each, for latency; many: four per CTA
+    const int threads = tokens <= 2 * sm_count() ? 64 : 256;
+    const int grid = div_ceil(tokens, threads / 64);
     if (dtype == B200_DTYPE_F32) {
-        B200_CHECK_CUDA(launch_kernel(latent_norm_store_kernel<float>, dim3(tokens), dim3(256), 0, stream, dim3(1, 1, 1),
+        B200_CHECK_CUDA(launch_kernel(latent_norm_store_kernel<float>, dim3(grid), dim3(threads), 0, stream, dim3(1, 1, 1),
                                       static_cast<float*>(q_latent), static_cast<float*>(cache),
                                       static_cast<const float*>(joint), static_cast<const float*>(q_weight),
-                                      static_cast<const float*>(kv_weight), out_loc, q_rank, qp, kv_rank, rp, num_slots,
+                                      static_cast<const float*>(kv_weight), out_loc, tokens, q_rank, qp, kv_rank, rp, num_slots,
                                       eps, status));
     } else {
         using B = __nv_bfloat16;
-        B200_CHECK_CUDA(launch_kernel(latent_norm_store_kernel<B>, dim3(tokens), dim3(256), 0, stream, dim3(1, 1, 1),
+        B200_CHECK_CUDA(launch_kernel(latent_norm_store_kernel<B>, dim3(grid), dim3(threads), 0, stream, dim3(1, 1, 1),
                                       static_cast<B*>(q_latent), static_cast<B*>(cache), static_cast<const B*>(joint),
-                                      static_cast<const B*>(q_weight), static_cast<const B*>(kv_weight), out_loc, q_rank,
+                                      static_cast<const B*>(q_weight), static_cast<const B*>(kv_weight), out_loc, tokens, q_rank,
                                       qp, kv_rank, rp, num_slots, eps, status));
     }
     return B200_OK;

@@ -8,23 +8,8 @@
 namespace b200 {
 namespace {
 
-constexpr int kVec = 8;   // float4 vectors a thread keeps; wider rows are read again from the residual
-
-template <typename T>
-__device__ __forceinline__ float4 load4(const T* p);
-template <>
-__device__ __forceinline__ float4 load4<float>(const float* p) {
-    return *reinterpret_cast<const float4*>(p);
-}
-template <>
-__device__ __forceinline__ float4 load4<__nv_bfloat16>(const __nv_bfloat16* p) {
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
-    return make_float4(bf16_lo(u.x), bf16_hi(u.x), bf16_lo(u.y), bf16_hi(u.y));
-}
-__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
-    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
-}
+// A thread works on pieces of 8 elements; it keeps up to VEC of them, wider rows are read again.
+constexpr int kRows = 16;   // row numbers of a token kept in shared memory; wider choices are read from global
 
 struct Args {
     void* out;
@@ -39,62 +24,94 @@ struct Args {
     int* status;
 };
 
-template <typename T>
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 residual_norm_kernel(const Args a) {
     __shared__ float red[8];
+    __shared__ int s_src[kRows], s_out[kRows];
     pdl_launch_dependents();
-    const int nvec = a.padded >> 2;
+    const int nvec = a.padded >> 3;
     const T* weight = static_cast<const T*>(a.weight);
     // the norm weights do not come from the kernel before this one
-    float4 w[kVec];
+    Vec8 w[VEC];
 #pragma unroll
-    for (int i = 0; i < kVec; ++i) {
+    for (int i = 0; i < VEC; ++i) {
         const int v = threadIdx.x + i * blockDim.x;
-        w[i] = v < nvec ? load4(weight + v * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+        if (v < nvec) w[i] = load8(weight + v * 8);
     }
     pdl_wait_prior();
     const int64_t t = blockIdx.x;
+    if (a.src_rows != nullptr || a.out_rows != nullptr) {
+        if (threadIdx.x < kRows) {
+            const int k = threadIdx.x;
+            if (a.src_rows != nullptr && k < a.src_top) s_src[k] = a.src_rows[t * a.src_top + k];
+            if (a.out_rows != nullptr && k < a.out_top) s_out[k] = a.out_rows[t * a.out_top + k];
+        }
+        __syncthreads();
+    }
     float* res = a.residual + t * a.padded;
     const T* src = static_cast<const T*>(a.src);
-    auto sum_at = [&](int v) {
-        float4 s = a.init ? make_float4(0.f, 0.f, 0.f, 0.f) : load4(static_cast<const float*>(res) + v * 4);
-        if (src != nullptr) {
-            float4 add = make_float4(0.f, 0.f, 0.f, 0.f);
-            for (int k = 0; k < a.src_top; ++k) {
-                const int64_t row = a.src_rows ? a.src_rows[t * a.src_top + k] : t;
-                if (row < 0 || row >= a.src_count) {
-                    if (v == 0) atomicExch(&a.status[kStatusBadIndex], static_cast<int>(row) + 1);
-                    continue;
-                }
-                const float4 x = load4(src + row * a.padded + v * 4);
-                add.x += x.x;
-                add.y += x.y;
-                add.z += x.z;
-                add.w += x.w;
-            }
-            s.x += a.src_scale * add.x;
-            s.y += a.src_scale * add.y;
-            s.z += a.src_scale * add.z;
-            s.w += a.src_scale * add.w;
-        }
-        return s;
+    // row k of what is added; a row outside the source adds nothing and is reported
+    auto src_row = [&](int k) -> int64_t {
+        if (a.src_rows == nullptr) return t;
+        const int64_t row = k < kRows ? s_src[k] : a.src_rows[t * a.src_top + k];
+        if (row >= 0 && row < a.src_count) return row;
+        if (threadIdx.x == 0) atomicExch(&a.status[kStatusBadIndex], static_cast<int>(row) + 1);
+        return -1;
     };
-    float4 val[kVec];
-    float ss = 0.f;
+    Vec8 val[VEC], add[VEC];
 #pragma unroll
-    for (int i = 0; i < kVec; ++i) {
+    for (int i = 0; i < VEC; ++i) {
         const int v = threadIdx.x + i * blockDim.x;
-        if (v < nvec) {
-            val[i] = sum_at(v);
-            if (src != nullptr) store4(res + v * 4, val[i]);
-            ss += val[i].x * val[i].x + val[i].y * val[i].y + val[i].z * val[i].z + val[i].w * val[i].w;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) val[i].v[j] = add[i].v[j] = 0.f;
+        if (v < nvec && !a.init) val[i] = load8(static_cast<const float*>(res) + v * 8);
+    }
+    if (src != nullptr) {
+#pragma unroll 4
+        for (int k = 0; k < a.src_top; ++k) {
+            const int64_t row = src_row(k);
+            if (row < 0) continue;
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) {
+                const int v = threadIdx.x + i * blockDim.x;
+                if (v < nvec) {
+                    const Vec8 x = load8(src + row * a.padded + v * 8);
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) add[i].v[j] += x.v[j];
+                }
+            }
         }
     }
-    for (int v = threadIdx.x + kVec * blockDim.x; v < nvec; v += blockDim.x) {
-        const float4 s = sum_at(v);
-        if (src != nullptr) store4(res + v * 4, s);
-        ss += s.x * s.x + s.y * s.y + s.z * s.z + s.w * s.w;
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+        const int v = threadIdx.x + i * blockDim.x;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            val[i].v[j] += a.src_scale * add[i].v[j];
+            ss += val[i].v[j] * val[i].v[j];
+        }
+        if (v < nvec && src != nullptr) store8(res + v * 8, val[i]);
+    }
+    for (int v = threadIdx.x + VEC * blockDim.x; v < nvec; v += blockDim.x) {   // rows wider than the registers
+        Vec8 x, y;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x.v[j] = y.v[j] = 0.f;
+        if (!a.init) x = load8(static_cast<const float*>(res) + v * 8);
+        for (int k = 0; src != nullptr && k < a.src_top; ++k) {
+            const int64_t row = src_row(k);
+            if (row < 0) continue;
+            const Vec8 z = load8(src + row * a.padded + v * 8);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) y.v[j] += z.v[j];
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            x.v[j] += a.src_scale * y.v[j];
+            ss += x.v[j] * x.v[j];
+        }
+        store8(res + v * 8, x);
     }
     ss = warp_sum(ss);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -103,23 +120,31 @@ residual_norm_kernel(const Args a) {
     ss = warp_sum(lane < static_cast<int>(blockDim.x >> 5) ? red[lane] : 0.f);
     const float scale = rsqrtf(ss / static_cast<float>(a.width) + a.eps) * a.out_scale;
     T* out = static_cast<T*>(a.out);
-    if (out == nullptr) return;
-    auto emit = [&](int v, float4 s, float4 g) {
-        const float o = a.weight_offset;
-        const float4 y = make_float4(s.x * scale * (g.x + o), s.y * scale * (g.y + o), s.z * scale * (g.z + o),
-                                     s.w * scale * (g.w + o));
+    auto emit = [&](int v, const Vec8& x, const Vec8& g) {
+        Vec8 y;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) y.v[j] = x.v[j] * scale * (g.v[j] + a.weight_offset);
+        if (a.out_rows == nullptr) {
+            store8(out + t * a.padded + v * 8, y);
+            return;
+        }
         for (int k = 0; k < a.out_top; ++k) {
-            const int64_t row = a.out_rows ? a.out_rows[t * a.out_top + k] : t;
-            store4(out + row * a.padded + v * 4, y);
+            const int64_t row = k < kRows ? s_out[k] : a.out_rows[t * a.out_top + k];
+            store8(out + row * a.padded + v * 8, y);
         }
     };
 #pragma unroll
-    for (int i = 0; i < kVec; ++i) {
+    for (int i = 0; i < VEC; ++i) {
         const int v = threadIdx.x + i * blockDim.x;
         if (v < nvec) emit(v, val[i], w[i]);
     }
-    for (int v = threadIdx.x + kVec * blockDim.x; v < nvec; v += blockDim.x)
-        emit(v, load4(static_cast<const float*>(res) + v * 4), load4(weight + v * 4));
+    for (int v = threadIdx.x + VEC * blockDim.x; v < nvec; v += blockDim.x)
+        emit(v, load8(static_cast<const float*>(res) + v * 8), load8(weight + v * 8));
+}
+
+template <typename T>
+auto kernel_for(int pieces) {   // pieces of 8 elements per thread
+    return pieces <= 1 ? residual_norm_kernel<T, 1> : pieces <= 2 ? residual_norm_kernel<T, 2> : residual_norm_kernel<T, 4>;
 }
 
 }  // namespace
@@ -144,9 +169,10 @@ int launch_residual_norm(const ResidualNorm& r, int dtype, int* status, cudaStre
     a.out_scale = r.out_scale;
     a.eps = r.eps;
     a.status = status;
-    int threads = 64;
+    int threads = 32;
     while (threads < 256 && threads * 8 < r.padded) threads *= 2;
-    auto kernel = dtype == B200_DTYPE_F32 ? residual_norm_kernel<float> : residual_norm_kernel<__nv_bfloat16>;
+    const int pieces = div_ceil(r.padded, threads * 8);
+    auto kernel = dtype == B200_DTYPE_F32 ? kernel_for<float>(pieces) : kernel_for<__nv_bfloat16>(pieces);
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(r.tokens), dim3(threads), 0, stream, dim3(1, 1, 1), a));
     return B200_OK;
 }

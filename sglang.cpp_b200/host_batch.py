@@ -266,7 +266,8 @@ class _Tables:
 
     def write_pages(self, rows, pos, slots) -> None:
         rows, pos, slots = (np.asarray(a, dtype=np.int32) for a in (rows, pos, slots))
-        self.page_table[rows, pos] = slots
+        ok = pos < self.page_table.shape[1]   # the last page may reach past the row (the device skips those too)
+        self.page_table[rows[ok], pos[ok]] = slots[ok]
         if self.engine is not None and len(rows):
             self.engine.write_page_table(rows, pos, slots)
 
