@@ -3,14 +3,16 @@
 // Every query row (one token) has H heads that all read the same latents, so one latent tile is loaded
 // once for all heads.  The products are turned around so that the long dimension, not the few heads, fills
 // the 128 rows of the MMA:
-//     S^T = C Q^T      128 keys x N heads, K = latent width: A is the latent tile as TMA delivers it
-//     O^T += C^T P^T   128 latent elements x N heads, K = 128 keys: A is the SAME tile read MN-major, so it
+//     S^T = C Q^T      KT keys x N heads, K = latent width: A is the latent tile as TMA delivers it
+//     O^T += C^T P^T   128 latent elements x N heads, K = KT keys: A is the SAME tile read MN-major, so it
 //                      is fetched from HBM once and never moved again
 // with N = 16, 32 or 64 heads per block (more heads run as further blocks of the same row) and S^T, O^T
 // accumulating in TMEM.
 //
-// A tile is 128 keys; it lives in shared memory as width / 128 units of 128 keys x 128 elements (32 KB), a
-// ring of which the producer keeps full; a unit is free again as soon as its O^T product has read it.
+// A tile is KT keys - 128, or 64 for wide latents, whose tiles stay in shared memory so long (until the softmax
+// of the whole tile is done) that 128 keys would leave no room to load ahead.  It lives in shared memory as
+// width / 128 units of KT keys x 128 elements, a ring of which the producer keeps full; a unit is free again
+// as soon as its O^T product has read it.
 // Softmax: one thread per key (= TMEM lane), all heads of the block in its registers.  The reference
 // maximum of a head only moves when some score exceeds it by more than 2^8, which a single block-wide vote
 // finds out; the running sum stays per thread until a row is finished.  Everything about scores and weights
@@ -33,11 +35,8 @@
 namespace b200 {
 namespace {
 
-constexpr int kTileKeys = 128;
 constexpr int kUnitElems = 128;                            // latent elements per unit
-constexpr uint32_t kAtomBytes = kTileKeys * 128;           // 128 keys x 64 elements, 128-byte rows
-constexpr uint32_t kUnitBytes = 2 * kAtomBytes;
-constexpr int kMaxUnits = 6;                               // units in the ring
+constexpr int kMaxUnits = 12;                              // units in the ring
 constexpr int kThreads = 224;
 constexpr int kMaxWidth = 512;
 constexpr uint32_t kColO = 0, kColS = 256;                 // TMEM columns: O^T (4 x 64), S^T (2 x 64)
@@ -69,10 +68,11 @@ struct LatentParams {
 
 // MN-major operand under the 128-byte swizzle (rows are keys, 64 latent elements per 128-byte row): the
 // next 64 elements one atom further, the next 8 keys 1024 bytes further.
+template <int KT>
 __device__ __forceinline__ uint64_t mnmajor_desc(uint32_t smem_addr) {
     uint64_t d = 0;
     d |= static_cast<uint64_t>((smem_addr >> 4) & 0x3FFFu);
-    d |= static_cast<uint64_t>(kAtomBytes >> 4) << 16;
+    d |= static_cast<uint64_t>((KT * 128) >> 4) << 16;
     d |= static_cast<uint64_t>(1024 >> 4) << 32;
     d |= static_cast<uint64_t>(1) << 46;
     d |= static_cast<uint64_t>(2) << 61;
@@ -140,6 +140,7 @@ struct Segment {
     int row, block, t0, t1, len;   // tiles [t0, t1) of an item whose row has len keys
     bool starts, ends;             // the item starts / ends inside this segment
 };
+template <int KT>
 __device__ __forceinline__ bool next_segment(Walk& w, const LatentParams& p, Segment& s) {
     if (w.left <= 0) return false;
     auto len_of = [&](int row) { return row - w.row0 < kLens ? w.lens[row - w.row0] : p.row_len[row]; };
@@ -150,7 +151,7 @@ __device__ __forceinline__ bool next_segment(Walk& w, const LatentParams& p, Seg
         if (w.row >= p.rows) return false;
         len = len_of(w.row);
     }
-    const int nt = (len + kTileKeys - 1) / kTileKeys;
+    const int nt = (len + KT - 1) / KT;
     s.row = w.row;
     s.block = w.block;
     s.len = len;
@@ -167,10 +168,12 @@ __device__ __forceinline__ bool next_segment(Walk& w, const LatentParams& p, Seg
     return true;
 }
 
-template <int N>
+template <int N, int KT>
 __global__ void __launch_bounds__(kThreads, 1)
 latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __grid_constant__ CUtensorMap tmap_q,
                            const LatentParams p) {
+    constexpr uint32_t kAtomBytes = KT * 128;        // KT keys x 64 elements, 128-byte rows
+    constexpr uint32_t kUnitBytes = 2 * kAtomBytes;
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t unit_full[kMaxUnits];
     __shared__ __align__(8) uint64_t unit_empty[kMaxUnits];
@@ -183,12 +186,13 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
     __shared__ float s_warp[4][N];
     __shared__ volatile int s_failed[2];
     __shared__ int s_len[kLens];
+    __shared__ int s_slot[128];     // the producer's current group of page-table look-ups
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t smem_base = (smem_u32(smem_raw) + 1023u) & ~1023u;
     const uint32_t q_base = smem_base + static_cast<uint32_t>(p.ring) * kUnitBytes;
     const uint32_t p_base = q_base + static_cast<uint32_t>(N) * static_cast<uint32_t>(p.width) * 2u;
-    constexpr uint32_t kPBytes = 2u * N * 128u;
+    constexpr uint32_t kPBytes = KT / 64 * N * 128u;
     const uint32_t stage_off = p_base + static_cast<uint32_t>(p.p_bufs) * kPBytes - smem_u32(smem_raw);   // output staging [16][128] fp32
     // The weights are the B operand of the second product: keys contiguous (one 2-byte store per head), or for
     // a full 64 heads heads contiguous, so that a thread stores its key's row in 16-byte pieces.
@@ -226,7 +230,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
         const int per = (p.rows + kThreads - 1) / kThreads;
         const int r0 = min(static_cast<int>(threadIdx.x) * per, p.rows), r1 = min(r0 + per, p.rows);
         int mine = 0;
-        for (int r = r0; r < r1; ++r) mine += (max(p.row_len[r], 0) + kTileKeys - 1) / kTileKeys * p.blocks;
+        for (int r = r0; r < r1; ++r) mine += (max(p.row_len[r], 0) + KT - 1) / KT * p.blocks;
         int incl = mine;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
@@ -246,7 +250,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
         if (g0 >= begin && g0 < begin + mine) {
             int at = begin;
             for (int r = r0; r < r1; ++r) {
-                const int nt = (max(p.row_len[r], 0) + kTileKeys - 1) / kTileKeys;
+                const int nt = (max(p.row_len[r], 0) + KT - 1) / KT;
                 if (g0 < at + nt * p.blocks) {
                     s_row = r;
                     s_block = (g0 - at) / nt;
@@ -279,20 +283,19 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
 
     if (warp == 0) {
         // ================= producer =================
-        const int copies = kTileKeys / p.kpc;
-        int ring_at = 0, unit = 0, nseg = 0;
-        uint32_t ring_parity = 1;          // of the slot's previous use
-        bool waited = !p.early;
-        // Page-table look-ups run a group of 128 copies (kpc tiles) ahead of the loads: copy i of a group is
-        // held, and issued, by lane i % 32.  A copy past the last key reads a row outside the tensor, which
-        // the copy engine fills with zeros.
+        // Page-table look-ups run a group of 128 copies ahead of the loads: the whole warp fetches the next
+        // group while one elected lane issues the copies of this one (copies issued lane by lane cost 250
+        // cycles each).  A copy past the last key reads a row outside the tensor, which the copy engine fills
+        // with zeros.
+        const int copies = KT / p.kpc, group_tiles = 128 / copies;
+        const bool whole_unit = p.kpc == KT;      // one copy brings both halves of a unit
         auto slots_of = [&](const Segment& g, int t0, int (&sl)[4]) {
             const int32_t* pt = p.page_table + static_cast<int64_t>(p.row_table[g.row]) * p.pt_stride;
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-                const int key = t0 * kTileKeys + (i * 32 + lane) * p.kpc;
+                const int key = t0 * KT + (i * 32 + lane) * p.kpc;
                 sl[i] = static_cast<int>(p.num_slots);
-                if (key < min(g.len, g.t1 * kTileKeys)) {
+                if (key < min(g.len, g.t1 * KT)) {
                     const int64_t v = pt[key];
                     if (v < 0 || v + p.kpc > p.num_slots)
                         atomicExch(&p.status[kStatusBadIndex], static_cast<int>(v) + 1);
@@ -301,86 +304,93 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                 }
             }
         };
-        int sl[4], sl_next[4];
-        bool have = next_segment(walk, p, seg);
-        if (have) slots_of(seg, seg.t0, sl_next);
+        int next[4];
+        int ring_at = 0, unit = 0, nseg = 0;
+        uint32_t ring_parity = 1;          // of the slot's previous use
+        bool waited = !p.early;
+        bool have = next_segment<KT>(walk, p, seg);
+        if (have) slots_of(seg, seg.t0, next);
+        int t = have ? seg.t0 : 0;
         while (have && !failed) {
-            Segment upcoming = seg;
-            bool more = false;
-            for (int t = seg.t0; t < seg.t1 && !failed; ++t) {
-                const int in_group = (t - seg.t0) & (p.kpc - 1);
-                if (in_group == 0) {
+            __syncwarp();
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) sl[i] = sl_next[i];
-                    if (t + p.kpc < seg.t1) {
-                        slots_of(seg, t + p.kpc, sl_next);
-                    } else {
-                        more = next_segment(walk, p, upcoming);
-                        if (more) slots_of(upcoming, upcoming.t0, sl_next);
-                    }
-                }
-                if (!waited && (t + 1) * kTileKeys >= seg.len) {   // this tile holds the newest key
+            for (int i = 0; i < 4; ++i) s_slot[i * 32 + lane] = next[i];
+            __syncwarp();
+            // the group's tiles are [t, t_end); what comes behind them is looked up meanwhile
+            const int t_end = min(t + group_tiles, seg.t1);
+            const Segment cur = seg;
+            if (t_end < seg.t1) {
+                slots_of(seg, t_end, next);
+            } else {
+                have = next_segment<KT>(walk, p, seg);
+                if (have) slots_of(seg, seg.t0, next);
+            }
+            const bool lead = elect_one();
+            for (int tt = t; tt < t_end && !failed; ++tt) {
+                if (!waited && (tt + 1) * KT >= cur.len) {   // this tile holds the newest key
                     pdl_wait_prior();
                     waited = true;
                 }
-                for (int u = 0; u < p.nb; ++u, ++unit) {
-                    const int s = ring_at;
-                    const bool ok = unit < p.ring || mbar_wait_bounded(smem_u32(&unit_empty[s]), ring_parity, p.status, 601);
-                    if (!__all_sync(0xffffffffu, ok)) {
-                        failed = true;
-                        break;
-                    }
-                    const uint32_t bar = smem_u32(&unit_full[s]);
-                    const uint32_t dst = smem_base + static_cast<uint32_t>(s) * kUnitBytes;
-                    if (lane == 0) mbar_arrive_expect_tx(bar, kUnitBytes);
-                    __syncwarp();
-#pragma unroll
-                    for (int i = 0; i < 4; ++i) {
-                        const int copy = i * 32 + lane - in_group * copies;
-                        if (copy >= 0 && copy < copies) {
-                            const uint32_t to = dst + static_cast<uint32_t>(copy * p.kpc) * 128u;
-                            tma_load_2d(to, &tmap_c, u * kUnitElems, sl[i], bar);
-                            tma_load_2d(to + kAtomBytes, &tmap_c, u * kUnitElems + 64, sl[i], bar);
+                bool ok = true;
+                if (lead) {
+                    for (int u = 0; u < p.nb && ok; ++u, ++unit) {
+                        if (unit >= p.ring &&
+                            !mbar_wait_bounded(smem_u32(&unit_empty[ring_at]), ring_parity, p.status, 601)) {
+                            ok = false;
+                            break;
+                        }
+                        const uint32_t bar = smem_u32(&unit_full[ring_at]);
+                        const uint32_t dst = smem_base + static_cast<uint32_t>(ring_at) * kUnitBytes;
+                        mbar_arrive_expect_tx(bar, kUnitBytes);
+                        if (whole_unit) {
+                            tma_load_3d(dst, &tmap_c, 0, s_slot[tt - t], 2 * u, bar);
+                        } else {
+                            for (int c = 0; c < copies; ++c) {
+                                const int sl = s_slot[(tt - t) * copies + c];
+                                const uint32_t to = dst + static_cast<uint32_t>(c * p.kpc) * 128u;
+                                tma_load_3d(to, &tmap_c, 0, sl, 2 * u, bar);
+                                tma_load_3d(to + kAtomBytes, &tmap_c, 0, sl, 2 * u + 1, bar);
+                            }
+                        }
+                        if (++ring_at == p.ring) {
+                            ring_at = 0;
+                            ring_parity ^= 1u;
                         }
                     }
-                    if (++ring_at == p.ring) {
-                        ring_at = 0;
-                        ring_parity ^= 1u;
-                    }
                 }
-                if (t == seg.t0 && !failed) {
+                if (tt == cur.t0) {
                     // the queries of this item, behind the first tile's latents
+                    __syncwarp();
                     if (!waited) {
                         pdl_wait_prior();
                         waited = true;
                     }
-                    const bool ok = nseg == 0 || mbar_wait_bounded(smem_u32(&q_empty), static_cast<uint32_t>(nseg - 1) & 1u,
-                                                                   p.status, 602);
-                    if (!__all_sync(0xffffffffu, ok)) {
-                        failed = true;
-                        break;
+                    if (lead && ok) {
+                        if (nseg > 0 && !mbar_wait_bounded(smem_u32(&q_empty), static_cast<uint32_t>(nseg - 1) & 1u, p.status, 602)) {
+                            ok = false;
+                        } else {
+                            const uint32_t bar = smem_u32(&q_full);
+                            mbar_arrive_expect_tx(bar, static_cast<uint32_t>(N) * p.width * 2u);
+                            for (int a = 0; a < p.width / 64; ++a)
+                                tma_load_2d(q_base + static_cast<uint32_t>(a) * N * 128u, &tmap_q, a * 64,
+                                            cur.row * p.heads + cur.block * p.per_block, bar);
+                        }
                     }
-                    const uint32_t bar = smem_u32(&q_full);
-                    if (lane == 0) mbar_arrive_expect_tx(bar, static_cast<uint32_t>(N) * p.width * 2u);
-                    __syncwarp();
-                    for (int a = lane; a < p.width / 64; a += 32)
-                        tma_load_2d(q_base + static_cast<uint32_t>(a) * N * 128u, &tmap_q, a * 64,
-                                    seg.row * p.heads + seg.block * p.per_block, bar);
+                    ++nseg;
                 }
+                failed = !__all_sync(0xffffffffu, ok);
             }
-            ++nseg;
-            have = more;
-            seg = upcoming;
+            t = t_end < cur.t1 ? t_end : seg.t0;
         }
         if (!waited) pdl_wait_prior();
     } else if (warp == 1) {
         // ================= S^T = C Q^T =================
         pdl_wait_prior();
         if (elect_one()) {
-            const uint32_t idesc = idesc_bf16_m128(N);
+            const uint32_t idesc = idesc_bf16(KT, N);
             int slot = 0, tiles = 0, nseg = 0;
             uint32_t parity = 0;
-            while (!failed && next_segment(walk, p, seg)) {
+            while (!failed && next_segment<KT>(walk, p, seg)) {
                 if (!mbar_wait_bounded(smem_u32(&q_full), static_cast<uint32_t>(nseg) & 1u, p.status, 603)) break;
                 for (int t = seg.t0; t < seg.t1 && !failed; ++t, ++tiles) {
                     const int buf = tiles & 1;
@@ -422,7 +432,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
             // A is MN-major; B is too where the heads of a key are contiguous
             const uint32_t idesc = idesc_bf16_m128(N) | (1u << 15) | (kHeadsContiguous ? 1u << 16 : 0u);
             int slot = 0, tiles = 0, nseg = 0;
-            while (!failed && next_segment(walk, p, seg)) {
+            while (!failed && next_segment<KT>(walk, p, seg)) {
                 for (int t = seg.t0; t < seg.t1; ++t, ++tiles) {
                     if (!mbar_wait_bounded(smem_u32(&p_full[tiles & 1]), static_cast<uint32_t>(tiles >> 1) & 1u, p.status, 606) ||
                         (t == seg.t0 && nseg > 0 &&
@@ -432,12 +442,12 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                     }
                     tc_fence_after();
                     const uint32_t pb = p_base + (p.p_bufs == 2 ? static_cast<uint32_t>(tiles & 1) * kPBytes : 0u);
-                    const uint64_t b = kHeadsContiguous ? mnmajor_desc(pb) : kmajor_sw128_desc(pb);
+                    const uint64_t b = kHeadsContiguous ? mnmajor_desc<KT>(pb) : kmajor_sw128_desc(pb);
                     uint32_t d = tmem_base + kColO;
                     for (int u = 0; u < p.nb; ++u, d += N) {
-                        const uint64_t a = mnmajor_desc(smem_base + static_cast<uint32_t>(slot) * kUnitBytes);
+                        const uint64_t a = mnmajor_desc<KT>(smem_base + static_cast<uint32_t>(slot) * kUnitBytes);
 #pragma unroll
-                        for (int ks = 0; ks < 8; ++ks)
+                        for (int ks = 0; ks < KT / 16; ++ks)
                             tc_mma_bf16(d, a + ks * 2048 / 16,
                                         b + (kHeadsContiguous ? ks * 2048 : (ks >> 2) * N * 128 + (ks & 3) * 32) / 16, idesc,
                                         (t > seg.t0 || ks > 0) ? 1u : 0u);
@@ -452,7 +462,10 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
     } else {
         // ================= softmax and output =================
         const int q = warp & 3;                 // TMEM lane quarter this warp may read
-        const int key = q * 32 + lane;          // key inside the tile = latent element inside a unit
+        const int elem = q * 32 + lane;         // latent element inside a unit = TMEM lane of O^T
+        // key inside the tile: a 64-row product sits in the first 16 lanes of every quarter
+        const int key = KT == 128 ? elem : q * 16 + (lane & 15);
+        const bool has_key = KT == 128 || lane < 16;
         const int st = static_cast<int>(threadIdx.x) - 64;   // 0..127
         const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(q * 32) << 16);
         const uint32_t p_key = p_base + static_cast<uint32_t>(key >> 6) * N * 128u + static_cast<uint32_t>(key & 7) * 2u;
@@ -461,7 +474,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
         int tiles = 0;
         float l[N];
         pdl_wait_prior();
-        while (!failed && next_segment(walk, p, seg)) {
+        while (!failed && next_segment<KT>(walk, p, seg)) {
 #pragma unroll
             for (int h = 0; h < N; ++h) l[h] = 0.f;
             if (st < N) s_ref[st] = -INFINITY;
@@ -472,7 +485,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                 tc_fence_after();
                 const uint32_t s_addr = lane_addr + kColS + static_cast<uint32_t>(buf) * 64u;
                 const uint32_t p_buf = p.p_bufs == 2 ? static_cast<uint32_t>(buf) * kPBytes : 0u;
-                const bool valid = t * kTileKeys + key < seg.len;
+                const bool valid = has_key && t * KT + key < seg.len;
                 // does any score outgrow its head's reference?
                 bool over = false;
 #pragma unroll
@@ -566,25 +579,28 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                     }
 #pragma unroll
                     for (int j = 0; j < 16; ++j) l[c * 16 + j] += w[j];
-                    if (kHeadsContiguous) {
+                    if (has_key) {
+                        if (kHeadsContiguous) {
 #pragma unroll
-                        for (int j = 0; j < 16; j += 8) {
-                            const uint32_t addr = swz128(p_base + p_buf + static_cast<uint32_t>(key) * 128u, c * 2 + j / 8);
-                            asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(addr), "r"(pack_bf16(w[j], w[j + 1])),
-                                         "r"(pack_bf16(w[j + 2], w[j + 3])), "r"(pack_bf16(w[j + 4], w[j + 5])),
-                                         "r"(pack_bf16(w[j + 6], w[j + 7]))
-                                         : "memory");
-                        }
-                    } else {
+                            for (int j = 0; j < 16; j += 8) {
+                                const uint32_t addr = swz128(p_base + p_buf + static_cast<uint32_t>(key) * 128u, c * 2 + j / 8);
+                                asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(addr), "r"(pack_bf16(w[j], w[j + 1])),
+                                             "r"(pack_bf16(w[j + 2], w[j + 3])), "r"(pack_bf16(w[j + 4], w[j + 5])),
+                                             "r"(pack_bf16(w[j + 6], w[j + 7]))
+                                             : "memory");
+                            }
+                        } else {
 #pragma unroll
-                        for (int j = 0; j < 16; ++j) {
-                            const int h = c * 16 + j;
-                            const __nv_bfloat16 b = __float2bfloat16_rn(w[j]);
-                            const uint32_t addr = p_key + p_buf + static_cast<uint32_t>(h) * 128u + ((p_chunk ^ (h & 7)) << 4);
-                            asm volatile("st.shared.b16 [%0], %1;" ::"r"(addr), "h"(*reinterpret_cast<const uint16_t*>(&b))
-                                         : "memory");
+                            for (int j = 0; j < 16; ++j) {
+                                const int h = c * 16 + j;
+                                const __nv_bfloat16 b = __float2bfloat16_rn(w[j]);
+                                const uint32_t addr = p_key + p_buf + static_cast<uint32_t>(h) * 128u + ((p_chunk ^ (h & 7)) << 4);
+                                asm volatile("st.shared.b16 [%0], %1;" ::"r"(addr), "h"(*reinterpret_cast<const uint16_t*>(&b))
+                                             : "memory");
+                            }
                         }
                     }
+                    __syncwarp();
                 }
                 fence_proxy_async_smem();
                 tc_fence_before();
@@ -621,7 +637,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
             }
             if (st == 0 && seg.starts) {
                 // the CTAs that share this item follow from its first tile's place in the sequence
-                const int nt = (seg.len + kTileKeys - 1) / kTileKeys;
+                const int nt = (seg.len + KT - 1) / KT;
                 const int first = g0 + tiles - (seg.t1 - seg.t0);
                 p.item_cta[2 * item] = static_cast<int>(blockIdx.x);
                 p.item_cta[2 * item + 1] = (first + nt - 1) / run;
@@ -637,7 +653,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                     tmem_ld_32x32b_x16(lane_addr + kColO + static_cast<uint32_t>(u * N + c * 16), ov);
                     tmem_ld_wait();
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) stage[j * kUnitElems + key] = __uint_as_float(ov[j]) * s_alpha[c * 16 + j];
+                    for (int j = 0; j < 16; ++j) stage[j * kUnitElems + elem] = __uint_as_float(ov[j]) * s_alpha[c * 16 + j];
                     softmax_sync();
                     // 16 heads x 128 elements, whole rows of a head at a time
                     if (whole) {
@@ -714,6 +730,27 @@ latent_merge_kernel(const LatentParams p, int N) {
         *reinterpret_cast<uint2*>(out + e) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
 }
 
+// The pool as [width / 64][num_slots][64], copied kpc slots and `halves` 64-element columns at a time.
+int make_latent_tmap(CUtensorMap* out, const void* cache, int width, int64_t num_slots, int kpc, int halves) {
+    EncodeTiledFn fn = encode_tiled_fn();
+    if (!fn) {
+        set_last_error("cuTensorMapEncodeTiled is not available from this driver");
+        return B200_ERR_CUDA;
+    }
+    const cuuint64_t dims[3] = {64, static_cast<cuuint64_t>(num_slots), static_cast<cuuint64_t>(width / 64)};
+    const cuuint64_t strides[2] = {static_cast<cuuint64_t>(width) * 2, 128};
+    const cuuint32_t box[3] = {64, static_cast<cuuint32_t>(kpc), static_cast<cuuint32_t>(halves)};
+    const cuuint32_t es[3] = {1, 1, 1};
+    CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(cache), dims, strides, box, es,
+                    CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                    CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) {
+        set_last_error("cuTensorMapEncodeTiled (latent pool) failed with CUresult %d", static_cast<int>(r));
+        return B200_ERR_CUDA;
+    }
+    return B200_OK;
+}
+
 struct Shape {
     int n, blocks, per_block;
 };
@@ -765,30 +802,35 @@ int launch_latent_attention_tc(const LatentAttention& a, int* status, cudaStream
     p.blocks = sh.blocks;
     p.per_block = sh.per_block;
     p.nb = a.width / kUnitElems;
-    p.kpc = a.page_size < kTileKeys ? a.page_size : kTileKeys;
+    const int kt = a.width > 256 ? 64 : 128;
+    p.kpc = a.page_size < kt ? a.page_size : kt;
     p.num_slots = a.num_slots;
     p.scale_log2 = a.scale * 1.4426950408889634f;
     p.early = a.only_last_key_new && pdl_launches_enabled() ? 1 : 0;
     p.status = status;
-    const uint32_t p_bytes = 2u * sh.n * 128u;
+    const uint32_t unit_bytes = static_cast<uint32_t>(kt) * 256u;
+    const uint32_t p_bytes = kt / 64 * sh.n * 128u;
     const uint32_t fixed = static_cast<uint32_t>(sh.n) * a.width * 2u + p_bytes + 16u * kUnitElems * 4u + 1024u;
     constexpr uint32_t kBudget = 224u * 1024u;
     int ring = kMaxUnits;
-    while (ring > p.nb && static_cast<uint32_t>(ring) * kUnitBytes + fixed > kBudget) --ring;
+    while (ring > p.nb && static_cast<uint32_t>(ring) * unit_bytes + fixed > kBudget) --ring;
     p.ring = ring;
-    uint32_t smem = static_cast<uint32_t>(ring) * kUnitBytes + fixed;
+    uint32_t smem = static_cast<uint32_t>(ring) * unit_bytes + fixed;
     p.p_bufs = smem + p_bytes <= kBudget ? 2 : 1;
     if (p.p_bufs == 2) smem += p_bytes;
 
     CUtensorMap tc, tq;
-    int err = cached_tmap(&tc, a.cache, static_cast<uint64_t>(a.width), static_cast<uint64_t>(a.num_slots),
-                          static_cast<uint64_t>(a.width) * 2, 64, static_cast<uint32_t>(p.kpc));
+    int err = make_latent_tmap(&tc, a.cache, a.width, a.num_slots, p.kpc, p.kpc == kt ? 2 : 1);
     if (err != B200_OK) return err;
     err = cached_tmap(&tq, a.q, static_cast<uint64_t>(a.width), static_cast<uint64_t>(a.rows) * a.heads,
                       static_cast<uint64_t>(a.width) * 2, 64, static_cast<uint32_t>(sh.n));
     if (err != B200_OK) return err;
-    auto kernel = sh.n == 16 ? latent_attention_tc_kernel<16> : sh.n == 32 ? latent_attention_tc_kernel<32>
-                                                                         : latent_attention_tc_kernel<64>;
+    auto kernel = kt == 64 ? (sh.n == 16   ? latent_attention_tc_kernel<16, 64>
+                              : sh.n == 32 ? latent_attention_tc_kernel<32, 64>
+                                           : latent_attention_tc_kernel<64, 64>)
+                           : (sh.n == 16   ? latent_attention_tc_kernel<16, 128>
+                              : sh.n == 32 ? latent_attention_tc_kernel<32, 128>
+                                           : latent_attention_tc_kernel<64, 128>);
     B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(grid), dim3(kThreads), smem, stream, dim3(1, 1, 1), tc, tq, p));
     B200_CHECK_CUDA(launch_kernel(latent_merge_kernel, dim3(a.rows * a.heads), dim3(128), 0, stream, dim3(1, 1, 1), p, sh.n));

@@ -104,10 +104,11 @@ __device__ __forceinline__ uint64_t kmajor_sw128_desc(uint32_t smem_addr) {
     return d;
 }
 
-// Instruction descriptor: bf16 x bf16 -> fp32, both operands K-major, M=128.
-__device__ __forceinline__ uint32_t idesc_bf16_m128(int n) {
+// Instruction descriptor: bf16 x bf16 -> fp32, both operands K-major.
+__device__ __forceinline__ uint32_t idesc_bf16(int m, int n) {
     return (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(n >> 3) << 17) |
-           (static_cast<uint32_t>(128 >> 4) << 24);
+           (static_cast<uint32_t>(m >> 4) << 24);
 }
+__device__ __forceinline__ uint32_t idesc_bf16_m128(int n) { return idesc_bf16(128, n); }
 
 }  // namespace b200
