@@ -1003,7 +1003,7 @@ int b200_engine_capture_graphs(b200_engine* e, const int32_t* batch_sizes, int c
             st.temperatures = variant ? &one : nullptr;   // non-NULL only switches the staging of sampling fields on
             int T = 0, max_ext = 0;
             B200_TRY(stage_step(e, &st, Bp, &T, &max_ext));
-            if (e->stack) B200_TRY(layer_stack_plan(e, &st, st.phase, Bp, T));
+            if (e->stack) B200_TRY(layer_stack_plan(e, &st, Bp));
             const size_t bytes = (variant ? b200_engine::step_index_offset(Bp) + 2 : 4 * Bp + 1) * sizeof(int32_t);
             B200_CHECK_CUDA(cudaMemcpyAsync(e->meta_dev, e->meta_host, bytes, cudaMemcpyHostToDevice, e->stream));
             B200_TRY(ensure_folded(e));
@@ -1065,7 +1065,7 @@ static int run_step(b200_engine* e, const b200_step* st, int32_t* next_tokens_ho
     const size_t meta_bytes =
         (sampling ? b200_engine::step_index_offset(Bg) + 2 : 4 * Bg + 1) * sizeof(int32_t);
     B200_CHECK_CUDA(cudaMemcpyAsync(e->meta_dev, e->meta_host, meta_bytes, cudaMemcpyHostToDevice, s));
-    if (e->stack) B200_TRY(layer_stack_plan(e, st, st->phase, Bg, T));
+    if (e->stack) B200_TRY(layer_stack_plan(e, st, Bg));
     B200_CHECK_CUDA(cudaEventRecord(e->ev_meta_done, s));
     e->meta_in_flight = true;
     // A captured graph covers all Bg rows; padded rows carry write_pos = -1 so nothing of

@@ -171,7 +171,7 @@ int layer_stack_create(b200_engine* e, const b200_stack_config* sc);
 void layer_stack_destroy(b200_engine* e);
 // Decides, on the host, which requests of a prefill step attend in the latent space and which through
 // expanded keys and values, and stages that plan behind the step's metadata copy.
-int layer_stack_plan(b200_engine* e, const b200_step* st, int phase, int Bp, int T);
+int layer_stack_plan(b200_engine* e, const b200_step* st, int Bp);
 // The layers on `T` tokens, as programmatic dependent launches if `pdl`; leaves the final-norm output in
 // stack_hidden().
 int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl);

@@ -18,7 +18,7 @@
 // are applied to the query and to the result.  Extensions of more than `expand_min` tokens expand keys and
 // values of the whole request once (two GEMMs) into a scratch that the prefill kernel of the
 // grouped-query models reads as if it were its paged pool.  A batch may hold both kinds of requests.
-#include <string.h>
+#include <stdlib.h>
 
 #include <string>
 #include <vector>
@@ -283,11 +283,11 @@ int32_t* stack_token_row(const b200_engine* e) { return e->stack->token_row; }
 int32_t* stack_token_len(const b200_engine* e) { return e->stack->token_len; }
 void stack_set_trace(b200_engine* e, float* host) { e->stack->trace = host; }
 
-int layer_stack_plan(b200_engine* e, const b200_step* st, int phase, int Bp, int T) {
+int layer_stack_plan(b200_engine* e, const b200_step* st, int Bp) {
     LayerStack* S = e->stack;
     S->plan_expanded = S->plan_latent = S->plan_max_extend = S->plan_max_len = 0;
     S->plan_rows = 0;
-    if (phase != B200_PHASE_PREFILL) return B200_OK;
+    if (st->phase != B200_PHASE_PREFILL) return B200_OK;
     int32_t* x_len = S->plan_host;
     int32_t* x_base = x_len + Bp;
     int32_t* g_base = x_base + Bp;
@@ -314,7 +314,6 @@ int layer_stack_plan(b200_engine* e, const b200_step* st, int phase, int Bp, int
     if (S->plan_expanded > 0)
         B200_CHECK_CUDA(cudaMemcpyAsync(S->plan_dev, S->plan_host, (3ll * Bp + S->plan_latent) * sizeof(int32_t),
                                         cudaMemcpyHostToDevice, e->stream));
-    (void)T;
     return B200_OK;
 }
 
@@ -406,7 +405,6 @@ int attend(b200_engine* e, const StackLayer& L, int phase, int Bp, int T) {
     S_TRY(launch_move_rows(S->qc, S->q, tokens, n, H * L.dp / 8, false, e->stream));
     S_TRY(attend_latent(e, L, S->ac, S->qc, S->compact_row, S->compact_len, n, false));
     return launch_move_rows(S->attn, S->ac, tokens, n, H * L.vp / 8, true, e->stream);
-    (void)T;
 }
 
 }  // namespace
