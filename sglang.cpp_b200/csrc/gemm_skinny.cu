@@ -684,6 +684,18 @@ static int env_int(const char* name, int dflt) {
     return (v && *v) ? atoi(v) : dflt;
 }
 
+// Split of `tiles` output tiles along K: at most one CTA per SM, and clusters of 8 only as many as the GPCs
+// hold at once with one CTA per SM (14 on B200; 16 of them ran in two waves: a [2048, 2048] projection took
+// 18 us with a split of 8 and 14 us with 4).
+static int cluster_split(int tiles, int kb_total) {
+    constexpr int kMaxClusters8 = 14;
+    int split = 1;
+    while (split < 8 && tiles * split * 2 <= sm_count() && split * 2 <= kb_total &&
+           (split < 4 || tiles <= kMaxClusters8))
+        split *= 2;
+    return split;
+}
+
 // K split of a slab: up to one CTA per SM in total, at most 8 ranks (portable cluster size).
 int skinny_gemm_split(int M, int N, int K, int epilogue) {
     (void)M;
@@ -694,10 +706,7 @@ int skinny_gemm_split(int M, int N, int K, int epilogue) {
     if (forced > 0) return forced;
     // One CTA per SM at most: a CTA holds its whole K slice plus the exchange buffer, so two
     // rarely fit on an SM, and a second wave would double the kernel's time.
-    int split = 1;
-    const int budget = sm_count();
-    while (split < 8 && n_tiles * split * 2 <= budget && split * 2 <= kb_total) split *= 2;
-    return split;
+    return cluster_split(n_tiles, kb_total);
 }
 
 // One slab of at most 256 rows.
@@ -855,8 +864,7 @@ int launch_linear_heads(void* y, const void* x, const void* w, int M, int heads,
     const int kb_total = K / kBlockK;
     const int n_tiles = div_ceil(N, kTileN);
     // the K split of the plain form, over all heads' tiles
-    int split = 1;
-    while (split < 8 && n_tiles * heads * split * 2 <= sm_count() && split * 2 <= kb_total) split *= 2;
+    const int split = cluster_split(n_tiles * heads, kb_total);
     const int kbp = div_ceil(kb_total, split);
     for (int m0 = 0; m0 < M; m0 += 256) {
         const int rows = M - m0 < 256 ? M - m0 : 256;

@@ -118,7 +118,7 @@ def read_rapizen(c: dict) -> StackConfig:
                 raise ValueError(f"layer {i}: unknown feed-forward {ff['kind']!r}")
         layers.append(spec)
     return StackConfig(c["width"], c["vocab"], float(c["norm"]["eps"]), layers, norm_offset=1.0,
-                       logit_scale=float(c["logit_scale"]))
+                       logit_scale=float(c.get("logit_scale", 1.0)))
 
 
 REGISTRY: dict[str, Callable] = {
