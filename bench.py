@@ -26,7 +26,8 @@ Other workloads (not the headline metric): --context N gives every prompt N toke
 of 4096 tokens prefilled in chunks, alternating with sampled decode steps of 56 running requests:
 prefill tokens/s, decode ms/step, fraction of the tensor-pipe rate); --workload c4 is Llama-3-8B under tensor parallelism and
 --workload c5 Qwen3-30B-A3B under expert parallelism + attention TP over the N ranks (strong
-scaling, weights drawn on the device); --eager / --profile-region / --profile-prefill shape a run
+scaling, weights drawn on the device); --workload rapizen is prefill and decode of the layer-stack
+design at three sizes beside Qwen3-MoE of the same sizes; --eager / --profile-region / --profile-prefill shape a run
 for a profiler's launch list.
 """
 from __future__ import annotations
