@@ -152,7 +152,14 @@ enum {
     B200_EPILOGUE_GEGLU = 2,     /* tanh-approximated GELU, as gelu_and_mul (src/layers/activation.cu:11-13) */
     B200_EPILOGUE_GEGLU_ERF = 3, /* exact GELU, as torch::gelu in MoELayer::forward (src/moe/moe.cc:80) */
     /* y[m, n] = max(acc[m, n], 0)^2, not gated: N outputs (no counterpart in the reference). */
-    B200_EPILOGUE_RELU2 = 4
+    B200_EPILOGUE_RELU2 = 4,
+    /* y[m, n] = gelu(acc[m, n]), exact, not gated: N outputs (no counterpart in the reference). */
+    B200_EPILOGUE_GELU_ERF = 5,
+    /* g = min(gate, limit), u = clamp(up, -limit, limit): y = g sigmoid(1.702 g) (u + 1); gated, with a
+     * limit beside it (no counterpart in the reference). */
+    B200_EPILOGUE_CLAMPED_SWIGLU = 6,
+    /* the fp32 accumulator itself: y is float [M, N] (no counterpart in the reference). */
+    B200_EPILOGUE_F32 = 7
 };
 
 /* LinearBase::forward (src/layers/linear.cc:24-26): y = x W^T (+ bias), bf16 in,
@@ -353,6 +360,103 @@ B200_API int b200_linear_f32(float* y, const float* x, const float* w, int max_r
                              int groups, const int32_t* counts, const int32_t* offsets, int epilogue,
                              b200_stream_t stream);
 
+/* b200_linear without a bias in either dtype, with the epilogues that take a limit (act_limit). */
+B200_API int b200_linear_act(void* y, const void* x, const void* w, int M, int N, int K, int epilogue,
+                             float act_limit, int dtype, b200_stream_t stream);
+
+/* The wiring with the norm on what a block returned:
+ *   a = sum_k src_weights[t, k] src[src_rows[t, k], :] + src2[t, :]   (src_rows NULL: src[t, :]; weights NULL: 1),
+ *   residual[t, :] += a / sqrt(mean(a^2) + eps) * add_weight          (add_weight NULL: += a; init: = instead of +=),
+ *   out[t, :] = residual, or its RMS norm with out_weight when there is one.
+ * Shapes as b200_residual_norm; every row of out is the token's own. */
+B200_API int b200_residual_post_norm(void* out, float* residual, const void* src, const int32_t* src_rows,
+                                     const float* src_weights, int src_top, int64_t src_count, const void* src2,
+                                     int init, const void* add_weight, const void* out_weight, int tokens,
+                                     int width, int padded, float eps, int dtype, b200_stream_t stream);
+
+/* Routing by sigmoid scores of fp32 logits [tokens, logits_ld]: only experts of the best keep_groups of
+ * `groups` equal groups (a group counts for the sum of its two best scores), the best `top` of those, weights =
+ * scores over their sum (+ 1e-20) times scale.  ids, weights, rows [tokens, top]: the chosen experts and the
+ * row each choice has in the expert-sorted order; counts [2 * experts] (the second half is scratch), offsets
+ * [experts + 1]; the token's row of x (row_bytes) is copied to its rows of xp. */
+B200_API int b200_score_route(int32_t* ids, float* weights, int32_t* rows, int32_t* counts, int32_t* offsets,
+                              void* xp, const void* x, int row_bytes, const float* logits, int64_t logits_ld,
+                              int tokens, int experts, int top, int groups, int keep_groups, float scale,
+                              b200_stream_t stream);
+
+/* What lies between the joint projection of an attention layer and the attention: joint [tokens, joint_ld]
+ * holds [heads * padded_dim | kv_heads * padded_dim | kv_heads * padded_value_dim | ...].  Queries (in place)
+ * and keys (to k_cache [num_slots, kv_heads, padded_dim]) are RMS-normalised over `dim` with q_norm / k_norm
+ * (NULL: not), then element i of the first rotary_dim turns with element i + rotary_dim / 2.  Values go to
+ * v_cache; mix 1 keeps a copy in first_values, mix 2 stores (1 - lambda) v + lambda first_values. */
+typedef struct b200_head_prepare_args {
+    void* joint;
+    int64_t joint_ld;
+    int32_t tokens, heads, kv_heads, dim, padded_dim, padded_value_dim;
+    const void *q_norm, *k_norm;
+    float eps;
+    int32_t rotary_dim, max_pos;
+    const float *cos_table, *sin_table;   /* [max_pos, rotary_dim / 2] */
+    const int32_t *positions, *out_loc;
+    void *k_cache, *v_cache;
+    int64_t num_slots;
+    int32_t mix;
+    const float* lambda;                  /* device */
+    void* first_values;                   /* [tokens, kv_heads, padded_value_dim] */
+} b200_head_prepare_args;
+B200_API int b200_head_prepare(const b200_head_prepare_args* args, int dtype, b200_stream_t stream);
+
+/* Paged grouped-query attention through a window: the query at position i sees key j <= i if i - j < window or
+ * j < keep_first.  out[t, h, :] = softmax(scale * q k) v, times sigmoid(gate[t, h, :]) when there is a gate.
+ * q: heads padded_dim apart; out [tokens, heads, padded_value_dim].  Requests by table_idx / seq_lens /
+ * qo_indptr (decode != 0: one token each), and per token its page-table row and the keys it could see without
+ * a window (row_table, row_len).  bf16 with both paddings 128 runs on the tensor-core kernels where they take
+ * the head counts, everything else (or plain != 0) on a plain kernel.
+ * workspace: b200_attention_decode_workspace_bytes, or any 16 bytes where that refuses the head counts. */
+typedef struct b200_window_attention_args {
+    void* out;
+    const void* q;
+    int64_t q_stride;
+    const void *k_cache, *v_cache;
+    int64_t num_slots;
+    const int32_t* page_table;
+    int64_t page_table_stride;
+    const int32_t *table_idx, *seq_lens, *qo_indptr, *row_table, *row_len;
+    int32_t tokens, batch, max_extend, decode, plain;
+    int32_t heads, kv_heads, padded_dim, padded_value_dim, page_size;
+    float scale;
+    int32_t window, keep_first;
+    const void* gate;
+    int64_t gate_stride;
+    void* workspace;
+    int64_t workspace_bytes;
+} b200_window_attention_args;
+B200_API int b200_window_attention(const b200_window_attention_args* args, int dtype, b200_stream_t stream);
+
+/* Gated linear attention with one decay per key channel.  Per head, with state S [dim, value dim]:
+ *   S <- diag(alpha) S + k v^T,   o = S^T (q * q_scale),   alpha = sigmoid(z)^(1 / tau),
+ *   z = a up^T + bias for the low-rank row a that the joint projection returns,
+ * and out = o / sqrt(mean(o^2) + eps) * norm * silu(gate) per head.  joint [tokens, joint_ld] holds
+ * [q | k: heads * padded_dim each | v | gate: heads * padded_value_dim each | a: padded rank]; up
+ * [heads * padded_dim, up_ld] of the dtype, bias fp32 [heads * padded_dim].  state fp32 [rows, heads, padded_dim,
+ * padded_value_dim]: row table_idx[b] belongs to request b, whose tokens are [qo_indptr[b], qo_indptr[b + 1])
+ * and whose first token has position cached[b]; a request that starts at position 0 starts from zeros.
+ * decode != 0: every request brings one token.  plain != 0: never the chunked tensor-core kernel. */
+typedef struct b200_linear_attention_args {
+    void* out;
+    const void* joint;
+    int64_t joint_ld;
+    int32_t tokens, batch, decode, plain;
+    const int32_t *table_idx, *cached, *qo_indptr;
+    float* state;
+    int32_t heads, dim, padded_dim, value_dim, padded_value_dim, rank, up_ld;
+    const void* up;
+    const float* bias;
+    const void* norm;
+    float tau, eps, q_scale;
+} b200_linear_attention_args;
+B200_API int b200_linear_attention(const b200_linear_attention_args* args, int dtype, b200_stream_t stream);
+
 /* ---- tensor-parallel all-reduce (include/sglang/distributed/distributed.h:24) --- */
 
 /* One process per GPU.  A communicator owns this rank's two exchange buffers (call parity 0 / 1)
@@ -476,23 +580,42 @@ typedef struct b200_engine b200_engine;
  * multiple of 64 (b200_pad_width; head and value dimensions up to 128 are padded to 128, latent widths
  * to a multiple of 128), vectors likewise; norms divide by the true width. */
 enum { B200_DTYPE_BF16 = 0, B200_DTYPE_F32 = 1 };
-enum { B200_MIXER_LATENT_ATTENTION = 0 };
-enum { B200_MLP_NONE = 0, B200_MLP_DENSE = 1, B200_MLP_TABLE_MOE = 2 };
+enum { B200_MIXER_LATENT_ATTENTION = 0, B200_MIXER_WINDOW_ATTENTION = 1, B200_MIXER_LINEAR_ATTENTION = 2 };
+enum { B200_MLP_NONE = 0, B200_MLP_DENSE = 1, B200_MLP_TABLE_MOE = 2, B200_MLP_SCORED_MOE = 3 };
 
 typedef struct b200_layer_config {
     int32_t mixer;         /* B200_MIXER_* */
     int32_t heads;
     int32_t head_dim;      /* query / key dimensions per head */
     int32_t value_dim;
-    int32_t q_rank;        /* width of the query latent */
-    int32_t kv_rank;       /* width of the key / value latent: what the cache holds per token */
+    int32_t q_rank;        /* latent attention: width of the query latent */
+    int32_t kv_rank;       /* latent attention: width of the key / value latent, what the cache holds per token */
     float score_scale;
     int32_t mlp;           /* B200_MLP_* */
     int32_t intermediate;  /* of the dense layer, or of each expert */
     int32_t epilogue;      /* B200_EPILOGUE_*: what is between the up and the down projection; a gated one
                               has gate and up stacked in "mlp_up" */
     int32_t num_experts;
-    int32_t experts_per_tok; /* width of the token-id -> experts table; each chosen expert weighs 1 / that */
+    int32_t experts_per_tok; /* table: width of the token-id -> experts table, each chosen expert weighs 1 / that;
+                                scored: experts with the largest scores */
+    /* window attention */
+    int32_t kv_heads;
+    int32_t window;          /* the query at position i sees key j <= i if i - j < window ... */
+    int32_t keep_first;      /* ... or j < keep_first */
+    int32_t rotary_dim;
+    double rope_base;
+    int32_t value_mix;       /* values mixed with those of the first layer that has this set */
+    /* linear attention */
+    int32_t decay_rank;
+    float decay_tau;
+    /* scored experts */
+    int32_t router_groups;
+    int32_t router_keep;     /* groups whose experts can be chosen */
+    float router_scale;
+    int32_t shared_intermediate; /* of the expert every token uses; 0: none */
+    /* limits of B200_EPILOGUE_CLAMPED_SWIGLU */
+    float act_limit;
+    float shared_act_limit;
 } b200_layer_config;
 
 typedef struct b200_stack_config {
@@ -501,6 +624,8 @@ typedef struct b200_stack_config {
     int32_t dtype;       /* B200_DTYPE_*: bf16 matrices and activations, or everything in fp32 */
     float norm_offset;   /* added to the stored weights of the layer norms and the final norm (0 or 1) */
     float logit_scale;
+    int32_t norm_output; /* 0: blocks read the normalised residual; 1: they read the residual, and what they
+                            return is normalised before it is added */
 } b200_stack_config;
 
 /* The padded size of a width / of a per-head dimension / of a latent width (see above). */
@@ -515,8 +640,8 @@ B200_API int b200_pad_latent(int n);
 B200_API int b200_engine_create(const b200_model_config* model, const b200_engine_config* config,
                                 b200_engine** out);
 /* The same for a model whose layers are listed one by one; of `model` only num_layers, hidden_size,
- * vocab_size, rms_norm_eps and tie_word_embeddings are read.  One latent pool per layer
- * [(num_pages+1)*page_size, pad(kv_rank)] stands where the K/V pools are.  tp_size must be 1. */
+ * vocab_size, rms_norm_eps and tie_word_embeddings are read.  Per layer a latent pool
+ * [(num_pages+1)*page_size, pad(kv_rank)], a K and a V pool, or a state per table row.  tp_size must be 1. */
 B200_API int b200_engine_create_stack(const b200_model_config* model, const b200_stack_config* stack,
                                       const b200_engine_config* config, b200_engine** out);
 B200_API int b200_engine_destroy(b200_engine* engine);
@@ -529,7 +654,12 @@ B200_API int b200_engine_destroy(b200_engine* engine);
  * "kv_latent_norm", "uq" [heads*dim, q latent], "uk" [heads*dim, kv latent], "uk_absorb" (per head the
  * transpose of its rows of uk: [heads, kv latent, dim]), "uv" [heads*vdim, kv latent], "o"
  * [hidden, heads*vdim], "mlp_up", "mlp_down" (experts stacked), "expert_table" int32 [vocab, experts
- * per token], "latent_cache". */
+ * per token], "latent_cache".  Window attention: "qkvg" [heads*dim + kv_heads*dim + kv_heads*vdim + heads*vdim,
+ * hidden], "q_head_norm", "k_head_norm" [dim], "value_mix" (one float), "o", "k_cache", "v_cache".  Linear
+ * attention (dimensions padded to a multiple of 64): "qkvga" [2 heads*dim + 2 heads*vdim + rank, hidden],
+ * "decay_up" [heads*dim, rank padded to 16], "decay_bias" fp32 [heads*dim], "head_norm" [vdim], "o",
+ * "state" fp32 [max_running_req + 1, heads, dim, vdim].  Scored experts: "router" [experts, hidden],
+ * "mlp_up", "mlp_down", "shared_up", "shared_down". */
 B200_API int b200_engine_tensor(b200_engine* engine, const char* name, int layer, void** device_ptr,
                                 int64_t* nbytes);
 /* Synchronous host-to-device copy into a named tensor (nbytes must equal its size). */

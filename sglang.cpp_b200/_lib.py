@@ -28,10 +28,18 @@ EPILOGUE_NONE = 0
 EPILOGUE_SWIGLU = 1
 EPILOGUE_GEGLU = 2
 EPILOGUE_RELU2 = 4
+EPILOGUE_GELU_ERF = 5
+EPILOGUE_CLAMPED_SWIGLU = 6
+EPILOGUE_F32 = 7
 
 DTYPE_BF16, DTYPE_F32 = 0, 1
-MIXER_LATENT_ATTENTION = 0
-MLP_NONE, MLP_DENSE, MLP_TABLE_MOE = 0, 1, 2
+MIXER_LATENT_ATTENTION, MIXER_WINDOW_ATTENTION, MIXER_LINEAR_ATTENTION = 0, 1, 2
+MLP_NONE, MLP_DENSE, MLP_TABLE_MOE, MLP_SCORED_MOE = 0, 1, 2, 3
+
+
+def epilogue_is_gated(epilogue: int) -> bool:
+    """Does the activation take two stacked halves (gate, up)?"""
+    return epilogue not in (EPILOGUE_NONE, EPILOGUE_RELU2, EPILOGUE_GELU_ERF, EPILOGUE_F32)
 
 
 class B200Error(RuntimeError):
@@ -103,6 +111,12 @@ PROTOTYPES: dict[str, tuple] = {
     "b200_table_route": (_I, [_P, _P, _P, _P, _P, _I, _I, _I, _I, _P]),
     "b200_linear_heads": (_I, [_P, _P, _P, _I, _I, _I, _I, _P]),
     "b200_linear_f32": (_I, [_P, _P, _P, _I, _I, _I, _I, _P, _P, _I, _P]),
+    "b200_linear_act": (_I, [_P, _P, _P, _I, _I, _I, _I, _F, _I, _P]),
+    "b200_residual_post_norm": (_I, [_P, _P, _P, _P, _P, _I, _L, _P, _I, _P, _P, _I, _I, _I, _F, _I, _P]),
+    "b200_score_route": (_I, [_P, _P, _P, _P, _P, _P, _P, _I, _P, _L, _I, _I, _I, _I, _I, _F, _P]),
+    "b200_head_prepare": (_I, [_P, _I, _P]),
+    "b200_window_attention": (_I, [_P, _I, _P]),
+    "b200_linear_attention": (_I, [_P, _I, _P]),
     "b200_pad_width": (_I, [_I]),
     "b200_pad_head_dim": (_I, [_I]),
     "b200_pad_latent": (_I, [_I]),
@@ -149,7 +163,45 @@ class LayerConfigStruct(ctypes.Structure):
         ("mixer", c_int32), ("heads", c_int32), ("head_dim", c_int32), ("value_dim", c_int32),
         ("q_rank", c_int32), ("kv_rank", c_int32), ("score_scale", c_float), ("mlp", c_int32),
         ("intermediate", c_int32), ("epilogue", c_int32), ("num_experts", c_int32),
-        ("experts_per_tok", c_int32),
+        ("experts_per_tok", c_int32), ("kv_heads", c_int32), ("window", c_int32), ("keep_first", c_int32),
+        ("rotary_dim", c_int32), ("rope_base", ctypes.c_double), ("value_mix", c_int32),
+        ("decay_rank", c_int32), ("decay_tau", c_float), ("router_groups", c_int32), ("router_keep", c_int32),
+        ("router_scale", c_float), ("shared_intermediate", c_int32), ("act_limit", c_float),
+        ("shared_act_limit", c_float),
+    ]
+
+
+class HeadPrepareArgs(ctypes.Structure):
+    """b200_head_prepare_args."""
+    _fields_ = [
+        ("joint", _P), ("joint_ld", _L), ("tokens", c_int32), ("heads", c_int32), ("kv_heads", c_int32),
+        ("dim", c_int32), ("padded_dim", c_int32), ("padded_value_dim", c_int32), ("q_norm", _P), ("k_norm", _P),
+        ("eps", c_float), ("rotary_dim", c_int32), ("max_pos", c_int32), ("cos_table", _P), ("sin_table", _P),
+        ("positions", _P), ("out_loc", _P), ("k_cache", _P), ("v_cache", _P), ("num_slots", _L), ("mix", c_int32),
+        ("lambda_", _P), ("first_values", _P),
+    ]
+
+
+class WindowAttentionArgs(ctypes.Structure):
+    """b200_window_attention_args."""
+    _fields_ = [
+        ("out", _P), ("q", _P), ("q_stride", _L), ("k_cache", _P), ("v_cache", _P), ("num_slots", _L),
+        ("page_table", _P), ("page_table_stride", _L), ("table_idx", _P), ("seq_lens", _P), ("qo_indptr", _P),
+        ("row_table", _P), ("row_len", _P), ("tokens", c_int32), ("batch", c_int32), ("max_extend", c_int32),
+        ("decode", c_int32), ("plain", c_int32), ("heads", c_int32), ("kv_heads", c_int32), ("padded_dim", c_int32),
+        ("padded_value_dim", c_int32), ("page_size", c_int32), ("scale", c_float), ("window", c_int32),
+        ("keep_first", c_int32), ("gate", _P), ("gate_stride", _L), ("workspace", _P), ("workspace_bytes", _L),
+    ]
+
+
+class LinearAttentionArgs(ctypes.Structure):
+    """b200_linear_attention_args."""
+    _fields_ = [
+        ("out", _P), ("joint", _P), ("joint_ld", _L), ("tokens", c_int32), ("batch", c_int32), ("decode", c_int32),
+        ("plain", c_int32), ("table_idx", _P), ("cached", _P), ("qo_indptr", _P), ("state", _P), ("heads", c_int32),
+        ("dim", c_int32), ("padded_dim", c_int32), ("value_dim", c_int32), ("padded_value_dim", c_int32),
+        ("rank", c_int32), ("up_ld", c_int32), ("up", _P), ("bias", _P), ("norm", _P), ("tau", c_float),
+        ("eps", c_float), ("q_scale", c_float),
     ]
 
 
@@ -157,7 +209,7 @@ class StackConfigStruct(ctypes.Structure):
     """b200_stack_config."""
     _fields_ = [
         ("num_layers", c_int32), ("layers", POINTER(LayerConfigStruct)), ("dtype", c_int32),
-        ("norm_offset", c_float), ("logit_scale", c_float),
+        ("norm_offset", c_float), ("logit_scale", c_float), ("norm_output", c_int32),
     ]
 
 

@@ -23,6 +23,9 @@
 //   * every warp writes an (m, l, O) partial (or, for a request that is a single partial, bf16
 //     outputs at once); a second, tiny kernel merges the partials of every request, one warp per
 //     (request, query head), so the streaming kernel ends with its last stage.
+// WINDOW: a sliding window with kept first keys.  A request's stages are then those that hold a kept key and
+// those from the oldest key in the window on; what lies between is never loaded.  The output passes a sigmoid
+// gate where it is written as bf16.
 #include <mutex>
 
 #include "common.cuh"
@@ -63,16 +66,37 @@ struct DecodeParams {
     int max_items;
     int* status;
     int kv_evict_first;   // stream K/V through L2 with the evict-first policy (read once per step)
+    int window, keep_first;       // 0x7fffffff, 0 without a window
+    const __nv_bfloat16* gate;    // WINDOW only
+    int64_t gate_st;
 };
+
+// Which stages of a request of `len` keys are read: stage numbers [0, head) and, `skip` further, [head, count).
+struct StageRange {
+    int count, head, skip;
+};
+__device__ __forceinline__ StageRange stage_range(int len, int stage_keys, int window, int keep_first) {
+    len = max(len, 0);
+    StageRange r;
+    r.head = (min(keep_first, len) + stage_keys - 1) / stage_keys;
+    r.skip = max(0, max(0, len - window) / stage_keys - r.head);
+    r.count = (len + stage_keys - 1) / stage_keys - r.skip;
+    return r;
+}
+__device__ __forceinline__ uint32_t gate_pair(uint32_t g, float lo, float hi) {
+    return pack_bf16(lo * sigmoid_f(bf16_lo(g)), hi * sigmoid_f(bf16_hi(g)));
+}
 
 struct ItemInfo {
     int b, len, s_begin, s_end, nchunks, item, first_slot;
+    int head, skip;   // stage_range
 };
 
 __device__ __forceinline__ void consumer_bar() {
     asm volatile("bar.sync 1, %0;" ::"n"(kConsumerThreads) : "memory");
 }
 
+template <bool WINDOW>
 __global__ void __launch_bounds__(kThreads, 1)
 attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
                         const __grid_constant__ CUtensorMap tmap_v, const DecodeParams p) {
@@ -117,7 +141,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
         int carry = 0;
         for (int base = 0; base < B; base += 32) {
             const int b = base + lane;
-            const int n = b < B ? (max(p.seq_lens[b], 0) + SK - 1) / SK : 0;
+            const int n = b < B ? stage_range(p.seq_lens[b], SK, p.window, p.keep_first).count : 0;
             int incl = n;
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -161,6 +185,9 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
         it.nchunks = (first + st - 1) / per - c0 + 1;   // CTAs that share this request
         it.first_slot = lo + c0;
         it.item = lo + static_cast<int>(blockIdx.x);
+        const StageRange range = stage_range(it.len, SK, p.window, p.keep_first);
+        it.head = range.head;
+        it.skip = range.skip;
         return it;
     };
 
@@ -178,14 +205,17 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
             const ItemInfo it = locate(gpos);
             gpos += it.s_end - it.s_begin;
             const int32_t* pt_row = p.page_table + static_cast<int64_t>(p.table_idx[it.b]) * p.pt_stride;
-            const int first_key = it.s_begin * SK;
-            const int item_keys = min(it.len, it.s_end * SK) - first_key;
-            const int item_copies = (item_keys + p.kpc - 1) / p.kpc;
+            auto stage_key = [&](int st) { return (WINDOW && st >= it.head ? st + it.skip : st) * SK; };
+            const int cps = SK / p.kpc;   // copies of a whole stage, a power of two
+            const int cps_shift = 31 - __clz(cps);
+            const int item_copies = (it.s_end - it.s_begin) * cps;
             // Slot of the first key of every copy of this item (the previous item's
             // table is no longer needed: all of its copies have been issued).
             __syncwarp();
-            for (int c = lane; c < min(item_copies, kSlotTab); c += 32)
-                s_slot_tab[c] = pt_row[first_key + c * p.kpc];
+            for (int c = lane; c < min(item_copies, kSlotTab); c += 32) {
+                const int key = stage_key(it.s_begin + (c >> cps_shift)) + (c & (cps - 1)) * p.kpc;
+                s_slot_tab[c] = key < it.len ? pt_row[key] : 0;
+            }
             __syncwarp();
             for (int st = it.s_begin; st < it.s_end; ++st, ++it_count) {
                 const uint32_t slot = it_count % kStages;
@@ -194,7 +224,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
                     failed = true;
                     break;
                 }
-                const int k0 = st * SK;
+                const int k0 = stage_key(st);
                 const int valid = min(SK, it.len - k0);
                 const int ncopies = (valid + p.kpc - 1) / p.kpc;
                 if (!waited && k0 + valid >= it.len) {  // this stage holds the key written just now
@@ -207,7 +237,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
                 const uint32_t stage_base = smem_base + slot * kStageBytes;
                 for (int ci = lane; ci < ncopies * 4; ci += 32) {
                     const int copy = ci >> 2, which = ci & 3;
-                    const int tab = (k0 - first_key) / p.kpc + copy;
+                    const int tab = (st - it.s_begin) * cps + copy;
                     int64_t sl = tab < kSlotTab ? s_slot_tab[tab] : pt_row[k0 + copy * p.kpc];
                     if (sl < 0 || sl + p.kpc > p.num_slots) {
                         atomicExch(&p.status[kStatusBadIndex], static_cast<int>(sl) + 1);
@@ -270,8 +300,11 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
             const uint32_t parity = (it_count / kStages) & 1u;
             if (!failed && !mbar_wait_bounded(smem_u32(&full_bar[slot]), parity, p.status, 202))
                 failed = true;
-            const int nvalid = it.len - (st * SK + kg * 16);  // valid keys in this warp's tile
-            if (!failed && nvalid > 0) {
+            const int key0 = (WINDOW && st >= it.head ? st + it.skip : st) * SK + kg * 16;   // first key of this warp's tile
+            const int nvalid = it.len - key0;  // valid keys in it
+            const int oldest = it.len - p.window;
+            const bool seen = !WINDOW || key0 + min(nvalid, 16) > oldest || key0 < p.keep_first;
+            if (!failed && nvalid > 0 && seen) {
                 const uint32_t stage_base = smem_base + slot * kStageBytes;
                 // Row of key j (0..15 of this warp's tile) inside a half tile.  A copy of
                 // kpc keys lands as [head][key] rows, so the keys of one head are adjacent
@@ -314,7 +347,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
                 for (int e = 0; e < 8; ++e) {
                     const float v = (e < 4 ? s0[e] : s1[e - 4]) * p.scale_log2;
                     const int key = (e >> 2) * 8 + 2 * t + (e & 1);
-                    x[e] = key < nvalid ? v : -INFINITY;
+                    const bool sees = key < nvalid && (!WINDOW || key0 + key >= oldest || key0 + key < p.keep_first);
+                    x[e] = sees ? v : -INFINITY;
                 }
                 float mx0 = fmaxf(fmaxf(x[0], x[1]), fmaxf(x[4], x[5]));
                 float mx1 = fmaxf(fmaxf(x[2], x[3]), fmaxf(x[6], x[7]));
@@ -322,7 +356,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
                 mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
                 mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
                 mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
-                const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);  // finite: key 0 is valid
+                const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);  // finite: a key of the tile is seen
                 const float al0 = exp2f(m0 - mn0), al1 = exp2f(m1 - mn1);
                 m0 = mn0;
                 m1 = mn1;
@@ -388,9 +422,14 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
                     const float inv = l > 0.f ? 1.f / l : 0.f;
                     __nv_bfloat16* dst = p.out + (static_cast<int64_t>(it.b) * Hq + h * G + row) * kD;
 #pragma unroll
-                    for (int i = 0; i < 16; ++i)
-                        *reinterpret_cast<uint32_t*>(dst + i * 8 + 2 * t) =
-                            pack_bf16(o[i][2 * rr] * inv, o[i][2 * rr + 1] * inv);
+                    for (int i = 0; i < 16; ++i) {
+                        const float a = o[i][2 * rr] * inv, b = o[i][2 * rr + 1] * inv;
+                        uint32_t packed = pack_bf16(a, b);
+                        if (WINDOW && p.gate != nullptr)
+                            packed = gate_pair(*reinterpret_cast<const uint32_t*>(p.gate + it.b * p.gate_st + (h * G + row) * kD +
+                                                                                  i * 8 + 2 * t), a, b);
+                        *reinterpret_cast<uint32_t*>(dst + i * 8 + 2 * t) = packed;
+                    }
                 }
             }
         } else {
@@ -438,7 +477,7 @@ attention_decode_merge_kernel(const DecodeParams p, int attn_grid) {
         int carry = 0, first = 0, mine = 0;
         for (int base = 0; base < p.batch; base += 32) {
             const int r = base + lane;
-            const int n = r < p.batch ? (max(p.seq_lens[r], 0) + SK - 1) / SK : 0;
+            const int n = r < p.batch ? stage_range(p.seq_lens[r], SK, p.window, p.keep_first).count : 0;
             int incl = n;
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -482,7 +521,7 @@ attention_decode_merge_kernel(const DecodeParams p, int attn_grid) {
         for (int j = 0; j < 8; ++j)
             rows[j] = j < n ? __ldcg(reinterpret_cast<const float4*>(po + (base + j) * o_stride))
                             : make_float4(0.f, 0.f, 0.f, 0.f);
-        const float Mc = fmaxf(M, warp_max(mine.x));   // finite: a request's first partial holds key 0
+        const float Mc = fmaxf(M, warp_max(mine.x));   // finite: a request's first stage holds a key that is seen
         const float rescale = exp2f(M - Mc);           // 0 on the first chunk (M = -inf)
         acc.x *= rescale;
         acc.y *= rescale;
@@ -514,6 +553,11 @@ attention_decode_merge_kernel(const DecodeParams p, int attn_grid) {
     uint2 packed;
     packed.x = pack_bf16(acc.x * inv, acc.y * inv);
     packed.y = pack_bf16(acc.z * inv, acc.w * inv);
+    if (p.gate != nullptr) {
+        const uint2 g = *reinterpret_cast<const uint2*>(p.gate + b * p.gate_st + head * kD + lane * 4);
+        packed.x = gate_pair(g.x, acc.x * inv, acc.y * inv);
+        packed.y = gate_pair(g.y, acc.z * inv, acc.w * inv);
+    }
     *reinterpret_cast<uint2*>(p.out + (static_cast<int64_t>(b) * Hq + head) * kD + lane * 4) = packed;
 }
 
@@ -531,7 +575,7 @@ int launch_attention_decode(void* out, const void* q, int64_t q_st, int64_t q_sh
                             const int32_t* page_table, int64_t pt_stride, const int32_t* table_idx,
                             const int32_t* seq_lens, int batch, int q_heads, int kv_heads,
                             int page_size, float sm_scale, void* workspace, int64_t workspace_bytes,
-                            int* status, cudaStream_t stream, bool kv_evict_first) {
+                            int* status, cudaStream_t stream, bool kv_evict_first, const AttentionWindow* window) {
     const int kg = kConsumerWarps / kv_heads;
     const int grid = sm_count();
     // Workspace layout: ws_ml | ws_o
@@ -569,12 +613,16 @@ int launch_attention_decode(void* out, const void* q, int64_t q_st, int64_t q_sh
     p.max_items = static_cast<int>(max_items < (1 << 30) ? max_items : (1 << 30));
     p.status = status;
     p.kv_evict_first = kv_evict_first ? 1 : 0;
+    p.window = window ? window->size : 0x7fffffff;
+    p.keep_first = window ? window->keep_first : 0;
+    p.gate = window ? static_cast<const __nv_bfloat16*>(window->gate) : nullptr;
+    p.gate_st = window ? window->gate_st : 0;
+    auto kernel = window ? attention_decode_kernel<true> : attention_decode_kernel<false>;
 
     const int smem = kStages * kStageBytes + 1024;
     // The attribute belongs to (function, device): set it on every launch, as the other launchers do.
-    B200_CHECK_CUDA(cudaFuncSetAttribute(attention_decode_kernel,
-                                         cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-    B200_CHECK_CUDA(launch_kernel(attention_decode_kernel, dim3(grid), dim3(kThreads), smem, stream,
+    B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    B200_CHECK_CUDA(launch_kernel(kernel, dim3(grid), dim3(kThreads), smem, stream,
                                   dim3(1, 1, 1), tmap_k, tmap_v, p));
     const int merge_ctas = batch * ((q_heads + kMergeWarps - 1) / kMergeWarps);
     B200_CHECK_CUDA(launch_kernel(attention_decode_merge_kernel, dim3(merge_ctas), dim3(kMergeWarps * 32), 0, stream,

@@ -20,6 +20,9 @@
 // TMEM lane; warps w and w+4 of a group share a lane quarter and take keys 0-63 / 64-127).
 // Queries are the LAST extend_len positions of the request, so tiles left of the diagonal need no mask
 // and tiles right of it are never loaded.
+//
+// WINDOW: a sliding window with kept first keys (tiles that no row of the block sees are never loaded; the
+// tiles at the window's edges are masked per element) and a sigmoid gate on the output.
 #include "common.cuh"
 #include "kernels.h"
 #include "tcgen05.cuh"
@@ -55,6 +58,9 @@ struct PrefillTc2Params {
     int64_t num_slots;
     float scale_log2;
     int* status;
+    int window, keep_first;     // WINDOW only
+    const __nv_bfloat16* gate;
+    int64_t gate_st;
 };
 
 // MN-major operand under the 128-byte swizzle (V as the B operand of P V: rows are keys, 64 head-dim
@@ -96,6 +102,7 @@ __device__ __forceinline__ void tmem_st_32x32b_x32(uint32_t taddr, const uint32_
         "r"(v[25]), "r"(v[26]), "r"(v[27]), "r"(v[28]), "r"(v[29]), "r"(v[30]), "r"(v[31])
         : "memory");
 }
+template <bool WINDOW>
 __global__ void __launch_bounds__(kThreads, 1)
 attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
                              const __grid_constant__ CUtensorMap tmap_v,
@@ -134,7 +141,11 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
     const int t_end = min(t0 + 2 * QB, ext);
     const int pos0 = len - ext;                   // position of query token 0
     const int kv_end = min(len, pos0 + t_end);    // keys [0, kv_end) are visible to this block
-    const int ntiles = (kv_end + kTile - 1) / kTile;
+    // tiles [0, head_tiles) and, `skip` tiles further, those from the oldest key that the first row sees
+    const int head_tiles = WINDOW ? (min(p.keep_first, kv_end) + kTile - 1) / kTile : 0;
+    const int skip = WINDOW ? max(0, max(0, pos0 + t0 - p.window + 1) / kTile - head_tiles) : 0;
+    const int ntiles = (kv_end + kTile - 1) / kTile - skip;
+    auto first_key = [&](int kt) { return (WINDOW && kt >= head_tiles ? kt + skip : kt) * kTile; };
 
     if (threadIdx.x == 0) {
         for (int s = 0; s < kStages; ++s) {
@@ -195,7 +206,7 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
         for (int kt = 0; kt < ntiles && !failed; ++kt) {
             const uint32_t slot = kt % kStages;
             const uint32_t parity = static_cast<uint32_t>(kt / kStages - 1) & 1u;
-            const int k0 = kt * kTile;
+            const int k0 = first_key(kt);
             const int valid = min(kTile, kv_end - k0);
             const int ncopies = (valid + p.kpc - 1) / p.kpc;
             const uint32_t stage_base = smem_base + kKVOff + slot * kStageBytes;
@@ -322,6 +333,8 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
         const int tok = t0 + tile * QB + r / G;
         const int head = h * G + r % G;
         const int limit = min(pos0 + tok, len - 1);   // last visible key of this row
+        const int oldest = WINDOW ? limit - p.window + 1 : 0;   // keys before it are seen below keep_first only
+        auto sees = [&](int k) { return k <= limit && (!WINDOW || k >= oldest || k < p.keep_first); };
         const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(qtr * 32) << 16);
         const uint32_t s_addr = lane_addr + kColS + static_cast<uint32_t>(tile) * 128u + static_cast<uint32_t>(half * 64);
         const uint32_t o_addr = lane_addr + kColO + static_cast<uint32_t>(tile) * 128u + static_cast<uint32_t>(half * 64);
@@ -341,9 +354,10 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
             if (!failed && !mbar_wait_bounded(smem_u32(&s_full[tile]), static_cast<uint32_t>(kt) & 1u, p.status, 324))
                 failed = true;
             tc_fence_after();
-            const int k0 = kt * kTile + half * 64;    // first key of this thread's columns
+            const int k0 = first_key(kt) + half * 64;    // first key of this thread's columns
             // (masking is decided per warp, so that the common case carries no per-element tests at all)
-            const bool need_mask = __any_sync(0xffffffffu, k0 + 63 > limit);
+            const bool need_mask =
+                __any_sync(0xffffffffu, k0 + 63 > limit || (WINDOW && k0 < oldest && k0 + 63 >= p.keep_first));
             // pass 1: the maximum of this thread's 64 scores (both loads in flight before the first wait)
             float mx = -INFINITY;
             {
@@ -354,8 +368,8 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
                 if (need_mask) {
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
-                        if (k0 + i <= limit) mx = fmaxf(mx, __uint_as_float(sa[i]));
-                        if (k0 + 32 + i <= limit) mx = fmaxf(mx, __uint_as_float(sb[i]));
+                        if (sees(k0 + i)) mx = fmaxf(mx, __uint_as_float(sa[i]));
+                        if (sees(k0 + 32 + i)) mx = fmaxf(mx, __uint_as_float(sb[i]));
                     }
                 } else {
                     float m0 = -INFINITY, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;
@@ -411,8 +425,8 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
                     for (int i = 0; i < 32; i += 2) {
                         float p0 = ex2(fmaf(__uint_as_float(sv[i]), sc, -mb));
                         float p1 = ex2(fmaf(__uint_as_float(sv[i + 1]), sc, -mb));
-                        if (k0 + c * 32 + i > limit) p0 = 0.f;
-                        if (k0 + c * 32 + i + 1 > limit) p1 = 0.f;
+                        if (!sees(k0 + c * 32 + i)) p0 = 0.f;
+                        if (!sees(k0 + c * 32 + i + 1)) p1 = 0.f;
                         sum0 += p0;
                         sum1 += p1;
                         packed[i >> 1] = pack_bf16(p0, p1);
@@ -455,12 +469,27 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
                 tmem_ld_32x32b_x32(o_addr + c * 32, ov);
                 tmem_ld_wait();
 #pragma unroll
+                for (int i = 0; i < 32; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * inv);
+                if (WINDOW && p.gate != nullptr && store) {
+                    const uint4* gate = reinterpret_cast<const uint4*>(p.gate + (q_begin + tok) * p.gate_st + head * kD + half * 64);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        const uint4 g4 = gate[c * 4 + j];
+                        const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) {
+                            ov[j * 8 + 2 * i] = __float_as_uint(__uint_as_float(ov[j * 8 + 2 * i]) * sigmoid_f(bf16_lo(gw[i])));
+                            ov[j * 8 + 2 * i + 1] = __float_as_uint(__uint_as_float(ov[j * 8 + 2 * i + 1]) * sigmoid_f(bf16_hi(gw[i])));
+                        }
+                    }
+                }
+#pragma unroll
                 for (int j = 0; j < 4; ++j) {
                     uint4 w;
-                    w.x = pack_bf16(__uint_as_float(ov[j * 8 + 0]) * inv, __uint_as_float(ov[j * 8 + 1]) * inv);
-                    w.y = pack_bf16(__uint_as_float(ov[j * 8 + 2]) * inv, __uint_as_float(ov[j * 8 + 3]) * inv);
-                    w.z = pack_bf16(__uint_as_float(ov[j * 8 + 4]) * inv, __uint_as_float(ov[j * 8 + 5]) * inv);
-                    w.w = pack_bf16(__uint_as_float(ov[j * 8 + 6]) * inv, __uint_as_float(ov[j * 8 + 7]) * inv);
+                    w.x = pack_bf16(__uint_as_float(ov[j * 8 + 0]), __uint_as_float(ov[j * 8 + 1]));
+                    w.y = pack_bf16(__uint_as_float(ov[j * 8 + 2]), __uint_as_float(ov[j * 8 + 3]));
+                    w.z = pack_bf16(__uint_as_float(ov[j * 8 + 4]), __uint_as_float(ov[j * 8 + 5]));
+                    w.w = pack_bf16(__uint_as_float(ov[j * 8 + 6]), __uint_as_float(ov[j * 8 + 7]));
                     if (store) dst[c * 4 + j] = w;
                 }
             }
@@ -499,7 +528,7 @@ int launch_attention_prefill_tc2(void* out, const void* q, int64_t q_st, int64_t
                                  int64_t pt_stride, const int32_t* table_idx, const int32_t* seq_lens,
                                  const int32_t* qo_indptr, int batch, int max_extend_len, int q_heads,
                                  int kv_heads, int page_size, float sm_scale, int* status,
-                                 cudaStream_t stream) {
+                                 cudaStream_t stream, const AttentionWindow* window) {
     if (batch == 0 || max_extend_len == 0) return B200_OK;
     PrefillTc2Params p;
     p.out = static_cast<__nv_bfloat16*>(out);
@@ -518,6 +547,10 @@ int launch_attention_prefill_tc2(void* out, const void* q, int64_t q_st, int64_t
     p.num_slots = num_slots;
     p.scale_log2 = sm_scale * 1.4426950408889634f;
     p.status = status;
+    p.window = window ? window->size : 0x7fffffff;
+    p.keep_first = window ? window->keep_first : 0;
+    p.gate = window ? static_cast<const __nv_bfloat16*>(window->gate) : nullptr;
+    p.gate_st = window ? window->gate_st : 0;
     CUtensorMap tk, tv;
     int err = make_kv_tmap_3d_tc2(&tk, k_cache, num_slots, kv_heads, p.kpc);
     if (err != B200_OK) return err;
@@ -532,10 +565,10 @@ int launch_attention_prefill_tc2(void* out, const void* q, int64_t q_st, int64_t
     if (err != B200_OK) return err;
     const int QB = kTile / p.group;
     const int smem = kSmemBytes + 1024;
-    B200_CHECK_CUDA(cudaFuncSetAttribute(attention_prefill_tc2_kernel,
-                                         cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    auto kernel = window ? attention_prefill_tc2_kernel<true> : attention_prefill_tc2_kernel<false>;
+    B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     dim3 grid(div_ceil(max_extend_len, 2 * QB), kv_heads, batch);
-    B200_CHECK_CUDA(launch_kernel(attention_prefill_tc2_kernel, grid, dim3(kThreads), smem, stream,
+    B200_CHECK_CUDA(launch_kernel(kernel, grid, dim3(kThreads), smem, stream,
                                   dim3(1, 1, 1), tk, tv, tk_tile, tv_tile, p));
     return B200_OK;
 }

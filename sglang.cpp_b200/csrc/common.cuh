@@ -108,6 +108,8 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&p);
 }
 
+__device__ __forceinline__ float sigmoid_f(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
+
 // Eight neighbouring elements of an fp32 or bf16 row (16-byte accesses).
 struct Vec8 {
     float v[8];
@@ -128,6 +130,15 @@ __device__ __forceinline__ void store8(float* p, const Vec8& x) {
 __device__ __forceinline__ void store8(__nv_bfloat16* p, const Vec8& x) {
     *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(x.v[0], x.v[1]), pack_bf16(x.v[2], x.v[3]),
                                               pack_bf16(x.v[4], x.v[5]), pack_bf16(x.v[6], x.v[7]));
+}
+
+// B200_EPILOGUE_CLAMPED_SWIGLU.  EXACT: the accurate exponential (fp32 models).
+template <bool EXACT>
+__device__ __forceinline__ float clamped_swiglu(float g, float u, float limit) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    const float e = EXACT ? expf(-1.702f * g) : __expf(-1.702f * g);
+    return (EXACT ? g / (1.0f + e) : __fdividef(g, 1.0f + e)) * (u + 1.0f);
 }
 
 __device__ __forceinline__ float round_bf16(float x) {

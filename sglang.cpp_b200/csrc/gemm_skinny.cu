@@ -83,6 +83,11 @@ __device__ __forceinline__ float gated_act(float g) {
     if (EPI == B200_EPILOGUE_GEGLU_ERF) return gelu_erf_f(g);
     return 0.5f * g * (1.0f + tanhf(0.7978845608f * (g + 0.044715f * g * g * g)));
 }
+template <int EPI>
+__device__ __forceinline__ float gated_pair(float g, float u, float limit) {
+    if (EPI == B200_EPILOGUE_CLAMPED_SWIGLU) return clamped_swiglu<false>(g, u, limit);
+    return gated_act<EPI>(g) * u;
+}
 __device__ __forceinline__ float gelu_tanh_f(float x) {
     return 0.5f * x * (1.0f + tanhf(0.7978845608f * (x + 0.044715f * x * x * x)));
 }
@@ -107,6 +112,7 @@ struct SkinnyParams {
     // Per-head mode: blockIdx.z = head; it reads columns [z * head_k, ...) of x and writes columns
     // [z * n_out, ...) of y with the weights of its own w_rows_per_group rows.
     int head_k;          // 0 = off
+    float act_limit;     // B200_EPILOGUE_CLAMPED_SWIGLU
     int64_t y_pitch;     // row pitch of y (n_out, or heads * n_out)
     // Fusions with the residual stream (split-K launches of the decode step; see SkinnyFusion in kernels.h).
     const unsigned long long* ssq_in;   // "normalised input": accumulator x rsqrt(ssq_in[m] / 2^24 / norm_width + eps)
@@ -398,12 +404,17 @@ skinny_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w,
                                 if (NUM_A == 2) {
                                     const float gv = round_bf16(__uint_as_float(g[j]));
                                     const float uv = round_bf16(__uint_as_float(u[j]));
-                                    v = gated_act<EPI>(gv) * uv;
+                                    v = gated_pair<EPI>(gv, uv, p.act_limit);
                                 } else {
                                     v = __uint_as_float(g[j]) + bias;
                                     if (EPI == B200_EPILOGUE_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
+                                    if (EPI == B200_EPILOGUE_GELU_ERF) v = gelu_erf_f(v);
                                 }
-                                p.y[static_cast<int64_t>(x_row0 + m) * p.y_pitch + y_col0 + n] = __float2bfloat16_rn(v);
+                                const int64_t at = static_cast<int64_t>(x_row0 + m) * p.y_pitch + y_col0 + n;
+                                if (EPI == B200_EPILOGUE_F32)
+                                    reinterpret_cast<float*>(p.y)[at] = v;
+                                else
+                                    p.y[at] = __float2bfloat16_rn(v);
                             }
                         }
                     }
@@ -593,14 +604,20 @@ skinny_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w,
                     for (int e = 0; e < 4; ++e) {
                         if (NUM_A == 2) {
                             const float gv = round_bf16(v[e]), uv = round_bf16(uu[e]);
-                            v[e] = gated_act<EPI>(gv) * uv;
+                            v[e] = gated_pair<EPI>(gv, uv, p.act_limit);
                         } else if (p.bias) {
                             v[e] += __bfloat162float(p.bias[n + e]);
                         }
                         if (EPI == B200_EPILOGUE_RELU2) v[e] = fmaxf(v[e], 0.f) * fmaxf(v[e], 0.f);
+                        if (EPI == B200_EPILOGUE_GELU_ERF) v[e] = gelu_erf_f(v[e]);
+                    }
+                    const int64_t at = static_cast<int64_t>(x_row0 + m) * p.y_pitch + y_col0 + n;
+                    if (EPI == B200_EPILOGUE_F32) {
+                        *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.y) + at) = make_float4(v[0], v[1], v[2], v[3]);
+                        continue;
                     }
                     uint2 packed = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
-                    *reinterpret_cast<uint2*>(p.y + static_cast<int64_t>(x_row0 + m) * p.y_pitch + y_col0 + n) = packed;
+                    *reinterpret_cast<uint2*>(p.y + at) = packed;
                 }
             }
         }
@@ -619,6 +636,9 @@ SkinnyKernel skinny_kernel_for(int epilogue, bool heads = false) {
         case B200_EPILOGUE_GEGLU: return skinny_gemm_kernel<B200_EPILOGUE_GEGLU>;
         case B200_EPILOGUE_GEGLU_ERF: return skinny_gemm_kernel<B200_EPILOGUE_GEGLU_ERF>;
         case B200_EPILOGUE_RELU2: return skinny_gemm_kernel<B200_EPILOGUE_RELU2>;
+        case B200_EPILOGUE_GELU_ERF: return skinny_gemm_kernel<B200_EPILOGUE_GELU_ERF>;
+        case B200_EPILOGUE_CLAMPED_SWIGLU: return skinny_gemm_kernel<B200_EPILOGUE_CLAMPED_SWIGLU>;
+        case B200_EPILOGUE_F32: return skinny_gemm_kernel<B200_EPILOGUE_F32>;
         default: return skinny_gemm_kernel<B200_EPILOGUE_NONE>;
     }
 }
@@ -712,7 +732,7 @@ int skinny_gemm_split(int M, int N, int K, int epilogue) {
 // One slab of at most 256 rows.
 int launch_skinny_gemm(void* y, const void* x, const void* w, const void* bias, int M, int N,
                        int K, int64_t ldx, int epilogue, int* status, cudaStream_t stream,
-                       const SkinnyFusion* fuse = nullptr) {
+                       const SkinnyFusion* fuse = nullptr, float act_limit = 0.f) {
     const bool gated = epilogue_is_gated(epilogue);
     const int n_out = gated ? N / 2 : N;
     // accumulator columns: 32, or a multiple of the 64-column exchange round (the epilogue walks whole rounds)
@@ -781,6 +801,7 @@ int launch_skinny_gemm(void* y, const void* x, const void* w, const void* bias, 
     p.group_offsets = nullptr;
     p.w_rows_per_group = 0;
     p.head_k = 0;
+    p.act_limit = act_limit;
     p.y_pitch = n_out;
     set_fusion(&p, fuse);
 
@@ -798,7 +819,7 @@ int launch_skinny_gemm(void* y, const void* x, const void* w, const void* bias, 
 int launch_grouped_gemm(void* y, const void* x, const void* w, const int32_t* counts,
                         const int32_t* offsets, int num_groups, int max_rows_per_group,
                         int64_t total_rows, int N, int K, int epilogue, int* status,
-                        cudaStream_t stream) {
+                        cudaStream_t stream, float act_limit) {
     const bool gated = epilogue_is_gated(epilogue);
     const int n_out = gated ? N / 2 : N;
     const int num_a = gated ? 2 : 1;
@@ -809,7 +830,7 @@ int launch_grouped_gemm(void* y, const void* x, const void* w, const int32_t* co
     // Many rows per group on average (prefill batches): tensor-bound, take the tile kernel.
     if (total_rows >= static_cast<int64_t>(num_groups) * env_int("B200_GROUPED_TILE_MIN_ROWS", 128) && num_groups <= 256)
         return launch_grouped_tile_gemm(y, x, w, counts, offsets, num_groups, total_rows, N, K, epilogue, status,
-                                        stream);
+                                        stream, act_limit);
     int nt_max = 32;
     while (nt_max < 256 && nt_max < max_rows_per_group) nt_max *= 2;
     const uint32_t stage_bytes = num_a * kTileN * kBlockK * 2 + nt_max * kBlockK * 2;
@@ -848,6 +869,7 @@ int launch_grouped_gemm(void* y, const void* x, const void* w, const int32_t* co
     p.group_offsets = offsets;
     p.w_rows_per_group = N;
     p.head_k = 0;
+    p.act_limit = act_limit;
     p.y_pitch = n_out;
     set_fusion(&p, nullptr);
     auto kernel = skinny_kernel_for(epilogue);
@@ -900,6 +922,7 @@ int launch_linear_heads(void* y, const void* x, const void* w, int M, int heads,
         p.group_offsets = nullptr;
         p.w_rows_per_group = N;
         p.head_k = K;
+        p.act_limit = 0.f;
         p.y_pitch = static_cast<int64_t>(heads) * N;
         set_fusion(&p, nullptr);
         auto kernel = skinny_kernel_for(B200_EPILOGUE_NONE);
@@ -912,23 +935,25 @@ int launch_linear_heads(void* y, const void* x, const void* w, int M, int heads,
 }
 
 int launch_linear(void* y, const void* x, const void* w, const void* bias, int M, int N, int K,
-                  int64_t ldx, int epilogue, int* status, cudaStream_t stream, const SkinnyFusion* fuse) {
+                  int64_t ldx, int epilogue, int* status, cudaStream_t stream, const SkinnyFusion* fuse,
+                  float act_limit) {
     // Few rows: stream the weights once (swap-AB, split-K).  Many rows: tensor-bound tiles.
     if (M >= env_int("B200_GEMM_TILE_MIN_M", 257)) {
         if (fuse != nullptr) {
             set_last_error("linear: the residual-stream fusions need at most 256 rows");
             return B200_ERR_UNSUPPORTED;
         }
-        return launch_tile_gemm(y, x, w, bias, M, N, K, ldx, epilogue, status, stream);
+        return launch_tile_gemm(y, x, w, bias, M, N, K, ldx, epilogue, status, stream, act_limit);
     }
     const int n_out = epilogue_is_gated(epilogue) ? N / 2 : N;
     const __nv_bfloat16* xp = static_cast<const __nv_bfloat16*>(x);
-    __nv_bfloat16* yp = static_cast<__nv_bfloat16*>(y);
+    char* yp = static_cast<char*>(y);
+    const int64_t y_row_bytes = static_cast<int64_t>(n_out) * (epilogue == B200_EPILOGUE_F32 ? 4 : 2);
     for (int m0 = 0; m0 < M; m0 += 256) {
         const int rows = (M - m0) < 256 ? (M - m0) : 256;
-        int err = launch_skinny_gemm(yp + static_cast<int64_t>(m0) * n_out,
+        int err = launch_skinny_gemm(yp + m0 * y_row_bytes,
                                      xp + static_cast<int64_t>(m0) * ldx, w, bias, rows, N, K, ldx,
-                                     epilogue, status, stream, fuse);
+                                     epilogue, status, stream, fuse, act_limit);
         if (err != B200_OK) return err;
     }
     return B200_OK;
@@ -948,6 +973,24 @@ int b200_linear_heads(void* y, const void* x, const void* w, int M, int heads, i
     int* status = b200::device_status_words(&err);
     if (err != B200_OK) return err;
     return b200::launch_linear_heads(y, x, w, M, heads, N, K, status, static_cast<cudaStream_t>(stream));
+}
+
+int b200_linear_act(void* y, const void* x, const void* w, int M, int N, int K, int epilogue, float act_limit, int dtype,
+                    b200_stream_t stream) {
+    B200_CHECK_ARG(M >= 0 && N > 0 && K > 0, "linear_act: bad shape");
+    B200_CHECK_ARG(M == 0 || (y && x && w), "linear_act: NULL tensor");
+    B200_CHECK_ARG(K % 64 == 0 && N % 16 == 0, "linear_act: K must be a multiple of 64, N of 16");
+    B200_CHECK_ARG(epilogue >= B200_EPILOGUE_NONE && epilogue <= B200_EPILOGUE_F32, "linear_act: unknown epilogue");
+    B200_CHECK_ARG(dtype == B200_DTYPE_BF16 || dtype == B200_DTYPE_F32, "linear_act: unknown dtype");
+    if (M == 0) return B200_OK;
+    int err = B200_OK;
+    int* status = b200::device_status_words(&err);
+    if (err != B200_OK) return err;
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    if (dtype == B200_DTYPE_F32)
+        return b200::launch_linear_f32(static_cast<float*>(y), static_cast<const float*>(x), static_cast<const float*>(w), M,
+                                       N, K, 1, nullptr, nullptr, epilogue, s, act_limit);
+    return b200::launch_linear(y, x, w, nullptr, M, N, K, K, epilogue, status, s, nullptr, act_limit);
 }
 
 int b200_linear(void* y, const void* x, const void* w, const void* bias, int M, int N, int K,

@@ -46,6 +46,7 @@ struct TileParams {
     const int32_t* group_offsets;
     int num_groups;
     int w_rows_per_group;
+    float act_limit;    // B200_EPILOGUE_CLAMPED_SWIGLU
 };
 
 constexpr int kMaxGroups = 256;
@@ -260,7 +261,8 @@ tile_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
                         if (GATED) {
                             const float gv = round_bf16(__uint_as_float(g[j]));
                             const float uv = round_bf16(__uint_as_float(u[j]));
-                            v[j] = gated_act_tile<EPI>(gv) * uv;
+                            v[j] = EPI == B200_EPILOGUE_CLAMPED_SWIGLU ? clamped_swiglu<false>(gv, uv, p.act_limit)
+                                                                       : gated_act_tile<EPI>(gv) * uv;
                         } else {
                             v[j] = __uint_as_float(g[j]);
                         }
@@ -273,6 +275,18 @@ tile_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
                     if (EPI == B200_EPILOGUE_RELU2) {
 #pragma unroll
                         for (int j = 0; j < 32; ++j) v[j] = fmaxf(v[j], 0.f) * fmaxf(v[j], 0.f);
+                    }
+                    if (EPI == B200_EPILOGUE_GELU_ERF) {
+#pragma unroll
+                        for (int j = 0; j < 32; ++j) v[j] = 0.5f * v[j] * (1.0f + erff(v[j] * 0.70710678118654752f));
+                    }
+                    if (EPI == B200_EPILOGUE_F32) {
+                        float* frow = reinterpret_cast<float*>(p.y) + static_cast<int64_t>(m) * p.n_out;
+#pragma unroll
+                        for (int j = 0; j < 32; j += 4)
+                            if (n + j < p.n_out)
+                                *reinterpret_cast<float4*>(frow + n + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+                        continue;
                     }
 #pragma unroll
                     for (int j = 0; j < 32; j += 8) {
@@ -301,7 +315,7 @@ tile_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
 }  // namespace
 
 int launch_tile_gemm(void* y, const void* x, const void* w, const void* bias, int M, int N, int K,
-                     int64_t ldx, int epilogue, int* status, cudaStream_t stream) {
+                     int64_t ldx, int epilogue, int* status, cudaStream_t stream, float act_limit) {
     const bool gated = epilogue_is_gated(epilogue);
     const int n_out = gated ? N / 2 : N;
     TileParams p;
@@ -319,6 +333,7 @@ int launch_tile_gemm(void* y, const void* x, const void* w, const void* bias, in
     p.group_offsets = nullptr;
     p.num_groups = 0;
     p.w_rows_per_group = 0;
+    p.act_limit = act_limit;
 
     CUtensorMap tmap_x, tmap_w;
     int err = cached_tmap(&tmap_x, x, static_cast<uint64_t>(K), static_cast<uint64_t>(M),
@@ -336,6 +351,9 @@ int launch_tile_gemm(void* y, const void* x, const void* w, const void* bias, in
     if (epilogue == B200_EPILOGUE_GEGLU) kernel = tile_gemm_kernel<B200_EPILOGUE_GEGLU>;
     if (epilogue == B200_EPILOGUE_GEGLU_ERF) kernel = tile_gemm_kernel<B200_EPILOGUE_GEGLU_ERF>;
     if (epilogue == B200_EPILOGUE_RELU2) kernel = tile_gemm_kernel<B200_EPILOGUE_RELU2>;
+    if (epilogue == B200_EPILOGUE_GELU_ERF) kernel = tile_gemm_kernel<B200_EPILOGUE_GELU_ERF>;
+    if (epilogue == B200_EPILOGUE_CLAMPED_SWIGLU) kernel = tile_gemm_kernel<B200_EPILOGUE_CLAMPED_SWIGLU>;
+    if (epilogue == B200_EPILOGUE_F32) kernel = tile_gemm_kernel<B200_EPILOGUE_F32>;
     B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(smem_bytes)));
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(grid), dim3(kThreads), smem_bytes, stream, dim3(1, 1, 1),
@@ -347,7 +365,7 @@ int launch_tile_gemm(void* y, const void* x, const void* w, const void* bias, in
 // [offsets[g], offsets[g] + counts[g]) of x [total_rows, K] by w[g] ([N, K], groups stacked).
 int launch_grouped_tile_gemm(void* y, const void* x, const void* w, const int32_t* counts,
                              const int32_t* offsets, int num_groups, int64_t total_rows, int N, int K,
-                             int epilogue, int* status, cudaStream_t stream) {
+                             int epilogue, int* status, cudaStream_t stream, float act_limit) {
     if (num_groups > kMaxGroups) {
         set_last_error("grouped GEMM: %d groups exceed %d", num_groups, kMaxGroups);
         return B200_ERR_UNSUPPORTED;
@@ -369,6 +387,7 @@ int launch_grouped_tile_gemm(void* y, const void* x, const void* w, const int32_
     p.group_offsets = offsets;
     p.num_groups = num_groups;
     p.w_rows_per_group = N;
+    p.act_limit = act_limit;
     CUtensorMap tmap_x, tmap_w;
     int err = cached_tmap(&tmap_x, x, static_cast<uint64_t>(K), static_cast<uint64_t>(total_rows),
                           static_cast<uint64_t>(K) * 2, kBK, kTM);
@@ -382,6 +401,9 @@ int launch_grouped_tile_gemm(void* y, const void* x, const void* w, const int32_
     if (epilogue == B200_EPILOGUE_GEGLU) kernel = tile_gemm_kernel<B200_EPILOGUE_GEGLU>;
     if (epilogue == B200_EPILOGUE_GEGLU_ERF) kernel = tile_gemm_kernel<B200_EPILOGUE_GEGLU_ERF>;
     if (epilogue == B200_EPILOGUE_RELU2) kernel = tile_gemm_kernel<B200_EPILOGUE_RELU2>;
+    if (epilogue == B200_EPILOGUE_GELU_ERF) kernel = tile_gemm_kernel<B200_EPILOGUE_GELU_ERF>;
+    if (epilogue == B200_EPILOGUE_CLAMPED_SWIGLU) kernel = tile_gemm_kernel<B200_EPILOGUE_CLAMPED_SWIGLU>;
+    if (epilogue == B200_EPILOGUE_F32) kernel = tile_gemm_kernel<B200_EPILOGUE_F32>;
     B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(smem_bytes)));
     // the number of tiles is only known on the device: one persistent CTA per SM

@@ -12,7 +12,8 @@ namespace b200 {
 
 // Gated epilogues take two stacked halves of W (gate, up); the others one.
 constexpr bool epilogue_is_gated(int epilogue) {
-    return epilogue != B200_EPILOGUE_NONE && epilogue != B200_EPILOGUE_RELU2;
+    return epilogue != B200_EPILOGUE_NONE && epilogue != B200_EPILOGUE_RELU2 && epilogue != B200_EPILOGUE_GELU_ERF &&
+           epilogue != B200_EPILOGUE_F32;
 }
 
 int launch_rmsnorm(void* out, const void* x, const void* weight, int rows, int hidden, float eps,
@@ -62,12 +63,13 @@ int cached_tmap(CUtensorMap* out, const void* base, uint64_t inner, uint64_t out
                 uint32_t box_inner, uint32_t box_outer);
 
 // Large-M GEMM (prefill batches): persistent 128 x 256 output tiles on the tcgen05 tensor cores.
+// act_limit (here and below): the limit of B200_EPILOGUE_CLAMPED_SWIGLU.
 int launch_tile_gemm(void* y, const void* x, const void* w, const void* bias, int M, int N, int K,
-                     int64_t ldx, int epilogue, int* status, cudaStream_t stream);
+                     int64_t ldx, int epilogue, int* status, cudaStream_t stream, float act_limit = 0.f);
 
 int launch_grouped_tile_gemm(void* y, const void* x, const void* w, const int32_t* counts,
                              const int32_t* offsets, int num_groups, int64_t total_rows, int N, int K,
-                             int epilogue, int* status, cudaStream_t stream);
+                             int epilogue, int* status, cudaStream_t stream, float act_limit = 0.f);
 
 // Fusions of a split-K GEMM of at most 256 rows with the residual stream of a decode step.  Row
 // statistics travel as sums of squares in 2^-24 fixed point (integer atomics: the same bits whatever
@@ -107,18 +109,19 @@ int skinny_gemm_split(int M, int N, int K, int epilogue);
 // y[M, n_out] = x[M, K] w[N, K]^T (+bias / gated epilogue); any M (slabs of 256 rows).
 int launch_linear(void* y, const void* x, const void* w, const void* bias, int M, int N, int K,
                   int64_t ldx, int epilogue, int* status, cudaStream_t stream,
-                  const SkinnyFusion* fuse = nullptr);
+                  const SkinnyFusion* fuse = nullptr, float act_limit = 0.f);
 
 int launch_grouped_gemm(void* y, const void* x, const void* w, const int32_t* counts,
                         const int32_t* offsets, int num_groups, int max_rows_per_group,
                         int64_t total_rows, int N, int K, int epilogue, int* status,
-                        cudaStream_t stream);
+                        cudaStream_t stream, float act_limit = 0.f);
 
 int launch_linear_heads(void* y, const void* x, const void* w, int M, int heads, int N, int K, int* status,
                         cudaStream_t stream);
 // fp32 GEMMs of every form the layer stack uses (linear_f32.cu); see b200_linear_f32.
 int launch_linear_f32(float* y, const float* x, const float* w, int max_rows, int N, int K, int groups,
-                      const int32_t* counts, const int32_t* offsets, int epilogue, cudaStream_t stream);
+                      const int32_t* counts, const int32_t* offsets, int epilogue, cudaStream_t stream,
+                      float act_limit = 0.f);
 
 // fp32 residual stream: add, norm, and the gather / scatter around them (residual.cu).
 struct ResidualNorm {
@@ -139,6 +142,28 @@ struct ResidualNorm {
 };
 int launch_residual_norm(const ResidualNorm& a, int dtype, int* status, cudaStream_t stream);
 
+// The wiring with the norm on what is added: residual += add_weight * rms_normalise(sum_k src_weights[k] *
+// src[src_rows[k]] + src2), out = residual (through the norm with out_weight if there is one).
+struct ResidualPostNorm {
+    void* out = nullptr;
+    float* residual = nullptr;
+    const void* src = nullptr;
+    const int32_t* src_rows = nullptr;      // NULL: the token's own row
+    const float* src_weights = nullptr;     // NULL: 1
+    int src_top = 1;
+    int64_t src_count = 0;
+    const void* src2 = nullptr;             // optional second row per token
+    bool init = false;                      // the sum replaces the residual
+    const void* add_weight = nullptr;       // NULL: what is added is not normalised
+    const void* out_weight = nullptr;       // NULL: out is the residual itself
+    float weight_offset = 0.f, out_scale = 1.f;   // as in ResidualNorm
+    int tokens = 0, width = 0, padded = 0;
+    float eps = 0.f;
+    int32_t* clear = nullptr;               // integers set to zero on the way (counters of a later kernel)
+    int clear_count = 0;
+};
+int launch_residual_post_norm(const ResidualPostNorm& a, int dtype, int* status, cudaStream_t stream);
+
 // Expert placement of every table-routed layer of a step in one launch (moe.cu): one CTA per layer.
 struct TableRouteLayer {
     const int32_t* table;     // [vocab, top]
@@ -148,6 +173,21 @@ struct TableRouteLayer {
 constexpr int kMaxTableExperts = 4096;
 int launch_table_route(const TableRouteLayer* layers_dev, int num_layers, int max_experts, const int32_t* token_ids,
                        int tokens, int vocab, int* status, cudaStream_t stream);
+
+// Routing by sigmoid scores (moe.cu): ids, weights and counts from fp32 logits, then a row for every choice
+// and the token's activations copied there.  counts [experts] and the cursor [experts] are zero before.
+struct ScoreRoute {
+    const float* logits = nullptr;   // [tokens, ld]
+    int64_t ld = 0;
+    int tokens = 0, experts = 0, top = 1, groups = 1, keep = 1;
+    float scale = 1.f;
+    int32_t* ids = nullptr;          // [tokens, top]
+    float* weights = nullptr;        // [tokens, top]
+    int32_t* counts = nullptr;
+};
+int launch_score_route(const ScoreRoute& r, cudaStream_t stream);
+int launch_score_place(void* xp, const void* x, int row_bytes, const ScoreRoute& r, int32_t* rows, int32_t* cursor,
+                       int32_t* offsets, cudaStream_t stream);
 
 // Latent attention (latent_attention.cu, latent_attention_tc.cu).
 // The output of the joint down-projection [tokens, qp + rp] -> RMS-normalised query latent [tokens, qp]
@@ -219,6 +259,16 @@ bool decode_chain_supported(int tokens, int hidden, int q_heads, int kv_heads, i
                             bool has_bias);
 int launch_decode_chain(const DecodeChainArgs& args, cudaStream_t stream);
 
+// A sliding window over the keys, the first ones kept, and a gate on the output (what the paged attention
+// kernels take beside causal attention): the query at position i sees key j <= i if i - j < size or
+// j < keep_first, and head h's output element c is multiplied by sigmoid(gate[token, h * 128 + c]).
+struct AttentionWindow {
+    int size = 0x7fffffff;
+    int keep_first = 0;
+    const void* gate = nullptr;   // bf16; NULL: no gate
+    int64_t gate_st = 0;          // its token stride in elements
+};
+
 int64_t decode_workspace_bytes(int max_batch, int q_heads, int kv_heads);
 int make_kv_tmap(CUtensorMap* out, const void* cache, int64_t num_slots, int kv_heads, int page_size);
 int launch_attention_decode(void* out, const void* q, int64_t q_st, int64_t q_sh,
@@ -226,7 +276,55 @@ int launch_attention_decode(void* out, const void* q, int64_t q_st, int64_t q_sh
                             const int32_t* page_table, int64_t pt_stride, const int32_t* table_idx,
                             const int32_t* seq_lens, int batch, int q_heads, int kv_heads,
                             int page_size, float sm_scale, void* workspace, int64_t workspace_bytes,
-                            int* status, cudaStream_t stream, bool kv_evict_first = false);
+                            int* status, cudaStream_t stream, bool kv_evict_first = false,
+                            const AttentionWindow* window = nullptr);
+// Attention of layer stacks (window_attention.cu).  head_prepare: the rows of the joint projection's output
+// [q heads | k heads | v heads | ...] to normalised, rotated queries (in place) and into the pools.
+struct HeadPrepare {
+    enum { kPlain = 0, kSave = 1, kMix = 2 };   // values: as they are, kept for later layers, mixed with the kept ones
+    void* joint = nullptr;
+    int64_t ld = 0;
+    int tokens = 0, heads = 0, kv_heads = 0, dim = 0, dp = 0, vp = 0;
+    const void *q_weight = nullptr, *k_weight = nullptr;   // [dp] or NULL
+    float eps = 0.f;
+    int rotary_dim = 0, max_pos = 1;
+    const float *cos_t = nullptr, *sin_t = nullptr;        // [max_pos, rotary_dim / 2]
+    const int32_t *positions = nullptr, *out_loc = nullptr;
+    void *k_cache = nullptr, *v_cache = nullptr;           // [num_slots, kv_heads, dp | vp]
+    int64_t num_slots = 0;
+    int mix = kPlain;
+    const float* lambda = nullptr;                         // v <- (1 - lambda) v + lambda first
+    void* first_values = nullptr;                          // [tokens, kv_heads, vp]
+    int* status = nullptr;
+};
+int launch_head_prepare(const HeadPrepare& a, int dtype, cudaStream_t stream);
+struct WindowAttention {
+    void* out = nullptr;               // [tokens, heads, vp]
+    const void* q = nullptr;           // token stride q_st, heads dp apart
+    int64_t q_st = 0;
+    const void *k_cache = nullptr, *v_cache = nullptr;
+    int64_t num_slots = 0;
+    const int32_t* page_table = nullptr;
+    int64_t pt_stride = 0;
+    const int32_t *table_idx = nullptr, *seq_lens = nullptr, *qo_indptr = nullptr;   // per request
+    const int32_t *row_table = nullptr, *row_len = nullptr;                          // per token
+    int tokens = 0, batch = 0, max_extend = 0;
+    bool decode = false;               // one token per request, the tables complete ahead of the launch
+    bool plain = false;                // never the tensor-core kernels
+    int heads = 0, kv_heads = 0, dp = 0, vp = 0, page_size = 1;
+    float scale = 1.f;
+    AttentionWindow window;
+    void* workspace = nullptr;
+    int64_t workspace_bytes = 0;       // decode_workspace_bytes
+    int* status = nullptr;
+};
+bool window_attention_tc_supported(const WindowAttention& a, int dtype);
+int launch_window_attention(const WindowAttention& a, int dtype, cudaStream_t stream);
+// Gated linear attention (linear_attention.cu): the recurrence, its norm and its gate; see
+// b200_linear_attention.
+using LinearAttention = b200_linear_attention_args;
+bool linear_attention_supported(int padded_value_dim, int padded_dim);
+int launch_linear_attention(const LinearAttention& a, int dtype, cudaStream_t stream);
 bool attention_prefill_tc_supported(const void* q, int64_t q_st, int64_t q_sh, const void* out);
 int launch_attention_prefill_tc(void* out, const void* q, int64_t q_st, int64_t q_sh, const void* k_cache,
                                 const void* v_cache, int64_t num_slots, const int32_t* page_table,
@@ -239,7 +337,7 @@ int launch_attention_prefill_tc2(void* out, const void* q, int64_t q_st, int64_t
                                 int64_t pt_stride, const int32_t* table_idx, const int32_t* seq_lens,
                                 const int32_t* qo_indptr, int batch, int max_extend_len, int q_heads,
                                 int kv_heads, int page_size, float sm_scale, int* status,
-                                cudaStream_t stream);
+                                cudaStream_t stream, const AttentionWindow* window = nullptr);
 int launch_attention_prefill(void* out, const void* q, int64_t q_st, int64_t q_sh, const void* k_cache,
                              const void* v_cache, int64_t num_slots, const int32_t* page_table,
                              int64_t pt_stride, const int32_t* table_idx, const int32_t* seq_lens,

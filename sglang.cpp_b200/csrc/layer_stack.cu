@@ -1,23 +1,31 @@
-// Models whose layers are listed one by one: allocation of their weights and latent pools, the per-step
+// Models whose layers are listed one by one: allocation of their weights, pools and states, the per-step
 // plan, and the layer stack the step runner (engine.cu) enqueues between its token preparation and its
 // output head.
 //
 // Per layer, on T tokens (fp32 residual stream r, everything else in the stack's dtype):
-//     x  = norm(r += previous block)              one kernel, residual.cu
-//     [cq | c] = x W_down                         both latents in one GEMM
-//     cq, pool[slot] = norm(cq), norm(c)          latent_attention.cu
-//     q  = cq W_uq
-//     o  = attention(q, pool)                     in the latent space, or over expanded keys and values
-//     y  = o W_o
-//     x  = norm(r += y), to the expert-sorted rows when the feed-forward is a mixture of experts
-//     y  = feed-forward(x)
-// The placement of tokens on experts depends on token ids only and is laid out for all layers at once
-// before the first.
+//     x = norm(r += previous block)       the norm on the input: one kernel, residual.cu
+//     x = r += norm(previous block)       or on the output of a block; one kernel as well
+//     y = mixer(x)
+//     x = ... once more
+//     y = feed-forward(x)
 //
-// Attention has two forms.  In the latent space (decode steps, short extensions) the per-head projections
+// Mixers
+//   latent attention:  [cq | c] = x W_down, both latents in one GEMM; cq, pool[slot] = norm(cq), norm(c)
+//                      (latent_attention.cu); q = cq W_uq; o = attention in the latent space, or over expanded
+//                      keys and values; y = o W_o
+//   window attention:  [q | k | v | gate] = x W in one GEMM; norms, rotation, value mixing and the K/V store in
+//                      one kernel; attention and its gate in the next (window_attention.cu); y = o W_o
+//   linear attention:  [q | k | v | gate | low-rank decay] = x W in one GEMM; recurrence, norm and gate
+//                      (linear_attention.cu); y = o W_o
+// Feed-forwards: dense; experts by token id, whose placement depends on token ids only and is laid out for all
+// layers at once before the first; experts by score (router logits in fp32, routing and placement in two
+// kernels, the weighted sum in the residual kernel that follows), beside one that every token uses.
+//
+// Latent attention has two forms.  In the latent space (decode steps, short extensions) the per-head projections
 // are applied to the query and to the result.  Extensions of more than `expand_min` tokens expand keys and
 // values of the whole request once (two GEMMs) into a scratch that the prefill kernel of the
 // grouped-query models reads as if it were its paged pool.  A batch may hold both kinds of requests.
+#include <math.h>
 #include <stdlib.h>
 
 #include <string>
@@ -41,6 +49,17 @@ struct StackLayer {
     int qp = 0, rp = 0, dp = 0, vp = 0, ip = 0;   // padded sizes
     void *norm1 = nullptr, *norm2 = nullptr, *down_qkv = nullptr, *q_norm = nullptr, *kv_norm = nullptr, *uq = nullptr,
          *uk = nullptr, *uk_absorb = nullptr, *uv = nullptr, *o = nullptr, *up = nullptr, *down = nullptr;
+    // window attention
+    void *qkvg = nullptr, *q_head_norm = nullptr, *k_head_norm = nullptr, *k_cache = nullptr, *v_cache = nullptr;
+    float *value_mix = nullptr, *cos_t = nullptr, *sin_t = nullptr;
+    int mix = HeadPrepare::kPlain;
+    // linear attention
+    void *qkvga = nullptr, *decay_up = nullptr, *head_norm = nullptr;
+    float *decay_bias = nullptr, *state = nullptr;
+    int up_ld = 0;
+    // scored experts
+    void *router = nullptr, *shared_up = nullptr, *shared_down = nullptr;
+    int isp = 0;
     int32_t* table = nullptr;
     void* cache = nullptr;
     int32_t *rows = nullptr, *counts = nullptr, *offsets = nullptr;   // expert placement of this step
@@ -53,6 +72,7 @@ struct LayerStack {
     int esz = 2;            // bytes per element
     int hp = 0, vocab_p = 0;
     float norm_offset = 0.f, logit_scale = 1.f;
+    bool norm_output = false;
     void *embed = nullptr, *head = nullptr, *final_norm = nullptr;
     float* residual = nullptr;
     void *x = nullptr, *joint = nullptr, *cq = nullptr, *q = nullptr, *attn = nullptr, *y = nullptr, *h = nullptr,
@@ -74,6 +94,13 @@ struct LayerStack {
     // the latent-space rows of a mixed step, compacted
     int32_t *compact_row = nullptr, *compact_len = nullptr;
     void *qc = nullptr, *ac = nullptr;
+    int max_extend = 0;        // longest extension of the current step
+    // window attention
+    void* first_values = nullptr;
+    // scored experts: the routing of the layer that is running
+    float *router_logits = nullptr, *route_weights = nullptr;
+    int32_t *route_ids = nullptr, *route_rows = nullptr, *route_counts = nullptr, *route_offsets = nullptr;
+    void *shared_h = nullptr, *shared_y = nullptr;
     std::vector<TableRouteLayer> routes;
     TableRouteLayer* routes_dev = nullptr;
     int max_experts = 0;
@@ -111,17 +138,209 @@ __global__ void compact_rows_kernel(int32_t* __restrict__ row, int32_t* __restri
 }
 
 int check_layer(const b200_layer_config& c, int l) {
-    B200_CHECK_ARG(c.mixer == B200_MIXER_LATENT_ATTENTION, "layer %d: unknown mixer %d", l, c.mixer);
-    B200_CHECK_ARG(c.heads > 0 && c.head_dim > 0 && c.value_dim > 0 && c.q_rank > 0 && c.kv_rank > 0,
-                   "layer %d: latent attention needs positive sizes", l);
-    B200_CHECK_ARG(c.mlp >= B200_MLP_NONE && c.mlp <= B200_MLP_TABLE_MOE, "layer %d: unknown feed-forward %d", l, c.mlp);
+    B200_CHECK_ARG(c.heads > 0 && c.heads <= 65535 && c.head_dim > 0 && c.value_dim > 0,
+                   "layer %d: head count and sizes must be positive", l);
+    if (c.mixer == B200_MIXER_LATENT_ATTENTION) {
+        B200_CHECK_ARG(c.q_rank > 0 && c.kv_rank > 0, "layer %d: latent attention needs positive ranks", l);
+    } else if (c.mixer == B200_MIXER_WINDOW_ATTENTION) {
+        B200_CHECK_ARG(c.kv_heads > 0 && c.heads % c.kv_heads == 0, "layer %d: %d heads over %d key/value heads", l, c.heads,
+                       c.kv_heads);
+        B200_CHECK_ARG(c.window > 0 && c.keep_first >= 0, "layer %d: bad window", l);
+        B200_CHECK_ARG(c.rotary_dim >= 0 && c.rotary_dim % 2 == 0 && c.rotary_dim <= c.head_dim &&
+                           (c.rotary_dim == 0 || c.rope_base > 0.0), "layer %d: bad rotation", l);
+        B200_CHECK_ARG(c.value_dim <= 1024 && c.head_dim <= 2048, "layer %d: heads are too wide", l);
+    } else if (c.mixer == B200_MIXER_LINEAR_ATTENTION) {
+        B200_CHECK_ARG(c.decay_rank > 0 && c.decay_tau > 0.f, "layer %d: bad decay", l);
+        B200_CHECK_ARG(linear_attention_supported(pad_width(c.value_dim), pad_width(c.head_dim)),
+                       "layer %d: heads are too wide", l);
+    } else {
+        B200_CHECK_ARG(false, "layer %d: unknown mixer %d", l, c.mixer);
+    }
+    B200_CHECK_ARG(c.mlp >= B200_MLP_NONE && c.mlp <= B200_MLP_SCORED_MOE, "layer %d: unknown feed-forward %d", l, c.mlp);
     if (c.mlp == B200_MLP_NONE) return B200_OK;
     B200_CHECK_ARG(c.intermediate > 0, "layer %d: feed-forward size must be positive", l);
-    B200_CHECK_ARG(c.epilogue > B200_EPILOGUE_NONE && c.epilogue <= B200_EPILOGUE_RELU2, "layer %d: unknown activation", l);
-    if (c.mlp == B200_MLP_TABLE_MOE)
+    B200_CHECK_ARG(c.epilogue > B200_EPILOGUE_NONE && c.epilogue <= B200_EPILOGUE_CLAMPED_SWIGLU, "layer %d: unknown activation", l);
+    if (c.mlp != B200_MLP_DENSE)
         B200_CHECK_ARG(c.num_experts > 0 && c.num_experts <= kMaxTableExperts && c.experts_per_tok > 0 &&
                            c.experts_per_tok <= c.num_experts,
                        "layer %d: %d of %d experts (at most %d)", l, c.experts_per_tok, c.num_experts, kMaxTableExperts);
+    if (c.mlp == B200_MLP_SCORED_MOE)
+        B200_CHECK_ARG(c.router_groups > 0 && c.num_experts % c.router_groups == 0 && c.router_keep > 0 &&
+                           c.router_keep <= c.router_groups &&
+                           c.experts_per_tok <= c.num_experts / c.router_groups * c.router_keep && c.shared_intermediate >= 0,
+                       "layer %d: bad expert groups", l);
+    return B200_OK;
+}
+
+// Sizes of the activation buffers: the widest of any layer, in elements per token (workspaces: bytes).
+struct Widths {
+    int64_t joint = 0, cq = 0, q = 0, attn = 0, h = 0, pairs = 0, latent = 0, xk = 0, xv = 0, xc = 0, ws = 0, first = 0,
+            experts = 0, router = 0, top = 0, shared = 0;
+    bool scored = false, any_expand = false;
+    static void widest(int64_t& a, int64_t b) { if (b > a) a = b; }
+};
+
+int alloc_latent(b200_engine* e, StackLayer& L, const std::string& sfx, Widths& w) {
+    LayerStack* S = e->stack;
+    const b200_layer_config& c = L.c;
+    L.qp = pad_width(c.q_rank);
+    L.rp = pad_latent(c.kv_rank);
+    L.dp = pad_head_dim(c.head_dim);
+    L.vp = pad_head_dim(c.value_dim);
+    const int64_t hp = S->hp, z = S->esz, H = c.heads, qp = L.qp, rp = L.rp, dp = L.dp, vp = L.vp;
+    S_TRY(named_bytes(e, &L.down_qkv, "down_qkv" + sfx, (qp + rp) * hp * z));
+    S_TRY(named_bytes(e, &L.q_norm, "q_latent_norm" + sfx, qp * z));
+    S_TRY(named_bytes(e, &L.kv_norm, "kv_latent_norm" + sfx, rp * z));
+    S_TRY(named_bytes(e, &L.uq, "uq" + sfx, H * dp * qp * z));
+    S_TRY(named_bytes(e, &L.uk_absorb, "uk_absorb" + sfx, H * rp * dp * z));
+    S_TRY(named_bytes(e, &L.uv, "uv" + sfx, H * vp * rp * z));
+    S_TRY(named_bytes(e, &L.cache, "latent_cache" + sfx, e->num_slots * rp * z));
+    // what the prefill kernel of the grouped-query models takes (and its positive score scale)
+    L.can_expand = S->dtype == B200_DTYPE_BF16 && dp == 128 && vp == 128 && c.score_scale > 0.f && H <= 65535;
+    if (L.can_expand) S_TRY(named_bytes(e, &L.uk, "uk" + sfx, H * dp * rp * z));
+    w.any_expand |= L.can_expand;
+    Widths::widest(w.joint, qp + rp);
+    Widths::widest(w.cq, qp);
+    Widths::widest(w.q, H * dp);
+    Widths::widest(w.latent, H * rp);
+    Widths::widest(w.ws, latent_attention_workspace_bytes(S->latent_rows, c.heads, L.rp));
+    if (L.can_expand) {
+        Widths::widest(w.xk, H * dp);
+        Widths::widest(w.xv, H * vp);
+        Widths::widest(w.xc, rp);
+    }
+    return B200_OK;
+}
+
+// cos / sin of position * base^(-2 i / dims), computed in double on the host; layers with the same rotation share
+// a table.
+int rope_table(b200_engine* e, StackLayer& L, int l) {
+    const b200_layer_config& c = L.c;
+    for (int o = 0; o < l; ++o) {
+        const StackLayer& other = e->stack->layers[o];
+        if (other.cos_t != nullptr && other.c.rotary_dim == c.rotary_dim && other.c.rope_base == c.rope_base) {
+            L.cos_t = other.cos_t;
+            L.sin_t = other.sin_t;
+            return B200_OK;
+        }
+    }
+    const int half = c.rotary_dim / 2;
+    const int64_t n = static_cast<int64_t>(e->pt_cols) * half;
+    std::vector<float> cs(n), sn(n);
+    for (int i = 0; i < half; ++i) {
+        const double f = pow(c.rope_base, -2.0 * i / c.rotary_dim);
+        for (int64_t p = 0; p < e->pt_cols; ++p) {
+            cs[p * half + i] = static_cast<float>(cos(static_cast<double>(p) * f));
+            sn[p * half + i] = static_cast<float>(sin(static_cast<double>(p) * f));
+        }
+    }
+    void* p = nullptr;
+    S_TRY(dev_alloc(e, &p, n * 4, true));
+    L.cos_t = static_cast<float*>(p);
+    S_TRY(dev_alloc(e, &p, n * 4, true));
+    L.sin_t = static_cast<float*>(p);
+    if (n == 0) return B200_OK;
+    B200_CHECK_CUDA(cudaMemcpy(L.cos_t, cs.data(), n * 4, cudaMemcpyHostToDevice));
+    B200_CHECK_CUDA(cudaMemcpy(L.sin_t, sn.data(), n * 4, cudaMemcpyHostToDevice));
+    return B200_OK;
+}
+
+int alloc_window(b200_engine* e, StackLayer& L, int l, const std::string& sfx, Widths& w) {
+    LayerStack* S = e->stack;
+    const b200_layer_config& c = L.c;
+    L.dp = pad_head_dim(c.head_dim);
+    L.vp = pad_head_dim(c.value_dim);
+    const int64_t hp = S->hp, z = S->esz, H = c.heads, G = c.kv_heads, dp = L.dp, vp = L.vp;
+    const int64_t joint = (H + G) * dp + (G + H) * vp;
+    S_TRY(named_bytes(e, &L.qkvg, "qkvg" + sfx, joint * hp * z));
+    S_TRY(named_bytes(e, &L.q_head_norm, "q_head_norm" + sfx, dp * z));
+    S_TRY(named_bytes(e, &L.k_head_norm, "k_head_norm" + sfx, dp * z));
+    S_TRY(named_bytes(e, &L.k_cache, "k_cache" + sfx, e->num_slots * G * dp * z));
+    S_TRY(named_bytes(e, &L.v_cache, "v_cache" + sfx, e->num_slots * G * vp * z));
+    S_TRY(rope_table(e, L, l));
+    if (c.value_mix) {
+        L.mix = HeadPrepare::kSave;
+        for (int o = 0; o < l; ++o) {
+            const b200_layer_config& f = S->layers[o].c;
+            if (f.mixer != B200_MIXER_WINDOW_ATTENTION || !f.value_mix) continue;
+            L.mix = HeadPrepare::kMix;
+            B200_CHECK_ARG(f.kv_heads == c.kv_heads && f.value_dim == c.value_dim,
+                           "layer %d: mixes %d x %d values with the %d x %d of layer %d", l, c.kv_heads, c.value_dim, f.kv_heads,
+                           f.value_dim, o);
+            break;
+        }
+        void* p = nullptr;
+        S_TRY(named_bytes(e, &p, "value_mix" + sfx, 4));
+        L.value_mix = static_cast<float*>(p);
+        Widths::widest(w.first, G * vp);
+    }
+    Widths::widest(w.joint, joint);
+    if (c.kv_heads <= 8 && 8 % c.kv_heads == 0)
+        Widths::widest(w.ws, decode_workspace_bytes(e->max_batch, c.heads, c.kv_heads));
+    return B200_OK;
+}
+
+int alloc_linear(b200_engine* e, StackLayer& L, const std::string& sfx, Widths& w) {
+    LayerStack* S = e->stack;
+    const b200_layer_config& c = L.c;
+    L.dp = pad_width(c.head_dim);
+    L.vp = pad_width(c.value_dim);
+    L.up_ld = pad_to(c.decay_rank, 16);
+    const int64_t hp = S->hp, z = S->esz, H = c.heads, dp = L.dp, vp = L.vp;
+    const int64_t joint = 2 * H * (dp + vp) + pad_width(c.decay_rank);
+    void* p = nullptr;
+    S_TRY(named_bytes(e, &L.qkvga, "qkvga" + sfx, joint * hp * z));
+    S_TRY(named_bytes(e, &L.decay_up, "decay_up" + sfx, H * dp * L.up_ld * z));
+    S_TRY(named_bytes(e, &p, "decay_bias" + sfx, H * dp * 4));
+    L.decay_bias = static_cast<float*>(p);
+    S_TRY(named_bytes(e, &L.head_norm, "head_norm" + sfx, vp * z));
+    S_TRY(named_bytes(e, &p, "state" + sfx, static_cast<int64_t>(e->pt_rows) * H * dp * vp * 4));
+    L.state = static_cast<float*>(p);
+    Widths::widest(w.joint, joint);
+    return B200_OK;
+}
+
+int alloc_feed_forward(b200_engine* e, StackLayer& L, const std::string& sfx, Widths& w) {
+    LayerStack* S = e->stack;
+    const b200_layer_config& c = L.c;
+    const int64_t hp = S->hp, z = S->esz, Tm = e->max_tokens;
+    L.ip = pad_width(c.intermediate);
+    const int64_t n_up = (epilogue_is_gated(c.epilogue) ? 2 : 1) * static_cast<int64_t>(L.ip);
+    const int64_t E = c.mlp == B200_MLP_DENSE ? 1 : c.num_experts;
+    S_TRY(named_bytes(e, &L.norm2, "norm2" + sfx, hp * z));
+    S_TRY(named_bytes(e, &L.up, "mlp_up" + sfx, E * n_up * hp * z));
+    S_TRY(named_bytes(e, &L.down, "mlp_down" + sfx, E * hp * L.ip * z));
+    if (c.mlp == B200_MLP_DENSE) {
+        Widths::widest(w.h, L.ip);
+        return B200_OK;
+    }
+    const int64_t top = c.experts_per_tok;
+    Widths::widest(w.h, top * L.ip);
+    Widths::widest(w.pairs, top);
+    void* p = nullptr;
+    if (c.mlp == B200_MLP_SCORED_MOE) {
+        w.scored = true;
+        S_TRY(named_bytes(e, &L.router, "router" + sfx, static_cast<int64_t>(pad_width(c.num_experts)) * hp * z));
+        Widths::widest(w.experts, E);
+        Widths::widest(w.router, pad_width(c.num_experts));
+        Widths::widest(w.top, top);
+        if (c.shared_intermediate > 0) {
+            L.isp = pad_width(c.shared_intermediate);
+            const int64_t n_shared = (epilogue_is_gated(c.epilogue) ? 2 : 1) * static_cast<int64_t>(L.isp);
+            S_TRY(named_bytes(e, &L.shared_up, "shared_up" + sfx, n_shared * hp * z));
+            S_TRY(named_bytes(e, &L.shared_down, "shared_down" + sfx, hp * L.isp * z));
+            Widths::widest(w.shared, L.isp);
+        }
+        return B200_OK;
+    }
+    S_TRY(named_bytes(e, &p, "expert_table" + sfx, static_cast<int64_t>(e->m.vocab_size) * top * 4));
+    L.table = static_cast<int32_t*>(p);
+    S_TRY(dev_alloc(e, &p, (Tm * top + 2 * E + 1) * 4, true));
+    L.rows = static_cast<int32_t*>(p);
+    L.counts = L.rows + Tm * top;
+    L.offsets = L.counts + E;
+    if (c.num_experts > S->max_experts) S->max_experts = c.num_experts;
+    S->routes.push_back(TableRouteLayer{L.table, L.rows, L.counts, L.offsets, c.experts_per_tok, c.num_experts});
     return B200_OK;
 }
 
@@ -136,6 +355,7 @@ int layer_stack_create(b200_engine* e, const b200_stack_config* sc) {
     S->esz = sc->dtype == B200_DTYPE_F32 ? 4 : 2;
     S->norm_offset = sc->norm_offset;
     S->logit_scale = sc->logit_scale;
+    S->norm_output = sc->norm_output != 0;
     S->hp = pad_width(e->m.hidden_size);
     S->vocab_p = pad_width(e->m.vocab_size);
     if (const char* v = getenv("B200_LATENT_EXPAND_MIN")) S->expand_min = atoi(v);
@@ -149,87 +369,43 @@ int layer_stack_create(b200_engine* e, const b200_stack_config* sc) {
     }
     S_TRY(named_bytes(e, &S->final_norm, "final_norm", hp * z));
 
-    int64_t joint = 0, cq = 0, q = 0, attn = 0, h = 0, pairs = 0, latent = 0, xk = 0, xv = 0, xc = 0, ws = 0;
+    Widths w;
     S->latent_rows = e->max_batch > 1024 ? e->max_batch : 1024;
     if (S->latent_rows > e->max_tokens) S->latent_rows = e->max_tokens;
-    bool any_expand = false;
-    auto widest = [](int64_t& a, int64_t b) { if (b > a) a = b; };
     S->layers.resize(sc->num_layers);
     for (int l = 0; l < sc->num_layers; ++l) {
         StackLayer& L = S->layers[l];
         L.c = sc->layers[l];
         const b200_layer_config& c = L.c;
         S_TRY(check_layer(c, l));
-        L.qp = pad_width(c.q_rank);
-        L.rp = pad_latent(c.kv_rank);
-        L.dp = pad_head_dim(c.head_dim);
-        L.vp = pad_head_dim(c.value_dim);
+        B200_CHECK_ARG(!(S->norm_output && c.mlp == B200_MLP_TABLE_MOE),
+                       "layer %d: experts by token id take the norm on their input", l);
         const std::string sfx = "." + std::to_string(l);
-        const int64_t H = c.heads, qp = L.qp, rp = L.rp, dp = L.dp, vp = L.vp;
         S_TRY(named_bytes(e, &L.norm1, "norm1" + sfx, hp * z));
-        S_TRY(named_bytes(e, &L.down_qkv, "down_qkv" + sfx, (qp + rp) * hp * z));
-        S_TRY(named_bytes(e, &L.q_norm, "q_latent_norm" + sfx, qp * z));
-        S_TRY(named_bytes(e, &L.kv_norm, "kv_latent_norm" + sfx, rp * z));
-        S_TRY(named_bytes(e, &L.uq, "uq" + sfx, H * dp * qp * z));
-        S_TRY(named_bytes(e, &L.uk_absorb, "uk_absorb" + sfx, H * rp * dp * z));
-        S_TRY(named_bytes(e, &L.uv, "uv" + sfx, H * vp * rp * z));
-        S_TRY(named_bytes(e, &L.o, "o" + sfx, hp * H * vp * z));
-        S_TRY(named_bytes(e, &L.cache, "latent_cache" + sfx, e->num_slots * rp * z));
-        // what the prefill kernel of the grouped-query models takes (and its positive score scale)
-        L.can_expand = S->dtype == B200_DTYPE_BF16 && dp == 128 && vp == 128 && c.score_scale > 0.f && H <= 65535;
-        if (L.can_expand) S_TRY(named_bytes(e, &L.uk, "uk" + sfx, H * dp * rp * z));
-        any_expand |= L.can_expand;
-        widest(joint, qp + rp);
-        widest(cq, qp);
-        widest(q, H * dp);
-        widest(attn, H * vp);
-        widest(latent, H * rp);
-        widest(ws, latent_attention_workspace_bytes(S->latent_rows, c.heads, L.rp));
-        if (L.can_expand) {
-            widest(xk, H * dp);
-            widest(xv, H * vp);
-            widest(xc, rp);
-        }
-        if (c.mlp == B200_MLP_NONE) continue;
-        L.ip = pad_width(c.intermediate);
-        const int64_t n_up = (epilogue_is_gated(c.epilogue) ? 2 : 1) * static_cast<int64_t>(L.ip);
-        const int64_t E = c.mlp == B200_MLP_TABLE_MOE ? c.num_experts : 1;
-        S_TRY(named_bytes(e, &L.norm2, "norm2" + sfx, hp * z));
-        S_TRY(named_bytes(e, &L.up, "mlp_up" + sfx, E * n_up * hp * z));
-        S_TRY(named_bytes(e, &L.down, "mlp_down" + sfx, E * hp * L.ip * z));
-        if (c.mlp == B200_MLP_DENSE) {
-            widest(h, L.ip);
-            continue;
-        }
-        const int64_t top = c.experts_per_tok;
-        void* p = nullptr;
-        S_TRY(named_bytes(e, &p, "expert_table" + sfx, static_cast<int64_t>(e->m.vocab_size) * top * 4));
-        L.table = static_cast<int32_t*>(p);
-        S_TRY(dev_alloc(e, &p, (Tm * top + 2 * E + 1) * 4, true));
-        L.rows = static_cast<int32_t*>(p);
-        L.counts = L.rows + Tm * top;
-        L.offsets = L.counts + E;
-        widest(h, top * L.ip);
-        widest(pairs, top);
-        if (c.num_experts > S->max_experts) S->max_experts = c.num_experts;
-        S->routes.push_back(TableRouteLayer{L.table, L.rows, L.counts, L.offsets, c.experts_per_tok, c.num_experts});
+        if (c.mixer == B200_MIXER_LATENT_ATTENTION) S_TRY(alloc_latent(e, L, sfx, w));
+        if (c.mixer == B200_MIXER_WINDOW_ATTENTION) S_TRY(alloc_window(e, L, l, sfx, w));
+        if (c.mixer == B200_MIXER_LINEAR_ATTENTION) S_TRY(alloc_linear(e, L, sfx, w));
+        const int64_t heads_out = static_cast<int64_t>(c.heads) * L.vp;
+        S_TRY(named_bytes(e, &L.o, "o" + sfx, hp * heads_out * z));
+        Widths::widest(w.attn, heads_out);
+        if (c.mlp != B200_MLP_NONE) S_TRY(alloc_feed_forward(e, L, sfx, w));
     }
     void* p = nullptr;
     S_TRY(dev_alloc(e, &p, Tm * hp * 4, true));
     S->residual = static_cast<float*>(p);
     S_TRY(dev_alloc(e, &S->x, Tm * hp * z, true));
     S_TRY(dev_alloc(e, &S->y, Tm * hp * z, true));
-    S_TRY(dev_alloc(e, &S->joint, Tm * joint * z, true));
-    S_TRY(dev_alloc(e, &S->cq, Tm * cq * z, true));
-    S_TRY(dev_alloc(e, &S->q, Tm * q * z, true));
-    S_TRY(dev_alloc(e, &S->attn, Tm * attn * z, true));
-    S_TRY(dev_alloc(e, &S->h, Tm * h * z, true));
-    S_TRY(dev_alloc(e, &S->xp, Tm * pairs * hp * z, true));
-    S_TRY(dev_alloc(e, &S->ye, Tm * pairs * hp * z, true));
-    S_TRY(dev_alloc(e, &S->qa, S->latent_rows * latent * z, true));
-    S_TRY(dev_alloc(e, &S->ol, S->latent_rows * latent * z, true));
-    S->ws_bytes = ws;
-    S_TRY(dev_alloc(e, &S->ws, ws, true));
+    S_TRY(dev_alloc(e, &S->joint, Tm * w.joint * z, true));
+    S_TRY(dev_alloc(e, &S->cq, Tm * w.cq * z, true));
+    S_TRY(dev_alloc(e, &S->q, Tm * w.q * z, true));
+    S_TRY(dev_alloc(e, &S->attn, Tm * w.attn * z, true));
+    S_TRY(dev_alloc(e, &S->h, Tm * w.h * z, true));
+    S_TRY(dev_alloc(e, &S->xp, Tm * w.pairs * hp * z, true));
+    S_TRY(dev_alloc(e, &S->ye, Tm * w.pairs * hp * z, true));
+    S_TRY(dev_alloc(e, &S->qa, S->latent_rows * w.latent * z, true));
+    S_TRY(dev_alloc(e, &S->ol, S->latent_rows * w.latent * z, true));
+    S->ws_bytes = w.ws;
+    S_TRY(dev_alloc(e, &S->ws, w.ws, true));
     S_TRY(dev_alloc(e, &p, Tm * 4, true));
     S->token_row = static_cast<int32_t*>(p);
     S_TRY(dev_alloc(e, &p, Tm * 4, true));
@@ -238,22 +414,38 @@ int layer_stack_create(b200_engine* e, const b200_stack_config* sc) {
     S->compact_row = static_cast<int32_t*>(p);
     S_TRY(dev_alloc(e, &p, Tm * 4, true));
     S->compact_len = static_cast<int32_t*>(p);
-    if (any_expand) {
+    if (w.first > 0) S_TRY(dev_alloc(e, &S->first_values, Tm * w.first * z, true));
+    if (w.scored) {
+        S_TRY(dev_alloc(e, &p, Tm * w.router * 4, true));
+        S->router_logits = static_cast<float*>(p);
+        S_TRY(dev_alloc(e, &p, Tm * w.top * 4, true));
+        S->route_weights = static_cast<float*>(p);
+        S_TRY(dev_alloc(e, &p, (2 * Tm * w.top + 3 * w.experts + 1) * 4, true));
+        S->route_ids = static_cast<int32_t*>(p);
+        S->route_rows = S->route_ids + Tm * w.top;
+        S->route_counts = S->route_rows + Tm * w.top;
+        S->route_offsets = S->route_counts + 2 * w.experts;
+        if (w.shared > 0) {
+            S_TRY(dev_alloc(e, &S->shared_h, Tm * w.shared * z, true));
+            S_TRY(dev_alloc(e, &S->shared_y, Tm * hp * z, true));
+        }
+    }
+    if (w.any_expand) {
         // room for the pool's tokens (each request rounded up to 64), at most 64 K of them, within 4 GB
         S->expand_cap = e->num_slots + 64ll * e->max_batch;
         if (S->expand_cap > 65536) S->expand_cap = 65536;
-        while (S->expand_cap > 4096 && S->expand_cap * (xk + xv) * 2 > (4ll << 30)) S->expand_cap /= 2;
+        while (S->expand_cap > 4096 && S->expand_cap * (w.xk + w.xv) * 2 > (4ll << 30)) S->expand_cap /= 2;
         S->expand_cap = S->expand_cap / 64 * 64 + 64;
-        S_TRY(dev_alloc(e, &S->xc, S->expand_cap * xc * 2, true));
-        S_TRY(dev_alloc(e, &S->xk, S->expand_cap * xk * 2, true));
-        S_TRY(dev_alloc(e, &S->xv, S->expand_cap * xv * 2, true));
+        S_TRY(dev_alloc(e, &S->xc, S->expand_cap * w.xc * 2, true));
+        S_TRY(dev_alloc(e, &S->xk, S->expand_cap * w.xk * 2, true));
+        S_TRY(dev_alloc(e, &S->xv, S->expand_cap * w.xv * 2, true));
         S_TRY(dev_alloc(e, &p, S->expand_cap * 4, false));
         S->iota = static_cast<int32_t*>(p);
         iota_kernel<<<static_cast<unsigned>((S->expand_cap + 255) / 256), 256>>>(S->iota, S->expand_cap);
         B200_CHECK_LAUNCH();
         // compacted queries and outputs of the requests that stay in the latent space beside expanded ones
-        S_TRY(dev_alloc(e, &S->qc, Tm * q * z, true));
-        S_TRY(dev_alloc(e, &S->ac, Tm * attn * z, true));
+        S_TRY(dev_alloc(e, &S->qc, Tm * w.q * z, true));
+        S_TRY(dev_alloc(e, &S->ac, Tm * w.attn * z, true));
     }
     const int64_t plan_ints = 3ll * e->max_batch + Tm;
     B200_CHECK_CUDA(cudaMallocHost(&S->plan_host, plan_ints * sizeof(int32_t)));
@@ -287,6 +479,7 @@ int layer_stack_plan(b200_engine* e, const b200_step* st, int Bp) {
     LayerStack* S = e->stack;
     S->plan_expanded = S->plan_latent = S->plan_max_extend = S->plan_max_len = 0;
     S->plan_rows = 0;
+    S->max_extend = 1;
     if (st->phase != B200_PHASE_PREFILL) return B200_OK;
     int32_t* x_len = S->plan_host;
     int32_t* x_base = x_len + Bp;
@@ -295,6 +488,7 @@ int layer_stack_plan(b200_engine* e, const b200_step* st, int Bp) {
     int at = 0;
     for (int b = 0; b < Bp; ++b) {
         const int ext = st->extend_lens[b], len = st->cached_lens[b] + ext;
+        if (ext > S->max_extend) S->max_extend = ext;
         const int64_t need = (len + 63) / 64 * 64;
         if (ext > S->expand_min && S->plan_rows + need <= S->expand_cap) {
             x_len[b] = len;
@@ -319,11 +513,11 @@ int layer_stack_plan(b200_engine* e, const b200_step* st, int Bp) {
 
 namespace {
 
-int project(b200_engine* e, void* y, const void* x, const void* w, int M, int N, int K, int epilogue) {
+int project(b200_engine* e, void* y, const void* x, const void* w, int M, int N, int K, int epilogue, float limit = 0.f) {
     if (e->stack->dtype == B200_DTYPE_F32)
         return launch_linear_f32(static_cast<float*>(y), static_cast<const float*>(x), static_cast<const float*>(w), M, N, K,
-                                 1, nullptr, nullptr, epilogue, e->stream);
-    return launch_linear(y, x, w, nullptr, M, N, K, K, epilogue, e->status, e->stream);
+                                 1, nullptr, nullptr, epilogue, e->stream, limit);
+    return launch_linear(y, x, w, nullptr, M, N, K, K, epilogue, e->status, e->stream, nullptr, limit);
 }
 
 int project_heads(b200_engine* e, void* y, const void* x, const void* w, int M, int heads, int N, int K) {
@@ -333,14 +527,14 @@ int project_heads(b200_engine* e, void* y, const void* x, const void* w, int M, 
     return launch_linear_heads(y, x, w, M, heads, N, K, e->status, e->stream);
 }
 
-int project_experts(b200_engine* e, void* y, const void* x, const void* w, const StackLayer& L, int T, int N, int K,
-                    int epilogue) {
+int project_experts(b200_engine* e, void* y, const void* x, const void* w, const StackLayer& L, const int32_t* counts,
+                    const int32_t* offsets, int T, int N, int K, int epilogue) {
     const int E = L.c.num_experts;
     if (e->stack->dtype == B200_DTYPE_F32)
         return launch_linear_f32(static_cast<float*>(y), static_cast<const float*>(x), static_cast<const float*>(w), T, N, K,
-                                 E, L.counts, L.offsets, epilogue, e->stream);
-    return launch_grouped_gemm(y, x, w, L.counts, L.offsets, E, T, static_cast<int64_t>(T) * L.c.experts_per_tok, N, K,
-                               epilogue, e->status, e->stream);
+                                 E, counts, offsets, epilogue, e->stream, L.c.act_limit);
+    return launch_grouped_gemm(y, x, w, counts, offsets, E, T, static_cast<int64_t>(T) * L.c.experts_per_tok, N, K,
+                               epilogue, e->status, e->stream, L.c.act_limit);
 }
 
 // Latent-space attention of `rows` query rows (q and out [rows, heads * dim], tables per row).
@@ -407,6 +601,191 @@ int attend(b200_engine* e, const StackLayer& L, int phase, int Bp, int T) {
     return launch_move_rows(S->attn, S->ac, tokens, n, H * L.vp / 8, true, e->stream);
 }
 
+int latent_mixer(b200_engine* e, const StackLayer& L, int T) {
+    LayerStack* S = e->stack;
+    const b200_layer_config& c = L.c;
+    S_TRY(project(e, S->joint, S->x, L.down_qkv, T, L.qp + L.rp, S->hp, B200_EPILOGUE_NONE));
+    S_TRY(launch_latent_norm_store(S->cq, L.cache, S->joint, L.q_norm, L.kv_norm, e->out_loc, T, c.q_rank, L.qp,
+                                   c.kv_rank, L.rp, e->num_slots, e->m.rms_norm_eps, S->dtype, e->status, e->stream));
+    return project(e, S->q, S->cq, L.uq, T, c.heads * L.dp, L.qp, B200_EPILOGUE_NONE);
+}
+
+int window_mixer(b200_engine* e, const StackLayer& L, int T) {
+    LayerStack* S = e->stack;
+    const b200_layer_config& c = L.c;
+    HeadPrepare a;
+    a.joint = S->joint;
+    a.ld = static_cast<int64_t>(c.heads + c.kv_heads) * (L.dp + L.vp);
+    S_TRY(project(e, S->joint, S->x, L.qkvg, T, static_cast<int>(a.ld), S->hp, B200_EPILOGUE_NONE));
+    a.tokens = T;
+    a.heads = c.heads;
+    a.kv_heads = c.kv_heads;
+    a.dim = c.head_dim;
+    a.dp = L.dp;
+    a.vp = L.vp;
+    a.q_weight = L.q_head_norm;
+    a.k_weight = L.k_head_norm;
+    a.eps = e->m.rms_norm_eps;
+    a.rotary_dim = c.rotary_dim;
+    a.max_pos = e->pt_cols;
+    a.cos_t = L.cos_t;
+    a.sin_t = L.sin_t;
+    a.positions = e->positions;
+    a.out_loc = e->out_loc;
+    a.k_cache = L.k_cache;
+    a.v_cache = L.v_cache;
+    a.num_slots = e->num_slots;
+    a.mix = L.mix;
+    a.lambda = L.value_mix;
+    a.first_values = S->first_values;
+    a.status = e->status;
+    return launch_head_prepare(a, S->dtype, e->stream);
+}
+
+int window_attend(b200_engine* e, const StackLayer& L, int phase, int Bp, int T) {
+    LayerStack* S = e->stack;
+    const b200_layer_config& c = L.c;
+    WindowAttention a;
+    a.out = S->attn;
+    a.q = S->joint;
+    a.q_st = static_cast<int64_t>(c.heads + c.kv_heads) * (L.dp + L.vp);
+    a.k_cache = L.k_cache;
+    a.v_cache = L.v_cache;
+    a.num_slots = e->num_slots;
+    a.page_table = e->page_table;
+    a.pt_stride = e->pt_cols;
+    a.table_idx = e->meta_dev;
+    a.seq_lens = e->seq_lens;
+    a.qo_indptr = e->meta_dev + 2 * Bp;
+    a.row_table = S->token_row;
+    a.row_len = S->token_len;
+    a.tokens = T;
+    a.batch = Bp;
+    a.max_extend = S->max_extend;
+    a.decode = phase == B200_PHASE_DECODE;
+    a.heads = c.heads;
+    a.kv_heads = c.kv_heads;
+    a.dp = L.dp;
+    a.vp = L.vp;
+    a.page_size = e->c.page_size;
+    a.scale = c.score_scale;
+    a.window.size = c.window;
+    a.window.keep_first = c.keep_first;
+    a.window.gate = static_cast<const char*>(S->joint) +
+                    (static_cast<int64_t>(c.heads + c.kv_heads) * L.dp + static_cast<int64_t>(c.kv_heads) * L.vp) * S->esz;
+    a.window.gate_st = a.q_st;
+    a.workspace = S->ws;
+    a.workspace_bytes = S->ws_bytes;
+    a.status = e->status;
+    return launch_window_attention(a, S->dtype, e->stream);
+}
+
+int linear_mixer(b200_engine* e, const StackLayer& L, int phase, int Bp, int T) {
+    LayerStack* S = e->stack;
+    const b200_layer_config& c = L.c;
+    LinearAttention a = {};
+    a.out = S->attn;
+    a.joint = S->joint;
+    a.joint_ld = 2ll * c.heads * (L.dp + L.vp) + pad_width(c.decay_rank);
+    S_TRY(project(e, S->joint, S->x, L.qkvga, T, static_cast<int>(a.joint_ld), S->hp, B200_EPILOGUE_NONE));
+    a.tokens = T;
+    a.batch = Bp;
+    a.decode = phase == B200_PHASE_DECODE ? 1 : 0;
+    a.table_idx = e->meta_dev;
+    a.cached = e->meta_dev + Bp;
+    a.qo_indptr = e->meta_dev + 2 * Bp;
+    a.state = L.state;
+    a.heads = c.heads;
+    a.dim = c.head_dim;
+    a.padded_dim = L.dp;
+    a.value_dim = c.value_dim;
+    a.padded_value_dim = L.vp;
+    a.rank = c.decay_rank;
+    a.up_ld = L.up_ld;
+    a.up = L.decay_up;
+    a.bias = L.decay_bias;
+    a.norm = L.head_norm;
+    a.tau = c.decay_tau;
+    a.eps = e->m.rms_norm_eps;
+    a.q_scale = static_cast<float>(1.0 / sqrt(static_cast<double>(c.head_dim)));
+    return launch_linear_attention(a, S->dtype, e->stream);
+}
+
+// S->x through the layer's mixer to S->y.
+int mix(b200_engine* e, int l, int phase, int Bp, int T) {
+    LayerStack* S = e->stack;
+    const StackLayer& L = S->layers[l];
+    cudaStream_t s = e->stream;
+    if (L.c.mixer == B200_MIXER_LINEAR_ATTENTION) {
+        S_TRY(linear_mixer(e, L, phase, Bp, T));
+        return project(e, S->y, S->attn, L.o, T, S->hp, L.c.heads * L.vp, B200_EPILOGUE_NONE);
+    }
+    const bool latent = L.c.mixer == B200_MIXER_LATENT_ATTENTION;
+    S_TRY(latent ? latent_mixer(e, L, T) : window_mixer(e, L, T));
+    const bool timed = e->profile_attention && !e->capturing;
+    const int at = e->prof_pairs_recorded;
+    if (timed) {
+        while (static_cast<int>(e->prof_events.size()) < 2 * (at + 1)) {
+            cudaEvent_t ev = nullptr;
+            B200_CHECK_CUDA(cudaEventCreate(&ev));
+            e->prof_events.push_back(ev);
+        }
+        B200_CHECK_CUDA(cudaEventRecord(e->prof_events[2 * at], s));
+    }
+    S_TRY(latent ? attend(e, L, phase, Bp, T) : window_attend(e, L, phase, Bp, T));
+    if (timed) {
+        B200_CHECK_CUDA(cudaEventRecord(e->prof_events[2 * at + 1], s));
+        e->prof_pairs_recorded = at + 1;
+    }
+    return project(e, S->y, S->attn, L.o, T, S->hp, L.c.heads * L.vp, B200_EPILOGUE_NONE);
+}
+
+// S->x through a dense layer to S->y, or through the experts its scores choose to S->ye (and the expert that
+// every token uses to S->shared_y).
+int feed_forward(b200_engine* e, const StackLayer& L, int T) {
+    LayerStack* S = e->stack;
+    const b200_layer_config& c = L.c;
+    const int hp = S->hp, gated = epilogue_is_gated(c.epilogue) ? 2 : 1;
+    if (c.mlp == B200_MLP_DENSE) {
+        S_TRY(project(e, S->h, S->x, L.up, T, gated * L.ip, hp, c.epilogue, c.act_limit));
+        return project(e, S->y, S->h, L.down, T, hp, L.ip, B200_EPILOGUE_NONE);
+    }
+    const int ep = pad_width(c.num_experts);
+    S_TRY(project(e, S->router_logits, S->x, L.router, T, ep, hp,
+                  S->dtype == B200_DTYPE_F32 ? B200_EPILOGUE_NONE : B200_EPILOGUE_F32));
+    ScoreRoute r;
+    r.logits = S->router_logits;
+    r.ld = ep;
+    r.tokens = T;
+    r.experts = c.num_experts;
+    r.top = c.experts_per_tok;
+    r.groups = c.router_groups;
+    r.keep = c.router_keep;
+    r.scale = c.router_scale;
+    r.ids = S->route_ids;
+    r.weights = S->route_weights;
+    r.counts = S->route_counts;
+    S_TRY(launch_score_route(r, e->stream));
+    S_TRY(launch_score_place(S->xp, S->x, hp * S->esz, r, S->route_rows, S->route_counts + c.num_experts, S->route_offsets,
+                             e->stream));
+    S_TRY(project_experts(e, S->h, S->xp, L.up, L, r.counts, S->route_offsets, T, gated * L.ip, hp, c.epilogue));
+    S_TRY(project_experts(e, S->ye, S->h, L.down, L, r.counts, S->route_offsets, T, hp, L.ip, B200_EPILOGUE_NONE));
+    if (L.isp == 0) return B200_OK;
+    S_TRY(project(e, S->shared_h, S->x, L.shared_up, T, gated * L.isp, hp, c.epilogue, c.shared_act_limit));
+    return project(e, S->shared_y, S->shared_h, L.shared_down, T, hp, L.isp, B200_EPILOGUE_NONE);
+}
+
+// What a block has left behind for the residual kernel that follows it.
+void take_block(LayerStack* S, const StackLayer* experts, int T, ResidualPostNorm& rn) {
+    rn.init = false;
+    rn.src = experts ? S->ye : S->y;
+    rn.src_rows = experts ? S->route_rows : nullptr;
+    rn.src_weights = experts ? S->route_weights : nullptr;
+    rn.src_top = experts ? experts->c.experts_per_tok : 1;
+    rn.src_count = static_cast<int64_t>(T) * rn.src_top;
+    rn.src2 = experts && experts->isp > 0 ? S->shared_y : nullptr;
+}
+
 }  // namespace
 
 int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
@@ -414,6 +793,7 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
     cudaStream_t s = e->stream;
     const int hp = S->hp, width = e->m.hidden_size;
     const int num_layers = static_cast<int>(S->layers.size());
+    e->prof_pairs_recorded = 0;
     if (!S->routes.empty())
         S_TRY(launch_table_route(S->routes_dev, static_cast<int>(S->routes.size()), S->max_experts, e->input_ids, T,
                                  e->m.vocab_size, e->status, s));
@@ -422,7 +802,8 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
                                       dim3(1, 1, 1), S->compact_row, S->compact_len,
                                       static_cast<const int32_t*>(S->token_row), static_cast<const int32_t*>(S->token_len),
                                       static_cast<const int32_t*>(S->plan_dev + 3 * Bp), S->plan_latent));
-    // What the next residual update adds: at first the embedding rows of the tokens.
+    // What the next residual update adds: at first the embedding rows of the tokens.  `rn` drives the kernel with
+    // the norm on what is read, `post` the one with the norm on what is added (and with weighted sources).
     ResidualNorm rn;
     rn.residual = S->residual;
     rn.weight_offset = S->norm_offset;
@@ -435,6 +816,20 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
     rn.src_top = 1;
     rn.src_count = e->m.vocab_size;
     rn.init = true;
+    ResidualPostNorm post;
+    post.out = S->x;
+    post.residual = S->residual;
+    post.src = S->embed;
+    post.src_rows = e->input_ids;
+    post.src_count = e->m.vocab_size;
+    post.init = true;
+    post.weight_offset = S->norm_offset;
+    post.tokens = T;
+    post.width = width;
+    post.padded = hp;
+    post.eps = e->m.rms_norm_eps;
+    const StackLayer* scored = nullptr;   // the last block was this layer's scored experts
+    const void* own_norm = nullptr;       // norm_output: the norm of the last block's output
     auto add_plain = [&]() {
         rn.src = S->y;
         rn.src_rows = nullptr;
@@ -442,14 +837,26 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
         rn.src_count = T;
         rn.src_scale = 1.f;
         rn.init = false;
+        scored = nullptr;
     };
-    auto norm_to = [&](const void* weight, void* out, const int32_t* rows, int top, float out_scale) -> int {
-        rn.weight = weight;
-        rn.out = out;
-        rn.out_rows = rows;
-        rn.out_top = top;
-        rn.out_scale = out_scale;
-        return launch_residual_norm(rn, S->dtype, e->status, s);
+    // Adds the last block and leaves what the next one reads: normalised with `weight`, or as it is.
+    auto advance = [&](const void* weight, void* out, const int32_t* rows, int top, float out_scale,
+                       const StackLayer* next_scored) -> int {
+        post.clear = next_scored ? S->route_counts : nullptr;
+        post.clear_count = next_scored ? 2 * next_scored->c.num_experts : 0;
+        if (!S->norm_output && scored == nullptr && next_scored == nullptr) {
+            rn.weight = weight;
+            rn.out = out;
+            rn.out_rows = rows;
+            rn.out_top = top;
+            rn.out_scale = out_scale;
+            return launch_residual_norm(rn, S->dtype, e->status, s);
+        }
+        if (!rn.init) take_block(S, scored, T, post);
+        post.add_weight = own_norm;
+        post.out_weight = weight;
+        post.out_scale = out_scale;
+        return launch_residual_post_norm(post, S->dtype, e->status, s);
     };
     // (the residual after layer l is complete once the kernel that opens what follows it has run)
     auto traced = [&](int layers_done) -> int {
@@ -463,49 +870,33 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
         const b200_layer_config& c = L.c;
         // The first norm is launched as an ordinary dependent of what prepares the step, so that every
         // kernel after it finds positions, slots and lengths complete even ahead of its own wait.
-        S_TRY(norm_to(L.norm1, S->x, nullptr, 1, 1.f));
+        S_TRY(advance(S->norm_output ? nullptr : L.norm1, S->x, nullptr, 1, 1.f, nullptr));
         if (l == 0) set_pdl_launches(pdl);
         S_TRY(traced(l));
-        S_TRY(project(e, S->joint, S->x, L.down_qkv, T, L.qp + L.rp, hp, B200_EPILOGUE_NONE));
-        S_TRY(launch_latent_norm_store(S->cq, L.cache, S->joint, L.q_norm, L.kv_norm, e->out_loc, T, c.q_rank, L.qp,
-                                       c.kv_rank, L.rp, e->num_slots, e->m.rms_norm_eps, S->dtype, e->status, s));
-        S_TRY(project(e, S->q, S->cq, L.uq, T, c.heads * L.dp, L.qp, B200_EPILOGUE_NONE));
-        const bool timed = e->profile_attention && !e->capturing;
-        if (timed) {
-            while (static_cast<int>(e->prof_events.size()) < 2 * num_layers) {
-                cudaEvent_t ev = nullptr;
-                B200_CHECK_CUDA(cudaEventCreate(&ev));
-                e->prof_events.push_back(ev);
-            }
-            B200_CHECK_CUDA(cudaEventRecord(e->prof_events[2 * l], s));
-        }
-        S_TRY(attend(e, L, phase, Bp, T));
-        if (timed) {
-            B200_CHECK_CUDA(cudaEventRecord(e->prof_events[2 * l + 1], s));
-            e->prof_pairs_recorded = l + 1;
-        }
-        S_TRY(project(e, S->y, S->attn, L.o, T, hp, c.heads * L.vp, B200_EPILOGUE_NONE));
+        S_TRY(mix(e, l, phase, Bp, T));
         add_plain();
+        if (S->norm_output) own_norm = L.norm1;
         if (c.mlp == B200_MLP_NONE) continue;
-        const int n_up = (epilogue_is_gated(c.epilogue) ? 2 : 1) * L.ip;
-        if (c.mlp == B200_MLP_DENSE) {
-            S_TRY(norm_to(L.norm2, S->x, nullptr, 1, 1.f));
-            S_TRY(project(e, S->h, S->x, L.up, T, n_up, hp, c.epilogue));
-            S_TRY(project(e, S->y, S->h, L.down, T, hp, L.ip, B200_EPILOGUE_NONE));
-            add_plain();
-        } else {
-            S_TRY(norm_to(L.norm2, S->xp, L.rows, c.experts_per_tok, 1.f));
-            S_TRY(project_experts(e, S->h, S->xp, L.up, L, T, n_up, hp, c.epilogue));
-            S_TRY(project_experts(e, S->ye, S->h, L.down, L, T, hp, L.ip, B200_EPILOGUE_NONE));
+        if (c.mlp == B200_MLP_TABLE_MOE) {
+            const int n_up = (epilogue_is_gated(c.epilogue) ? 2 : 1) * L.ip;
+            S_TRY(advance(L.norm2, S->xp, L.rows, c.experts_per_tok, 1.f, nullptr));
+            S_TRY(project_experts(e, S->h, S->xp, L.up, L, L.counts, L.offsets, T, n_up, hp, c.epilogue));
+            S_TRY(project_experts(e, S->ye, S->h, L.down, L, L.counts, L.offsets, T, hp, L.ip, B200_EPILOGUE_NONE));
             rn.src = S->ye;
             rn.src_rows = L.rows;
             rn.src_top = c.experts_per_tok;
             rn.src_count = static_cast<int64_t>(T) * c.experts_per_tok;
             rn.src_scale = 1.f / static_cast<float>(c.experts_per_tok);
             rn.init = false;
+            continue;
         }
+        S_TRY(advance(S->norm_output ? nullptr : L.norm2, S->x, nullptr, 1, 1.f, c.mlp == B200_MLP_SCORED_MOE ? &L : nullptr));
+        S_TRY(feed_forward(e, L, T));
+        add_plain();
+        if (c.mlp == B200_MLP_SCORED_MOE) scored = &L;
+        if (S->norm_output) own_norm = L.norm2;
     }
-    S_TRY(norm_to(S->final_norm, S->x, nullptr, 1, S->logit_scale));
+    S_TRY(advance(S->final_norm, S->x, nullptr, 1, S->logit_scale, nullptr));
     return traced(num_layers);
 }
 

@@ -19,6 +19,7 @@ struct F32Params {
     const int32_t* counts;     // grouped mode
     const int32_t* offsets;
     int per_head;              // z selects a column block of x and y
+    float act_limit;
 };
 
 __device__ __forceinline__ float gate_f32(int epi, float g) {
@@ -91,7 +92,11 @@ linear_f32_kernel(const F32Params p) {
             const int n = n0 + tx * 4 + j;
             if (n >= p.n_out) continue;
             float v = acc[i][j];
-            if (GATED) v = gate_f32(EPI, v) * up[GATED ? i : 0][j];
+            if (EPI == B200_EPILOGUE_CLAMPED_SWIGLU)
+                v = clamped_swiglu<true>(v, up[GATED ? i : 0][j], p.act_limit);
+            else if (GATED)
+                v = gate_f32(EPI, v) * up[GATED ? i : 0][j];
+            if (EPI == B200_EPILOGUE_GELU_ERF) v = gate_f32(B200_EPILOGUE_GEGLU_ERF, v);
             if (EPI == B200_EPILOGUE_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
             y[static_cast<int64_t>(m) * p.y_pitch + n] = v;
         }
@@ -101,7 +106,8 @@ linear_f32_kernel(const F32Params p) {
 }  // namespace
 
 int launch_linear_f32(float* y, const float* x, const float* w, int max_rows, int N, int K, int groups,
-                      const int32_t* counts, const int32_t* offsets, int epilogue, cudaStream_t stream) {
+                      const int32_t* counts, const int32_t* offsets, int epilogue, cudaStream_t stream,
+                      float act_limit) {
     if (max_rows == 0 || groups == 0) return B200_OK;
     const bool per_head = counts == nullptr && groups > 1;
     F32Params p;
@@ -117,11 +123,14 @@ int launch_linear_f32(float* y, const float* x, const float* w, int max_rows, in
     p.counts = counts;
     p.offsets = offsets;
     p.per_head = per_head ? 1 : 0;
+    p.act_limit = act_limit;
     void (*kernel)(F32Params) = linear_f32_kernel<B200_EPILOGUE_NONE>;
     if (epilogue == B200_EPILOGUE_SWIGLU) kernel = linear_f32_kernel<B200_EPILOGUE_SWIGLU>;
     if (epilogue == B200_EPILOGUE_GEGLU) kernel = linear_f32_kernel<B200_EPILOGUE_GEGLU>;
     if (epilogue == B200_EPILOGUE_GEGLU_ERF) kernel = linear_f32_kernel<B200_EPILOGUE_GEGLU_ERF>;
     if (epilogue == B200_EPILOGUE_RELU2) kernel = linear_f32_kernel<B200_EPILOGUE_RELU2>;
+    if (epilogue == B200_EPILOGUE_GELU_ERF) kernel = linear_f32_kernel<B200_EPILOGUE_GELU_ERF>;
+    if (epilogue == B200_EPILOGUE_CLAMPED_SWIGLU) kernel = linear_f32_kernel<B200_EPILOGUE_CLAMPED_SWIGLU>;
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(div_ceil(p.n_out, kTile), div_ceil(max_rows, kTile), groups), dim3(256), 0,
                                   stream, dim3(1, 1, 1), p));
     return B200_OK;

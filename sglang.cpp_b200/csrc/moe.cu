@@ -220,6 +220,150 @@ table_route_kernel(const TableRouteLayer* __restrict__ layers, const int32_t* __
     for (int i = threadIdx.x; i < pairs; i += blockDim.x) L.rows[i] = atomicAdd(&s_cnt[expert_of(i)], 1);
 }
 
+// Scored routing: sigmoid scores in fp32, optionally only inside the best groups of neighbouring experts (a
+// group counts for the sum of its two best), the best `top` of them, weights = scores over their sum.  One
+// warp per token; ties go to the lower index.
+struct ScoreRouteArgs {
+    const float* logits;     // [tokens, ld]
+    int64_t ld;
+    int tokens, experts, top, groups, keep;
+    float scale;
+    int32_t* ids;            // [tokens, top]
+    float* weights;          // [tokens, top]
+    int32_t* counts;         // [experts], zero before
+    int smem_floats;         // per warp: scores | group scores | chosen scores
+};
+
+__device__ __forceinline__ void warp_argmax(float& best, int& at) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float b = __shfl_xor_sync(0xffffffffu, best, o);
+        const int i = __shfl_xor_sync(0xffffffffu, at, o);
+        if (b > best || (b == best && i < at)) {
+            best = b;
+            at = i;
+        }
+    }
+}
+
+__global__ void __launch_bounds__(128)
+score_route_kernel(const ScoreRouteArgs a) {
+    extern __shared__ float s_route[];
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int64_t t = static_cast<int64_t>(blockIdx.x) * (blockDim.x >> 5) + warp;
+    if (t >= a.tokens) return;
+    constexpr float kTaken = -2.f, kOut = -1.f;   // below every score
+    float* score = s_route + static_cast<int64_t>(warp) * a.smem_floats;
+    float* group = score + a.experts;
+    float* chosen = group + a.groups;
+    for (int e = lane; e < a.experts; e += 32) score[e] = 1.f / (1.f + expf(-a.logits[t * a.ld + e]));
+    __syncwarp();
+    if (a.keep < a.groups) {
+        const int size = a.experts / a.groups;
+        for (int g = lane; g < a.groups; g += 32) {
+            float first = kOut, second = kOut;
+            for (int i = 0; i < size; ++i) {
+                const float s = score[g * size + i];
+                if (s > first) {
+                    second = first;
+                    first = s;
+                } else if (s > second) {
+                    second = s;
+                }
+            }
+            group[g] = first + (size > 1 ? second : 0.f);
+        }
+        __syncwarp();
+        for (int k = 0; k < a.keep; ++k) {
+            float best = kOut;
+            int at = 0x7fffffff;
+            for (int g = lane; g < a.groups; g += 32)
+                if (group[g] > best) {
+                    best = group[g];
+                    at = g;
+                }
+            warp_argmax(best, at);
+            if (lane == 0 && at < a.groups) group[at] = kTaken;
+            __syncwarp();
+        }
+        for (int e = lane; e < a.experts; e += 32)
+            if (group[e / size] != kTaken) score[e] = kOut;
+        __syncwarp();
+    }
+    float sum = 0.f;
+    for (int k = 0; k < a.top; ++k) {
+        float best = kOut;
+        int at = 0x7fffffff;
+        for (int e = lane; e < a.experts; e += 32)
+            if (score[e] > best) {
+                best = score[e];
+                at = e;
+            }
+        warp_argmax(best, at);
+        if (at >= a.experts) {   // NaN logits: a valid expert all the same
+            at = 0;
+            best = 0.f;
+        }
+        sum += best;
+        if (lane == 0) {
+            score[at] = kTaken;
+            chosen[k] = best;
+            a.ids[t * a.top + k] = at;
+            atomicAdd(&a.counts[at], 1);
+        }
+        __syncwarp();
+    }
+    for (int k = lane; k < a.top; k += 32) a.weights[t * a.top + k] = chosen[k] / (sum + 1e-20f) * a.scale;
+}
+
+// A row among its expert's for every choice of a token, and the token's activations copied there.  The first
+// rows of the experts follow from the counts, so no scan runs in between; one CTA per token.
+__global__ void __launch_bounds__(128)
+score_place_kernel(uint4* __restrict__ xp, const uint4* __restrict__ x, int32_t* __restrict__ rows,
+                   const int32_t* __restrict__ ids, const int32_t* __restrict__ counts, int32_t* __restrict__ cursor,
+                   int32_t* __restrict__ offsets, int experts, int top, int vec_per_row) {
+    extern __shared__ int s_place[];
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    const int64_t t = blockIdx.x;
+    for (int k = warp; k < top; k += warps) {
+        const int e = ids[t * top + k];
+        int before = 0;
+        for (int i = lane; i < e; i += 32) before += counts[i];
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) before += __shfl_xor_sync(0xffffffffu, before, o);
+        if (lane == 0) {
+            const int row = before + atomicAdd(&cursor[e], 1);
+            s_place[k] = row;
+            rows[t * top + k] = row;
+        }
+    }
+    if (t == 0 && warp == warps - 1) {
+        int carry = 0;
+        for (int base = 0; base < experts; base += 32) {
+            const int e = base + lane;
+            const int n = e < experts ? counts[e] : 0;
+            int incl = n;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int up = __shfl_up_sync(0xffffffffu, incl, o);
+                if (lane >= o) incl += up;
+            }
+            if (e < experts) offsets[e] = carry + incl - n;
+            carry += __shfl_sync(0xffffffffu, incl, 31);
+        }
+        if (lane == 0) offsets[experts] = carry;
+    }
+    __syncthreads();
+    for (int v = threadIdx.x; v < vec_per_row; v += blockDim.x) {
+        const uint4 u = x[t * vec_per_row + v];
+        for (int k = 0; k < top; ++k) xp[static_cast<int64_t>(s_place[k]) * vec_per_row + v] = u;
+    }
+}
+
 struct MoeWorkspace {
     int32_t *ids, *counts, *offsets, *cursor, *pos;
     float* weights;
@@ -260,6 +404,38 @@ int launch_table_route(const TableRouteLayer* layers_dev, int num_layers, int ma
     if (tokens == 0 || num_layers == 0) return B200_OK;
     B200_CHECK_CUDA(launch_kernel(table_route_kernel, dim3(num_layers), dim3(1024), max_experts * sizeof(int), stream,
                                   dim3(1, 1, 1), layers_dev, token_ids, tokens, vocab, status));
+    return B200_OK;
+}
+
+int launch_score_route(const ScoreRoute& r, cudaStream_t stream) {
+    if (r.tokens == 0) return B200_OK;
+    ScoreRouteArgs a;
+    a.logits = r.logits;
+    a.ld = r.ld;
+    a.tokens = r.tokens;
+    a.experts = r.experts;
+    a.top = r.top;
+    a.groups = r.groups;
+    a.keep = r.keep;
+    a.scale = r.scale;
+    a.ids = r.ids;
+    a.weights = r.weights;
+    a.counts = r.counts;
+    a.smem_floats = r.experts + r.groups + r.top;
+    // few tokens: one warp per CTA, spread over the SMs
+    const int warps = r.tokens >= 1024 && r.experts <= 1024 ? 4 : 1;
+    B200_CHECK_CUDA(launch_kernel(score_route_kernel, dim3(div_ceil(r.tokens, warps)), dim3(32 * warps),
+                                  static_cast<size_t>(warps) * a.smem_floats * 4, stream, dim3(1, 1, 1), a));
+    return B200_OK;
+}
+
+int launch_score_place(void* xp, const void* x, int row_bytes, const ScoreRoute& r, int32_t* rows, int32_t* cursor,
+                       int32_t* offsets, cudaStream_t stream) {
+    if (r.tokens == 0) return B200_OK;
+    B200_CHECK_CUDA(launch_kernel(score_place_kernel, dim3(r.tokens), dim3(128), static_cast<size_t>(r.top) * 4, stream,
+                                  dim3(1, 1, 1), static_cast<uint4*>(xp), static_cast<const uint4*>(x), rows,
+                                  static_cast<const int32_t*>(r.ids), static_cast<const int32_t*>(r.counts), cursor,
+                                  offsets, r.experts, r.top, row_bytes / 16));
     return B200_OK;
 }
 
@@ -355,6 +531,34 @@ int b200_table_route(int32_t* rows, int32_t* counts, int32_t* offsets, const int
     cudaFree(dev);
     B200_CHECK_CUDA(ce);
     return err;
+}
+
+int b200_score_route(int32_t* ids, float* weights, int32_t* rows, int32_t* counts, int32_t* offsets, void* xp,
+                     const void* x, int row_bytes, const float* logits, int64_t logits_ld, int tokens, int experts,
+                     int top, int groups, int keep_groups, float scale, b200_stream_t stream) {
+    B200_CHECK_ARG(tokens >= 0 && experts > 0 && experts <= b200::kMaxTableExperts && top > 0 && groups > 0 &&
+                       experts % groups == 0 && keep_groups > 0 && keep_groups <= groups &&
+                       top <= experts / groups * keep_groups, "score_route: bad shape");
+    B200_CHECK_ARG(row_bytes > 0 && row_bytes % 16 == 0 && logits_ld >= experts, "score_route: bad row size");
+    if (tokens == 0) return B200_OK;
+    B200_CHECK_ARG(ids && weights && rows && counts && offsets && xp && x && logits, "score_route: NULL tensor");
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    B200_CHECK_CUDA(cudaMemsetAsync(counts, 0, 2ll * experts * 4, s));
+    b200::ScoreRoute r;
+    r.logits = logits;
+    r.ld = logits_ld;
+    r.tokens = tokens;
+    r.experts = experts;
+    r.top = top;
+    r.groups = groups;
+    r.keep = keep_groups;
+    r.scale = scale;
+    r.ids = ids;
+    r.weights = weights;
+    r.counts = counts;
+    int err = b200::launch_score_route(r, s);
+    if (err != B200_OK) return err;
+    return b200::launch_score_place(xp, x, row_bytes, r, rows, counts + experts, offsets, s);
 }
 
 int b200_moe_forward_local(void* out, const void* hidden_states, const void* router_logits,

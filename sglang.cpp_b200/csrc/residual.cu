@@ -2,6 +2,9 @@
 // embedding row, a projection's output, or the weighted outputs of a token's experts), stores the sum and
 // writes its RMS norm for the next block - to the token's own row, or straight into the expert-sorted
 // rows that the next block's grouped GEMM reads.  One CTA per token, the row in registers.
+//
+// Two wirings: the norm on what the next block reads (residual_norm_kernel), or on what the previous block
+// returned, before it is added (residual_post_norm_kernel).
 #include "common.cuh"
 #include "kernels.h"
 
@@ -147,7 +150,201 @@ auto kernel_for(int pieces) {   // pieces of 8 elements per thread
     return pieces <= 1 ? residual_norm_kernel<T, 1> : pieces <= 2 ? residual_norm_kernel<T, 2> : residual_norm_kernel<T, 4>;
 }
 
+struct PostArgs {
+    void* out;
+    float* residual;
+    const void* src;
+    const int32_t* src_rows;
+    const float* src_weights;
+    const void* src2;
+    const void* add_weight;
+    const void* out_weight;
+    int64_t src_count;
+    int src_top, init, width, padded;
+    float weight_offset, out_scale, eps;
+    int32_t* clear;
+    int clear_count;
+    int* status;
+};
+
+// What is added is a token's row of the source, or the weighted rows src_rows names, plus its row of a second
+// source; it is RMS-normalised when there is a weight for it.  The sum goes to the residual and, rounded (or
+// normalised once more, before the output head), to `out`.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+residual_post_norm_kernel(const PostArgs a) {
+    __shared__ float red[2][8];
+    __shared__ int s_row[kRows];
+    __shared__ float s_weight[kRows];
+    pdl_launch_dependents();
+    const int nvec = a.padded >> 3;
+    const T* add_weight = static_cast<const T*>(a.add_weight);
+    const T* out_weight = static_cast<const T*>(a.out_weight);
+    // the norm weights do not come from the kernel before this one
+    Vec8 w[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+        const int v = threadIdx.x + i * blockDim.x;
+        if (v < nvec && add_weight != nullptr) w[i] = load8(add_weight + v * 8);
+    }
+    pdl_wait_prior();
+    const int64_t t = blockIdx.x;
+    if (blockIdx.x == 0)
+        for (int i = threadIdx.x; i < a.clear_count; i += blockDim.x) a.clear[i] = 0;
+    if (a.src_rows != nullptr) {
+        if (threadIdx.x < kRows && threadIdx.x < a.src_top) {
+            s_row[threadIdx.x] = a.src_rows[t * a.src_top + threadIdx.x];
+            s_weight[threadIdx.x] = a.src_weights != nullptr ? a.src_weights[t * a.src_top + threadIdx.x] : 1.f;
+        }
+        __syncthreads();
+    }
+    float* res = a.residual + t * a.padded;
+    const T* src = static_cast<const T*>(a.src);
+    const T* src2 = static_cast<const T*>(a.src2);
+    auto addend = [&](int v) {
+        Vec8 y;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) y.v[j] = 0.f;
+        if (a.src_rows == nullptr) {
+            y = load8(src + t * a.padded + v * 8);
+        } else {
+#pragma unroll 4
+            for (int k = 0; k < a.src_top; ++k) {
+                const int64_t row = k < kRows ? s_row[k] : a.src_rows[t * a.src_top + k];
+                const float g = k < kRows ? s_weight[k] : a.src_weights != nullptr ? a.src_weights[t * a.src_top + k] : 1.f;
+                if (row < 0 || row >= a.src_count) {   // adds nothing and is reported
+                    if (v == 0) atomicExch(&a.status[kStatusBadIndex], static_cast<int>(row) + 1);
+                    continue;
+                }
+                const Vec8 x = load8(src + row * a.padded + v * 8);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) y.v[j] += g * x.v[j];
+            }
+        }
+        if (src2 != nullptr) {
+            const Vec8 x = load8(src2 + t * a.padded + v * 8);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) y.v[j] += x.v[j];
+        }
+        return y;
+    };
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    auto block_sum = [&](float x, float* scratch) {
+        x = warp_sum(x);
+        if (lane == 0) scratch[warp] = x;
+        __syncthreads();
+        return warp_sum(lane < static_cast<int>(blockDim.x >> 5) ? scratch[lane] : 0.f);
+    };
+    Vec8 val[VEC], add[VEC];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+        const int v = threadIdx.x + i * blockDim.x;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) val[i].v[j] = add[i].v[j] = 0.f;
+        if (v < nvec) {
+            if (!a.init) val[i] = load8(static_cast<const float*>(res) + v * 8);
+            add[i] = addend(v);
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ss += add[i].v[j] * add[i].v[j];
+    }
+    const int wide0 = threadIdx.x + VEC * static_cast<int>(blockDim.x);   // rows wider than the registers
+    float scale = 1.f;
+    if (add_weight != nullptr) {
+        for (int v = wide0; v < nvec; v += blockDim.x) {
+            const Vec8 y = addend(v);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) ss += y.v[j] * y.v[j];
+        }
+        scale = rsqrtf(block_sum(ss, red[0]) / static_cast<float>(a.width) + a.eps);
+    }
+    float ss2 = 0.f;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+        const int v = threadIdx.x + i * blockDim.x;
+        if (v >= nvec) continue;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            val[i].v[j] += add_weight != nullptr ? add[i].v[j] * scale * (w[i].v[j] + a.weight_offset) : add[i].v[j];
+            ss2 += val[i].v[j] * val[i].v[j];
+        }
+        store8(res + v * 8, val[i]);
+    }
+    for (int v = wide0; v < nvec; v += blockDim.x) {
+        const Vec8 y = addend(v);
+        Vec8 x, g;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            x.v[j] = 0.f;
+            g.v[j] = 1.f - a.weight_offset;
+        }
+        if (!a.init) x = load8(static_cast<const float*>(res) + v * 8);
+        if (add_weight != nullptr) g = load8(add_weight + v * 8);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            x.v[j] += y.v[j] * scale * (g.v[j] + a.weight_offset);
+            ss2 += x.v[j] * x.v[j];
+        }
+        store8(res + v * 8, x);
+    }
+    float out_scale = 1.f;
+    if (out_weight != nullptr)
+        out_scale = rsqrtf(block_sum(ss2, red[1]) / static_cast<float>(a.width) + a.eps) * a.out_scale;
+    T* out = static_cast<T*>(a.out) + t * a.padded;
+    auto emit = [&](int v, Vec8 x) {
+        if (out_weight != nullptr) {
+            const Vec8 g = load8(out_weight + v * 8);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x.v[j] *= out_scale * (g.v[j] + a.weight_offset);
+        }
+        store8(out + v * 8, x);
+    };
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+        const int v = threadIdx.x + i * blockDim.x;
+        if (v < nvec) emit(v, val[i]);
+    }
+    for (int v = wide0; v < nvec; v += blockDim.x) emit(v, load8(static_cast<const float*>(res) + v * 8));
+}
+
+template <typename T>
+auto post_kernel_for(int pieces) {
+    return pieces <= 1 ? residual_post_norm_kernel<T, 1>
+                       : pieces <= 2 ? residual_post_norm_kernel<T, 2> : residual_post_norm_kernel<T, 4>;
+}
+
 }  // namespace
+
+int launch_residual_post_norm(const ResidualPostNorm& r, int dtype, int* status, cudaStream_t stream) {
+    if (r.tokens == 0) return B200_OK;
+    PostArgs a;
+    a.out = r.out;
+    a.residual = r.residual;
+    a.src = r.src;
+    a.src_rows = r.src_rows;
+    a.src_weights = r.src_weights;
+    a.src2 = r.src2;
+    a.add_weight = r.add_weight;
+    a.out_weight = r.out_weight;
+    a.src_count = r.src_count;
+    a.src_top = r.src_rows ? r.src_top : 1;
+    a.init = r.init ? 1 : 0;
+    a.width = r.width;
+    a.padded = r.padded;
+    a.weight_offset = r.weight_offset;
+    a.out_scale = r.out_scale;
+    a.eps = r.eps;
+    a.clear = r.clear;
+    a.clear_count = r.clear ? r.clear_count : 0;
+    a.status = status;
+    int threads = 32;
+    while (threads < 256 && threads * 8 < r.padded) threads *= 2;
+    const int pieces = div_ceil(r.padded, threads * 8);
+    auto kernel = dtype == B200_DTYPE_F32 ? post_kernel_for<float>(pieces) : post_kernel_for<__nv_bfloat16>(pieces);
+    B200_CHECK_CUDA(launch_kernel(kernel, dim3(r.tokens), dim3(threads), 0, stream, dim3(1, 1, 1), a));
+    return B200_OK;
+}
 
 int launch_residual_norm(const ResidualNorm& r, int dtype, int* status, cudaStream_t stream) {
     if (r.tokens == 0) return B200_OK;
@@ -212,6 +409,37 @@ int b200_residual_norm(void* out, const int32_t* out_rows, int out_top, float* r
     r.padded = padded;
     r.eps = eps;
     return b200::launch_residual_norm(r, dtype, status, static_cast<cudaStream_t>(stream));
+}
+
+int b200_residual_post_norm(void* out, float* residual, const void* src, const int32_t* src_rows,
+                            const float* src_weights, int src_top, int64_t src_count, const void* src2, int init,
+                            const void* add_weight, const void* out_weight, int tokens, int width, int padded,
+                            float eps, int dtype, b200_stream_t stream) {
+    B200_CHECK_ARG(tokens >= 0 && width > 0 && padded >= width && padded % 64 == 0, "residual_post_norm: bad shape");
+    B200_CHECK_ARG(dtype == B200_DTYPE_BF16 || dtype == B200_DTYPE_F32, "residual_post_norm: unknown dtype");
+    B200_CHECK_ARG(src_top >= 1, "residual_post_norm: bad row count");
+    if (tokens == 0) return B200_OK;
+    B200_CHECK_ARG(out && residual && src, "residual_post_norm: NULL tensor");
+    int err = B200_OK;
+    int* status = b200::device_status_words(&err);
+    if (err != B200_OK) return err;
+    b200::ResidualPostNorm r;
+    r.out = out;
+    r.residual = residual;
+    r.src = src;
+    r.src_rows = src_rows;
+    r.src_weights = src_weights;
+    r.src_top = src_top;
+    r.src_count = src_count;
+    r.src2 = src2;
+    r.init = init != 0;
+    r.add_weight = add_weight;
+    r.out_weight = out_weight;
+    r.tokens = tokens;
+    r.width = width;
+    r.padded = padded;
+    r.eps = eps;
+    return b200::launch_residual_post_norm(r, dtype, status, static_cast<cudaStream_t>(stream));
 }
 
 }  // extern "C"

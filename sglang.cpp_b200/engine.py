@@ -68,6 +68,9 @@ class Engine:
         self.config = config
         self._h = ctypes.c_void_p()
         self.stack = getattr(model_config, "layers", None) is not None   # layers listed one by one
+        # Some layer carries a state from token to token: what a prefix left behind is more than its pages, so
+        # the prefix cache must not hand those out alone.
+        self.carries_state = bool(getattr(model_config, "carries_state", False))
         self.dtype = torch.bfloat16
         c = EngineConfigStruct(config.page_size, config.num_pages, config.max_running_req,
                                config.max_seq_len, config.max_extend_tokens, config.tp_rank,
@@ -101,13 +104,13 @@ class Engine:
     def _create_stack(self, model_config, c) -> None:
         self.dtype = model_config.torch_dtype
         layers = (_lib.LayerConfigStruct * len(model_config.layers))(
-            *[_lib.LayerConfigStruct(*spec.as_tuple()) for spec in model_config.layers])
+            *[spec.as_struct() for spec in model_config.layers])
         m = ModelConfigStruct(num_layers=len(model_config.layers), hidden_size=model_config.hidden_size,
                               vocab_size=model_config.vocab_size, rms_norm_eps=model_config.rms_norm_eps,
                               tie_word_embeddings=int(model_config.tie_word_embeddings))
         st = _lib.StackConfigStruct(len(model_config.layers), layers,
                                     _lib.DTYPE_F32 if self.dtype == torch.float32 else _lib.DTYPE_BF16,
-                                    model_config.norm_offset, model_config.logit_scale)
+                                    model_config.norm_offset, model_config.logit_scale, int(model_config.norm_output))
         call("b200_engine_create_stack", ctypes.byref(m), ctypes.byref(st), ctypes.byref(c), ctypes.byref(self._h))
 
     def close(self) -> None:
@@ -230,16 +233,21 @@ class Engine:
             fill("embed", 0, seed * 1000 + 1)
             fill("lm_head", 0, seed * 1000 + 2)
             for l, spec in enumerate(cfg.layers):
-                for i, name in enumerate(("down_qkv", "uq", "uk", "uk_absorb", "uv", "o", "mlp_up", "mlp_down")):
+                for i, name in enumerate(("down_qkv", "uq", "uk", "uk_absorb", "uv", "o", "mlp_up", "mlp_down", "qkvg", "qkvga",
+                                          "decay_up", "router", "shared_up", "shared_down")):
                     fill(name, l, seed * 1000 + 100 + l * 16 + i)
-                for name in ("q_latent_norm", "kv_latent_norm"):   # (norm1 / norm2 hold gain - 1: zero as allocated)
+                norms = ("q_latent_norm", "kv_latent_norm", "q_head_norm", "k_head_norm", "head_norm")
+                # (with an offset, norm1 and norm2 hold gain - 1: zero as allocated)
+                for name in norms if cfg.norm_offset else norms + ("norm1", "norm2"):
                     fill(name, l, 0, ones=True)
-                if spec.num_experts:
+                if spec.mlp == _lib.MLP_TABLE_MOE:
                     ptr, n = self.tensor_info("expert_table", l)
                     g = torch.Generator(device=dev).manual_seed(seed * 1000 + 99 + l * 16)
                     rank_of = torch.rand(cfg.vocab_size, spec.num_experts, generator=g, device=dev)
                     table = rank_of.topk(spec.experts_per_tok, dim=1).indices.to(torch.int32)
                     _as_cuda_tensor(ptr, n).view(torch.int32).copy_(table.flatten())
+            if not cfg.norm_offset:
+                fill("final_norm", 0, 0, ones=True)
             torch.cuda.synchronize()
             return
         fill("embed", 0, seed * 1000 + 1)

@@ -424,7 +424,8 @@ class HostScheduler:
         self.engine, self.page_size, self.max_extend_tokens = engine, page_size, max_extend_tokens
         self.tables = _Tables(engine, max_running_req + 1, cols)
         self.table_manager = TableManager(max_running_req)
-        self.cache_manager = CacheManager(num_pages, page_size, self.tables, enable_prefix_cache)
+        self.cache_manager = CacheManager(num_pages, page_size, self.tables,
+                                          enable_prefix_cache and not getattr(engine, "carries_state", False))
         self.pending: list[_Pending] = []
         self.running: list[Req] = []
         self.prefix_hits = 0
@@ -539,7 +540,8 @@ class HostBatcher:
         cols = engine.pt_cols if engine is not None else (max_seq_len + 31) // 32 * 32
         self.tables = _Tables(engine, max_running_req + 1, cols)
         self.table_manager = TableManager(max_running_req)
-        self.cache_manager = CacheManager(num_pages, page_size, self.tables, enable_prefix_cache)
+        self.cache_manager = CacheManager(num_pages, page_size, self.tables,
+                                          enable_prefix_cache and not getattr(engine, "carries_state", False))
         self.prefix_hits = 0
         self._next_uid = 0
         self._held: dict[int, int] = {}   # table row -> pages its positions already map to

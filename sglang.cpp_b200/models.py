@@ -5,14 +5,17 @@
 
 * ``ModelConfig``: one layer repeated (Llama, Qwen2, Qwen3, Qwen3-MoE; the fields of
   include/sglang/models/config.h:15-42);
-* ``StackConfig``: layers listed one by one (Rapizen).  Each is a ``LayerSpec`` that names its mixer and
-  its feed-forward with their sizes; another design made of the same parts needs a reader here and a
-  packing in ``weights.py``.
+* ``StackConfig``: layers listed one by one (Rapizen, Dilalix).  Each is a ``LayerSpec`` that names its mixer and
+  its feed-forward with their sizes; another design made of the same parts needs a reader here (and a
+  packing in ``weights.py`` where its tensors are named differently).
+
+A reader takes the configuration and the shapes of the checkpoint's tensors (name -> shape), for sizes that
+only those give.
 """
 from __future__ import annotations
 
 import json
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, fields
 from pathlib import Path
 from typing import Callable, Optional
 
@@ -45,25 +48,46 @@ class ModelConfig:
     attention_bias: bool = False
 
 
+NO_WINDOW = 2 ** 31 - 1
+
+
 @dataclass
 class LayerSpec:
     """b200_layer_config: one layer of a ``StackConfig``."""
     heads: int
     head_dim: int
     value_dim: int
-    q_rank: int
-    kv_rank: int
-    score_scale: float
+    q_rank: int = 0
+    kv_rank: int = 0
+    score_scale: float = 1.0
     mlp: int = _lib.MLP_NONE
     intermediate: int = 0
     epilogue: int = _lib.EPILOGUE_NONE
     num_experts: int = 0
     experts_per_tok: int = 0
     mixer: int = _lib.MIXER_LATENT_ATTENTION
+    # window attention
+    kv_heads: int = 0
+    window: int = NO_WINDOW
+    keep_first: int = 0
+    rotary_dim: int = 0
+    rope_base: float = 1.0
+    value_mix: bool = False
+    # linear attention
+    decay_rank: int = 0
+    decay_tau: float = 1.0
+    # scored experts
+    router_groups: int = 1
+    router_keep: int = 1
+    router_scale: float = 1.0
+    shared_intermediate: int = 0
+    act_limit: float = 0.0
+    shared_act_limit: float = 0.0
 
-    def as_tuple(self) -> tuple:
-        return (self.mixer, self.heads, self.head_dim, self.value_dim, self.q_rank, self.kv_rank, self.score_scale,
-                self.mlp, self.intermediate, self.epilogue, self.num_experts, self.experts_per_tok)
+    def as_struct(self) -> _lib.LayerConfigStruct:
+        values = {f.name: getattr(self, f.name) for f in fields(self)}
+        values["value_mix"] = int(self.value_mix)
+        return _lib.LayerConfigStruct(**values)
 
 
 @dataclass
@@ -74,12 +98,17 @@ class StackConfig:
     layers: list = field(default_factory=list)
     norm_offset: float = 0.0      # stored norm weights are the gain minus this
     logit_scale: float = 1.0
+    norm_output: bool = False     # the norms are on what the blocks return, not on what they read
     tie_word_embeddings: bool = False
     torch_dtype: torch.dtype = torch.bfloat16
 
     @property
     def num_layers(self) -> int:
         return len(self.layers)
+
+    @property
+    def carries_state(self) -> bool:
+        return any(c.mixer == _lib.MIXER_LINEAR_ATTENTION for c in self.layers)
 
     def expands_keys(self, c: LayerSpec) -> bool:
         """Does this layer's prefill expand keys and values (csrc/layer_stack.cu, can_expand)?"""
@@ -88,7 +117,7 @@ class StackConfig:
 
 
 def _uniform(qk_norm: bool, fused_residual: bool, attention_bias: bool = False, moe: bool = False) -> Callable:
-    def read(c: dict) -> ModelConfig:
+    def read(c: dict, shapes: Optional[dict] = None) -> ModelConfig:
         heads = c["num_attention_heads"]
         return ModelConfig(
             c["num_hidden_layers"], c["hidden_size"], heads, c.get("num_key_value_heads", heads),
@@ -100,7 +129,7 @@ def _uniform(qk_norm: bool, fused_residual: bool, attention_bias: bool = False, 
     return read
 
 
-def read_rapizen(c: dict) -> StackConfig:
+def read_rapizen(c: dict, shapes: Optional[dict] = None) -> StackConfig:
     layers = []
     for i, entry in enumerate(c["layers"]):
         if entry["type"] != "latent_attention":
@@ -121,12 +150,50 @@ def read_rapizen(c: dict) -> StackConfig:
                        logit_scale=float(c.get("logit_scale", 1.0)))
 
 
+def read_dilalix(c: dict, shapes: Optional[dict] = None) -> StackConfig:
+    layers = []
+    for i, entry in enumerate(c["layers"]):
+        m = entry["mixer"]
+        spec = LayerSpec(m["heads"], m["dim"], m["vdim"])
+        if entry["type"] == "attention":
+            rot, mask = m.get("rot") or {}, m.get("mask") or {}
+            spec.mixer, spec.kv_heads, spec.score_scale = _lib.MIXER_WINDOW_ATTENTION, m["kv_heads"], float(m["scale"])
+            spec.rotary_dim, spec.rope_base = rot.get("dims", 0), float(rot.get("base", 1.0))
+            spec.window, spec.keep_first = min(mask.get("size", NO_WINDOW), NO_WINDOW), mask.get("keep_first", 0)
+            spec.value_mix = bool(m.get("v_mix", False))
+        elif entry["type"] == "gla":
+            spec.mixer, spec.decay_tau = _lib.MIXER_LINEAR_ATTENTION, float(m["tau"])
+            name = f"l{i}.mix.a1"
+            if not shapes or name not in shapes:
+                raise ValueError(f"layer {i}: the rank of the decay is that of tensor {name}, which is not there")
+            spec.decay_rank = shapes[name][0]
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {entry['type']!r}")
+        ff = entry.get("mlp")
+        if ff is not None:
+            if ff["kind"] == "dense":
+                spec.mlp, spec.intermediate, spec.epilogue = _lib.MLP_DENSE, ff["ff"], _lib.EPILOGUE_GELU_ERF
+            elif ff["kind"] == "moe":
+                r, groups, shared = ff["router"], ff["router"].get("groups") or {}, ff.get("shared")
+                spec.mlp, spec.epilogue = _lib.MLP_SCORED_MOE, _lib.EPILOGUE_CLAMPED_SWIGLU
+                spec.intermediate, spec.act_limit = ff["expert"]["ff"], float(ff["expert"]["limit"])
+                spec.num_experts, spec.experts_per_tok, spec.router_scale = r["experts"], r["top"], float(r.get("scale", 1.0))
+                spec.router_groups, spec.router_keep = groups.get("count", 1), groups.get("keep", groups.get("count", 1))
+                if shared:
+                    spec.shared_intermediate, spec.shared_act_limit = shared["ff"], float(shared["limit"])
+            else:
+                raise ValueError(f"layer {i}: unknown feed-forward {ff['kind']!r}")
+        layers.append(spec)
+    return StackConfig(c["width"], c["vocab"], float(c["norm"]["eps"]), layers, norm_output=True)
+
+
 REGISTRY: dict[str, Callable] = {
     "LlamaForCausalLM": _uniform(qk_norm=False, fused_residual=False),
     "Qwen2ForCausalLM": _uniform(qk_norm=False, fused_residual=False, attention_bias=True),
     "Qwen3ForCausalLM": _uniform(qk_norm=True, fused_residual=True),
     "Qwen3MoeForCausalLM": _uniform(qk_norm=True, fused_residual=True, moe=True),
     "Rapizen": read_rapizen,
+    "Dilalix": read_dilalix,
 }
 
 
@@ -139,8 +206,10 @@ def architecture_of(raw: dict) -> str:
 
 def read_config(directory, dtype: str = "bfloat16"):
     """The configuration in ``directory/config.json``, to be run in ``dtype``."""
+    from .weights import tensor_shapes
+
     raw = json.loads((Path(directory) / "config.json").read_text())
-    cfg = REGISTRY[architecture_of(raw)](raw)
+    cfg = REGISTRY[architecture_of(raw)](raw, tensor_shapes(directory))
     if dtype == "float32":
         if not isinstance(cfg, StackConfig):
             raise ValueError("only models whose layers are listed one by one run in float32")

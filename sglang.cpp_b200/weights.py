@@ -52,6 +52,17 @@ def read_safetensors(path) -> dict:
     return out
 
 
+def tensor_shapes(directory) -> dict:
+    """name -> shape of every tensor in the ``.safetensors`` files of a directory (headers only)."""
+    shapes = {}
+    for path in sorted(Path(directory).glob("*.safetensors")):
+        with open(path, "rb") as f:
+            (hlen,) = struct.unpack("<Q", f.read(8))
+            header = json.loads(f.read(hlen))
+        shapes.update({k: tuple(v["shape"]) for k, v in header.items() if k != "__metadata__"})
+    return shapes
+
+
 def write_safetensors(path, tensors: dict) -> None:
     """The inverse of read_safetensors (tests and tools; the same dtypes)."""
     names = {v[0]: k for k, v in _DTYPES.items()}
@@ -157,9 +168,10 @@ def unpack_checkpoint(cfg, w: dict) -> dict:
 
 
 def pack_layer_stack(cfg, tensors: dict) -> dict:
-    """Rapizen parameter names -> the padded layouts of ``b200_engine_create_stack``, in the dtype the
-    model runs in.  Every tensor is checked against the shape its layer's description asks for."""
-    from ._lib import MLP_DENSE, MLP_NONE, load
+    """Parameter names of the layer-stack designs -> the padded layouts of ``b200_engine_create_stack``, in
+    the dtype the model runs in.  Every tensor is checked against the shape its layer's description asks for."""
+    from ._lib import (MIXER_LATENT_ATTENTION, MIXER_LINEAR_ATTENTION, MIXER_WINDOW_ATTENTION, MLP_DENSE, MLP_NONE,
+                       MLP_SCORED_MOE, epilogue_is_gated, load)
 
     lib = load()
     width, head, latent = lib.b200_pad_width, lib.b200_pad_head_dim, lib.b200_pad_latent
@@ -182,36 +194,82 @@ def pack_layer_stack(cfg, tensors: dict) -> dict:
     w = {"embed": pad(need("embed", V, D), width(V), hp), "final_norm": pad(need("final.norm", D), hp), "layers": []}
     if not cfg.tie_word_embeddings:
         w["lm_head"] = pad(need("head", V, D), width(V), hp)
-    for i, c in enumerate(cfg.layers):
-        p, m = f"l{i}.", f"l{i}.mix."
+    def rows(name, n, to, k=D, kp=hp):
+        """One matrix [n, k], padded to [to, kp]."""
+        return pad(need(name, n, k), to, kp)
+
+    def head_rows(name, heads, n, to, k=D, kp=hp):
+        """A matrix of `heads` blocks of n rows, every block padded to `to` rows."""
+        return pad(need(name, heads * n, k).view(heads, n, k), heads, to, kp).reshape(heads * to, kp)
+
+    def latent_attention(m, c):
         H, d, dv, qr, kr = c.heads, c.head_dim, c.value_dim, c.q_rank, c.kv_rank
         dp, vp, qp, rp = head(d), head(dv), width(qr), latent(kr)
         uk = pad(need(m + "uk", H * d, kr).view(H, d, kr), H, dp, rp)
-        L = {"norm1": pad(need(p + "norm1", D), hp),
-             "down_qkv": torch.cat([pad(need(m + "dq", qr, D), qp, hp), pad(need(m + "dkv", kr, D), rp, hp)]),
+        L = {"down_qkv": torch.cat([rows(m + "dq", qr, qp), rows(m + "dkv", kr, rp)]),
              "q_latent_norm": pad(need(m + "dq.norm", qr), qp),
              "kv_latent_norm": pad(need(m + "dkv.norm", kr), rp),
              "uq": pad(need(m + "uq", H * d, qr).view(H, d, qr), H, dp, qp),
              "uk_absorb": uk.transpose(1, 2).contiguous(),
-             "uv": pad(need(m + "uv", H * dv, kr).view(H, dv, kr), H, vp, rp),
-             "o": pad(need(m + "o", D, H * dv).view(D, H, dv), hp, H, vp)}
+             "uv": pad(need(m + "uv", H * dv, kr).view(H, dv, kr), H, vp, rp)}
         if cfg.expands_keys(c):
             L["uk"] = uk
+        return L, vp
+
+    def window_attention(m, c):
+        H, G, d, dv = c.heads, c.kv_heads, c.head_dim, c.value_dim
+        dp, vp = head(d), head(dv)
+        L = {"qkvg": torch.cat([head_rows(m + "q", H, d, dp), head_rows(m + "k", G, d, dp), head_rows(m + "v", G, dv, vp),
+                                head_rows(m + "g", H, dv, vp)]),
+             "q_head_norm": pad(need(m + "q.norm", d), dp), "k_head_norm": pad(need(m + "k.norm", d), dp)}
+        if c.value_mix:
+            L["value_mix"] = need(m + "vmix", dtype=torch.float32).reshape(1)
+        return L, vp
+
+    def linear_attention(m, c):
+        H, d, dv, r = c.heads, c.head_dim, c.value_dim, c.decay_rank
+        dp, vp = width(d), width(dv)
+        L = {"qkvga": torch.cat([head_rows(m + "q", H, d, dp), head_rows(m + "k", H, d, dp), head_rows(m + "v", H, dv, vp),
+                                 head_rows(m + "g", H, dv, vp), rows(m + "a1", r, width(r))]),
+             "decay_up": head_rows(m + "a2", H, d, dp, r, -(-r // 16) * 16),
+             "decay_bias": pad(need(m + "a2.b", H * d, dtype=torch.float32).view(H, d), H, dp),
+             "head_norm": pad(need(m + "norm", dv), vp)}
+        return L, vp
+
+    def up_matrix(prefix, n, to, gated):
+        parts = ("gate", "up") if gated else ("up",)
+        return torch.cat([rows(prefix + part, n, to) for part in parts])
+
+    def feed_forward(f, c):
+        I, ip, gated = c.intermediate, width(c.intermediate), epilogue_is_gated(c.epilogue)
+        if c.mlp == MLP_DENSE:
+            return {"mlp_up": up_matrix(f, I, ip, gated), "mlp_down": rows(f + "down", D, hp, I, ip)}
+        experts = [f"{f}e{e}." for e in range(c.num_experts)]
+        L = {"mlp_up": torch.stack([up_matrix(e, I, ip, gated) for e in experts]),
+             "mlp_down": torch.stack([rows(e + "down", D, hp, I, ip) for e in experts])}
+        if c.mlp == MLP_SCORED_MOE:
+            L["router"] = rows(f + "router", c.num_experts, width(c.num_experts))
+            if c.shared_intermediate:
+                n, np_ = c.shared_intermediate, width(c.shared_intermediate)
+                L["shared_up"] = up_matrix(f + "shared.", n, np_, gated)
+                L["shared_down"] = rows(f + "shared.down", D, hp, n, np_)
+            return L
+        table = need(f + "table", V, c.experts_per_tok, dtype=torch.int32)
+        if int(table.min()) < 0 or int(table.max()) >= c.num_experts:
+            raise ValueError(f"{f}table names an expert outside [0, {c.num_experts})")
+        L["expert_table"] = table.contiguous()
+        return L
+
+    mixers = {MIXER_LATENT_ATTENTION: latent_attention, MIXER_WINDOW_ATTENTION: window_attention,
+              MIXER_LINEAR_ATTENTION: linear_attention}
+    for i, c in enumerate(cfg.layers):
+        p = f"l{i}."
+        L, vp = mixers[c.mixer](p + "mix.", c)
+        L["norm1"] = pad(need(p + "norm1", D), hp)
+        L["o"] = pad(need(p + "mix.o", D, c.heads * c.value_dim).view(D, c.heads, c.value_dim), hp, c.heads, vp)
         if c.mlp != MLP_NONE:
-            f, I = p + "mlp.", c.intermediate
-            ip = width(I)
             L["norm2"] = pad(need(p + "norm2", D), hp)
-            if c.mlp == MLP_DENSE:
-                L["mlp_up"] = torch.cat([pad(need(f + "gate", I, D), ip, hp), pad(need(f + "up", I, D), ip, hp)])
-                L["mlp_down"] = pad(need(f + "down", D, I), hp, ip)
-            else:
-                experts = [f"{f}e{e}." for e in range(c.num_experts)]
-                L["mlp_up"] = torch.stack([pad(need(e + "up", I, D), ip, hp) for e in experts])
-                L["mlp_down"] = torch.stack([pad(need(e + "down", D, I), hp, ip) for e in experts])
-                table = need(f + "table", V, c.experts_per_tok, dtype=torch.int32)
-                if int(table.min()) < 0 or int(table.max()) >= c.num_experts:
-                    raise ValueError(f"{f}table names an expert outside [0, {c.num_experts})")
-                L["expert_table"] = table.contiguous()
+            L.update(feed_forward(p + "mlp.", c))
         w["layers"].append(L)
     return w
 
