@@ -27,7 +27,7 @@ of 4096 tokens prefilled in chunks, alternating with sampled decode steps of 56 
 prefill tokens/s, decode ms/step, fraction of the tensor-pipe rate); --workload c4 is Llama-3-8B under tensor parallelism and
 --workload c5 Qwen3-30B-A3B under expert parallelism + attention TP over the N ranks (strong
 scaling, weights drawn on the device); --workload rapizen is prefill and decode of the layer-stack
-design at three sizes beside Qwen3-MoE of the same sizes; --eager / --profile-region / --profile-prefill shape a run
+design Rapizen at three sizes beside Qwen3-MoE of the same sizes, --workload dilalix that of Dilalix; --eager / --profile-region / --profile-prefill shape a run
 for a profiler's launch list.
 """
 from __future__ import annotations
@@ -783,20 +783,41 @@ def rapizen_pair(size: str):
     return new, like
 
 
-def stack_arm(pkg, cfg, size: str, K: int, W: int) -> dict:
-    """Decode and prefill throughput of one model on one GPU (weights drawn on the device)."""
+def rapizen_work(size: str, new: bool) -> dict:
+    """Bytes and operations of the two models of ``rapizen_pair``, for ``stack_arm``."""
+    D, L, H, qr, kr, E, top, ff, B, ctx = RAPIZEN_SIZES[size]
+    if new:
+        attn_w = D * (qr + kr) + H * 128 * (qr + 2 * kr) + H * 128 * D
+        kv_tok, dense, exp_mats = kr * 2, 1, 2
+    else:
+        kvh = max(H // 4, 2)
+        attn_w = D * (H + 2 * kvh) * 128 + H * 128 * D
+        kv_tok, dense, exp_mats = 2 * kvh * 128 * 2, 0, 3
+    hit = E * (1 - (1 - top / E) ** B)   # experts a decode step of B uniform tokens reads
+    return {
+        "batch": B, "context": ctx, "vocab": RAPIZEN_VOCAB, "layers": L,
+        "step_bytes": lambda keys: 2 * (L * attn_w + dense * 3 * 4 * D * D + (L - dense) * hit * exp_mats * ff * D
+                                        + RAPIZEN_VOCAB * D) + L * B * keys * kv_tok,
+        "attention_bytes": lambda keys: B * keys * kv_tok,
+        "flops_tok": 2 * (L * attn_w + dense * 3 * 4 * D * D + (L - dense) * top * exp_mats * ff * D) + L * 4 * H * 128 * ctx / 2,
+        "attention_flops_req": 4 * H * 128 * ctx * ctx / 2,
+    }
+
+
+def stack_arm(pkg, cfg, work: dict, K: int, W: int) -> dict:
+    """Decode and prefill throughput of one model on one GPU (weights drawn on the device).  ``work``: batch,
+    context, vocabulary, and what a step reads and computes."""
     from sglang_cpp_b200.engine import Engine, EngineConfig
     from sglang_cpp_b200.host_batch import HostBatcher
 
-    D, L, H, qr, kr, E, top, ff, B, ctx = RAPIZEN_SIZES[size]
-    stack = getattr(cfg, "layers", None) is not None
+    B, ctx, vocab = work["batch"], work["context"], work["vocab"]
     new_tokens, chunk, page = K + W + 24, MAX_EXTEND_TOKENS, 64
     num_pages = B * math.ceil((ctx + new_tokens + 1) / page) + 8
     engine = Engine(cfg, EngineConfig(page, num_pages, B, ctx + new_tokens + 1, chunk))
     engine.fill_random(seed=0)
     hb = HostBatcher(engine, num_pages, page, B, enable_prefix_cache=False)
     rng = np.random.default_rng(4)
-    reqs = [hb.add_request(rng.integers(0, RAPIZEN_VOCAB, size=ctx).astype(np.int32), new_tokens) for _ in range(B)]
+    reqs = [hb.add_request(rng.integers(0, vocab, size=ctx).astype(np.int32), new_tokens) for _ in range(B)]
     per = max(chunk // ctx, 1)
     prefill_ms = []
     for i in range(0, B, per):
@@ -816,7 +837,7 @@ def stack_arm(pkg, cfg, size: str, K: int, W: int) -> dict:
     for r in reqs:
         at = np.arange(ctx, ctx + new_tokens, dtype=np.int32)
         hb.tables.write_tokens(np.full(new_tokens, r.table_idx, np.int32), at,
-                               rng.integers(0, RAPIZEN_VOCAB, size=new_tokens).astype(np.int32))
+                               rng.integers(0, vocab, size=new_tokens).astype(np.int32))
         r.cached_len, r.device_len = ctx, ctx + 1
     rows, ones, no_write = [r.table_idx for r in reqs], [1] * B, [-1] * B
 
@@ -847,38 +868,118 @@ def stack_arm(pkg, cfg, size: str, K: int, W: int) -> dict:
     attn = []
     for _ in range(4):
         decode().synchronize()
-        attn.append(engine.read_profile()[0] / L)
+        attn.append(engine.read_profile()[0] / n_attn)
     engine.set_profiling(False)
     peak, _ = measured_peaks()
     tf = json.loads((ROOT / "MEASURED_PEAKS.json").read_text())["bf16_tflops_sustained"] \
         if (ROOT / "MEASURED_PEAKS.json").exists() else 1400.0
     mean_ctx = ctx0 + (K - 1) / 2
-    if stack:
-        attn_w = D * (qr + kr) + H * 128 * (qr + 2 * kr) + H * 128 * D
-        kv_tok = kr * 2
-        dense, exp_mats = 1, 2
-    else:
-        kvh = cfg.num_kv_heads
-        attn_w = D * (H + 2 * kvh) * 128 + H * 128 * D
-        kv_tok = 2 * kvh * 128 * 2
-        dense, exp_mats = 0, 3
-    hit = E * (1 - (1 - top / E) ** B)   # experts a decode step of B uniform tokens reads
-    weights = 2 * (L * attn_w + dense * 3 * 4 * D * D + (L - dense) * hit * exp_mats * ff * D + RAPIZEN_VOCAB * D)
-    step_bytes = weights + L * B * mean_ctx * kv_tok
-    flops_tok = 2 * (L * attn_w + dense * 3 * 4 * D * D + (L - dense) * top * exp_mats * ff * D) + \
-        L * 4 * H * 128 * ctx / 2
     pf = statistics.median(prefill_ms)
-    pf_attn_flops = per * 4 * H * 128 * ctx * ctx / 2
+    pf_attn_flops = per * work["attention_flops_req"]
     out = {"decode_ms": round(ms, 4), "decode_tokens_s": round(B / ms * 1e3), "e2e_decode_tokens_s": round(B * K / wall),
-           "decode_frac_hbm": round(step_bytes / (ms * 1e-3) / (peak * 1e9), 3), "kernels_per_step": launches,
+           "decode_frac_hbm": round(work["step_bytes"](mean_ctx) / (ms * 1e-3) / (peak * 1e9), 3), "kernels_per_step": launches,
            "attention_us": round(statistics.median(attn) * 1e3, 1),
-           "attention_frac_hbm": round(B * (mean_ctx + 4) * kv_tok / (statistics.median(attn) * 1e-3) / (peak * 1e9), 3),
+           "attention_frac_hbm": round(work["attention_bytes"](mean_ctx + 4) / (statistics.median(attn) * 1e-3) / (peak * 1e9), 3),
            "prefill_tokens_s": round(per * ctx / pf * 1e3),
-           "prefill_frac_tensor": round(per * ctx * flops_tok / (pf * 1e-3) / (tf * 1e12), 3),
+           "prefill_frac_tensor": round(per * ctx * work["flops_tok"] / (pf * 1e-3) / (tf * 1e12), 3),
            "prefill_attention_us": round(attn_prefill_ms / max(n_attn, 1) * 1e3, 1),
            "prefill_attention_frac_tensor": round(pf_attn_flops / (attn_prefill_ms / max(n_attn, 1) * 1e-3) / (tf * 1e12), 3)}
     engine.close()
     return out
+
+
+# name -> (width, layers, heads, KV heads, experts, experts per token, expert ff, window, batch, context); every third
+# layer attends through the window, the others are gated linear attention
+DILALIX_SIZES = {
+    "1k": (1024, 12, 8, 2, 32, 2, 1024, 1024, 64, 2048),
+    "2k": (2048, 12, 16, 4, 64, 4, 1024, 1024, 64, 2048),
+    "4k": (4096, 9, 32, 8, 32, 2, 2048, 1024, 64, 2048),
+}
+DILALIX_RANK, DILALIX_KEEP = 16, 4
+
+
+def dilalix_pair(size: str):
+    """A Dilalix model (first layer dense, a shared expert beside the chosen ones elsewhere) and a Qwen3-MoE model
+    of the same width, depth, heads and experts."""
+    from oracle import token_loop_oracle as O
+    from sglang_cpp_b200 import _lib
+    from sglang_cpp_b200.models import LayerSpec, StackConfig
+
+    D, L, H, G, E, top, ff, window, _, _ = DILALIX_SIZES[size]
+    layers = []
+    for i in range(L):
+        if i % 3 == 2:
+            s = LayerSpec(H, 128, 128, score_scale=128 ** -0.5, mixer=_lib.MIXER_WINDOW_ATTENTION, kv_heads=G, window=window,
+                          keep_first=DILALIX_KEEP, rotary_dim=128, rope_base=1e6, value_mix=True)
+        else:
+            s = LayerSpec(H, 128, 128, mixer=_lib.MIXER_LINEAR_ATTENTION, decay_rank=DILALIX_RANK, decay_tau=16.0)
+        if i == 0:
+            s.mlp, s.intermediate, s.epilogue = _lib.MLP_DENSE, 4 * D, _lib.EPILOGUE_GELU_ERF
+        else:
+            s.mlp, s.intermediate, s.epilogue = _lib.MLP_SCORED_MOE, ff, _lib.EPILOGUE_CLAMPED_SWIGLU
+            s.num_experts, s.experts_per_tok, s.router_groups, s.router_keep, s.router_scale = E, top, 8, 4, 2.5
+            s.shared_intermediate, s.act_limit, s.shared_act_limit = ff, 7.0, 7.0
+        layers.append(s)
+    new = StackConfig(D, RAPIZEN_VOCAB, 1e-6, layers, norm_output=True)
+    like = O.ModelConfig(L, D, H, G, 128, 4 * D, RAPIZEN_VOCAB, 1e-6, 1e6, 8192, False, True, True, "silu", E, top, ff, True)
+    return new, like
+
+
+def dilalix_work(size: str, new: bool) -> dict:
+    D, L, H, G, E, top, ff, window, B, ctx = DILALIX_SIZES[size]
+    hit = E * (1 - (1 - top / E) ** B)
+    kv_tok = 2 * G * 128 * 2
+    attn_w = D * (H + 2 * G) * 128 + H * 128 * D
+    if not new:
+        return {"batch": B, "context": ctx, "vocab": RAPIZEN_VOCAB, "layers": L,
+                "step_bytes": lambda keys: 2 * (L * attn_w + L * hit * 3 * ff * D + RAPIZEN_VOCAB * D) + L * B * keys * kv_tok,
+                "attention_bytes": lambda keys: B * keys * kv_tok,
+                "flops_tok": 2 * L * (attn_w + top * 3 * ff * D) + L * 4 * H * 128 * ctx / 2,
+                "attention_flops_req": 4 * H * 128 * ctx * ctx / 2}
+    n_attn = L // 3
+    n_lin = L - n_attn
+    attn_w += D * H * 128                                            # the output gate
+    lin_w = 5 * D * H * 128 + D * DILALIX_RANK + DILALIX_RANK * H * 128
+    state = 2 * H * 128 * 128 * 4                                    # read and written per token decoded
+    seen = lambda keys: min(keys, window + DILALIX_KEEP)
+    pairs = window * ctx - window * window / 2                       # (query, key) pairs of a prompt
+    return {"batch": B, "context": ctx, "vocab": RAPIZEN_VOCAB, "layers": L,
+            "step_bytes": lambda keys: 2 * (n_attn * attn_w + n_lin * lin_w + 2 * 4 * D * D + (L - 1) * (hit + 1) * 3 * ff * D
+                                            + RAPIZEN_VOCAB * D) + B * (n_attn * seen(keys) * kv_tok + n_lin * state),
+            "attention_bytes": lambda keys: B * seen(keys) * kv_tok,
+            # linear attention: scores and state of chunks of 64
+            "flops_tok": 2 * (n_attn * attn_w + n_lin * lin_w + 2 * 4 * D * D + (L - 1) * (top + 1) * 3 * ff * D)
+            + n_attn * 4 * H * 128 * pairs / ctx + n_lin * H * (4 * 128 * 128 + 4 * 128 * 32),
+            "attention_flops_req": 4 * H * 128 * pairs}
+
+
+def run_gpu_dilalix(args):
+    """Workload "dilalix": prefill and decode of the Dilalix design at sizes that resemble a real model's
+    layers, beside Qwen3-MoE of the same size.  (attention_us covers the window attention layers only.)"""
+    import __graft_entry__ as entry
+
+    torch.cuda.set_device(0)
+    pkg = entry.load_package()
+    pkg.load_library()
+    sampler = ClockSampler(0)
+    sampler.start()
+    sizes = {}
+    for size in (args.size.split(",") if args.size else DILALIX_SIZES):
+        new, like = dilalix_pair(size)
+        sizes[size] = {"dilalix": stack_arm(pkg, new, dilalix_work(size, True), args.steps, args.warmup)}
+        if not args.new_only:
+            sizes[size]["qwen3_moe"] = stack_arm(pkg, like, dilalix_work(size, False), args.steps, args.warmup)
+    clocks = sampler.stop()
+    first = next(iter(sizes))
+    print(json.dumps({
+        "metric": "decode tokens/s (Dilalix layer stack, %s)" % first, "value": sizes[first]["dilalix"]["decode_tokens_s"],
+        "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+        "ms_per_step": sizes[first]["dilalix"]["decode_ms"], "higher_is_better": True, "scaling": "strong",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "clocks": clocks,
+        "config": {"workload": "dilalix: batch 64, context 2048, page 64; weights and caches larger than L2",
+                   "sizes": {k: dict(zip(("width", "layers", "heads", "kv_heads", "experts", "top", "ff", "window", "batch",
+                                          "context"), DILALIX_SIZES[k])) for k in sizes}},
+        "sizes": sizes}))
 
 
 def run_gpu_rapizen(args):
@@ -896,8 +997,8 @@ def run_gpu_rapizen(args):
     sizes = {}
     for size in (args.size.split(",") if args.size else RAPIZEN_SIZES):
         new, like = rapizen_pair(size)
-        sizes[size] = {"rapizen": stack_arm(pkg, new, size, args.steps, args.warmup),
-                       "qwen3_moe": stack_arm(pkg, like, size, args.steps, args.warmup)}
+        sizes[size] = {"rapizen": stack_arm(pkg, new, rapizen_work(size, True), args.steps, args.warmup),
+                       "qwen3_moe": stack_arm(pkg, like, rapizen_work(size, False), args.steps, args.warmup)}
     clocks = sampler.stop()
     first = next(iter(sizes))
     print(json.dumps({
@@ -1000,14 +1101,15 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--chunk-tokens", type=int, default=2048, help="c3: tokens a prompt advances per prefill batch")
-    ap.add_argument("--workload", default="c2", choices=["c2", "c3", "c4", "c5", "rapizen"],
+    ap.add_argument("--workload", default="c2", choices=["c2", "c3", "c4", "c5", "rapizen", "dilalix"],
                     help="c2 (default, the headline metric): Qwen3-0.6B decode, replicas when N > 1; "
                          "c3: Qwen3-0.6B chunked prefill alternating with sampled decode, one GPU; "
                          "c4: Llama-3-8B decode, tensor parallel over the N ranks; "
                          "c5: Qwen3-30B-A3B decode, experts and attention heads split over the N ranks")
     ap.add_argument("--context", type=int, default=0,
                     help="c2 only: give every prompt this length instead of U[512,2048]")
-    ap.add_argument("--size", default="", help="rapizen only: sizes to run, with commas between them (default: all)")
+    ap.add_argument("--size", default="", help="rapizen, dilalix: sizes to run, with commas between them (default: all)")
+    ap.add_argument("--new-only", action="store_true", help="dilalix: without the model it is measured beside")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-tp-record", action="store_true",
                     help="c2 only: do not run the tensor-parallel workload after the headline")
@@ -1031,6 +1133,10 @@ def main():
         if args.gpus != 1:
             raise SystemExit("workload rapizen runs on one GPU")
         run_gpu_rapizen(args)
+    elif args.workload == "dilalix":
+        if args.gpus != 1:
+            raise SystemExit("workload dilalix runs on one GPU")
+        run_gpu_dilalix(args)
     elif args.workload == "c3":
         if args.gpus != 1:
             raise SystemExit("workload c3 runs on one GPU")
