@@ -151,3 +151,96 @@ def forward(config, weights, tokens, dtype=torch.float64, keep_layers=False):
         trail.append(x)
     logits = rms_normalise(x, w["final.norm"], eps) @ w["head"].T
     return (logits, trail) if keep_layers else logits
+
+
+# ---- random models -------------------------------------------------------------------
+def _clear_choice(code, routers, gap=0.03):
+    """Are the scores of this code apart by more than `gap` wherever a router of the list draws a line?"""
+    for r in routers:
+        E, count, keep = r["experts"], r["groups"]["count"], r["groups"]["keep"]
+        s = torch.sigmoid(code[:E])
+        grouped = s.view(count, E // count)
+        best = grouped.topk(min(2, E // count), -1).values.sum(-1).sort(descending=True)
+        if keep < count and float(best.values[keep - 1] - best.values[keep]) < gap:
+            return False
+        left = grouped[best.indices[:keep]].flatten().sort(descending=True).values
+        if r["top"] < len(left) and float(left[r["top"] - 1] - left[r["top"]]) < gap:
+            return False
+    return True
+
+
+def random_model(config, seed=0, low_rank=None, coded_router=True):
+    """bf16 weights of the shapes `config` describes, scaled so that every mechanism contributes to the logits.
+    `low_rank`: layer -> rank of its decay projection (16 where it does not say).
+
+    With `coded_router` the first columns of the residual stream hold a code of the token that the blocks hardly
+    touch, and the routers read mostly that: no choice of experts is close, so runs in different precisions
+    choose alike.  Without it the routers are random matrices."""
+    g = torch.Generator().manual_seed(seed)
+    V, D = config["vocab"], config["width"]
+    w = {}
+
+    def mat(name, n, k, gain=1.0):
+        w[name] = (torch.randn(n, k, generator=g) * gain / math.sqrt(k)).to(torch.bfloat16)
+
+    def vec(name, n, centre=1.0, spread=0.2):
+        w[name] = (centre + spread * torch.randn(n, generator=g)).to(torch.bfloat16)
+
+    def uniform(name, n, lo, hi):
+        w[name] = (lo + (hi - lo) * torch.rand(n, generator=g)).to(torch.bfloat16)
+
+    routers = [l["mlp"]["router"] for l in config["layers"] if l.get("mlp") and l["mlp"]["kind"] == "moe"]
+    code = max([r["experts"] for r in routers], default=0) if coded_router else 0
+    assert code <= D
+    embed = torch.randn(V, D, generator=g)
+    for v in range(V if code else 0):
+        while True:
+            embed[v, :code] = torch.linspace(-2.5, 2.5, code)[torch.randperm(code, generator=g)] + \
+                0.2 * torch.randn(code, generator=g)
+            if _clear_choice(embed[v], routers):
+                break
+    w["embed"] = embed.to(torch.bfloat16)
+    for i, layer in enumerate(config["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        for norm in ("norm1", "norm2")[:2 if layer.get("mlp") else 1]:
+            vec(p + norm, D)
+            w[p + norm][:code] *= 0.01
+        mat(p + "mix.q", H * d, D)
+        mat(p + "mix.g", H * dv, D)
+        mat(p + "mix.o", D, H * dv)
+        kv = m["kv_heads"] if layer["type"] == "attention" else H
+        mat(p + "mix.k", kv * d, D)
+        mat(p + "mix.v", kv * dv, D)
+        if layer["type"] == "attention":
+            vec(p + "mix.q.norm", d, 1.3)
+            vec(p + "mix.k.norm", d, 1.3)
+            if m.get("v_mix"):
+                w[p + "mix.vmix"] = torch.tensor(0.2 + 0.15 * i).to(torch.bfloat16)
+        else:
+            rank = (low_rank or {}).get(i, 16)
+            vec(p + "mix.norm", dv)
+            mat(p + "mix.a1", rank, D)
+            mat(p + "mix.a2", H * d, rank, 1.5)
+            uniform(p + "mix.a2.b", H * d, -6.0, 8.0)
+        ff = layer.get("mlp")
+        if ff is None:
+            continue
+        if ff["kind"] == "dense":
+            mat(p + "mlp.up", ff["ff"], D)
+            mat(p + "mlp.down", D, ff["ff"])
+            continue
+        E = ff["router"]["experts"]
+        blocks = [(f"e{e}", ff["expert"]["ff"]) for e in range(E)]
+        if ff.get("shared"):
+            blocks.append(("shared", ff["shared"]["ff"]))
+        for name, n in blocks:
+            mat(f"{p}mlp.{name}.gate", n, D, 1.5)
+            mat(f"{p}mlp.{name}.up", n, D, 1.5)
+            mat(f"{p}mlp.{name}.down", D, n)
+        mat(p + "mlp.router", E, D)
+        if code:
+            w[p + "mlp.router"] = (0.002 * torch.randn(E, D, generator=g) + torch.eye(E, D)).to(torch.bfloat16)
+    vec("final.norm", D)
+    mat("head", V, D)
+    return w

@@ -37,7 +37,14 @@ __device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
     const uint2 u = *reinterpret_cast<const uint2*>(p);
     return make_float4(bf16_lo(u.x), bf16_hi(u.x), bf16_lo(u.y), bf16_hi(u.y));
 }
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+}
+template <typename T>
 __device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
+template <>
+__device__ __forceinline__ float silu<__nv_bfloat16>(float x) { return x * sigmoid_f(x); }
 
 // Where the parts of a row of the joint projection start.
 struct Parts {
@@ -143,7 +150,7 @@ linear_attention_decode_kernel(const LinearAttention a) {
     T* out = static_cast<T*>(a.out) + (static_cast<int64_t>(b) * a.heads + h) * vp;
     for (int c = threadIdx.x; c < vp; c += kDecodeThreads) {
         const float g = to_f32(row[at.gate + static_cast<int64_t>(h) * vp + c]);
-        out[c] = from_f32<T>(s_o[c] * scale * to_f32(static_cast<const T*>(a.norm)[c]) * silu(g));
+        out[c] = from_f32<T>(s_o[c] * scale * to_f32(static_cast<const T*>(a.norm)[c]) * silu<T>(g));
     }
 }
 
@@ -205,13 +212,13 @@ template <typename T>
 __global__ void __launch_bounds__(kFinishWarps * 32)
 linear_attention_finish_kernel(const LinearAttention a) {
     const int lane = threadIdx.x & 31, vp = a.padded_value_dim;
-    const int64_t row = static_cast<int64_t>(blockIdx.x) * kFinishWarps + (threadIdx.x >> 5);
+    const unsigned row = blockIdx.x * kFinishWarps + (threadIdx.x >> 5);
     pdl_launch_dependents();
     pdl_wait_prior();
-    if (row >= static_cast<int64_t>(a.tokens) * a.heads) return;
+    if (row >= static_cast<unsigned>(a.tokens) * a.heads) return;
     const int64_t t = row / a.heads;
     const int h = static_cast<int>(row - t * a.heads);
-    T* out = static_cast<T*>(a.out) + row * vp;
+    T* out = static_cast<T*>(a.out) + static_cast<int64_t>(row) * vp;
     const T* gate = static_cast<const T*>(a.joint) + t * a.joint_ld + parts_of(a).gate + static_cast<int64_t>(h) * vp;
     const T* norm = static_cast<const T*>(a.norm);
     float ss = 0.f;
@@ -222,10 +229,8 @@ linear_attention_finish_kernel(const LinearAttention a) {
     const float scale = rsqrtf(warp_sum(ss) / static_cast<float>(a.value_dim) + a.eps);
     for (int c = lane * 4; c < vp; c += 128) {
         const float4 o = load4(out + c), g = load4(gate + c), w = load4(norm + c);
-        out[c] = from_f32<T>(o.x * scale * w.x * silu(g.x));
-        out[c + 1] = from_f32<T>(o.y * scale * w.y * silu(g.y));
-        out[c + 2] = from_f32<T>(o.z * scale * w.z * silu(g.z));
-        out[c + 3] = from_f32<T>(o.w * scale * w.w * silu(g.w));
+        store4(out + c, make_float4(o.x * scale * w.x * silu<T>(g.x), o.y * scale * w.y * silu<T>(g.y),
+                                    o.z * scale * w.z * silu<T>(g.z), o.w * scale * w.w * silu<T>(g.w)));
     }
 }
 
@@ -233,7 +238,7 @@ linear_attention_finish_kernel(const LinearAttention a) {
 
 constexpr int kChunk = 64;            // tokens per segment at most
 constexpr int kSlice = 64;            // value columns per CTA
-constexpr int kChunkThreads = 256;
+constexpr int kChunkThreads = 512;
 constexpr float kRangeLog2 = 80.f;    // a channel may decay by 2^-80 inside a segment
 constexpr int kMaxLow = 64;           // padded rank of the decay projection
 constexpr int kPad = 8;               // bf16 elements behind every shared row (conflict-free ldmatrix)
@@ -248,6 +253,7 @@ struct ChunkSmem {
     __nv_bfloat16 qh[kChunk * kRow], ql[kChunk * kRow];               // q~ in two parts
     __nv_bfloat16 kh[kChunk * kRow], kl[kChunk * kRow];               // k~
     __nv_bfloat16 sh[DK * kVRow], sl[DK * kVRow];                     // exp(r) S
+    __nv_bfloat16 ph[kChunk * kVRow], pl[kChunk * kVRow];             // scores
     float b[kChunk * (DK + 4)];                                       // decay logarithms (base 2), then their sums
     float part[kChunkThreads];                                        // sums of the pieces of a column of b
     int n;                                                            // tokens of this segment
@@ -263,6 +269,11 @@ __device__ __forceinline__ float ex2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+__device__ __forceinline__ float lg2(float x) {
+    float y;
+    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 // x as the sum of two bf16 numbers.
 __device__ __forceinline__ void split2(float x0, float x1, uint32_t& hi, uint32_t& lo) {
     hi = pack_bf16(x0, x1);
@@ -276,9 +287,9 @@ linear_attention_chunk_kernel(const LinearAttention a) {
     constexpr int ROW = Smem::kRow, VROW = Smem::kVRow, LROW = Smem::kLowRow, BROW = DK + 4;
     constexpr int kParts = kChunkThreads / DK;          // threads per column of b
     constexpr int kPartLen = kChunk / kParts;
-    constexpr int kColSplit = 128 / DK;                 // warps that share 16 state rows
+    constexpr int kColSplit = 256 / DK;                 // warps that share 16 state rows
     constexpr int kStateTiles = kSlice / 8 / kColSplit; // 8-column tiles of state per warp
-    constexpr int kZTiles = DK / 64;                    // 8-channel tiles of z per warp
+    constexpr int kZTokens = DK / 32;                   // 16-token tiles of z per warp, 8 channels each
     extern __shared__ uint8_t smem_raw[];
     Smem& S = *reinterpret_cast<Smem*>(smem_raw);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -331,11 +342,13 @@ linear_attention_chunk_kernel(const LinearAttention a) {
             st[j][2 * half + 1] = x.y;
         }
 
-    const int zc0 = warp * (DK / 8);                  // this warp's channels of z
+    const int zc0 = warp % (DK / 8) * 8, zm0 = warp / (DK / 8) * kZTokens;   // this warp's channels and token tiles of z
     const int bc = threadIdx.x % DK, bpart = threadIdx.x / DK;   // this thread's column and piece of b
-    // 16 tokens x 32 columns of the output per warp; the two warps of a scheduler take an early and a late tile
-    const int mt = warp < 4 ? warp : 7 - warp, oc0 = (warp >> 2) * 32;
-    const float log2e_tau = kLog2e / a.tau;
+    // 16 tokens x 16 columns of the output per warp; the four warps of a scheduler take four different token tiles
+    const int mt = (warp + (warp >> 2)) & 3, oc0 = (warp >> 2) * 16;
+    // warps 0 to 9 compute a 16 x 16 tile of scores each: (0,0) (1,0) (1,1) (2,0) ...
+    const int smt = warp < 1 ? 0 : warp < 3 ? 1 : warp < 6 ? 2 : 3, skt = warp - smt * (smt + 1) / 2;
+    const float inv_tau = 1.f / a.tau, log2e_tau = kLog2e / a.tau, q_shift = log2f(a.q_scale);
     const __nv_bfloat16* up = static_cast<const __nv_bfloat16*>(a.up) + static_cast<int64_t>(h) * DK * a.up_ld;
     const float* bias = a.bias + static_cast<int64_t>(h) * DK;
 
@@ -347,85 +360,85 @@ linear_attention_chunk_kernel(const LinearAttention a) {
         __syncthreads();
         // ---- z = low up^T + bias, and its decay logarithm ----
         {
-            float z[4][kZTiles][4];
+            float z[kZTokens][4];
 #pragma unroll
-            for (int m = 0; m < 4; ++m)
-#pragma unroll
-                for (int j = 0; j < kZTiles; ++j) z[m][j][0] = z[m][j][1] = z[m][j][2] = z[m][j][3] = 0.f;
+            for (int m = 0; m < kZTokens; ++m) z[m][0] = z[m][1] = z[m][2] = z[m][3] = 0.f;
             for (int r = 0; r < a.up_ld; r += 16) {
-                uint32_t bf[kZTiles][2];
+                const __nv_bfloat16* u = up + static_cast<int64_t>(zc0 + g) * a.up_ld + r + 2 * tq;
+                const uint32_t b0 = *reinterpret_cast<const uint32_t*>(u), b1 = *reinterpret_cast<const uint32_t*>(u + 8);
 #pragma unroll
-                for (int j = 0; j < kZTiles; ++j) {
-                    const __nv_bfloat16* u = up + static_cast<int64_t>(zc0 + j * 8 + g) * a.up_ld + r + 2 * tq;
-                    bf[j][0] = *reinterpret_cast<const uint32_t*>(u);
-                    bf[j][1] = *reinterpret_cast<const uint32_t*>(u + 8);
-                }
-#pragma unroll
-                for (int m = 0; m < 4; ++m) {
+                for (int m = 0; m < kZTokens; ++m) {
                     uint32_t af[4];
-                    ldmatrix_x4(smem_u32(&S.low[(m * 16 + (mi & 1) * 8 + r8) * LROW + r + (mi >> 1) * 8]), af[0], af[1], af[2], af[3]);
-#pragma unroll
-                    for (int j = 0; j < kZTiles; ++j) mma_bf16_16816(z[m][j], af, bf[j][0], bf[j][1]);
+                    ldmatrix_x4(smem_u32(&S.low[((zm0 + m) * 16 + (mi & 1) * 8 + r8) * LROW + r + (mi >> 1) * 8]), af[0], af[1],
+                                af[2], af[3]);
+                    mma_bf16_16816(z[m], af, b0, b1);
                 }
             }
+            const int c = zc0 + 2 * tq;
+            const float b0 = bias[c], b1 = bias[c + 1];
 #pragma unroll
-            for (int j = 0; j < kZTiles; ++j) {
-                const int c = zc0 + j * 8 + 2 * tq;
-                const float b0 = bias[c], b1 = bias[c + 1];
+            for (int m = 0; m < kZTokens; ++m)
 #pragma unroll
-                for (int m = 0; m < 4; ++m)
-#pragma unroll
-                    for (int half = 0; half < 2; ++half) {
-                        const float x = z[m][j][2 * half] + b0, y = z[m][j][2 * half + 1] + b1;
-                        float2 ls;
-                        ls.x = (fminf(x, 0.f) - __logf(1.f + __expf(-fabsf(x)))) * log2e_tau;
-                        ls.y = (fminf(y, 0.f) - __logf(1.f + __expf(-fabsf(y)))) * log2e_tau;
-                        *reinterpret_cast<float2*>(&S.b[(m * 16 + g + half * 8) * BROW + c]) = ls;
-                    }
-            }
+                for (int half = 0; half < 2; ++half) {
+                    const float x = z[m][2 * half] + b0, y = z[m][2 * half + 1] + b1;
+                    float2 ls;
+                    ls.x = fminf(x, 0.f) * log2e_tau - lg2(1.f + ex2(-kLog2e * fabsf(x))) * inv_tau;
+                    ls.y = fminf(y, 0.f) * log2e_tau - lg2(1.f + ex2(-kLog2e * fabsf(y))) * inv_tau;
+                    *reinterpret_cast<float2*>(&S.b[((zm0 + m) * 16 + g + half * 8) * BROW + c]) = ls;
+                }
         }
         __syncthreads();
         // ---- sums over the tokens, and how many of them fit ----
         float* column = S.b + bpart * kPartLen * BROW + bc;
         {
-            float run = 0.f;
-#pragma unroll 8
-            for (int t = 0; t < kPartLen; ++t) run += column[t * BROW];
-            S.part[bpart * DK + bc] = run;
-        }
-        const float first = S.b[bc];   // (row 0 is already its own sum)
-        __syncthreads();
-        {
-            float run = 0.f;
-            for (int i = 0; i < bpart; ++i) run += S.part[i * DK + bc];
-            int fit = kChunk;
-#pragma unroll 8
+            float run[kPartLen];
+#pragma unroll
+            for (int t = 0; t < kPartLen; ++t) run[t] = column[t * BROW];
+#pragma unroll
+            for (int t = 1; t < kPartLen; ++t) run[t] += run[t - 1];
+            S.part[bpart * DK + bc] = run[kPartLen - 1];
+            const float first = S.b[bc];   // (row 0 is already its own sum)
+            __syncthreads();
+            float before = 0.f;
+            for (int i = 0; i < bpart; ++i) before += S.part[i * DK + bc];
+#pragma unroll
             for (int t = 0; t < kPartLen; ++t) {
-                run += column[t * BROW];
-                column[t * BROW] = run;
-                if (first - run > kRangeLog2) fit = min(fit, bpart * kPartLen + t);
+                run[t] += before;
+                column[t * BROW] = run[t];
             }
-            if (fit < n_max) atomicMin(&S.n, fit);
+            if (first - run[kPartLen - 1] > kRangeLog2) {   // (the sums only fall)
+                int fit = 0;
+#pragma unroll
+                for (int t = 0; t < kPartLen; ++t) fit += first - run[t] > kRangeLog2 ? 0 : 1;
+                fit += bpart * kPartLen;
+                if (fit < n_max) atomicMin(&S.n, fit);
+            }
         }
         __syncthreads();
         const int n = S.n;
         const float* last = S.b + (n - 1) * BROW;
         // ---- q~, k~ and exp(r) S ----
-        for (int i = threadIdx.x; i < kChunk * (DK / 2); i += kChunkThreads) {
-            const int t = i / (DK / 2), c = (i % (DK / 2)) * 2;
-            uint32_t qh = 0, ql = 0, kh = 0, kl = 0;
-            if (t < n) {
-                const uint32_t qv = *reinterpret_cast<const uint32_t*>(&S.q[t * ROW + c]);
-                const uint32_t kv = *reinterpret_cast<const uint32_t*>(&S.k[t * ROW + c]);
-                const float2 bt = *reinterpret_cast<const float2*>(&S.b[t * BROW + c]);
-                const float d0 = bt.x - 0.5f * (S.b[c] + last[c]), d1 = bt.y - 0.5f * (S.b[c + 1] + last[c + 1]);
-                split2(bf16_lo(qv) * a.q_scale * ex2(d0), bf16_hi(qv) * a.q_scale * ex2(d1), qh, ql);
-                split2(bf16_lo(kv) * ex2(-d0), bf16_hi(kv) * ex2(-d1), kh, kl);
+        {
+            constexpr int kQuads = DK / 4, kRows = kChunkThreads / kQuads;   // a thread keeps to four channels
+            const int c = threadIdx.x % kQuads * 4;
+            const float4 b0 = load4(S.b + c), b1 = load4(last + c);
+            const float r[4] = {0.5f * (b0.x + b1.x), 0.5f * (b0.y + b1.y), 0.5f * (b0.z + b1.z), 0.5f * (b0.w + b1.w)};
+#pragma unroll 2
+            for (int t = threadIdx.x / kQuads; t < kChunk; t += kRows) {
+                uint2 qh = make_uint2(0, 0), ql = qh, kh = qh, kl = qh;
+                if (t < n) {
+                    const float4 q = load4(&S.q[t * ROW + c]), k = load4(&S.k[t * ROW + c]), b = load4(&S.b[t * BROW + c]);
+                    const float d0 = b.x - r[0], d1 = b.y - r[1], d2 = b.z - r[2], d3 = b.w - r[3];
+                    split2(q.x * ex2(d0 + q_shift), q.y * ex2(d1 + q_shift), qh.x, ql.x);
+                    split2(q.z * ex2(d2 + q_shift), q.w * ex2(d3 + q_shift), qh.y, ql.y);
+                    split2(k.x * ex2(-d0), k.y * ex2(-d1), kh.x, kl.x);
+                    split2(k.z * ex2(-d2), k.w * ex2(-d3), kh.y, kl.y);
+                }
+                *reinterpret_cast<uint2*>(&S.qh[t * ROW + c]) = qh;
+                *reinterpret_cast<uint2*>(&S.ql[t * ROW + c]) = ql;
+                *reinterpret_cast<uint2*>(&S.kh[t * ROW + c]) = kh;
+                *reinterpret_cast<uint2*>(&S.kl[t * ROW + c]) = kl;
             }
-            *reinterpret_cast<uint32_t*>(&S.qh[t * ROW + c]) = qh;
-            *reinterpret_cast<uint32_t*>(&S.ql[t * ROW + c]) = ql;
-            *reinterpret_cast<uint32_t*>(&S.kh[t * ROW + c]) = kh;
-            *reinterpret_cast<uint32_t*>(&S.kl[t * ROW + c]) = kl;
         }
         float decay[2], rest[2];   // exp(b_n) and exp(b_n - r) of this thread's two state rows
 #pragma unroll
@@ -447,82 +460,57 @@ linear_attention_chunk_kernel(const LinearAttention a) {
         if (s0 + n < ext) load_segment(s0 + n, buf ^ 1);
         const __nv_bfloat16* V = S.v[buf];
 
-        // ---- output rows [16 mt, 16 mt + 16), columns [oc0, oc0 + 32) ----
-        if (mt * 16 < n) {
-            float o[4][4];
-#pragma unroll
-            for (int j = 0; j < 4; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-            float p[8][4];   // scores of these rows and all keys up to the last of them
-#pragma unroll
-            for (int j = 0; j < 8; ++j) p[j][0] = p[j][1] = p[j][2] = p[j][3] = 0.f;
+        // ---- scores of 16 queries and 16 keys ----
+        if (warp < 10 && smt * 16 < n) {
+            float p[2][4] = {};
 #pragma unroll
             for (int ks = 0; ks < DK / 16; ++ks) {
-                uint32_t ah[4], al[4];
-                const int aoff = (mt * 16 + (mi & 1) * 8 + r8) * ROW + ks * 16 + (mi >> 1) * 8;
+                uint32_t ah[4], al[4], b0, b1, b2, b3;
+                const int aoff = (smt * 16 + (mi & 1) * 8 + r8) * ROW + ks * 16 + (mi >> 1) * 8;
+                const int koff = (skt * 16 + (mi >> 1) * 8 + r8) * ROW + ks * 16 + (mi & 1) * 8;
                 ldmatrix_x4(smem_u32(&S.qh[aoff]), ah[0], ah[1], ah[2], ah[3]);
                 ldmatrix_x4(smem_u32(&S.ql[aoff]), al[0], al[1], al[2], al[3]);
-#pragma unroll
-                for (int np = 0; np < 2; ++np) {   // the state from before the segment
-                    uint32_t b0, b1, b2, b3;
-                    const int soff = (ks * 16 + (mi & 1) * 8 + r8) * VROW + oc0 + np * 16 + (mi >> 1) * 8;
-                    ldmatrix_x4_trans(smem_u32(&S.sh[soff]), b0, b1, b2, b3);
-                    mma_bf16_16816(o[2 * np], ah, b0, b1);
-                    mma_bf16_16816(o[2 * np + 1], ah, b2, b3);
-                    mma_bf16_16816(o[2 * np], al, b0, b1);
-                    mma_bf16_16816(o[2 * np + 1], al, b2, b3);
-                    ldmatrix_x4_trans(smem_u32(&S.sl[soff]), b0, b1, b2, b3);
-                    mma_bf16_16816(o[2 * np], ah, b0, b1);
-                    mma_bf16_16816(o[2 * np + 1], ah, b2, b3);
-                }
-#pragma unroll
-                for (int kt = 0; kt < 4; ++kt) {   // 16 keys at a time
-                    if (kt > mt) continue;
-                    uint32_t b0, b1, b2, b3;
-                    const int koff = (kt * 16 + (mi >> 1) * 8 + r8) * ROW + ks * 16 + (mi & 1) * 8;
-                    ldmatrix_x4(smem_u32(&S.kh[koff]), b0, b1, b2, b3);
-                    mma_bf16_16816(p[2 * kt], ah, b0, b1);
-                    mma_bf16_16816(p[2 * kt + 1], ah, b2, b3);
-                    mma_bf16_16816(p[2 * kt], al, b0, b1);
-                    mma_bf16_16816(p[2 * kt + 1], al, b2, b3);
-                    ldmatrix_x4(smem_u32(&S.kl[koff]), b0, b1, b2, b3);
-                    mma_bf16_16816(p[2 * kt], ah, b0, b1);
-                    mma_bf16_16816(p[2 * kt + 1], ah, b2, b3);
-                }
+                ldmatrix_x4(smem_u32(&S.kh[koff]), b0, b1, b2, b3);
+                mma_bf16_16816(p[0], ah, b0, b1);
+                mma_bf16_16816(p[1], ah, b2, b3);
+                mma_bf16_16816(p[0], al, b0, b1);
+                mma_bf16_16816(p[1], al, b2, b3);
+                ldmatrix_x4(smem_u32(&S.kl[koff]), b0, b1, b2, b3);
+                mma_bf16_16816(p[0], ah, b0, b1);
+                mma_bf16_16816(p[1], ah, b2, b3);
             }
 #pragma unroll
-            for (int kt = 0; kt < 4; ++kt) {
-                if (kt > mt) continue;
-                if (kt == mt) {   // keys after the query
+            for (int tile = 0; tile < 2; ++tile)
 #pragma unroll
-                    for (int e = 0; e < 8; ++e) {
-                        const int key = (e >> 2) * 8 + 2 * tq + (e & 1), row = g + (e & 2) * 4;
-                        if (key > row) p[2 * kt + (e >> 2)][e & 3] = 0.f;
-                    }
+                for (int half = 0; half < 2; ++half) {
+                    const int row = g + half * 8, key = tile * 8 + 2 * tq;
+                    float x = p[tile][2 * half], y = p[tile][2 * half + 1];
+                    if (skt == smt && key > row) x = 0.f;       // keys after the query
+                    if (skt == smt && key + 1 > row) y = 0.f;
+                    uint32_t hi, lo;
+                    split2(x, y, hi, lo);
+                    *reinterpret_cast<uint32_t*>(&S.ph[(smt * 16 + row) * VROW + skt * 16 + key]) = hi;
+                    *reinterpret_cast<uint32_t*>(&S.pl[(smt * 16 + row) * VROW + skt * 16 + key]) = lo;
                 }
-                uint32_t ph[4], pl[4];
-                split2(p[2 * kt][0], p[2 * kt][1], ph[0], pl[0]);
-                split2(p[2 * kt][2], p[2 * kt][3], ph[1], pl[1]);
-                split2(p[2 * kt + 1][0], p[2 * kt + 1][1], ph[2], pl[2]);
-                split2(p[2 * kt + 1][2], p[2 * kt + 1][3], ph[3], pl[3]);
+        }
+        // ---- what the state from before the segment adds to output rows [16 mt, +16), columns [oc0, +16) ----
+        float o[2][4] = {};
+        if (mt * 16 < n) {
 #pragma unroll
-                for (int np = 0; np < 2; ++np) {
-                    uint32_t b0, b1, b2, b3;
-                    ldmatrix_x4_trans(smem_u32(&V[(kt * 16 + (mi & 1) * 8 + r8) * VROW + oc0 + np * 16 + (mi >> 1) * 8]), b0, b1, b2, b3);
-                    mma_bf16_16816(o[2 * np], ph, b0, b1);
-                    mma_bf16_16816(o[2 * np + 1], ph, b2, b3);
-                    mma_bf16_16816(o[2 * np], pl, b0, b1);
-                    mma_bf16_16816(o[2 * np + 1], pl, b2, b3);
-                }
-            }
-            __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + static_cast<int64_t>(h) * vp + v0 + oc0;
-#pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                const int t = mt * 16 + g + half * 8;
-                if (t >= n) continue;
-                __nv_bfloat16* dst = out + static_cast<int64_t>(begin + s0 + t) * a.heads * vp;
-#pragma unroll
-                for (int j = 0; j < 4; ++j)
-                    *reinterpret_cast<uint32_t*>(dst + j * 8 + 2 * tq) = pack_bf16(o[j][2 * half], o[j][2 * half + 1]);
+            for (int ks = 0; ks < DK / 16; ++ks) {
+                uint32_t ah[4], al[4], b0, b1, b2, b3;
+                const int aoff = (mt * 16 + (mi & 1) * 8 + r8) * ROW + ks * 16 + (mi >> 1) * 8;
+                const int soff = (ks * 16 + (mi & 1) * 8 + r8) * VROW + oc0 + (mi >> 1) * 8;
+                ldmatrix_x4(smem_u32(&S.qh[aoff]), ah[0], ah[1], ah[2], ah[3]);
+                ldmatrix_x4(smem_u32(&S.ql[aoff]), al[0], al[1], al[2], al[3]);
+                ldmatrix_x4_trans(smem_u32(&S.sh[soff]), b0, b1, b2, b3);
+                mma_bf16_16816(o[0], ah, b0, b1);
+                mma_bf16_16816(o[1], ah, b2, b3);
+                mma_bf16_16816(o[0], al, b0, b1);
+                mma_bf16_16816(o[1], al, b2, b3);
+                ldmatrix_x4_trans(smem_u32(&S.sl[soff]), b0, b1, b2, b3);
+                mma_bf16_16816(o[0], ah, b0, b1);
+                mma_bf16_16816(o[1], ah, b2, b3);
             }
         }
         // ---- the state after the segment ----
@@ -551,9 +539,34 @@ linear_attention_chunk_kernel(const LinearAttention a) {
 #pragma unroll
                 for (int e = 0; e < 4; ++e) st[j][e] = decay[e >> 1] * st[j][e] + rest[e >> 1] * u[j][e];
         }
+        __syncthreads();   // the scores are complete
+        if (mt * 16 < n) {
+#pragma unroll
+            for (int kt = 0; kt < 4; ++kt) {
+                if (kt > mt) continue;
+                uint32_t ah[4], al[4], b0, b1, b2, b3;
+                const int poff = (mt * 16 + (mi & 1) * 8 + r8) * VROW + kt * 16 + (mi >> 1) * 8;
+                ldmatrix_x4(smem_u32(&S.ph[poff]), ah[0], ah[1], ah[2], ah[3]);
+                ldmatrix_x4(smem_u32(&S.pl[poff]), al[0], al[1], al[2], al[3]);
+                ldmatrix_x4_trans(smem_u32(&V[(kt * 16 + (mi & 1) * 8 + r8) * VROW + oc0 + (mi >> 1) * 8]), b0, b1, b2, b3);
+                mma_bf16_16816(o[0], ah, b0, b1);
+                mma_bf16_16816(o[1], ah, b2, b3);
+                mma_bf16_16816(o[0], al, b0, b1);
+                mma_bf16_16816(o[1], al, b2, b3);
+            }
+            __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + static_cast<int64_t>(h) * vp + v0 + oc0;
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int t = mt * 16 + g + half * 8;
+                if (t >= n) continue;
+                __nv_bfloat16* dst = out + static_cast<int64_t>(begin + s0 + t) * a.heads * vp;
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+                    *reinterpret_cast<uint32_t*>(dst + j * 8 + 2 * tq) = pack_bf16(o[j][2 * half], o[j][2 * half + 1]);
+            }
+        }
         s0 += n;
         buf ^= 1;
-        __syncthreads();   // q~, k~, S and b are written again
     }
 #pragma unroll
     for (int j = 0; j < kStateTiles; ++j)
@@ -626,6 +639,7 @@ int b200_linear_attention(const b200_linear_attention_args* p, int dtype, b200_s
                        b200::linear_attention_supported(p->padded_value_dim, p->padded_dim), "linear_attention: bad head sizes");
     B200_CHECK_ARG(p->rank > 0 && p->up_ld >= p->rank && p->up_ld % 16 == 0 && p->joint_ld % 8 == 0 && p->tau > 0.f,
                    "linear_attention: bad decay projection");
+    B200_CHECK_ARG(static_cast<int64_t>(p->tokens) * p->heads < (1ll << 31), "linear_attention: too many tokens");
     B200_CHECK_ARG(!p->decode || p->tokens == p->batch, "linear_attention: a decode step brings one token per request");
     if (p->tokens == 0 || p->batch == 0) return B200_OK;
     B200_CHECK_ARG(p->out && p->joint && p->table_idx && p->cached && (p->decode || p->qo_indptr) && p->state && p->up &&

@@ -119,6 +119,86 @@ head_prepare_kernel(const HeadPrepare a) {
     }
 }
 
+// The same for heads of 128 whose rotation pairs lie whole groups of four elements apart: a lane keeps four elements
+// of a row and gets their partners from another lane; one CTA per token, a warp has the loads of kFastRows rows in flight.
+constexpr int kFastRows = 4;
+
+template <typename T>
+__global__ void __launch_bounds__(kPrepareWarps * 32)
+head_prepare_128_kernel(const HeadPrepare a) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, e0 = lane * 4;
+    const int rows = a.heads + 2 * a.kv_heads;
+    const int64_t t = blockIdx.x;
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int half = a.rotary_dim >> 1;
+    const bool turns = e0 < a.rotary_dim;
+    const int pair = !turns ? lane : e0 < half ? lane + half / 4 : lane - half / 4;
+    const int64_t slot = a.out_loc[t];
+    int pos = a.positions[t];
+    const bool slot_ok = slot >= 0 && slot < a.num_slots;
+    if (threadIdx.x == 0 && !slot_ok) atomicExch(&a.status[kStatusBadIndex], static_cast<int>(slot) + 1);
+    if (pos < 0 || pos >= a.max_pos) {
+        if (threadIdx.x == 0) atomicExch(&a.status[kStatusBadIndex], pos + 1);
+        pos = min(max(pos, 0), a.max_pos - 1);
+    }
+    float4 c = make_float4(1.f, 1.f, 1.f, 1.f), s = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (turns) {
+        const int64_t at = static_cast<int64_t>(pos) * half + (e0 < half ? e0 : e0 - half);
+        c = load4(a.cos_t + at);
+        s = load4(a.sin_t + at);
+        if (e0 < half) s = make_float4(-s.x, -s.y, -s.z, -s.w);
+    }
+    const float4 one = make_float4(1.f, 1.f, 1.f, 1.f);
+    const float4 wq = a.q_weight != nullptr ? load4(static_cast<const T*>(a.q_weight) + e0) : one;
+    const float4 wk = a.k_weight != nullptr ? load4(static_cast<const T*>(a.k_weight) + e0) : one;
+    const float lambda = a.mix == HeadPrepare::kMix ? *a.lambda : 0.f;
+    T* joint = static_cast<T*>(a.joint) + t * a.ld;
+    for (int r0 = warp; r0 < rows; r0 += kPrepareWarps * kFastRows) {
+        float4 x[kFastRows];
+#pragma unroll
+        for (int i = 0; i < kFastRows; ++i) {
+            const int r = r0 + i * kPrepareWarps;
+            if (r < rows) x[i] = load4(joint + r * 128 + e0);
+        }
+#pragma unroll
+        for (int i = 0; i < kFastRows; ++i) {
+            const int r = r0 + i * kPrepareWarps;
+            if (r >= rows) break;
+            float4 v = x[i];
+            const bool is_q = r < a.heads;
+            if (r >= a.heads + a.kv_heads) {   // a value row
+                const int h = r - a.heads - a.kv_heads;
+                T* first = static_cast<T*>(a.first_values) + (t * a.kv_heads + h) * 128 + e0;
+                if (a.mix == HeadPrepare::kSave) store4(first, v);
+                if (a.mix == HeadPrepare::kMix) {
+                    const float4 f = load4(first);
+                    v.x = (1.f - lambda) * v.x + lambda * f.x;
+                    v.y = (1.f - lambda) * v.y + lambda * f.y;
+                    v.z = (1.f - lambda) * v.z + lambda * f.z;
+                    v.w = (1.f - lambda) * v.w + lambda * f.w;
+                }
+                if (slot_ok) store4(static_cast<T*>(a.v_cache) + (slot * a.kv_heads + h) * 128 + e0, v);
+                continue;
+            }
+            if ((is_q ? a.q_weight : a.k_weight) != nullptr) {
+                const float scale =
+                    rsqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / static_cast<float>(a.dim) + a.eps);
+                const float4 w = is_q ? wq : wk;
+                v = make_float4(v.x * scale * w.x, v.y * scale * w.y, v.z * scale * w.z, v.w * scale * w.w);
+            }
+            float4 o;
+            o.x = __shfl_sync(0xffffffffu, v.x, pair);
+            o.y = __shfl_sync(0xffffffffu, v.y, pair);
+            o.z = __shfl_sync(0xffffffffu, v.z, pair);
+            o.w = __shfl_sync(0xffffffffu, v.w, pair);
+            v = make_float4(v.x * c.x + o.x * s.x, v.y * c.y + o.y * s.y, v.z * c.z + o.z * s.z, v.w * c.w + o.w * s.w);
+            T* dst = is_q ? joint + r * 128 : static_cast<T*>(a.k_cache) + (slot * a.kv_heads + (r - a.heads)) * 128;
+            if (is_q || slot_ok) store4(dst + e0, v);
+        }
+    }
+}
+
 // ---- plain attention: any sizes, fp32 or bf16 ------------------------------------
 
 constexpr int kPlainThreads = 128;
@@ -221,6 +301,11 @@ window_attention_plain_kernel(const WindowAttention a) {
 int launch_head_prepare(const HeadPrepare& a, int dtype, cudaStream_t stream) {
     if (a.tokens == 0) return B200_OK;
     const int64_t rows = static_cast<int64_t>(a.tokens) * (a.heads + 2 * a.kv_heads);
+    if (a.dp == 128 && a.vp == 128 && a.rotary_dim % 8 == 0 && rows >= 4096) {
+        auto fast = dtype == B200_DTYPE_F32 ? head_prepare_128_kernel<float> : head_prepare_128_kernel<__nv_bfloat16>;
+        B200_CHECK_CUDA(launch_kernel(fast, dim3(a.tokens), dim3(kPrepareWarps * 32), 0, stream, dim3(1, 1, 1), a));
+        return B200_OK;
+    }
     auto kernel = dtype == B200_DTYPE_F32 ? head_prepare_kernel<float> : head_prepare_kernel<__nv_bfloat16>;
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(static_cast<unsigned>((rows + kPrepareWarps - 1) / kPrepareWarps)),
                                   dim3(kPrepareWarps * 32), static_cast<size_t>(kPrepareWarps) * a.dp * 4, stream,

@@ -69,7 +69,7 @@ def write_safetensors(path, tensors: dict) -> None:
     header, blobs, off = {}, [], 0
     for name, t in tensors.items():
         t = t.contiguous()
-        raw = t.view(torch.uint8).numpy().tobytes() if t.numel() else b""
+        raw = t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b""
         header[name] = {"dtype": names[t.dtype], "shape": list(t.shape), "data_offsets": [off, off + len(raw)]}
         blobs.append(raw)
         off += len(raw)
