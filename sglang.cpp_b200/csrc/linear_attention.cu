@@ -352,6 +352,22 @@ linear_attention_chunk_kernel(const LinearAttention a) {
     const __nv_bfloat16* up = static_cast<const __nv_bfloat16*>(a.up) + static_cast<int64_t>(h) * DK * a.up_ld;
     const float* bias = a.bias + static_cast<int64_t>(h) * DK;
 
+    // the first 16 ranks of this warp's channels and their bias, fetched a segment ahead (shared memory leaves no
+    // room for them to stay in L1)
+    uint32_t up0, up1;
+    float bias0, bias1;
+    auto fetch_up = [&](int r, uint32_t& b0, uint32_t& b1) {
+        const __nv_bfloat16* u = up + static_cast<int64_t>(zc0 + g) * a.up_ld + r + 2 * tq;
+        b0 = *reinterpret_cast<const uint32_t*>(u);
+        b1 = *reinterpret_cast<const uint32_t*>(u + 8);
+    };
+    auto fetch_decay = [&]() {
+        fetch_up(0, up0, up1);
+        bias0 = bias[zc0 + 2 * tq];
+        bias1 = bias[zc0 + 2 * tq + 1];
+    };
+    fetch_decay();
+
     int buf = 0;
     for (int s0 = 0; s0 < ext;) {
         const int n_max = min(kChunk, ext - s0);
@@ -364,8 +380,8 @@ linear_attention_chunk_kernel(const LinearAttention a) {
 #pragma unroll
             for (int m = 0; m < kZTokens; ++m) z[m][0] = z[m][1] = z[m][2] = z[m][3] = 0.f;
             for (int r = 0; r < a.up_ld; r += 16) {
-                const __nv_bfloat16* u = up + static_cast<int64_t>(zc0 + g) * a.up_ld + r + 2 * tq;
-                const uint32_t b0 = *reinterpret_cast<const uint32_t*>(u), b1 = *reinterpret_cast<const uint32_t*>(u + 8);
+                uint32_t b0 = up0, b1 = up1;
+                if (r > 0) fetch_up(r, b0, b1);
 #pragma unroll
                 for (int m = 0; m < kZTokens; ++m) {
                     uint32_t af[4];
@@ -375,12 +391,11 @@ linear_attention_chunk_kernel(const LinearAttention a) {
                 }
             }
             const int c = zc0 + 2 * tq;
-            const float b0 = bias[c], b1 = bias[c + 1];
 #pragma unroll
             for (int m = 0; m < kZTokens; ++m)
 #pragma unroll
                 for (int half = 0; half < 2; ++half) {
-                    const float x = z[m][2 * half] + b0, y = z[m][2 * half + 1] + b1;
+                    const float x = z[m][2 * half] + bias0, y = z[m][2 * half + 1] + bias1;
                     float2 ls;
                     ls.x = fminf(x, 0.f) * log2e_tau - lg2(1.f + ex2(-kLog2e * fabsf(x))) * inv_tau;
                     ls.y = fminf(y, 0.f) * log2e_tau - lg2(1.f + ex2(-kLog2e * fabsf(y))) * inv_tau;
@@ -540,6 +555,7 @@ linear_attention_chunk_kernel(const LinearAttention a) {
                 for (int e = 0; e < 4; ++e) st[j][e] = decay[e >> 1] * st[j][e] + rest[e >> 1] * u[j][e];
         }
         __syncthreads();   // the scores are complete
+        fetch_decay();
         if (mt * 16 < n) {
 #pragma unroll
             for (int kt = 0; kt < 4; ++kt) {
