@@ -75,9 +75,15 @@ struct DecodeParams {
 struct StageRange {
     int count, head, skip;
 };
+template <bool WINDOW>
 __device__ __forceinline__ StageRange stage_range(int len, int stage_keys, int window, int keep_first) {
     len = max(len, 0);
     StageRange r;
+    if (!WINDOW) {
+        r.head = r.skip = 0;
+        r.count = (len + stage_keys - 1) / stage_keys;
+        return r;
+    }
     r.head = (min(keep_first, len) + stage_keys - 1) / stage_keys;
     r.skip = max(0, max(0, len - window) / stage_keys - r.head);
     r.count = (len + stage_keys - 1) / stage_keys - r.skip;
@@ -141,7 +147,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
         int carry = 0;
         for (int base = 0; base < B; base += 32) {
             const int b = base + lane;
-            const int n = b < B ? stage_range(p.seq_lens[b], SK, p.window, p.keep_first).count : 0;
+            const int n = b < B ? stage_range<WINDOW>(p.seq_lens[b], SK, p.window, p.keep_first).count : 0;
             int incl = n;
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -185,9 +191,12 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
         it.nchunks = (first + st - 1) / per - c0 + 1;   // CTAs that share this request
         it.first_slot = lo + c0;
         it.item = lo + static_cast<int>(blockIdx.x);
-        const StageRange range = stage_range(it.len, SK, p.window, p.keep_first);
-        it.head = range.head;
-        it.skip = range.skip;
+        it.head = it.skip = 0;
+        if (WINDOW) {
+            const StageRange range = stage_range<WINDOW>(it.len, SK, p.window, p.keep_first);
+            it.head = range.head;
+            it.skip = range.skip;
+        }
         return it;
     };
 
@@ -208,11 +217,17 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
             auto stage_key = [&](int st) { return (WINDOW && st >= it.head ? st + it.skip : st) * SK; };
             const int cps = SK / p.kpc;   // copies of a whole stage, a power of two
             const int cps_shift = 31 - __clz(cps);
-            const int item_copies = (it.s_end - it.s_begin) * cps;
+            const int first_key = it.s_begin * SK;
+            const int item_copies = WINDOW ? (it.s_end - it.s_begin) * cps
+                                           : (min(it.len, it.s_end * SK) - first_key + p.kpc - 1) / p.kpc;
             // Slot of the first key of every copy of this item (the previous item's
             // table is no longer needed: all of its copies have been issued).
             __syncwarp();
             for (int c = lane; c < min(item_copies, kSlotTab); c += 32) {
+                if (!WINDOW) {
+                    s_slot_tab[c] = pt_row[first_key + c * p.kpc];
+                    continue;
+                }
                 const int key = stage_key(it.s_begin + (c >> cps_shift)) + (c & (cps - 1)) * p.kpc;
                 s_slot_tab[c] = key < it.len ? pt_row[key] : 0;
             }
@@ -237,7 +252,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
                 const uint32_t stage_base = smem_base + slot * kStageBytes;
                 for (int ci = lane; ci < ncopies * 4; ci += 32) {
                     const int copy = ci >> 2, which = ci & 3;
-                    const int tab = (st - it.s_begin) * cps + copy;
+                    const int tab = (WINDOW ? (st - it.s_begin) * cps : (k0 - first_key) / p.kpc) + copy;
                     int64_t sl = tab < kSlotTab ? s_slot_tab[tab] : pt_row[k0 + copy * p.kpc];
                     if (sl < 0 || sl + p.kpc > p.num_slots) {
                         atomicExch(&p.status[kStatusBadIndex], static_cast<int>(sl) + 1);
@@ -462,6 +477,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
 // of the streaming kernel on purpose: there the CTA that happened to deliver a request's last partial
 // merged it behind its own last stage, a chain of fences, a ticket and three dependent trips to L2 that
 // left the other 147 SMs and HBM idle for about 12 us per launch.
+template <bool WINDOW>
 __global__ void __launch_bounds__(kMergeWarps * 32)
 attention_decode_merge_kernel(const DecodeParams p, int attn_grid) {
     __shared__ int s_first, s_stages, s_total;
@@ -477,7 +493,7 @@ attention_decode_merge_kernel(const DecodeParams p, int attn_grid) {
         int carry = 0, first = 0, mine = 0;
         for (int base = 0; base < p.batch; base += 32) {
             const int r = base + lane;
-            const int n = r < p.batch ? stage_range(p.seq_lens[r], SK, p.window, p.keep_first).count : 0;
+            const int n = r < p.batch ? stage_range<WINDOW>(p.seq_lens[r], SK, p.window, p.keep_first).count : 0;
             int incl = n;
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -553,7 +569,7 @@ attention_decode_merge_kernel(const DecodeParams p, int attn_grid) {
     uint2 packed;
     packed.x = pack_bf16(acc.x * inv, acc.y * inv);
     packed.y = pack_bf16(acc.z * inv, acc.w * inv);
-    if (p.gate != nullptr) {
+    if (WINDOW && p.gate != nullptr) {
         const uint2 g = *reinterpret_cast<const uint2*>(p.gate + b * p.gate_st + head * kD + lane * 4);
         packed.x = gate_pair(g.x, acc.x * inv, acc.y * inv);
         packed.y = gate_pair(g.y, acc.z * inv, acc.w * inv);
@@ -625,7 +641,8 @@ int launch_attention_decode(void* out, const void* q, int64_t q_st, int64_t q_sh
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(grid), dim3(kThreads), smem, stream,
                                   dim3(1, 1, 1), tmap_k, tmap_v, p));
     const int merge_ctas = batch * ((q_heads + kMergeWarps - 1) / kMergeWarps);
-    B200_CHECK_CUDA(launch_kernel(attention_decode_merge_kernel, dim3(merge_ctas), dim3(kMergeWarps * 32), 0, stream,
+    auto merge = window ? attention_decode_merge_kernel<true> : attention_decode_merge_kernel<false>;
+    B200_CHECK_CUDA(launch_kernel(merge, dim3(merge_ctas), dim3(kMergeWarps * 32), 0, stream,
                                   dim3(1, 1, 1), p, grid));
     return B200_OK;
 }
