@@ -327,6 +327,14 @@ B200_API int b200_latent_attention(void* out, const void* q, const void* cache, 
                                    const int32_t* row_table, const int32_t* row_len, int rows, int heads,
                                    int width, int page_size, float scale, int dtype, int plain,
                                    void* workspace, int64_t workspace_bytes, b200_stream_t stream);
+/* The same where only the first out_width columns of a latent are averaged (out [rows, heads, out_width], a multiple
+ * of 128): the others, a rotated part of the keys for instance, take part in the scores alone.  The tensor-core
+ * kernel takes widths of up to 640 with up to 512 of them averaged. */
+B200_API int b200_latent_attention_part(void* out, const void* q, const void* cache, int64_t num_slots,
+                                        const int32_t* page_table, int64_t page_table_stride,
+                                        const int32_t* row_table, const int32_t* row_len, int rows, int heads,
+                                        int width, int out_width, int page_size, float scale, int dtype, int plain,
+                                        void* workspace, int64_t workspace_bytes, b200_stream_t stream);
 
 /* residual[t, :] += sum_k src_scale * src[src_rows[t * src_top + k], :]   (src NULL: nothing added;
  * src_rows NULL: row t; init != 0: the sum replaces the residual instead, e.g. an embedding lookup), then
@@ -430,6 +438,11 @@ typedef struct b200_window_attention_args {
     int64_t gate_stride;
     void* workspace;
     int64_t workspace_bytes;
+    int32_t chunk;           /* > 0, instead of the window: key j is seen if i / chunk = j / chunk */
+    const float* sinks;      /* [heads] or NULL: exp(sinks[h]) joins the softmax's denominator */
+    int32_t gate_per_head;   /* the gate is [tokens, heads]: one number per head */
+    float out_scale;         /* a factor on the output; 0 means 1 */
+    int64_t out_stride;      /* token stride of out in elements; 0: dense */
 } b200_window_attention_args;
 B200_API int b200_window_attention(const b200_window_attention_args* args, int dtype, b200_stream_t stream);
 
@@ -456,6 +469,59 @@ typedef struct b200_linear_attention_args {
     float tau, eps, q_scale;
 } b200_linear_attention_args;
 B200_API int b200_linear_attention(const b200_linear_attention_args* args, int dtype, b200_stream_t stream);
+
+/* Recurrences with one decay per head, behind a short causal convolution.  joint [tokens, joint_ld] holds
+ * [gate | v: heads * padded_value_dim each | k | q: kv_heads * padded_dim each | a of every head, and for the delta
+ * rule b of every head]; head h uses k / q head h / (heads / kv_heads).
+ *   v, k, q <- silu(conv(.) + conv_bias): conv [taps, channels] per channel of [v | k | q], the last tap the
+ *   current token's; conv_state [rows, taps, channels] of the dtype keeps the last inputs, that of position p at
+ *   p mod taps
+ * B200_RULE_STATE_SPACE:  dt = softplus(a + step_bias), g = exp(-exp(decay_log) dt)
+ *   S <- g S + dt k v^T,  o = S^T q + skip * v,  out = rms(o * silu(gate)) * norm in norm_groups equal parts of the
+ *   concatenated (true) heads; norm [heads * padded_value_dim]
+ * B200_RULE_DELTA:  g = exp(-exp(decay_log) softplus(a + step_bias)), beta = sigmoid(b); k and q divided by
+ *   sqrt(sum of squares + 1e-6), q also by sqrt(dim)
+ *   S <- g S,  u = beta (v - S^T k),  S <- S + k u^T,  o = S^T q,  out = rms(o) * norm * silu(gate) per head; norm
+ *   [padded_value_dim]
+ * out [tokens, out_ld] is also multiplied by out_scale.  state fp32 [rows, heads, padded_dim, padded_value_dim];
+ * rows, requests, decode and plain as for b200_linear_attention; a request brings at most max_extend tokens.  conv,
+ * conv_bias (NULL: 0), decay_log, step_bias, skip are fp32.  Scratch: b200_recurrence_scratch. */
+enum { B200_RULE_STATE_SPACE = 0, B200_RULE_DELTA = 1 };
+typedef struct b200_recurrence_args {
+    void* out;
+    int64_t out_ld;
+    const void* joint;
+    int64_t joint_ld;
+    int32_t rule, tokens, batch, max_extend, decode, plain;
+    const int32_t *table_idx, *cached, *qo_indptr;
+    float* state;
+    void* conv_state;
+    int32_t heads, kv_heads, dim, padded_dim, value_dim, padded_value_dim, taps, norm_groups;
+    const float *conv, *conv_bias, *decay_log, *step_bias, *skip;
+    const void* norm;
+    float eps, out_scale;
+    void* mixed;       /* [tokens, channels] of the dtype */
+    float* steps;      /* [tokens, heads, 2]: log2 of the decay, weight of what is written */
+    float* units;      /* delta rule [tokens, 2 kv_heads]: factors that make k and q unit vectors */
+    void* chunks;      /* per 64 tokens and head: matrices of the chunked kernel */
+} b200_recurrence_args;
+B200_API int b200_recurrence(const b200_recurrence_args* args, int dtype, b200_stream_t stream);
+/* Bytes of mixed, steps, units and chunks for steps of at most max_tokens tokens of max_batch requests. */
+B200_API int b200_recurrence_scratch(int rule, int max_tokens, int max_batch, int heads, int kv_heads, int padded_dim,
+                                     int padded_value_dim, int dtype, int64_t* bytes);
+
+/* residual_post_norm where what is added is the sum of two rows per token, each RMS-normalised with its own weight,
+ * times pair_scale. */
+B200_API int b200_residual_pair_norm(void* out, float* residual, const void* src, const void* src2,
+                                     const void* weight, const void* weight2, float pair_scale, const void* add_weight,
+                                     const void* out_weight, int tokens, int width, int padded, float eps, int dtype,
+                                     b200_stream_t stream);
+
+/* The first `dims` elements of every head of x [tokens, heads, ld] rotated in place, element 2i with its
+ * neighbour, by the angles whose cosines and sines are in the tables [max_pos, dims / 2]. */
+B200_API int b200_rotate_pairs(void* x, int tokens, int heads, int ld, int dims, const float* cos_table,
+                               const float* sin_table, const int32_t* positions, int max_pos, int dtype,
+                               b200_stream_t stream);
 
 /* ---- tensor-parallel all-reduce (include/sglang/distributed/distributed.h:24) --- */
 
@@ -580,7 +646,20 @@ typedef struct b200_engine b200_engine;
  * multiple of 64 (b200_pad_width; head and value dimensions up to 128 are padded to 128, latent widths
  * to a multiple of 128), vectors likewise; norms divide by the true width. */
 enum { B200_DTYPE_BF16 = 0, B200_DTYPE_F32 = 1 };
-enum { B200_MIXER_LATENT_ATTENTION = 0, B200_MIXER_WINDOW_ATTENTION = 1, B200_MIXER_LINEAR_ATTENTION = 2 };
+enum {
+    B200_MIXER_LATENT_ATTENTION = 0,
+    B200_MIXER_WINDOW_ATTENTION = 1,
+    B200_MIXER_LINEAR_ATTENTION = 2,
+    B200_MIXER_STATE_SPACE = 3,   /* b200_recurrence, either rule */
+    B200_MIXER_DELTA_RULE = 4
+};
+enum { B200_GATE_NONE = 0, B200_GATE_ELEMENT = 1, B200_GATE_HEAD = 2 };
+/* How the outputs of two mixers side by side become one. */
+enum {
+    B200_JOIN_SUM = 0,      /* added, each times its out_scale, by one output projection */
+    B200_JOIN_NORMED = 1    /* each RMS-normalised with its own weight, then half of their sum */
+};
+enum { B200_NORM_INPUT = 0, B200_NORM_OUTPUT = 1, B200_NORM_BOTH = 2 };
 enum { B200_MLP_NONE = 0, B200_MLP_DENSE = 1, B200_MLP_TABLE_MOE = 2, B200_MLP_SCORED_MOE = 3 };
 
 typedef struct b200_layer_config {
@@ -616,6 +695,24 @@ typedef struct b200_layer_config {
     /* limits of B200_EPILOGUE_CLAMPED_SWIGLU */
     float act_limit;
     float shared_act_limit;
+    /* window attention */
+    int32_t head_norm;       /* RMS norms on queries and keys */
+    int32_t gate;            /* B200_GATE_* on the output */
+    int32_t qkv_bias;
+    int32_t sink;            /* a score per head that joins the softmax's denominator */
+    int32_t chunk;           /* > 0, instead of the window: keys of the query's own chunk of the sequence */
+    /* rotations (latent attention: of the rotary_dim key dimensions that all heads share, in neighbouring pairs):
+     * frequencies divided by rope_factor where their wavelength exceeds rope_original / rope_low, kept below
+     * rope_original / rope_high, blended between; factor 0: none */
+    double rope_factor, rope_low, rope_high, rope_original;
+    int32_t kv_from;         /* latent attention: the layer whose latents this one reads, -1: its own */
+    /* recurrences (head_dim: state rows; kv_heads: heads of k and q) */
+    int32_t conv_taps;
+    int32_t norm_groups;
+    /* a second mixer that reads the same input */
+    int32_t beside;          /* index into the stack's `beside`, -1: none */
+    int32_t join;            /* B200_JOIN_* */
+    float out_scale;         /* of this mixer's output (window attention, recurrences) */
 } b200_layer_config;
 
 typedef struct b200_stack_config {
@@ -624,14 +721,19 @@ typedef struct b200_stack_config {
     int32_t dtype;       /* B200_DTYPE_*: bf16 matrices and activations, or everything in fp32 */
     float norm_offset;   /* added to the stored weights of the layer norms and the final norm (0 or 1) */
     float logit_scale;
-    int32_t norm_output; /* 0: blocks read the normalised residual; 1: they read the residual, and what they
-                            return is normalised before it is added */
+    int32_t norm_output; /* B200_NORM_*: blocks read the normalised residual; or they read the residual, and what
+                            they return is normalised before it is added; or both */
+    int32_t num_beside;
+    const b200_layer_config* beside;   /* mixers that run beside another one (only mixer fields are read) */
 } b200_stack_config;
 
 /* The padded size of a width / of a per-head dimension / of a latent width (see above). */
 B200_API int b200_pad_width(int n);
 B200_API int b200_pad_head_dim(int n);
 B200_API int b200_pad_latent(int n);
+/* The column where the rotated part of a latent row starts (latents with one are kv_rank numbers, padding up to
+ * there, and the rotated part, padded as a whole). */
+B200_API int b200_latent_rope_at(int kv_rank);
 
 /* Engine::Engine (src/engine/engine.cc:412-489): allocates weights (uninitialised), the KV
  * pool [2, L, (num_pages+1)*page_size, kv_heads/tp, head_dim], the page table and token pool
@@ -658,7 +760,13 @@ B200_API int b200_engine_destroy(b200_engine* engine);
  * hidden], "q_head_norm", "k_head_norm" [dim], "value_mix" (one float), "o", "k_cache", "v_cache".  Linear
  * attention (dimensions padded to a multiple of 64): "qkvga" [2 heads*dim + 2 heads*vdim + rank, hidden],
  * "decay_up" [heads*dim, rank padded to 16], "decay_bias" fp32 [heads*dim], "head_norm" [vdim], "o",
- * "state" fp32 [max_running_req + 1, heads, dim, vdim].  Scored experts: "router" [experts, hidden],
+ * "state" fp32 [max_running_req + 1, heads, dim, vdim].  Recurrences (dimensions padded the same way): "recurrence"
+ * [the columns of b200_recurrence's joint rows, hidden], "conv" [taps, channels], "conv_bias" [channels], "decay_log",
+ * "step_bias", "skip" [heads], all fp32, "head_norm", "o", "state", "conv_state".  Optional: "joint_bias" of the
+ * input projection, "sinks" fp32 [heads], "norm1_out", "norm2_out".  Two mixers side by side share the input
+ * projection "joint" [left columns + right columns, hidden], and under B200_JOIN_SUM "o" [hidden, left + right];
+ * under B200_JOIN_NORMED there are "side_norm" [hidden] and the right one's "beside_o", "beside_side_norm".  The names
+ * of the right one's other tensors start with "beside_".  Scored experts: "router" [experts, hidden],
  * "mlp_up", "mlp_down", "shared_up", "shared_down". */
 B200_API int b200_engine_tensor(b200_engine* engine, const char* name, int layer, void** device_ptr,
                                 int64_t* nbytes);

@@ -33,7 +33,11 @@ EPILOGUE_CLAMPED_SWIGLU = 6
 EPILOGUE_F32 = 7
 
 DTYPE_BF16, DTYPE_F32 = 0, 1
-MIXER_LATENT_ATTENTION, MIXER_WINDOW_ATTENTION, MIXER_LINEAR_ATTENTION = 0, 1, 2
+MIXER_LATENT_ATTENTION, MIXER_WINDOW_ATTENTION, MIXER_LINEAR_ATTENTION, MIXER_STATE_SPACE, MIXER_DELTA_RULE = 0, 1, 2, 3, 4
+RULE_STATE_SPACE, RULE_DELTA = 0, 1
+GATE_NONE, GATE_ELEMENT, GATE_HEAD = 0, 1, 2
+JOIN_SUM, JOIN_NORMED = 0, 1
+NORM_INPUT, NORM_OUTPUT, NORM_BOTH = 0, 1, 2
 MLP_NONE, MLP_DENSE, MLP_TABLE_MOE, MLP_SCORED_MOE = 0, 1, 2, 3
 
 
@@ -107,6 +111,11 @@ PROTOTYPES: dict[str, tuple] = {
     "b200_engine_comm_connect": (_I, [_P, _P]),
     "b200_latent_attention_workspace_bytes": (_L, [_I, _I, _I]),
     "b200_latent_attention": (_I, [_P, _P, _P, _L, _P, _L, _P, _P, _I, _I, _I, _I, _F, _I, _I, _P, _L, _P]),
+    "b200_latent_attention_part": (_I, [_P, _P, _P, _L, _P, _L, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P, _L, _P]),
+    "b200_rotate_pairs": (_I, [_P, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P]),
+    "b200_residual_pair_norm": (_I, [_P, _P, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _F, _I, _P]),
+    "b200_recurrence": (_I, [_P, _I, _P]),
+    "b200_recurrence_scratch": (_I, [_I, _I, _I, _I, _I, _I, _I, _I, POINTER(c_int64)]),
     "b200_residual_norm": (_I, [_P, _P, _I, _P, _P, _P, _I, _L, _F, _I, _P, _F, _F, _I, _I, _I, _F, _I, _P]),
     "b200_table_route": (_I, [_P, _P, _P, _P, _P, _I, _I, _I, _I, _P]),
     "b200_linear_heads": (_I, [_P, _P, _P, _I, _I, _I, _I, _P]),
@@ -120,6 +129,7 @@ PROTOTYPES: dict[str, tuple] = {
     "b200_pad_width": (_I, [_I]),
     "b200_pad_head_dim": (_I, [_I]),
     "b200_pad_latent": (_I, [_I]),
+    "b200_latent_rope_at": (_I, [_I]),
     "b200_engine_create_stack": (_I, [_P, _P, _P, POINTER(c_void_p)]),
     "b200_engine_token_logits": (_I, [_P, _P, _I, _P]),
     "b200_engine_trace_residual": (_I, [_P, _P]),
@@ -167,7 +177,10 @@ class LayerConfigStruct(ctypes.Structure):
         ("rotary_dim", c_int32), ("rope_base", ctypes.c_double), ("value_mix", c_int32),
         ("decay_rank", c_int32), ("decay_tau", c_float), ("router_groups", c_int32), ("router_keep", c_int32),
         ("router_scale", c_float), ("shared_intermediate", c_int32), ("act_limit", c_float),
-        ("shared_act_limit", c_float),
+        ("shared_act_limit", c_float), ("head_norm", c_int32), ("gate", c_int32), ("qkv_bias", c_int32),
+        ("sink", c_int32), ("chunk", c_int32), ("rope_factor", ctypes.c_double), ("rope_low", ctypes.c_double),
+        ("rope_high", ctypes.c_double), ("rope_original", ctypes.c_double), ("kv_from", c_int32),
+        ("conv_taps", c_int32), ("norm_groups", c_int32), ("beside", c_int32), ("join", c_int32), ("out_scale", c_float),
     ]
 
 
@@ -191,6 +204,7 @@ class WindowAttentionArgs(ctypes.Structure):
         ("decode", c_int32), ("plain", c_int32), ("heads", c_int32), ("kv_heads", c_int32), ("padded_dim", c_int32),
         ("padded_value_dim", c_int32), ("page_size", c_int32), ("scale", c_float), ("window", c_int32),
         ("keep_first", c_int32), ("gate", _P), ("gate_stride", _L), ("workspace", _P), ("workspace_bytes", _L),
+        ("chunk", c_int32), ("sinks", _P), ("gate_per_head", c_int32), ("out_scale", c_float), ("out_stride", _L),
     ]
 
 
@@ -205,11 +219,25 @@ class LinearAttentionArgs(ctypes.Structure):
     ]
 
 
+class RecurrenceArgs(ctypes.Structure):
+    """b200_recurrence_args."""
+    _fields_ = [
+        ("out", _P), ("out_ld", _L), ("joint", _P), ("joint_ld", _L), ("rule", c_int32), ("tokens", c_int32),
+        ("batch", c_int32), ("max_extend", c_int32), ("decode", c_int32), ("plain", c_int32), ("table_idx", _P),
+        ("cached", _P), ("qo_indptr", _P), ("state", _P), ("conv_state", _P), ("heads", c_int32), ("kv_heads", c_int32),
+        ("dim", c_int32), ("padded_dim", c_int32), ("value_dim", c_int32), ("padded_value_dim", c_int32),
+        ("taps", c_int32), ("norm_groups", c_int32), ("conv", _P), ("conv_bias", _P), ("decay_log", _P),
+        ("step_bias", _P), ("skip", _P), ("norm", _P), ("eps", c_float), ("out_scale", c_float), ("mixed", _P),
+        ("steps", _P), ("units", _P), ("chunks", _P),
+    ]
+
+
 class StackConfigStruct(ctypes.Structure):
     """b200_stack_config."""
     _fields_ = [
         ("num_layers", c_int32), ("layers", POINTER(LayerConfigStruct)), ("dtype", c_int32),
-        ("norm_offset", c_float), ("logit_scale", c_float), ("norm_output", c_int32),
+        ("norm_offset", c_float), ("logit_scale", c_float), ("norm_output", c_int32), ("num_beside", c_int32),
+        ("beside", POINTER(LayerConfigStruct)),
     ]
 
 

@@ -23,9 +23,9 @@
 //   * every warp writes an (m, l, O) partial (or, for a request that is a single partial, bf16
 //     outputs at once); a second, tiny kernel merges the partials of every request, one warp per
 //     (request, query head), so the streaming kernel ends with its last stage.
-// WINDOW: a sliding window with kept first keys.  A request's stages are then those that hold a kept key and
-// those from the oldest key in the window on; what lies between is never loaded.  The output passes a sigmoid
-// gate where it is written as bf16.
+// WINDOW: everything AttentionWindow has.  A request's stages are then those that hold a kept key and those from
+// the oldest key in the window on; what lies between is never loaded.  Sinks, gates and the output's factor are
+// applied where it is written as bf16.
 #include <mutex>
 
 #include "common.cuh"
@@ -66,9 +66,7 @@ struct DecodeParams {
     int max_items;
     int* status;
     int kv_evict_first;   // stream K/V through L2 with the evict-first policy (read once per step)
-    int window, keep_first;       // 0x7fffffff, 0 without a window
-    const __nv_bfloat16* gate;    // WINDOW only
-    int64_t gate_st;
+    AttentionWindow w;            // WINDOW only
 };
 
 // Which stages of a request of `len` keys are read: stage numbers [0, head) and, `skip` further, [head, count).
@@ -76,7 +74,7 @@ struct StageRange {
     int count, head, skip;
 };
 template <bool WINDOW>
-__device__ __forceinline__ StageRange stage_range(int len, int stage_keys, int window, int keep_first) {
+__device__ __forceinline__ StageRange stage_range(int len, int stage_keys, const AttentionWindow& w) {
     len = max(len, 0);
     StageRange r;
     if (!WINDOW) {
@@ -84,14 +82,20 @@ __device__ __forceinline__ StageRange stage_range(int len, int stage_keys, int w
         r.count = (len + stage_keys - 1) / stage_keys;
         return r;
     }
-    r.head = (min(keep_first, len) + stage_keys - 1) / stage_keys;
-    r.skip = max(0, max(0, len - window) / stage_keys - r.head);
+    r.head = (min(w.keep_first, len) + stage_keys - 1) / stage_keys;
+    r.skip = max(0, (len > 0 ? w.oldest(len - 1) : 0) / stage_keys - r.head);
     r.count = (len + stage_keys - 1) / stage_keys - r.skip;
     return r;
 }
 __device__ __forceinline__ uint32_t gate_pair(uint32_t g, float lo, float hi) {
     return pack_bf16(lo * sigmoid_f(bf16_lo(g)), hi * sigmoid_f(bf16_hi(g)));
 }
+// What every element of a head's output is multiplied by, the softmax denominator apart.
+__device__ __forceinline__ float head_factor(const AttentionWindow& w, int b, int head) {
+    if (w.gate == nullptr || !w.gate_per_head) return w.out_scale;
+    return w.out_scale * sigmoid_f(__bfloat162float(static_cast<const __nv_bfloat16*>(w.gate)[b * w.gate_st + head]));
+}
+constexpr float kLog2e = 1.4426950408889634f;
 
 struct ItemInfo {
     int b, len, s_begin, s_end, nchunks, item, first_slot;
@@ -147,7 +151,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
         int carry = 0;
         for (int base = 0; base < B; base += 32) {
             const int b = base + lane;
-            const int n = b < B ? stage_range<WINDOW>(p.seq_lens[b], SK, p.window, p.keep_first).count : 0;
+            const int n = b < B ? stage_range<WINDOW>(p.seq_lens[b], SK, p.w).count : 0;
             int incl = n;
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -193,7 +197,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
         it.item = lo + static_cast<int>(blockIdx.x);
         it.head = it.skip = 0;
         if (WINDOW) {
-            const StageRange range = stage_range<WINDOW>(it.len, SK, p.window, p.keep_first);
+            const StageRange range = stage_range<WINDOW>(it.len, SK, p.w);
             it.head = range.head;
             it.skip = range.skip;
         }
@@ -317,8 +321,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
                 failed = true;
             const int key0 = (WINDOW && st >= it.head ? st + it.skip : st) * SK + kg * 16;   // first key of this warp's tile
             const int nvalid = it.len - key0;  // valid keys in it
-            const int oldest = it.len - p.window;
-            const bool seen = !WINDOW || key0 + min(nvalid, 16) > oldest || key0 < p.keep_first;
+            const int oldest = WINDOW ? p.w.oldest(it.len - 1) : 0;
+            const bool seen = !WINDOW || key0 + min(nvalid, 16) > oldest || key0 < p.w.keep_first;
             if (!failed && nvalid > 0 && seen) {
                 const uint32_t stage_base = smem_base + slot * kStageBytes;
                 // Row of key j (0..15 of this warp's tile) inside a half tile.  A copy of
@@ -362,7 +366,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
                 for (int e = 0; e < 8; ++e) {
                     const float v = (e < 4 ? s0[e] : s1[e - 4]) * p.scale_log2;
                     const int key = (e >> 2) * 8 + 2 * t + (e & 1);
-                    const bool sees = key < nvalid && (!WINDOW || key0 + key >= oldest || key0 + key < p.keep_first);
+                    const bool sees = key < nvalid && (!WINDOW || key0 + key >= oldest || key0 + key < p.w.keep_first);
                     x[e] = sees ? v : -INFINITY;
                 }
                 float mx0 = fmaxf(fmaxf(x[0], x[1]), fmaxf(x[4], x[5]));
@@ -433,16 +437,20 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
             for (int rr = 0; rr < 2; ++rr) {
                 const int row = g + rr * 8;
                 if (row < G) {
-                    const float l = rr ? l1 : l0;
-                    const float inv = l > 0.f ? 1.f / l : 0.f;
-                    __nv_bfloat16* dst = p.out + (static_cast<int64_t>(it.b) * Hq + h * G + row) * kD;
+                    const int head = h * G + row;
+                    float l = rr ? l1 : l0;
+                    if (WINDOW && p.w.sinks != nullptr) l += exp2f(p.w.sinks[head] * kLog2e - (rr ? m1 : m0));
+                    float inv = l > 0.f ? 1.f / l : 0.f;
+                    if (WINDOW) inv *= head_factor(p.w, it.b, head);
+                    __nv_bfloat16* dst = p.out + (WINDOW ? it.b * p.w.out_st : static_cast<int64_t>(it.b) * Hq * kD) + head * kD;
+                    const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(p.w.gate);
 #pragma unroll
                     for (int i = 0; i < 16; ++i) {
                         const float a = o[i][2 * rr] * inv, b = o[i][2 * rr + 1] * inv;
                         uint32_t packed = pack_bf16(a, b);
-                        if (WINDOW && p.gate != nullptr)
-                            packed = gate_pair(*reinterpret_cast<const uint32_t*>(p.gate + it.b * p.gate_st + (h * G + row) * kD +
-                                                                                  i * 8 + 2 * t), a, b);
+                        if (WINDOW && gate != nullptr && !p.w.gate_per_head)
+                            packed = gate_pair(*reinterpret_cast<const uint32_t*>(gate + it.b * p.w.gate_st + head * kD + i * 8 + 2 * t),
+                                               a, b);
                         *reinterpret_cast<uint32_t*>(dst + i * 8 + 2 * t) = packed;
                     }
                 }
@@ -493,7 +501,7 @@ attention_decode_merge_kernel(const DecodeParams p, int attn_grid) {
         int carry = 0, first = 0, mine = 0;
         for (int base = 0; base < p.batch; base += 32) {
             const int r = base + lane;
-            const int n = r < p.batch ? stage_range<WINDOW>(p.seq_lens[r], SK, p.window, p.keep_first).count : 0;
+            const int n = r < p.batch ? stage_range<WINDOW>(p.seq_lens[r], SK, p.w).count : 0;
             int incl = n;
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -565,16 +573,19 @@ attention_decode_merge_kernel(const DecodeParams p, int attn_grid) {
             acc.w += r.w * w;
         }
     }
-    const float inv = Lsum > 0.f ? 1.f / Lsum : 0.f;
+    if (WINDOW && p.w.sinks != nullptr) Lsum += exp2f(p.w.sinks[head] * kLog2e - M);
+    float inv = Lsum > 0.f ? 1.f / Lsum : 0.f;
+    if (WINDOW) inv *= head_factor(p.w, b, head);
     uint2 packed;
     packed.x = pack_bf16(acc.x * inv, acc.y * inv);
     packed.y = pack_bf16(acc.z * inv, acc.w * inv);
-    if (WINDOW && p.gate != nullptr) {
-        const uint2 g = *reinterpret_cast<const uint2*>(p.gate + b * p.gate_st + head * kD + lane * 4);
+    if (WINDOW && p.w.gate != nullptr && !p.w.gate_per_head) {
+        const uint2 g = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.w.gate) + b * p.w.gate_st + head * kD +
+                                                        lane * 4);
         packed.x = gate_pair(g.x, acc.x * inv, acc.y * inv);
         packed.y = gate_pair(g.y, acc.z * inv, acc.w * inv);
     }
-    *reinterpret_cast<uint2*>(p.out + (static_cast<int64_t>(b) * Hq + head) * kD + lane * 4) = packed;
+    *reinterpret_cast<uint2*>(p.out + (WINDOW ? b * p.w.out_st : static_cast<int64_t>(b) * Hq * kD) + head * kD + lane * 4) = packed;
 }
 
 }  // namespace
@@ -629,10 +640,8 @@ int launch_attention_decode(void* out, const void* q, int64_t q_st, int64_t q_sh
     p.max_items = static_cast<int>(max_items < (1 << 30) ? max_items : (1 << 30));
     p.status = status;
     p.kv_evict_first = kv_evict_first ? 1 : 0;
-    p.window = window ? window->size : 0x7fffffff;
-    p.keep_first = window ? window->keep_first : 0;
-    p.gate = window ? static_cast<const __nv_bfloat16*>(window->gate) : nullptr;
-    p.gate_st = window ? window->gate_st : 0;
+    if (window) p.w = *window;
+    if (p.w.out_st == 0) p.w.out_st = static_cast<int64_t>(q_heads) * kD;
     auto kernel = window ? attention_decode_kernel<true> : attention_decode_kernel<false>;
 
     const int smem = kStages * kStageBytes + 1024;

@@ -21,8 +21,8 @@
 // Queries are the LAST extend_len positions of the request, so tiles left of the diagonal need no mask
 // and tiles right of it are never loaded.
 //
-// WINDOW: a sliding window with kept first keys (tiles that no row of the block sees are never loaded; the
-// tiles at the window's edges are masked per element) and a sigmoid gate on the output.
+// WINDOW: everything AttentionWindow has (tiles that no row of the block sees are never loaded; the tiles at a
+// window's or a chunk's edges are masked per element).
 #include "common.cuh"
 #include "kernels.h"
 #include "tcgen05.cuh"
@@ -58,9 +58,7 @@ struct PrefillTc2Params {
     int64_t num_slots;
     float scale_log2;
     int* status;
-    int window, keep_first;     // WINDOW only
-    const __nv_bfloat16* gate;
-    int64_t gate_st;
+    AttentionWindow w;          // WINDOW only
 };
 
 // MN-major operand under the 128-byte swizzle (V as the B operand of P V: rows are keys, 64 head-dim
@@ -142,8 +140,8 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
     const int pos0 = len - ext;                   // position of query token 0
     const int kv_end = min(len, pos0 + t_end);    // keys [0, kv_end) are visible to this block
     // tiles [0, head_tiles) and, `skip` tiles further, those from the oldest key that the first row sees
-    const int head_tiles = WINDOW ? (min(p.keep_first, kv_end) + kTile - 1) / kTile : 0;
-    const int skip = WINDOW ? max(0, max(0, pos0 + t0 - p.window + 1) / kTile - head_tiles) : 0;
+    const int head_tiles = WINDOW ? (min(p.w.keep_first, kv_end) + kTile - 1) / kTile : 0;
+    const int skip = WINDOW ? max(0, p.w.oldest(pos0 + t0) / kTile - head_tiles) : 0;
     const int ntiles = (kv_end + kTile - 1) / kTile - skip;
     auto first_key = [&](int kt) { return (WINDOW && kt >= head_tiles ? kt + skip : kt) * kTile; };
 
@@ -333,8 +331,8 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
         const int tok = t0 + tile * QB + r / G;
         const int head = h * G + r % G;
         const int limit = min(pos0 + tok, len - 1);   // last visible key of this row
-        const int oldest = WINDOW ? limit - p.window + 1 : 0;   // keys before it are seen below keep_first only
-        auto sees = [&](int k) { return k <= limit && (!WINDOW || k >= oldest || k < p.keep_first); };
+        const int oldest = WINDOW ? p.w.oldest(limit) : 0;   // keys before it are seen below keep_first only
+        auto sees = [&](int k) { return k <= limit && (!WINDOW || k >= oldest || k < p.w.keep_first); };
         const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(qtr * 32) << 16);
         const uint32_t s_addr = lane_addr + kColS + static_cast<uint32_t>(tile) * 128u + static_cast<uint32_t>(half * 64);
         const uint32_t o_addr = lane_addr + kColO + static_cast<uint32_t>(tile) * 128u + static_cast<uint32_t>(half * 64);
@@ -357,7 +355,7 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
             const int k0 = first_key(kt) + half * 64;    // first key of this thread's columns
             // (masking is decided per warp, so that the common case carries no per-element tests at all)
             const bool need_mask =
-                __any_sync(0xffffffffu, k0 + 63 > limit || (WINDOW && k0 < oldest && k0 + 63 >= p.keep_first));
+                __any_sync(0xffffffffu, k0 + 63 > limit || (WINDOW && k0 < oldest && k0 + 63 >= p.w.keep_first));
             // pass 1: the maximum of this thread's 64 scores (both loads in flight before the first wait)
             float mx = -INFINITY;
             {
@@ -456,12 +454,17 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
         tc_fence_after();
         s_sum[tile][half][r] = l_run;
         pair_sync();
-        const float l_tot = l_run + s_sum[tile][half ^ 1][r];
+        float l_tot = l_run + s_sum[tile][half ^ 1][r];
+        if (WINDOW && p.w.sinks != nullptr) l_tot += ex2(fmaf(p.w.sinks[head], 1.4426950408889634f, -m_ref * sc));
         {
             // (the TMEM loads are warp-wide: every lane takes part, only the stores are per row)
             const bool store = !failed && tok < t_end;
-            const float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
-            uint4* dst = reinterpret_cast<uint4*>(p.out + (static_cast<int64_t>(q_begin + (store ? tok : 0)) * p.q_heads + head) * kD +
+            float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
+            const int64_t row = q_begin + (store ? tok : 0);
+            const __nv_bfloat16* gates = WINDOW ? static_cast<const __nv_bfloat16*>(p.w.gate) : nullptr;
+            if (WINDOW) inv *= p.w.out_scale;
+            if (WINDOW && gates != nullptr && p.w.gate_per_head) inv *= sigmoid_f(__bfloat162float(gates[row * p.w.gate_st + head]));
+            uint4* dst = reinterpret_cast<uint4*>(p.out + row * (WINDOW ? p.w.out_st : static_cast<int64_t>(p.q_heads) * kD) + head * kD +
                                                   half * 64);
 #pragma unroll
             for (int c = 0; c < 2; ++c) {
@@ -470,8 +473,8 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
                 tmem_ld_wait();
 #pragma unroll
                 for (int i = 0; i < 32; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * inv);
-                if (WINDOW && p.gate != nullptr && store) {
-                    const uint4* gate = reinterpret_cast<const uint4*>(p.gate + (q_begin + tok) * p.gate_st + head * kD + half * 64);
+                if (WINDOW && gates != nullptr && !p.w.gate_per_head && store) {
+                    const uint4* gate = reinterpret_cast<const uint4*>(gates + row * p.w.gate_st + head * kD + half * 64);
 #pragma unroll
                     for (int j = 0; j < 4; ++j) {
                         const uint4 g4 = gate[c * 4 + j];
@@ -547,10 +550,8 @@ int launch_attention_prefill_tc2(void* out, const void* q, int64_t q_st, int64_t
     p.num_slots = num_slots;
     p.scale_log2 = sm_scale * 1.4426950408889634f;
     p.status = status;
-    p.window = window ? window->size : 0x7fffffff;
-    p.keep_first = window ? window->keep_first : 0;
-    p.gate = window ? static_cast<const __nv_bfloat16*>(window->gate) : nullptr;
-    p.gate_st = window ? window->gate_st : 0;
+    if (window) p.w = *window;
+    if (p.w.out_st == 0) p.w.out_st = static_cast<int64_t>(q_heads) * kD;
     CUtensorMap tk, tv;
     int err = make_kv_tmap_3d_tc2(&tk, k_cache, num_slots, kv_heads, p.kpc);
     if (err != B200_OK) return err;

@@ -121,7 +121,7 @@ int launch_linear_heads(void* y, const void* x, const void* w, int M, int heads,
 // fp32 GEMMs of every form the layer stack uses (linear_f32.cu); see b200_linear_f32.
 int launch_linear_f32(float* y, const float* x, const float* w, int max_rows, int N, int K, int groups,
                       const int32_t* counts, const int32_t* offsets, int epilogue, cudaStream_t stream,
-                      float act_limit = 0.f);
+                      float act_limit = 0.f, const float* bias = nullptr);
 
 // fp32 residual stream: add, norm, and the gather / scatter around them (residual.cu).
 struct ResidualNorm {
@@ -153,6 +153,10 @@ struct ResidualPostNorm {
     int src_top = 1;
     int64_t src_count = 0;
     const void* src2 = nullptr;             // optional second row per token
+    // Both set: src and src2 are RMS-normalised with a weight each before they are added, and the sum is
+    // multiplied by pair_scale.
+    const void *pair_weight = nullptr, *pair_weight2 = nullptr;
+    float pair_scale = 1.f;
     bool init = false;                      // the sum replaces the residual
     const void* add_weight = nullptr;       // NULL: what is added is not normalised
     const void* out_weight = nullptr;       // NULL: out is the residual itself
@@ -191,13 +195,26 @@ int launch_score_place(void* xp, const void* x, int row_bytes, const ScoreRoute&
 
 // Latent attention (latent_attention.cu, latent_attention_tc.cu).
 // The output of the joint down-projection [tokens, qp + rp] -> RMS-normalised query latent [tokens, qp]
-// and RMS-normalised key/value latent straight into the pool.
-int launch_latent_norm_store(void* q_latent, void* cache, const void* joint, const void* q_weight,
-                             const void* kv_weight, const int32_t* out_loc, int tokens, int q_rank, int qp,
-                             int kv_rank, int rp, int64_t num_slots, float eps, int dtype, int* status,
-                             cudaStream_t stream);
+// and RMS-normalised key/value latent straight into the pool (cache NULL: the joint rows are the query latent
+// alone).  With a rotation, columns [rope_at, rope_at + rope_dim) of the key/value part are not normalised but
+// rotated in neighbouring pairs; rope_at is a multiple of 8.
+struct LatentNorm {
+    void *q_latent = nullptr, *cache = nullptr;
+    const void *joint = nullptr, *q_weight = nullptr, *kv_weight = nullptr;
+    const int32_t *out_loc = nullptr, *positions = nullptr;
+    int tokens = 0, q_rank = 0, qp = 0, kv_rank = 0, rp = 0;
+    int rope_at = 0, rope_dim = 0, max_pos = 1;
+    const float *cos_t = nullptr, *sin_t = nullptr;   // [max_pos, rope_dim / 2]
+    int64_t num_slots = 0;
+    float eps = 0.f;
+    int* status = nullptr;
+};
+int launch_latent_norm_store(const LatentNorm& a, int dtype, cudaStream_t stream);
+// The first `dims` elements of every head of x [tokens, heads, ld] rotated in place, in neighbouring pairs.
+int launch_rotate_pairs(void* x, int tokens, int heads, int ld, int dims, const float* cos_t, const float* sin_t,
+                        const int32_t* positions, int max_pos, int dtype, int* status, cudaStream_t stream);
 struct LatentAttention {
-    void* out = nullptr;              // [rows, heads, width]
+    void* out = nullptr;              // [rows, heads, out_width]
     const void* q = nullptr;          // [rows, heads, width]
     const void* cache = nullptr;      // [num_slots, width]
     int64_t num_slots = 0;
@@ -206,6 +223,7 @@ struct LatentAttention {
     const int32_t* row_table = nullptr;   // page-table row of every query row
     const int32_t* row_len = nullptr;     // keys it sees
     int rows = 0, heads = 0, width = 0, page_size = 1;
+    int out_width = 0;                    // only the first columns of a latent are averaged; 0: all of them
     float scale = 1.f;
     // Only key row_len[i] - 1 of row i was written by kernels that may still be running when this one
     // starts (a decode step), and the tables and lengths are complete: the rest is read ahead of them.
@@ -259,14 +277,29 @@ bool decode_chain_supported(int tokens, int hidden, int q_heads, int kv_heads, i
                             bool has_bias);
 int launch_decode_chain(const DecodeChainArgs& args, cudaStream_t stream);
 
-// A sliding window over the keys, the first ones kept, and a gate on the output (what the paged attention
-// kernels take beside causal attention): the query at position i sees key j <= i if i - j < size or
-// j < keep_first, and head h's output element c is multiplied by sigmoid(gate[token, h * 128 + c]).
+// What the paged attention kernels take beside causal attention.
+//  - A sliding window over the keys, the first ones kept: the query at position i sees key j <= i if
+//    i - j < size or j < keep_first.  Or chunks of the sequence (chunk > 0, which replaces size): it sees j if
+//    i / chunk = j / chunk.
+//  - A sink: exp(sinks[h]) is added to the denominator of head h's softmax.
+//  - A gate on the output: head h's element c is multiplied by sigmoid(gate[token, h * vdim + c]), or the whole
+//    head by sigmoid(gate[token, h]).
+//  - A constant factor on the output, whose rows may be part of wider ones.
 struct AttentionWindow {
     int size = 0x7fffffff;
     int keep_first = 0;
-    const void* gate = nullptr;   // bf16; NULL: no gate
-    int64_t gate_st = 0;          // its token stride in elements
+    int chunk = 0;
+    const float* sinks = nullptr;   // [heads]; NULL: none
+    const void* gate = nullptr;     // of the attention's dtype; NULL: no gate
+    int64_t gate_st = 0;            // its token stride in elements
+    bool gate_per_head = false;
+    float out_scale = 1.f;
+    int64_t out_st = 0;             // token stride of the output; 0: its rows are dense
+    // the oldest key in the window of the query at position `pos` (kept ones aside)
+    __host__ __device__ int oldest(int pos) const {
+        const int o = chunk > 0 ? pos / chunk * chunk : pos - size + 1;
+        return o > 0 ? o : 0;
+    }
 };
 
 int64_t decode_workspace_bytes(int max_batch, int q_heads, int kv_heads);
@@ -320,6 +353,16 @@ struct WindowAttention {
 };
 bool window_attention_tc_supported(const WindowAttention& a, int dtype);
 int launch_window_attention(const WindowAttention& a, int dtype, cudaStream_t stream);
+// Recurrences with one decay per head (recurrence.cu); see b200_recurrence.
+using Recurrence = b200_recurrence_args;
+// Bytes of a step's scratch arrays.
+struct RecurrenceScratch {
+    int64_t mixed, steps, units, chunks;
+};
+RecurrenceScratch recurrence_scratch(int rule, int max_tokens, int max_batch, int heads, int kv_heads, int padded_dim,
+                                     int padded_value_dim, int dtype);
+bool recurrence_supported(int padded_value_dim, int padded_dim, int taps);
+int launch_recurrence(const Recurrence& a, int dtype, cudaStream_t stream);
 // Gated linear attention (linear_attention.cu): the recurrence, its norm and its gate; see
 // b200_linear_attention.
 using LinearAttention = b200_linear_attention_args;

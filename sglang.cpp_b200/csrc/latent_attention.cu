@@ -25,27 +25,27 @@ __device__ __forceinline__ void put(float* p, float v) { *p = v; }
 __device__ __forceinline__ void put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 
 // Columns [0, qp) of a token's joint row are its query latent, [qp, qp + rp) its key/value latent; each is
-// divided by its own root mean square (over the true widths) and scaled by its own weight.  One warp per
-// latent: warps 0 and 1 of a pair take the two latents of one token, four tokens per CTA, the row in
-// registers (latents of up to 8 x 256 elements; wider ones are read again).
+// divided by its own root mean square (over the true widths) and scaled by its own weight, but for the part of
+// the key/value latent that turns with the position instead.  One warp per latent: warps 0 and 1 of a pair take
+// the two latents of one token, four tokens per CTA, the row in registers (latents of up to 8 x 256 elements;
+// wider ones are read again).
 template <typename T>
 __global__ void __launch_bounds__(256)
-latent_norm_store_kernel(T* __restrict__ q_latent, T* __restrict__ cache, const T* __restrict__ joint,
-                         const T* __restrict__ q_weight, const T* __restrict__ kv_weight,
-                         const int32_t* __restrict__ out_loc, int tokens, int q_rank, int qp, int kv_rank, int rp,
-                         int64_t num_slots, float eps, int* status) {
+latent_norm_store_kernel(const LatentNorm a) {
     constexpr int kKeep = 8;
     pdl_launch_dependents();
     pdl_wait_prior();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int64_t t = static_cast<int64_t>(blockIdx.x) * (blockDim.x >> 6) + (warp >> 1);
-    if (t >= tokens) return;
+    if (t >= a.tokens) return;
     const bool kv = (warp & 1) != 0;
-    const T* src = joint + t * (qp + rp) + (kv ? qp : 0);
-    const T* weight = kv ? kv_weight : q_weight;
-    const int nvec = (kv ? rp : qp) >> 3;
+    if (kv && a.cache == nullptr) return;
+    const T* src = static_cast<const T*>(a.joint) + t * (a.qp + a.rp) + (kv ? a.qp : 0);
+    const T* weight = static_cast<const T*>(kv ? a.kv_weight : a.q_weight);
+    const int nvec = (kv ? a.rp : a.qp) >> 3;
+    const int rope0 = kv && a.rope_dim > 0 ? a.rope_at >> 3 : nvec;   // the first vector that turns
     int64_t slot = 0;
-    if (kv) slot = out_loc[t];
+    if (kv) slot = a.out_loc[t];
     Vec8 x[kKeep];
     float ss = 0.f;
 #pragma unroll
@@ -54,34 +54,84 @@ latent_norm_store_kernel(T* __restrict__ q_latent, T* __restrict__ cache, const 
         if (v < nvec) {
             x[i] = load8(src + v * 8);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) ss += x[i].v[j] * x[i].v[j];
+            for (int j = 0; j < 8; ++j) ss += v < rope0 ? x[i].v[j] * x[i].v[j] : 0.f;
         }
     }
-    for (int v = lane + kKeep * 32; v < nvec; v += 32) {
+    for (int v = lane + kKeep * 32; v < rope0; v += 32) {
         const Vec8 y = load8(src + v * 8);
 #pragma unroll
         for (int j = 0; j < 8; ++j) ss += y.v[j] * y.v[j];
     }
-    const float r = rsqrtf(warp_sum(ss) / static_cast<float>(kv ? kv_rank : q_rank) + eps);
-    T* dst = q_latent + t * qp;
+    const float r = rsqrtf(warp_sum(ss) / static_cast<float>(kv ? a.kv_rank : a.q_rank) + a.eps);
+    T* dst = static_cast<T*>(a.q_latent) + t * a.qp;
     if (kv) {
-        if (slot < 0 || slot >= num_slots) {
-            if (lane == 0) atomicExch(&status[kStatusBadIndex], static_cast<int>(slot) + 1);
+        if (slot < 0 || slot >= a.num_slots) {
+            if (lane == 0) atomicExch(&a.status[kStatusBadIndex], static_cast<int>(slot) + 1);
             return;
         }
-        dst = cache + slot * rp;
+        dst = static_cast<T*>(a.cache) + slot * a.rp;
+    }
+    int pos = 0;
+    if (kv && a.rope_dim > 0) {
+        pos = a.positions[t];
+        if (pos < 0 || pos >= a.max_pos) {
+            if (lane == 0) atomicExch(&a.status[kStatusBadIndex], pos + 1);
+            pos = min(max(pos, 0), a.max_pos - 1);
+        }
     }
     auto emit = [&](int v, const Vec8& y) {
-        const Vec8 g = load8(weight + v * 8);
         Vec8 o;
+        if (v < rope0) {
+            const Vec8 g = load8(weight + v * 8);
 #pragma unroll
-        for (int j = 0; j < 8; ++j) o.v[j] = y.v[j] * r * g.v[j];
+            for (int j = 0; j < 8; ++j) o.v[j] = y.v[j] * r * g.v[j];
+        } else {
+            const int half = a.rope_dim >> 1;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int pair = (v - rope0) * 4 + j;
+                const float c = pair < half ? a.cos_t[static_cast<int64_t>(pos) * half + pair] : 0.f;
+                const float s = pair < half ? a.sin_t[static_cast<int64_t>(pos) * half + pair] : 0.f;
+                o.v[2 * j] = y.v[2 * j] * c - y.v[2 * j + 1] * s;
+                o.v[2 * j + 1] = y.v[2 * j + 1] * c + y.v[2 * j] * s;
+            }
+        }
         store8(dst + v * 8, o);
     };
 #pragma unroll
     for (int i = 0; i < kKeep; ++i)
         if (lane + i * 32 < nvec) emit(lane + i * 32, x[i]);
     for (int v = lane + kKeep * 32; v < nvec; v += 32) emit(v, load8(src + v * 8));
+}
+
+// One thread per 8 elements of a head's rotated part.
+template <typename T>
+__global__ void __launch_bounds__(256)
+rotate_pairs_kernel(T* __restrict__ x, int64_t count, int vecs, int heads, int ld, int dims, const float* __restrict__ cos_t,
+                    const float* __restrict__ sin_t, const int32_t* __restrict__ positions, int max_pos, int* status) {
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+    if (i >= count) return;
+    const int64_t row = i / vecs;
+    const int v = static_cast<int>(i - row * vecs), half = dims >> 1;
+    int pos = positions[row / heads];
+    if (pos < 0 || pos >= max_pos) {
+        atomicExch(&status[kStatusBadIndex], pos + 1);
+        pos = min(max(pos, 0), max_pos - 1);
+    }
+    T* p = x + row * ld + v * 8;
+    Vec8 y = load8(p);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const int pair = v * 4 + j;
+        if (pair >= half) break;
+        const float c = cos_t[static_cast<int64_t>(pos) * half + pair], s = sin_t[static_cast<int64_t>(pos) * half + pair];
+        const float a = y.v[2 * j], b = y.v[2 * j + 1];
+        y.v[2 * j] = a * c - b * s;
+        y.v[2 * j + 1] = b * c + a * s;
+    }
+    store8(p, y);
 }
 
 // One CTA per (query row, head); its warps take every fourth key each with an online softmax whose
@@ -91,7 +141,7 @@ __global__ void __launch_bounds__(128)
 latent_attention_plain_kernel(T* __restrict__ out, const T* __restrict__ q, const T* __restrict__ cache,
                               int64_t num_slots, const int32_t* __restrict__ page_table, int64_t pt_stride,
                               const int32_t* __restrict__ row_table, const int32_t* __restrict__ row_len, int heads,
-                              int width, float scale, int* status) {
+                              int width, int out_width, float scale, int* status) {
     extern __shared__ float smem[];   // q [width], then o [4][width]
     __shared__ float s_m[4], s_l[4];
     pdl_launch_dependents();
@@ -103,7 +153,7 @@ latent_attention_plain_kernel(T* __restrict__ out, const T* __restrict__ q, cons
     float* so = smem + (1 + warp) * width;
     const T* qr = q + (row * heads + h) * width;
     for (int i = threadIdx.x; i < width; i += blockDim.x) sq[i] = as_float(qr[i]);
-    for (int i = lane; i < width; i += 32) so[i] = 0.f;
+    for (int i = lane; i < out_width; i += 32) so[i] = 0.f;
     __syncthreads();
     const int32_t* pt = page_table + static_cast<int64_t>(row_table[row]) * pt_stride;
     const int len = row_len[row];
@@ -122,7 +172,7 @@ latent_attention_plain_kernel(T* __restrict__ out, const T* __restrict__ q, cons
         const float alpha = expf(m - m_new), p = expf(s - m_new);
         l = l * alpha + p;
         m = m_new;
-        for (int i = lane; i < width; i += 32) so[i] = so[i] * alpha + p * as_float(c[i]);
+        for (int i = lane; i < out_width; i += 32) so[i] = so[i] * alpha + p * as_float(c[i]);
     }
     if (lane == 0) {
         s_m[warp] = m;
@@ -138,11 +188,11 @@ latent_attention_plain_kernel(T* __restrict__ out, const T* __restrict__ q, cons
         tot += f[w] * s_l[w];
     }
     const float inv = tot > 0.f ? 1.f / tot : 0.f;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    for (int i = threadIdx.x; i < out_width; i += blockDim.x) {
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < 4; ++w) v += f[w] * smem[(1 + w) * width + i];
-        put(out + (row * heads + h) * width + i, v * inv);
+        put(out + (row * heads + h) * out_width + i, v * inv);
     }
 }
 
@@ -186,28 +236,29 @@ move_rows_kernel(uint4* __restrict__ out, const uint4* __restrict__ in, const in
 
 }  // namespace
 
-int launch_latent_norm_store(void* q_latent, void* cache, const void* joint, const void* q_weight,
-                             const void* kv_weight, const int32_t* out_loc, int tokens, int q_rank, int qp,
-                             int kv_rank, int rp, int64_t num_slots, float eps, int dtype, int* status,
-                             cudaStream_t stream) {
-    if (tokens == 0) return B200_OK;
+int launch_latent_norm_store(const LatentNorm& a, int dtype, cudaStream_t stream) {
+    if (a.tokens == 0) return B200_OK;
     // few tokens: a CTA each, for latency; many: four per CTA
-    const int threads = tokens <= 2 * sm_count() ? 64 : 256;
-    const int grid = div_ceil(tokens, threads / 64);
-    if (dtype == B200_DTYPE_F32) {
-        B200_CHECK_CUDA(launch_kernel(latent_norm_store_kernel<float>, dim3(grid), dim3(threads), 0, stream, dim3(1, 1, 1),
-                                      static_cast<float*>(q_latent), static_cast<float*>(cache),
-                                      static_cast<const float*>(joint), static_cast<const float*>(q_weight),
-                                      static_cast<const float*>(kv_weight), out_loc, tokens, q_rank, qp, kv_rank, rp, num_slots,
-                                      eps, status));
-    } else {
-        using B = __nv_bfloat16;
-        B200_CHECK_CUDA(launch_kernel(latent_norm_store_kernel<B>, dim3(grid), dim3(threads), 0, stream, dim3(1, 1, 1),
-                                      static_cast<B*>(q_latent), static_cast<B*>(cache), static_cast<const B*>(joint),
-                                      static_cast<const B*>(q_weight), static_cast<const B*>(kv_weight), out_loc, tokens, q_rank,
-                                      qp, kv_rank, rp, num_slots, eps, status));
-    }
+    const int threads = a.tokens <= 2 * sm_count() ? 64 : 256;
+    const int grid = div_ceil(a.tokens, threads / 64);
+    auto kernel = dtype == B200_DTYPE_F32 ? latent_norm_store_kernel<float> : latent_norm_store_kernel<__nv_bfloat16>;
+    B200_CHECK_CUDA(launch_kernel(kernel, dim3(grid), dim3(threads), 0, stream, dim3(1, 1, 1), a));
     return B200_OK;
+}
+
+int launch_rotate_pairs(void* x, int tokens, int heads, int ld, int dims, const float* cos_t, const float* sin_t,
+                        const int32_t* positions, int max_pos, int dtype, int* status, cudaStream_t stream) {
+    if (tokens == 0 || dims == 0) return B200_OK;
+    const int vecs = div_ceil(dims, 8);
+    const int64_t count = static_cast<int64_t>(tokens) * heads * vecs;
+    const dim3 grid(static_cast<unsigned>(div_ceil64(count, 256)));
+    auto run = [&](auto* p) -> int {
+        using T = typename std::remove_pointer<decltype(p)>::type;
+        B200_CHECK_CUDA(launch_kernel(rotate_pairs_kernel<T>, grid, dim3(256), 0, stream, dim3(1, 1, 1), p, count, vecs, heads,
+                                      ld, dims, cos_t, sin_t, positions, max_pos, status));
+        return B200_OK;
+    };
+    return dtype == B200_DTYPE_F32 ? run(static_cast<float*>(x)) : run(static_cast<__nv_bfloat16*>(x));
 }
 
 int launch_latent_attention_plain(const LatentAttention& a, int dtype, int* status, cudaStream_t stream) {
@@ -224,7 +275,8 @@ int launch_latent_attention_plain(const LatentAttention& a, int dtype, int* stat
         B200_CHECK_CUDA(launch_kernel(kernel, dim3(a.rows, a.heads), dim3(128), smem, stream, dim3(1, 1, 1),
                                       static_cast<T*>(a.out), static_cast<const T*>(a.q),
                                       static_cast<const T*>(a.cache), a.num_slots, a.page_table, a.pt_stride,
-                                      a.row_table, a.row_len, a.heads, a.width, a.scale, status));
+                                      a.row_table, a.row_len, a.heads, a.width, a.out_width > 0 ? a.out_width : a.width, a.scale,
+                                      status));
         return B200_OK;
     };
     return dtype == B200_DTYPE_F32 ? run(static_cast<float*>(nullptr)) : run(static_cast<__nv_bfloat16*>(nullptr));
@@ -265,6 +317,15 @@ int b200_latent_attention(void* out, const void* q, const void* cache, int64_t n
                           int64_t page_table_stride, const int32_t* row_table, const int32_t* row_len, int rows,
                           int heads, int width, int page_size, float scale, int dtype, int plain, void* workspace,
                           int64_t workspace_bytes, b200_stream_t stream) {
+    return b200_latent_attention_part(out, q, cache, num_slots, page_table, page_table_stride, row_table, row_len, rows, heads,
+                                      width, width, page_size, scale, dtype, plain, workspace, workspace_bytes, stream);
+}
+
+int b200_latent_attention_part(void* out, const void* q, const void* cache, int64_t num_slots, const int32_t* page_table,
+                               int64_t page_table_stride, const int32_t* row_table, const int32_t* row_len, int rows,
+                               int heads, int width, int out_width, int page_size, float scale, int dtype, int plain,
+                               void* workspace, int64_t workspace_bytes, b200_stream_t stream) {
+    B200_CHECK_ARG(out_width > 0 && out_width <= width && out_width % 128 == 0, "latent_attention: bad output width");
     B200_CHECK_ARG(rows >= 0 && heads > 0 && width > 0 && width % 128 == 0 && num_slots > 0,
                    "latent_attention: bad shape");
     B200_CHECK_ARG(page_size >= 1 && (page_size & (page_size - 1)) == 0, "latent_attention: page_size must be a power of two");
@@ -286,6 +347,7 @@ int b200_latent_attention(void* out, const void* q, const void* cache, int64_t n
     a.rows = rows;
     a.heads = heads;
     a.width = width;
+    a.out_width = out_width;
     a.page_size = page_size;
     a.scale = scale;
     a.workspace = workspace;
@@ -297,6 +359,20 @@ int b200_latent_attention(void* out, const void* q, const void* cache, int64_t n
         return b200::launch_latent_attention_tc(a, status, s);
     }
     return b200::launch_latent_attention_plain(a, dtype, status, s);
+}
+
+int b200_rotate_pairs(void* x, int tokens, int heads, int ld, int dims, const float* cos_table, const float* sin_table,
+                      const int32_t* positions, int max_pos, int dtype, b200_stream_t stream) {
+    B200_CHECK_ARG(tokens >= 0 && heads > 0 && ld > 0 && ld % 8 == 0 && dims >= 0 && dims % 2 == 0 && dims <= ld && max_pos > 0,
+                   "rotate_pairs: bad shape");
+    B200_CHECK_ARG(dtype == B200_DTYPE_BF16 || dtype == B200_DTYPE_F32, "rotate_pairs: unknown dtype");
+    if (tokens == 0 || dims == 0) return B200_OK;
+    B200_CHECK_ARG(x && cos_table && sin_table && positions, "rotate_pairs: NULL tensor");
+    int err = B200_OK;
+    int* status = b200::device_status_words(&err);
+    if (err != B200_OK) return err;
+    return b200::launch_rotate_pairs(x, tokens, heads, ld, dims, cos_table, sin_table, positions, max_pos, dtype, status,
+                                     static_cast<cudaStream_t>(stream));
 }
 
 }  // extern "C"

@@ -5,7 +5,8 @@
 // the 128 rows of the MMA:
 //     S^T = C Q^T      KT keys x N heads, K = latent width: A is the latent tile as TMA delivers it
 //     O^T += C^T P^T   128 latent elements x N heads, K = KT keys: A is the SAME tile read MN-major, so it
-//                      is fetched from HBM once and never moved again
+//                      is fetched from HBM once and never moved again (columns from out_width on, which only
+//                      take part in the scores, are left out)
 // with N = 16, 32 or 64 heads per block (more heads run as further blocks of the same row) and S^T, O^T
 // accumulating in TMEM.
 //
@@ -38,14 +39,14 @@ namespace {
 constexpr int kUnitElems = 128;                            // latent elements per unit
 constexpr int kMaxUnits = 12;                              // units in the ring
 constexpr int kThreads = 224;
-constexpr int kMaxWidth = 512;
+constexpr int kMaxWidth = 640, kMaxOutWidth = 512;
 constexpr uint32_t kColO = 0, kColS = 256;                 // TMEM columns: O^T (4 x 64), S^T (2 x 64)
 constexpr float kLazyLog2 = 8.0f;
 constexpr int kLens = 64;
 
 struct LatentParams {
-    __nv_bfloat16* out;         // [rows, heads, width]
-    float* part_o;              // [2 * grid][N][width] un-normalised
+    __nv_bfloat16* out;         // [rows, heads, out_width]
+    float* part_o;              // [2 * grid][N][out_width] un-normalised
     float* part_m;              // [2 * grid][N]
     float* part_l;
     int32_t* item_cta;          // [2 * items]: first and last CTA of an item
@@ -53,9 +54,9 @@ struct LatentParams {
     int64_t pt_stride;
     const int32_t* row_table;
     const int32_t* row_len;
-    int rows, heads, width;
+    int rows, heads, width, out_width;
     int blocks, per_block;      // head blocks per row, heads per block (<= N)
-    int nb;                     // units per tile
+    int nb, no;                 // units per tile, and those of them that are averaged
     int ring;                   // units in the ring (>= nb)
     int p_bufs;                 // buffers of P, 1 or 2
     int kpc;                    // keys per TMA copy
@@ -413,6 +414,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                             tc_mma_bf16(d, a + ((ks >> 2) * kAtomBytes + (ks & 3) * 32) / 16,
                                         b + ((ks >> 2) * N * 128 + (ks & 3) * 32) / 16, idesc, (u > 0 || ks > 0) ? 1u : 0u);
                         b += 2 * N * 128 / 16;
+                        if (u >= p.no) tc_commit(smem_u32(&unit_empty[slot]));   // nobody else reads it
                         if (++slot == p.ring) {
                             slot = 0;
                             parity ^= 1u;
@@ -444,7 +446,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                     const uint32_t pb = p_base + (p.p_bufs == 2 ? static_cast<uint32_t>(tiles & 1) * kPBytes : 0u);
                     const uint64_t b = kHeadsContiguous ? mnmajor_desc<KT>(pb) : kmajor_sw128_desc(pb);
                     uint32_t d = tmem_base + kColO;
-                    for (int u = 0; u < p.nb; ++u, d += N) {
+                    for (int u = 0; u < p.no; ++u, d += N) {
                         const uint64_t a = mnmajor_desc<KT>(smem_base + static_cast<uint32_t>(slot) * kUnitBytes);
 #pragma unroll
                         for (int ks = 0; ks < KT / 16; ++ks)
@@ -454,6 +456,8 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                         tc_commit(smem_u32(&unit_empty[slot]));
                         if (++slot == p.ring) slot = 0;
                     }
+                    slot += p.nb - p.no;
+                    if (slot >= p.ring) slot -= p.ring;
                     tc_commit(smem_u32(&pv_done[tiles & 1]));
                 }
                 ++nseg;
@@ -544,7 +548,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                         tc_fence_after();
 #pragma unroll
                         for (int h = 0; h < N; ++h) l[h] *= s_alpha[h];
-                        for (int u = 0; u < p.nb; ++u)
+                        for (int u = 0; u < p.no; ++u)
 #pragma unroll
                             for (int c = 0; c < N / 16; ++c) {
                                 const uint32_t o_addr = lane_addr + kColO + static_cast<uint32_t>(u * N + c * 16);
@@ -645,7 +649,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
             softmax_sync();
             const int h0 = seg.block * p.per_block;
             const int nh = min(p.per_block, p.heads - h0);
-            for (int u = 0; u < p.nb; ++u) {
+            for (int u = 0; u < p.no; ++u) {
 #pragma unroll
                 for (int c = 0; c < N / 16; ++c) {
                     if (c * 16 >= nh) break;
@@ -663,7 +667,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                             if (h < nh) {
                                 const float* v = stage + (i / (kUnitElems / 8)) * kUnitElems + e;
                                 const float4 a = *reinterpret_cast<const float4*>(v), b = *reinterpret_cast<const float4*>(v + 4);
-                                *reinterpret_cast<uint4*>(p.out + (static_cast<int64_t>(seg.row) * p.heads + h0 + h) * p.width +
+                                *reinterpret_cast<uint4*>(p.out + (static_cast<int64_t>(seg.row) * p.heads + h0 + h) * p.out_width +
                                                           u * kUnitElems + e) =
                                     make_uint4(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w), pack_bf16(b.x, b.y), pack_bf16(b.z, b.w));
                             }
@@ -673,7 +677,7 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_c, const __g
                         for (int i = st; i < 16 * kUnitElems / 4; i += 128) {
                             const int h = c * 16 + i / (kUnitElems / 4), e = i % (kUnitElems / 4) * 4;
                             if (h < nh)
-                                *reinterpret_cast<float4*>(p.part_o + (slot * N + h) * p.width + u * kUnitElems + e) =
+                                *reinterpret_cast<float4*>(p.part_o + (slot * N + h) * p.out_width + u * kUnitElems + e) =
                                     *reinterpret_cast<const float4*>(stage + (i / (kUnitElems / 4)) * kUnitElems + e);
                         }
                     }
@@ -699,9 +703,9 @@ latent_merge_kernel(const LatentParams p, int N) {
     const int row = blockIdx.x / p.heads, head = blockIdx.x - row * p.heads;
     const int block = head / p.per_block, h = head - block * p.per_block;
     const int item = row * p.blocks + block;
-    __nv_bfloat16* out = p.out + (static_cast<int64_t>(row) * p.heads + head) * p.width;
+    __nv_bfloat16* out = p.out + (static_cast<int64_t>(row) * p.heads + head) * p.out_width;
     if (p.row_len[row] <= 0) {   // no keys: zeros
-        for (int i = threadIdx.x; i < p.width; i += blockDim.x) out[i] = __float2bfloat16_rn(0.f);
+        for (int i = threadIdx.x; i < p.out_width; i += blockDim.x) out[i] = __float2bfloat16_rn(0.f);
         return;
     }
     const int c0 = p.item_cta[2 * item], c1 = p.item_cta[2 * item + 1];
@@ -717,8 +721,8 @@ latent_merge_kernel(const LatentParams p, int N) {
         const int64_t s = slot_of(c);
         const float f = ex2(p.part_m[s] - mx);
         tot += f * p.part_l[s];
-        if (e < p.width) {
-            const float4 v = *reinterpret_cast<const float4*>(p.part_o + s * p.width + e);
+        if (e < p.out_width) {
+            const float4 v = *reinterpret_cast<const float4*>(p.part_o + s * p.out_width + e);
             acc.x += f * v.x;
             acc.y += f * v.y;
             acc.z += f * v.z;
@@ -726,7 +730,7 @@ latent_merge_kernel(const LatentParams p, int N) {
         }
     }
     const float inv = tot > 0.f ? 1.f / tot : 0.f;
-    if (e < p.width)
+    if (e < p.out_width)
         *reinterpret_cast<uint2*>(out + e) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
 }
 
@@ -773,7 +777,8 @@ int64_t latent_attention_workspace_bytes(int rows, int heads, int width) {
 }
 
 bool latent_attention_tc_supported(const LatentAttention& a) {
-    return a.width % kUnitElems == 0 && a.width <= kMaxWidth && a.scale > 0.f && sm_count() <= 160 &&
+    const int out_width = a.out_width > 0 ? a.out_width : a.width;
+    return a.width % kUnitElems == 0 && a.width <= kMaxWidth && out_width % kUnitElems == 0 && out_width <= kMaxOutWidth && a.scale > 0.f && sm_count() <= 160 &&
            (reinterpret_cast<uintptr_t>(a.cache) & 15u) == 0 && (reinterpret_cast<uintptr_t>(a.q) & 15u) == 0;
 }
 
@@ -799,9 +804,11 @@ int launch_latent_attention_tc(const LatentAttention& a, int* status, cudaStream
     p.rows = a.rows;
     p.heads = a.heads;
     p.width = a.width;
+    p.out_width = a.out_width > 0 ? a.out_width : a.width;
     p.blocks = sh.blocks;
     p.per_block = sh.per_block;
     p.nb = a.width / kUnitElems;
+    p.no = p.out_width / kUnitElems;
     const int kt = a.width > 256 ? 64 : 128;
     p.kpc = a.page_size < kt ? a.page_size : kt;
     p.num_slots = a.num_slots;

@@ -4,7 +4,7 @@
 //
 // Per layer, on T tokens (fp32 residual stream r, everything else in the stack's dtype):
 //     x = norm(r += previous block)       the norm on the input: one kernel, residual.cu
-//     x = r += norm(previous block)       or on the output of a block; one kernel as well
+//     x = r += norm(previous block)       or on the output of a block, or both; one kernel as well
 //     y = mixer(x)
 //     x = ... once more
 //     y = feed-forward(x)
@@ -12,11 +12,17 @@
 // Mixers
 //   latent attention:  [cq | c] = x W_down, both latents in one GEMM; cq, pool[slot] = norm(cq), norm(c)
 //                      (latent_attention.cu); q = cq W_uq; o = attention in the latent space, or over expanded
-//                      keys and values; y = o W_o
+//                      keys and values; y = o W_o.  A part of the key may turn with the position instead of being
+//                      normalised; a layer may read the pool of another one
 //   window attention:  [q | k | v | gate] = x W in one GEMM; norms, rotation, value mixing and the K/V store in
 //                      one kernel; attention and its gate in the next (window_attention.cu); y = o W_o
 //   linear attention:  [q | k | v | gate | low-rank decay] = x W in one GEMM; recurrence, norm and gate
 //                      (linear_attention.cu); y = o W_o
+//   state space, delta rule:  [gate | v | k | q | steps] = x W in one GEMM; convolution, recurrence, norm and gate
+//                      (recurrence.cu); y = o W_o
+//   two of the last kinds (window attention, recurrences) side by side: one GEMM makes both rows; one output
+//                      projection over both results adds them up, or each has its own and they meet, normalised, in
+//                      the residual kernel
 // Feed-forwards: dense; experts by token id, whose placement depends on token ids only and is laid out for all
 // layers at once before the first; experts by score (router logits in fp32, routing and placement in two
 // kernels, the weighted sum in the residual kernel that follows), beside one that every token uses.
@@ -42,21 +48,35 @@ int pad_to(int n, int m) { return (n + m - 1) / m * m; }
 int pad_width(int n) { return pad_to(n, 64); }
 int pad_head_dim(int n) { return n <= 128 ? 128 : pad_to(n, 64); }
 int pad_latent(int n) { return pad_to(n, 128); }
+int latent_rope_at(int kv_rank) { return pad_to(kv_rank, 8); }   // where the rotated part of a latent row starts
+int latent_width(int kv_rank, int rope_dim) { return pad_latent(rope_dim > 0 ? latent_rope_at(kv_rank) + rope_dim : kv_rank); }
+bool is_recurrence(int mixer) { return mixer == B200_MIXER_STATE_SPACE || mixer == B200_MIXER_DELTA_RULE; }
 }  // namespace
 
 struct StackLayer {
     b200_layer_config c;
-    int qp = 0, rp = 0, dp = 0, vp = 0, ip = 0;   // padded sizes
+    int qp = 0, rp = 0, op = 0, dp = 0, vp = 0, ip = 0;   // padded sizes
+    void *norm1_out = nullptr, *norm2_out = nullptr;       // of what the blocks return, where both sides have one
     void *norm1 = nullptr, *norm2 = nullptr, *down_qkv = nullptr, *q_norm = nullptr, *kv_norm = nullptr, *uq = nullptr,
          *uk = nullptr, *uk_absorb = nullptr, *uv = nullptr, *o = nullptr, *up = nullptr, *down = nullptr;
+    // the projection that a mixer's (or both mixers') rows come from, and this mixer's columns in them
+    void *joint = nullptr, *joint_bias = nullptr;
+    int64_t joint_ld = 0, joint_at = 0;
+    // where this mixer's result goes: element offset in the result buffer, distance of its rows
+    int64_t out_at = 0, out_ld = 0;
+    StackLayer* beside = nullptr;
+    void* side_norm = nullptr;    // of this mixer's result, under B200_JOIN_NORMED
     // window attention
-    void *qkvg = nullptr, *q_head_norm = nullptr, *k_head_norm = nullptr, *k_cache = nullptr, *v_cache = nullptr;
-    float *value_mix = nullptr, *cos_t = nullptr, *sin_t = nullptr;
+    void *q_head_norm = nullptr, *k_head_norm = nullptr, *k_cache = nullptr, *v_cache = nullptr;
+    float *value_mix = nullptr, *cos_t = nullptr, *sin_t = nullptr, *sinks = nullptr;
     int mix = HeadPrepare::kPlain;
     // linear attention
-    void *qkvga = nullptr, *decay_up = nullptr, *head_norm = nullptr;
+    void *decay_up = nullptr, *head_norm = nullptr;
     float *decay_bias = nullptr, *state = nullptr;
     int up_ld = 0;
+    // recurrences
+    float *conv = nullptr, *conv_bias = nullptr, *decay_log = nullptr, *step_bias = nullptr, *skip = nullptr;
+    void* conv_state = nullptr;
     // scored experts
     void *router = nullptr, *shared_up = nullptr, *shared_down = nullptr;
     int isp = 0;
@@ -67,12 +87,17 @@ struct StackLayer {
 };
 
 struct LayerStack {
-    std::vector<StackLayer> layers;
+    std::vector<StackLayer> layers, besides;
+    struct RopeTable {
+        b200_layer_config c;
+        float *cos_t, *sin_t;
+    };
+    std::vector<RopeTable> ropes;
     int dtype = B200_DTYPE_BF16;
     int esz = 2;            // bytes per element
     int hp = 0, vocab_p = 0;
     float norm_offset = 0.f, logit_scale = 1.f;
-    bool norm_output = false;
+    bool norm_input = true, norm_output = false;
     void *embed = nullptr, *head = nullptr, *final_norm = nullptr;
     float* residual = nullptr;
     void *x = nullptr, *joint = nullptr, *cq = nullptr, *q = nullptr, *attn = nullptr, *y = nullptr, *h = nullptr,
@@ -97,6 +122,10 @@ struct LayerStack {
     int max_extend = 0;        // longest extension of the current step
     // window attention
     void* first_values = nullptr;
+    // recurrences
+    void *mixed = nullptr, *chunks = nullptr;
+    float *steps = nullptr, *units = nullptr;
+    void* y2 = nullptr;        // the right one of two results under B200_JOIN_NORMED
     // scored experts: the routing of the layer that is running
     float *router_logits = nullptr, *route_weights = nullptr;
     int32_t *route_ids = nullptr, *route_rows = nullptr, *route_counts = nullptr, *route_offsets = nullptr;
@@ -137,25 +166,47 @@ __global__ void compact_rows_kernel(int32_t* __restrict__ row, int32_t* __restri
     len[i] = token_len[tokens[i]];
 }
 
-int check_layer(const b200_layer_config& c, int l) {
+// A rotation whose frequencies may be stretched.
+bool rope_ok(const b200_layer_config& c, int widest) {
+    return c.rotary_dim >= 0 && c.rotary_dim % 2 == 0 && c.rotary_dim <= widest && (c.rotary_dim == 0 || c.rope_base > 0.0) &&
+           (c.rope_factor == 0.0 || (c.rope_factor > 0.0 && c.rope_low > 0.0 && c.rope_high > c.rope_low && c.rope_original > 0.0));
+}
+bool same_rope(const b200_layer_config& a, const b200_layer_config& b) {
+    if (a.rotary_dim != b.rotary_dim || a.rope_base != b.rope_base || a.rope_factor != b.rope_factor) return false;
+    return a.rope_factor == 0.0 || (a.rope_low == b.rope_low && a.rope_high == b.rope_high && a.rope_original == b.rope_original);
+}
+
+int check_mixer(const b200_layer_config& c, int l) {
     B200_CHECK_ARG(c.heads > 0 && c.heads <= 65535 && c.head_dim > 0 && c.value_dim > 0,
                    "layer %d: head count and sizes must be positive", l);
     if (c.mixer == B200_MIXER_LATENT_ATTENTION) {
         B200_CHECK_ARG(c.q_rank > 0 && c.kv_rank > 0, "layer %d: latent attention needs positive ranks", l);
+        B200_CHECK_ARG(rope_ok(c, c.head_dim), "layer %d: bad rotation", l);
     } else if (c.mixer == B200_MIXER_WINDOW_ATTENTION) {
         B200_CHECK_ARG(c.kv_heads > 0 && c.heads % c.kv_heads == 0, "layer %d: %d heads over %d key/value heads", l, c.heads,
                        c.kv_heads);
-        B200_CHECK_ARG(c.window > 0 && c.keep_first >= 0, "layer %d: bad window", l);
-        B200_CHECK_ARG(c.rotary_dim >= 0 && c.rotary_dim % 2 == 0 && c.rotary_dim <= c.head_dim &&
-                           (c.rotary_dim == 0 || c.rope_base > 0.0), "layer %d: bad rotation", l);
+        B200_CHECK_ARG(c.window > 0 && c.keep_first >= 0 && c.chunk >= 0, "layer %d: bad window", l);
+        B200_CHECK_ARG(c.gate >= B200_GATE_NONE && c.gate <= B200_GATE_HEAD, "layer %d: unknown gate", l);
+        B200_CHECK_ARG(rope_ok(c, c.head_dim), "layer %d: bad rotation", l);
         B200_CHECK_ARG(c.value_dim <= 1024 && c.head_dim <= 2048, "layer %d: heads are too wide", l);
     } else if (c.mixer == B200_MIXER_LINEAR_ATTENTION) {
         B200_CHECK_ARG(c.decay_rank > 0 && c.decay_tau > 0.f, "layer %d: bad decay", l);
         B200_CHECK_ARG(linear_attention_supported(pad_width(c.value_dim), pad_width(c.head_dim)),
                        "layer %d: heads are too wide", l);
+    } else if (is_recurrence(c.mixer)) {
+        B200_CHECK_ARG(c.kv_heads > 0 && c.heads % c.kv_heads == 0, "layer %d: %d heads over %d key heads", l, c.heads, c.kv_heads);
+        B200_CHECK_ARG(recurrence_supported(pad_width(c.value_dim), pad_width(c.head_dim), c.conv_taps),
+                       "layer %d: heads or convolution too wide", l);
+        B200_CHECK_ARG(c.mixer == B200_MIXER_DELTA_RULE || (c.norm_groups > 0 && c.heads * c.value_dim % c.norm_groups == 0),
+                       "layer %d: bad norm groups", l);
     } else {
         B200_CHECK_ARG(false, "layer %d: unknown mixer %d", l, c.mixer);
     }
+    return B200_OK;
+}
+
+int check_layer(const b200_layer_config& c, int l) {
+    S_TRY(check_mixer(c, l));
     B200_CHECK_ARG(c.mlp >= B200_MLP_NONE && c.mlp <= B200_MLP_SCORED_MOE, "layer %d: unknown feed-forward %d", l, c.mlp);
     if (c.mlp == B200_MLP_NONE) return B200_OK;
     B200_CHECK_ARG(c.intermediate > 0, "layer %d: feed-forward size must be positive", l);
@@ -175,26 +226,78 @@ int check_layer(const b200_layer_config& c, int l) {
 // Sizes of the activation buffers: the widest of any layer, in elements per token (workspaces: bytes).
 struct Widths {
     int64_t joint = 0, cq = 0, q = 0, attn = 0, h = 0, pairs = 0, latent = 0, xk = 0, xv = 0, xc = 0, ws = 0, first = 0,
-            experts = 0, router = 0, top = 0, shared = 0;
+            experts = 0, router = 0, top = 0, shared = 0, mixed = 0, steps = 0, units = 0, chunks = 0;
+    bool normed_pair = false;
     bool scored = false, any_expand = false;
     static void widest(int64_t& a, int64_t b) { if (b > a) a = b; }
 };
 
-int alloc_latent(b200_engine* e, StackLayer& L, const std::string& sfx, Widths& w) {
+// cos / sin of position * frequency, computed in double on the host; layers with the same rotation share a table.
+int rope_table(b200_engine* e, StackLayer& L) {
+    LayerStack* S = e->stack;
+    const b200_layer_config& c = L.c;
+    for (const LayerStack::RopeTable& t : S->ropes)
+        if (same_rope(t.c, c)) {
+            L.cos_t = t.cos_t;
+            L.sin_t = t.sin_t;
+            return B200_OK;
+        }
+    constexpr double kTwoPi = 6.283185307179586476925286766559;
+    const int half = c.rotary_dim / 2;
+    const int64_t n = static_cast<int64_t>(e->pt_cols) * half;
+    std::vector<float> cs(n), sn(n);
+    for (int i = 0; i < half; ++i) {
+        double f = pow(c.rope_base, -2.0 * i / c.rotary_dim);
+        if (c.rope_factor > 0.0) {
+            const double wave = kTwoPi / f;
+            const double s = (c.rope_original / wave - c.rope_low) / (c.rope_high - c.rope_low);
+            if (wave > c.rope_original / c.rope_low)
+                f /= c.rope_factor;
+            else if (wave >= c.rope_original / c.rope_high)
+                f = (1.0 - s) * f / c.rope_factor + s * f;
+        }
+        for (int64_t p = 0; p < e->pt_cols; ++p) {
+            cs[p * half + i] = static_cast<float>(cos(static_cast<double>(p) * f));
+            sn[p * half + i] = static_cast<float>(sin(static_cast<double>(p) * f));
+        }
+    }
+    void* p = nullptr;
+    S_TRY(dev_alloc(e, &p, n * 4, true));
+    L.cos_t = static_cast<float*>(p);
+    S_TRY(dev_alloc(e, &p, n * 4, true));
+    L.sin_t = static_cast<float*>(p);
+    S->ropes.push_back({c, L.cos_t, L.sin_t});
+    if (n == 0) return B200_OK;
+    B200_CHECK_CUDA(cudaMemcpy(L.cos_t, cs.data(), n * 4, cudaMemcpyHostToDevice));
+    B200_CHECK_CUDA(cudaMemcpy(L.sin_t, sn.data(), n * 4, cudaMemcpyHostToDevice));
+    return B200_OK;
+}
+
+int alloc_latent(b200_engine* e, StackLayer& L, int l, const std::string& sfx, Widths& w) {
     LayerStack* S = e->stack;
     const b200_layer_config& c = L.c;
     L.qp = pad_width(c.q_rank);
-    L.rp = pad_latent(c.kv_rank);
+    L.rp = latent_width(c.kv_rank, c.rotary_dim);
+    L.op = pad_latent(c.kv_rank);
     L.dp = pad_head_dim(c.head_dim);
     L.vp = pad_head_dim(c.value_dim);
-    const int64_t hp = S->hp, z = S->esz, H = c.heads, qp = L.qp, rp = L.rp, dp = L.dp, vp = L.vp;
-    S_TRY(named_bytes(e, &L.down_qkv, "down_qkv" + sfx, (qp + rp) * hp * z));
+    const int64_t hp = S->hp, z = S->esz, H = c.heads, qp = L.qp, rp = L.rp, op = L.op, dp = L.dp, vp = L.vp;
+    const bool own = c.kv_from < 0;
+    if (!own) {
+        B200_CHECK_ARG(c.kv_from < l && S->layers[c.kv_from].c.mixer == B200_MIXER_LATENT_ATTENTION &&
+                           S->layers[c.kv_from].c.kv_from < 0, "layer %d: layer %d has no latents of its own", l, c.kv_from);
+        const b200_layer_config& from = S->layers[c.kv_from].c;
+        B200_CHECK_ARG(from.kv_rank == c.kv_rank && same_rope(from, c), "layer %d: its latents are not those of layer %d", l, c.kv_from);
+        L.cache = S->layers[c.kv_from].cache;
+    }
+    S_TRY(named_bytes(e, &L.down_qkv, "down_qkv" + sfx, (qp + (own ? rp : 0)) * hp * z));
     S_TRY(named_bytes(e, &L.q_norm, "q_latent_norm" + sfx, qp * z));
-    S_TRY(named_bytes(e, &L.kv_norm, "kv_latent_norm" + sfx, rp * z));
+    if (own) S_TRY(named_bytes(e, &L.kv_norm, "kv_latent_norm" + sfx, rp * z));
+    S_TRY(rope_table(e, L));
     S_TRY(named_bytes(e, &L.uq, "uq" + sfx, H * dp * qp * z));
     S_TRY(named_bytes(e, &L.uk_absorb, "uk_absorb" + sfx, H * rp * dp * z));
-    S_TRY(named_bytes(e, &L.uv, "uv" + sfx, H * vp * rp * z));
-    S_TRY(named_bytes(e, &L.cache, "latent_cache" + sfx, e->num_slots * rp * z));
+    S_TRY(named_bytes(e, &L.uv, "uv" + sfx, H * vp * op * z));
+    if (own) S_TRY(named_bytes(e, &L.cache, "latent_cache" + sfx, e->num_slots * rp * z));
     // what the prefill kernel of the grouped-query models takes (and its positive score scale)
     L.can_expand = S->dtype == B200_DTYPE_BF16 && dp == 128 && vp == 128 && c.score_scale > 0.f && H <= 65535;
     if (L.can_expand) S_TRY(named_bytes(e, &L.uk, "uk" + sfx, H * dp * rp * z));
@@ -212,52 +315,33 @@ int alloc_latent(b200_engine* e, StackLayer& L, const std::string& sfx, Widths& 
     return B200_OK;
 }
 
-// cos / sin of position * base^(-2 i / dims), computed in double on the host; layers with the same rotation share
-// a table.
-int rope_table(b200_engine* e, StackLayer& L, int l) {
+// Columns of the joint projection's rows.
+int64_t joint_width(const StackLayer& L) {
     const b200_layer_config& c = L.c;
-    for (int o = 0; o < l; ++o) {
-        const StackLayer& other = e->stack->layers[o];
-        if (other.cos_t != nullptr && other.c.rotary_dim == c.rotary_dim && other.c.rope_base == c.rope_base) {
-            L.cos_t = other.cos_t;
-            L.sin_t = other.sin_t;
-            return B200_OK;
-        }
-    }
-    const int half = c.rotary_dim / 2;
-    const int64_t n = static_cast<int64_t>(e->pt_cols) * half;
-    std::vector<float> cs(n), sn(n);
-    for (int i = 0; i < half; ++i) {
-        const double f = pow(c.rope_base, -2.0 * i / c.rotary_dim);
-        for (int64_t p = 0; p < e->pt_cols; ++p) {
-            cs[p * half + i] = static_cast<float>(cos(static_cast<double>(p) * f));
-            sn[p * half + i] = static_cast<float>(sin(static_cast<double>(p) * f));
-        }
-    }
-    void* p = nullptr;
-    S_TRY(dev_alloc(e, &p, n * 4, true));
-    L.cos_t = static_cast<float*>(p);
-    S_TRY(dev_alloc(e, &p, n * 4, true));
-    L.sin_t = static_cast<float*>(p);
-    if (n == 0) return B200_OK;
-    B200_CHECK_CUDA(cudaMemcpy(L.cos_t, cs.data(), n * 4, cudaMemcpyHostToDevice));
-    B200_CHECK_CUDA(cudaMemcpy(L.sin_t, sn.data(), n * 4, cudaMemcpyHostToDevice));
-    return B200_OK;
+    const int64_t H = c.heads, G = c.kv_heads, dp = L.dp, vp = L.vp;
+    if (c.mixer == B200_MIXER_LINEAR_ATTENTION) return 2 * H * (dp + vp) + pad_width(c.decay_rank);
+    if (c.mixer == B200_MIXER_WINDOW_ATTENTION)
+        return (H + G) * dp + G * vp + (c.gate == B200_GATE_ELEMENT ? H * vp : c.gate == B200_GATE_HEAD ? pad_width(c.heads) : 0);
+    return 2 * H * vp + 2 * G * dp + pad_width(c.mixer == B200_MIXER_DELTA_RULE ? 2 * c.heads : c.heads);
 }
 
-int alloc_window(b200_engine* e, StackLayer& L, int l, const std::string& sfx, Widths& w) {
+// (names of a mixer's tensors start with `pre`)
+int alloc_window(b200_engine* e, StackLayer& L, int l, const std::string& pre, const std::string& sfx, Widths& w) {
     LayerStack* S = e->stack;
     const b200_layer_config& c = L.c;
-    L.dp = pad_head_dim(c.head_dim);
-    L.vp = pad_head_dim(c.value_dim);
-    const int64_t hp = S->hp, z = S->esz, H = c.heads, G = c.kv_heads, dp = L.dp, vp = L.vp;
-    const int64_t joint = (H + G) * dp + (G + H) * vp;
-    S_TRY(named_bytes(e, &L.qkvg, "qkvg" + sfx, joint * hp * z));
-    S_TRY(named_bytes(e, &L.q_head_norm, "q_head_norm" + sfx, dp * z));
-    S_TRY(named_bytes(e, &L.k_head_norm, "k_head_norm" + sfx, dp * z));
-    S_TRY(named_bytes(e, &L.k_cache, "k_cache" + sfx, e->num_slots * G * dp * z));
-    S_TRY(named_bytes(e, &L.v_cache, "v_cache" + sfx, e->num_slots * G * vp * z));
-    S_TRY(rope_table(e, L, l));
+    const int64_t z = S->esz, G = c.kv_heads, dp = L.dp, vp = L.vp;
+    if (c.head_norm) {
+        S_TRY(named_bytes(e, &L.q_head_norm, pre + "q_head_norm" + sfx, dp * z));
+        S_TRY(named_bytes(e, &L.k_head_norm, pre + "k_head_norm" + sfx, dp * z));
+    }
+    S_TRY(named_bytes(e, &L.k_cache, pre + "k_cache" + sfx, e->num_slots * G * dp * z));
+    S_TRY(named_bytes(e, &L.v_cache, pre + "v_cache" + sfx, e->num_slots * G * vp * z));
+    S_TRY(rope_table(e, L));
+    void* p = nullptr;
+    if (c.sink) {
+        S_TRY(named_bytes(e, &p, pre + "sinks" + sfx, c.heads * 4ll));
+        L.sinks = static_cast<float*>(p);
+    }
     if (c.value_mix) {
         L.mix = HeadPrepare::kSave;
         for (int o = 0; o < l; ++o) {
@@ -269,34 +353,113 @@ int alloc_window(b200_engine* e, StackLayer& L, int l, const std::string& sfx, W
                            f.value_dim, o);
             break;
         }
-        void* p = nullptr;
-        S_TRY(named_bytes(e, &p, "value_mix" + sfx, 4));
+        S_TRY(named_bytes(e, &p, pre + "value_mix" + sfx, 4));
         L.value_mix = static_cast<float*>(p);
         Widths::widest(w.first, G * vp);
     }
-    Widths::widest(w.joint, joint);
     if (c.kv_heads <= 8 && 8 % c.kv_heads == 0)
         Widths::widest(w.ws, decode_workspace_bytes(e->max_batch, c.heads, c.kv_heads));
     return B200_OK;
 }
 
-int alloc_linear(b200_engine* e, StackLayer& L, const std::string& sfx, Widths& w) {
+int alloc_linear(b200_engine* e, StackLayer& L, const std::string& pre, const std::string& sfx) {
     LayerStack* S = e->stack;
     const b200_layer_config& c = L.c;
-    L.dp = pad_width(c.head_dim);
-    L.vp = pad_width(c.value_dim);
     L.up_ld = pad_to(c.decay_rank, 16);
-    const int64_t hp = S->hp, z = S->esz, H = c.heads, dp = L.dp, vp = L.vp;
-    const int64_t joint = 2 * H * (dp + vp) + pad_width(c.decay_rank);
+    const int64_t z = S->esz, H = c.heads, dp = L.dp, vp = L.vp;
     void* p = nullptr;
-    S_TRY(named_bytes(e, &L.qkvga, "qkvga" + sfx, joint * hp * z));
-    S_TRY(named_bytes(e, &L.decay_up, "decay_up" + sfx, H * dp * L.up_ld * z));
-    S_TRY(named_bytes(e, &p, "decay_bias" + sfx, H * dp * 4));
+    S_TRY(named_bytes(e, &L.decay_up, pre + "decay_up" + sfx, H * dp * L.up_ld * z));
+    S_TRY(named_bytes(e, &p, pre + "decay_bias" + sfx, H * dp * 4));
     L.decay_bias = static_cast<float*>(p);
-    S_TRY(named_bytes(e, &L.head_norm, "head_norm" + sfx, vp * z));
-    S_TRY(named_bytes(e, &p, "state" + sfx, static_cast<int64_t>(e->pt_rows) * H * dp * vp * 4));
+    S_TRY(named_bytes(e, &L.head_norm, pre + "head_norm" + sfx, vp * z));
+    S_TRY(named_bytes(e, &p, pre + "state" + sfx, static_cast<int64_t>(e->pt_rows) * H * dp * vp * 4));
     L.state = static_cast<float*>(p);
-    Widths::widest(w.joint, joint);
+    return B200_OK;
+}
+
+int alloc_recurrence(b200_engine* e, StackLayer& L, const std::string& pre, const std::string& sfx, Widths& w) {
+    LayerStack* S = e->stack;
+    const b200_layer_config& c = L.c;
+    const bool delta = c.mixer == B200_MIXER_DELTA_RULE;
+    const int64_t z = S->esz, H = c.heads, dp = L.dp, vp = L.vp, channels = H * vp + 2 * c.kv_heads * dp;
+    void* p = nullptr;
+    auto floats = [&](float*& to, const char* name, int64_t n) -> int {
+        S_TRY(named_bytes(e, &p, pre + name + sfx, n * 4));
+        to = static_cast<float*>(p);
+        return B200_OK;
+    };
+    S_TRY(floats(L.conv, "conv", c.conv_taps * channels));
+    S_TRY(floats(L.conv_bias, "conv_bias", channels));
+    S_TRY(floats(L.decay_log, "decay_log", H));
+    S_TRY(floats(L.step_bias, "step_bias", H));
+    if (!delta) S_TRY(floats(L.skip, "skip", H));
+    S_TRY(named_bytes(e, &L.head_norm, pre + "head_norm" + sfx, (delta ? vp : H * vp) * z));
+    S_TRY(floats(L.state, "state", static_cast<int64_t>(e->pt_rows) * H * dp * vp));
+    S_TRY(named_bytes(e, &L.conv_state, pre + "conv_state" + sfx, static_cast<int64_t>(e->pt_rows) * c.conv_taps * channels * z));
+    const RecurrenceScratch need = recurrence_scratch(delta ? B200_RULE_DELTA : B200_RULE_STATE_SPACE, e->max_tokens, e->max_batch,
+                                                      c.heads, c.kv_heads, L.dp, L.vp, S->dtype);
+    Widths::widest(w.mixed, need.mixed);
+    Widths::widest(w.steps, need.steps);
+    Widths::widest(w.units, need.units);
+    Widths::widest(w.chunks, need.chunks);
+    return B200_OK;
+}
+
+// What a mixer other than latent attention has beside its input and output projections.
+int alloc_mixer(b200_engine* e, StackLayer& L, int l, const std::string& pre, const std::string& sfx, Widths& w) {
+    const b200_layer_config& c = L.c;
+    const bool window = c.mixer == B200_MIXER_WINDOW_ATTENTION;
+    L.dp = window ? pad_head_dim(c.head_dim) : pad_width(c.head_dim);
+    L.vp = window ? pad_head_dim(c.value_dim) : pad_width(c.value_dim);
+    L.out_ld = static_cast<int64_t>(c.heads) * L.vp;
+    L.joint_ld = joint_width(L);
+    if (window) return alloc_window(e, L, l, pre, sfx, w);
+    if (is_recurrence(c.mixer)) return alloc_recurrence(e, L, pre, sfx, w);
+    return alloc_linear(e, L, pre, sfx);
+}
+
+// Mixer (or both mixers) of a layer: the projections around it, then the rest.
+int alloc_layer_mixer(b200_engine* e, StackLayer& L, int l, const std::string& sfx, Widths& w) {
+    LayerStack* S = e->stack;
+    const b200_layer_config& c = L.c;
+    const int64_t hp = S->hp, z = S->esz;
+    if (c.mixer == B200_MIXER_LATENT_ATTENTION) {
+        B200_CHECK_ARG(c.beside < 0, "layer %d: nothing runs beside latent attention", l);
+        S_TRY(alloc_latent(e, L, l, sfx, w));
+        L.out_ld = static_cast<int64_t>(c.heads) * L.vp;
+        Widths::widest(w.attn, L.out_ld);
+        return named_bytes(e, &L.o, "o" + sfx, hp * L.out_ld * z);
+    }
+    S_TRY(alloc_mixer(e, L, l, "", sfx, w));
+    StackLayer* R = L.beside;
+    const char* name = c.mixer == B200_MIXER_WINDOW_ATTENTION ? "qkvg" : c.mixer == B200_MIXER_LINEAR_ATTENTION ? "qkvga" : "recurrence";
+    const int64_t left_out = L.out_ld;
+    if (R != nullptr) {
+        B200_CHECK_ARG(c.mixer != B200_MIXER_LINEAR_ATTENTION && R->c.mixer != B200_MIXER_LINEAR_ATTENTION &&
+                           R->c.mixer != B200_MIXER_LATENT_ATTENTION && !R->c.value_mix, "layer %d: mixers that do not run side by side", l);
+        B200_CHECK_ARG(c.join == B200_JOIN_SUM || c.join == B200_JOIN_NORMED, "layer %d: unknown join", l);
+        S_TRY(check_mixer(R->c, l));
+        S_TRY(alloc_mixer(e, *R, l, "beside_", sfx, w));
+        name = "joint";
+        R->joint_at = L.joint_ld;
+        L.joint_ld = R->joint_ld = L.joint_ld + R->joint_ld;
+        Widths::widest(w.attn, left_out + R->out_ld);
+        if (c.join == B200_JOIN_SUM) {
+            R->out_at = left_out;
+            L.out_ld = R->out_ld = left_out + R->out_ld;
+        } else {
+            w.normed_pair = true;
+            R->out_at = static_cast<int64_t>(e->max_tokens) * left_out;
+            S_TRY(named_bytes(e, &R->o, "beside_o" + sfx, hp * R->out_ld * z));
+            S_TRY(named_bytes(e, &L.side_norm, "side_norm" + sfx, hp * z));
+            S_TRY(named_bytes(e, &R->side_norm, "beside_side_norm" + sfx, hp * z));
+        }
+    }
+    S_TRY(named_bytes(e, &L.joint, name + sfx, L.joint_ld * hp * z));
+    if (c.qkv_bias || (R != nullptr && R->c.qkv_bias)) S_TRY(named_bytes(e, &L.joint_bias, "joint_bias" + sfx, L.joint_ld * z));
+    S_TRY(named_bytes(e, &L.o, "o" + sfx, hp * L.out_ld * z));
+    Widths::widest(w.joint, L.joint_ld);
+    Widths::widest(w.attn, L.out_ld);
     return B200_OK;
 }
 
@@ -308,6 +471,7 @@ int alloc_feed_forward(b200_engine* e, StackLayer& L, const std::string& sfx, Wi
     const int64_t n_up = (epilogue_is_gated(c.epilogue) ? 2 : 1) * static_cast<int64_t>(L.ip);
     const int64_t E = c.mlp == B200_MLP_DENSE ? 1 : c.num_experts;
     S_TRY(named_bytes(e, &L.norm2, "norm2" + sfx, hp * z));
+    if (S->norm_input && S->norm_output) S_TRY(named_bytes(e, &L.norm2_out, "norm2_out" + sfx, hp * z));
     S_TRY(named_bytes(e, &L.up, "mlp_up" + sfx, E * n_up * hp * z));
     S_TRY(named_bytes(e, &L.down, "mlp_down" + sfx, E * hp * L.ip * z));
     if (c.mlp == B200_MLP_DENSE) {
@@ -355,7 +519,10 @@ int layer_stack_create(b200_engine* e, const b200_stack_config* sc) {
     S->esz = sc->dtype == B200_DTYPE_F32 ? 4 : 2;
     S->norm_offset = sc->norm_offset;
     S->logit_scale = sc->logit_scale;
-    S->norm_output = sc->norm_output != 0;
+    B200_CHECK_ARG(sc->norm_output >= B200_NORM_INPUT && sc->norm_output <= B200_NORM_BOTH, "layer stack: unknown norm placement");
+    B200_CHECK_ARG(sc->num_beside >= 0 && (sc->num_beside == 0 || sc->beside), "layer stack: no mixers to run beside others");
+    S->norm_input = sc->norm_output != B200_NORM_OUTPUT;
+    S->norm_output = sc->norm_output != B200_NORM_INPUT;
     S->hp = pad_width(e->m.hidden_size);
     S->vocab_p = pad_width(e->m.vocab_size);
     if (const char* v = getenv("B200_LATENT_EXPAND_MIN")) S->expand_min = atoi(v);
@@ -373,6 +540,8 @@ int layer_stack_create(b200_engine* e, const b200_stack_config* sc) {
     S->latent_rows = e->max_batch > 1024 ? e->max_batch : 1024;
     if (S->latent_rows > e->max_tokens) S->latent_rows = e->max_tokens;
     S->layers.resize(sc->num_layers);
+    S->besides.resize(sc->num_beside);
+    for (int i = 0; i < sc->num_beside; ++i) S->besides[i].c = sc->beside[i];
     for (int l = 0; l < sc->num_layers; ++l) {
         StackLayer& L = S->layers[l];
         L.c = sc->layers[l];
@@ -382,12 +551,10 @@ int layer_stack_create(b200_engine* e, const b200_stack_config* sc) {
                        "layer %d: experts by token id take the norm on their input", l);
         const std::string sfx = "." + std::to_string(l);
         S_TRY(named_bytes(e, &L.norm1, "norm1" + sfx, hp * z));
-        if (c.mixer == B200_MIXER_LATENT_ATTENTION) S_TRY(alloc_latent(e, L, sfx, w));
-        if (c.mixer == B200_MIXER_WINDOW_ATTENTION) S_TRY(alloc_window(e, L, l, sfx, w));
-        if (c.mixer == B200_MIXER_LINEAR_ATTENTION) S_TRY(alloc_linear(e, L, sfx, w));
-        const int64_t heads_out = static_cast<int64_t>(c.heads) * L.vp;
-        S_TRY(named_bytes(e, &L.o, "o" + sfx, hp * heads_out * z));
-        Widths::widest(w.attn, heads_out);
+        if (S->norm_input && S->norm_output) S_TRY(named_bytes(e, &L.norm1_out, "norm1_out" + sfx, hp * z));
+        B200_CHECK_ARG(c.beside < sc->num_beside, "layer %d: no mixer %d to run beside", l, c.beside);
+        if (c.beside >= 0) L.beside = &S->besides[c.beside];
+        S_TRY(alloc_layer_mixer(e, L, l, sfx, w));
         if (c.mlp != B200_MLP_NONE) S_TRY(alloc_feed_forward(e, L, sfx, w));
     }
     void* p = nullptr;
@@ -414,6 +581,15 @@ int layer_stack_create(b200_engine* e, const b200_stack_config* sc) {
     S->compact_row = static_cast<int32_t*>(p);
     S_TRY(dev_alloc(e, &p, Tm * 4, true));
     S->compact_len = static_cast<int32_t*>(p);
+    if (w.mixed > 0) {
+        S_TRY(dev_alloc(e, &S->mixed, w.mixed, true));
+        S_TRY(dev_alloc(e, &p, w.steps, true));
+        S->steps = static_cast<float*>(p);
+        S_TRY(dev_alloc(e, &p, w.units, true));
+        S->units = static_cast<float*>(p);
+        S_TRY(dev_alloc(e, &S->chunks, w.chunks, true));
+    }
+    if (w.normed_pair) S_TRY(dev_alloc(e, &S->y2, Tm * hp * z, true));
     if (w.first > 0) S_TRY(dev_alloc(e, &S->first_values, Tm * w.first * z, true));
     if (w.scored) {
         S_TRY(dev_alloc(e, &p, Tm * w.router * 4, true));
@@ -513,11 +689,12 @@ int layer_stack_plan(b200_engine* e, const b200_step* st, int Bp) {
 
 namespace {
 
-int project(b200_engine* e, void* y, const void* x, const void* w, int M, int N, int K, int epilogue, float limit = 0.f) {
+int project(b200_engine* e, void* y, const void* x, const void* w, int M, int N, int K, int epilogue, float limit = 0.f,
+            const void* bias = nullptr) {
     if (e->stack->dtype == B200_DTYPE_F32)
         return launch_linear_f32(static_cast<float*>(y), static_cast<const float*>(x), static_cast<const float*>(w), M, N, K,
-                                 1, nullptr, nullptr, epilogue, e->stream, limit);
-    return launch_linear(y, x, w, nullptr, M, N, K, K, epilogue, e->status, e->stream, nullptr, limit);
+                                 1, nullptr, nullptr, epilogue, e->stream, limit, static_cast<const float*>(bias));
+    return launch_linear(y, x, w, bias, M, N, K, K, epilogue, e->status, e->stream, nullptr, limit);
 }
 
 int project_heads(b200_engine* e, void* y, const void* x, const void* w, int M, int heads, int N, int K) {
@@ -559,6 +736,7 @@ int attend_latent(b200_engine* e, const StackLayer& L, void* out, const void* q,
         a.rows = n;
         a.heads = H;
         a.width = L.rp;
+        a.out_width = L.op;
         a.page_size = e->c.page_size;
         a.scale = L.c.score_scale;
         a.only_last_key_new = decode;
@@ -568,7 +746,7 @@ int attend_latent(b200_engine* e, const StackLayer& L, void* out, const void* q,
             S_TRY(launch_latent_attention_tc(a, e->status, e->stream));
         else
             S_TRY(launch_latent_attention_plain(a, S->dtype, e->status, e->stream));
-        S_TRY(project_heads(e, os, S->ol, L.uv, n, H, L.vp, L.rp));
+        S_TRY(project_heads(e, os, S->ol, L.uv, n, H, L.vp, L.op));
     }
     return B200_OK;
 }
@@ -588,7 +766,7 @@ int attend(b200_engine* e, const StackLayer& L, int phase, int Bp, int T) {
     S_TRY(launch_gather_latents(S->xc, L.cache, e->num_slots, e->page_table, e->pt_cols, table_idx, x_len, g_base, Bp,
                                 S->plan_max_len, L.rp, e->status, e->stream));
     S_TRY(project(e, S->xk, S->xc, L.uk, rows, H * L.dp, L.rp, B200_EPILOGUE_NONE));
-    S_TRY(project(e, S->xv, S->xc, L.uv, rows, H * L.vp, L.rp, B200_EPILOGUE_NONE));
+    S_TRY(launch_linear(S->xv, S->xc, L.uv, nullptr, rows, H * L.vp, L.op, L.rp, B200_EPILOGUE_NONE, e->status, e->stream));
     // request b's expanded rows start at x_base[b]: with the identity row as the page table and a row
     // stride of one, "table row x_base[b]" maps position p to x_base[b] + p
     S_TRY(launch_attention_prefill(S->attn, S->q, static_cast<int64_t>(H) * L.dp, L.dp, S->xk, S->xv, rows, S->iota, 1,
@@ -604,19 +782,45 @@ int attend(b200_engine* e, const StackLayer& L, int phase, int Bp, int T) {
 int latent_mixer(b200_engine* e, const StackLayer& L, int T) {
     LayerStack* S = e->stack;
     const b200_layer_config& c = L.c;
-    S_TRY(project(e, S->joint, S->x, L.down_qkv, T, L.qp + L.rp, S->hp, B200_EPILOGUE_NONE));
-    S_TRY(launch_latent_norm_store(S->cq, L.cache, S->joint, L.q_norm, L.kv_norm, e->out_loc, T, c.q_rank, L.qp,
-                                   c.kv_rank, L.rp, e->num_slots, e->m.rms_norm_eps, S->dtype, e->status, e->stream));
-    return project(e, S->q, S->cq, L.uq, T, c.heads * L.dp, L.qp, B200_EPILOGUE_NONE);
+    const bool own = c.kv_from < 0;
+    LatentNorm n;
+    n.q_latent = S->cq;
+    n.cache = own ? L.cache : nullptr;
+    n.joint = S->joint;
+    n.q_weight = L.q_norm;
+    n.kv_weight = L.kv_norm;
+    n.out_loc = e->out_loc;
+    n.positions = e->positions;
+    n.tokens = T;
+    n.q_rank = c.q_rank;
+    n.qp = L.qp;
+    n.kv_rank = c.kv_rank;
+    n.rp = own ? L.rp : 0;
+    n.rope_at = latent_rope_at(c.kv_rank);
+    n.rope_dim = c.rotary_dim;
+    n.max_pos = e->pt_cols;
+    n.cos_t = L.cos_t;
+    n.sin_t = L.sin_t;
+    n.num_slots = e->num_slots;
+    n.eps = e->m.rms_norm_eps;
+    n.status = e->status;
+    S_TRY(project(e, S->joint, S->x, L.down_qkv, T, n.qp + n.rp, S->hp, B200_EPILOGUE_NONE));
+    S_TRY(launch_latent_norm_store(n, S->dtype, e->stream));
+    S_TRY(project(e, S->q, S->cq, L.uq, T, c.heads * L.dp, L.qp, B200_EPILOGUE_NONE));
+    return launch_rotate_pairs(S->q, T, c.heads, L.dp, c.rotary_dim, L.cos_t, L.sin_t, e->positions, e->pt_cols, S->dtype,
+                               e->status, e->stream);
 }
 
-int window_mixer(b200_engine* e, const StackLayer& L, int T) {
+// A mixer's columns of the joint rows, and its place in the result buffer.
+char* joint_of(const LayerStack* S, const StackLayer& L) { return static_cast<char*>(S->joint) + L.joint_at * S->esz; }
+char* result_of(const LayerStack* S, const StackLayer& L) { return static_cast<char*>(S->attn) + L.out_at * S->esz; }
+
+int window_prepare(b200_engine* e, const StackLayer& L, int T) {
     LayerStack* S = e->stack;
     const b200_layer_config& c = L.c;
     HeadPrepare a;
-    a.joint = S->joint;
-    a.ld = static_cast<int64_t>(c.heads + c.kv_heads) * (L.dp + L.vp);
-    S_TRY(project(e, S->joint, S->x, L.qkvg, T, static_cast<int>(a.ld), S->hp, B200_EPILOGUE_NONE));
+    a.joint = joint_of(S, L);
+    a.ld = L.joint_ld;
     a.tokens = T;
     a.heads = c.heads;
     a.kv_heads = c.kv_heads;
@@ -646,9 +850,9 @@ int window_attend(b200_engine* e, const StackLayer& L, int phase, int Bp, int T)
     LayerStack* S = e->stack;
     const b200_layer_config& c = L.c;
     WindowAttention a;
-    a.out = S->attn;
-    a.q = S->joint;
-    a.q_st = static_cast<int64_t>(c.heads + c.kv_heads) * (L.dp + L.vp);
+    a.out = result_of(S, L);
+    a.q = joint_of(S, L);
+    a.q_st = L.joint_ld;
     a.k_cache = L.k_cache;
     a.v_cache = L.v_cache;
     a.num_slots = e->num_slots;
@@ -671,9 +875,16 @@ int window_attend(b200_engine* e, const StackLayer& L, int phase, int Bp, int T)
     a.scale = c.score_scale;
     a.window.size = c.window;
     a.window.keep_first = c.keep_first;
-    a.window.gate = static_cast<const char*>(S->joint) +
-                    (static_cast<int64_t>(c.heads + c.kv_heads) * L.dp + static_cast<int64_t>(c.kv_heads) * L.vp) * S->esz;
-    a.window.gate_st = a.q_st;
+    a.window.chunk = c.chunk;
+    a.window.sinks = L.sinks;
+    if (c.gate != B200_GATE_NONE) {
+        a.window.gate = joint_of(S, L) +
+                        (static_cast<int64_t>(c.heads + c.kv_heads) * L.dp + static_cast<int64_t>(c.kv_heads) * L.vp) * S->esz;
+        a.window.gate_st = a.q_st;
+        a.window.gate_per_head = c.gate == B200_GATE_HEAD;
+    }
+    a.window.out_scale = c.out_scale;
+    a.window.out_st = L.out_ld;
     a.workspace = S->ws;
     a.workspace_bytes = S->ws_bytes;
     a.status = e->status;
@@ -686,8 +897,7 @@ int linear_mixer(b200_engine* e, const StackLayer& L, int phase, int Bp, int T) 
     LinearAttention a = {};
     a.out = S->attn;
     a.joint = S->joint;
-    a.joint_ld = 2ll * c.heads * (L.dp + L.vp) + pad_width(c.decay_rank);
-    S_TRY(project(e, S->joint, S->x, L.qkvga, T, static_cast<int>(a.joint_ld), S->hp, B200_EPILOGUE_NONE));
+    a.joint_ld = L.joint_ld;
     a.tokens = T;
     a.batch = Bp;
     a.decode = phase == B200_PHASE_DECODE ? 1 : 0;
@@ -711,17 +921,50 @@ int linear_mixer(b200_engine* e, const StackLayer& L, int phase, int Bp, int T) 
     return launch_linear_attention(a, S->dtype, e->stream);
 }
 
-// S->x through the layer's mixer to S->y.
-int mix(b200_engine* e, int l, int phase, int Bp, int T) {
+int recurrence_mixer(b200_engine* e, const StackLayer& L, int phase, int Bp, int T) {
     LayerStack* S = e->stack;
-    const StackLayer& L = S->layers[l];
-    cudaStream_t s = e->stream;
-    if (L.c.mixer == B200_MIXER_LINEAR_ATTENTION) {
-        S_TRY(linear_mixer(e, L, phase, Bp, T));
-        return project(e, S->y, S->attn, L.o, T, S->hp, L.c.heads * L.vp, B200_EPILOGUE_NONE);
-    }
-    const bool latent = L.c.mixer == B200_MIXER_LATENT_ATTENTION;
-    S_TRY(latent ? latent_mixer(e, L, T) : window_mixer(e, L, T));
+    const b200_layer_config& c = L.c;
+    Recurrence a = {};
+    a.out = result_of(S, L);
+    a.out_ld = L.out_ld;
+    a.joint = joint_of(S, L);
+    a.joint_ld = L.joint_ld;
+    a.rule = c.mixer == B200_MIXER_DELTA_RULE ? B200_RULE_DELTA : B200_RULE_STATE_SPACE;
+    a.tokens = T;
+    a.batch = Bp;
+    a.max_extend = S->max_extend;
+    a.decode = phase == B200_PHASE_DECODE ? 1 : 0;
+    a.table_idx = e->meta_dev;
+    a.cached = e->meta_dev + Bp;
+    a.qo_indptr = e->meta_dev + 2 * Bp;
+    a.state = L.state;
+    a.conv_state = L.conv_state;
+    a.heads = c.heads;
+    a.kv_heads = c.kv_heads;
+    a.dim = c.head_dim;
+    a.padded_dim = L.dp;
+    a.value_dim = c.value_dim;
+    a.padded_value_dim = L.vp;
+    a.taps = c.conv_taps;
+    a.norm_groups = c.norm_groups;
+    a.conv = L.conv;
+    a.conv_bias = L.conv_bias;
+    a.decay_log = L.decay_log;
+    a.step_bias = L.step_bias;
+    a.skip = L.skip;
+    a.norm = L.head_norm;
+    a.eps = e->m.rms_norm_eps;
+    a.out_scale = c.out_scale;
+    a.mixed = S->mixed;
+    a.steps = S->steps;
+    a.units = S->units;
+    a.chunks = S->chunks;
+    return launch_recurrence(a, S->dtype, e->stream);
+}
+
+// Attention launches bracketed by events while the engine is being profiled.
+template <typename F>
+int timed_attention(b200_engine* e, F launch) {
     const bool timed = e->profile_attention && !e->capturing;
     const int at = e->prof_pairs_recorded;
     if (timed) {
@@ -730,14 +973,40 @@ int mix(b200_engine* e, int l, int phase, int Bp, int T) {
             B200_CHECK_CUDA(cudaEventCreate(&ev));
             e->prof_events.push_back(ev);
         }
-        B200_CHECK_CUDA(cudaEventRecord(e->prof_events[2 * at], s));
+        B200_CHECK_CUDA(cudaEventRecord(e->prof_events[2 * at], e->stream));
     }
-    S_TRY(latent ? attend(e, L, phase, Bp, T) : window_attend(e, L, phase, Bp, T));
+    S_TRY(launch());
     if (timed) {
-        B200_CHECK_CUDA(cudaEventRecord(e->prof_events[2 * at + 1], s));
+        B200_CHECK_CUDA(cudaEventRecord(e->prof_events[2 * at + 1], e->stream));
         e->prof_pairs_recorded = at + 1;
     }
-    return project(e, S->y, S->attn, L.o, T, S->hp, L.c.heads * L.vp, B200_EPILOGUE_NONE);
+    return B200_OK;
+}
+
+// A mixer between the joint projection and the output projection.
+int run_mixer(b200_engine* e, const StackLayer& L, int phase, int Bp, int T) {
+    if (L.c.mixer == B200_MIXER_LINEAR_ATTENTION) return linear_mixer(e, L, phase, Bp, T);
+    if (is_recurrence(L.c.mixer)) return recurrence_mixer(e, L, phase, Bp, T);
+    S_TRY(window_prepare(e, L, T));
+    return timed_attention(e, [&] { return window_attend(e, L, phase, Bp, T); });
+}
+
+// S->x through the layer's mixer, or both of them, to S->y (under B200_JOIN_NORMED the right one's result to S->y2).
+int mix(b200_engine* e, int l, int phase, int Bp, int T) {
+    LayerStack* S = e->stack;
+    const StackLayer& L = S->layers[l];
+    if (L.c.mixer == B200_MIXER_LATENT_ATTENTION) {
+        S_TRY(latent_mixer(e, L, T));
+        S_TRY(timed_attention(e, [&] { return attend(e, L, phase, Bp, T); }));
+    } else {
+        S_TRY(project(e, S->joint, S->x, L.joint, T, static_cast<int>(L.joint_ld), S->hp, B200_EPILOGUE_NONE, 0.f, L.joint_bias));
+        S_TRY(run_mixer(e, L, phase, Bp, T));
+        if (L.beside != nullptr) S_TRY(run_mixer(e, *L.beside, phase, Bp, T));
+        if (L.side_norm != nullptr)
+            S_TRY(project(e, S->y2, result_of(S, *L.beside), L.beside->o, T, S->hp, static_cast<int>(L.beside->out_ld),
+                          B200_EPILOGUE_NONE));
+    }
+    return project(e, S->y, S->attn, L.o, T, S->hp, static_cast<int>(L.out_ld), B200_EPILOGUE_NONE);
 }
 
 // S->x through a dense layer to S->y, or through the experts its scores choose to S->ye (and the expert that
@@ -776,14 +1045,17 @@ int feed_forward(b200_engine* e, const StackLayer& L, int T) {
 }
 
 // What a block has left behind for the residual kernel that follows it.
-void take_block(LayerStack* S, const StackLayer* experts, int T, ResidualPostNorm& rn) {
+void take_block(LayerStack* S, const StackLayer* experts, const StackLayer* pair, int T, ResidualPostNorm& rn) {
     rn.init = false;
     rn.src = experts ? S->ye : S->y;
     rn.src_rows = experts ? S->route_rows : nullptr;
     rn.src_weights = experts ? S->route_weights : nullptr;
     rn.src_top = experts ? experts->c.experts_per_tok : 1;
     rn.src_count = static_cast<int64_t>(T) * rn.src_top;
-    rn.src2 = experts && experts->isp > 0 ? S->shared_y : nullptr;
+    rn.src2 = pair ? S->y2 : experts && experts->isp > 0 ? S->shared_y : nullptr;
+    rn.pair_weight = pair ? pair->side_norm : nullptr;
+    rn.pair_weight2 = pair ? pair->beside->side_norm : nullptr;
+    rn.pair_scale = 0.5f;
 }
 
 }  // namespace
@@ -829,6 +1101,7 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
     post.padded = hp;
     post.eps = e->m.rms_norm_eps;
     const StackLayer* scored = nullptr;   // the last block was this layer's scored experts
+    const StackLayer* pair = nullptr;     // the last block was this layer's two mixers, normalised each
     const void* own_norm = nullptr;       // norm_output: the norm of the last block's output
     auto add_plain = [&]() {
         rn.src = S->y;
@@ -837,14 +1110,14 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
         rn.src_count = T;
         rn.src_scale = 1.f;
         rn.init = false;
-        scored = nullptr;
+        scored = pair = nullptr;
     };
     // Adds the last block and leaves what the next one reads: normalised with `weight`, or as it is.
     auto advance = [&](const void* weight, void* out, const int32_t* rows, int top, float out_scale,
                        const StackLayer* next_scored) -> int {
         post.clear = next_scored ? S->route_counts : nullptr;
         post.clear_count = next_scored ? 2 * next_scored->c.num_experts : 0;
-        if (!S->norm_output && scored == nullptr && next_scored == nullptr) {
+        if (!S->norm_output && scored == nullptr && pair == nullptr && next_scored == nullptr) {
             rn.weight = weight;
             rn.out = out;
             rn.out_rows = rows;
@@ -852,7 +1125,7 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
             rn.out_scale = out_scale;
             return launch_residual_norm(rn, S->dtype, e->status, s);
         }
-        if (!rn.init) take_block(S, scored, T, post);
+        if (!rn.init) take_block(S, scored, pair, T, post);
         post.add_weight = own_norm;
         post.out_weight = weight;
         post.out_scale = out_scale;
@@ -870,18 +1143,20 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
         const b200_layer_config& c = L.c;
         // The first norm is launched as an ordinary dependent of what prepares the step, so that every
         // kernel after it finds positions, slots and lengths complete even ahead of its own wait.
-        S_TRY(advance(S->norm_output ? nullptr : L.norm1, S->x, nullptr, 1, 1.f, nullptr));
+        S_TRY(advance(S->norm_input ? L.norm1 : nullptr, S->x, nullptr, 1, 1.f, nullptr));
         if (l == 0) set_pdl_launches(pdl);
         S_TRY(traced(l));
         S_TRY(mix(e, l, phase, Bp, T));
         add_plain();
-        if (S->norm_output) own_norm = L.norm1;
+        if (L.side_norm != nullptr) pair = &L;
+        if (S->norm_output) own_norm = S->norm_input ? L.norm1_out : L.norm1;
         if (c.mlp == B200_MLP_NONE) continue;
         if (c.mlp == B200_MLP_TABLE_MOE) {
             const int n_up = (epilogue_is_gated(c.epilogue) ? 2 : 1) * L.ip;
             S_TRY(advance(L.norm2, S->xp, L.rows, c.experts_per_tok, 1.f, nullptr));
             S_TRY(project_experts(e, S->h, S->xp, L.up, L, L.counts, L.offsets, T, n_up, hp, c.epilogue));
             S_TRY(project_experts(e, S->ye, S->h, L.down, L, L.counts, L.offsets, T, hp, L.ip, B200_EPILOGUE_NONE));
+            pair = nullptr;
             rn.src = S->ye;
             rn.src_rows = L.rows;
             rn.src_top = c.experts_per_tok;
@@ -890,11 +1165,11 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
             rn.init = false;
             continue;
         }
-        S_TRY(advance(S->norm_output ? nullptr : L.norm2, S->x, nullptr, 1, 1.f, c.mlp == B200_MLP_SCORED_MOE ? &L : nullptr));
+        S_TRY(advance(S->norm_input ? L.norm2 : nullptr, S->x, nullptr, 1, 1.f, c.mlp == B200_MLP_SCORED_MOE ? &L : nullptr));
         S_TRY(feed_forward(e, L, T));
         add_plain();
         if (c.mlp == B200_MLP_SCORED_MOE) scored = &L;
-        if (S->norm_output) own_norm = L.norm2;
+        if (S->norm_output) own_norm = S->norm_input ? L.norm2_out : L.norm2;
     }
     S_TRY(advance(S->final_norm, S->x, nullptr, 1, S->logit_scale, nullptr));
     return traced(num_layers);
@@ -912,5 +1187,6 @@ extern "C" {
 int b200_pad_width(int n) { return b200::pad_width(n); }
 int b200_pad_head_dim(int n) { return b200::pad_head_dim(n); }
 int b200_pad_latent(int n) { return b200::pad_latent(n); }
+int b200_latent_rope_at(int kv_rank) { return b200::latent_rope_at(kv_rank); }
 
 }  // extern "C"

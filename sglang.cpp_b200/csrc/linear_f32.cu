@@ -19,6 +19,7 @@ struct F32Params {
     const int32_t* counts;     // grouped mode
     const int32_t* offsets;
     int per_head;              // z selects a column block of x and y
+    const float* bias;         // [n_out] or NULL, before the activation
     float act_limit;
 };
 
@@ -92,6 +93,7 @@ linear_f32_kernel(const F32Params p) {
             const int n = n0 + tx * 4 + j;
             if (n >= p.n_out) continue;
             float v = acc[i][j];
+            if (p.bias != nullptr) v += p.bias[n];
             if (EPI == B200_EPILOGUE_CLAMPED_SWIGLU)
                 v = clamped_swiglu<true>(v, up[GATED ? i : 0][j], p.act_limit);
             else if (GATED)
@@ -107,7 +109,7 @@ linear_f32_kernel(const F32Params p) {
 
 int launch_linear_f32(float* y, const float* x, const float* w, int max_rows, int N, int K, int groups,
                       const int32_t* counts, const int32_t* offsets, int epilogue, cudaStream_t stream,
-                      float act_limit) {
+                      float act_limit, const float* bias) {
     if (max_rows == 0 || groups == 0) return B200_OK;
     const bool per_head = counts == nullptr && groups > 1;
     F32Params p;
@@ -124,6 +126,7 @@ int launch_linear_f32(float* y, const float* x, const float* w, int max_rows, in
     p.offsets = offsets;
     p.per_head = per_head ? 1 : 0;
     p.act_limit = act_limit;
+    p.bias = bias;
     void (*kernel)(F32Params) = linear_f32_kernel<B200_EPILOGUE_NONE>;
     if (epilogue == B200_EPILOGUE_SWIGLU) kernel = linear_f32_kernel<B200_EPILOGUE_SWIGLU>;
     if (epilogue == B200_EPILOGUE_GEGLU) kernel = linear_f32_kernel<B200_EPILOGUE_GEGLU>;

@@ -1,0 +1,1109 @@
+// Recurrences with one decay per head and step, behind a short causal convolution: a scalar-decay state space
+//     S <- g S + dt k v^T,                    o = S^T q + skip v
+// and the gated delta rule (k and q unit vectors)
+//     S <- g S,  u = beta (v - S^T k),  S <- S + k u^T,    o = S^T q.
+// The matrix state is fp32 and lives in a slot per page-table row, as do the convolution's last inputs (a ring: the
+// input of position p is at p mod taps, so that a step writes a place that nobody reads in the same step).
+//
+//   * decode: one CTA per (request, head) convolves its channels, streams the state once - read, decayed, updated,
+//     read out, written, in registers between its first and its last use - and, for the delta rule, applies the
+//     head's norm and gate.  Everything that the projection before it does not write is read ahead of
+//     griddepcontrol.wait.
+//   * prefill: mix_kernel convolves all channels and leaves steps (decay logarithm, weight of what is written) and
+//     unit factors in fp32; the recurrence itself follows in chunks of 64 tokens (bf16) or token by token.
+//   * chunked: with B_t the decay logarithms summed up inside a chunk, G_t = exp(B_t), and S the state before it,
+//         P_ts = exp(B_t - B_s) q_t . k_s  (s <= t),     A_ts = beta_t exp(B_t - B_s) k_t . k_s  (s < t)
+//         U = (I + A)^-1 diag(beta) (V - diag(G) K S)     (state space: U = diag(dt) V)
+//         O = diag(G) Q S + P U
+//         S <- G_n S + K^T diag(exp(B_n - B_s)) U
+//     No exponent is positive, however steep the decay.  P and the inverse do not depend on the state: prepare_kernel
+//     makes them for all chunks at once (the inverse by substitution in fp32) and stores them in the order in which
+//     chunk_kernel's threads hold MMA operands.  chunk_kernel walks a request's chunks, one CTA per head and 64
+//     value columns.  k, q and v enter the products as the bf16 numbers the convolution returned, unit factors, steps
+//     and decays being applied to fp32 results; everything derived from those or from the state enters as the
+//     sum of two bf16 numbers.
+//   * a last kernel applies norm and gate where the recurrence did not.
+#include <math.h>
+
+#include "common.cuh"
+#include "kernels.h"
+
+namespace b200 {
+namespace {
+
+template <typename T>
+__device__ __forceinline__ float to_f32(T x) { return static_cast<float>(x); }
+template <>
+__device__ __forceinline__ float to_f32(__nv_bfloat16 x) { return __bfloat162float(x); }
+template <typename T>
+__device__ __forceinline__ T from_f32(float x) { return static_cast<T>(x); }
+template <>
+__device__ __forceinline__ __nv_bfloat16 from_f32(float x) { return __float2bfloat16_rn(x); }
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <typename T>
+__device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
+template <>
+__device__ __forceinline__ float silu<__nv_bfloat16>(float x) { return x * sigmoid_f(x); }
+
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr float kUnitEps = 1e-6f;
+constexpr int kMaxTaps = 32;
+constexpr int kStateSpace = B200_RULE_STATE_SPACE, kDelta = B200_RULE_DELTA;
+
+// Channel c of [v | k | q] is column values() + c of a row of the joint projection.
+__device__ __forceinline__ int64_t values(const Recurrence& a) { return static_cast<int64_t>(a.heads) * a.padded_value_dim; }
+__device__ __forceinline__ int64_t channels(const Recurrence& a) { return values(a) + 2ll * a.kv_heads * a.padded_dim; }
+
+// log2 of a step's decay and the weight of what it writes.
+template <typename T>
+__device__ __forceinline__ float2 step_of(const Recurrence& a, const T* row, int h) {
+    const T* tail = row + values(a) + channels(a);
+    const float x = to_f32(tail[h]) + a.step_bias[h];
+    const float dt = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
+    float2 s;
+    s.x = -expf(a.decay_log[h]) * dt * kLog2e;
+    s.y = a.rule == kStateSpace ? dt : 1.f / (1.f + expf(-to_f32(tail[a.heads + h])));
+    return s;
+}
+
+// ---- convolution, steps, unit factors ------------------------------------------------
+
+constexpr int kMixThreads = 128;
+constexpr int kMixTokens = 32;
+
+// Grid: blocks of tokens, blocks of channels (8 per thread; those of k and q cover whole heads) and one for the
+// steps, requests.  TAPS 0: any number of them.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(kMixThreads)
+mix_kernel(const Recurrence a, int v_blocks, int heads_per_block) {
+    __shared__ float s_part[kMixTokens][kMixThreads];
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int b = blockIdx.z, begin = a.qo_indptr[b], ext = a.qo_indptr[b + 1] - begin;
+    const int t0 = blockIdx.x * kMixTokens;
+    if (t0 >= ext) return;
+    const int n = min(kMixTokens, ext - t0);
+    const T* joint = static_cast<const T*>(a.joint) + static_cast<int64_t>(begin) * a.joint_ld;
+    if (blockIdx.y == gridDim.y - 1) {
+        for (int i = threadIdx.x; i < n * a.heads; i += kMixThreads) {
+            const int t = t0 + i / a.heads, h = i % a.heads;
+            reinterpret_cast<float2*>(a.steps)[static_cast<int64_t>(begin + t) * a.heads + h] = step_of(a, joint + t * a.joint_ld, h);
+        }
+        return;
+    }
+    const int64_t nv = values(a), nc = channels(a);
+    const bool heads = static_cast<int>(blockIdx.y) >= v_blocks;
+    const int per_head = a.padded_dim >> 3, head0 = (static_cast<int>(blockIdx.y) - v_blocks) * heads_per_block;
+    int64_t c;
+    bool active;
+    if (heads) {
+        const int head = static_cast<int>(threadIdx.x) / per_head;
+        active = head < heads_per_block && head0 + head < 2 * a.kv_heads;
+        c = nv + static_cast<int64_t>(head0) * a.padded_dim + threadIdx.x * 8;
+    } else {
+        c = (static_cast<int64_t>(blockIdx.y) * kMixThreads + threadIdx.x) * 8;
+        active = c < nv;
+    }
+    const int taps = TAPS > 0 ? TAPS : a.taps, cached = a.cached[b];
+    T* ring = static_cast<T*>(a.conv_state) + static_cast<int64_t>(a.table_idx[b]) * taps * nc + c;
+    const T* in = joint + nv + c;
+    // the input of token r of this step, or of one before it
+    auto input = [&](int r) {
+        if (r >= 0) return load8(in + r * a.joint_ld);
+        Vec8 x;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x.v[j] = 0.f;
+        return cached + r >= 0 ? load8(ring + (cached + r) % taps * nc) : x;
+    };
+    if (active) {
+        constexpr int kWindow = TAPS > 0 ? TAPS : 1;
+        Vec8 w[kWindow], x[kWindow], bias;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) bias.v[j] = 0.f;
+        if (a.conv_bias != nullptr) bias = load8(a.conv_bias + c);
+        if (TAPS > 0) {
+#pragma unroll
+            for (int i = 0; i < kWindow; ++i) {
+                w[i] = load8(a.conv + i * nc + c);
+                if (i + 1 < kWindow) x[i + 1] = input(t0 - (kWindow - 1) + i);
+            }
+        }
+        T* out = static_cast<T*>(a.mixed) + static_cast<int64_t>(begin) * nc + c;
+        for (int t = t0; t < t0 + n; ++t) {
+            Vec8 y = bias;
+            if (TAPS > 0) {
+#pragma unroll
+                for (int i = 0; i + 1 < kWindow; ++i) x[i] = x[i + 1];
+                x[kWindow - 1] = load8(in + t * a.joint_ld);
+#pragma unroll
+                for (int i = 0; i < kWindow; ++i)
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) y.v[j] = fmaf(w[i].v[j], x[i].v[j], y.v[j]);
+            } else {
+                for (int i = 0; i < taps; ++i) {
+                    const Vec8 wi = load8(a.conv + i * nc + c), xi = input(t - (taps - 1) + i);
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) y.v[j] = fmaf(wi.v[j], xi.v[j], y.v[j]);
+                }
+            }
+            float ss = 0.f;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                y.v[j] = to_f32(from_f32<T>(silu<T>(y.v[j])));
+                ss += y.v[j] * y.v[j];
+            }
+            store8(out + t * nc, y);
+            s_part[t - t0][threadIdx.x] = ss;
+        }
+        // (a request's first block is the only one that reads the ring)
+        if (blockIdx.x == 0)
+            for (int r = max(0, ext - (taps - 1)); r < ext; ++r) store8(ring + (cached + r) % taps * nc, load8(in + r * a.joint_ld));
+    }
+    if (!heads || a.rule != kDelta) return;
+    __syncthreads();
+    const int here = min(heads_per_block, 2 * a.kv_heads - head0);
+    for (int i = threadIdx.x; i < n * here; i += kMixThreads) {
+        const int t = i / here, head = i - t * here;
+        float ss = 0.f;
+        for (int j = 0; j < per_head; ++j) ss += s_part[t][head * per_head + j];
+        float f = 1.f / sqrtf(ss + kUnitEps);
+        if (head0 + head >= a.kv_heads) f /= sqrtf(static_cast<float>(a.dim));
+        a.units[static_cast<int64_t>(begin + t0 + t) * 2 * a.kv_heads + head0 + head] = f;
+    }
+}
+
+// ---- token by token: decode, and prompts that the chunked kernels do not take ------------
+
+constexpr int kStepThreads = 256;
+constexpr int kAhead = 16;   // state rows per thread, in registers
+
+// Grid: heads, requests, blocks of 4 << log_cols value columns.
+template <typename T, int RULE, bool DECODE>
+__global__ void __launch_bounds__(kStepThreads)
+step_kernel(const Recurrence a, int log_cols, bool finish) {
+    extern __shared__ __align__(16) float smem[];
+    __shared__ float s_ss[kStepThreads / 32];
+    const int dk = a.padded_dim, vp = a.padded_value_dim;
+    const int nv4 = 1 << log_cols, cols = nv4 * 4, groups = kStepThreads >> log_cols;
+    float *s_v = smem, *s_k = s_v + cols, *s_q = s_k + dk, *s_red = s_q + dk, *s_o = s_red + kStepThreads * 4;
+    const int h = blockIdx.x, b = blockIdx.y, col0 = blockIdx.z * cols;
+    const int kvh = h / (a.heads / a.kv_heads);
+    const int group = threadIdx.x >> log_cols, col = (threadIdx.x & (nv4 - 1)) * 4;
+    const bool active = col0 + col < vp;
+    const int64_t nv = values(a), nc = channels(a);
+    float* state = a.state + (static_cast<int64_t>(a.table_idx[b]) * a.heads + h) * dk * vp + col0 + col;
+    const int cached = a.cached[b];
+    pdl_launch_dependents();
+    float4 x[kAhead];
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) {
+        const int r = group + i * groups;
+        x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (active && cached > 0 && r < dk) x[i] = load4(state + static_cast<int64_t>(r) * vp);
+    }
+    // this CTA's channels: its value columns, the head's k and q
+    const int own_v = min(cols, vp - col0), own = own_v + 2 * dk;
+    auto channel = [&](int i) -> int64_t {
+        if (i < own_v) return static_cast<int64_t>(h) * vp + col0 + i;
+        i -= own_v;
+        return nv + (i < dk ? static_cast<int64_t>(kvh) * dk + i : static_cast<int64_t>(a.kv_heads + kvh) * dk + i - dk);
+    };
+    auto place = [&](int i) -> float& { return i < own_v ? s_v[i] : s_k[i - own_v]; };   // (s_q follows s_k)
+    T* ring = static_cast<T*>(a.conv_state) + static_cast<int64_t>(a.table_idx[b]) * a.taps * nc;
+    if (DECODE) {
+        for (int i = threadIdx.x; i < own; i += kStepThreads) {
+            const int64_t c = channel(i);
+            float y = a.conv_bias != nullptr ? a.conv_bias[c] : 0.f;
+            for (int j = 0; j + 1 < a.taps; ++j) {
+                const int pos = cached - (a.taps - 1) + j;
+                if (pos >= 0) y = fmaf(a.conv[j * nc + c], to_f32(ring[pos % a.taps * nc + c]), y);
+            }
+            place(i) = y;
+        }
+    }
+    pdl_wait_prior();
+    const int begin = DECODE ? b : a.qo_indptr[b], end = DECODE ? b + 1 : a.qo_indptr[b + 1];
+    const float skip = RULE == kStateSpace ? a.skip[h] : 0.f;
+    for (int64_t t = begin; t < end; ++t) {
+        const T* row = static_cast<const T*>(a.joint) + t * a.joint_ld;
+        float2 step;
+        if (DECODE) {
+            T* now = ring + static_cast<int64_t>(cached % a.taps) * nc;
+            const bool keeps = h % (a.heads / a.kv_heads) == 0 && blockIdx.z == 0;   // k and q are shared
+            for (int i = threadIdx.x; i < own; i += kStepThreads) {
+                const int64_t c = channel(i);
+                const T in = row[nv + c];
+                place(i) = to_f32(from_f32<T>(silu<T>(fmaf(a.conv[(a.taps - 1) * nc + c], to_f32(in), place(i)))));
+                if (i < own_v || keeps) now[c] = in;
+            }
+            step = step_of(a, row, h);
+        } else {
+            const T* mixed = static_cast<const T*>(a.mixed) + t * nc;
+            for (int i = threadIdx.x; i < own; i += kStepThreads) place(i) = to_f32(mixed[channel(i)]);
+            step = reinterpret_cast<const float2*>(a.steps)[t * a.heads + h];
+        }
+        __syncthreads();
+        float kf = step.y, qf = 1.f;   // factors of k and q
+        const float g = exp2f(step.x);
+        if (RULE == kDelta) {
+            if (DECODE) {
+                const int lane = threadIdx.x & 31;
+                float sk = 0.f, sq = 0.f;
+                for (int i = lane; i < dk; i += 32) {
+                    sk += s_k[i] * s_k[i];
+                    sq += s_q[i] * s_q[i];
+                }
+                kf = 1.f / sqrtf(warp_sum(sk) + kUnitEps);
+                qf = 1.f / sqrtf(warp_sum(sq) + kUnitEps) / sqrtf(static_cast<float>(a.dim));
+            } else {
+                kf = a.units[t * 2 * a.kv_heads + kvh];
+                qf = a.units[t * 2 * a.kv_heads + a.kv_heads + kvh];
+            }
+        }
+        float4 u = active ? *reinterpret_cast<const float4*>(s_v + col) : make_float4(0.f, 0.f, 0.f, 0.f);
+        if (RULE == kDelta) {
+            float4 p = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int i = 0; i < kAhead; ++i) {
+                const int r = group + i * groups;
+                if (r < dk) {
+                    const float k = s_k[r];
+                    p.x = fmaf(k, x[i].x, p.x);
+                    p.y = fmaf(k, x[i].y, p.y);
+                    p.z = fmaf(k, x[i].z, p.z);
+                    p.w = fmaf(k, x[i].w, p.w);
+                }
+            }
+            *reinterpret_cast<float4*>(s_red + group * cols + col) = p;
+            __syncthreads();
+            p = make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int i = 0; i < groups; ++i) {
+                const float4 y = load4(s_red + i * cols + col);
+                p.x += y.x;
+                p.y += y.y;
+                p.z += y.z;
+                p.w += y.w;
+            }
+            const float f = g * kf;
+            u = make_float4(step.y * (u.x - f * p.x), step.y * (u.y - f * p.y), step.y * (u.z - f * p.z), step.y * (u.w - f * p.w));
+            __syncthreads();
+        }
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < kAhead; ++i) {
+            const int r = group + i * groups;
+            if (r < dk) {
+                const float k = kf * s_k[r], q = s_q[r];
+                x[i].x = fmaf(k, u.x, g * x[i].x);
+                x[i].y = fmaf(k, u.y, g * x[i].y);
+                x[i].z = fmaf(k, u.z, g * x[i].z);
+                x[i].w = fmaf(k, u.w, g * x[i].w);
+                o.x = fmaf(q, x[i].x, o.x);
+                o.y = fmaf(q, x[i].y, o.y);
+                o.z = fmaf(q, x[i].z, o.z);
+                o.w = fmaf(q, x[i].w, o.w);
+                if (DECODE && active) *reinterpret_cast<float4*>(state + static_cast<int64_t>(r) * vp) = x[i];
+            }
+        }
+        *reinterpret_cast<float4*>(s_red + group * cols + col) = o;
+        __syncthreads();
+        T* out = static_cast<T*>(a.out) + t * a.out_ld + static_cast<int64_t>(h) * vp + col0;
+        float ss = 0.f;
+        for (int c = threadIdx.x; c < own_v; c += kStepThreads) {
+            float y = 0.f;
+            for (int i = 0; i < groups; ++i) y += s_red[i * cols + c];
+            y *= qf;
+            if (RULE == kStateSpace) y = fmaf(skip, s_v[c], y);
+            if (!finish) out[c] = from_f32<T>(y);
+            s_o[c] = y;
+            ss += y * y;
+        }
+        if (finish) {   // the whole head is here: norm and gate
+            const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+            ss = warp_sum(ss);
+            if (lane == 0) s_ss[warp] = ss;
+            __syncthreads();
+            ss = warp_sum(lane < kStepThreads / 32 ? s_ss[lane] : 0.f);
+            const float scale = rsqrtf(ss / static_cast<float>(a.value_dim) + a.eps) * a.out_scale;
+            for (int c = threadIdx.x; c < own_v; c += kStepThreads)
+                out[c] = from_f32<T>(s_o[c] * scale * to_f32(static_cast<const T*>(a.norm)[c]) *
+                                     silu<T>(to_f32(row[static_cast<int64_t>(h) * vp + c])));
+        }
+        if (!DECODE) __syncthreads();   // everything in shared memory has been used
+    }
+    if (DECODE || !active || begin >= end) return;
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) {
+        const int r = group + i * groups;
+        if (r < dk) *reinterpret_cast<float4*>(state + static_cast<int64_t>(r) * vp) = x[i];
+    }
+}
+
+// ---- norm and gate of raw outputs, in place ------------------------------------------------
+
+// Delta rule: one warp per (token, head).
+constexpr int kFinishWarps = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(kFinishWarps * 32)
+finish_heads_kernel(const Recurrence a) {
+    const int lane = threadIdx.x & 31, vp = a.padded_value_dim;
+    const unsigned row = blockIdx.x * kFinishWarps + (threadIdx.x >> 5);
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    if (row >= static_cast<unsigned>(a.tokens) * a.heads) return;
+    const int64_t t = row / a.heads;
+    const int h = static_cast<int>(row - t * a.heads);
+    T* out = static_cast<T*>(a.out) + t * a.out_ld + static_cast<int64_t>(h) * vp;
+    const T* gate = static_cast<const T*>(a.joint) + t * a.joint_ld + static_cast<int64_t>(h) * vp;
+    const T* norm = static_cast<const T*>(a.norm);
+    float ss = 0.f;
+    for (int c = lane * 8; c < vp; c += 256) {
+        const Vec8 o = load8(out + c);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ss += o.v[j] * o.v[j];
+    }
+    const float scale = rsqrtf(warp_sum(ss) / static_cast<float>(a.value_dim) + a.eps) * a.out_scale;
+    for (int c = lane * 8; c < vp; c += 256) {
+        Vec8 o = load8(out + c);
+        const Vec8 g = load8(gate + c), w = load8(norm + c);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) o.v[j] *= scale * w.v[j] * silu<T>(g.v[j]);
+        store8(out + c, o);
+    }
+}
+
+// State space: one CTA per (token, part of the norm).  A part is a run of the concatenated heads without their
+// padding, so it may begin and end inside one; VEC elements at a time.
+constexpr int kPartThreads = 128;
+constexpr int kPartKeep = 4;   // pieces of VEC elements a thread keeps in registers
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kPartThreads)
+finish_parts_kernel(const Recurrence a) {
+    __shared__ float red[kPartThreads / 32];
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int64_t t = blockIdx.x;
+    const int per = a.heads * a.value_dim / a.norm_groups, from = blockIdx.y * per;
+    T* out = static_cast<T*>(a.out) + t * a.out_ld;
+    const T* gate = static_cast<const T*>(a.joint) + t * a.joint_ld;
+    const T* norm = static_cast<const T*>(a.norm);
+    auto place = [&](int i) { return (from + i) / a.value_dim * a.padded_value_dim + (from + i) % a.value_dim; };
+    auto gated = [&](int at, float (&y)[VEC]) {
+        if (VEC == 8) {
+            const Vec8 o = load8(out + at), z = load8(gate + at);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) y[j] = o.v[j & 7] * silu<T>(z.v[j & 7]);
+        } else {
+            y[0] = to_f32(out[at]) * silu<T>(to_f32(gate[at]));
+        }
+    };
+    float kept[kPartKeep][VEC], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kPartKeep; ++i) {
+        const int e = (threadIdx.x + i * kPartThreads) * VEC;
+        if (e >= per) continue;
+        gated(place(e), kept[i]);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) ss += kept[i][j] * kept[i][j];
+    }
+    for (int e = (threadIdx.x + kPartKeep * kPartThreads) * VEC; e < per; e += kPartThreads * VEC) {
+        float y[VEC];
+        gated(place(e), y);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) ss += y[j] * y[j];
+    }
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    ss = warp_sum(ss);
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    ss = warp_sum(lane < kPartThreads / 32 ? red[lane] : 0.f);
+    const float scale = rsqrtf(ss / static_cast<float>(per) + a.eps) * a.out_scale;
+    auto emit = [&](int at, const float (&y)[VEC]) {
+        if (VEC == 8) {
+            const Vec8 w = load8(norm + at);
+            Vec8 o;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) o.v[j] = y[j % VEC] * scale * w.v[j];
+            store8(out + at, o);
+        } else {
+            out[at] = from_f32<T>(y[0] * scale * to_f32(norm[at]));
+        }
+    };
+#pragma unroll
+    for (int i = 0; i < kPartKeep; ++i) {
+        const int e = (threadIdx.x + i * kPartThreads) * VEC;
+        if (e < per) emit(place(e), kept[i]);
+    }
+    for (int e = (threadIdx.x + kPartKeep * kPartThreads) * VEC; e < per; e += kPartThreads * VEC) {
+        float y[VEC];
+        gated(place(e), y);
+        emit(place(e), y);
+    }
+}
+
+// ---- chunked ---------------------------------------------------------------------------------
+
+constexpr int kChunk = 64;            // tokens per chunk
+constexpr int kSlice = 64;            // value columns per CTA
+constexpr int kPad = 8;               // bf16 elements behind every shared row (conflict-free ldmatrix)
+constexpr int kTiles = 10;            // 16 x 16 tiles on and below the diagonal
+constexpr int kMatrixVecs = kTiles * 2 * 32;   // uint4 per matrix: [tile][upper / lower part][lane]
+
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid) {
+    const int bytes = valid ? 16 : 0;   // 0: the 16 bytes are filled with zeros
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+// x as the sum of two bf16 numbers.
+__device__ __forceinline__ void split2(float x0, float x1, uint32_t& hi, uint32_t& lo) {
+    hi = pack_bf16(x0, x1);
+    lo = pack_bf16(x0 - bf16_lo(hi), x1 - bf16_hi(hi));
+}
+// Chunk i of request b, which brings the tokens from `begin` on: numbers that no two requests share.
+__device__ __forceinline__ int64_t chunk_number(int begin, int b, int i) { return begin / kChunk + b + i; }
+
+// Sums of a chunk's decay logarithms over its tokens: the calling warp's lane holds those of tokens 2 lane and
+// 2 lane + 1.
+__device__ __forceinline__ float2 running_sums(float2 x) {
+    const int lane = threadIdx.x & 31;
+    float s = x.x + x.y;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const float up = __shfl_up_sync(0xffffffffu, s, o);
+        if (lane >= o) s += up;
+    }
+    return make_float2(s - x.y, s);
+}
+
+constexpr int kPrepareThreads = 128;
+constexpr int kARow = kChunk + 4;
+struct PrepareSmem {
+    union {
+        struct {
+            __nv_bfloat16 k[kChunk * (64 + kPad)], q[kChunk * (64 + kPad)];   // 64 columns at a time
+        };
+        float a[2][kChunk * kARow];   // two heads' A, then their inverses
+    };
+    float sum[2][kChunk], weight[2][kChunk], kf[kChunk], qf[kChunk];
+};
+
+// The columns of (I + A)^-1 from BASE on, one per lane, by forward substitution; those before it are zero in rows
+// below BASE.
+template <int BASE>
+__device__ __forceinline__ void invert_columns(float* a) {
+    const int lane = threadIdx.x & 31;
+    float x[kChunk];
+#pragma unroll
+    for (int i = BASE; i < kChunk; ++i) {
+        float acc[4] = {i == BASE + lane ? 1.f : 0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int s = BASE; s < i; s += 4) {
+            const float4 r = load4(a + i * kARow + s);
+            acc[0] = fmaf(-r.x, x[s], acc[0]);
+            if (s + 1 < i) acc[1] = fmaf(-r.y, x[s + 1], acc[1]);
+            if (s + 2 < i) acc[2] = fmaf(-r.z, x[s + 2], acc[2]);
+            if (s + 3 < i) acc[3] = fmaf(-r.w, x[s + 3], acc[3]);
+        }
+        x[i] = (acc[0] + acc[1]) + (acc[2] + acc[3]);
+    }
+    const int pair = 1 + (static_cast<int>(threadIdx.x) >> 6);
+    asm volatile("bar.sync %0, 64;" ::"r"(pair) : "memory");   // both warps have read A
+#pragma unroll
+    for (int i = 0; i < kChunk; ++i) a[i * kARow + BASE + lane] = i < BASE ? 0.f : x[i < BASE ? BASE : i];
+    asm volatile("bar.sync %0, 64;" ::"r"(pair) : "memory");
+}
+
+// Grid: chunks of the longest request, k / q heads, requests.
+template <int RULE>
+__global__ void __launch_bounds__(kPrepareThreads)
+prepare_kernel(const Recurrence a) {
+    extern __shared__ __align__(16) uint8_t smem_raw[];
+    PrepareSmem& S = *reinterpret_cast<PrepareSmem*>(smem_raw);
+    constexpr int ROW = 64 + kPad, kMatrices = RULE == kDelta ? 2 : 1;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int g = lane >> 2, tq = lane & 3, mi = lane >> 3, r8 = lane & 7;
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int b = blockIdx.z, kvh = blockIdx.y, begin = a.qo_indptr[b], ext = a.qo_indptr[b + 1] - begin;
+    const int s0 = blockIdx.x * kChunk;
+    if (s0 >= ext) return;
+    const int n = min(kChunk, ext - s0);
+    const int64_t nc = channels(a), first = begin + s0;
+    const __nv_bfloat16* k0 = static_cast<const __nv_bfloat16*>(a.mixed) + first * nc + values(a) + static_cast<int64_t>(kvh) * a.padded_dim;
+    const int64_t to_q = static_cast<int64_t>(a.kv_heads) * a.padded_dim;
+    if (threadIdx.x < kChunk) {
+        float kf = 1.f, qf = 1.f;
+        if (RULE == kDelta && threadIdx.x < n) {
+            kf = a.units[(first + threadIdx.x) * 2 * a.kv_heads + kvh];
+            qf = a.units[(first + threadIdx.x) * 2 * a.kv_heads + a.kv_heads + kvh];
+        }
+        S.kf[threadIdx.x] = kf;
+        S.qf[threadIdx.x] = qf;
+    }
+    // ---- k . k and q . k of this warp's 16 rows ----
+    float kk[8][4] = {}, qk[8][4] = {};
+    for (int d0 = 0; d0 < a.padded_dim; d0 += 64) {
+        if (d0 > 0) __syncthreads();
+        for (int i = threadIdx.x; i < kChunk * 8; i += kPrepareThreads) {
+            const int t = i >> 3, c = (i & 7) * 8;
+            const __nv_bfloat16* row = k0 + (t < n ? t : 0) * nc + d0 + c;
+            cp_async16(smem_u32(&S.k[t * ROW + c]), row, t < n);
+            cp_async16(smem_u32(&S.q[t * ROW + c]), row + to_q, t < n);
+        }
+        cp_async_wait_all();
+        __syncthreads();
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) {
+            uint32_t ak[4], aq[4], b0, b1, b2, b3;
+            const int aoff = (warp * 16 + (mi & 1) * 8 + r8) * ROW + ks * 16 + (mi >> 1) * 8;
+            ldmatrix_x4(smem_u32(&S.q[aoff]), aq[0], aq[1], aq[2], aq[3]);
+            if (RULE == kDelta) ldmatrix_x4(smem_u32(&S.k[aoff]), ak[0], ak[1], ak[2], ak[3]);
+#pragma unroll
+            for (int kt = 0; kt < 4; ++kt) {
+                if (kt > warp) continue;
+                ldmatrix_x4(smem_u32(&S.k[(kt * 16 + (mi >> 1) * 8 + r8) * ROW + ks * 16 + (mi & 1) * 8]), b0, b1, b2, b3);
+                mma_bf16_16816(qk[2 * kt], aq, b0, b1);
+                mma_bf16_16816(qk[2 * kt + 1], aq, b2, b3);
+                if (RULE == kDelta) {
+                    mma_bf16_16816(kk[2 * kt], ak, b0, b1);
+                    mma_bf16_16816(kk[2 * kt + 1], ak, b2, b3);
+                }
+            }
+        }
+    }
+    // ---- per head: P and, two heads at a time, the inverse ----
+    const int group = a.heads / a.kv_heads;
+    uint4* chunks = static_cast<uint4*>(a.chunks) + chunk_number(begin, b, blockIdx.x) * a.heads * kMatrices * kMatrixVecs;
+    for (int h0 = 0; h0 < group; h0 += 2) {
+        __syncthreads();
+        if ((warp & 1) == 0 && h0 + (warp >> 1) < group) {
+            const int h = kvh * group + h0 + (warp >> 1);
+            const float2* steps = reinterpret_cast<const float2*>(a.steps) + first * a.heads + h;
+            const float2 none = make_float2(0.f, 0.f);
+            const float2 x = 2 * lane < n ? steps[static_cast<int64_t>(2 * lane) * a.heads] : none;
+            const float2 y = 2 * lane + 1 < n ? steps[static_cast<int64_t>(2 * lane + 1) * a.heads] : none;
+            *reinterpret_cast<float2*>(&S.sum[warp >> 1][2 * lane]) = running_sums(make_float2(x.x, y.x));
+            *reinterpret_cast<float2*>(&S.weight[warp >> 1][2 * lane]) = make_float2(x.y, y.y);
+        }
+        __syncthreads();
+#pragma unroll
+        for (int hp = 0; hp < 2; ++hp) {
+            if (h0 + hp >= group) continue;
+            uint4* out = chunks + (static_cast<int64_t>(kvh * group + h0 + hp) * kMatrices) * kMatrixVecs + lane;
+            const float* sum = S.sum[hp];
+            const float* weight = S.weight[hp];
+#pragma unroll
+            for (int kt = 0; kt < 4; ++kt) {
+                if (kt > warp) continue;
+                uint32_t hi[4], lo[4];
+#pragma unroll
+                for (int part = 0; part < 4; ++part) {   // rows g, g + 8 of the left tile, then of the right one
+                    const int t = warp * 16 + g + (part & 1) * 8, s = kt * 16 + (part >> 1) * 8 + 2 * tq;
+                    const float* src = qk[2 * kt + (part >> 1)] + (part & 1) * 2;
+                    float p[2];
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        const float ratio = s + e <= t ? ex2(sum[t] - sum[s + e]) : 0.f;
+                        p[e] = src[e] * ratio * (RULE == kDelta ? S.qf[t] * S.kf[s + e] : weight[s + e]);
+                        if (RULE == kDelta)
+                            S.a[hp][t * kARow + s + e] = s + e < t ? kk[2 * kt + (part >> 1)][(part & 1) * 2 + e] * ratio *
+                                                                         (S.kf[t] * S.kf[s + e]) * weight[t]
+                                                                   : 0.f;
+                    }
+                    split2(p[0], p[1], hi[part], lo[part]);
+                }
+                const int tile = warp * (warp + 1) / 2 + kt;
+                out[tile * 64] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                out[tile * 64 + 32] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            }
+        }
+        if (RULE != kDelta) continue;
+        __syncthreads();
+        const int hp = warp >> 1;
+        if (h0 + hp >= group) continue;   // (both warps of the pair)
+        float* m = S.a[hp];
+        if ((warp & 1) == 0) invert_columns<0>(m);
+        else invert_columns<32>(m);
+        uint4* out = chunks + (static_cast<int64_t>(kvh * group + h0 + hp) * kMatrices + 1) * kMatrixVecs + lane;
+        // tiles of the pair's warps: rows 0 and 3, rows 1 and 2
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int mt = (warp & 1) == 0 ? i * 3 : 1 + i;
+            for (int kt = 0; kt <= mt; ++kt) {
+                uint32_t hi[4], lo[4];
+#pragma unroll
+                for (int part = 0; part < 4; ++part) {
+                    const float2 v = *reinterpret_cast<const float2*>(m + (mt * 16 + g + (part & 1) * 8) * kARow + kt * 16 +
+                                                                      (part >> 1) * 8 + 2 * tq);
+                    split2(v.x, v.y, hi[part], lo[part]);
+                }
+                const int tile = mt * (mt + 1) / 2 + kt;
+                out[tile * 64] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                out[tile * 64 + 32] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            }
+        }
+    }
+}
+
+constexpr int kWalkThreads = 256;
+
+template <int DK, int RULE>
+struct WalkSmem {
+    static constexpr int kRow = DK + kPad, kVRow = kSlice + kPad;
+    __nv_bfloat16 k[2][kChunk * kRow], q[2][kChunk * kRow], v[2][kChunk * kVRow];   // this chunk's and the next one's
+    __nv_bfloat16 sh[DK * kVRow], sl[DK * kVRow];                                   // the state
+    __nv_bfloat16 rh[RULE == kDelta ? kChunk * kVRow : 8], rl[RULE == kDelta ? kChunk * kVRow : 8];   // beta (V - G K S)
+    __nv_bfloat16 uh[RULE == kDelta ? kChunk * kVRow : 8], ul[RULE == kDelta ? kChunk * kVRow : 8];   // U
+    __nv_bfloat16 wh[kChunk * kVRow], wl[kChunk * kVRow];                           // U as it enters the state
+    float out[2][kChunk];      // G_t times q's factor
+    float beta[2][kChunk], read[2][kChunk];   // beta_t; beta_t G_t times k's factor
+    float write[2][kChunk];    // exp(B_n - B_t) times k's factor (or times dt)
+    float keep[2];             // G_n
+};
+
+// Grid: slices of 64 value columns, heads, requests.
+template <int DK, int RULE>
+__global__ void __launch_bounds__(kWalkThreads, 1)
+chunk_kernel(const Recurrence a) {
+    using Smem = WalkSmem<DK, RULE>;
+    constexpr int ROW = Smem::kRow, VROW = Smem::kVRow, kMatrices = RULE == kDelta ? 2 : 1;
+    constexpr int kColSplit = 128 / DK;                  // warps that share 16 state rows
+    constexpr int kStateTiles = kSlice / 8 / kColSplit;  // 8-column tiles of state per warp
+    extern __shared__ __align__(16) uint8_t smem_raw[];
+    Smem& S = *reinterpret_cast<Smem*>(smem_raw);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int g = lane >> 2, tq = lane & 3, mi = lane >> 3, r8 = lane & 7;
+    const int h = blockIdx.y, req = blockIdx.z, v0 = blockIdx.x * kSlice;
+    const int vp = a.padded_value_dim, kvh = h / (a.heads / a.kv_heads);
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int begin = a.qo_indptr[req], ext = a.qo_indptr[req + 1] - begin;
+    if (ext <= 0) return;
+    const int64_t nc = channels(a);
+    const __nv_bfloat16* mixed = static_cast<const __nv_bfloat16*>(a.mixed) + begin * nc;
+    const int64_t at_k = values(a) + static_cast<int64_t>(kvh) * DK, to_q = static_cast<int64_t>(a.kv_heads) * DK;
+    const int64_t at_v = static_cast<int64_t>(h) * vp + v0;
+
+    auto load_chunk = [&](int s0, int buf) {
+        const int n = min(kChunk, ext - s0);
+        for (int i = threadIdx.x; i < kChunk * (DK / 8); i += kWalkThreads) {
+            const int t = i / (DK / 8), c = (i % (DK / 8)) * 8;
+            const __nv_bfloat16* row = mixed + static_cast<int64_t>(t < n ? s0 + t : s0) * nc + at_k + c;
+            cp_async16(smem_u32(&S.k[buf][t * ROW + c]), row, t < n);
+            cp_async16(smem_u32(&S.q[buf][t * ROW + c]), row + to_q, t < n);
+        }
+        for (int i = threadIdx.x; i < kChunk * (kSlice / 8); i += kWalkThreads) {
+            const int t = i / (kSlice / 8), c = (i % (kSlice / 8)) * 8;
+            cp_async16(smem_u32(&S.v[buf][t * VROW + c]), mixed + static_cast<int64_t>(t < n ? s0 + t : s0) * nc + at_v + c, t < n);
+        }
+    };
+    // Factors of a chunk's tokens: the first warp fetches them a chunk ahead and works them out behind it.
+    float2 st0, st1, un0, un1;
+    auto fetch_factors = [&](int s0) {
+        const int n = min(kChunk, ext - s0);
+        const float2* steps = reinterpret_cast<const float2*>(a.steps) + static_cast<int64_t>(begin + s0) * a.heads + h;
+        st0 = st1 = make_float2(0.f, 0.f);
+        un0 = un1 = make_float2(1.f, 1.f);
+        auto unit = [&](int t) {
+            const float* u = a.units + static_cast<int64_t>(begin + s0 + t) * 2 * a.kv_heads + kvh;
+            return make_float2(u[0], u[a.kv_heads]);
+        };
+        if (2 * lane < n) {
+            st0 = steps[static_cast<int64_t>(2 * lane) * a.heads];
+            if (RULE == kDelta) un0 = unit(2 * lane);
+        }
+        if (2 * lane + 1 < n) {
+            st1 = steps[static_cast<int64_t>(2 * lane + 1) * a.heads];
+            if (RULE == kDelta) un1 = unit(2 * lane + 1);
+        }
+    };
+    auto put_factors = [&](int buf) {
+        const float2 B = running_sums(make_float2(st0.x, st1.x));
+        const float last = __shfl_sync(0xffffffffu, B.y, 31);
+        const float g0 = ex2(B.x), g1 = ex2(B.y), w0 = ex2(last - B.x), w1 = ex2(last - B.y);
+        *reinterpret_cast<float2*>(&S.out[buf][2 * lane]) = make_float2(g0 * un0.y, g1 * un1.y);
+        if (RULE == kDelta) {
+            *reinterpret_cast<float2*>(&S.beta[buf][2 * lane]) = make_float2(st0.y, st1.y);
+            *reinterpret_cast<float2*>(&S.read[buf][2 * lane]) = make_float2(st0.y * g0 * un0.x, st1.y * g1 * un1.x);
+            *reinterpret_cast<float2*>(&S.write[buf][2 * lane]) = make_float2(w0 * un0.x, w1 * un1.x);
+        } else {
+            *reinterpret_cast<float2*>(&S.write[buf][2 * lane]) = make_float2(w0 * st0.y, w1 * st1.y);
+        }
+        if (lane == 0) S.keep[buf] = ex2(last);
+    };
+    load_chunk(0, 0);
+
+    // This warp's part of the state: 16 rows from row0, kStateTiles tiles of 8 columns from col0, in the layout of an
+    // MMA accumulator.
+    const int row0 = warp / kColSplit * 16, col0 = warp % kColSplit * (kSlice / kColSplit);
+    float* state = a.state + (static_cast<int64_t>(a.table_idx[req]) * a.heads + h) * DK * vp + v0;
+    float st[kStateTiles][4];
+    const bool fresh = a.cached[req] == 0;
+    auto put_state = [&]() {
+#pragma unroll
+        for (int j = 0; j < kStateTiles; ++j)
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                uint32_t hi, lo;
+                split2(st[j][2 * half], st[j][2 * half + 1], hi, lo);
+                const int at = (row0 + g + half * 8) * VROW + col0 + j * 8 + 2 * tq;
+                *reinterpret_cast<uint32_t*>(&S.sh[at]) = hi;
+                *reinterpret_cast<uint32_t*>(&S.sl[at]) = lo;
+            }
+    };
+#pragma unroll
+    for (int j = 0; j < kStateTiles; ++j)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const float2 x = fresh ? make_float2(0.f, 0.f)
+                                   : *reinterpret_cast<const float2*>(state + static_cast<int64_t>(row0 + g + half * 8) * vp + col0 +
+                                                                      j * 8 + 2 * tq);
+            st[j][2 * half] = x.x;
+            st[j][2 * half + 1] = x.y;
+        }
+    put_state();
+    if (warp == 0) {
+        fetch_factors(0);
+        put_factors(0);
+    }
+    // 16 tokens x 32 columns of the products per warp; the two warps of a scheduler share out the triangle evenly
+    const int mt = warp < 4 ? warp : 7 - warp, oc0 = (warp >> 2) * 32;
+    const float skip = RULE == kStateSpace ? a.skip[h] : 0.f;
+    const uint4* chunks = static_cast<const uint4*>(a.chunks) +
+                          (chunk_number(begin, req, 0) * a.heads + h) * kMatrices * kMatrixVecs + mt * (mt + 1) / 2 * 64 + lane;
+    const int64_t chunk_vecs = static_cast<int64_t>(a.heads) * kMatrices * kMatrixVecs;
+
+    // acc += M X for this warp's rows: M's tiles from memory, X [kChunk][kSlice] in shared memory as one or two parts
+    auto load_matrix = [&](const uint4* m, uint4 (&hi)[4], uint4 (&lo)[4]) {
+#pragma unroll
+        for (int kt = 0; kt < 4; ++kt)
+            if (kt <= mt) {
+                hi[kt] = __ldg(m + kt * 64);
+                lo[kt] = __ldg(m + kt * 64 + 32);
+            }
+    };
+    auto multiply = [&](float (&acc)[4][4], const uint4 (&hi)[4], const uint4 (&lo)[4], const __nv_bfloat16* xh, const __nv_bfloat16* xl) {
+#pragma unroll
+        for (int kt = 0; kt < 4; ++kt) {
+            if (kt > mt) continue;
+            const uint32_t ah[4] = {hi[kt].x, hi[kt].y, hi[kt].z, hi[kt].w}, al[4] = {lo[kt].x, lo[kt].y, lo[kt].z, lo[kt].w};
+#pragma unroll
+            for (int np = 0; np < 2; ++np) {
+                const int off = (kt * 16 + (mi & 1) * 8 + r8) * VROW + oc0 + np * 16 + (mi >> 1) * 8;
+                uint32_t b0, b1, b2, b3;
+                ldmatrix_x4_trans(smem_u32(xh + off), b0, b1, b2, b3);
+                mma_bf16_16816(acc[2 * np], ah, b0, b1);
+                mma_bf16_16816(acc[2 * np + 1], ah, b2, b3);
+                mma_bf16_16816(acc[2 * np], al, b0, b1);
+                mma_bf16_16816(acc[2 * np + 1], al, b2, b3);
+                if (xl != nullptr) {
+                    ldmatrix_x4_trans(smem_u32(xl + off), b0, b1, b2, b3);
+                    mma_bf16_16816(acc[2 * np], ah, b0, b1);
+                    mma_bf16_16816(acc[2 * np + 1], ah, b2, b3);
+                }
+            }
+        }
+    };
+
+    int buf = 0;
+    for (int s0 = 0; s0 < ext; s0 += kChunk, buf ^= 1, chunks += chunk_vecs) {
+        const int n = min(kChunk, ext - s0);
+        const bool more = s0 + kChunk < ext, mine = mt * 16 < n;
+        cp_async_wait_all();
+        __syncthreads();   // this chunk, its factors and the state are in place; nobody needs the last chunk's
+        if (more) {
+            load_chunk(s0 + kChunk, buf ^ 1);
+            if (warp == 0) fetch_factors(s0 + kChunk);
+        }
+        uint4 ph[4], pl[4], th[4], tl[4];
+        if (mine) {
+            if (RULE == kDelta) load_matrix(chunks + kMatrixVecs, th, tl);
+            load_matrix(chunks, ph, pl);
+        }
+        const __nv_bfloat16 *K = S.k[buf], *Q = S.q[buf], *V = S.v[buf];
+        const int ta = mt * 16 + g, tb = ta + 8;   // this thread's rows of the products
+        // ---- Q S and K S ----
+        float o[4][4] = {}, u[4][4] = {};
+        if (mine) {
+#pragma unroll
+            for (int ks = 0; ks < DK / 16; ++ks) {
+                uint32_t aq[4], ak[4], b0, b1, b2, b3;
+                const int aoff = (mt * 16 + (mi & 1) * 8 + r8) * ROW + ks * 16 + (mi >> 1) * 8;
+                ldmatrix_x4(smem_u32(&Q[aoff]), aq[0], aq[1], aq[2], aq[3]);
+                if (RULE == kDelta) ldmatrix_x4(smem_u32(&K[aoff]), ak[0], ak[1], ak[2], ak[3]);
+#pragma unroll
+                for (int np = 0; np < 2; ++np) {
+                    const int soff = (ks * 16 + (mi & 1) * 8 + r8) * VROW + oc0 + np * 16 + (mi >> 1) * 8;
+#pragma unroll
+                    for (int part = 0; part < 2; ++part) {
+                        ldmatrix_x4_trans(smem_u32(part == 0 ? &S.sh[soff] : &S.sl[soff]), b0, b1, b2, b3);
+                        mma_bf16_16816(o[2 * np], aq, b0, b1);
+                        mma_bf16_16816(o[2 * np + 1], aq, b2, b3);
+                        if (RULE == kDelta) {
+                            mma_bf16_16816(u[2 * np], ak, b0, b1);
+                            mma_bf16_16816(u[2 * np + 1], ak, b2, b3);
+                        }
+                    }
+                }
+            }
+        }
+        if (RULE == kDelta) {
+            // ---- U = (I + A)^-1 (beta V - beta G K S) ----
+            if (mine) {
+                const float ba = S.beta[buf][ta], bb = S.beta[buf][tb], ra = S.read[buf][ta], rb = S.read[buf][tb];
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+#pragma unroll
+                    for (int half = 0; half < 2; ++half) {
+                        const int at = (half ? tb : ta) * VROW + oc0 + j * 8 + 2 * tq;
+                        const uint32_t v = *reinterpret_cast<const uint32_t*>(&V[at]);
+                        const float beta = half ? bb : ba, r = half ? rb : ra;
+                        uint32_t hi, lo;
+                        split2(beta * bf16_lo(v) - r * u[j][2 * half], beta * bf16_hi(v) - r * u[j][2 * half + 1], hi, lo);
+                        *reinterpret_cast<uint32_t*>(&S.rh[at]) = hi;
+                        *reinterpret_cast<uint32_t*>(&S.rl[at]) = lo;
+                        u[j][2 * half] = u[j][2 * half + 1] = 0.f;
+                    }
+            }
+            __syncthreads();
+            if (mine) multiply(u, th, tl, S.rh, S.rl);
+        }
+        if (mine) {
+            const float wa = S.write[buf][ta], wb = S.write[buf][tb];
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    const int at = (half ? tb : ta) * VROW + oc0 + j * 8 + 2 * tq;
+                    const float w = half ? wb : wa;
+                    float x = u[j][2 * half], y = u[j][2 * half + 1];
+                    uint32_t hi, lo;
+                    if (RULE == kDelta) {
+                        split2(x, y, hi, lo);
+                        *reinterpret_cast<uint32_t*>(&S.uh[at]) = hi;
+                        *reinterpret_cast<uint32_t*>(&S.ul[at]) = lo;
+                    } else {
+                        const uint32_t v = *reinterpret_cast<const uint32_t*>(&V[at]);
+                        x = bf16_lo(v);
+                        y = bf16_hi(v);
+                    }
+                    split2(x * w, y * w, hi, lo);
+                    *reinterpret_cast<uint32_t*>(&S.wh[at]) = hi;
+                    *reinterpret_cast<uint32_t*>(&S.wl[at]) = lo;
+                }
+        }
+        __syncthreads();
+        // ---- O = G Q S + P U (+ skip V) ----
+        if (mine) {
+            const float ga = S.out[buf][ta], gb = S.out[buf][tb];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                o[j][0] *= ga;
+                o[j][1] *= ga;
+                o[j][2] *= gb;
+                o[j][3] *= gb;
+            }
+            if (RULE == kDelta) multiply(o, ph, pl, S.uh, S.ul);
+            else multiply(o, ph, pl, V, nullptr);
+            __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + static_cast<int64_t>(begin + s0) * a.out_ld + at_v + oc0 + 2 * tq;
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int t = half ? tb : ta;
+                if (t >= n) continue;
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    float x = o[j][2 * half], y = o[j][2 * half + 1];
+                    if (RULE == kStateSpace) {
+                        const uint32_t v = *reinterpret_cast<const uint32_t*>(&V[t * VROW + oc0 + j * 8 + 2 * tq]);
+                        x = fmaf(skip, bf16_lo(v), x);
+                        y = fmaf(skip, bf16_hi(v), y);
+                    }
+                    *reinterpret_cast<uint32_t*>(out + t * a.out_ld + j * 8) = pack_bf16(x, y);
+                }
+            }
+        }
+        // ---- the state after the chunk ----
+        const float keep = S.keep[buf];
+#pragma unroll
+        for (int j = 0; j < kStateTiles; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) st[j][e] *= keep;
+#pragma unroll
+        for (int kt = 0; kt < kChunk / 16; ++kt) {
+            if (kt * 16 >= n) continue;
+            uint32_t ak[4];
+            ldmatrix_x4_trans(smem_u32(&K[(kt * 16 + (mi >> 1) * 8 + r8) * ROW + row0 + (mi & 1) * 8]), ak[0], ak[1], ak[2], ak[3]);
+#pragma unroll
+            for (int np = 0; np < kStateTiles / 2; ++np) {
+                const int off = (kt * 16 + (mi & 1) * 8 + r8) * VROW + col0 + np * 16 + (mi >> 1) * 8;
+                uint32_t b0, b1, b2, b3;
+                ldmatrix_x4_trans(smem_u32(&S.wh[off]), b0, b1, b2, b3);
+                mma_bf16_16816(st[2 * np], ak, b0, b1);
+                mma_bf16_16816(st[2 * np + 1], ak, b2, b3);
+                ldmatrix_x4_trans(smem_u32(&S.wl[off]), b0, b1, b2, b3);
+                mma_bf16_16816(st[2 * np], ak, b0, b1);
+                mma_bf16_16816(st[2 * np + 1], ak, b2, b3);
+            }
+        }
+        if (more) {
+            put_state();
+            if (warp == 0) put_factors(buf ^ 1);
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < kStateTiles; ++j)
+#pragma unroll
+        for (int half = 0; half < 2; ++half)
+            *reinterpret_cast<float2*>(state + static_cast<int64_t>(row0 + g + half * 8) * vp + col0 + j * 8 + 2 * tq) =
+                make_float2(st[j][2 * half], st[j][2 * half + 1]);
+}
+
+bool chunked_supported(const Recurrence& a, int dtype) {
+    return dtype == B200_DTYPE_BF16 && !a.plain && (a.padded_dim == 64 || a.padded_dim == 128) && a.padded_value_dim % kSlice == 0;
+}
+
+int max_smem(const void* kernel, size_t bytes) {
+    B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)));
+    return B200_OK;
+}
+
+template <typename T>
+int launch_mix(const Recurrence& a, cudaStream_t stream) {
+    auto kernel = a.taps == 2 ? mix_kernel<T, 2> : a.taps == 3 ? mix_kernel<T, 3> : a.taps == 4 ? mix_kernel<T, 4> : mix_kernel<T, 0>;
+    const int v_blocks = div_ceil(a.heads * a.padded_value_dim, kMixThreads * 8);
+    const int per_block = kMixThreads / (a.padded_dim / 8);
+    const dim3 grid(div_ceil(a.max_extend, kMixTokens), v_blocks + div_ceil(2 * a.kv_heads, per_block) + 1, a.batch);
+    B200_CHECK_CUDA(launch_kernel(kernel, grid, dim3(kMixThreads), 0, stream, dim3(1, 1, 1), a, v_blocks, per_block));
+    return B200_OK;
+}
+
+template <int RULE>
+int launch_chunked(const Recurrence& a, cudaStream_t stream) {
+    auto prepare = prepare_kernel<RULE>;
+    int err = max_smem(reinterpret_cast<const void*>(prepare), sizeof(PrepareSmem));
+    if (err != B200_OK) return err;
+    B200_CHECK_CUDA(launch_kernel(prepare, dim3(div_ceil(a.max_extend, kChunk), a.kv_heads, a.batch), dim3(kPrepareThreads),
+                                  sizeof(PrepareSmem), stream, dim3(1, 1, 1), a));
+    auto kernel = a.padded_dim == 64 ? chunk_kernel<64, RULE> : chunk_kernel<128, RULE>;
+    const size_t smem = a.padded_dim == 64 ? sizeof(WalkSmem<64, RULE>) : sizeof(WalkSmem<128, RULE>);
+    err = max_smem(reinterpret_cast<const void*>(kernel), smem);
+    if (err != B200_OK) return err;
+    B200_CHECK_CUDA(launch_kernel(kernel, dim3(a.padded_value_dim / kSlice, a.heads, a.batch), dim3(kWalkThreads), smem, stream,
+                                  dim3(1, 1, 1), a));
+    return B200_OK;
+}
+
+template <typename T, int RULE>
+int launch_steps(const Recurrence& a, int log_cols, int slices, bool finish, cudaStream_t stream) {
+    const size_t smem = (2ull * (4u << log_cols) + 2ull * a.padded_dim + kStepThreads * 4) * 4;
+    auto kernel = a.decode ? step_kernel<T, RULE, true> : step_kernel<T, RULE, false>;
+    B200_CHECK_CUDA(launch_kernel(kernel, dim3(a.heads, a.batch, slices), dim3(kStepThreads), smem, stream, dim3(1, 1, 1), a,
+                                  log_cols, finish));
+    return B200_OK;
+}
+
+template <typename T>
+int run(const Recurrence& a, int dtype, cudaStream_t stream) {
+    const bool delta = a.rule == kDelta;
+    int err = B200_OK;
+    if (!a.decode) err = launch_mix<T>(a, stream);
+    if (err != B200_OK) return err;
+    bool finished = false;
+    if (!a.decode && chunked_supported(a, dtype)) {
+        err = delta ? launch_chunked<kDelta>(a, stream) : launch_chunked<kStateSpace>(a, stream);
+    } else {
+        // groups of four columns per CTA: a thread has room for kAhead rows
+        const int most = kAhead * kStepThreads / a.padded_dim;
+        int log_cols = 0;
+        while ((4 << log_cols) < a.padded_value_dim && (2 << log_cols) <= most && (2 << log_cols) <= kStepThreads) ++log_cols;
+        const int slices = div_ceil(a.padded_value_dim, 4 << log_cols);
+        finished = a.decode && delta && slices == 1;
+        err = delta ? launch_steps<T, kDelta>(a, log_cols, slices, finished, stream)
+                    : launch_steps<T, kStateSpace>(a, log_cols, slices, finished, stream);
+    }
+    if (err != B200_OK || finished) return err;
+    if (delta) {
+        const int64_t rows = static_cast<int64_t>(a.tokens) * a.heads;
+        B200_CHECK_CUDA(launch_kernel(finish_heads_kernel<T>, dim3(static_cast<unsigned>(div_ceil64(rows, kFinishWarps))),
+                                      dim3(kFinishWarps * 32), 0, stream, dim3(1, 1, 1), a));
+    } else {
+        const int per = a.heads * a.value_dim / a.norm_groups;
+        auto kernel = per % 8 == 0 && a.value_dim % 8 == 0 ? finish_parts_kernel<T, 8> : finish_parts_kernel<T, 1>;
+        B200_CHECK_CUDA(launch_kernel(kernel, dim3(a.tokens, a.norm_groups), dim3(kPartThreads), 0, stream, dim3(1, 1, 1), a));
+    }
+    return B200_OK;
+}
+
+}  // namespace
+
+// A thread of the step kernel holds kAhead state rows of four columns.
+bool recurrence_supported(int padded_value_dim, int padded_dim, int taps) {
+    return padded_value_dim <= 65535 && padded_dim <= 1024 && taps >= 1 && taps <= kMaxTaps;
+}
+
+RecurrenceScratch recurrence_scratch(int rule, int max_tokens, int max_batch, int heads, int kv_heads, int padded_dim,
+                                     int padded_value_dim, int dtype) {
+    RecurrenceScratch s;
+    const int64_t T = max_tokens, esz = dtype == B200_DTYPE_F32 ? 4 : 2;
+    s.mixed = T * (static_cast<int64_t>(heads) * padded_value_dim + 2ll * kv_heads * padded_dim) * esz;
+    s.steps = T * heads * 8;
+    s.units = rule == kDelta ? T * kv_heads * 8 : 0;
+    s.chunks = dtype == B200_DTYPE_F32 || padded_dim > 128
+                   ? 0
+                   : (T / kChunk + max_batch + 1) * heads * (rule == kDelta ? 2 : 1) * kMatrixVecs * 16;
+    return s;
+}
+
+int launch_recurrence(const Recurrence& a, int dtype, cudaStream_t stream) {
+    if (a.tokens == 0 || a.batch == 0) return B200_OK;
+    return dtype == B200_DTYPE_F32 ? run<float>(a, dtype, stream) : run<__nv_bfloat16>(a, dtype, stream);
+}
+
+}  // namespace b200
+
+extern "C" {
+
+int b200_recurrence_scratch(int rule, int max_tokens, int max_batch, int heads, int kv_heads, int padded_dim,
+                            int padded_value_dim, int dtype, int64_t* bytes) {
+    B200_CHECK_ARG(bytes && max_tokens >= 0 && max_batch >= 0 && heads > 0 && kv_heads > 0 && padded_dim > 0 && padded_value_dim > 0,
+                   "recurrence_scratch: bad sizes");
+    const b200::RecurrenceScratch s =
+        b200::recurrence_scratch(rule, max_tokens, max_batch, heads, kv_heads, padded_dim, padded_value_dim, dtype);
+    bytes[0] = s.mixed;
+    bytes[1] = s.steps;
+    bytes[2] = s.units;
+    bytes[3] = s.chunks;
+    return B200_OK;
+}
+
+int b200_recurrence(const b200_recurrence_args* p, int dtype, b200_stream_t stream) {
+    B200_CHECK_ARG(p, "recurrence: NULL argument");
+    B200_CHECK_ARG(dtype == B200_DTYPE_BF16 || dtype == B200_DTYPE_F32, "recurrence: unknown dtype");
+    B200_CHECK_ARG(p->rule == B200_RULE_STATE_SPACE || p->rule == B200_RULE_DELTA, "recurrence: unknown rule");
+    B200_CHECK_ARG(p->tokens >= 0 && p->batch >= 0 && p->batch <= 65535 && p->heads > 0 && p->heads <= 65535 && p->kv_heads > 0 &&
+                       p->heads % p->kv_heads == 0, "recurrence: bad sizes");
+    B200_CHECK_ARG(p->dim > 0 && p->padded_dim >= p->dim && p->padded_dim % 64 == 0 && p->value_dim > 0 &&
+                       p->padded_value_dim >= p->value_dim && p->padded_value_dim % 64 == 0 &&
+                       b200::recurrence_supported(p->padded_value_dim, p->padded_dim, p->taps), "recurrence: bad head sizes");
+    B200_CHECK_ARG(p->joint_ld % 8 == 0 && p->out_ld % 8 == 0 && p->out_ld >= static_cast<int64_t>(p->heads) * p->padded_value_dim,
+                   "recurrence: bad strides");
+    B200_CHECK_ARG(p->rule == B200_RULE_DELTA || (p->norm_groups > 0 && p->heads * p->value_dim % p->norm_groups == 0),
+                   "recurrence: bad norm groups");
+    B200_CHECK_ARG(static_cast<int64_t>(p->tokens) * p->heads < (1ll << 31), "recurrence: too many tokens");
+    B200_CHECK_ARG(!p->decode || p->tokens == p->batch, "recurrence: a decode step brings one token per request");
+    if (p->tokens == 0 || p->batch == 0) return B200_OK;
+    B200_CHECK_ARG(p->out && p->joint && p->table_idx && p->cached && p->state && p->conv_state && p->conv && p->decay_log &&
+                       p->step_bias && p->norm && (p->rule == B200_RULE_DELTA || p->skip), "recurrence: NULL tensor");
+    B200_CHECK_ARG(p->decode || (p->qo_indptr && p->mixed && p->steps && (p->units || p->rule != B200_RULE_DELTA) && p->chunks &&
+                                 p->max_extend > 0), "recurrence: NULL scratch");
+    return b200::launch_recurrence(*p, dtype, static_cast<cudaStream_t>(stream));
+}
+
+}  // extern "C"

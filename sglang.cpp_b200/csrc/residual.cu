@@ -3,8 +3,8 @@
 // writes its RMS norm for the next block - to the token's own row, or straight into the expert-sorted
 // rows that the next block's grouped GEMM reads.  One CTA per token, the row in registers.
 //
-// Two wirings: the norm on what the next block reads (residual_norm_kernel), or on what the previous block
-// returned, before it is added (residual_post_norm_kernel).
+// Wirings: the norm on what the next block reads (residual_norm_kernel), or on what the previous block
+// returned, before it is added, or both (residual_post_norm_kernel).
 #include "common.cuh"
 #include "kernels.h"
 
@@ -157,6 +157,9 @@ struct PostArgs {
     const int32_t* src_rows;
     const float* src_weights;
     const void* src2;
+    const void* pair_weight;
+    const void* pair_weight2;
+    float pair_scale;
     const void* add_weight;
     const void* out_weight;
     int64_t src_count;
@@ -168,12 +171,13 @@ struct PostArgs {
 };
 
 // What is added is a token's row of the source, or the weighted rows src_rows names, plus its row of a second
-// source; it is RMS-normalised when there is a weight for it.  The sum goes to the residual and, rounded (or
+// source (PAIR: both normalised by themselves first, the sum scaled); it is RMS-normalised when there is a weight
+// for it.  The sum goes to the residual and, rounded (or
 // normalised once more, before the output head), to `out`.
-template <typename T, int VEC>
+template <typename T, int VEC, bool PAIR>
 __global__ void __launch_bounds__(256)
 residual_post_norm_kernel(const PostArgs a) {
-    __shared__ float red[2][8];
+    __shared__ float red[PAIR ? 4 : 2][8];
     __shared__ int s_row[kRows];
     __shared__ float s_weight[kRows];
     pdl_launch_dependents();
@@ -201,8 +205,17 @@ residual_post_norm_kernel(const PostArgs a) {
     float* res = a.residual + t * a.padded;
     const T* src = static_cast<const T*>(a.src);
     const T* src2 = static_cast<const T*>(a.src2);
+    float scale_a = 1.f, scale_b = 1.f;   // PAIR: one over the root mean square of either row
     auto addend = [&](int v) {
         Vec8 y;
+        if (PAIR) {
+            y = load8(src + t * a.padded + v * 8);
+            const Vec8 x = load8(src2 + t * a.padded + v * 8);
+            const Vec8 ga = load8(static_cast<const T*>(a.pair_weight) + v * 8), gb = load8(static_cast<const T*>(a.pair_weight2) + v * 8);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) y.v[j] = a.pair_scale * (y.v[j] * scale_a * ga.v[j] + x.v[j] * scale_b * gb.v[j]);
+            return y;
+        }
 #pragma unroll
         for (int j = 0; j < 8; ++j) y.v[j] = 0.f;
         if (a.src_rows == nullptr) {
@@ -235,6 +248,19 @@ residual_post_norm_kernel(const PostArgs a) {
         __syncthreads();
         return warp_sum(lane < static_cast<int>(blockDim.x >> 5) ? scratch[lane] : 0.f);
     };
+    if (PAIR) {
+        float sa = 0.f, sb = 0.f;
+        for (int v = threadIdx.x; v < nvec; v += blockDim.x) {
+            const Vec8 x = load8(src + t * a.padded + v * 8), y = load8(src2 + t * a.padded + v * 8);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                sa += x.v[j] * x.v[j];
+                sb += y.v[j] * y.v[j];
+            }
+        }
+        scale_a = rsqrtf(block_sum(sa, red[PAIR ? 2 : 0]) / static_cast<float>(a.width) + a.eps);
+        scale_b = rsqrtf(block_sum(sb, red[PAIR ? 3 : 0]) / static_cast<float>(a.width) + a.eps);
+    }
     Vec8 val[VEC], add[VEC];
     float ss = 0.f;
 #pragma unroll
@@ -308,10 +334,10 @@ residual_post_norm_kernel(const PostArgs a) {
     for (int v = wide0; v < nvec; v += blockDim.x) emit(v, load8(static_cast<const float*>(res) + v * 8));
 }
 
-template <typename T>
+template <typename T, bool PAIR>
 auto post_kernel_for(int pieces) {
-    return pieces <= 1 ? residual_post_norm_kernel<T, 1>
-                       : pieces <= 2 ? residual_post_norm_kernel<T, 2> : residual_post_norm_kernel<T, 4>;
+    return pieces <= 1 ? residual_post_norm_kernel<T, 1, PAIR>
+                       : pieces <= 2 ? residual_post_norm_kernel<T, 2, PAIR> : residual_post_norm_kernel<T, 4, PAIR>;
 }
 
 }  // namespace
@@ -325,6 +351,9 @@ int launch_residual_post_norm(const ResidualPostNorm& r, int dtype, int* status,
     a.src_rows = r.src_rows;
     a.src_weights = r.src_weights;
     a.src2 = r.src2;
+    a.pair_weight = r.pair_weight;
+    a.pair_weight2 = r.pair_weight2;
+    a.pair_scale = r.pair_scale;
     a.add_weight = r.add_weight;
     a.out_weight = r.out_weight;
     a.src_count = r.src_count;
@@ -341,7 +370,10 @@ int launch_residual_post_norm(const ResidualPostNorm& r, int dtype, int* status,
     int threads = 32;
     while (threads < 256 && threads * 8 < r.padded) threads *= 2;
     const int pieces = div_ceil(r.padded, threads * 8);
-    auto kernel = dtype == B200_DTYPE_F32 ? post_kernel_for<float>(pieces) : post_kernel_for<__nv_bfloat16>(pieces);
+    const bool f32 = dtype == B200_DTYPE_F32;
+    auto kernel = r.pair_weight != nullptr
+                      ? (f32 ? post_kernel_for<float, true>(pieces) : post_kernel_for<__nv_bfloat16, true>(pieces))
+                      : (f32 ? post_kernel_for<float, false>(pieces) : post_kernel_for<__nv_bfloat16, false>(pieces));
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(r.tokens), dim3(threads), 0, stream, dim3(1, 1, 1), a));
     return B200_OK;
 }
@@ -433,6 +465,34 @@ int b200_residual_post_norm(void* out, float* residual, const void* src, const i
     r.src_count = src_count;
     r.src2 = src2;
     r.init = init != 0;
+    r.add_weight = add_weight;
+    r.out_weight = out_weight;
+    r.tokens = tokens;
+    r.width = width;
+    r.padded = padded;
+    r.eps = eps;
+    return b200::launch_residual_post_norm(r, dtype, status, static_cast<cudaStream_t>(stream));
+}
+
+int b200_residual_pair_norm(void* out, float* residual, const void* src, const void* src2, const void* weight,
+                            const void* weight2, float pair_scale, const void* add_weight, const void* out_weight,
+                            int tokens, int width, int padded, float eps, int dtype, b200_stream_t stream) {
+    B200_CHECK_ARG(tokens >= 0 && width > 0 && padded >= width && padded % 64 == 0, "residual_pair_norm: bad shape");
+    B200_CHECK_ARG(dtype == B200_DTYPE_BF16 || dtype == B200_DTYPE_F32, "residual_pair_norm: unknown dtype");
+    if (tokens == 0) return B200_OK;
+    B200_CHECK_ARG(out && residual && src && src2 && weight && weight2, "residual_pair_norm: NULL tensor");
+    int err = B200_OK;
+    int* status = b200::device_status_words(&err);
+    if (err != B200_OK) return err;
+    b200::ResidualPostNorm r;
+    r.out = out;
+    r.residual = residual;
+    r.src = src;
+    r.src_count = tokens;
+    r.src2 = src2;
+    r.pair_weight = weight;
+    r.pair_weight2 = weight2;
+    r.pair_scale = pair_scale;
     r.add_weight = add_weight;
     r.out_weight = out_weight;
     r.tokens = tokens;

@@ -1,5 +1,6 @@
 // Softmax attention of layer stacks: per-head query and key norms, partial rotation, values mixed with those of
-// an earlier layer, a sliding window that keeps the first keys, and a gate on the output.
+// an earlier layer, a sliding window that keeps the first keys or chunks of the sequence, sinks, and gates on the
+// output (AttentionWindow).
 //
 //   * head_prepare_kernel: between the joint projection and the attention.  One warp per (token, head) row of
 //     the joint output [q heads | k heads | v heads | gate]: queries are normalised and rotated in place, keys
@@ -221,7 +222,7 @@ window_attention_plain_kernel(const WindowAttention a) {
     for (int i = threadIdx.x; i < a.dp; i += kPlainThreads) s_q[i] = to_f32(q[i]) * a.scale;
     const int32_t* pages = a.page_table + static_cast<int64_t>(a.row_table[t]) * a.pt_stride;
     const int len = a.row_len[t];
-    const int oldest = max(0, len - a.window.size);
+    const int oldest = len > 0 ? a.window.oldest(len - 1) : 0;
     const int kept = min(a.window.keep_first, oldest);
     const int count = kept + len - oldest;             // keys it sees: [0, kept) and [oldest, len)
     float acc[kPlainMaxVec];
@@ -282,10 +283,15 @@ window_attention_plain_kernel(const WindowAttention a) {
             }
         }
     }
-    T* out = static_cast<T*>(a.out) + (t * a.heads + h) * a.vp;
-    const T* gate = a.window.gate == nullptr ? nullptr
-                                             : static_cast<const T*>(a.window.gate) + t * a.window.gate_st + static_cast<int64_t>(h) * a.vp;
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    T* out = static_cast<T*>(a.out) + t * a.window.out_st + static_cast<int64_t>(h) * a.vp;
+    const T* gate = a.window.gate == nullptr ? nullptr : static_cast<const T*>(a.window.gate) + t * a.window.gate_st;
+    if (a.window.sinks != nullptr) l += expf(a.window.sinks[h] - m);
+    float inv = l > 0.f ? a.window.out_scale / l : 0.f;
+    if (gate != nullptr && a.window.gate_per_head) {
+        inv *= 1.f / (1.f + expf(-to_f32(gate[h])));
+        gate = nullptr;
+    }
+    if (gate != nullptr) gate += static_cast<int64_t>(h) * a.vp;
 #pragma unroll
     for (int i = 0; i < kPlainMaxVec; ++i) {
         const int c = threadIdx.x + i * kPlainThreads;
@@ -316,7 +322,7 @@ int launch_head_prepare(const HeadPrepare& a, int dtype, cudaStream_t stream) {
 bool window_attention_tc_supported(const WindowAttention& a, int dtype) {
     const int group = a.heads / a.kv_heads;
     if (dtype != B200_DTYPE_BF16 || a.plain || a.dp != 128 || a.vp != 128 || a.scale <= 0.f || group > 16) return false;
-    if (a.window.gate_st % 8 != 0 || !attention_prefill_tc_supported(a.q, a.q_st, a.dp, a.out)) return false;
+    if (a.window.gate_st % 8 != 0 || a.window.out_st % 8 != 0 || !attention_prefill_tc_supported(a.q, a.q_st, a.dp, a.out)) return false;
     if (a.decode) return a.kv_heads <= 8 && 8 % a.kv_heads == 0 && a.batch <= 1024;
     return (group & (group - 1)) == 0;
 }
@@ -337,9 +343,11 @@ int launch_window_attention(const WindowAttention& a, int dtype, cudaStream_t st
                                        a.table_idx, a.seq_lens, a.batch, a.heads, a.kv_heads, a.page_size, a.scale,
                                        a.workspace, a.workspace_bytes, a.status, stream, true, &a.window);
     }
+    WindowAttention plain = a;
+    if (plain.window.out_st == 0) plain.window.out_st = static_cast<int64_t>(a.heads) * a.vp;
     auto kernel = dtype == B200_DTYPE_F32 ? window_attention_plain_kernel<float> : window_attention_plain_kernel<__nv_bfloat16>;
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(a.tokens, a.heads), dim3(kPlainThreads), static_cast<size_t>(a.dp) * 4, stream,
-                                  dim3(1, 1, 1), a));
+                                  dim3(1, 1, 1), plain));
     return B200_OK;
 }
 
@@ -398,7 +406,9 @@ int b200_window_attention(const b200_window_attention_args* p, int dtype, b200_s
                        p->padded_value_dim % 64 == 0 && p->padded_value_dim <= b200::kPlainMaxVec * b200::kPlainThreads,
                    "window_attention: bad head sizes");
     B200_CHECK_ARG(p->page_size >= 1 && (p->page_size & (p->page_size - 1)) == 0, "window_attention: page_size must be a power of two");
-    B200_CHECK_ARG(p->window >= 1 && p->keep_first >= 0, "window_attention: bad window");
+    B200_CHECK_ARG(p->window >= 1 && p->keep_first >= 0 && p->chunk >= 0, "window_attention: bad window");
+    B200_CHECK_ARG(p->out_stride == 0 || p->out_stride >= static_cast<int64_t>(p->heads) * p->padded_value_dim,
+                   "window_attention: bad output stride");
     if (p->tokens == 0) return B200_OK;
     B200_CHECK_ARG(p->out && p->q && p->k_cache && p->v_cache && p->page_table && p->table_idx && p->seq_lens && p->qo_indptr &&
                        p->row_table && p->row_len && p->workspace, "window_attention: NULL tensor");
@@ -434,6 +444,11 @@ int b200_window_attention(const b200_window_attention_args* p, int dtype, b200_s
     a.window.keep_first = p->keep_first;
     a.window.gate = p->gate;
     a.window.gate_st = p->gate_stride;
+    a.window.gate_per_head = p->gate_per_head != 0;
+    a.window.chunk = p->chunk;
+    a.window.sinks = p->sinks;
+    a.window.out_scale = p->out_scale == 0.f ? 1.f : p->out_scale;
+    a.window.out_st = p->out_stride;
     a.workspace = p->workspace;
     a.workspace_bytes = p->workspace_bytes;
     return b200::launch_window_attention(a, dtype, static_cast<cudaStream_t>(stream));

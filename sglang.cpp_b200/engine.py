@@ -105,12 +105,17 @@ class Engine:
         self.dtype = model_config.torch_dtype
         layers = (_lib.LayerConfigStruct * len(model_config.layers))(
             *[spec.as_struct() for spec in model_config.layers])
+        pairs = [(i, spec.beside) for i, spec in enumerate(model_config.layers) if spec.beside is not None]
+        beside = (_lib.LayerConfigStruct * max(len(pairs), 1))(*[spec.as_struct() for _, spec in pairs])
+        for n, (i, _) in enumerate(pairs):
+            layers[i].beside = n
         m = ModelConfigStruct(num_layers=len(model_config.layers), hidden_size=model_config.hidden_size,
                               vocab_size=model_config.vocab_size, rms_norm_eps=model_config.rms_norm_eps,
                               tie_word_embeddings=int(model_config.tie_word_embeddings))
         st = _lib.StackConfigStruct(len(model_config.layers), layers,
                                     _lib.DTYPE_F32 if self.dtype == torch.float32 else _lib.DTYPE_BF16,
-                                    model_config.norm_offset, model_config.logit_scale, int(model_config.norm_output))
+                                    model_config.norm_offset, model_config.logit_scale, int(model_config.norm_output),
+                                    len(pairs), beside)
         call("b200_engine_create_stack", ctypes.byref(m), ctypes.byref(st), ctypes.byref(c), ctypes.byref(self._h))
 
     def close(self) -> None:
@@ -234,15 +239,24 @@ class Engine:
             fill("lm_head", 0, seed * 1000 + 2)
             for l, spec in enumerate(cfg.layers):
                 for i, name in enumerate(("down_qkv", "uq", "uk", "uk_absorb", "uv", "o", "mlp_up", "mlp_down", "qkvg", "qkvga",
-                                          "decay_up", "router", "shared_up", "shared_down")):
-                    fill(name, l, seed * 1000 + 100 + l * 16 + i)
-                norms = ("q_latent_norm", "kv_latent_norm", "q_head_norm", "k_head_norm", "head_norm")
-                # (with an offset, norm1 and norm2 hold gain - 1: zero as allocated)
-                for name in norms if cfg.norm_offset else norms + ("norm1", "norm2"):
+                                          "decay_up", "router", "shared_up", "shared_down", "joint", "recurrence", "beside_o")):
+                    fill(name, l, seed * 1000 + 100 + l * 32 + i)
+                norms = ("q_latent_norm", "kv_latent_norm", "q_head_norm", "k_head_norm", "head_norm", "beside_head_norm",
+                         "side_norm", "beside_side_norm")
+                # (with an offset, the layer norms hold gain - 1: zero as allocated)
+                for name in norms if cfg.norm_offset else norms + ("norm1", "norm2", "norm1_out", "norm2_out"):
                     fill(name, l, 0, ones=True)
+                for name in ("conv", "beside_conv"):      # (fp32; decays, biases and skips stay zero)
+                    try:
+                        ptr, n = self.tensor_info(name, l)
+                    except B200Error:
+                        continue
+                    g = torch.Generator(device=dev).manual_seed(seed * 1000 + 131 + l * 32)
+                    taps = _as_cuda_tensor(ptr, n).view(torch.float32)
+                    taps.copy_(torch.randn(taps.numel(), generator=g, device=dev))
                 if spec.mlp == _lib.MLP_TABLE_MOE:
                     ptr, n = self.tensor_info("expert_table", l)
-                    g = torch.Generator(device=dev).manual_seed(seed * 1000 + 99 + l * 16)
+                    g = torch.Generator(device=dev).manual_seed(seed * 1000 + 99 + l * 32)
                     rank_of = torch.rand(cfg.vocab_size, spec.num_experts, generator=g, device=dev)
                     table = rank_of.topk(spec.experts_per_tok, dim=1).indices.to(torch.int32)
                     _as_cuda_tensor(ptr, n).view(torch.int32).copy_(table.flatten())

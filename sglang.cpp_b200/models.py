@@ -5,7 +5,7 @@
 
 * ``ModelConfig``: one layer repeated (Llama, Qwen2, Qwen3, Qwen3-MoE; the fields of
   include/sglang/models/config.h:15-42);
-* ``StackConfig``: layers listed one by one (Rapizen, Dilalix).  Each is a ``LayerSpec`` that names its mixer and
+* ``StackConfig``: layers listed one by one (Rapizen, Dilalix, Saluzen).  Each is a ``LayerSpec`` that names its mixer and
   its feed-forward with their sizes; another design made of the same parts needs a reader here (and a
   packing in ``weights.py`` where its tensors are named differently).
 
@@ -83,11 +83,32 @@ class LayerSpec:
     shared_intermediate: int = 0
     act_limit: float = 0.0
     shared_act_limit: float = 0.0
+    # window attention
+    head_norm: bool = True
+    gate: int = _lib.GATE_ELEMENT
+    qkv_bias: bool = False
+    sink: bool = False            # a score per head in the softmax's denominator ...
+    sink_learned: bool = True     # ... from the checkpoint, or 0
+    chunk: int = 0                # keys of the query's own chunk, instead of a window
+    # rotations whose long wavelengths are stretched; latent attention counts its rotary_dim rotated dimensions in
+    # head_dim
+    rope_factor: float = 0.0
+    rope_low: float = 1.0
+    rope_high: float = 1.0
+    rope_original: float = 0.0
+    kv_from: int = -1             # latent attention: the layer whose latents are read
+    # recurrences: head_dim state rows, kv_heads heads of k and q
+    conv_taps: int = 1
+    norm_groups: int = 1
+    # a second mixer on the same input, and how the results meet
+    beside: Optional["LayerSpec"] = None
+    join: int = _lib.JOIN_SUM
+    out_scale: float = 1.0
 
     def as_struct(self) -> _lib.LayerConfigStruct:
-        values = {f.name: getattr(self, f.name) for f in fields(self)}
-        values["value_mix"] = int(self.value_mix)
-        return _lib.LayerConfigStruct(**values)
+        """(``beside`` becomes an index once the whole stack is known: Engine.)"""
+        values = {f.name: getattr(self, f.name) for f in fields(self) if f.name not in ("beside", "sink_learned")}
+        return _lib.LayerConfigStruct(beside=-1, **{k: int(v) if isinstance(v, bool) else v for k, v in values.items()})
 
 
 @dataclass
@@ -98,7 +119,7 @@ class StackConfig:
     layers: list = field(default_factory=list)
     norm_offset: float = 0.0      # stored norm weights are the gain minus this
     logit_scale: float = 1.0
-    norm_output: bool = False     # the norms are on what the blocks return, not on what they read
+    norm_output: int = _lib.NORM_INPUT   # norms on what the blocks read, on what they return, or on both
     tie_word_embeddings: bool = False
     torch_dtype: torch.dtype = torch.bfloat16
 
@@ -108,7 +129,8 @@ class StackConfig:
 
     @property
     def carries_state(self) -> bool:
-        return any(c.mixer == _lib.MIXER_LINEAR_ATTENTION for c in self.layers)
+        kinds = (_lib.MIXER_LINEAR_ATTENTION, _lib.MIXER_STATE_SPACE, _lib.MIXER_DELTA_RULE)
+        return any(m is not None and m.mixer in kinds for c in self.layers for m in (c, c.beside))
 
     def expands_keys(self, c: LayerSpec) -> bool:
         """Does this layer's prefill expand keys and values (csrc/layer_stack.cu, can_expand)?"""
@@ -184,7 +206,62 @@ def read_dilalix(c: dict, shapes: Optional[dict] = None) -> StackConfig:
             else:
                 raise ValueError(f"layer {i}: unknown feed-forward {ff['kind']!r}")
         layers.append(spec)
-    return StackConfig(c["width"], c["vocab"], float(c["norm"]["eps"]), layers, norm_output=True)
+    return StackConfig(c["width"], c["vocab"], float(c["norm"]["eps"]), layers, norm_output=_lib.NORM_OUTPUT)
+
+
+def _set_rotation(spec: LayerSpec, rot: dict) -> None:
+    spec.rotary_dim, spec.rope_base = rot["dims"], float(rot["base"])
+    s = rot.get("scaling")
+    if s:
+        spec.rope_factor, spec.rope_low, spec.rope_high = float(s["factor"]), float(s["low"]), float(s["high"])
+        spec.rope_original = float(s["original"])
+
+
+def _biased_attention(m: dict) -> LayerSpec:
+    """Grouped-query attention with projection biases and a sink, without norms on queries and keys."""
+    spec = LayerSpec(m["heads"], m["dim"], m["vdim"], score_scale=float(m["scale"]), mixer=_lib.MIXER_WINDOW_ATTENTION,
+                     kv_heads=m["kv_heads"], head_norm=False, qkv_bias=True, sink=True)
+    _set_rotation(spec, m["rot"])
+    return spec
+
+
+def _state_space(m: dict) -> LayerSpec:
+    return LayerSpec(m["heads"], m["state"], m["vdim"], mixer=_lib.MIXER_STATE_SPACE, kv_heads=m["groups"],
+                     conv_taps=m["conv"], norm_groups=m["norm_groups"])
+
+
+def _delta_rule(m: dict) -> LayerSpec:
+    return LayerSpec(m["heads"], m["dim"], m["vdim"], mixer=_lib.MIXER_DELTA_RULE, kv_heads=m["kv_heads"],
+                     conv_taps=m["conv"])
+
+
+def read_saluzen(c: dict, shapes: Optional[dict] = None) -> StackConfig:
+    layers = []
+    for i, entry in enumerate(c["layers"]):
+        m = entry["mixer"]
+        if entry["type"] == "parallel":
+            spec = _biased_attention(m["left"])
+            spec.sink_learned = False
+            spec.beside, spec.join = _state_space(m["right"]), _lib.JOIN_NORMED
+        elif entry["type"] == "parallel_2":
+            spec = _biased_attention(m["left"])
+            spec.chunk, spec.gate, spec.out_scale = m["left"]["mask"]["size"], _lib.GATE_HEAD, float(m["left_scale"])
+            spec.beside, spec.join = _delta_rule(m["right"]), _lib.JOIN_SUM
+            spec.beside.out_scale = float(m["right_scale"])
+        elif entry["type"] == "latent_attention":
+            spec = LayerSpec(m["heads"], m["dim"] + m["rot_dim"], m["vdim"], m["q_rank"], m["kv_rank"], float(m["scale"]))
+            _set_rotation(spec, {**m["rot"], "dims": m["rot_dim"]})
+            if m.get("kv_from") is not None:
+                spec.kv_from = m["kv_from"]
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {entry['type']!r}")
+        ff = entry.get("mlp")
+        if ff is not None:
+            if ff["kind"] != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward {ff['kind']!r}")
+            spec.mlp, spec.intermediate, spec.epilogue = _lib.MLP_DENSE, ff["ff"], _lib.EPILOGUE_SWIGLU
+        layers.append(spec)
+    return StackConfig(c["width"], c["vocab"], float(c["norm"]["eps"]), layers, norm_output=_lib.NORM_BOTH)
 
 
 REGISTRY: dict[str, Callable] = {
@@ -194,6 +271,7 @@ REGISTRY: dict[str, Callable] = {
     "Qwen3MoeForCausalLM": _uniform(qk_norm=True, fused_residual=True, moe=True),
     "Rapizen": read_rapizen,
     "Dilalix": read_dilalix,
+    "Saluzen": read_saluzen,
 }
 
 

@@ -170,8 +170,9 @@ def unpack_checkpoint(cfg, w: dict) -> dict:
 def pack_layer_stack(cfg, tensors: dict) -> dict:
     """Parameter names of the layer-stack designs -> the padded layouts of ``b200_engine_create_stack``, in
     the dtype the model runs in.  Every tensor is checked against the shape its layer's description asks for."""
-    from ._lib import (MIXER_LATENT_ATTENTION, MIXER_LINEAR_ATTENTION, MIXER_WINDOW_ATTENTION, MLP_DENSE, MLP_NONE,
-                       MLP_SCORED_MOE, epilogue_is_gated, load)
+    from ._lib import (GATE_ELEMENT, GATE_HEAD, JOIN_NORMED, MIXER_DELTA_RULE, MIXER_LATENT_ATTENTION, MIXER_LINEAR_ATTENTION,
+                       MIXER_STATE_SPACE, MIXER_WINDOW_ATTENTION, MLP_DENSE, MLP_NONE, MLP_SCORED_MOE, NORM_BOTH,
+                       epilogue_is_gated, load)
 
     lib = load()
     width, head, latent = lib.b200_pad_width, lib.b200_pad_head_dim, lib.b200_pad_latent
@@ -203,38 +204,122 @@ def pack_layer_stack(cfg, tensors: dict) -> dict:
         return pad(need(name, heads * n, k).view(heads, n, k), heads, to, kp).reshape(heads * to, kp)
 
     def latent_attention(m, c):
-        H, d, dv, qr, kr = c.heads, c.head_dim, c.value_dim, c.q_rank, c.kv_rank
-        dp, vp, qp, rp = head(d), head(dv), width(qr), latent(kr)
-        uk = pad(need(m + "uk", H * d, kr).view(H, d, kr), H, dp, rp)
-        L = {"down_qkv": torch.cat([rows(m + "dq", qr, qp), rows(m + "dkv", kr, rp)]),
-             "q_latent_norm": pad(need(m + "dq.norm", qr), qp),
-             "kv_latent_norm": pad(need(m + "dkv.norm", kr), rp),
-             "uq": pad(need(m + "uq", H * d, qr).view(H, d, qr), H, dp, qp),
-             "uk_absorb": uk.transpose(1, 2).contiguous(),
-             "uv": pad(need(m + "uv", H * dv, kr).view(H, dv, kr), H, vp, rp)}
+        H, dr, dv, qr, kr = c.heads, c.rotary_dim, c.value_dim, c.q_rank, c.kv_rank
+        d, at = c.head_dim - dr, lib.b200_latent_rope_at(kr) if dr else kr
+        dp, vp, qp, rp, op = head(d + dr), head(dv), width(qr), latent(at + dr), latent(kr)
+        # A head's rotated dimensions come first.  Keys take them from the latent as they are, so that one matrix per
+        # head turns a latent into its whole key.
+        uk = torch.zeros(H, dp, rp, dtype=cfg.torch_dtype)
+        uk[:, dr:dr + d, :kr] = need(m + "uk", H * d, kr).view(H, d, kr)
+        uk[:, range(dr), range(at, at + dr)] = 1
+        uq = need(m + "uq", H * (d + dr), qr).view(H, d + dr, qr)
+        L = {"down_qkv": rows(m + "dq", qr, qp), "q_latent_norm": pad(need(m + "dq.norm", qr), qp),
+             "uq": pad(torch.cat([uq[:, d:], uq[:, :d]], 1), H, dp, qp), "uk_absorb": uk.transpose(1, 2).contiguous(),
+             "uv": pad(need(m + "uv", H * dv, kr).view(H, dv, kr), H, vp, op)}
+        if c.kv_from < 0:
+            dkv, down = need(m + "dkv", kr + dr, D), torch.zeros(rp, hp, dtype=cfg.torch_dtype)
+            down[:kr, :D], down[at:at + dr, :D] = dkv[:kr], dkv[kr:]
+            L["down_qkv"] = torch.cat([L["down_qkv"], down])
+            L["kv_latent_norm"] = pad(need(m + "dkv.norm", kr), rp)
         if cfg.expands_keys(c):
             L["uk"] = uk
         return L, vp
 
+    # The mixers below return (rows of the input projection, their bias or None, other tensors, padded value dimension).
     def window_attention(m, c):
         H, G, d, dv = c.heads, c.kv_heads, c.head_dim, c.value_dim
         dp, vp = head(d), head(dv)
-        L = {"qkvg": torch.cat([head_rows(m + "q", H, d, dp), head_rows(m + "k", G, d, dp), head_rows(m + "v", G, dv, vp),
-                                head_rows(m + "g", H, dv, vp)]),
-             "q_head_norm": pad(need(m + "q.norm", d), dp), "k_head_norm": pad(need(m + "k.norm", d), dp)}
+        parts = [("q", H, d, dp), ("k", G, d, dp), ("v", G, dv, vp)]
+        joint = [head_rows(m + name, n, k, kp) for name, n, k, kp in parts]
+        if c.gate == GATE_ELEMENT:
+            joint.append(head_rows(m + "g", H, dv, vp))
+        elif c.gate == GATE_HEAD:
+            joint.append(rows(m + "g", H, width(H)))
+        joint, L, bias = torch.cat(joint), {}, None
+        if c.qkv_bias:
+            bias = torch.cat([pad(need(f"{m}{name}.b", n * k).view(n, k), n, kp).flatten() for name, n, k, kp in parts])
+            bias = pad(bias, len(joint))
+        if c.head_norm:
+            L.update(q_head_norm=pad(need(m + "q.norm", d), dp), k_head_norm=pad(need(m + "k.norm", d), dp))
         if c.value_mix:
             L["value_mix"] = need(m + "vmix", dtype=torch.float32).reshape(1)
-        return L, vp
+        if c.sink:
+            L["sinks"] = need(m + "sink", H, dtype=torch.float32) if c.sink_learned else torch.zeros(H)
+        return joint, bias, L, vp
 
     def linear_attention(m, c):
         H, d, dv, r = c.heads, c.head_dim, c.value_dim, c.decay_rank
         dp, vp = width(d), width(dv)
-        L = {"qkvga": torch.cat([head_rows(m + "q", H, d, dp), head_rows(m + "k", H, d, dp), head_rows(m + "v", H, dv, vp),
-                                 head_rows(m + "g", H, dv, vp), rows(m + "a1", r, width(r))]),
-             "decay_up": head_rows(m + "a2", H, d, dp, r, -(-r // 16) * 16),
+        joint = torch.cat([head_rows(m + "q", H, d, dp), head_rows(m + "k", H, d, dp), head_rows(m + "v", H, dv, vp),
+                           head_rows(m + "g", H, dv, vp), rows(m + "a1", r, width(r))])
+        L = {"decay_up": head_rows(m + "a2", H, d, dp, r, -(-r // 16) * 16),
              "decay_bias": pad(need(m + "a2.b", H * d, dtype=torch.float32).view(H, d), H, dp),
              "head_norm": pad(need(m + "norm", dv), vp)}
-        return L, vp
+        return joint, None, L, vp
+
+    def by_head(t, heads, n, to):
+        """The first dimension as `heads` blocks of n, each padded to `to`."""
+        return pad(t.reshape(heads, n, *t.shape[1:]), heads, to, *t.shape[1:]).flatten(0, 1)
+
+    def state_space(m, c):
+        H, G, N, dv, taps = c.heads, c.kv_heads, c.head_dim, c.value_dim, c.conv_taps
+        dp, vp, inner = width(N), width(dv), H * dv
+        f32 = dict(dtype=torch.float32)
+        blocks = [(H, dv, vp), (G, N, dp), (G, N, dp)]              # x, B, C: the convolution's channels
+        split = [n * k for n, k, _ in blocks]
+        z, xbc, dt = need(m + "in", 2 * inner + 2 * G * N + H, D).split([inner, sum(split), H])
+        joint = torch.cat([by_head(z, H, dv, vp)] + [by_head(t, *b) for t, b in zip(xbc.split(split), blocks)] + [pad(dt, width(H), D)])
+        conv = [by_head(t, *b) for t, b in zip(need(m + "conv", sum(split), taps, **f32).split(split), blocks)]
+        bias = [by_head(t, *b) for t, b in zip(need(m + "conv.b", sum(split), **f32).split(split), blocks)]
+        L = {"conv": torch.cat(conv).T.contiguous(), "conv_bias": torch.cat(bias), "decay_log": need(m + "A_log", H, **f32),
+             "step_bias": need(m + "dt_bias", H, **f32), "skip": need(m + "D", H, **f32),
+             "head_norm": by_head(need(m + "norm", inner), H, dv, vp)}
+        return pad(joint, len(joint), hp), None, L, vp
+
+    def delta_rule(m, c):
+        H, G, d, dv, taps = c.heads, c.kv_heads, c.head_dim, c.value_dim, c.conv_taps
+        dp, vp = width(d), width(dv)
+        f32 = dict(dtype=torch.float32)
+        blocks = {"v": (H, dv, vp), "k": (G, d, dp), "q": (G, d, dp)}
+        steps = torch.cat([need(m + "a", H, D), need(m + "b", H, D)])
+        joint = torch.cat([head_rows(m + "g", H, dv, vp)] + [head_rows(m + n, *b) for n, b in blocks.items()] +
+                          [pad(steps, width(2 * H), hp)])
+        conv = torch.cat([by_head(need(f"{m}{n}.conv", b[0] * b[1], taps, **f32), *b) for n, b in blocks.items()])
+        L = {"conv": conv.T.contiguous(), "conv_bias": torch.zeros(len(conv)), "decay_log": need(m + "A_log", H, **f32),
+             "step_bias": need(m + "dt_bias", H, **f32), "head_norm": pad(need(m + "norm", dv), vp)}
+        return joint, None, L, vp
+
+    def output(m, c, vp):
+        return pad(need(m + "o", D, c.heads * c.value_dim).view(D, c.heads, c.value_dim), hp, c.heads, vp)
+
+    joint_names = {MIXER_WINDOW_ATTENTION: "qkvg", MIXER_LINEAR_ATTENTION: "qkvga", MIXER_STATE_SPACE: "recurrence",
+                   MIXER_DELTA_RULE: "recurrence"}
+    mixers = {MIXER_WINDOW_ATTENTION: window_attention, MIXER_LINEAR_ATTENTION: linear_attention, MIXER_STATE_SPACE: state_space,
+              MIXER_DELTA_RULE: delta_rule}
+
+    def one_mixer(m, c):
+        if c.mixer == MIXER_LATENT_ATTENTION:
+            L, vp = latent_attention(m, c)
+        else:
+            joint, bias, L, vp = mixers[c.mixer](m, c)
+            L[joint_names[c.mixer]] = joint
+            if bias is not None:
+                L["joint_bias"] = bias
+        L["o"] = output(m, c, vp)
+        return L
+
+    def two_mixers(m, c):
+        (ja, ba, L, va), (jb, bb, R, vb) = mixers[c.mixer](m + "left.", c), mixers[c.beside.mixer](m + "right.", c.beside)
+        L["joint"] = torch.cat([ja, jb])
+        if ba is not None or bb is not None:
+            L["joint_bias"] = torch.cat([torch.zeros(len(j), dtype=cfg.torch_dtype) if b is None else b for j, b in ((ja, ba), (jb, bb))])
+        L.update({"beside_" + k: t for k, t in R.items()})
+        oa, ob = output(m + "left.", c, va).flatten(1), output(m + "right.", c.beside, vb).flatten(1)
+        if c.join == JOIN_NORMED:
+            L.update(o=oa, beside_o=ob, side_norm=pad(need(m + "left.out", D), hp), beside_side_norm=pad(need(m + "right.out", D), hp))
+        else:
+            L["o"] = torch.cat([oa, ob], 1)
+        return L
 
     def up_matrix(prefix, n, to, gated):
         parts = ("gate", "up") if gated else ("up",)
@@ -260,15 +345,16 @@ def pack_layer_stack(cfg, tensors: dict) -> dict:
         L["expert_table"] = table.contiguous()
         return L
 
-    mixers = {MIXER_LATENT_ATTENTION: latent_attention, MIXER_WINDOW_ATTENTION: window_attention,
-              MIXER_LINEAR_ATTENTION: linear_attention}
     for i, c in enumerate(cfg.layers):
         p = f"l{i}."
-        L, vp = mixers[c.mixer](p + "mix.", c)
+        L = one_mixer(p + "mix.", c) if c.beside is None else two_mixers(p + "mix.", c)
         L["norm1"] = pad(need(p + "norm1", D), hp)
-        L["o"] = pad(need(p + "mix.o", D, c.heads * c.value_dim).view(D, c.heads, c.value_dim), hp, c.heads, vp)
+        if cfg.norm_output == NORM_BOTH:
+            L["norm1_out"] = pad(need(p + "norm1b", D), hp)
         if c.mlp != MLP_NONE:
             L["norm2"] = pad(need(p + "norm2", D), hp)
+            if cfg.norm_output == NORM_BOTH:
+                L["norm2_out"] = pad(need(p + "norm2b", D), hp)
             L.update(feed_forward(p + "mlp.", c))
         w["layers"].append(L)
     return w
