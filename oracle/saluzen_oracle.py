@@ -235,3 +235,84 @@ def forward(config, weights, tokens, dtype=torch.float64, keep_layers=False):
         trail.append(x)
     logits = rms_normalise(x, w["final.norm"], eps) @ w["head"].T
     return (logits, trail) if keep_layers else logits
+
+
+# ---- random models -------------------------------------------------------------------
+def random_model(config, seed=0):
+    """bf16 weights of the shapes `config` describes, scaled so that every mechanism contributes to the logits:
+    scores spread over a few units, decays from a few tokens to hundreds of them."""
+    g = torch.Generator().manual_seed(seed)
+    V, D = config["vocab"], config["width"]
+    w = {}
+
+    def mat(name, n, k, gain=1.0):
+        w[name] = (torch.randn(n, k, generator=g) * gain / math.sqrt(k)).to(torch.bfloat16)
+
+    def vec(name, n, centre=1.0, spread=0.2):
+        w[name] = (centre + spread * torch.randn(n, generator=g)).to(torch.bfloat16)
+
+    def uniform(name, n, lo, hi):
+        w[name] = (lo + (hi - lo) * torch.rand(n, generator=g)).to(torch.bfloat16)
+
+    def taps(name, n, t):
+        w[name] = (torch.randn(n, t, generator=g) * 1.5 / math.sqrt(t)).to(torch.bfloat16)
+
+    def attention(p, m, gate):
+        H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        for name, n, gain in (("q", H * d, 1.3), ("k", G * d, 1.3), ("v", G * dv, 1.0)):
+            mat(p + name, n, D, gain)
+            vec(f"{p}{name}.b", n, 0.0, 0.3)
+        mat(p + "g", gate, D, 1.5)
+        mat(p + "o", D, H * dv)
+
+    w["embed"] = torch.randn(V, D, generator=g).to(torch.bfloat16)
+    for i, layer in enumerate(config["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        for norm in ("norm1", "norm1b", "norm2", "norm2b")[:4 if layer.get("mlp") else 2]:
+            vec(p + norm, D)
+        if layer["type"] == "latent_attention":
+            H, d, dr, dv, r = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+            mat(p + "mix.dq", m["q_rank"], D)
+            vec(p + "mix.dq.norm", m["q_rank"])
+            mat(p + "mix.uq", H * (d + dr), m["q_rank"], 1.3)
+            if m.get("kv_from") is None:
+                mat(p + "mix.dkv", r + dr, D, 1.3)
+                vec(p + "mix.dkv.norm", r)
+            mat(p + "mix.uk", H * d, r, 1.3)
+            mat(p + "mix.uv", H * dv, r)
+            mat(p + "mix.o", D, H * dv)
+        else:
+            left, right, r = p + "mix.left.", p + "mix.right.", m["right"]
+            H, dv = r["heads"], r["vdim"]
+            if layer["type"] == "parallel":
+                attention(left, m["left"], m["left"]["heads"] * m["left"]["vdim"])
+                inner, gn = H * dv, r["groups"] * r["state"]
+                mat(right + "in", 2 * inner + 2 * gn + H, D, 1.2)
+                taps(right + "conv", inner + 2 * gn, r["conv"])
+                vec(right + "conv.b", inner + 2 * gn, 0.0, 0.3)
+                vec(right + "D", H, 0.5, 0.5)
+                vec(right + "norm", inner)
+                vec(p + "mix.left.out", D)
+                vec(p + "mix.right.out", D)
+            else:
+                attention(left, m["left"], m["left"]["heads"])
+                vec(left + "sink", m["left"]["heads"], 0.5, 1.0)
+                G, d = r["kv_heads"], r["dim"]
+                for name, n in (("q", G * d), ("k", G * d), ("v", H * dv)):
+                    mat(right + name, n, D, 1.2)
+                    taps(f"{right}{name}.conv", n, r["conv"])
+                mat(right + "a", H, D)
+                mat(right + "b", H, D, 1.5)
+                mat(right + "g", H * dv, D)
+                vec(right + "norm", dv)
+            uniform(right + "A_log", H, -2.0, 1.0)
+            uniform(right + "dt_bias", H, -5.0, 0.0)
+            mat(right + "o", D, H * dv)
+        if layer.get("mlp"):
+            n = layer["mlp"]["ff"]
+            mat(p + "mlp.gate", n, D)
+            mat(p + "mlp.up", n, D)
+            mat(p + "mlp.down", D, n)
+    vec("final.norm", D)
+    mat("head", V, D)
+    return w
