@@ -27,7 +27,7 @@ of 4096 tokens prefilled in chunks, alternating with sampled decode steps of 56 
 prefill tokens/s, decode ms/step, fraction of the tensor-pipe rate); --workload c4 is Llama-3-8B under tensor parallelism and
 --workload c5 Qwen3-30B-A3B under expert parallelism + attention TP over the N ranks (strong
 scaling, weights drawn on the device); --workload rapizen is prefill and decode of the layer-stack
-design Rapizen at three sizes beside Qwen3-MoE of the same sizes, --workload dilalix that of Dilalix; --eager / --profile-region / --profile-prefill shape a run
+design Rapizen at three sizes beside Qwen3-MoE of the same sizes, --workload dilalix that of Dilalix, --workload saluzen that of Saluzen beside Qwen3; --eager / --profile-region / --profile-prefill shape a run
 for a profiler's launch list.
 """
 from __future__ import annotations
@@ -953,6 +953,104 @@ def dilalix_work(size: str, new: bool) -> dict:
             "attention_flops_req": 4 * H * 128 * pairs}
 
 
+# name -> (width, layers, heads, KV heads, query latent, kv latent, ff, chunk, batch, context); layers in turn: attention in
+# chunks beside the delta rule, latent attention (every other one reads the latents of the one before it), attention beside
+# the state space
+SALUZEN_SIZES = {
+    "1k": (1024, 12, 8, 2, 384, 256, 3072, 1024, 64, 2048),
+    "2k": (2048, 12, 16, 4, 768, 512, 6144, 1024, 64, 2048),
+    "4k": (4096, 9, 32, 8, 1536, 512, 12288, 1024, 64, 2048),
+}
+SALUZEN_STATE, SALUZEN_TAPS, SALUZEN_ROT = 128, 4, 64    # state of the state space, taps, rotated latent dimensions
+
+
+def saluzen_pair(size: str):
+    """A Saluzen model and a Qwen3 model of the same width, depth, heads and feed-forward."""
+    from oracle import token_loop_oracle as O
+    from sglang_cpp_b200 import _lib
+    from sglang_cpp_b200.models import LayerSpec, StackConfig
+
+    D, L, H, G, qr, kr, ff, chunk, _, _ = SALUZEN_SIZES[size]
+    attention = dict(score_scale=128 ** -0.5, mixer=_lib.MIXER_WINDOW_ATTENTION, kv_heads=G, rotary_dim=128, rope_base=1e6,
+                     head_norm=False, qkv_bias=True, sink=True)
+    layers = []
+    for i in range(L):
+        if i % 3 == 0:
+            s = LayerSpec(H, 128, 128, chunk=chunk, gate=_lib.GATE_HEAD, out_scale=0.8, **attention)
+            s.beside = LayerSpec(H, 128, 128, mixer=_lib.MIXER_DELTA_RULE, kv_heads=H // 2, conv_taps=SALUZEN_TAPS)
+        elif i % 3 == 1:
+            s = LayerSpec(H, 128, 128, qr, kr, 128 ** -0.5, rotary_dim=SALUZEN_ROT, rope_base=1e4, kv_from=i - 3 if i % 6 == 4 else -1)
+        else:
+            s = LayerSpec(H, 128, 128, rope_factor=8.0, rope_low=1.0, rope_high=4.0, rope_original=8192.0, **attention)
+            s.join = _lib.JOIN_NORMED
+            s.beside = LayerSpec(D // 64, SALUZEN_STATE, 64, mixer=_lib.MIXER_STATE_SPACE, kv_heads=1, conv_taps=SALUZEN_TAPS)
+        s.mlp, s.intermediate, s.epilogue = _lib.MLP_DENSE, ff, _lib.EPILOGUE_SWIGLU
+        layers.append(s)
+    new = StackConfig(D, RAPIZEN_VOCAB, 1e-6, layers, norm_output=_lib.NORM_BOTH)
+    like = O.ModelConfig(L, D, H, G, 128, ff, RAPIZEN_VOCAB, 1e-6, 1e6, 8192, False, True, True)
+    return new, like
+
+
+def saluzen_work(size: str, new: bool) -> dict:
+    D, L, H, G, qr, kr, ff, chunk, B, ctx = SALUZEN_SIZES[size]
+    kv_tok, mlp_w, attn_w = 2 * G * 128 * 2, 3 * ff * D, D * (H + 2 * G) * 128 + H * 128 * D
+    pairs = ctx * ctx / 2                                            # (query, key) pairs of a prompt
+    if not new:
+        return {"batch": B, "context": ctx, "vocab": RAPIZEN_VOCAB, "layers": L,
+                "step_bytes": lambda keys: 2 * (L * (attn_w + mlp_w) + RAPIZEN_VOCAB * D) + L * B * keys * kv_tok,
+                "attention_bytes": lambda keys: B * keys * kv_tok,
+                "flops_tok": 2 * L * (attn_w + mlp_w) + L * 4 * H * 128 * pairs / ctx,
+                "attention_flops_req": 4 * H * 128 * pairs}
+    n_delta, n_latent, n_ssd = (sum(i % 3 == k for i in range(L)) for k in range(3))
+    n_shared = sum(i % 6 == 4 for i in range(L))
+    delta_w = attn_w + D * H + D * (3 * H * 128 + 2 * (H // 2) * 128 + 2 * H)
+    ssd_w = attn_w + D * H * 128 + D * (2 * D + 2 * SALUZEN_STATE + D // 64) + D * D
+    row = kr + SALUZEN_ROT
+    latent_w = n_latent * (D * qr + H * 128 * qr + H * (64 + 128) * kr + H * 128 * D) + (n_latent - n_shared) * D * row
+    state = 2 * 4 * (n_delta * H * 128 * 128 + n_ssd * D * SALUZEN_STATE)          # read and written per token decoded
+    in_chunk = lambda keys: (keys - 1) % chunk + 1
+    keys_read = lambda keys: n_delta * in_chunk(keys) * kv_tok + n_ssd * keys * kv_tok + n_latent * keys * row * 2
+    chunk_pairs = ctx // chunk * chunk * chunk / 2
+    recurrent = n_delta * H * (6 * 128 * 128 + 3 * 128 * 64) + n_ssd * (D // 64) * (4 * 128 * 64 + 2 * 64 * 64 + 128 * 64)
+    matrices = n_delta * delta_w + latent_w + n_ssd * ssd_w + L * mlp_w
+    attn_flops = 4 * H * 128 * (n_delta * chunk_pairs + (n_latent + n_ssd) * pairs)
+    return {"batch": B, "context": ctx, "vocab": RAPIZEN_VOCAB, "layers": L,
+            "step_bytes": lambda keys: 2 * (matrices + RAPIZEN_VOCAB * D) + B * (keys_read(keys) + state),
+            "attention_bytes": lambda keys: B * keys_read(keys) / L,
+            "flops_tok": 2 * matrices + attn_flops / ctx + recurrent,
+            "attention_flops_req": attn_flops / L}
+
+
+def run_gpu_saluzen(args):
+    """Workload "saluzen": prefill and decode of the Saluzen design at sizes that resemble a real model's layers,
+    beside Qwen3 of the same size.  (attention_us: the mean of the layers' attention launches, for latent attention
+    with its absorbed projections.)"""
+    import __graft_entry__ as entry
+
+    torch.cuda.set_device(0)
+    pkg = entry.load_package()
+    pkg.load_library()
+    sampler = ClockSampler(0)
+    sampler.start()
+    sizes = {}
+    for size in (args.size.split(",") if args.size else SALUZEN_SIZES):
+        new, like = saluzen_pair(size)
+        sizes[size] = {"saluzen": stack_arm(pkg, new, saluzen_work(size, True), args.steps, args.warmup)}
+        if not args.new_only:
+            sizes[size]["qwen3"] = stack_arm(pkg, like, saluzen_work(size, False), args.steps, args.warmup)
+    clocks = sampler.stop()
+    first = next(iter(sizes))
+    print(json.dumps({
+        "metric": "decode tokens/s (Saluzen layer stack, %s)" % first, "value": sizes[first]["saluzen"]["decode_tokens_s"],
+        "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+        "ms_per_step": sizes[first]["saluzen"]["decode_ms"], "higher_is_better": True, "scaling": "strong",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "clocks": clocks,
+        "config": {"workload": "saluzen: batch 64, context 2048, page 64; weights and caches larger than L2",
+                   "sizes": {k: dict(zip(("width", "layers", "heads", "kv_heads", "q_rank", "kv_rank", "ff", "chunk", "batch",
+                                          "context"), SALUZEN_SIZES[k])) for k in sizes}},
+        "sizes": sizes}))
+
+
 def run_gpu_dilalix(args):
     """Workload "dilalix": prefill and decode of the Dilalix design at sizes that resemble a real model's
     layers, beside Qwen3-MoE of the same size.  (attention_us covers the window attention layers only.)"""
@@ -1101,15 +1199,15 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--chunk-tokens", type=int, default=2048, help="c3: tokens a prompt advances per prefill batch")
-    ap.add_argument("--workload", default="c2", choices=["c2", "c3", "c4", "c5", "rapizen", "dilalix"],
+    ap.add_argument("--workload", default="c2", choices=["c2", "c3", "c4", "c5", "rapizen", "dilalix", "saluzen"],
                     help="c2 (default, the headline metric): Qwen3-0.6B decode, replicas when N > 1; "
                          "c3: Qwen3-0.6B chunked prefill alternating with sampled decode, one GPU; "
                          "c4: Llama-3-8B decode, tensor parallel over the N ranks; "
                          "c5: Qwen3-30B-A3B decode, experts and attention heads split over the N ranks")
     ap.add_argument("--context", type=int, default=0,
                     help="c2 only: give every prompt this length instead of U[512,2048]")
-    ap.add_argument("--size", default="", help="rapizen, dilalix: sizes to run, with commas between them (default: all)")
-    ap.add_argument("--new-only", action="store_true", help="dilalix: without the model it is measured beside")
+    ap.add_argument("--size", default="", help="rapizen, dilalix, saluzen: sizes to run, with commas between them (default: all)")
+    ap.add_argument("--new-only", action="store_true", help="dilalix, saluzen: without the model it is measured beside")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-tp-record", action="store_true",
                     help="c2 only: do not run the tensor-parallel workload after the headline")
@@ -1137,6 +1235,10 @@ def main():
         if args.gpus != 1:
             raise SystemExit("workload dilalix runs on one GPU")
         run_gpu_dilalix(args)
+    elif args.workload == "saluzen":
+        if args.gpus != 1:
+            raise SystemExit("workload saluzen runs on one GPU")
+        run_gpu_saluzen(args)
     elif args.workload == "c3":
         if args.gpus != 1:
             raise SystemExit("workload c3 runs on one GPU")
