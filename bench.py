@@ -957,9 +957,9 @@ def dilalix_work(size: str, new: bool) -> dict:
 # chunks beside the delta rule, latent attention (every other one reads the latents of the one before it), attention beside
 # the state space
 SALUZEN_SIZES = {
-    "1k": (1024, 12, 8, 2, 384, 256, 3072, 1024, 64, 2048),
-    "2k": (2048, 12, 16, 4, 768, 512, 6144, 1024, 64, 2048),
-    "4k": (4096, 9, 32, 8, 1536, 512, 12288, 1024, 64, 2048),
+    "1k": (1024, 12, 8, 2, 384, 256, 3072, 1536, 64, 2048),
+    "2k": (2048, 12, 16, 4, 768, 512, 6144, 1536, 64, 2048),
+    "4k": (4096, 9, 32, 8, 1536, 512, 12288, 1536, 64, 2048),
 }
 SALUZEN_STATE, SALUZEN_TAPS, SALUZEN_ROT = 128, 4, 64    # state of the state space, taps, rotated latent dimensions
 
@@ -1010,7 +1010,7 @@ def saluzen_work(size: str, new: bool) -> dict:
     state = 2 * 4 * (n_delta * H * 128 * 128 + n_ssd * D * SALUZEN_STATE)          # read and written per token decoded
     in_chunk = lambda keys: (keys - 1) % chunk + 1
     keys_read = lambda keys: n_delta * in_chunk(keys) * kv_tok + n_ssd * keys * kv_tok + n_latent * keys * row * 2
-    chunk_pairs = ctx // chunk * chunk * chunk / 2
+    chunk_pairs = (ctx // chunk * chunk ** 2 + (ctx % chunk) ** 2) / 2
     recurrent = n_delta * H * (6 * 128 * 128 + 3 * 128 * 64) + n_ssd * (D // 64) * (4 * 128 * 64 + 2 * 64 * 64 + 128 * 64)
     matrices = n_delta * delta_w + latent_w + n_ssd * ssd_w + L * mlp_w
     attn_flops = 4 * H * 128 * (n_delta * chunk_pairs + (n_latent + n_ssd) * pairs)

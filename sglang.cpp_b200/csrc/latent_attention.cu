@@ -27,12 +27,11 @@ __device__ __forceinline__ void put(__nv_bfloat16* p, float v) { *p = __float2bf
 // Columns [0, qp) of a token's joint row are its query latent, [qp, qp + rp) its key/value latent; each is
 // divided by its own root mean square (over the true widths) and scaled by its own weight, but for the part of
 // the key/value latent that turns with the position instead.  One warp per latent: warps 0 and 1 of a pair take
-// the two latents of one token, four tokens per CTA, the row in registers (latents of up to 8 x 256 elements;
+// the two latents of one token, four tokens per CTA, the row in registers (latents of up to kKeep x 256 elements;
 // wider ones are read again).
-template <typename T>
+template <typename T, int kKeep>
 __global__ void __launch_bounds__(256)
 latent_norm_store_kernel(const LatentNorm a) {
-    constexpr int kKeep = 8;
     pdl_launch_dependents();
     pdl_wait_prior();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -46,6 +45,11 @@ latent_norm_store_kernel(const LatentNorm a) {
     const int rope0 = kv && a.rope_dim > 0 ? a.rope_at >> 3 : nvec;   // the first vector that turns
     int64_t slot = 0;
     if (kv) slot = a.out_loc[t];
+    int pos = kv && a.rope_dim > 0 ? a.positions[t] : 0;
+    if (pos < 0 || pos >= a.max_pos) {
+        if (lane == 0) atomicExch(&a.status[kStatusBadIndex], pos + 1);
+        pos = min(max(pos, 0), a.max_pos - 1);
+    }
     Vec8 x[kKeep];
     float ss = 0.f;
 #pragma unroll
@@ -71,14 +75,6 @@ latent_norm_store_kernel(const LatentNorm a) {
         }
         dst = static_cast<T*>(a.cache) + slot * a.rp;
     }
-    int pos = 0;
-    if (kv && a.rope_dim > 0) {
-        pos = a.positions[t];
-        if (pos < 0 || pos >= a.max_pos) {
-            if (lane == 0) atomicExch(&a.status[kStatusBadIndex], pos + 1);
-            pos = min(max(pos, 0), a.max_pos - 1);
-        }
-    }
     auto emit = [&](int v, const Vec8& y) {
         Vec8 o;
         if (v < rope0) {
@@ -86,14 +82,28 @@ latent_norm_store_kernel(const LatentNorm a) {
 #pragma unroll
             for (int j = 0; j < 8; ++j) o.v[j] = y.v[j] * r * g.v[j];
         } else {
-            const int half = a.rope_dim >> 1;
+            const int half = a.rope_dim >> 1, pair0 = (v - rope0) * 4;
+            const float* ct = a.cos_t + static_cast<int64_t>(pos) * half + pair0;
+            const float* st = a.sin_t + static_cast<int64_t>(pos) * half + pair0;
+            float c[4] = {0.f, 0.f, 0.f, 0.f}, s[4] = {0.f, 0.f, 0.f, 0.f};
+            if (half % 4 == 0) {
+                if (pair0 < half) {
+                    const float4 c4 = *reinterpret_cast<const float4*>(ct), s4 = *reinterpret_cast<const float4*>(st);
+                    c[0] = c4.x, c[1] = c4.y, c[2] = c4.z, c[3] = c4.w;
+                    s[0] = s4.x, s[1] = s4.y, s[2] = s4.z, s[3] = s4.w;
+                }
+            } else {
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+                    if (pair0 + j < half) {
+                        c[j] = ct[j];
+                        s[j] = st[j];
+                    }
+            }
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                const int pair = (v - rope0) * 4 + j;
-                const float c = pair < half ? a.cos_t[static_cast<int64_t>(pos) * half + pair] : 0.f;
-                const float s = pair < half ? a.sin_t[static_cast<int64_t>(pos) * half + pair] : 0.f;
-                o.v[2 * j] = y.v[2 * j] * c - y.v[2 * j + 1] * s;
-                o.v[2 * j + 1] = y.v[2 * j + 1] * c + y.v[2 * j] * s;
+                o.v[2 * j] = y.v[2 * j] * c[j] - y.v[2 * j + 1] * s[j];
+                o.v[2 * j + 1] = y.v[2 * j + 1] * c[j] + y.v[2 * j] * s[j];
             }
         }
         store8(dst + v * 8, o);
@@ -241,7 +251,11 @@ int launch_latent_norm_store(const LatentNorm& a, int dtype, cudaStream_t stream
     // few tokens: a CTA each, for latency; many: four per CTA
     const int threads = a.tokens <= 2 * sm_count() ? 64 : 256;
     const int grid = div_ceil(a.tokens, threads / 64);
-    auto kernel = dtype == B200_DTYPE_F32 ? latent_norm_store_kernel<float> : latent_norm_store_kernel<__nv_bfloat16>;
+    const bool f32 = dtype == B200_DTYPE_F32;
+    const int widest = a.qp > a.rp ? a.qp : a.rp;
+    auto kernel = widest <= 512    ? (f32 ? latent_norm_store_kernel<float, 2> : latent_norm_store_kernel<__nv_bfloat16, 2>)
+                  : widest <= 1024 ? (f32 ? latent_norm_store_kernel<float, 4> : latent_norm_store_kernel<__nv_bfloat16, 4>)
+                                   : (f32 ? latent_norm_store_kernel<float, 8> : latent_norm_store_kernel<__nv_bfloat16, 8>);
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(grid), dim3(threads), 0, stream, dim3(1, 1, 1), a));
     return B200_OK;
 }

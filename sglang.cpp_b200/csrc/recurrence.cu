@@ -40,6 +40,14 @@ __device__ __forceinline__ T from_f32(float x) { return static_cast<T>(x); }
 template <>
 __device__ __forceinline__ __nv_bfloat16 from_f32(float x) { return __float2bfloat16_rn(x); }
 __device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    return make_float4(bf16_lo(u.x), bf16_hi(u.x), bf16_lo(u.y), bf16_hi(u.y));
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+}
 template <typename T>
 __device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
 template <>
@@ -54,22 +62,17 @@ constexpr int kStateSpace = B200_RULE_STATE_SPACE, kDelta = B200_RULE_DELTA;
 __device__ __forceinline__ int64_t values(const Recurrence& a) { return static_cast<int64_t>(a.heads) * a.padded_value_dim; }
 __device__ __forceinline__ int64_t channels(const Recurrence& a) { return values(a) + 2ll * a.kv_heads * a.padded_dim; }
 
-// log2 of a step's decay and the weight of what it writes.
-template <typename T>
-__device__ __forceinline__ float2 step_of(const Recurrence& a, const T* row, int h) {
-    const T* tail = row + values(a) + channels(a);
-    const float x = to_f32(tail[h]) + a.step_bias[h];
-    const float dt = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
-    float2 s;
-    s.x = -expf(a.decay_log[h]) * dt * kLog2e;
-    s.y = a.rule == kStateSpace ? dt : 1.f / (1.f + expf(-to_f32(tail[a.heads + h])));
-    return s;
+// log2 of a step's decay and the weight of what it writes, from a head's columns of the joint projection.
+__device__ __forceinline__ float2 make_step(int rule, float za, float zb, float step_bias, float decay_log) {
+    const float x = za + step_bias, dt = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
+    return make_float2(-expf(decay_log) * dt * kLog2e, rule == kStateSpace ? dt : 1.f / (1.f + expf(-zb)));
 }
 
 // ---- convolution, steps, unit factors ------------------------------------------------
 
 constexpr int kMixThreads = 128;
 constexpr int kMixTokens = 32;
+constexpr int kMixAhead = 4;   // tokens whose inputs are in flight
 
 // Grid: blocks of tokens, blocks of channels (8 per thread; those of k and q cover whole heads) and one for the
 // steps, requests.  TAPS 0: any number of them.
@@ -87,7 +90,9 @@ mix_kernel(const Recurrence a, int v_blocks, int heads_per_block) {
     if (blockIdx.y == gridDim.y - 1) {
         for (int i = threadIdx.x; i < n * a.heads; i += kMixThreads) {
             const int t = t0 + i / a.heads, h = i % a.heads;
-            reinterpret_cast<float2*>(a.steps)[static_cast<int64_t>(begin + t) * a.heads + h] = step_of(a, joint + t * a.joint_ld, h);
+            const T* tail = joint + t * a.joint_ld + values(a) + channels(a) + h;
+            reinterpret_cast<float2*>(a.steps)[static_cast<int64_t>(begin + t) * a.heads + h] =
+                make_step(a.rule, to_f32(tail[0]), a.rule == kDelta ? to_f32(tail[a.heads]) : 0.f, a.step_bias[h], a.decay_log[h]);
         }
         return;
     }
@@ -129,23 +134,7 @@ mix_kernel(const Recurrence a, int v_blocks, int heads_per_block) {
             }
         }
         T* out = static_cast<T*>(a.mixed) + static_cast<int64_t>(begin) * nc + c;
-        for (int t = t0; t < t0 + n; ++t) {
-            Vec8 y = bias;
-            if (TAPS > 0) {
-#pragma unroll
-                for (int i = 0; i + 1 < kWindow; ++i) x[i] = x[i + 1];
-                x[kWindow - 1] = load8(in + t * a.joint_ld);
-#pragma unroll
-                for (int i = 0; i < kWindow; ++i)
-#pragma unroll
-                    for (int j = 0; j < 8; ++j) y.v[j] = fmaf(w[i].v[j], x[i].v[j], y.v[j]);
-            } else {
-                for (int i = 0; i < taps; ++i) {
-                    const Vec8 wi = load8(a.conv + i * nc + c), xi = input(t - (taps - 1) + i);
-#pragma unroll
-                    for (int j = 0; j < 8; ++j) y.v[j] = fmaf(wi.v[j], xi.v[j], y.v[j]);
-                }
-            }
+        auto emit = [&](int t, Vec8 y) {
             float ss = 0.f;
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
@@ -154,6 +143,36 @@ mix_kernel(const Recurrence a, int v_blocks, int heads_per_block) {
             }
             store8(out + t * nc, y);
             s_part[t - t0][threadIdx.x] = ss;
+        };
+        if (TAPS > 0) {
+            for (int t = t0; t < t0 + n; t += kMixAhead) {
+                Vec8 next[kMixAhead];
+#pragma unroll
+                for (int e = 0; e < kMixAhead; ++e) next[e] = load8(in + min(t + e, t0 + n - 1) * a.joint_ld);
+#pragma unroll
+                for (int e = 0; e < kMixAhead; ++e) {
+                    if (t + e >= t0 + n) break;
+                    Vec8 y = bias;
+#pragma unroll
+                    for (int i = 0; i + 1 < kWindow; ++i) x[i] = x[i + 1];
+                    x[kWindow - 1] = next[e];
+#pragma unroll
+                    for (int i = 0; i < kWindow; ++i)
+#pragma unroll
+                        for (int j = 0; j < 8; ++j) y.v[j] = fmaf(w[i].v[j], x[i].v[j], y.v[j]);
+                    emit(t + e, y);
+                }
+            }
+        } else {
+            for (int t = t0; t < t0 + n; ++t) {
+                Vec8 y = bias;
+                for (int i = 0; i < taps; ++i) {
+                    const Vec8 wi = load8(a.conv + i * nc + c), xi = input(t - (taps - 1) + i);
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) y.v[j] = fmaf(wi.v[j], xi.v[j], y.v[j]);
+                }
+                emit(t, y);
+            }
         }
         // (a request's first block is the only one that reads the ring)
         if (blockIdx.x == 0)
@@ -175,28 +194,30 @@ mix_kernel(const Recurrence a, int v_blocks, int heads_per_block) {
 // ---- token by token: decode, and prompts that the chunked kernels do not take ------------
 
 constexpr int kStepThreads = 256;
-constexpr int kAhead = 16;   // state rows per thread, in registers
+constexpr int kMaxAhead = 16;   // state rows per thread, in registers
+constexpr int kTapsAhead = 3;   // earlier inputs of a channel fetched together
 
-// Grid: heads, requests, blocks of 4 << log_cols value columns.
-template <typename T, int RULE, bool DECODE>
-__global__ void __launch_bounds__(kStepThreads)
+// Grid: heads, requests, blocks of 4 << log_cols value columns (at most kStepThreads).
+template <typename T, int RULE, bool DECODE, int AHEAD>
+__global__ void __launch_bounds__(kStepThreads, AHEAD > 8 ? 2 : 3)
 step_kernel(const Recurrence a, int log_cols, bool finish) {
     extern __shared__ __align__(16) float smem[];
     __shared__ float s_ss[kStepThreads / 32];
     const int dk = a.padded_dim, vp = a.padded_value_dim;
     const int nv4 = 1 << log_cols, cols = nv4 * 4, groups = kStepThreads >> log_cols;
-    float *s_v = smem, *s_k = s_v + cols, *s_q = s_k + dk, *s_red = s_q + dk, *s_o = s_red + kStepThreads * 4;
+    float *s_v = smem, *s_k = s_v + cols, *s_q = s_k + dk, *s_red = s_q + dk;
     const int h = blockIdx.x, b = blockIdx.y, col0 = blockIdx.z * cols;
     const int kvh = h / (a.heads / a.kv_heads);
     const int group = threadIdx.x >> log_cols, col = (threadIdx.x & (nv4 - 1)) * 4;
     const bool active = col0 + col < vp;
     const int64_t nv = values(a), nc = channels(a);
-    float* state = a.state + (static_cast<int64_t>(a.table_idx[b]) * a.heads + h) * dk * vp + col0 + col;
+    const int64_t row_state = static_cast<int64_t>(a.table_idx[b]);
+    float* state = a.state + (row_state * a.heads + h) * dk * vp + col0 + col;
     const int cached = a.cached[b];
     pdl_launch_dependents();
-    float4 x[kAhead];
+    float4 x[AHEAD];
 #pragma unroll
-    for (int i = 0; i < kAhead; ++i) {
+    for (int i = 0; i < AHEAD; ++i) {
         const int r = group + i * groups;
         x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (active && cached > 0 && r < dk) x[i] = load4(state + static_cast<int64_t>(r) * vp);
@@ -209,34 +230,74 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
         return nv + (i < dk ? static_cast<int64_t>(kvh) * dk + i : static_cast<int64_t>(a.kv_heads + kvh) * dk + i - dk);
     };
     auto place = [&](int i) -> float& { return i < own_v ? s_v[i] : s_k[i - own_v]; };   // (s_q follows s_k)
-    T* ring = static_cast<T*>(a.conv_state) + static_cast<int64_t>(a.table_idx[b]) * a.taps * nc;
+    T* ring = static_cast<T*>(a.conv_state) + row_state * a.taps * nc;
+    const int now = DECODE ? cached % a.taps : 0;
+    float step_bias = 0.f, decay = 0.f, norm = 0.f;
     if (DECODE) {
-        for (int i = threadIdx.x; i < own; i += kStepThreads) {
-            const int64_t c = channel(i);
-            float y = a.conv_bias != nullptr ? a.conv_bias[c] : 0.f;
-            for (int j = 0; j + 1 < a.taps; ++j) {
-                const int pos = cached - (a.taps - 1) + j;
-                if (pos >= 0) y = fmaf(a.conv[j * nc + c], to_f32(ring[pos % a.taps * nc + c]), y);
+        // what the inputs before this one add to the channels, two of them at a time
+        for (int i0 = threadIdx.x; i0 < own; i0 += 2 * kStepThreads) {
+            float y[2] = {0.f, 0.f}, w[2][kTapsAhead], in[2][kTapsAhead];
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int i = i0 + e * kStepThreads;
+                const int64_t c = channel(i < own ? i : 0);
+                if (a.conv_bias != nullptr) y[e] = a.conv_bias[c];
+#pragma unroll
+                for (int m = 0; m < kTapsAhead; ++m) {
+                    const bool there = m + 1 < a.taps && cached > m;
+                    const int slot = now - 1 - m + (now - 1 - m < 0 ? a.taps : 0);
+                    w[e][m] = there ? a.conv[(a.taps - 2 - m) * nc + c] : 0.f;
+                    in[e][m] = there ? to_f32(ring[slot * nc + c]) : 0.f;
+                }
             }
-            place(i) = y;
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int i = i0 + e * kStepThreads;
+                if (i >= own) continue;
+                const int64_t c = channel(i);
+                for (int m = a.taps - 2; m >= kTapsAhead; --m)
+                    if (cached > m) y[e] = fmaf(a.conv[(a.taps - 2 - m) * nc + c], to_f32(ring[(cached - 1 - m) % a.taps * nc + c]), y[e]);
+#pragma unroll
+                for (int m = kTapsAhead - 1; m >= 0; --m) y[e] = fmaf(w[e][m], in[e][m], y[e]);
+                place(i) = y[e];
+            }
         }
+        step_bias = a.step_bias[h];
+        decay = a.decay_log[h];
+        if (finish && threadIdx.x < own_v) norm = to_f32(static_cast<const T*>(a.norm)[threadIdx.x]);
     }
+    const float skip = RULE == kStateSpace ? a.skip[h] : 0.f;
     pdl_wait_prior();
     const int begin = DECODE ? b : a.qo_indptr[b], end = DECODE ? b + 1 : a.qo_indptr[b + 1];
-    const float skip = RULE == kStateSpace ? a.skip[h] : 0.f;
     for (int64_t t = begin; t < end; ++t) {
         const T* row = static_cast<const T*>(a.joint) + t * a.joint_ld;
         float2 step;
+        float gate = 0.f;
         if (DECODE) {
-            T* now = ring + static_cast<int64_t>(cached % a.taps) * nc;
+            const T* tail = row + nv + nc;
+            const float za = to_f32(tail[h]), zb = RULE == kDelta ? to_f32(tail[a.heads + h]) : 0.f;
+            if (finish && threadIdx.x < own_v) gate = to_f32(row[static_cast<int64_t>(h) * vp + threadIdx.x]);
+            T* keep = ring + static_cast<int64_t>(now) * nc;
             const bool keeps = h % (a.heads / a.kv_heads) == 0 && blockIdx.z == 0;   // k and q are shared
-            for (int i = threadIdx.x; i < own; i += kStepThreads) {
-                const int64_t c = channel(i);
-                const T in = row[nv + c];
-                place(i) = to_f32(from_f32<T>(silu<T>(fmaf(a.conv[(a.taps - 1) * nc + c], to_f32(in), place(i)))));
-                if (i < own_v || keeps) now[c] = in;
+            for (int i0 = threadIdx.x; i0 < own; i0 += 2 * kStepThreads) {
+                T in[2];
+                float w[2];
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int i = i0 + e * kStepThreads;
+                    const int64_t c = channel(i < own ? i : 0);
+                    in[e] = row[nv + c];
+                    w[e] = a.conv[(a.taps - 1) * nc + c];
+                }
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int i = i0 + e * kStepThreads;
+                    if (i >= own) continue;
+                    place(i) = to_f32(from_f32<T>(silu<T>(fmaf(w[e], to_f32(in[e]), place(i)))));
+                    if (i < own_v || keeps) keep[channel(i)] = in[e];
+                }
             }
-            step = step_of(a, row, h);
+            step = make_step(RULE, za, zb, step_bias, decay);
         } else {
             const T* mixed = static_cast<const T*>(a.mixed) + t * nc;
             for (int i = threadIdx.x; i < own; i += kStepThreads) place(i) = to_f32(mixed[channel(i)]);
@@ -264,7 +325,7 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
         if (RULE == kDelta) {
             float4 p = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-            for (int i = 0; i < kAhead; ++i) {
+            for (int i = 0; i < AHEAD; ++i) {
                 const int r = group + i * groups;
                 if (r < dk) {
                     const float k = s_k[r];
@@ -290,7 +351,7 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
         }
         float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-        for (int i = 0; i < kAhead; ++i) {
+        for (int i = 0; i < AHEAD; ++i) {
             const int r = group + i * groups;
             if (r < dk) {
                 const float k = kf * s_k[r], q = s_q[r];
@@ -308,32 +369,28 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
         *reinterpret_cast<float4*>(s_red + group * cols + col) = o;
         __syncthreads();
         T* out = static_cast<T*>(a.out) + t * a.out_ld + static_cast<int64_t>(h) * vp + col0;
-        float ss = 0.f;
-        for (int c = threadIdx.x; c < own_v; c += kStepThreads) {
-            float y = 0.f;
+        const int c = threadIdx.x;
+        float y = 0.f;
+        if (c < own_v) {
             for (int i = 0; i < groups; ++i) y += s_red[i * cols + c];
             y *= qf;
             if (RULE == kStateSpace) y = fmaf(skip, s_v[c], y);
             if (!finish) out[c] = from_f32<T>(y);
-            s_o[c] = y;
-            ss += y * y;
         }
-        if (finish) {   // the whole head is here: norm and gate
+        if (DECODE && RULE == kDelta && finish) {   // the whole head is here: norm and gate
             const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-            ss = warp_sum(ss);
+            float ss = warp_sum(y * y);
             if (lane == 0) s_ss[warp] = ss;
             __syncthreads();
             ss = warp_sum(lane < kStepThreads / 32 ? s_ss[lane] : 0.f);
             const float scale = rsqrtf(ss / static_cast<float>(a.value_dim) + a.eps) * a.out_scale;
-            for (int c = threadIdx.x; c < own_v; c += kStepThreads)
-                out[c] = from_f32<T>(s_o[c] * scale * to_f32(static_cast<const T*>(a.norm)[c]) *
-                                     silu<T>(to_f32(row[static_cast<int64_t>(h) * vp + c])));
+            if (c < own_v) out[c] = from_f32<T>(y * scale * norm * silu<T>(gate));
         }
         if (!DECODE) __syncthreads();   // everything in shared memory has been used
     }
     if (DECODE || !active || begin >= end) return;
 #pragma unroll
-    for (int i = 0; i < kAhead; ++i) {
+    for (int i = 0; i < AHEAD; ++i) {
         const int r = group + i * groups;
         if (r < dk) *reinterpret_cast<float4*>(state + static_cast<int64_t>(r) * vp) = x[i];
     }
@@ -341,7 +398,7 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
 
 // ---- norm and gate of raw outputs, in place ------------------------------------------------
 
-// Delta rule: one warp per (token, head).
+// Delta rule: one warp per (token, head), four elements per lane in registers (more, for wide heads, read again).
 constexpr int kFinishWarps = 8;
 
 template <typename T>
@@ -353,24 +410,28 @@ finish_heads_kernel(const Recurrence a) {
     pdl_wait_prior();
     if (row >= static_cast<unsigned>(a.tokens) * a.heads) return;
     const int64_t t = row / a.heads;
-    const int h = static_cast<int>(row - t * a.heads);
+    const int h = static_cast<int>(row - t * a.heads), c0 = lane * 4;
     T* out = static_cast<T*>(a.out) + t * a.out_ld + static_cast<int64_t>(h) * vp;
     const T* gate = static_cast<const T*>(a.joint) + t * a.joint_ld + static_cast<int64_t>(h) * vp;
     const T* norm = static_cast<const T*>(a.norm);
-    float ss = 0.f;
-    for (int c = lane * 8; c < vp; c += 256) {
-        const Vec8 o = load8(out + c);
-#pragma unroll
-        for (int j = 0; j < 8; ++j) ss += o.v[j] * o.v[j];
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f), g = o, w = o;
+    if (c0 < vp) {
+        o = load4(out + c0);
+        g = load4(gate + c0);
+        w = load4(norm + c0);
+    }
+    float ss = o.x * o.x + o.y * o.y + o.z * o.z + o.w * o.w;
+    for (int c = c0 + 128; c < vp; c += 128) {
+        const float4 y = load4(out + c);
+        ss += y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w;
     }
     const float scale = rsqrtf(warp_sum(ss) / static_cast<float>(a.value_dim) + a.eps) * a.out_scale;
-    for (int c = lane * 8; c < vp; c += 256) {
-        Vec8 o = load8(out + c);
-        const Vec8 g = load8(gate + c), w = load8(norm + c);
-#pragma unroll
-        for (int j = 0; j < 8; ++j) o.v[j] *= scale * w.v[j] * silu<T>(g.v[j]);
-        store8(out + c, o);
-    }
+    auto emit = [&](int c, const float4& y, const float4& z, const float4& n) {
+        store4(out + c, make_float4(y.x * scale * n.x * silu<T>(z.x), y.y * scale * n.y * silu<T>(z.y),
+                                    y.z * scale * n.z * silu<T>(z.z), y.w * scale * n.w * silu<T>(z.w)));
+    };
+    if (c0 < vp) emit(c0, o, g, w);
+    for (int c = c0 + 128; c < vp; c += 128) emit(c, load4(out + c), load4(gate + c), load4(norm + c));
 }
 
 // State space: one CTA per (token, part of the norm).  A part is a run of the concatenated heads without their
@@ -446,7 +507,6 @@ finish_parts_kernel(const Recurrence a) {
 // ---- chunked ---------------------------------------------------------------------------------
 
 constexpr int kChunk = 64;            // tokens per chunk
-constexpr int kSlice = 64;            // value columns per CTA
 constexpr int kPad = 8;               // bf16 elements behind every shared row (conflict-free ldmatrix)
 constexpr int kTiles = 10;            // 16 x 16 tiles on and below the diagonal
 constexpr int kMatrixVecs = kTiles * 2 * 32;   // uint4 per matrix: [tile][upper / lower part][lane]
@@ -494,6 +554,12 @@ struct PrepareSmem {
     float sum[2][kChunk], weight[2][kChunk], kf[kChunk], qf[kChunk];
 };
 
+// Barrier of the two warps that work on one head.
+__device__ __forceinline__ void pair_sync() {
+    if (threadIdx.x < 64) asm volatile("bar.sync 1, 64;" ::: "memory");
+    else asm volatile("bar.sync 2, 64;" ::: "memory");
+}
+
 // The columns of (I + A)^-1 from BASE on, one per lane, by forward substitution; those before it are zero in rows
 // below BASE.
 template <int BASE>
@@ -513,11 +579,10 @@ __device__ __forceinline__ void invert_columns(float* a) {
         }
         x[i] = (acc[0] + acc[1]) + (acc[2] + acc[3]);
     }
-    const int pair = 1 + (static_cast<int>(threadIdx.x) >> 6);
-    asm volatile("bar.sync %0, 64;" ::"r"(pair) : "memory");   // both warps have read A
+    pair_sync();   // both warps have read A
 #pragma unroll
     for (int i = 0; i < kChunk; ++i) a[i * kARow + BASE + lane] = i < BASE ? 0.f : x[i < BASE ? BASE : i];
-    asm volatile("bar.sync %0, 64;" ::"r"(pair) : "memory");
+    pair_sync();
 }
 
 // Grid: chunks of the longest request, k / q heads, requests.
@@ -597,27 +662,40 @@ prepare_kernel(const Recurrence a) {
         for (int hp = 0; hp < 2; ++hp) {
             if (h0 + hp >= group) continue;
             uint4* out = chunks + (static_cast<int64_t>(kvh * group + h0 + hp) * kMatrices) * kMatrixVecs + lane;
-            const float* sum = S.sum[hp];
-            const float* weight = S.weight[hp];
+            const int t0 = warp * 16 + g;
+            const float sum_t[2] = {S.sum[hp][t0], S.sum[hp][t0 + 8]};
+            float q_t[2] = {1.f, 1.f}, k_t[2] = {0.f, 0.f};
+            if (RULE == kDelta) {
+                q_t[0] = S.qf[t0];
+                q_t[1] = S.qf[t0 + 8];
+                k_t[0] = S.kf[t0] * S.weight[hp][t0];
+                k_t[1] = S.kf[t0 + 8] * S.weight[hp][t0 + 8];
+            }
 #pragma unroll
             for (int kt = 0; kt < 4; ++kt) {
                 if (kt > warp) continue;
                 uint32_t hi[4], lo[4];
 #pragma unroll
-                for (int part = 0; part < 4; ++part) {   // rows g, g + 8 of the left tile, then of the right one
-                    const int t = warp * 16 + g + (part & 1) * 8, s = kt * 16 + (part >> 1) * 8 + 2 * tq;
-                    const float* src = qk[2 * kt + (part >> 1)] + (part & 1) * 2;
-                    float p[2];
+                for (int side = 0; side < 2; ++side) {
+                    const int s = kt * 16 + side * 8 + 2 * tq;
+                    const float2 sum_s = *reinterpret_cast<const float2*>(&S.sum[hp][s]);
+                    const float2 f_s = RULE == kDelta ? *reinterpret_cast<const float2*>(&S.kf[s])
+                                                      : *reinterpret_cast<const float2*>(&S.weight[hp][s]);
+                    float2 am[2];
 #pragma unroll
-                    for (int e = 0; e < 2; ++e) {
-                        const float ratio = s + e <= t ? ex2(sum[t] - sum[s + e]) : 0.f;
-                        p[e] = src[e] * ratio * (RULE == kDelta ? S.qf[t] * S.kf[s + e] : weight[s + e]);
-                        if (RULE == kDelta)
-                            S.a[hp][t * kARow + s + e] = s + e < t ? kk[2 * kt + (part >> 1)][(part & 1) * 2 + e] * ratio *
-                                                                         (S.kf[t] * S.kf[s + e]) * weight[t]
-                                                                   : 0.f;
+                    for (int half = 0; half < 2; ++half) {   // rows g, g + 8
+                        const int t = t0 + half * 8, tile = 2 * kt + side;
+                        const float rx = (s <= t ? ex2(sum_t[half] - sum_s.x) : 0.f) * f_s.x;
+                        const float ry = (s + 1 <= t ? ex2(sum_t[half] - sum_s.y) : 0.f) * f_s.y;
+                        split2(qk[tile][2 * half] * (rx * q_t[half]), qk[tile][2 * half + 1] * (ry * q_t[half]), hi[2 * side + half],
+                               lo[2 * side + half]);
+                        am[half] = make_float2(s < t ? kk[tile][2 * half] * (rx * k_t[half]) : 0.f,
+                                               s + 1 < t ? kk[tile][2 * half + 1] * (ry * k_t[half]) : 0.f);
                     }
-                    split2(p[0], p[1], hi[part], lo[part]);
+                    if (RULE == kDelta) {
+                        *reinterpret_cast<float2*>(&S.a[hp][t0 * kARow + s]) = am[0];
+                        *reinterpret_cast<float2*>(&S.a[hp][(t0 + 8) * kARow + s]) = am[1];
+                    }
                 }
                 const int tile = warp * (warp + 1) / 2 + kt;
                 out[tile * 64] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
@@ -652,11 +730,10 @@ prepare_kernel(const Recurrence a) {
     }
 }
 
-constexpr int kWalkThreads = 256;
-
-template <int DK, int RULE>
+// SLICE value columns per CTA, 16 per warp.
+template <int DK, int RULE, int SLICE>
 struct WalkSmem {
-    static constexpr int kRow = DK + kPad, kVRow = kSlice + kPad;
+    static constexpr int kRow = DK + kPad, kVRow = SLICE + kPad;
     __nv_bfloat16 k[2][kChunk * kRow], q[2][kChunk * kRow], v[2][kChunk * kVRow];   // this chunk's and the next one's
     __nv_bfloat16 sh[DK * kVRow], sl[DK * kVRow];                                   // the state
     __nv_bfloat16 rh[RULE == kDelta ? kChunk * kVRow : 8], rl[RULE == kDelta ? kChunk * kVRow : 8];   // beta (V - G K S)
@@ -668,19 +745,20 @@ struct WalkSmem {
     float keep[2];             // G_n
 };
 
-// Grid: slices of 64 value columns, heads, requests.
-template <int DK, int RULE>
-__global__ void __launch_bounds__(kWalkThreads, 1)
+// Grid: slices of the value columns, heads, requests.
+template <int DK, int RULE, int SLICE>
+__global__ void __launch_bounds__(SLICE * 8, 512 / (SLICE * 8))
 chunk_kernel(const Recurrence a) {
-    using Smem = WalkSmem<DK, RULE>;
+    using Smem = WalkSmem<DK, RULE, SLICE>;
+    constexpr int kWalkThreads = SLICE * 8;             // four tiles of tokens times 16 columns per warp
     constexpr int ROW = Smem::kRow, VROW = Smem::kVRow, kMatrices = RULE == kDelta ? 2 : 1;
-    constexpr int kColSplit = 128 / DK;                  // warps that share 16 state rows
-    constexpr int kStateTiles = kSlice / 8 / kColSplit;  // 8-column tiles of state per warp
+    constexpr int kColSplit = SLICE * 4 / DK;            // warps that share 16 state rows
+    constexpr int kStateTiles = SLICE / 8 / kColSplit;   // 8-column tiles of state per warp
     extern __shared__ __align__(16) uint8_t smem_raw[];
     Smem& S = *reinterpret_cast<Smem*>(smem_raw);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, tq = lane & 3, mi = lane >> 3, r8 = lane & 7;
-    const int h = blockIdx.y, req = blockIdx.z, v0 = blockIdx.x * kSlice;
+    const int h = blockIdx.y, req = blockIdx.z, v0 = blockIdx.x * SLICE;
     const int vp = a.padded_value_dim, kvh = h / (a.heads / a.kv_heads);
     pdl_launch_dependents();
     pdl_wait_prior();
@@ -699,8 +777,8 @@ chunk_kernel(const Recurrence a) {
             cp_async16(smem_u32(&S.k[buf][t * ROW + c]), row, t < n);
             cp_async16(smem_u32(&S.q[buf][t * ROW + c]), row + to_q, t < n);
         }
-        for (int i = threadIdx.x; i < kChunk * (kSlice / 8); i += kWalkThreads) {
-            const int t = i / (kSlice / 8), c = (i % (kSlice / 8)) * 8;
+        for (int i = threadIdx.x; i < kChunk * (SLICE / 8); i += kWalkThreads) {
+            const int t = i / (SLICE / 8), c = (i % (SLICE / 8)) * 8;
             cp_async16(smem_u32(&S.v[buf][t * VROW + c]), mixed + static_cast<int64_t>(t < n ? s0 + t : s0) * nc + at_v + c, t < n);
         }
     };
@@ -742,7 +820,7 @@ chunk_kernel(const Recurrence a) {
 
     // This warp's part of the state: 16 rows from row0, kStateTiles tiles of 8 columns from col0, in the layout of an
     // MMA accumulator.
-    const int row0 = warp / kColSplit * 16, col0 = warp % kColSplit * (kSlice / kColSplit);
+    const int row0 = warp / kColSplit * 16, col0 = warp % kColSplit * (SLICE / kColSplit);
     float* state = a.state + (static_cast<int64_t>(a.table_idx[req]) * a.heads + h) * DK * vp + v0;
     float st[kStateTiles][4];
     const bool fresh = a.cached[req] == 0;
@@ -773,8 +851,8 @@ chunk_kernel(const Recurrence a) {
         fetch_factors(0);
         put_factors(0);
     }
-    // 16 tokens x 32 columns of the products per warp; the two warps of a scheduler share out the triangle evenly
-    const int mt = warp < 4 ? warp : 7 - warp, oc0 = (warp >> 2) * 32;
+    // 16 tokens x 16 columns of the products per warp; the warps of a scheduler share out the triangle evenly
+    const int mt = (warp + (warp >> 2)) & 3, oc0 = (warp >> 2) * 16;
     const float skip = RULE == kStateSpace ? a.skip[h] : 0.f;
     const uint4* chunks = static_cast<const uint4*>(a.chunks) +
                           (chunk_number(begin, req, 0) * a.heads + h) * kMatrices * kMatrixVecs + mt * (mt + 1) / 2 * 64 + lane;
@@ -789,25 +867,22 @@ chunk_kernel(const Recurrence a) {
                 lo[kt] = __ldg(m + kt * 64 + 32);
             }
     };
-    auto multiply = [&](float (&acc)[4][4], const uint4 (&hi)[4], const uint4 (&lo)[4], const __nv_bfloat16* xh, const __nv_bfloat16* xl) {
+    auto multiply = [&](float (&acc)[2][4], const uint4 (&hi)[4], const uint4 (&lo)[4], const __nv_bfloat16* xh, const __nv_bfloat16* xl) {
 #pragma unroll
         for (int kt = 0; kt < 4; ++kt) {
             if (kt > mt) continue;
             const uint32_t ah[4] = {hi[kt].x, hi[kt].y, hi[kt].z, hi[kt].w}, al[4] = {lo[kt].x, lo[kt].y, lo[kt].z, lo[kt].w};
-#pragma unroll
-            for (int np = 0; np < 2; ++np) {
-                const int off = (kt * 16 + (mi & 1) * 8 + r8) * VROW + oc0 + np * 16 + (mi >> 1) * 8;
-                uint32_t b0, b1, b2, b3;
-                ldmatrix_x4_trans(smem_u32(xh + off), b0, b1, b2, b3);
-                mma_bf16_16816(acc[2 * np], ah, b0, b1);
-                mma_bf16_16816(acc[2 * np + 1], ah, b2, b3);
-                mma_bf16_16816(acc[2 * np], al, b0, b1);
-                mma_bf16_16816(acc[2 * np + 1], al, b2, b3);
-                if (xl != nullptr) {
-                    ldmatrix_x4_trans(smem_u32(xl + off), b0, b1, b2, b3);
-                    mma_bf16_16816(acc[2 * np], ah, b0, b1);
-                    mma_bf16_16816(acc[2 * np + 1], ah, b2, b3);
-                }
+            const int off = (kt * 16 + (mi & 1) * 8 + r8) * VROW + oc0 + (mi >> 1) * 8;
+            uint32_t b0, b1, b2, b3;
+            ldmatrix_x4_trans(smem_u32(xh + off), b0, b1, b2, b3);
+            mma_bf16_16816(acc[0], ah, b0, b1);
+            mma_bf16_16816(acc[1], ah, b2, b3);
+            mma_bf16_16816(acc[0], al, b0, b1);
+            mma_bf16_16816(acc[1], al, b2, b3);
+            if (xl != nullptr) {
+                ldmatrix_x4_trans(smem_u32(xl + off), b0, b1, b2, b3);
+                mma_bf16_16816(acc[0], ah, b0, b1);
+                mma_bf16_16816(acc[1], ah, b2, b3);
             }
         }
     };
@@ -822,15 +897,12 @@ chunk_kernel(const Recurrence a) {
             load_chunk(s0 + kChunk, buf ^ 1);
             if (warp == 0) fetch_factors(s0 + kChunk);
         }
-        uint4 ph[4], pl[4], th[4], tl[4];
-        if (mine) {
-            if (RULE == kDelta) load_matrix(chunks + kMatrixVecs, th, tl);
-            load_matrix(chunks, ph, pl);
-        }
+        uint4 mh[4], ml[4];   // the inverse, then P
+        if (mine) load_matrix(RULE == kDelta ? chunks + kMatrixVecs : chunks, mh, ml);
         const __nv_bfloat16 *K = S.k[buf], *Q = S.q[buf], *V = S.v[buf];
         const int ta = mt * 16 + g, tb = ta + 8;   // this thread's rows of the products
         // ---- Q S and K S ----
-        float o[4][4] = {}, u[4][4] = {};
+        float o[2][4] = {}, u[2][4] = {};
         if (mine) {
 #pragma unroll
             for (int ks = 0; ks < DK / 16; ++ks) {
@@ -838,18 +910,15 @@ chunk_kernel(const Recurrence a) {
                 const int aoff = (mt * 16 + (mi & 1) * 8 + r8) * ROW + ks * 16 + (mi >> 1) * 8;
                 ldmatrix_x4(smem_u32(&Q[aoff]), aq[0], aq[1], aq[2], aq[3]);
                 if (RULE == kDelta) ldmatrix_x4(smem_u32(&K[aoff]), ak[0], ak[1], ak[2], ak[3]);
+                const int soff = (ks * 16 + (mi & 1) * 8 + r8) * VROW + oc0 + (mi >> 1) * 8;
 #pragma unroll
-                for (int np = 0; np < 2; ++np) {
-                    const int soff = (ks * 16 + (mi & 1) * 8 + r8) * VROW + oc0 + np * 16 + (mi >> 1) * 8;
-#pragma unroll
-                    for (int part = 0; part < 2; ++part) {
-                        ldmatrix_x4_trans(smem_u32(part == 0 ? &S.sh[soff] : &S.sl[soff]), b0, b1, b2, b3);
-                        mma_bf16_16816(o[2 * np], aq, b0, b1);
-                        mma_bf16_16816(o[2 * np + 1], aq, b2, b3);
-                        if (RULE == kDelta) {
-                            mma_bf16_16816(u[2 * np], ak, b0, b1);
-                            mma_bf16_16816(u[2 * np + 1], ak, b2, b3);
-                        }
+                for (int part = 0; part < 2; ++part) {
+                    ldmatrix_x4_trans(smem_u32(part == 0 ? &S.sh[soff] : &S.sl[soff]), b0, b1, b2, b3);
+                    mma_bf16_16816(o[0], aq, b0, b1);
+                    mma_bf16_16816(o[1], aq, b2, b3);
+                    if (RULE == kDelta) {
+                        mma_bf16_16816(u[0], ak, b0, b1);
+                        mma_bf16_16816(u[1], ak, b2, b3);
                     }
                 }
             }
@@ -859,7 +928,7 @@ chunk_kernel(const Recurrence a) {
             if (mine) {
                 const float ba = S.beta[buf][ta], bb = S.beta[buf][tb], ra = S.read[buf][ta], rb = S.read[buf][tb];
 #pragma unroll
-                for (int j = 0; j < 4; ++j)
+                for (int j = 0; j < 2; ++j)
 #pragma unroll
                     for (int half = 0; half < 2; ++half) {
                         const int at = (half ? tb : ta) * VROW + oc0 + j * 8 + 2 * tq;
@@ -873,12 +942,15 @@ chunk_kernel(const Recurrence a) {
                     }
             }
             __syncthreads();
-            if (mine) multiply(u, th, tl, S.rh, S.rl);
+            if (mine) {
+                multiply(u, mh, ml, S.rh, S.rl);
+                load_matrix(chunks, mh, ml);
+            }
         }
         if (mine) {
             const float wa = S.write[buf][ta], wb = S.write[buf][tb];
 #pragma unroll
-            for (int j = 0; j < 4; ++j)
+            for (int j = 0; j < 2; ++j)
 #pragma unroll
                 for (int half = 0; half < 2; ++half) {
                     const int at = (half ? tb : ta) * VROW + oc0 + j * 8 + 2 * tq;
@@ -904,21 +976,21 @@ chunk_kernel(const Recurrence a) {
         if (mine) {
             const float ga = S.out[buf][ta], gb = S.out[buf][tb];
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
+            for (int j = 0; j < 2; ++j) {
                 o[j][0] *= ga;
                 o[j][1] *= ga;
                 o[j][2] *= gb;
                 o[j][3] *= gb;
             }
-            if (RULE == kDelta) multiply(o, ph, pl, S.uh, S.ul);
-            else multiply(o, ph, pl, V, nullptr);
+            if (RULE == kDelta) multiply(o, mh, ml, S.uh, S.ul);
+            else multiply(o, mh, ml, V, nullptr);
             __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + static_cast<int64_t>(begin + s0) * a.out_ld + at_v + oc0 + 2 * tq;
 #pragma unroll
             for (int half = 0; half < 2; ++half) {
                 const int t = half ? tb : ta;
                 if (t >= n) continue;
 #pragma unroll
-                for (int j = 0; j < 4; ++j) {
+                for (int j = 0; j < 2; ++j) {
                     float x = o[j][2 * half], y = o[j][2 * half + 1];
                     if (RULE == kStateSpace) {
                         const uint32_t v = *reinterpret_cast<const uint32_t*>(&V[t * VROW + oc0 + j * 8 + 2 * tq]);
@@ -966,7 +1038,7 @@ chunk_kernel(const Recurrence a) {
 }
 
 bool chunked_supported(const Recurrence& a, int dtype) {
-    return dtype == B200_DTYPE_BF16 && !a.plain && (a.padded_dim == 64 || a.padded_dim == 128) && a.padded_value_dim % kSlice == 0;
+    return dtype == B200_DTYPE_BF16 && !a.plain && (a.padded_dim == 64 || a.padded_dim == 128) && a.padded_value_dim % 64 == 0;
 }
 
 int max_smem(const void* kernel, size_t bytes) {
@@ -991,19 +1063,23 @@ int launch_chunked(const Recurrence& a, cudaStream_t stream) {
     if (err != B200_OK) return err;
     B200_CHECK_CUDA(launch_kernel(prepare, dim3(div_ceil(a.max_extend, kChunk), a.kv_heads, a.batch), dim3(kPrepareThreads),
                                   sizeof(PrepareSmem), stream, dim3(1, 1, 1), a));
-    auto kernel = a.padded_dim == 64 ? chunk_kernel<64, RULE> : chunk_kernel<128, RULE>;
-    const size_t smem = a.padded_dim == 64 ? sizeof(WalkSmem<64, RULE>) : sizeof(WalkSmem<128, RULE>);
+    // the state space has room for two CTAs per SM
+    constexpr int SLICE = RULE == kDelta ? 64 : 32;
+    auto kernel = a.padded_dim == 64 ? chunk_kernel<64, RULE, SLICE> : chunk_kernel<128, RULE, SLICE>;
+    const size_t smem = a.padded_dim == 64 ? sizeof(WalkSmem<64, RULE, SLICE>) : sizeof(WalkSmem<128, RULE, SLICE>);
     err = max_smem(reinterpret_cast<const void*>(kernel), smem);
     if (err != B200_OK) return err;
-    B200_CHECK_CUDA(launch_kernel(kernel, dim3(a.padded_value_dim / kSlice, a.heads, a.batch), dim3(kWalkThreads), smem, stream,
+    B200_CHECK_CUDA(launch_kernel(kernel, dim3(a.padded_value_dim / SLICE, a.heads, a.batch), dim3(SLICE * 8), smem, stream,
                                   dim3(1, 1, 1), a));
     return B200_OK;
 }
 
 template <typename T, int RULE>
 int launch_steps(const Recurrence& a, int log_cols, int slices, bool finish, cudaStream_t stream) {
-    const size_t smem = (2ull * (4u << log_cols) + 2ull * a.padded_dim + kStepThreads * 4) * 4;
-    auto kernel = a.decode ? step_kernel<T, RULE, true> : step_kernel<T, RULE, false>;
+    const size_t smem = ((4ull << log_cols) + 2ull * a.padded_dim + kStepThreads * 4) * 4;
+    const bool few = div_ceil(a.padded_dim, kStepThreads >> log_cols) <= 8;
+    auto kernel = a.decode ? (few ? step_kernel<T, RULE, true, 8> : step_kernel<T, RULE, true, kMaxAhead>)
+                           : (few ? step_kernel<T, RULE, false, 8> : step_kernel<T, RULE, false, kMaxAhead>);
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(a.heads, a.batch, slices), dim3(kStepThreads), smem, stream, dim3(1, 1, 1), a,
                                   log_cols, finish));
     return B200_OK;
@@ -1019,10 +1095,10 @@ int run(const Recurrence& a, int dtype, cudaStream_t stream) {
     if (!a.decode && chunked_supported(a, dtype)) {
         err = delta ? launch_chunked<kDelta>(a, stream) : launch_chunked<kStateSpace>(a, stream);
     } else {
-        // groups of four columns per CTA: a thread has room for kAhead rows
-        const int most = kAhead * kStepThreads / a.padded_dim;
+        // groups of four columns per CTA: a thread has room for kMaxAhead rows, and one output column
+        const int most = kMaxAhead * kStepThreads / a.padded_dim;
         int log_cols = 0;
-        while ((4 << log_cols) < a.padded_value_dim && (2 << log_cols) <= most && (2 << log_cols) <= kStepThreads) ++log_cols;
+        while ((4 << log_cols) < a.padded_value_dim && (2 << log_cols) <= most && (8 << log_cols) <= kStepThreads) ++log_cols;
         const int slices = div_ceil(a.padded_value_dim, 4 << log_cols);
         finished = a.decode && delta && slices == 1;
         err = delta ? launch_steps<T, kDelta>(a, log_cols, slices, finished, stream)
@@ -1043,7 +1119,7 @@ int run(const Recurrence& a, int dtype, cudaStream_t stream) {
 
 }  // namespace
 
-// A thread of the step kernel holds kAhead state rows of four columns.
+// A thread of the step kernel holds kMaxAhead state rows of four columns.
 bool recurrence_supported(int padded_value_dim, int padded_dim, int taps) {
     return padded_value_dim <= 65535 && padded_dim <= 1024 && taps >= 1 && taps <= kMaxTaps;
 }
