@@ -70,9 +70,36 @@ __device__ __forceinline__ float2 make_step(int rule, float za, float zb, float 
 
 // ---- convolution, steps, unit factors ------------------------------------------------
 
+// Eight elements as they are in memory.
+template <typename T>
+struct Packed8;
+template <>
+struct __align__(16) Packed8<__nv_bfloat16> {
+    uint4 u;
+};
+template <>
+struct __align__(16) Packed8<float> {
+    float4 a, b;
+};
+template <typename T>
+__device__ __forceinline__ Packed8<T> pack8(const Vec8& x);
+template <>
+__device__ __forceinline__ Packed8<float> pack8(const Vec8& x) {
+    return {make_float4(x.v[0], x.v[1], x.v[2], x.v[3]), make_float4(x.v[4], x.v[5], x.v[6], x.v[7])};
+}
+template <>
+__device__ __forceinline__ Packed8<__nv_bfloat16> pack8(const Vec8& x) {
+    return {make_uint4(pack_bf16(x.v[0], x.v[1]), pack_bf16(x.v[2], x.v[3]), pack_bf16(x.v[4], x.v[5]), pack_bf16(x.v[6], x.v[7]))};
+}
+__device__ __forceinline__ Vec8 unpack8(const Packed8<float>& p) { return {{p.a.x, p.a.y, p.a.z, p.a.w, p.b.x, p.b.y, p.b.z, p.b.w}}; }
+__device__ __forceinline__ Vec8 unpack8(const Packed8<__nv_bfloat16>& p) {
+    return {{bf16_lo(p.u.x), bf16_hi(p.u.x), bf16_lo(p.u.y), bf16_hi(p.u.y), bf16_lo(p.u.z), bf16_hi(p.u.z), bf16_lo(p.u.w),
+             bf16_hi(p.u.w)}};
+}
+
 constexpr int kMixThreads = 128;
 constexpr int kMixTokens = 32;
-constexpr int kMixAhead = 4;   // tokens whose inputs are in flight
+constexpr int kMixAhead = 2;   // tokens whose inputs are in flight
 
 // Grid: blocks of tokens, blocks of channels (8 per thread; those of k and q cover whole heads) and one for the
 // steps, requests.  TAPS 0: any number of them.
@@ -134,28 +161,32 @@ mix_kernel(const Recurrence a, int v_blocks, int heads_per_block) {
             }
         }
         T* out = static_cast<T*>(a.mixed) + static_cast<int64_t>(begin) * nc + c;
+        const bool units = heads && a.rule == kDelta;
         auto emit = [&](int t, Vec8 y) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) y.v[j] = silu<T>(y.v[j]);
+            const auto packed = pack8<T>(y);
+            *reinterpret_cast<Packed8<T>*>(out + t * nc) = packed;
+            if (!units) return;
+            y = unpack8(packed);
             float ss = 0.f;
 #pragma unroll
-            for (int j = 0; j < 8; ++j) {
-                y.v[j] = to_f32(from_f32<T>(silu<T>(y.v[j])));
-                ss += y.v[j] * y.v[j];
-            }
-            store8(out + t * nc, y);
+            for (int j = 0; j < 8; ++j) ss += y.v[j] * y.v[j];
             s_part[t - t0][threadIdx.x] = ss;
         };
         if (TAPS > 0) {
             for (int t = t0; t < t0 + n; t += kMixAhead) {
-                Vec8 next[kMixAhead];
+                Packed8<T> next[kMixAhead];
 #pragma unroll
-                for (int e = 0; e < kMixAhead; ++e) next[e] = load8(in + min(t + e, t0 + n - 1) * a.joint_ld);
+                for (int e = 0; e < kMixAhead; ++e)
+                    next[e] = *reinterpret_cast<const Packed8<T>*>(in + min(t + e, t0 + n - 1) * a.joint_ld);
 #pragma unroll
                 for (int e = 0; e < kMixAhead; ++e) {
                     if (t + e >= t0 + n) break;
                     Vec8 y = bias;
 #pragma unroll
                     for (int i = 0; i + 1 < kWindow; ++i) x[i] = x[i + 1];
-                    x[kWindow - 1] = next[e];
+                    x[kWindow - 1] = unpack8(next[e]);
 #pragma unroll
                     for (int i = 0; i < kWindow; ++i)
 #pragma unroll
@@ -543,6 +574,7 @@ __device__ __forceinline__ float2 running_sums(float2 x) {
 }
 
 constexpr int kPrepareThreads = 128;
+constexpr int kPrepareHeads = 4;   // heads per CTA
 constexpr int kARow = kChunk + 4;
 struct PrepareSmem {
     union {
@@ -560,17 +592,16 @@ __device__ __forceinline__ void pair_sync() {
     else asm volatile("bar.sync 2, 64;" ::: "memory");
 }
 
-// The columns of (I + A)^-1 from BASE on, one per lane, by forward substitution; those before it are zero in rows
-// below BASE.
-template <int BASE>
-__device__ __forceinline__ void invert_columns(float* a) {
+// (I + A)^-1 of the 32 x 32 block at `a`, in its place: a column per lane, by forward substitution.
+__device__ __forceinline__ void invert_block(float* a) {
+    constexpr int N = kChunk / 2;
     const int lane = threadIdx.x & 31;
-    float x[kChunk];
+    float x[N];
 #pragma unroll
-    for (int i = BASE; i < kChunk; ++i) {
-        float acc[4] = {i == BASE + lane ? 1.f : 0.f, 0.f, 0.f, 0.f};
+    for (int i = 0; i < N; ++i) {
+        float acc[4] = {i == lane ? 1.f : 0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int s = BASE; s < i; s += 4) {
+        for (int s = 0; s < i; s += 4) {
             const float4 r = load4(a + i * kARow + s);
             acc[0] = fmaf(-r.x, x[s], acc[0]);
             if (s + 1 < i) acc[1] = fmaf(-r.y, x[s + 1], acc[1]);
@@ -579,16 +610,68 @@ __device__ __forceinline__ void invert_columns(float* a) {
         }
         x[i] = (acc[0] + acc[1]) + (acc[2] + acc[3]);
     }
-    pair_sync();   // both warps have read A
+    __syncwarp();
 #pragma unroll
-    for (int i = 0; i < kChunk; ++i) a[i * kARow + BASE + lane] = i < BASE ? 0.f : x[i < BASE ? BASE : i];
+    for (int i = 0; i < N; ++i) a[i * kARow + lane] = x[i];
+}
+
+// 16 rows of a product of 32 x 32 blocks in shared memory, every factor as the sum of two bf16 numbers.
+__device__ __forceinline__ void multiply_block(float (&acc)[4][4], const float* left, const float* right) {
+    const int lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+#pragma unroll
+    for (int kt = 0; kt < 2; ++kt) {
+        uint32_t ah[4], al[4];
+#pragma unroll
+        for (int p = 0; p < 4; ++p) {
+            const float2 v = *reinterpret_cast<const float2*>(left + (g + (p & 1) * 8) * kARow + kt * 16 + (p >> 1) * 8 + 2 * tq);
+            split2(v.x, v.y, ah[p], al[p]);
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            uint32_t bh[2], bl[2];
+#pragma unroll
+            for (int p = 0; p < 2; ++p) {
+                const float* r = right + (kt * 16 + p * 8 + 2 * tq) * kARow + j * 8 + g;
+                split2(r[0], r[kARow], bh[p], bl[p]);
+            }
+            mma_bf16_16816(acc[j], ah, bh[0], bh[1]);
+            mma_bf16_16816(acc[j], al, bh[0], bh[1]);
+            mma_bf16_16816(acc[j], ah, bl[0], bl[1]);
+        }
+    }
+}
+
+// (I + A)^-1 of a head's chunk, in the place of A, by the pair of warps that works on it: the diagonal blocks by
+// substitution, the block below them as -inverse(lower) A inverse(upper).
+__device__ __forceinline__ void invert_chunk(float* a, int half) {
+    constexpr int N = kChunk / 2;
+    const int lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
+    float *upper = a, *lower = a + N * kARow + N, *below = a + N * kARow, *spare = a + N;
+    auto put = [&](float* to, const float (&acc)[4][4], float sign) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int p = 0; p < 2; ++p)
+                *reinterpret_cast<float2*>(to + (half * 16 + g + p * 8) * kARow + j * 8 + 2 * tq) =
+                    make_float2(sign * acc[j][2 * p], sign * acc[j][2 * p + 1]);
+    };
+    invert_block(half ? lower : upper);
+    pair_sync();
+    float acc[4][4];
+    multiply_block(acc, below + half * 16 * kARow, upper);
+    put(spare, acc, 1.f);
+    pair_sync();
+    multiply_block(acc, lower + half * 16 * kARow, spare);
+    put(below, acc, -1.f);
     pair_sync();
 }
 
-// Grid: chunks of the longest request, k / q heads, requests.
+// Grid: chunks of the longest request, k / q heads times the parts that their heads are dealt with in, requests.
 template <int RULE>
-__global__ void __launch_bounds__(kPrepareThreads)
-prepare_kernel(const Recurrence a) {
+__global__ void __launch_bounds__(kPrepareThreads, 4)
+prepare_kernel(const Recurrence a, int parts) {
     extern __shared__ __align__(16) uint8_t smem_raw[];
     PrepareSmem& S = *reinterpret_cast<PrepareSmem*>(smem_raw);
     constexpr int ROW = 64 + kPad, kMatrices = RULE == kDelta ? 2 : 1;
@@ -596,7 +679,7 @@ prepare_kernel(const Recurrence a) {
     const int g = lane >> 2, tq = lane & 3, mi = lane >> 3, r8 = lane & 7;
     pdl_launch_dependents();
     pdl_wait_prior();
-    const int b = blockIdx.z, kvh = blockIdx.y, begin = a.qo_indptr[b], ext = a.qo_indptr[b + 1] - begin;
+    const int b = blockIdx.z, kvh = blockIdx.y / parts, begin = a.qo_indptr[b], ext = a.qo_indptr[b + 1] - begin;
     const int s0 = blockIdx.x * kChunk;
     if (s0 >= ext) return;
     const int n = min(kChunk, ext - s0);
@@ -644,11 +727,12 @@ prepare_kernel(const Recurrence a) {
         }
     }
     // ---- per head: P and, two heads at a time, the inverse ----
-    const int group = a.heads / a.kv_heads;
+    const int group = a.heads / a.kv_heads, part = blockIdx.y % parts;
+    const int from = part * kPrepareHeads, to = min(group, from + kPrepareHeads);
     uint4* chunks = static_cast<uint4*>(a.chunks) + chunk_number(begin, b, blockIdx.x) * a.heads * kMatrices * kMatrixVecs;
-    for (int h0 = 0; h0 < group; h0 += 2) {
+    for (int h0 = from; h0 < to; h0 += 2) {
         __syncthreads();
-        if ((warp & 1) == 0 && h0 + (warp >> 1) < group) {
+        if ((warp & 1) == 0 && h0 + (warp >> 1) < to) {
             const int h = kvh * group + h0 + (warp >> 1);
             const float2* steps = reinterpret_cast<const float2*>(a.steps) + first * a.heads + h;
             const float2 none = make_float2(0.f, 0.f);
@@ -660,7 +744,7 @@ prepare_kernel(const Recurrence a) {
         __syncthreads();
 #pragma unroll
         for (int hp = 0; hp < 2; ++hp) {
-            if (h0 + hp >= group) continue;
+            if (h0 + hp >= to) continue;
             uint4* out = chunks + (static_cast<int64_t>(kvh * group + h0 + hp) * kMatrices) * kMatrixVecs + lane;
             const int t0 = warp * 16 + g;
             const float sum_t[2] = {S.sum[hp][t0], S.sum[hp][t0 + 8]};
@@ -705,10 +789,9 @@ prepare_kernel(const Recurrence a) {
         if (RULE != kDelta) continue;
         __syncthreads();
         const int hp = warp >> 1;
-        if (h0 + hp >= group) continue;   // (both warps of the pair)
+        if (h0 + hp >= to) continue;   // (both warps of the pair)
         float* m = S.a[hp];
-        if ((warp & 1) == 0) invert_columns<0>(m);
-        else invert_columns<32>(m);
+        invert_chunk(m, warp & 1);
         uint4* out = chunks + (static_cast<int64_t>(kvh * group + h0 + hp) * kMatrices + 1) * kMatrixVecs + lane;
         // tiles of the pair's warps: rows 0 and 3, rows 1 and 2
 #pragma unroll
@@ -730,35 +813,43 @@ prepare_kernel(const Recurrence a) {
     }
 }
 
-// SLICE value columns per CTA, 16 per warp.
-template <int DK, int RULE, int SLICE>
+// An 8 x 8 matrix of bf16 pairs, one per lane, transposed across the warp.
+__device__ __forceinline__ uint32_t transpose_8x8(uint32_t x) {
+    uint32_t y;
+    asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(y) : "r"(x));
+    return y;
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int LEFT>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(LEFT) : "memory"); }
+
+constexpr int kWalkThreads = 128;
+constexpr int kSlice = 64;            // value columns per CTA, 16 per warp
+
+template <int DK, int RULE>
 struct WalkSmem {
-    static constexpr int kRow = DK + kPad, kVRow = SLICE + kPad;
+    static constexpr int kRow = DK + kPad, kVRow = kSlice + kPad;
     __nv_bfloat16 k[2][kChunk * kRow], q[2][kChunk * kRow], v[2][kChunk * kVRow];   // this chunk's and the next one's
-    __nv_bfloat16 sh[DK * kVRow], sl[DK * kVRow];                                   // the state
-    __nv_bfloat16 rh[RULE == kDelta ? kChunk * kVRow : 8], rl[RULE == kDelta ? kChunk * kVRow : 8];   // beta (V - G K S)
-    __nv_bfloat16 uh[RULE == kDelta ? kChunk * kVRow : 8], ul[RULE == kDelta ? kChunk * kVRow : 8];   // U
-    __nv_bfloat16 wh[kChunk * kVRow], wl[kChunk * kVRow];                           // U as it enters the state
+    uint4 m[(RULE == kDelta ? 2 : 1) * kMatrixVecs];   // this chunk's P and inverse
     float out[2][kChunk];      // G_t times q's factor
     float beta[2][kChunk], read[2][kChunk];   // beta_t; beta_t G_t times k's factor
     float write[2][kChunk];    // exp(B_n - B_t) times k's factor (or times dt)
     float keep[2];             // G_n
 };
 
-// Grid: slices of the value columns, heads, requests.
-template <int DK, int RULE, int SLICE>
-__global__ void __launch_bounds__(SLICE * 8, 512 / (SLICE * 8))
+// Grid: slices of 64 value columns, heads, requests.  All products are formed transposed, 16 value columns by tokens (or
+// by state rows) per warp, so that what one leaves in a warp's accumulators is the next one's left operand where it
+// is: nothing but the chunk's k, q, v and matrices goes through shared memory, and warps do not wait for one another.
+template <int DK, int RULE>
+__global__ void __launch_bounds__(kWalkThreads, 2)
 chunk_kernel(const Recurrence a) {
-    using Smem = WalkSmem<DK, RULE, SLICE>;
-    constexpr int kWalkThreads = SLICE * 8;             // four tiles of tokens times 16 columns per warp
+    using Smem = WalkSmem<DK, RULE>;
     constexpr int ROW = Smem::kRow, VROW = Smem::kVRow, kMatrices = RULE == kDelta ? 2 : 1;
-    constexpr int kColSplit = SLICE * 4 / DK;            // warps that share 16 state rows
-    constexpr int kStateTiles = SLICE / 8 / kColSplit;   // 8-column tiles of state per warp
     extern __shared__ __align__(16) uint8_t smem_raw[];
     Smem& S = *reinterpret_cast<Smem*>(smem_raw);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, tq = lane & 3, mi = lane >> 3, r8 = lane & 7;
-    const int h = blockIdx.y, req = blockIdx.z, v0 = blockIdx.x * SLICE;
+    const int h = blockIdx.y, req = blockIdx.z, v0 = blockIdx.x * kSlice, col0 = warp * 16;
     const int vp = a.padded_value_dim, kvh = h / (a.heads / a.kv_heads);
     pdl_launch_dependents();
     pdl_wait_prior();
@@ -777,8 +868,8 @@ chunk_kernel(const Recurrence a) {
             cp_async16(smem_u32(&S.k[buf][t * ROW + c]), row, t < n);
             cp_async16(smem_u32(&S.q[buf][t * ROW + c]), row + to_q, t < n);
         }
-        for (int i = threadIdx.x; i < kChunk * (SLICE / 8); i += kWalkThreads) {
-            const int t = i / (SLICE / 8), c = (i % (SLICE / 8)) * 8;
+        for (int i = threadIdx.x; i < kChunk * (kSlice / 8); i += kWalkThreads) {
+            const int t = i / (kSlice / 8), c = (i % (kSlice / 8)) * 8;
             cp_async16(smem_u32(&S.v[buf][t * VROW + c]), mixed + static_cast<int64_t>(t < n ? s0 + t : s0) * nc + at_v + c, t < n);
         }
     };
@@ -817,228 +908,213 @@ chunk_kernel(const Recurrence a) {
         if (lane == 0) S.keep[buf] = ex2(last);
     };
     load_chunk(0, 0);
+    cp_async_commit();
 
-    // This warp's part of the state: 16 rows from row0, kStateTiles tiles of 8 columns from col0, in the layout of an
-    // MMA accumulator.
-    const int row0 = warp / kColSplit * 16, col0 = warp % kColSplit * (SLICE / kColSplit);
-    float* state = a.state + (static_cast<int64_t>(a.table_idx[req]) * a.heads + h) * DK * vp + v0;
-    float st[kStateTiles][4];
+    // This warp's 16 columns of the state, transposed: tile j holds state rows 8 j + 2 tq, + 1 of columns g and g + 8.
+    float* state = a.state + (static_cast<int64_t>(a.table_idx[req]) * a.heads + h) * DK * vp + v0 + col0 + g;
+    float st[DK / 8][4];
     const bool fresh = a.cached[req] == 0;
-    auto put_state = [&]() {
 #pragma unroll
-        for (int j = 0; j < kStateTiles; ++j)
+    for (int j = 0; j < DK / 8; ++j)
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                uint32_t hi, lo;
-                split2(st[j][2 * half], st[j][2 * half + 1], hi, lo);
-                const int at = (row0 + g + half * 8) * VROW + col0 + j * 8 + 2 * tq;
-                *reinterpret_cast<uint32_t*>(&S.sh[at]) = hi;
-                *reinterpret_cast<uint32_t*>(&S.sl[at]) = lo;
-            }
-    };
-#pragma unroll
-    for (int j = 0; j < kStateTiles; ++j)
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-            const float2 x = fresh ? make_float2(0.f, 0.f)
-                                   : *reinterpret_cast<const float2*>(state + static_cast<int64_t>(row0 + g + half * 8) * vp + col0 +
-                                                                      j * 8 + 2 * tq);
-            st[j][2 * half] = x.x;
-            st[j][2 * half + 1] = x.y;
-        }
-    put_state();
+        for (int e = 0; e < 4; ++e) st[j][e] = fresh ? 0.f : state[static_cast<int64_t>(8 * j + 2 * tq + (e & 1)) * vp + (e >> 1) * 8];
     if (warp == 0) {
         fetch_factors(0);
         put_factors(0);
     }
-    // 16 tokens x 16 columns of the products per warp; the warps of a scheduler share out the triangle evenly
-    const int mt = (warp + (warp >> 2)) & 3, oc0 = (warp >> 2) * 16;
     const float skip = RULE == kStateSpace ? a.skip[h] : 0.f;
-    const uint4* chunks = static_cast<const uint4*>(a.chunks) +
-                          (chunk_number(begin, req, 0) * a.heads + h) * kMatrices * kMatrixVecs + mt * (mt + 1) / 2 * 64 + lane;
+    const uint4* chunks = static_cast<const uint4*>(a.chunks) + (chunk_number(begin, req, 0) * a.heads + h) * kMatrices * kMatrixVecs;
     const int64_t chunk_vecs = static_cast<int64_t>(a.heads) * kMatrices * kMatrixVecs;
 
-    // acc += M X for this warp's rows: M's tiles from memory, X [kChunk][kSlice] in shared memory as one or two parts
-    auto load_matrix = [&](const uint4* m, uint4 (&hi)[4], uint4 (&lo)[4]) {
-#pragma unroll
-        for (int kt = 0; kt < 4; ++kt)
-            if (kt <= mt) {
-                hi[kt] = __ldg(m + kt * 64);
-                lo[kt] = __ldg(m + kt * 64 + 32);
-            }
-    };
-    auto multiply = [&](float (&acc)[2][4], const uint4 (&hi)[4], const uint4 (&lo)[4], const __nv_bfloat16* xh, const __nv_bfloat16* xl) {
+    // acc (16 columns by tokens) += X M^T for a lower triangular M, X as left operands of 16 tokens each
+    auto multiply = [&](float (&acc)[8][4], const uint32_t (&xh)[4][4], const uint32_t (*xl)[4], const uint4* m, int n) {
+        // (neighbouring products go to different accumulators)
 #pragma unroll
         for (int kt = 0; kt < 4; ++kt) {
-            if (kt > mt) continue;
-            const uint32_t ah[4] = {hi[kt].x, hi[kt].y, hi[kt].z, hi[kt].w}, al[4] = {lo[kt].x, lo[kt].y, lo[kt].z, lo[kt].w};
-            const int off = (kt * 16 + (mi & 1) * 8 + r8) * VROW + oc0 + (mi >> 1) * 8;
-            uint32_t b0, b1, b2, b3;
-            ldmatrix_x4_trans(smem_u32(xh + off), b0, b1, b2, b3);
-            mma_bf16_16816(acc[0], ah, b0, b1);
-            mma_bf16_16816(acc[1], ah, b2, b3);
-            mma_bf16_16816(acc[0], al, b0, b1);
-            mma_bf16_16816(acc[1], al, b2, b3);
+            if (kt * 16 >= n) continue;
+            uint4 b[4];
+#pragma unroll
+            for (int mt = kt; mt < 4; ++mt) b[mt] = m[(mt * (mt + 1) / 2 + kt) * 64 + lane];
+#pragma unroll
+            for (int mt = kt; mt < 4; ++mt) {
+                mma_bf16_16816(acc[2 * mt], xh[kt], b[mt].x, b[mt].z);
+                mma_bf16_16816(acc[2 * mt + 1], xh[kt], b[mt].y, b[mt].w);
+            }
             if (xl != nullptr) {
-                ldmatrix_x4_trans(smem_u32(xl + off), b0, b1, b2, b3);
-                mma_bf16_16816(acc[0], ah, b0, b1);
-                mma_bf16_16816(acc[1], ah, b2, b3);
+#pragma unroll
+                for (int mt = kt; mt < 4; ++mt) {
+                    mma_bf16_16816(acc[2 * mt], xl[kt], b[mt].x, b[mt].z);
+                    mma_bf16_16816(acc[2 * mt + 1], xl[kt], b[mt].y, b[mt].w);
+                }
+            }
+#pragma unroll
+            for (int mt = kt; mt < 4; ++mt) b[mt] = m[(mt * (mt + 1) / 2 + kt) * 64 + 32 + lane];
+#pragma unroll
+            for (int mt = kt; mt < 4; ++mt) {
+                mma_bf16_16816(acc[2 * mt], xh[kt], b[mt].x, b[mt].z);
+                mma_bf16_16816(acc[2 * mt + 1], xh[kt], b[mt].y, b[mt].w);
             }
         }
+    };
+    // accumulators of 16 tokens as a left operand in two parts
+    auto split_tile = [&](const float (&acc)[8][4], int kt, uint32_t (&hi)[4], uint32_t (&lo)[4]) {
+#pragma unroll
+        for (int p = 0; p < 4; ++p) split2(acc[2 * kt + (p >> 1)][(p & 1) * 2], acc[2 * kt + (p >> 1)][(p & 1) * 2 + 1], hi[p], lo[p]);
     };
 
     int buf = 0;
     for (int s0 = 0; s0 < ext; s0 += kChunk, buf ^= 1, chunks += chunk_vecs) {
         const int n = min(kChunk, ext - s0);
-        const bool more = s0 + kChunk < ext, mine = mt * 16 < n;
-        cp_async_wait_all();
-        __syncthreads();   // this chunk, its factors and the state are in place; nobody needs the last chunk's
+        const bool more = s0 + kChunk < ext;
+        cp_async_wait<0>();
+        __syncthreads();   // this chunk and its factors are in place; nobody needs the last one's
+        for (int i = threadIdx.x; i < kMatrices * kMatrixVecs; i += kWalkThreads) cp_async16(smem_u32(&S.m[i]), chunks + i, true);
+        cp_async_commit();
         if (more) {
             load_chunk(s0 + kChunk, buf ^ 1);
             if (warp == 0) fetch_factors(s0 + kChunk);
         }
-        uint4 mh[4], ml[4];   // the inverse, then P
-        if (mine) load_matrix(RULE == kDelta ? chunks + kMatrixVecs : chunks, mh, ml);
+        cp_async_commit();
         const __nv_bfloat16 *K = S.k[buf], *Q = S.q[buf], *V = S.v[buf];
-        const int ta = mt * 16 + g, tb = ta + 8;   // this thread's rows of the products
-        // ---- Q S and K S ----
-        float o[2][4] = {}, u[2][4] = {};
-        if (mine) {
+        // ---- S^T Q^T and S^T K^T ----
+        float o[8][4] = {}, u[8][4] = {};
+        constexpr int kPairs = RULE == kDelta ? 2 : 4;   // 16-token operands at a time
 #pragma unroll
-            for (int ks = 0; ks < DK / 16; ++ks) {
-                uint32_t aq[4], ak[4], b0, b1, b2, b3;
-                const int aoff = (mt * 16 + (mi & 1) * 8 + r8) * ROW + ks * 16 + (mi >> 1) * 8;
-                ldmatrix_x4(smem_u32(&Q[aoff]), aq[0], aq[1], aq[2], aq[3]);
-                if (RULE == kDelta) ldmatrix_x4(smem_u32(&K[aoff]), ak[0], ak[1], ak[2], ak[3]);
-                const int soff = (ks * 16 + (mi & 1) * 8 + r8) * VROW + oc0 + (mi >> 1) * 8;
+        for (int ks = 0; ks < DK / 16; ++ks) {
+            uint32_t ah[4], al[4];
 #pragma unroll
-                for (int part = 0; part < 2; ++part) {
-                    ldmatrix_x4_trans(smem_u32(part == 0 ? &S.sh[soff] : &S.sl[soff]), b0, b1, b2, b3);
-                    mma_bf16_16816(o[0], aq, b0, b1);
-                    mma_bf16_16816(o[1], aq, b2, b3);
-                    if (RULE == kDelta) {
-                        mma_bf16_16816(u[0], ak, b0, b1);
-                        mma_bf16_16816(u[1], ak, b2, b3);
-                    }
+            for (int p = 0; p < 4; ++p) split2(st[2 * ks + (p >> 1)][(p & 1) * 2], st[2 * ks + (p >> 1)][(p & 1) * 2 + 1], ah[p], al[p]);
+#pragma unroll
+            for (int tp0 = 0; tp0 < 4; tp0 += kPairs) {
+                if (tp0 * 16 >= n) continue;
+                uint32_t bq[kPairs][4], bk[kPairs][4];
+#pragma unroll
+                for (int e = 0; e < kPairs; ++e) {
+                    const int off = ((tp0 + e) * 16 + (mi >> 1) * 8 + r8) * ROW + ks * 16 + (mi & 1) * 8;
+                    ldmatrix_x4(smem_u32(&Q[off]), bq[e][0], bq[e][1], bq[e][2], bq[e][3]);
+                    if (RULE == kDelta) ldmatrix_x4(smem_u32(&K[off]), bk[e][0], bk[e][1], bk[e][2], bk[e][3]);
                 }
+#pragma unroll
+                for (int part = 0; part < 2; ++part)
+#pragma unroll
+                    for (int e = 0; e < kPairs; ++e) {
+                        const uint32_t(&x)[4] = part == 0 ? ah : al;
+                        mma_bf16_16816(o[2 * (tp0 + e)], x, bq[e][0], bq[e][1]);
+                        mma_bf16_16816(o[2 * (tp0 + e) + 1], x, bq[e][2], bq[e][3]);
+                        if (RULE == kDelta) {
+                            mma_bf16_16816(u[2 * (tp0 + e)], x, bk[e][0], bk[e][1]);
+                            mma_bf16_16816(u[2 * (tp0 + e) + 1], x, bk[e][2], bk[e][3]);
+                        }
+                    }
             }
         }
+        // V^T of 16 tokens: token pairs 2 tq of columns g and g + 8, then eight tokens on
+        auto values_of = [&](int tp, uint32_t (&x)[4]) {
+            ldmatrix_x4_trans(smem_u32(&V[(tp * 16 + (mi >> 1) * 8 + r8) * VROW + col0 + (mi & 1) * 8]), x[0], x[1], x[2], x[3]);
+        };
+        uint32_t xh[4][4], xl[RULE == kDelta ? 4 : 1][4];
         if (RULE == kDelta) {
             // ---- U = (I + A)^-1 (beta V - beta G K S) ----
-            if (mine) {
-                const float ba = S.beta[buf][ta], bb = S.beta[buf][tb], ra = S.read[buf][ta], rb = S.read[buf][tb];
 #pragma unroll
-                for (int j = 0; j < 2; ++j)
+            for (int tp = 0; tp < 4; ++tp) {
+                uint32_t x[4];
+                values_of(tp, x);
 #pragma unroll
-                    for (int half = 0; half < 2; ++half) {
-                        const int at = (half ? tb : ta) * VROW + oc0 + j * 8 + 2 * tq;
-                        const uint32_t v = *reinterpret_cast<const uint32_t*>(&V[at]);
-                        const float beta = half ? bb : ba, r = half ? rb : ra;
-                        uint32_t hi, lo;
-                        split2(beta * bf16_lo(v) - r * u[j][2 * half], beta * bf16_hi(v) - r * u[j][2 * half + 1], hi, lo);
-                        *reinterpret_cast<uint32_t*>(&S.rh[at]) = hi;
-                        *reinterpret_cast<uint32_t*>(&S.rl[at]) = lo;
-                        u[j][2 * half] = u[j][2 * half + 1] = 0.f;
-                    }
-            }
-            __syncthreads();
-            if (mine) {
-                multiply(u, mh, ml, S.rh, S.rl);
-                load_matrix(chunks, mh, ml);
-            }
-        }
-        if (mine) {
-            const float wa = S.write[buf][ta], wb = S.write[buf][tb];
-#pragma unroll
-            for (int j = 0; j < 2; ++j)
-#pragma unroll
-                for (int half = 0; half < 2; ++half) {
-                    const int at = (half ? tb : ta) * VROW + oc0 + j * 8 + 2 * tq;
-                    const float w = half ? wb : wa;
-                    float x = u[j][2 * half], y = u[j][2 * half + 1];
-                    uint32_t hi, lo;
-                    if (RULE == kDelta) {
-                        split2(x, y, hi, lo);
-                        *reinterpret_cast<uint32_t*>(&S.uh[at]) = hi;
-                        *reinterpret_cast<uint32_t*>(&S.ul[at]) = lo;
-                    } else {
-                        const uint32_t v = *reinterpret_cast<const uint32_t*>(&V[at]);
-                        x = bf16_lo(v);
-                        y = bf16_hi(v);
-                    }
-                    split2(x * w, y * w, hi, lo);
-                    *reinterpret_cast<uint32_t*>(&S.wh[at]) = hi;
-                    *reinterpret_cast<uint32_t*>(&S.wl[at]) = lo;
+                for (int side = 0; side < 2; ++side) {
+                    const int t = tp * 16 + side * 8 + 2 * tq;
+                    const float2 be = *reinterpret_cast<const float2*>(&S.beta[buf][t]), rd = *reinterpret_cast<const float2*>(&S.read[buf][t]);
+                    float* c = u[2 * tp + side];
+                    c[0] = be.x * bf16_lo(x[2 * side]) - rd.x * c[0];
+                    c[1] = be.y * bf16_hi(x[2 * side]) - rd.y * c[1];
+                    c[2] = be.x * bf16_lo(x[2 * side + 1]) - rd.x * c[2];
+                    c[3] = be.y * bf16_hi(x[2 * side + 1]) - rd.y * c[3];
                 }
+                split_tile(u, tp, xh[tp], xl[tp]);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) u[2 * tp + (e >> 2)][e & 3] = 0.f;
+            }
+        } else {
+#pragma unroll
+            for (int tp = 0; tp < 4; ++tp) values_of(tp, xh[tp]);
         }
-        __syncthreads();
+        cp_async_wait<1>();
+        __syncthreads();   // the matrices
+        if (RULE == kDelta) {
+            multiply(u, xh, xl, S.m + kMatrixVecs, n);
+#pragma unroll
+            for (int tp = 0; tp < 4; ++tp) split_tile(u, tp, xh[tp], xl[tp]);
+        }
         // ---- O = G Q S + P U (+ skip V) ----
-        if (mine) {
-            const float ga = S.out[buf][ta], gb = S.out[buf][tb];
 #pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                o[j][0] *= ga;
-                o[j][1] *= ga;
-                o[j][2] *= gb;
-                o[j][3] *= gb;
+        for (int j = 0; j < 8; ++j) {
+            const float2 f = *reinterpret_cast<const float2*>(&S.out[buf][8 * j + 2 * tq]);
+            o[j][0] *= f.x;
+            o[j][1] *= f.y;
+            o[j][2] *= f.x;
+            o[j][3] *= f.y;
+            if (RULE == kStateSpace) {
+                const uint32_t *x = &xh[j >> 1][(j & 1) * 2];
+                o[j][0] = fmaf(skip, bf16_lo(x[0]), o[j][0]);
+                o[j][1] = fmaf(skip, bf16_hi(x[0]), o[j][1]);
+                o[j][2] = fmaf(skip, bf16_lo(x[1]), o[j][2]);
+                o[j][3] = fmaf(skip, bf16_hi(x[1]), o[j][3]);
             }
-            if (RULE == kDelta) multiply(o, mh, ml, S.uh, S.ul);
-            else multiply(o, mh, ml, V, nullptr);
-            __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + static_cast<int64_t>(begin + s0) * a.out_ld + at_v + oc0 + 2 * tq;
+        }
+        multiply(o, xh, RULE == kDelta ? xl : nullptr, S.m, n);
+        {
+            __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + static_cast<int64_t>(begin + s0 + g) * a.out_ld + at_v + col0 + 2 * tq;
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                const int t = half ? tb : ta;
-                if (t >= n) continue;
-#pragma unroll
-                for (int j = 0; j < 2; ++j) {
-                    float x = o[j][2 * half], y = o[j][2 * half + 1];
-                    if (RULE == kStateSpace) {
-                        const uint32_t v = *reinterpret_cast<const uint32_t*>(&V[t * VROW + oc0 + j * 8 + 2 * tq]);
-                        x = fmaf(skip, bf16_lo(v), x);
-                        y = fmaf(skip, bf16_hi(v), y);
-                    }
-                    *reinterpret_cast<uint32_t*>(out + t * a.out_ld + j * 8) = pack_bf16(x, y);
-                }
+            for (int j = 0; j < 8; ++j) {
+                const uint32_t left = transpose_8x8(pack_bf16(o[j][0], o[j][1])), right = transpose_8x8(pack_bf16(o[j][2], o[j][3]));
+                if (8 * j + g >= n) continue;
+                *reinterpret_cast<uint32_t*>(out + static_cast<int64_t>(8 * j) * a.out_ld) = left;
+                *reinterpret_cast<uint32_t*>(out + static_cast<int64_t>(8 * j) * a.out_ld + 8) = right;
             }
         }
         // ---- the state after the chunk ----
         const float keep = S.keep[buf];
 #pragma unroll
-        for (int j = 0; j < kStateTiles; ++j)
+        for (int j = 0; j < DK / 8; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) st[j][e] *= keep;
 #pragma unroll
-        for (int kt = 0; kt < kChunk / 16; ++kt) {
+        for (int kt = 0; kt < 4; ++kt) {
             if (kt * 16 >= n) continue;
-            uint32_t ak[4];
-            ldmatrix_x4_trans(smem_u32(&K[(kt * 16 + (mi >> 1) * 8 + r8) * ROW + row0 + (mi & 1) * 8]), ak[0], ak[1], ak[2], ak[3]);
+            uint32_t wh[4], wl[4];
 #pragma unroll
-            for (int np = 0; np < kStateTiles / 2; ++np) {
-                const int off = (kt * 16 + (mi & 1) * 8 + r8) * VROW + col0 + np * 16 + (mi >> 1) * 8;
-                uint32_t b0, b1, b2, b3;
-                ldmatrix_x4_trans(smem_u32(&S.wh[off]), b0, b1, b2, b3);
-                mma_bf16_16816(st[2 * np], ak, b0, b1);
-                mma_bf16_16816(st[2 * np + 1], ak, b2, b3);
-                ldmatrix_x4_trans(smem_u32(&S.wl[off]), b0, b1, b2, b3);
-                mma_bf16_16816(st[2 * np], ak, b0, b1);
-                mma_bf16_16816(st[2 * np + 1], ak, b2, b3);
+            for (int p = 0; p < 4; ++p) {
+                const float2 w = *reinterpret_cast<const float2*>(&S.write[buf][kt * 16 + (p >> 1) * 8 + 2 * tq]);
+                const float* c = &u[2 * kt + (p >> 1)][(p & 1) * 2];
+                const float x = RULE == kDelta ? c[0] : bf16_lo(xh[kt][p]), y = RULE == kDelta ? c[1] : bf16_hi(xh[kt][p]);
+                split2(x * w.x, y * w.y, wh[p], wl[p]);
+            }
+#pragma unroll
+            for (int dp0 = 0; dp0 < DK / 16; dp0 += 4) {
+                uint32_t bk[4][4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    ldmatrix_x4_trans(smem_u32(&K[(kt * 16 + (mi & 1) * 8 + r8) * ROW + (dp0 + e) * 16 + (mi >> 1) * 8]), bk[e][0], bk[e][1],
+                                      bk[e][2], bk[e][3]);
+#pragma unroll
+                for (int part = 0; part < 2; ++part)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const uint32_t(&x)[4] = part == 0 ? wh : wl;
+                        mma_bf16_16816(st[2 * (dp0 + e)], x, bk[e][0], bk[e][1]);
+                        mma_bf16_16816(st[2 * (dp0 + e) + 1], x, bk[e][2], bk[e][3]);
+                    }
             }
         }
-        if (more) {
-            put_state();
-            if (warp == 0) put_factors(buf ^ 1);
-        }
+        if (more && warp == 0) put_factors(buf ^ 1);
     }
 #pragma unroll
-    for (int j = 0; j < kStateTiles; ++j)
+    for (int j = 0; j < DK / 8; ++j)
 #pragma unroll
-        for (int half = 0; half < 2; ++half)
-            *reinterpret_cast<float2*>(state + static_cast<int64_t>(row0 + g + half * 8) * vp + col0 + j * 8 + 2 * tq) =
-                make_float2(st[j][2 * half], st[j][2 * half + 1]);
+        for (int e = 0; e < 4; ++e) state[static_cast<int64_t>(8 * j + 2 * tq + (e & 1)) * vp + (e >> 1) * 8] = st[j][e];
 }
 
 bool chunked_supported(const Recurrence& a, int dtype) {
-    return dtype == B200_DTYPE_BF16 && !a.plain && (a.padded_dim == 64 || a.padded_dim == 128) && a.padded_value_dim % 64 == 0;
+    return dtype == B200_DTYPE_BF16 && !a.plain && (a.padded_dim == 64 || a.padded_dim == 128) && a.padded_value_dim % kSlice == 0;
 }
 
 int max_smem(const void* kernel, size_t bytes) {
@@ -1061,15 +1137,14 @@ int launch_chunked(const Recurrence& a, cudaStream_t stream) {
     auto prepare = prepare_kernel<RULE>;
     int err = max_smem(reinterpret_cast<const void*>(prepare), sizeof(PrepareSmem));
     if (err != B200_OK) return err;
-    B200_CHECK_CUDA(launch_kernel(prepare, dim3(div_ceil(a.max_extend, kChunk), a.kv_heads, a.batch), dim3(kPrepareThreads),
-                                  sizeof(PrepareSmem), stream, dim3(1, 1, 1), a));
-    // the state space has room for two CTAs per SM
-    constexpr int SLICE = RULE == kDelta ? 64 : 32;
-    auto kernel = a.padded_dim == 64 ? chunk_kernel<64, RULE, SLICE> : chunk_kernel<128, RULE, SLICE>;
-    const size_t smem = a.padded_dim == 64 ? sizeof(WalkSmem<64, RULE, SLICE>) : sizeof(WalkSmem<128, RULE, SLICE>);
+    const int parts = div_ceil(a.heads / a.kv_heads, kPrepareHeads);
+    B200_CHECK_CUDA(launch_kernel(prepare, dim3(div_ceil(a.max_extend, kChunk), a.kv_heads * parts, a.batch), dim3(kPrepareThreads),
+                                  sizeof(PrepareSmem), stream, dim3(1, 1, 1), a, parts));
+    auto kernel = a.padded_dim == 64 ? chunk_kernel<64, RULE> : chunk_kernel<128, RULE>;
+    const size_t smem = a.padded_dim == 64 ? sizeof(WalkSmem<64, RULE>) : sizeof(WalkSmem<128, RULE>);
     err = max_smem(reinterpret_cast<const void*>(kernel), smem);
     if (err != B200_OK) return err;
-    B200_CHECK_CUDA(launch_kernel(kernel, dim3(a.padded_value_dim / SLICE, a.heads, a.batch), dim3(SLICE * 8), smem, stream,
+    B200_CHECK_CUDA(launch_kernel(kernel, dim3(a.padded_value_dim / kSlice, a.heads, a.batch), dim3(kWalkThreads), smem, stream,
                                   dim3(1, 1, 1), a));
     return B200_OK;
 }
