@@ -819,18 +819,20 @@ __device__ __forceinline__ uint32_t transpose_8x8(uint32_t x) {
     asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(y) : "r"(x));
     return y;
 }
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int LEFT>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(LEFT) : "memory"); }
 
-constexpr int kWalkThreads = 128;
-constexpr int kSlice = 64;            // value columns per CTA, 16 per warp
+constexpr int kWalkThreads = 256;
+constexpr int kSlice = 64;            // value columns per CTA, 16 per pair of warps
 
 template <int DK, int RULE>
 struct WalkSmem {
     static constexpr int kRow = DK + kPad, kVRow = kSlice + kPad;
     __nv_bfloat16 k[2][kChunk * kRow], q[2][kChunk * kRow], v[2][kChunk * kVRow];   // this chunk's and the next one's
-    uint4 m[(RULE == kDelta ? 2 : 1) * kMatrixVecs];   // this chunk's P and inverse
+    uint4 m[2][(RULE == kDelta ? 2 : 1) * kMatrixVecs];   // P and inverse
+    // what the warps of a pair hand to one another as left operands, per 16 tokens upper and lower parts:
+    // beta (V - G K S), U, U as it enters the state
+    uint4 hand[RULE == kDelta ? 3 : 1][kSlice / 16][RULE == kDelta ? 4 : 1][2][32];
+    // and what a warp's state rows add to the other one's tokens: [pair][warp][token tile][Q S, K S][8 tokens]
+    float4 sums[kSlice / 16][2][2][RULE == kDelta ? 2 : 1][2][32];
     float out[2][kChunk];      // G_t times q's factor
     float beta[2][kChunk], read[2][kChunk];   // beta_t; beta_t G_t times k's factor
     float write[2][kChunk];    // exp(B_n - B_t) times k's factor (or times dt)
@@ -838,10 +840,11 @@ struct WalkSmem {
 };
 
 // Grid: slices of 64 value columns, heads, requests.  All products are formed transposed, 16 value columns by tokens (or
-// by state rows) per warp, so that what one leaves in a warp's accumulators is the next one's left operand where it
-// is: nothing but the chunk's k, q, v and matrices goes through shared memory, and warps do not wait for one another.
+// by state rows), so that what one leaves in a warp's accumulators is the next one's left operand where it is.  Two
+// warps share 16 columns: each keeps half of the state rows and works out the results of half of the tokens (tiles 0
+// and 3, tiles 1 and 2).
 template <int DK, int RULE>
-__global__ void __launch_bounds__(kWalkThreads, 2)
+__global__ void __launch_bounds__(kWalkThreads, 1)
 chunk_kernel(const Recurrence a) {
     using Smem = WalkSmem<DK, RULE>;
     constexpr int ROW = Smem::kRow, VROW = Smem::kVRow, kMatrices = RULE == kDelta ? 2 : 1;
@@ -849,8 +852,10 @@ chunk_kernel(const Recurrence a) {
     Smem& S = *reinterpret_cast<Smem*>(smem_raw);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, tq = lane & 3, mi = lane >> 3, r8 = lane & 7;
-    const int h = blockIdx.y, req = blockIdx.z, v0 = blockIdx.x * kSlice, col0 = warp * 16;
+    const int h = blockIdx.y, req = blockIdx.z, v0 = blockIdx.x * kSlice, pair = warp >> 1, half = warp & 1, col0 = pair * 16;
     const int vp = a.padded_value_dim, kvh = h / (a.heads / a.kv_heads);
+    const int own[4] = {half, 3 - half, 1 - half, 2 + half};   // this warp's 16-token tiles, then the other one's
+    constexpr int kRows = DK / 2;                              // state rows per warp
     pdl_launch_dependents();
     pdl_wait_prior();
     const int begin = a.qo_indptr[req], ext = a.qo_indptr[req + 1] - begin;
@@ -907,15 +912,20 @@ chunk_kernel(const Recurrence a) {
         }
         if (lane == 0) S.keep[buf] = ex2(last);
     };
+    const uint4* chunks = static_cast<const uint4*>(a.chunks) + (chunk_number(begin, req, 0) * a.heads + h) * kMatrices * kMatrixVecs;
+    const int64_t chunk_vecs = static_cast<int64_t>(a.heads) * kMatrices * kMatrixVecs;
+    auto load_matrices = [&](const uint4* m, int buf) {
+        for (int i = threadIdx.x; i < kMatrices * kMatrixVecs; i += kWalkThreads) cp_async16(smem_u32(&S.m[buf][i]), m + i, true);
+    };
     load_chunk(0, 0);
-    cp_async_commit();
+    load_matrices(chunks, 0);
 
-    // This warp's 16 columns of the state, transposed: tile j holds state rows 8 j + 2 tq, + 1 of columns g and g + 8.
-    float* state = a.state + (static_cast<int64_t>(a.table_idx[req]) * a.heads + h) * DK * vp + v0 + col0 + g;
-    float st[DK / 8][4];
+    // This warp's part of the state, transposed: tile j holds rows 8 j + 2 tq, + 1 of its half, of columns g and g + 8.
+    float* state = a.state + ((static_cast<int64_t>(a.table_idx[req]) * a.heads + h) * DK + half * kRows) * vp + v0 + col0 + g;
+    float st[kRows / 8][4];
     const bool fresh = a.cached[req] == 0;
 #pragma unroll
-    for (int j = 0; j < DK / 8; ++j)
+    for (int j = 0; j < kRows / 8; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) st[j][e] = fresh ? 0.f : state[static_cast<int64_t>(8 * j + 2 * tq + (e & 1)) * vp + (e >> 1) * 8];
     if (warp == 0) {
@@ -923,192 +933,245 @@ chunk_kernel(const Recurrence a) {
         put_factors(0);
     }
     const float skip = RULE == kStateSpace ? a.skip[h] : 0.f;
-    const uint4* chunks = static_cast<const uint4*>(a.chunks) + (chunk_number(begin, req, 0) * a.heads + h) * kMatrices * kMatrixVecs;
-    const int64_t chunk_vecs = static_cast<int64_t>(a.heads) * kMatrices * kMatrixVecs;
 
-    // acc (16 columns by tokens) += X M^T for a lower triangular M, X as left operands of 16 tokens each
-    auto multiply = [&](float (&acc)[8][4], const uint32_t (&xh)[4][4], const uint32_t (*xl)[4], const uint4* m, int n) {
-        // (neighbouring products go to different accumulators)
+    // acc (16 columns by this warp's tokens) += X M^T for a lower triangular M, X as left operands of 16 tokens each
+    // (neighbouring products go to different accumulators)
+    auto multiply = [&](float (&acc)[2][2][4], const uint32_t (&xh)[4][4], const uint32_t (*xl)[4], const uint4* m) {
 #pragma unroll
         for (int kt = 0; kt < 4; ++kt) {
-            if (kt * 16 >= n) continue;
-            uint4 b[4];
+            uint4 hi[2], lo[2];
 #pragma unroll
-            for (int mt = kt; mt < 4; ++mt) b[mt] = m[(mt * (mt + 1) / 2 + kt) * 64 + lane];
-#pragma unroll
-            for (int mt = kt; mt < 4; ++mt) {
-                mma_bf16_16816(acc[2 * mt], xh[kt], b[mt].x, b[mt].z);
-                mma_bf16_16816(acc[2 * mt + 1], xh[kt], b[mt].y, b[mt].w);
-            }
-            if (xl != nullptr) {
-#pragma unroll
-                for (int mt = kt; mt < 4; ++mt) {
-                    mma_bf16_16816(acc[2 * mt], xl[kt], b[mt].x, b[mt].z);
-                    mma_bf16_16816(acc[2 * mt + 1], xl[kt], b[mt].y, b[mt].w);
-                }
-            }
-#pragma unroll
-            for (int mt = kt; mt < 4; ++mt) b[mt] = m[(mt * (mt + 1) / 2 + kt) * 64 + 32 + lane];
-#pragma unroll
-            for (int mt = kt; mt < 4; ++mt) {
-                mma_bf16_16816(acc[2 * mt], xh[kt], b[mt].x, b[mt].z);
-                mma_bf16_16816(acc[2 * mt + 1], xh[kt], b[mt].y, b[mt].w);
-            }
-        }
-    };
-    // accumulators of 16 tokens as a left operand in two parts
-    auto split_tile = [&](const float (&acc)[8][4], int kt, uint32_t (&hi)[4], uint32_t (&lo)[4]) {
-#pragma unroll
-        for (int p = 0; p < 4; ++p) split2(acc[2 * kt + (p >> 1)][(p & 1) * 2], acc[2 * kt + (p >> 1)][(p & 1) * 2 + 1], hi[p], lo[p]);
-    };
-
-    int buf = 0;
-    for (int s0 = 0; s0 < ext; s0 += kChunk, buf ^= 1, chunks += chunk_vecs) {
-        const int n = min(kChunk, ext - s0);
-        const bool more = s0 + kChunk < ext;
-        cp_async_wait<0>();
-        __syncthreads();   // this chunk and its factors are in place; nobody needs the last one's
-        for (int i = threadIdx.x; i < kMatrices * kMatrixVecs; i += kWalkThreads) cp_async16(smem_u32(&S.m[i]), chunks + i, true);
-        cp_async_commit();
-        if (more) {
-            load_chunk(s0 + kChunk, buf ^ 1);
-            if (warp == 0) fetch_factors(s0 + kChunk);
-        }
-        cp_async_commit();
-        const __nv_bfloat16 *K = S.k[buf], *Q = S.q[buf], *V = S.v[buf];
-        // ---- S^T Q^T and S^T K^T ----
-        float o[8][4] = {}, u[8][4] = {};
-        constexpr int kPairs = RULE == kDelta ? 2 : 4;   // 16-token operands at a time
-#pragma unroll
-        for (int ks = 0; ks < DK / 16; ++ks) {
-            uint32_t ah[4], al[4];
-#pragma unroll
-            for (int p = 0; p < 4; ++p) split2(st[2 * ks + (p >> 1)][(p & 1) * 2], st[2 * ks + (p >> 1)][(p & 1) * 2 + 1], ah[p], al[p]);
-#pragma unroll
-            for (int tp0 = 0; tp0 < 4; tp0 += kPairs) {
-                if (tp0 * 16 >= n) continue;
-                uint32_t bq[kPairs][4], bk[kPairs][4];
-#pragma unroll
-                for (int e = 0; e < kPairs; ++e) {
-                    const int off = ((tp0 + e) * 16 + (mi >> 1) * 8 + r8) * ROW + ks * 16 + (mi & 1) * 8;
-                    ldmatrix_x4(smem_u32(&Q[off]), bq[e][0], bq[e][1], bq[e][2], bq[e][3]);
-                    if (RULE == kDelta) ldmatrix_x4(smem_u32(&K[off]), bk[e][0], bk[e][1], bk[e][2], bk[e][3]);
+            for (int i = 0; i < 2; ++i)
+                if (kt <= own[i]) {
+                    hi[i] = m[(own[i] * (own[i] + 1) / 2 + kt) * 64 + lane];
+                    lo[i] = m[(own[i] * (own[i] + 1) / 2 + kt) * 64 + 32 + lane];
                 }
 #pragma unroll
-                for (int part = 0; part < 2; ++part)
+            for (int part = 0; part < 3; ++part) {
+                if (part == 2 && xl == nullptr) continue;
 #pragma unroll
-                    for (int e = 0; e < kPairs; ++e) {
-                        const uint32_t(&x)[4] = part == 0 ? ah : al;
-                        mma_bf16_16816(o[2 * (tp0 + e)], x, bq[e][0], bq[e][1]);
-                        mma_bf16_16816(o[2 * (tp0 + e) + 1], x, bq[e][2], bq[e][3]);
-                        if (RULE == kDelta) {
-                            mma_bf16_16816(u[2 * (tp0 + e)], x, bk[e][0], bk[e][1]);
-                            mma_bf16_16816(u[2 * (tp0 + e) + 1], x, bk[e][2], bk[e][3]);
-                        }
+                for (int i = 0; i < 2; ++i)
+                    if (kt <= own[i]) {
+                        const uint4 b = part == 1 ? lo[i] : hi[i];
+                        mma_bf16_16816(acc[i][0], part == 2 ? xl[kt] : xh[kt], b.x, b.z);
+                        mma_bf16_16816(acc[i][1], part == 2 ? xl[kt] : xh[kt], b.y, b.w);
                     }
             }
         }
-        // V^T of 16 tokens: token pairs 2 tq of columns g and g + 8, then eight tokens on
-        auto values_of = [&](int tp, uint32_t (&x)[4]) {
-            ldmatrix_x4_trans(smem_u32(&V[(tp * 16 + (mi >> 1) * 8 + r8) * VROW + col0 + (mi & 1) * 8]), x[0], x[1], x[2], x[3]);
-        };
-        uint32_t xh[4][4], xl[RULE == kDelta ? 4 : 1][4];
+    };
+    // V^T of 16 tokens: token pairs 2 tq of columns g and g + 8, then eight tokens on
+    auto values_of = [&](const __nv_bfloat16* V, int tile, uint32_t (&x)[4]) {
+        ldmatrix_x4_trans(smem_u32(&V[(tile * 16 + (mi >> 1) * 8 + r8) * VROW + col0 + (mi & 1) * 8]), x[0], x[1], x[2], x[3]);
+    };
+    // accumulators of 16 tokens (tile, eight tokens further) as a left operand in two parts, for the pair
+    auto hand_over = [&](int which, int tile, const float (&c)[2][4]) {
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int p = 0; p < 4; ++p) split2(c[p >> 1][(p & 1) * 2], c[p >> 1][(p & 1) * 2 + 1], hi[p], lo[p]);
+        S.hand[which][pair][tile][0][lane] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        S.hand[which][pair][tile][1][lane] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    };
+    auto take = [&](int which, int tile, uint32_t (&hi)[4], uint32_t (&lo)[4]) {
+        const uint4 x = S.hand[which][pair][tile][0][lane], y = S.hand[which][pair][tile][1][lane];
+        hi[0] = x.x, hi[1] = x.y, hi[2] = x.z, hi[3] = x.w;
+        lo[0] = y.x, lo[1] = y.y, lo[2] = y.z, lo[3] = y.w;
+    };
+    auto pair_barrier = [&]() { asm volatile("bar.sync %0, 64;" ::"r"(1 + pair) : "memory"); };
+
+    int buf = 0;
+    for (int s0 = 0; s0 < ext; s0 += kChunk, buf ^= 1) {
+        const int n = min(kChunk, ext - s0);
+        const bool more = s0 + kChunk < ext;
+        cp_async_wait_all();
+        __syncthreads();   // this chunk and its factors are in place; nobody needs the last one's
+        if (more) {
+            chunks += chunk_vecs;
+            load_chunk(s0 + kChunk, buf ^ 1);
+            load_matrices(chunks, buf ^ 1);
+            if (warp == 0) fetch_factors(s0 + kChunk);
+        }
+        const __nv_bfloat16 *K = S.k[buf], *Q = S.q[buf], *V = S.v[buf];
+        // ---- S^T Q^T and S^T K^T ----
+        float o[2][2][4], u[2][2][4];
+        {
+            float po[4][2][4] = {}, pu[4][2][4] = {};
+#pragma unroll
+            for (int ks = 0; ks < kRows / 16; ++ks) {
+                uint32_t ah[4], al[4];
+#pragma unroll
+                for (int p = 0; p < 4; ++p)
+                    split2(st[2 * ks + (p >> 1)][(p & 1) * 2], st[2 * ks + (p >> 1)][(p & 1) * 2 + 1], ah[p], al[p]);
+#pragma unroll
+                for (int i0 = 0; i0 < 4; i0 += 2) {
+                    uint32_t bq[2][4], bk[2][4];
+#pragma unroll
+                    for (int i = 0; i < 2; ++i) {
+                        const int off = (own[i0 + i] * 16 + (mi >> 1) * 8 + r8) * ROW + half * kRows + ks * 16 + (mi & 1) * 8;
+                        ldmatrix_x4(smem_u32(&Q[off]), bq[i][0], bq[i][1], bq[i][2], bq[i][3]);
+                        if (RULE == kDelta) ldmatrix_x4(smem_u32(&K[off]), bk[i][0], bk[i][1], bk[i][2], bk[i][3]);
+                    }
+#pragma unroll
+                    for (int part = 0; part < 2; ++part) {
+                        const uint32_t(&x)[4] = part == 0 ? ah : al;
+#pragma unroll
+                        for (int i = 0; i < 2; ++i) {
+                            mma_bf16_16816(po[i0 + i][0], x, bq[i][0], bq[i][1]);
+                            mma_bf16_16816(po[i0 + i][1], x, bq[i][2], bq[i][3]);
+                            if (RULE == kDelta) {
+                                mma_bf16_16816(pu[i0 + i][0], x, bk[i][0], bk[i][1]);
+                                mma_bf16_16816(pu[i0 + i][1], x, bk[i][2], bk[i][3]);
+                            }
+                        }
+                    }
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int side = 0; side < 2; ++side) {
+                    const float *x = po[2 + i][side], *y = pu[2 + i][side];
+                    S.sums[pair][half][i][0][side][lane] = make_float4(x[0], x[1], x[2], x[3]);
+                    if (RULE == kDelta) S.sums[pair][half][i][RULE == kDelta ? 1 : 0][side][lane] = make_float4(y[0], y[1], y[2], y[3]);
+                }
+            pair_barrier();
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int side = 0; side < 2; ++side) {
+                    const float4 x = S.sums[pair][half ^ 1][i][0][side][lane];
+                    o[i][side][0] = po[i][side][0] + x.x;
+                    o[i][side][1] = po[i][side][1] + x.y;
+                    o[i][side][2] = po[i][side][2] + x.z;
+                    o[i][side][3] = po[i][side][3] + x.w;
+                    if (RULE == kDelta) {
+                        const float4 y = S.sums[pair][half ^ 1][i][RULE == kDelta ? 1 : 0][side][lane];
+                        u[i][side][0] = pu[i][side][0] + y.x;
+                        u[i][side][1] = pu[i][side][1] + y.y;
+                        u[i][side][2] = pu[i][side][2] + y.z;
+                        u[i][side][3] = pu[i][side][3] + y.w;
+                    }
+                }
+        }
+        uint32_t xh[4][4], xl[4][4];
         if (RULE == kDelta) {
             // ---- U = (I + A)^-1 (beta V - beta G K S) ----
 #pragma unroll
-            for (int tp = 0; tp < 4; ++tp) {
+            for (int i = 0; i < 2; ++i) {
                 uint32_t x[4];
-                values_of(tp, x);
+                values_of(V, own[i], x);
 #pragma unroll
                 for (int side = 0; side < 2; ++side) {
-                    const int t = tp * 16 + side * 8 + 2 * tq;
+                    const int t = own[i] * 16 + side * 8 + 2 * tq;
                     const float2 be = *reinterpret_cast<const float2*>(&S.beta[buf][t]), rd = *reinterpret_cast<const float2*>(&S.read[buf][t]);
-                    float* c = u[2 * tp + side];
+                    float* c = u[i][side];
                     c[0] = be.x * bf16_lo(x[2 * side]) - rd.x * c[0];
                     c[1] = be.y * bf16_hi(x[2 * side]) - rd.y * c[1];
                     c[2] = be.x * bf16_lo(x[2 * side + 1]) - rd.x * c[2];
                     c[3] = be.y * bf16_hi(x[2 * side + 1]) - rd.y * c[3];
                 }
-                split_tile(u, tp, xh[tp], xl[tp]);
+                hand_over(0, own[i], u[i]);
 #pragma unroll
-                for (int e = 0; e < 8; ++e) u[2 * tp + (e >> 2)][e & 3] = 0.f;
+                for (int e = 0; e < 8; ++e) u[i][e >> 2][e & 3] = 0.f;
+            }
+            pair_barrier();
+#pragma unroll
+            for (int kt = 0; kt < 4; ++kt) take(0, kt, xh[kt], xl[kt]);
+            multiply(u, xh, xl, S.m[buf] + kMatrixVecs);
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                hand_over(1, own[i], u[i]);
+#pragma unroll
+                for (int side = 0; side < 2; ++side) {
+                    const float2 w = *reinterpret_cast<const float2*>(&S.write[buf][own[i] * 16 + side * 8 + 2 * tq]);
+                    u[i][side][0] *= w.x;
+                    u[i][side][1] *= w.y;
+                    u[i][side][2] *= w.x;
+                    u[i][side][3] *= w.y;
+                }
+                hand_over(2, own[i], u[i]);
             }
         } else {
 #pragma unroll
-            for (int tp = 0; tp < 4; ++tp) values_of(tp, xh[tp]);
-        }
-        cp_async_wait<1>();
-        __syncthreads();   // the matrices
-        if (RULE == kDelta) {
-            multiply(u, xh, xl, S.m + kMatrixVecs, n);
-#pragma unroll
-            for (int tp = 0; tp < 4; ++tp) split_tile(u, tp, xh[tp], xl[tp]);
+            for (int kt = 0; kt < 4; ++kt) values_of(V, kt, xh[kt]);
         }
         // ---- O = G Q S + P U (+ skip V) ----
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            const float2 f = *reinterpret_cast<const float2*>(&S.out[buf][8 * j + 2 * tq]);
-            o[j][0] *= f.x;
-            o[j][1] *= f.y;
-            o[j][2] *= f.x;
-            o[j][3] *= f.y;
-            if (RULE == kStateSpace) {
-                const uint32_t *x = &xh[j >> 1][(j & 1) * 2];
-                o[j][0] = fmaf(skip, bf16_lo(x[0]), o[j][0]);
-                o[j][1] = fmaf(skip, bf16_hi(x[0]), o[j][1]);
-                o[j][2] = fmaf(skip, bf16_lo(x[1]), o[j][2]);
-                o[j][3] = fmaf(skip, bf16_hi(x[1]), o[j][3]);
+        for (int i = 0; i < 2; ++i) {
+            uint32_t x[4];
+            if (RULE == kStateSpace) values_of(V, own[i], x);
+#pragma unroll
+            for (int side = 0; side < 2; ++side) {
+                const float2 f = *reinterpret_cast<const float2*>(&S.out[buf][own[i] * 16 + side * 8 + 2 * tq]);
+                float* c = o[i][side];
+                c[0] *= f.x;
+                c[1] *= f.y;
+                c[2] *= f.x;
+                c[3] *= f.y;
+                if (RULE == kStateSpace) {
+                    c[0] = fmaf(skip, bf16_lo(x[2 * side]), c[0]);
+                    c[1] = fmaf(skip, bf16_hi(x[2 * side]), c[1]);
+                    c[2] = fmaf(skip, bf16_lo(x[2 * side + 1]), c[2]);
+                    c[3] = fmaf(skip, bf16_hi(x[2 * side + 1]), c[3]);
+                }
             }
         }
-        multiply(o, xh, RULE == kDelta ? xl : nullptr, S.m, n);
-        {
-            __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + static_cast<int64_t>(begin + s0 + g) * a.out_ld + at_v + col0 + 2 * tq;
+        if (RULE == kDelta) {
+            pair_barrier();
 #pragma unroll
-            for (int j = 0; j < 8; ++j) {
-                const uint32_t left = transpose_8x8(pack_bf16(o[j][0], o[j][1])), right = transpose_8x8(pack_bf16(o[j][2], o[j][3]));
-                if (8 * j + g >= n) continue;
-                *reinterpret_cast<uint32_t*>(out + static_cast<int64_t>(8 * j) * a.out_ld) = left;
-                *reinterpret_cast<uint32_t*>(out + static_cast<int64_t>(8 * j) * a.out_ld + 8) = right;
-            }
+            for (int kt = 0; kt < 4; ++kt) take(1, kt, xh[kt], xl[kt]);
+        }
+        multiply(o, xh, RULE == kDelta ? xl : nullptr, S.m[buf]);
+        {
+            __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + static_cast<int64_t>(begin + s0) * a.out_ld + at_v + col0 + 2 * tq;
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int side = 0; side < 2; ++side) {
+                    const float* c = o[i][side];
+                    const uint32_t left = transpose_8x8(pack_bf16(c[0], c[1])), right = transpose_8x8(pack_bf16(c[2], c[3]));
+                    const int t = own[i] * 16 + side * 8 + g;
+                    if (t >= n) continue;
+                    *reinterpret_cast<uint32_t*>(out + t * a.out_ld) = left;
+                    *reinterpret_cast<uint32_t*>(out + t * a.out_ld + 8) = right;
+                }
         }
         // ---- the state after the chunk ----
         const float keep = S.keep[buf];
 #pragma unroll
-        for (int j = 0; j < DK / 8; ++j)
+        for (int j = 0; j < kRows / 8; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) st[j][e] *= keep;
 #pragma unroll
         for (int kt = 0; kt < 4; ++kt) {
             if (kt * 16 >= n) continue;
             uint32_t wh[4], wl[4];
+            if (RULE == kDelta) {
+                take(2, kt, wh, wl);
+            } else {
 #pragma unroll
-            for (int p = 0; p < 4; ++p) {
-                const float2 w = *reinterpret_cast<const float2*>(&S.write[buf][kt * 16 + (p >> 1) * 8 + 2 * tq]);
-                const float* c = &u[2 * kt + (p >> 1)][(p & 1) * 2];
-                const float x = RULE == kDelta ? c[0] : bf16_lo(xh[kt][p]), y = RULE == kDelta ? c[1] : bf16_hi(xh[kt][p]);
-                split2(x * w.x, y * w.y, wh[p], wl[p]);
+                for (int p = 0; p < 4; ++p) {
+                    const float2 w = *reinterpret_cast<const float2*>(&S.write[buf][kt * 16 + (p >> 1) * 8 + 2 * tq]);
+                    split2(bf16_lo(xh[kt][p]) * w.x, bf16_hi(xh[kt][p]) * w.y, wh[p], wl[p]);
+                }
             }
+            uint32_t bk[kRows / 16][4];
 #pragma unroll
-            for (int dp0 = 0; dp0 < DK / 16; dp0 += 4) {
-                uint32_t bk[4][4];
+            for (int e = 0; e < kRows / 16; ++e)
+                ldmatrix_x4_trans(smem_u32(&K[(kt * 16 + (mi & 1) * 8 + r8) * ROW + half * kRows + e * 16 + (mi >> 1) * 8]), bk[e][0],
+                                  bk[e][1], bk[e][2], bk[e][3]);
 #pragma unroll
-                for (int e = 0; e < 4; ++e)
-                    ldmatrix_x4_trans(smem_u32(&K[(kt * 16 + (mi & 1) * 8 + r8) * ROW + (dp0 + e) * 16 + (mi >> 1) * 8]), bk[e][0], bk[e][1],
-                                      bk[e][2], bk[e][3]);
+            for (int part = 0; part < 2; ++part)
 #pragma unroll
-                for (int part = 0; part < 2; ++part)
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        const uint32_t(&x)[4] = part == 0 ? wh : wl;
-                        mma_bf16_16816(st[2 * (dp0 + e)], x, bk[e][0], bk[e][1]);
-                        mma_bf16_16816(st[2 * (dp0 + e) + 1], x, bk[e][2], bk[e][3]);
-                    }
-            }
+                for (int e = 0; e < kRows / 16; ++e) {
+                    const uint32_t(&x)[4] = part == 0 ? wh : wl;
+                    mma_bf16_16816(st[2 * e], x, bk[e][0], bk[e][1]);
+                    mma_bf16_16816(st[2 * e + 1], x, bk[e][2], bk[e][3]);
+                }
         }
         if (more && warp == 0) put_factors(buf ^ 1);
     }
 #pragma unroll
-    for (int j = 0; j < DK / 8; ++j)
+    for (int j = 0; j < kRows / 8; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) state[static_cast<int64_t>(8 * j + 2 * tq + (e & 1)) * vp + (e >> 1) * 8] = st[j][e];
 }
