@@ -216,24 +216,25 @@ mix_kernel(const Recurrence a, int v_blocks, int heads_per_block) {
         const int t = i / here, head = i - t * here;
         float ss = 0.f;
         for (int j = 0; j < per_head; ++j) ss += s_part[t][head * per_head + j];
-        float f = 1.f / sqrtf(ss + kUnitEps);
-        if (head0 + head >= a.kv_heads) f /= sqrtf(static_cast<float>(a.dim));
+        float f = rsqrtf(ss + kUnitEps);
+        if (head0 + head >= a.kv_heads) f *= rsqrtf(static_cast<float>(a.dim));
         a.units[static_cast<int64_t>(begin + t0 + t) * 2 * a.kv_heads + head0 + head] = f;
     }
 }
 
 // ---- token by token: decode, and prompts that the chunked kernels do not take ------------
 
-constexpr int kStepThreads = 256;
-constexpr int kMaxAhead = 16;   // state rows per thread, in registers
+constexpr int kStepThreads = 512;
+constexpr int kMaxAhead = 8;   // state rows per thread, in registers
 constexpr int kTapsAhead = 3;   // earlier inputs of a channel fetched together
 
 // Grid: heads, requests, blocks of 4 << log_cols value columns (at most kStepThreads).
 template <typename T, int RULE, bool DECODE, int AHEAD>
-__global__ void __launch_bounds__(kStepThreads, AHEAD > 8 ? 2 : 3)
+__global__ void __launch_bounds__(kStepThreads, 2)
 step_kernel(const Recurrence a, int log_cols, bool finish) {
     extern __shared__ __align__(16) float smem[];
     __shared__ float s_ss[kStepThreads / 32];
+    __shared__ float2 s_step;
     const int dk = a.padded_dim, vp = a.padded_value_dim;
     const int nv4 = 1 << log_cols, cols = nv4 * 4, groups = kStepThreads >> log_cols;
     float *s_v = smem, *s_k = s_v + cols, *s_q = s_k + dk, *s_red = s_q + dk;
@@ -243,15 +244,16 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
     const bool active = col0 + col < vp;
     const int64_t nv = values(a), nc = channels(a);
     const int64_t row_state = static_cast<int64_t>(a.table_idx[b]);
-    float* state = a.state + (row_state * a.heads + h) * dk * vp + col0 + col;
+    // this thread's rows: group, group + groups, ...
+    float* state = a.state + ((row_state * a.heads + h) * dk + group) * vp + col0 + col;
+    const int rows = group < dk ? (dk - group + groups - 1) >> (31 - __clz(groups)) : 0, row_step = groups * vp;
     const int cached = a.cached[b];
     pdl_launch_dependents();
     float4 x[AHEAD];
 #pragma unroll
     for (int i = 0; i < AHEAD; ++i) {
-        const int r = group + i * groups;
         x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (active && cached > 0 && r < dk) x[i] = load4(state + static_cast<int64_t>(r) * vp);
+        if (active && cached > 0 && i < rows) x[i] = load4(state + i * row_step);
     }
     // this CTA's channels: its value columns, the head's k and q
     const int own_v = min(cols, vp - col0), own = own_v + 2 * dk;
@@ -263,6 +265,7 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
     auto place = [&](int i) -> float& { return i < own_v ? s_v[i] : s_k[i - own_v]; };   // (s_q follows s_k)
     T* ring = static_cast<T*>(a.conv_state) + row_state * a.taps * nc;
     const int now = DECODE ? cached % a.taps : 0;
+    const bool steps = threadIdx.x == kStepThreads - 1;   // this thread works out the step
     float step_bias = 0.f, decay = 0.f, norm = 0.f;
     if (DECODE) {
         // what the inputs before this one add to the channels, two of them at a time
@@ -293,8 +296,10 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
                 place(i) = y[e];
             }
         }
-        step_bias = a.step_bias[h];
-        decay = a.decay_log[h];
+        if (steps) {
+            step_bias = a.step_bias[h];
+            decay = a.decay_log[h];
+        }
         if (finish && threadIdx.x < own_v) norm = to_f32(static_cast<const T*>(a.norm)[threadIdx.x]);
     }
     const float skip = RULE == kStateSpace ? a.skip[h] : 0.f;
@@ -306,7 +311,11 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
         float gate = 0.f;
         if (DECODE) {
             const T* tail = row + nv + nc;
-            const float za = to_f32(tail[h]), zb = RULE == kDelta ? to_f32(tail[a.heads + h]) : 0.f;
+            float za = 0.f, zb = 0.f;
+            if (steps) {
+                za = to_f32(tail[h]);
+                if (RULE == kDelta) zb = to_f32(tail[a.heads + h]);
+            }
             if (finish && threadIdx.x < own_v) gate = to_f32(row[static_cast<int64_t>(h) * vp + threadIdx.x]);
             T* keep = ring + static_cast<int64_t>(now) * nc;
             const bool keeps = h % (a.heads / a.kv_heads) == 0 && blockIdx.z == 0;   // k and q are shared
@@ -328,13 +337,14 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
                     if (i < own_v || keeps) keep[channel(i)] = in[e];
                 }
             }
-            step = make_step(RULE, za, zb, step_bias, decay);
+            if (steps) s_step = make_step(RULE, za, zb, step_bias, decay);
         } else {
             const T* mixed = static_cast<const T*>(a.mixed) + t * nc;
             for (int i = threadIdx.x; i < own; i += kStepThreads) place(i) = to_f32(mixed[channel(i)]);
             step = reinterpret_cast<const float2*>(a.steps)[t * a.heads + h];
         }
         __syncthreads();
+        if (DECODE) step = s_step;
         float kf = step.y, qf = 1.f;   // factors of k and q
         const float g = exp2f(step.x);
         if (RULE == kDelta) {
@@ -345,8 +355,8 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
                     sk += s_k[i] * s_k[i];
                     sq += s_q[i] * s_q[i];
                 }
-                kf = 1.f / sqrtf(warp_sum(sk) + kUnitEps);
-                qf = 1.f / sqrtf(warp_sum(sq) + kUnitEps) / sqrtf(static_cast<float>(a.dim));
+                kf = rsqrtf(warp_sum(sk) + kUnitEps);
+                qf = rsqrtf(warp_sum(sq) + kUnitEps) * rsqrtf(static_cast<float>(a.dim));
             } else {
                 kf = a.units[t * 2 * a.kv_heads + kvh];
                 qf = a.units[t * 2 * a.kv_heads + a.kv_heads + kvh];
@@ -357,9 +367,8 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
             float4 p = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
             for (int i = 0; i < AHEAD; ++i) {
-                const int r = group + i * groups;
-                if (r < dk) {
-                    const float k = s_k[r];
+                if (i < rows) {
+                    const float k = s_k[group + i * groups];
                     p.x = fmaf(k, x[i].x, p.x);
                     p.y = fmaf(k, x[i].y, p.y);
                     p.z = fmaf(k, x[i].z, p.z);
@@ -383,9 +392,8 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
         float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i) {
-            const int r = group + i * groups;
-            if (r < dk) {
-                const float k = kf * s_k[r], q = s_q[r];
+            if (i < rows) {
+                const float k = kf * s_k[group + i * groups], q = s_q[group + i * groups];
                 x[i].x = fmaf(k, u.x, g * x[i].x);
                 x[i].y = fmaf(k, u.y, g * x[i].y);
                 x[i].z = fmaf(k, u.z, g * x[i].z);
@@ -394,7 +402,7 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
                 o.y = fmaf(q, x[i].y, o.y);
                 o.z = fmaf(q, x[i].z, o.z);
                 o.w = fmaf(q, x[i].w, o.w);
-                if (DECODE && active) *reinterpret_cast<float4*>(state + static_cast<int64_t>(r) * vp) = x[i];
+                if (DECODE && active) *reinterpret_cast<float4*>(state + i * row_step) = x[i];
             }
         }
         *reinterpret_cast<float4*>(s_red + group * cols + col) = o;
@@ -421,10 +429,8 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
     }
     if (DECODE || !active || begin >= end) return;
 #pragma unroll
-    for (int i = 0; i < AHEAD; ++i) {
-        const int r = group + i * groups;
-        if (r < dk) *reinterpret_cast<float4*>(state + static_cast<int64_t>(r) * vp) = x[i];
-    }
+    for (int i = 0; i < AHEAD; ++i)
+        if (i < rows) *reinterpret_cast<float4*>(state + i * row_step) = x[i];
 }
 
 // ---- norm and gate of raw outputs, in place ------------------------------------------------
@@ -1215,9 +1221,9 @@ int launch_chunked(const Recurrence& a, cudaStream_t stream) {
 template <typename T, int RULE>
 int launch_steps(const Recurrence& a, int log_cols, int slices, bool finish, cudaStream_t stream) {
     const size_t smem = ((4ull << log_cols) + 2ull * a.padded_dim + kStepThreads * 4) * 4;
-    const bool few = div_ceil(a.padded_dim, kStepThreads >> log_cols) <= 8;
-    auto kernel = a.decode ? (few ? step_kernel<T, RULE, true, 8> : step_kernel<T, RULE, true, kMaxAhead>)
-                           : (few ? step_kernel<T, RULE, false, 8> : step_kernel<T, RULE, false, kMaxAhead>);
+    const bool few = div_ceil(a.padded_dim, kStepThreads >> log_cols) <= 4;
+    auto kernel = a.decode ? (few ? step_kernel<T, RULE, true, 4> : step_kernel<T, RULE, true, kMaxAhead>)
+                           : (few ? step_kernel<T, RULE, false, 4> : step_kernel<T, RULE, false, kMaxAhead>);
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(a.heads, a.batch, slices), dim3(kStepThreads), smem, stream, dim3(1, 1, 1), a,
                                   log_cols, finish));
     return B200_OK;
