@@ -55,7 +55,7 @@ __device__ __forceinline__ float silu<__nv_bfloat16>(float x) { return x * sigmo
 
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kUnitEps = 1e-6f;
-constexpr int kMaxTaps = 32;
+constexpr int kMaxTaps = 16;
 constexpr int kStateSpace = B200_RULE_STATE_SPACE, kDelta = B200_RULE_DELTA;
 
 // Channel c of [v | k | q] is column values() + c of a row of the joint projection.
@@ -98,7 +98,7 @@ __device__ __forceinline__ Vec8 unpack8(const Packed8<__nv_bfloat16>& p) {
 }
 
 constexpr int kMixThreads = 128;
-constexpr int kMixTokens = 32;
+constexpr int kMixTokens = 16;
 constexpr int kMixAhead = 2;   // tokens whose inputs are in flight
 
 // Grid: blocks of tokens, blocks of channels (8 per thread; those of k and q cover whole heads) and one for the
