@@ -372,7 +372,7 @@ B200_API int b200_linear_f32(float* y, const float* x, const float* w, int max_r
 B200_API int b200_linear_act(void* y, const void* x, const void* w, int M, int N, int K, int epilogue,
                              float act_limit, int dtype, b200_stream_t stream);
 
-/* The wiring with the norm on what a block returned:
+/* The wiring with the norm on what a block returned (layer_norm below: the same with layer norms):
  *   a = sum_k src_weights[t, k] src[src_rows[t, k], :] + src2[t, :]   (src_rows NULL: src[t, :]; weights NULL: 1),
  *   residual[t, :] += a / sqrt(mean(a^2) + eps) * add_weight          (add_weight NULL: += a; init: = instead of +=),
  *   out[t, :] = residual, or its RMS norm with out_weight when there is one.
@@ -382,21 +382,36 @@ B200_API int b200_residual_post_norm(void* out, float* residual, const void* src
                                      int init, const void* add_weight, const void* out_weight, int tokens,
                                      int width, int padded, float eps, int dtype, b200_stream_t stream);
 
-/* Routing by sigmoid scores of fp32 logits [tokens, logits_ld]: only experts of the best keep_groups of
+/* With y -> (y - mean) / sqrt(mean squared deviation + eps) * weight + bias as the norm:
+ *   a = sum_k src_weights[t, k] src[src_rows[t, k], :]   (a row of -1: the token's own row of `self` instead),
+ *   residual[t, :] += norm(a; add_weight, add_bias)      (NULL: += a; init: = a * src_scale instead of +=),
+ *   out[t, :] = norm(residual; out_weight, out_bias), or the residual without a weight. */
+B200_API int b200_residual_layer_norm(void* out, float* residual, const void* src, const int32_t* src_rows,
+                                      const float* src_weights, int src_top, int64_t src_count, const void* self,
+                                      float src_scale, int init, const void* add_weight, const void* add_bias,
+                                      const void* out_weight, const void* out_bias, int tokens, int width, int padded,
+                                      float eps, int dtype, b200_stream_t stream);
+
+enum { B200_SCORE_SIGMOID = 0, B200_SCORE_SOFTMAX = 1 };
+/* Routing by scores of fp32 logits [tokens, logits_ld], one per expert and then one per identity expert.
+ * B200_SCORE_SIGMOID: only experts of the best keep_groups of
  * `groups` equal groups (a group counts for the sum of its two best scores), the best `top` of those, weights =
- * scores over their sum (+ 1e-20) times scale.  ids, weights, rows [tokens, top]: the chosen experts and the
- * row each choice has in the expert-sorted order; counts [2 * experts] (the second half is scratch), offsets
+ * scores over their sum (+ 1e-20) times scale.  B200_SCORE_SOFTMAX: groups (which count for their best) and experts
+ * are chosen by softmax score + correction (fp32 per output, or NULL), weights = softmax scores times scale.  ids, weights,
+ * rows [tokens, top]: the chosen experts and the row each choice has in the expert-sorted order, -1 for an identity
+ * expert; counts [2 * experts] (the second half is scratch), offsets
  * [experts + 1]; the token's row of x (row_bytes) is copied to its rows of xp. */
 B200_API int b200_score_route(int32_t* ids, float* weights, int32_t* rows, int32_t* counts, int32_t* offsets,
                               void* xp, const void* x, int row_bytes, const float* logits, int64_t logits_ld,
                               int tokens, int experts, int top, int groups, int keep_groups, float scale,
-                              b200_stream_t stream);
+                              int score, int identity_experts, const float* correction, b200_stream_t stream);
 
 /* What lies between the joint projection of an attention layer and the attention: joint [tokens, joint_ld]
  * holds [heads * padded_dim | kv_heads * padded_dim | kv_heads * padded_value_dim | ...].  Queries (in place)
  * and keys (to k_cache [num_slots, kv_heads, padded_dim]) are RMS-normalised over `dim` with q_norm / k_norm
- * (NULL: not), then element i of the first rotary_dim turns with element i + rotary_dim / 2.  Values go to
- * v_cache; mix 1 keeps a copy in first_values, mix 2 stores (1 - lambda) v + lambda first_values. */
+ * (NULL: not; unit_norm: without a weight), then element i of the first rotary_dim turns with element i + rotary_dim / 2.
+ * Values go to v_cache; mix 1 keeps a copy in first_values, mix 2 stores (1 - lambda) v + lambda first_values.
+ * value_rotary > 0: element i of the first value_rotary of a value turns with element i + value_rotary / 2. */
 typedef struct b200_head_prepare_args {
     void* joint;
     int64_t joint_ld;
@@ -411,6 +426,8 @@ typedef struct b200_head_prepare_args {
     int32_t mix;
     const float* lambda;                  /* device */
     void* first_values;                   /* [tokens, kv_heads, padded_value_dim] */
+    int32_t unit_norm, value_rotary;
+    const float *value_cos, *value_sin;   /* [max_pos, value_rotary / 2] */
 } b200_head_prepare_args;
 B200_API int b200_head_prepare(const b200_head_prepare_args* args, int dtype, b200_stream_t stream);
 
@@ -443,7 +460,21 @@ typedef struct b200_window_attention_args {
     int32_t gate_per_head;   /* the gate is [tokens, heads]: one number per head */
     float out_scale;         /* a factor on the output; 0 means 1 */
     int64_t out_stride;      /* token stride of out in elements; 0: dense */
+    /* Heads that mix their weights: with p_g the softmax weights of head g, head h applies sum_g head_mix[h, g] p_g to
+     * the values of its own key / value head.  value_rotary > 0: the result at position p is then turned back by p,
+     * element i of the first value_rotary with element i + value_rotary / 2, before the gate.  No sinks. */
+    const float* head_mix;   /* [heads, heads] or NULL */
+    int32_t value_rotary, max_pos;
+    const float *value_cos, *value_sin;   /* [max_pos, value_rotary / 2] */
+    const int32_t* positions;             /* [tokens] */
+    float score_bound;       /* no q . k is larger than this; 0: not known.  (A bound lets the tensor-core kernels of mixing
+                                heads run without a running maximum; without one the plain kernel is used.) */
+    void* mix_scratch;       /* b200_head_mix_scratch_bytes */
 } b200_window_attention_args;
+/* Per (token, head), what the head's weights make of the values of every key / value head. */
+B200_API int64_t b200_head_mix_scratch_bytes(int tokens, int heads, int kv_heads, int padded_value_dim, int dtype);
+/* The workspace of mixing heads instead of b200_attention_decode_workspace_bytes. */
+B200_API int64_t b200_head_mix_workspace_bytes(int max_batch, int heads, int kv_heads);
 B200_API int b200_window_attention(const b200_window_attention_args* args, int dtype, b200_stream_t stream);
 
 /* Gated linear attention with one decay per key channel.  Per head, with state S [dim, value dim]:
@@ -470,9 +501,9 @@ typedef struct b200_linear_attention_args {
 } b200_linear_attention_args;
 B200_API int b200_linear_attention(const b200_linear_attention_args* args, int dtype, b200_stream_t stream);
 
-/* Recurrences with one decay per head, behind a short causal convolution.  joint [tokens, joint_ld] holds
- * [gate | v: heads * padded_value_dim each | k | q: kv_heads * padded_dim each | a of every head, and for the delta
- * rule b of every head]; head h uses k / q head h / (heads / kv_heads).
+/* Recurrences with one decay per head, the first two behind a short causal convolution.  joint [tokens, joint_ld] holds
+ * [gate | v: heads * padded_value_dim each | k | q: kv_heads * padded_dim each | a of every head (none for lightning),
+ * and for the delta rule and the matrix memory b of every head]; head h uses k / q head h / (heads / kv_heads).
  *   v, k, q <- silu(conv(.) + conv_bias): conv [taps, channels] per channel of [v | k | q], the last tap the
  *   current token's; conv_state [rows, taps, channels] of the dtype keeps the last inputs, that of position p at
  *   p mod taps
@@ -483,10 +514,17 @@ B200_API int b200_linear_attention(const b200_linear_attention_args* args, int d
  *   sqrt(sum of squares + 1e-6), q also by sqrt(dim)
  *   S <- g S,  u = beta (v - S^T k),  S <- S + k u^T,  o = S^T q,  out = rms(o) * norm * silu(gate) per head; norm
  *   [padded_value_dim]
+ * B200_RULE_LIGHTNING: v, k, q <- silu(.), g = exp(decay_log)
+ *   S <- g S + k v^T,  o = S^T q,  out = rms(o) * norm * sigmoid(gate) in norm_groups parts as above
+ * B200_RULE_MATRIX_MEMORY: v, k as they are, q / sqrt(dim); i = c tanh((a + step_bias[h]) / c),
+ *   f = log sigmoid(c tanh((b + step_bias[heads + h]) / c)) with c = gate_cap; from S = 0, n = 0, m = 0
+ *   m' = max(f + m, i),  S <- exp(f + m - m') S + exp(i - m') k v^T,  n likewise with k alone,  m <- m'
+ *   o = S^T q / (max(|n . q|, exp(-m)) + 1e-6),  out = rms(o) * norm * sigmoid(gate) in norm_groups parts;
+ *   memory fp32 [rows, heads, b200_recurrence_memory_bytes / 4] holds n and m
  * out [tokens, out_ld] is also multiplied by out_scale.  state fp32 [rows, heads, padded_dim, padded_value_dim];
  * rows, requests, decode and plain as for b200_linear_attention; a request brings at most max_extend tokens.  conv,
  * conv_bias (NULL: 0), decay_log, step_bias, skip are fp32.  Scratch: b200_recurrence_scratch. */
-enum { B200_RULE_STATE_SPACE = 0, B200_RULE_DELTA = 1 };
+enum { B200_RULE_STATE_SPACE = 0, B200_RULE_DELTA = 1, B200_RULE_LIGHTNING = 2, B200_RULE_MATRIX_MEMORY = 3 };
 typedef struct b200_recurrence_args {
     void* out;
     int64_t out_ld;
@@ -501,11 +539,16 @@ typedef struct b200_recurrence_args {
     const void* norm;
     float eps, out_scale;
     void* mixed;       /* [tokens, channels] of the dtype */
-    float* steps;      /* [tokens, heads, 2]: log2 of the decay, weight of what is written */
-    float* units;      /* delta rule [tokens, 2 kv_heads]: factors that make k and q unit vectors */
+    float* steps;      /* [tokens, heads, 2]: log2 of the decay, weight of what is written (matrix memory: its log2) */
+    float* units;      /* delta rule [tokens, 2 kv_heads]: factors that make k and q unit vectors; matrix memory
+                          [tokens, heads]: what a chunk's tokens add to n . q */
     void* chunks;      /* per 64 tokens and head: matrices of the chunked kernel */
+    float gate_cap;    /* matrix memory */
+    float* memory;
 } b200_recurrence_args;
 B200_API int b200_recurrence(const b200_recurrence_args* args, int dtype, b200_stream_t stream);
+/* Bytes per head of the matrix memory's n and m (one copy for every group of value columns that a CTA may work on). */
+B200_API int64_t b200_recurrence_memory_bytes(int padded_dim, int padded_value_dim);
 /* Bytes of mixed, steps, units and chunks for steps of at most max_tokens tokens of max_batch requests. */
 B200_API int b200_recurrence_scratch(int rule, int max_tokens, int max_batch, int heads, int kv_heads, int padded_dim,
                                      int padded_value_dim, int dtype, int64_t* bytes);
@@ -651,8 +694,12 @@ enum {
     B200_MIXER_WINDOW_ATTENTION = 1,
     B200_MIXER_LINEAR_ATTENTION = 2,
     B200_MIXER_STATE_SPACE = 3,   /* b200_recurrence, either rule */
-    B200_MIXER_DELTA_RULE = 4
+    B200_MIXER_DELTA_RULE = 4,
+    B200_MIXER_LIGHTNING = 5,     /* b200_recurrence as well */
+    B200_MIXER_MATRIX_MEMORY = 6
 };
+/* Norms on queries and keys: none, RMS norms with a weight, or division by the root mean square alone. */
+enum { B200_HEAD_NORM_NONE = 0, B200_HEAD_NORM_WEIGHTED = 1, B200_HEAD_NORM_UNIT = 2 };
 enum { B200_GATE_NONE = 0, B200_GATE_ELEMENT = 1, B200_GATE_HEAD = 2 };
 /* How the outputs of two mixers side by side become one. */
 enum {
@@ -660,6 +707,8 @@ enum {
     B200_JOIN_NORMED = 1    /* each RMS-normalised with its own weight, then half of their sum */
 };
 enum { B200_NORM_INPUT = 0, B200_NORM_OUTPUT = 1, B200_NORM_BOTH = 2 };
+/* The norms around blocks and before the output head: RMS norms, or layer norms with a weight and a bias. */
+enum { B200_NORM_RMS = 0, B200_NORM_LAYER = 1 };
 enum { B200_MLP_NONE = 0, B200_MLP_DENSE = 1, B200_MLP_TABLE_MOE = 2, B200_MLP_SCORED_MOE = 3 };
 
 typedef struct b200_layer_config {
@@ -696,16 +745,16 @@ typedef struct b200_layer_config {
     float act_limit;
     float shared_act_limit;
     /* window attention */
-    int32_t head_norm;       /* RMS norms on queries and keys */
+    int32_t head_norm;       /* B200_HEAD_NORM_* on queries and keys */
     int32_t gate;            /* B200_GATE_* on the output */
     int32_t qkv_bias;
     int32_t sink;            /* a score per head that joins the softmax's denominator */
     int32_t chunk;           /* > 0, instead of the window: keys of the query's own chunk of the sequence */
     /* rotations (latent attention: of the rotary_dim key dimensions that all heads share, in neighbouring pairs):
      * frequencies divided by rope_factor where their wavelength exceeds rope_original / rope_low, kept below
-     * rope_original / rope_high, blended between; factor 0: none */
+     * rope_original / rope_high, blended between; rope_original 0: all of them divided; factor 0: none */
     double rope_factor, rope_low, rope_high, rope_original;
-    int32_t kv_from;         /* latent attention: the layer whose latents this one reads, -1: its own */
+    int32_t kv_from;         /* latent and window attention: the layer whose cache this one reads, -1: its own */
     /* recurrences (head_dim: state rows; kv_heads: heads of k and q) */
     int32_t conv_taps;
     int32_t norm_groups;
@@ -713,6 +762,15 @@ typedef struct b200_layer_config {
     int32_t beside;          /* index into the stack's `beside`, -1: none */
     int32_t join;            /* B200_JOIN_* */
     float out_scale;         /* of this mixer's output (window attention, recurrences) */
+    /* window attention */
+    int32_t value_rotary;    /* cached values are rotated by their position over all of value_dim (base rope_base, no
+                                stretching), and what a query at position i gets out is turned back by i */
+    int32_t head_mix;        /* the softmax weights of every head become a sum over all heads' weights */
+    /* matrix memory */
+    float gate_cap;
+    /* scored experts */
+    int32_t score;           /* B200_SCORE_* */
+    int32_t identity_experts; /* the last outputs of the router: experts that return their input */
 } b200_layer_config;
 
 typedef struct b200_stack_config {
@@ -725,6 +783,8 @@ typedef struct b200_stack_config {
                             they return is normalised before it is added; or both */
     int32_t num_beside;
     const b200_layer_config* beside;   /* mixers that run beside another one (only mixer fields are read) */
+    int32_t norm_kind;   /* B200_NORM_RMS or B200_NORM_LAYER */
+    float embed_scale;   /* a factor on the embedding rows; 0 means 1 */
 } b200_stack_config;
 
 /* The padded size of a width / of a per-head dimension / of a latent width (see above). */
@@ -767,7 +827,9 @@ B200_API int b200_engine_destroy(b200_engine* engine);
  * projection "joint" [left columns + right columns, hidden], and under B200_JOIN_SUM "o" [hidden, left + right];
  * under B200_JOIN_NORMED there are "side_norm" [hidden] and the right one's "beside_o", "beside_side_norm".  The names
  * of the right one's other tensors start with "beside_".  Scored experts: "router" [experts, hidden],
- * "mlp_up", "mlp_down", "shared_up", "shared_down". */
+ * "mlp_up", "mlp_down", "shared_up", "shared_down", and with B200_SCORE_SOFTMAX "router_correction" fp32.  Layer norms
+ * add "norm1_bias", "norm2_bias", "norm1_out_bias", "norm2_out_bias" and "final_norm_bias".  "head_mix" fp32 [heads,
+ * heads] (also, as the identity, where only the values are rotated); "memory" fp32, see b200_recurrence. */
 B200_API int b200_engine_tensor(b200_engine* engine, const char* name, int layer, void** device_ptr,
                                 int64_t* nbytes);
 /* Synchronous host-to-device copy into a named tensor (nbytes must equal its size). */

@@ -34,10 +34,14 @@ EPILOGUE_F32 = 7
 
 DTYPE_BF16, DTYPE_F32 = 0, 1
 MIXER_LATENT_ATTENTION, MIXER_WINDOW_ATTENTION, MIXER_LINEAR_ATTENTION, MIXER_STATE_SPACE, MIXER_DELTA_RULE = 0, 1, 2, 3, 4
-RULE_STATE_SPACE, RULE_DELTA = 0, 1
+MIXER_LIGHTNING, MIXER_MATRIX_MEMORY = 5, 6
+RULE_STATE_SPACE, RULE_DELTA, RULE_LIGHTNING, RULE_MATRIX_MEMORY = 0, 1, 2, 3
+HEAD_NORM_NONE, HEAD_NORM_WEIGHTED, HEAD_NORM_UNIT = 0, 1, 2
 GATE_NONE, GATE_ELEMENT, GATE_HEAD = 0, 1, 2
 JOIN_SUM, JOIN_NORMED = 0, 1
 NORM_INPUT, NORM_OUTPUT, NORM_BOTH = 0, 1, 2
+NORM_RMS, NORM_LAYER = 0, 1
+SCORE_SIGMOID, SCORE_SOFTMAX = 0, 1
 MLP_NONE, MLP_DENSE, MLP_TABLE_MOE, MLP_SCORED_MOE = 0, 1, 2, 3
 
 
@@ -122,7 +126,11 @@ PROTOTYPES: dict[str, tuple] = {
     "b200_linear_f32": (_I, [_P, _P, _P, _I, _I, _I, _I, _P, _P, _I, _P]),
     "b200_linear_act": (_I, [_P, _P, _P, _I, _I, _I, _I, _F, _I, _P]),
     "b200_residual_post_norm": (_I, [_P, _P, _P, _P, _P, _I, _L, _P, _I, _P, _P, _I, _I, _I, _F, _I, _P]),
-    "b200_score_route": (_I, [_P, _P, _P, _P, _P, _P, _P, _I, _P, _L, _I, _I, _I, _I, _I, _F, _P]),
+    "b200_residual_layer_norm": (_I, [_P, _P, _P, _P, _P, _I, _L, _P, _F, _I, _P, _P, _P, _P, _I, _I, _I, _F, _I, _P]),
+    "b200_score_route": (_I, [_P, _P, _P, _P, _P, _P, _P, _I, _P, _L, _I, _I, _I, _I, _I, _F, _I, _I, _P, _P]),
+    "b200_head_mix_scratch_bytes": (_L, [_I, _I, _I, _I, _I]),
+    "b200_head_mix_workspace_bytes": (_L, [_I, _I, _I]),
+    "b200_recurrence_memory_bytes": (_L, [_I, _I]),
     "b200_head_prepare": (_I, [_P, _I, _P]),
     "b200_window_attention": (_I, [_P, _I, _P]),
     "b200_linear_attention": (_I, [_P, _I, _P]),
@@ -181,6 +189,8 @@ class LayerConfigStruct(ctypes.Structure):
         ("sink", c_int32), ("chunk", c_int32), ("rope_factor", ctypes.c_double), ("rope_low", ctypes.c_double),
         ("rope_high", ctypes.c_double), ("rope_original", ctypes.c_double), ("kv_from", c_int32),
         ("conv_taps", c_int32), ("norm_groups", c_int32), ("beside", c_int32), ("join", c_int32), ("out_scale", c_float),
+        ("value_rotary", c_int32), ("head_mix", c_int32), ("gate_cap", c_float), ("score", c_int32),
+        ("identity_experts", c_int32),
     ]
 
 
@@ -191,7 +201,8 @@ class HeadPrepareArgs(ctypes.Structure):
         ("dim", c_int32), ("padded_dim", c_int32), ("padded_value_dim", c_int32), ("q_norm", _P), ("k_norm", _P),
         ("eps", c_float), ("rotary_dim", c_int32), ("max_pos", c_int32), ("cos_table", _P), ("sin_table", _P),
         ("positions", _P), ("out_loc", _P), ("k_cache", _P), ("v_cache", _P), ("num_slots", _L), ("mix", c_int32),
-        ("lambda_", _P), ("first_values", _P),
+        ("lambda_", _P), ("first_values", _P), ("unit_norm", c_int32), ("value_rotary", c_int32), ("value_cos", _P),
+        ("value_sin", _P),
     ]
 
 
@@ -205,6 +216,8 @@ class WindowAttentionArgs(ctypes.Structure):
         ("padded_value_dim", c_int32), ("page_size", c_int32), ("scale", c_float), ("window", c_int32),
         ("keep_first", c_int32), ("gate", _P), ("gate_stride", _L), ("workspace", _P), ("workspace_bytes", _L),
         ("chunk", c_int32), ("sinks", _P), ("gate_per_head", c_int32), ("out_scale", c_float), ("out_stride", _L),
+        ("head_mix", _P), ("value_rotary", c_int32), ("max_pos", c_int32), ("value_cos", _P), ("value_sin", _P),
+        ("positions", _P), ("score_bound", c_float), ("mix_scratch", _P),
     ]
 
 
@@ -228,7 +241,7 @@ class RecurrenceArgs(ctypes.Structure):
         ("dim", c_int32), ("padded_dim", c_int32), ("value_dim", c_int32), ("padded_value_dim", c_int32),
         ("taps", c_int32), ("norm_groups", c_int32), ("conv", _P), ("conv_bias", _P), ("decay_log", _P),
         ("step_bias", _P), ("skip", _P), ("norm", _P), ("eps", c_float), ("out_scale", c_float), ("mixed", _P),
-        ("steps", _P), ("units", _P), ("chunks", _P),
+        ("steps", _P), ("units", _P), ("chunks", _P), ("gate_cap", c_float), ("memory", _P),
     ]
 
 
@@ -237,7 +250,7 @@ class StackConfigStruct(ctypes.Structure):
     _fields_ = [
         ("num_layers", c_int32), ("layers", POINTER(LayerConfigStruct)), ("dtype", c_int32),
         ("norm_offset", c_float), ("logit_scale", c_float), ("norm_output", c_int32), ("num_beside", c_int32),
-        ("beside", POINTER(LayerConfigStruct)),
+        ("beside", POINTER(LayerConfigStruct)), ("norm_kind", c_int32), ("embed_scale", c_float),
     ]
 
 

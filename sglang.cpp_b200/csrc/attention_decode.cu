@@ -26,9 +26,14 @@
 // WINDOW: everything AttentionWindow has.  A request's stages are then those that hold a kept key and those from
 // the oldest key in the window on; what lies between is never loaded.  Sinks, gates and the output's factor are
 // applied where it is written as bf16.
+// MT: mixing heads (head_mix.cuh).  All heads' weights of a stage go through shared memory, and every warp then
+// multiplies them with its key / value head's values of the whole stage, 16 * 8 / kv_heads columns of them: O_gc for all
+// pairs, in MT tiles of 16 heads g.  Scores are bounded, so there is no running maximum and partials simply add up; a
+// second kernel adds them, mixes and finishes.
 #include <mutex>
 
 #include "common.cuh"
+#include "head_mix.cuh"
 #include "kernels.h"
 #include "tensormap.cuh"
 
@@ -67,6 +72,7 @@ struct DecodeParams {
     int* status;
     int kv_evict_first;   // stream K/V through L2 with the evict-first policy (read once per step)
     AttentionWindow w;            // WINDOW only
+    float* ws_l;          // mixing heads: [max_items * KG, q_heads] sums of weights; ws_o [max_items, q_heads, kv_heads, 128]
 };
 
 // Which stages of a request of `len` keys are read: stage numbers [0, head) and, `skip` further, [head, count).
@@ -106,7 +112,8 @@ __device__ __forceinline__ void consumer_bar() {
     asm volatile("bar.sync 1, %0;" ::"n"(kConsumerThreads) : "memory");
 }
 
-template <bool WINDOW>
+// KEY_GROUPS: 16-key groups per stage (8 / kv_heads), with MT only.
+template <bool WINDOW, int MT, int KEY_GROUPS>
 __global__ void __launch_bounds__(kThreads, 1)
 attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
                         const __grid_constant__ CUtensorMap tmap_v, const DecodeParams p) {
@@ -116,6 +123,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
     __shared__ int s_prefix[kMaxBatch + 1];  // exclusive scan of items per request
     __shared__ int s_len[kMaxBatch];         // seq_lens, read once
     __shared__ int s_slot_tab[kSlotTab];
+    constexpr int kPRow = KEY_GROUPS * 16 + 8;   // mixing heads: a head's weights of a stage, padded for ldmatrix
+    __shared__ __align__(16) __nv_bfloat16 s_p[MT > 0 ? 2 : 1][MT > 0 ? MT * 16 * kPRow : 8];
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t smem_base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -129,6 +138,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
         }
         fence_mbar_init();
     }
+    if (MT > 0)
+        for (int i = threadIdx.x; i < 2 * MT * 16 * kPRow; i += kThreads) s_p[0][i] = __float2bfloat16_rn(0.f);
     if (warp == kConsumerWarps && lane == 0) {
         tma_prefetch_desc(&tmap_k);
         tma_prefetch_desc(&tmap_v);
@@ -300,6 +311,114 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
     const int Hq = p.q_heads;
 
     pdl_wait_prior();  // q comes from the kernel before this one
+    if constexpr (MT > 0) {
+        constexpr int NT = 16 / KEY_GROUPS;   // 8-column tiles of this warp
+        auto stage_row = [&](int j) -> uint32_t {   // of key j of a stage, of this warp's key / value head
+            return static_cast<uint32_t>((j & ~(p.kpc - 1)) * Hkv + h * p.kpc + (j & (p.kpc - 1)));
+        };
+        for (int at = g_begin; at < g_end;) {
+            const ItemInfo it = locate(at);
+            at += it.s_end - it.s_begin;
+            load_q(it.b);
+            float o[MT][NT][4], l0 = 0.f, l1 = 0.f;
+#pragma unroll
+            for (int i = 0; i < MT * NT * 4; ++i) o[i / (NT * 4)][i / 4 % NT][i % 4] = 0.f;
+            const int oldest = p.w.oldest(it.len - 1);
+            for (int st = it.s_begin; st < it.s_end; ++st, ++it_count) {
+                const uint32_t slot = it_count % kStages;
+                if (!failed && !mbar_wait_bounded(smem_u32(&full_bar[slot]), (it_count / kStages) & 1u, p.status, 203)) failed = true;
+                const uint32_t stage_base = smem_base + slot * kStageBytes;
+                const int stage_key = (st >= it.head ? st + it.skip : st) * SK;
+                const int key0 = stage_key + kg * 16, nvalid = it.len - key0;
+                // ---- this warp's weights: the heads of key head h, 16 keys ----
+                uint32_t w[4] = {0u, 0u, 0u, 0u};
+                if (!failed && nvalid > 0 && (key0 + min(nvalid, 16) > oldest || key0 < p.w.keep_first)) {
+                    if (nvalid < 16) {   // rows past the end hold stale bytes: 0 * garbage must stay 0
+                        for (int i = lane; i < (16 - nvalid) * 16; i += 32) {
+                            const int c16 = i & 15;
+                            const uint32_t a = stage_base + (2 + (c16 >> 3)) * kHalfBytes + stage_row(kg * 16 + nvalid + (i >> 4)) * 128u +
+                                               (c16 & 7) * 16u;
+                            asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(a), "r"(0u) : "memory");
+                        }
+                        fence_proxy_async_smem();
+                    }
+                    float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+                    const uint32_t rowoff = stage_row(kg * 16 + (mi >> 1) * 8 + r8) * 128u;
+#pragma unroll
+                    for (int ks = 0; ks < 8; ++ks) {
+                        const int c16 = ks * 2 + (mi & 1);
+                        uint32_t b00, b01, b10, b11;
+                        ldmatrix_x4(swz128(stage_base + (c16 >> 3) * kHalfBytes + rowoff, c16 & 7), b00, b01, b10, b11);
+                        mma_bf16_16816(s0, qa[ks], b00, b01);
+                        mma_bf16_16816(s1, qa[ks], b10, b11);
+                    }
+                    float x[8];
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) {
+                        const int key = (e >> 2) * 8 + 2 * t + (e & 1);
+                        const bool sees = key < nvalid && (key0 + key >= oldest || key0 + key < p.w.keep_first);
+                        x[e] = sees ? exp2f((e < 4 ? s0[e] : s1[e - 4]) * p.scale_log2) : 0.f;
+                    }
+                    l0 += (x[0] + x[1]) + (x[4] + x[5]);
+                    l1 += (x[2] + x[3]) + (x[6] + x[7]);
+                    w[0] = pack_bf16(x[0], x[1]);
+                    w[1] = pack_bf16(x[2], x[3]);
+                    w[2] = pack_bf16(x[4], x[5]);
+                    w[3] = pack_bf16(x[6], x[7]);
+                }
+                __nv_bfloat16* P = s_p[it_count & 1];
+                {
+                    uint32_t* row = reinterpret_cast<uint32_t*>(P + (h * G + g) * kPRow + kg * 16 + 2 * t);
+                    if (g < G) row[0] = w[0], row[4] = w[2];
+                    row += 8 * (kPRow / 2);
+                    if (g + 8 < G) row[0] = w[1], row[4] = w[3];
+                }
+                consumer_bar();   // (the other buffer's readers are through: they have been at this barrier)
+                // ---- all heads' weights times this warp's columns of its head's values ----
+#pragma unroll
+                for (int ks = 0; ks < KEY_GROUPS; ++ks) {
+                    if (failed || stage_key + ks * 16 >= it.len) break;
+                    uint32_t pa[MT][4];
+#pragma unroll
+                    for (int i = 0; i < MT; ++i)
+                        ldmatrix_x4(smem_u32(P + (i * 16 + (lane & 15)) * kPRow + ks * 16 + (lane >> 4) * 8), pa[i][0], pa[i][1], pa[i][2],
+                                    pa[i][3]);
+                    const uint32_t rowoff = stage_row(ks * 16 + (mi & 1) * 8 + r8) * 128u;
+#pragma unroll
+                    for (int np = 0; np < NT / 2; ++np) {
+                        const int c16 = kg * NT + np * 2 + (mi >> 1);
+                        uint32_t v0, v1, v2, v3;
+                        ldmatrix_x4_trans(swz128(stage_base + (2 + (c16 >> 3)) * kHalfBytes + rowoff, c16 & 7), v0, v1, v2, v3);
+#pragma unroll
+                        for (int i = 0; i < MT; ++i) {
+                            mma_bf16_16816(o[i][2 * np], pa[i], v0, v1);
+                            mma_bf16_16816(o[i][2 * np + 1], pa[i], v2, v3);
+                        }
+                    }
+                }
+                __syncwarp();
+                if (lane == 0) mbar_arrive(smem_u32(&empty_bar[slot]));
+            }
+            l0 += __shfl_xor_sync(0xffffffffu, l0, 1);
+            l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
+            l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
+            l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+            float* l = p.ws_l + (static_cast<int64_t>(it.item) * KG + kg) * Hq + h * G + g;
+            if (t == 0 && g < G) l[0] = l0;
+            if (t == 0 && g + 8 < G) l[8] = l1;
+#pragma unroll
+            for (int i = 0; i < MT; ++i)
+#pragma unroll
+                for (int rr = 0; rr < 2; ++rr) {
+                    const int head = i * 16 + g + rr * 8;
+                    if (head >= Hq) continue;
+                    float* dst = p.ws_o + ((static_cast<int64_t>(it.item) * Hq + head) * Hkv + h) * kD + kg * NT * 8 + 2 * t;
+#pragma unroll
+                    for (int n = 0; n < NT; ++n) *reinterpret_cast<float2*>(dst + n * 8) = make_float2(o[i][n][2 * rr], o[i][n][2 * rr + 1]);
+                }
+        }
+        return;
+    }
     int gpos = g_begin;
     bool have = gpos < g_end;
     ItemInfo it = {};
@@ -485,6 +604,29 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
 // of the streaming kernel on purpose: there the CTA that happened to deliver a request's last partial
 // merged it behind its own last stage, a chain of fences, a ticket and three dependent trips to L2 that
 // left the other 147 SMs and HBM idle for about 12 us per launch.
+// The first stage of request b, its stages, and those of all requests, as the attention kernel counts them (one warp).
+template <bool WINDOW>
+__device__ __forceinline__ int3 request_stages(const DecodeParams& p, int b) {
+    const int lane = threadIdx.x & 31;
+    int carry = 0, first = 0, mine = 0;
+    for (int base = 0; base < p.batch; base += 32) {
+        const int r = base + lane;
+        const int n = r < p.batch ? stage_range<WINDOW>(p.seq_lens[r], p.stage_keys, p.w).count : 0;
+        int incl = n;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int t = __shfl_up_sync(0xffffffffu, incl, o);
+            if (lane >= o) incl += t;
+        }
+        if (b >= base && b < base + 32) {
+            first = carry + __shfl_sync(0xffffffffu, incl - n, b - base);
+            mine = __shfl_sync(0xffffffffu, n, b - base);
+        }
+        carry += __shfl_sync(0xffffffffu, incl, 31);
+    }
+    return make_int3(first, mine, carry);
+}
+
 template <bool WINDOW>
 __global__ void __launch_bounds__(kMergeWarps * 32)
 attention_decode_merge_kernel(const DecodeParams p, int attn_grid) {
@@ -494,30 +636,14 @@ attention_decode_merge_kernel(const DecodeParams p, int attn_grid) {
     const int ctas_per_req = (p.q_heads + heads_per_cta - 1) / heads_per_cta;
     const int b = static_cast<int>(blockIdx.x) / ctas_per_req;
     const int head = (static_cast<int>(blockIdx.x) % ctas_per_req) * heads_per_cta + warp;
-    const int SK = p.stage_keys;
     pdl_launch_dependents();
     // seq_lens were complete before the attention kernel started: the split runs ahead of the wait
     if (warp == 0) {
-        int carry = 0, first = 0, mine = 0;
-        for (int base = 0; base < p.batch; base += 32) {
-            const int r = base + lane;
-            const int n = r < p.batch ? stage_range<WINDOW>(p.seq_lens[r], SK, p.w).count : 0;
-            int incl = n;
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const int t = __shfl_up_sync(0xffffffffu, incl, o);
-                if (lane >= o) incl += t;
-            }
-            if (b >= base && b < base + 32) {
-                first = carry + __shfl_sync(0xffffffffu, incl - n, b - base);
-                mine = __shfl_sync(0xffffffffu, n, b - base);
-            }
-            carry += __shfl_sync(0xffffffffu, incl, 31);
-        }
+        const int3 r = request_stages<WINDOW>(p, b);
         if (lane == 0) {
-            s_first = first;
-            s_stages = mine;
-            s_total = carry;
+            s_first = r.x;
+            s_stages = r.y;
+            s_total = r.z;
         }
     }
     __syncthreads();
@@ -588,7 +714,147 @@ attention_decode_merge_kernel(const DecodeParams p, int attn_grid) {
     *reinterpret_cast<uint2*>(p.out + (WINDOW ? b * p.w.out_st : static_cast<int64_t>(b) * Hq * kD) + head * kD + lane * 4) = packed;
 }
 
+// Mixing heads: the partials of a request added up, mixed and finished.  One CTA per (request, key / value head); its warps
+// share the heads that are summed over.  HC: room for the heads of a group.
+constexpr int kMixThreads = 256, kMixWarps = kMixThreads / 32;
+
+template <int HC>
+__global__ void __launch_bounds__(kMixThreads)
+decode_mix_kernel(const DecodeParams p, const MixOutput a, int attn_grid) {
+    __shared__ int3 s_split;
+    constexpr int kOnce = HC < 8 ? HC : 8;   // heads added up at a time
+    __shared__ float4 s_part[kMixWarps][kOnce][32];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int b = blockIdx.x, c = blockIdx.y, H = a.heads, group = p.group, pairs = a.pairs();
+    pdl_launch_dependents();
+    if (warp == 0) {
+        const int3 r = request_stages<true>(p, b);
+        if (lane == 0) s_split = r;
+    }
+    __syncthreads();
+    const int first = s_split.x, st = s_split.y;
+    const int per = max((s_split.z + attn_grid - 1) / attn_grid, kMinStagesPerCta), c0 = first / per;
+    const int items = st > 0 ? (first + st - 1) / per - c0 + 1 : 0;
+    const int KG = kConsumerWarps / p.kv_heads;
+    const int64_t item0 = b + c0;
+    const bool even = (pairs & 1) == 0;
+    const int m = 2 * lane;
+    float2 u[HC], v[HC];
+#pragma unroll
+    for (int i = 0; i < HC; ++i) u[i] = v[i] = make_float2(0.f, 0.f);
+    pdl_wait_prior();
+    for (int g = warp; g < H; g += kMixWarps) {
+        float l = 0.f;
+        for (int i = lane; i < items * KG; i += 32) l += __ldcg(p.ws_l + (item0 * KG + i) * H + g);
+        l = warp_sum(l);
+        float2 x = make_float2(0.f, 0.f), y = x;
+        if (m < pairs) {
+            const float* o = p.ws_o + ((item0 * H + g) * p.kv_heads + c) * kD + m;
+            const int64_t step = static_cast<int64_t>(H) * p.kv_heads * kD;
+#pragma unroll 4
+            for (int i = 0; i < items; ++i, o += step) {
+                const float2 d = load_pair(o, true);
+                const float2 e = m + 1 < pairs ? load_pair(o + pairs, even) : make_float2(o[pairs], 0.f);
+                x.x += d.x, x.y += d.y, y.x += e.x, y.y += e.y;
+            }
+        }
+        const float inv = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+        for (int i = 0; i < HC; ++i) {
+            if (i >= group) break;
+            const float f = a.weights[static_cast<int64_t>(c * group + i) * H + g] * inv;
+            u[i].x = fmaf(f, x.x, u[i].x);
+            u[i].y = fmaf(f, x.y, u[i].y);
+            v[i].x = fmaf(f, y.x, v[i].x);
+            v[i].y = fmaf(f, y.y, v[i].y);
+        }
+    }
+#pragma unroll
+    for (int h0 = 0; h0 < HC; h0 += kOnce) {
+        if (h0 > 0) __syncthreads();
+#pragma unroll
+        for (int i = 0; i < kOnce; ++i) s_part[warp][i][lane] = make_float4(u[h0 + i].x, u[h0 + i].y, v[h0 + i].x, v[h0 + i].y);
+        __syncthreads();
+        for (int i = warp; i < min(kOnce, group - h0); i += kMixWarps) {
+            float4 s = s_part[0][i][lane];
+#pragma unroll
+            for (int w = 1; w < kMixWarps; ++w) {
+                const float4 x = s_part[w][i][lane];
+                s.x += x.x, s.y += x.y, s.z += x.z, s.w += x.w;
+            }
+            const int head = c * group + h0 + i;
+            if (m < pairs) finish_mixed<__nv_bfloat16>(a, b, head, m, make_float2(s.x, s.y), make_float2(s.z, s.w));
+            clear_padding<__nv_bfloat16>(a, b, head);
+        }
+    }
+}
+
+// The attention kernel of mixing heads for these counts, or NULL.
+auto talking_kernel(int heads, int kv_heads) -> decltype(&attention_decode_kernel<true, 1, 1>) {
+    if (kv_heads < 1 || kv_heads > 8 || 8 % kv_heads != 0 || heads % kv_heads != 0 || heads / kv_heads > 16) return nullptr;
+    const int tiles = div_ceil(heads, 16);
+    switch (kv_heads) {
+        case 1: return attention_decode_kernel<true, 1, 8>;
+        case 2: return tiles == 1 ? attention_decode_kernel<true, 1, 4> : attention_decode_kernel<true, 2, 4>;
+        case 4: return tiles == 1 ? attention_decode_kernel<true, 1, 2>
+                                  : tiles == 2 ? attention_decode_kernel<true, 2, 2> : attention_decode_kernel<true, 4, 2>;
+        default: return tiles == 1 ? attention_decode_kernel<true, 1, 1> : tiles == 2 ? attention_decode_kernel<true, 2, 1> : nullptr;
+    }
+}
+
 }  // namespace
+
+bool talking_decode_supported(int heads, int kv_heads) { return talking_kernel(heads, kv_heads) != nullptr; }
+
+int64_t head_mix_workspace_bytes(int max_batch, int heads, int kv_heads) {
+    const int64_t items = static_cast<int64_t>(sm_count()) + max_batch;
+    return items * heads * (static_cast<int64_t>(kv_heads) * kD + kConsumerWarps / kv_heads) * 4 + 512;
+}
+
+int launch_talking_decode(const WindowAttention& a, cudaStream_t stream) {
+    const int grid = sm_count();
+    if (a.workspace_bytes < head_mix_workspace_bytes(a.batch, a.heads, a.kv_heads)) {
+        set_last_error("talking heads: workspace of %lld bytes is too small (need %lld)", static_cast<long long>(a.workspace_bytes),
+                       static_cast<long long>(head_mix_workspace_bytes(a.batch, a.heads, a.kv_heads)));
+        return B200_ERR_INVALID_ARGUMENT;
+    }
+    DecodeParams p = {};
+    p.q = static_cast<const __nv_bfloat16*>(a.q);
+    p.q_st = a.q_st;
+    p.q_sh = a.dp;
+    p.page_table = a.page_table;
+    p.pt_stride = a.pt_stride;
+    p.table_idx = a.table_idx;
+    p.seq_lens = a.seq_lens;
+    p.batch = a.batch;
+    p.q_heads = a.heads;
+    p.kv_heads = a.kv_heads;
+    p.group = a.heads / a.kv_heads;
+    p.stage_keys = kStageRows / a.kv_heads;
+    p.kpc = a.page_size < p.stage_keys ? a.page_size : p.stage_keys;
+    p.num_slots = a.num_slots;
+    p.scale_log2 = a.scale * kLog2e;
+    p.max_items = grid + a.batch;
+    p.status = a.status;
+    p.kv_evict_first = 1;
+    p.w = a.window;
+    p.ws_o = reinterpret_cast<float*>((reinterpret_cast<uintptr_t>(a.workspace) + 255) & ~uintptr_t(255));
+    p.ws_l = p.ws_o + static_cast<int64_t>(p.max_items) * a.heads * a.kv_heads * kD;
+    CUtensorMap tk, tv;
+    int err = make_kv_tmap(&tk, a.k_cache, a.num_slots, a.kv_heads, a.page_size);
+    if (err != B200_OK) return err;
+    err = make_kv_tmap(&tv, a.v_cache, a.num_slots, a.kv_heads, a.page_size);
+    if (err != B200_OK) return err;
+    auto kernel = talking_kernel(a.heads, a.kv_heads);
+    const int smem = kStages * kStageBytes + 1024;
+    B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    B200_CHECK_CUDA(launch_kernel(kernel, dim3(grid), dim3(kThreads), smem, stream, dim3(1, 1, 1), tk, tv, p));
+    const int g = p.group;
+    auto mix = g <= 1 ? decode_mix_kernel<1> : g <= 2 ? decode_mix_kernel<2> : g <= 4 ? decode_mix_kernel<4>
+               : g <= 8 ? decode_mix_kernel<8> : decode_mix_kernel<16>;
+    B200_CHECK_CUDA(launch_kernel(mix, dim3(a.batch, a.kv_heads), dim3(kMixThreads), 0, stream, dim3(1, 1, 1), p, mix_output(a), grid));
+    return B200_OK;
+}
 
 int64_t decode_workspace_bytes(int max_batch, int q_heads, int kv_heads) {
     const int kg = kConsumerWarps / kv_heads;
@@ -642,7 +908,7 @@ int launch_attention_decode(void* out, const void* q, int64_t q_st, int64_t q_sh
     p.kv_evict_first = kv_evict_first ? 1 : 0;
     if (window) p.w = *window;
     if (p.w.out_st == 0) p.w.out_st = static_cast<int64_t>(q_heads) * kD;
-    auto kernel = window ? attention_decode_kernel<true> : attention_decode_kernel<false>;
+    auto kernel = window ? attention_decode_kernel<true, 0, 1> : attention_decode_kernel<false, 0, 1>;
 
     const int smem = kStages * kStageBytes + 1024;
     // The attribute belongs to (function, device): set it on every launch, as the other launchers do.

@@ -61,45 +61,6 @@ struct PrefillTc2Params {
     AttentionWindow w;          // WINDOW only
 };
 
-// MN-major operand under the 128-byte swizzle (V as the B operand of P V: rows are keys, 64 head-dim
-// elements per 128-byte row): 8-key groups 1024 bytes apart along K, the second 64 head-dim elements one
-// atom (16 KB) further.
-__device__ __forceinline__ uint64_t mnmajor_sw128_desc2(uint32_t smem_addr) {
-    uint64_t d = 0;
-    d |= static_cast<uint64_t>((smem_addr >> 4) & 0x3FFFu);
-    d |= static_cast<uint64_t>(kAtomBytes >> 4) << 16;
-    d |= static_cast<uint64_t>(1024 >> 4) << 32;
-    d |= static_cast<uint64_t>(1) << 46;
-    d |= static_cast<uint64_t>(2) << 61;
-    return d;
-}
-__device__ __forceinline__ uint32_t idesc2_128x128(bool b_mn_major) {
-    return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn_major ? (1u << 16) : 0u) |
-           (static_cast<uint32_t>(128 >> 3) << 17) | (static_cast<uint32_t>(128 >> 4) << 24);
-}
-// D[tmem] (+)= A[tmem] * B[smem]
-__device__ __forceinline__ void tc_mma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc,
-                                               uint32_t accumulate) {
-    asm volatile(
-        "{\n\t"
-        ".reg .pred p;\n\t"
-        "setp.ne.b32 p, %4, 0;\n\t"
-        "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t"
-        "}\n" ::"r"(tmem_d),
-        "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate)
-        : "memory");
-}
-__device__ __forceinline__ void tmem_st_32x32b_x32(uint32_t taddr, const uint32_t (&v)[32]) {
-    asm volatile(
-        "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-        "{%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,"
-        "%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31,%32};" ::"r"(taddr),
-        "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]),
-        "r"(v[9]), "r"(v[10]), "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15]), "r"(v[16]),
-        "r"(v[17]), "r"(v[18]), "r"(v[19]), "r"(v[20]), "r"(v[21]), "r"(v[22]), "r"(v[23]), "r"(v[24]),
-        "r"(v[25]), "r"(v[26]), "r"(v[27]), "r"(v[28]), "r"(v[29]), "r"(v[30]), "r"(v[31])
-        : "memory");
-}
 template <bool WINDOW>
 __global__ void __launch_bounds__(kThreads, 1)
 attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
@@ -260,8 +221,8 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
     } else if (warp == 1) {
         // ================= MMA issuer =================
         if (lane == 0) {
-            const uint32_t idesc_s = idesc2_128x128(false);
-            const uint32_t idesc_pv = idesc2_128x128(true);
+            const uint32_t idesc_s = idesc_bf16_128x128(false);
+            const uint32_t idesc_pv = idesc_bf16_128x128(true);
             bool failed = false;
             // S_i = Q_i K^T of K/V tile kt (the K tile's barrier is waited for by whoever comes first)
             auto issue_s = [&](int i, int kt) {
@@ -300,7 +261,7 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
                 for (int ks = 0; ks < 8; ++ks) {
                     // keys ks*16 .. +15: eight packed columns; keys 64-127 start at column 64
                     const uint32_t a = s_base + static_cast<uint32_t>((ks >> 2) * 64 + (ks & 3) * 8);
-                    tc_mma_bf16_ts(d, a, mnmajor_sw128_desc2(v_addr + ks * 2048), idesc_pv, (kt > 0 || ks > 0) ? 1u : 0u);
+                    tc_mma_bf16_ts(d, a, mnmajor_sw128_desc(v_addr + ks * 2048), idesc_pv, (kt > 0 || ks > 0) ? 1u : 0u);
                 }
                 tc_commit(smem_u32(&pv_done[i]));
                 if (i == 1) tc_commit(smem_u32(&v_empty[slot]));   // both tiles have read this V tile
@@ -504,7 +465,9 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap tmap_k,
     if (warp == 1) tmem_dealloc(tmem_base, 512);
 }
 
-int make_kv_tmap_3d_tc2(CUtensorMap* out, const void* cache, int64_t num_slots, int kv_heads, int kpc) {
+}  // namespace
+
+int make_kv_tile_tmap(CUtensorMap* out, const void* cache, int64_t num_slots, int kv_heads, int kpc) {
     EncodeTiledFn fn = encode_tiled_fn();
     if (!fn) {
         set_last_error("cuTensorMapEncodeTiled is not available from this driver");
@@ -523,8 +486,6 @@ int make_kv_tmap_3d_tc2(CUtensorMap* out, const void* cache, int64_t num_slots, 
     }
     return B200_OK;
 }
-
-}  // namespace
 
 int launch_attention_prefill_tc2(void* out, const void* q, int64_t q_st, int64_t q_sh, const void* k_cache,
                                  const void* v_cache, int64_t num_slots, const int32_t* page_table,
@@ -553,16 +514,16 @@ int launch_attention_prefill_tc2(void* out, const void* q, int64_t q_st, int64_t
     if (window) p.w = *window;
     if (p.w.out_st == 0) p.w.out_st = static_cast<int64_t>(q_heads) * kD;
     CUtensorMap tk, tv;
-    int err = make_kv_tmap_3d_tc2(&tk, k_cache, num_slots, kv_heads, p.kpc);
+    int err = make_kv_tile_tmap(&tk, k_cache, num_slots, kv_heads, p.kpc);
     if (err != B200_OK) return err;
-    err = make_kv_tmap_3d_tc2(&tv, v_cache, num_slots, kv_heads, p.kpc);
+    err = make_kv_tile_tmap(&tv, v_cache, num_slots, kv_heads, p.kpc);
     if (err != B200_OK) return err;
     CUtensorMap tk_tile, tv_tile;   // 128-key boxes for tiles whose pages are consecutive slots
     const int tile_box = num_slots >= kTile ? kTile : p.kpc;
     p.whole_tile_boxes = (tile_box == kTile && p.kpc < kTile) ? 1 : 0;
-    err = make_kv_tmap_3d_tc2(&tk_tile, k_cache, num_slots, kv_heads, tile_box);
+    err = make_kv_tile_tmap(&tk_tile, k_cache, num_slots, kv_heads, tile_box);
     if (err != B200_OK) return err;
-    err = make_kv_tmap_3d_tc2(&tv_tile, v_cache, num_slots, kv_heads, tile_box);
+    err = make_kv_tile_tmap(&tv_tile, v_cache, num_slots, kv_heads, tile_box);
     if (err != B200_OK) return err;
     const int QB = kTile / p.group;
     const int smem = kSmemBytes + 1024;

@@ -160,6 +160,11 @@ struct ResidualPostNorm {
     bool init = false;                      // the sum replaces the residual
     const void* add_weight = nullptr;       // NULL: what is added is not normalised
     const void* out_weight = nullptr;       // NULL: out is the residual itself
+    // Layer norms instead of RMS norms (weight_offset and out_scale do not apply, nor do pairs).
+    bool layer = false;
+    const void *add_bias = nullptr, *out_bias = nullptr;
+    const void* self = nullptr;             // what a source row of -1 stands for: the token's own row here
+    float src_scale = 1.f;                  // with init: a factor on what is added
     float weight_offset = 0.f, out_scale = 1.f;   // as in ResidualNorm
     int tokens = 0, width = 0, padded = 0;
     float eps = 0.f;
@@ -178,13 +183,16 @@ constexpr int kMaxTableExperts = 4096;
 int launch_table_route(const TableRouteLayer* layers_dev, int num_layers, int max_experts, const int32_t* token_ids,
                        int tokens, int vocab, int* status, cudaStream_t stream);
 
-// Routing by sigmoid scores (moe.cu): ids, weights and counts from fp32 logits, then a row for every choice
+// Routing by scores (moe.cu; b200_score_route): ids, weights and counts from fp32 logits, then a row for every choice
 // and the token's activations copied there.  counts [experts] and the cursor [experts] are zero before.
 struct ScoreRoute {
     const float* logits = nullptr;   // [tokens, ld]
     int64_t ld = 0;
     int tokens = 0, experts = 0, top = 1, groups = 1, keep = 1;
     float scale = 1.f;
+    int score = B200_SCORE_SIGMOID;
+    int identity = 0;                // logits behind those of the experts: experts that return their input
+    const float* correction = nullptr;   // softmax scores: what a choice adds to a score, or NULL
     int32_t* ids = nullptr;          // [tokens, top]
     float* weights = nullptr;        // [tokens, top]
     int32_t* counts = nullptr;
@@ -302,6 +310,8 @@ struct AttentionWindow {
     }
 };
 
+// A pool [slots, kv heads, 128] in boxes of 64 elements of one head of kpc slots (attention_prefill_tc2.cu).
+int make_kv_tile_tmap(CUtensorMap* out, const void* cache, int64_t num_slots, int kv_heads, int kpc);
 int64_t decode_workspace_bytes(int max_batch, int q_heads, int kv_heads);
 int make_kv_tmap(CUtensorMap* out, const void* cache, int64_t num_slots, int kv_heads, int page_size);
 int launch_attention_decode(void* out, const void* q, int64_t q_st, int64_t q_sh,
@@ -328,9 +338,22 @@ struct HeadPrepare {
     int mix = kPlain;
     const float* lambda = nullptr;                         // v <- (1 - lambda) v + lambda first
     void* first_values = nullptr;                          // [tokens, kv_heads, vp]
+    bool unit_norm = false;                                // RMS norms without weights
+    int value_rotary = 0;                                  // values rotate over their first value_rotary elements
+    const float *value_cos = nullptr, *value_sin = nullptr;
     int* status = nullptr;
 };
 int launch_head_prepare(const HeadPrepare& a, int dtype, cudaStream_t stream);
+// Heads that mix their softmax weights, and values that are turned back (head_mix.cuh); see
+// b200_window_attention_args.
+struct HeadMix {
+    const float* weights = nullptr;    // [heads, heads]; NULL: off
+    int rotary = 0, max_pos = 1;
+    const float *cos_t = nullptr, *sin_t = nullptr;
+    const int32_t* positions = nullptr;
+    float score_bound = 0.f;
+    void* scratch = nullptr;           // [tokens, heads, kv_heads, vp] of the dtype
+};
 struct WindowAttention {
     void* out = nullptr;               // [tokens, heads, vp]
     const void* q = nullptr;           // token stride q_st, heads dp apart
@@ -347,12 +370,21 @@ struct WindowAttention {
     int heads = 0, kv_heads = 0, dp = 0, vp = 0, page_size = 1;
     float scale = 1.f;
     AttentionWindow window;
+    HeadMix mix;
     void* workspace = nullptr;
-    int64_t workspace_bytes = 0;       // decode_workspace_bytes
+    int64_t workspace_bytes = 0;       // decode_workspace_bytes, or head_mix_workspace_bytes
     int* status = nullptr;
 };
+// The plain kernel over all key / value heads' values: what every head's weights make of each of them, in a.mix.scratch.
+int launch_plain_all_values(const WindowAttention& a, int dtype, cudaStream_t stream);
 bool window_attention_tc_supported(const WindowAttention& a, int dtype);
 int launch_window_attention(const WindowAttention& a, int dtype, cudaStream_t stream);
+// Mixing heads (talking_heads.cu; the decode kernel is attention_decode.cu's).
+bool talking_heads_tc_supported(const WindowAttention& a, int dtype);
+int launch_talking_heads(const WindowAttention& a, int dtype, cudaStream_t stream);
+bool talking_decode_supported(int heads, int kv_heads);
+int64_t head_mix_workspace_bytes(int max_batch, int heads, int kv_heads);
+int launch_talking_decode(const WindowAttention& a, cudaStream_t stream);
 // Recurrences with one decay per head (recurrence.cu); see b200_recurrence.
 using Recurrence = b200_recurrence_args;
 // Bytes of a step's scratch arrays.
@@ -362,6 +394,7 @@ struct RecurrenceScratch {
 RecurrenceScratch recurrence_scratch(int rule, int max_tokens, int max_batch, int heads, int kv_heads, int padded_dim,
                                      int padded_value_dim, int dtype);
 bool recurrence_supported(int padded_value_dim, int padded_dim, int taps);
+int64_t recurrence_memory_floats(int padded_dim, int padded_value_dim);   // per head
 int launch_recurrence(const Recurrence& a, int dtype, cudaStream_t stream);
 // Gated linear attention (linear_attention.cu): the recurrence, its norm and its gate; see
 // b200_linear_attention.

@@ -4,7 +4,7 @@
 //
 // Per layer, on T tokens (fp32 residual stream r, everything else in the stack's dtype):
 //     x = norm(r += previous block)       the norm on the input: one kernel, residual.cu
-//     x = r += norm(previous block)       or on the output of a block, or both; one kernel as well
+//     x = r += norm(previous block)       or on the output of a block, or both; one kernel as well (RMS or layer norms)
 //     y = mixer(x)
 //     x = ... once more
 //     y = feed-forward(x)
@@ -15,11 +15,12 @@
 //                      keys and values; y = o W_o.  A part of the key may turn with the position instead of being
 //                      normalised; a layer may read the pool of another one
 //   window attention:  [q | k | v | gate] = x W in one GEMM; norms, rotation, value mixing and the K/V store in
-//                      one kernel; attention and its gate in the next (window_attention.cu); y = o W_o
+//                      one kernel; attention and its gate in the next (window_attention.cu); y = o W_o.  Heads may mix
+//                      their weights (talking_heads.cu), values turn with the position, a layer read the pools of another
 //   linear attention:  [q | k | v | gate | low-rank decay] = x W in one GEMM; recurrence, norm and gate
 //                      (linear_attention.cu); y = o W_o
-//   state space, delta rule:  [gate | v | k | q | steps] = x W in one GEMM; convolution, recurrence, norm and gate
-//                      (recurrence.cu); y = o W_o
+//   state space, delta rule, lightning, matrix memory:  [gate | v | k | q | steps] = x W in one GEMM; convolution,
+//                      recurrence, norm and gate (recurrence.cu); y = o W_o
 //   two of the last kinds (window attention, recurrences) side by side: one GEMM makes both rows; one output
 //                      projection over both results adds them up, or each has its own and they meet, normalised, in
 //                      the residual kernel
@@ -50,13 +51,21 @@ int pad_head_dim(int n) { return n <= 128 ? 128 : pad_to(n, 64); }
 int pad_latent(int n) { return pad_to(n, 128); }
 int latent_rope_at(int kv_rank) { return pad_to(kv_rank, 8); }   // where the rotated part of a latent row starts
 int latent_width(int kv_rank, int rope_dim) { return pad_latent(rope_dim > 0 ? latent_rope_at(kv_rank) + rope_dim : kv_rank); }
-bool is_recurrence(int mixer) { return mixer == B200_MIXER_STATE_SPACE || mixer == B200_MIXER_DELTA_RULE; }
+bool is_recurrence(int mixer) {
+    return mixer == B200_MIXER_STATE_SPACE || mixer == B200_MIXER_DELTA_RULE || mixer == B200_MIXER_LIGHTNING ||
+           mixer == B200_MIXER_MATRIX_MEMORY;
+}
+int rule_of(int mixer) {
+    return mixer == B200_MIXER_DELTA_RULE ? B200_RULE_DELTA : mixer == B200_MIXER_LIGHTNING ? B200_RULE_LIGHTNING
+           : mixer == B200_MIXER_MATRIX_MEMORY ? B200_RULE_MATRIX_MEMORY : B200_RULE_STATE_SPACE;
+}
 }  // namespace
 
 struct StackLayer {
     b200_layer_config c;
     int qp = 0, rp = 0, op = 0, dp = 0, vp = 0, ip = 0;   // padded sizes
     void *norm1_out = nullptr, *norm2_out = nullptr;       // of what the blocks return, where both sides have one
+    void *norm1_bias = nullptr, *norm2_bias = nullptr, *norm1_out_bias = nullptr, *norm2_out_bias = nullptr;   // layer norms
     void *norm1 = nullptr, *norm2 = nullptr, *down_qkv = nullptr, *q_norm = nullptr, *kv_norm = nullptr, *uq = nullptr,
          *uk = nullptr, *uk_absorb = nullptr, *uv = nullptr, *o = nullptr, *up = nullptr, *down = nullptr;
     // the projection that a mixer's (or both mixers') rows come from, and this mixer's columns in them
@@ -69,6 +78,7 @@ struct StackLayer {
     // window attention
     void *q_head_norm = nullptr, *k_head_norm = nullptr, *k_cache = nullptr, *v_cache = nullptr;
     float *value_mix = nullptr, *cos_t = nullptr, *sin_t = nullptr, *sinks = nullptr;
+    float *value_cos = nullptr, *value_sin = nullptr, *head_mix = nullptr;
     int mix = HeadPrepare::kPlain;
     // linear attention
     void *decay_up = nullptr, *head_norm = nullptr;
@@ -77,8 +87,10 @@ struct StackLayer {
     // recurrences
     float *conv = nullptr, *conv_bias = nullptr, *decay_log = nullptr, *step_bias = nullptr, *skip = nullptr;
     void* conv_state = nullptr;
+    float* memory = nullptr;
     // scored experts
     void *router = nullptr, *shared_up = nullptr, *shared_down = nullptr;
+    float* correction = nullptr;
     int isp = 0;
     int32_t* table = nullptr;
     void* cache = nullptr;
@@ -97,8 +109,9 @@ struct LayerStack {
     int esz = 2;            // bytes per element
     int hp = 0, vocab_p = 0;
     float norm_offset = 0.f, logit_scale = 1.f;
-    bool norm_input = true, norm_output = false;
-    void *embed = nullptr, *head = nullptr, *final_norm = nullptr;
+    bool norm_input = true, norm_output = false, layer_norm = false;
+    float embed_scale = 1.f;
+    void *embed = nullptr, *head = nullptr, *final_norm = nullptr, *final_norm_bias = nullptr;
     float* residual = nullptr;
     void *x = nullptr, *joint = nullptr, *cq = nullptr, *q = nullptr, *attn = nullptr, *y = nullptr, *h = nullptr,
          *xp = nullptr, *ye = nullptr;
@@ -121,7 +134,7 @@ struct LayerStack {
     void *qc = nullptr, *ac = nullptr;
     int max_extend = 0;        // longest extension of the current step
     // window attention
-    void* first_values = nullptr;
+    void *first_values = nullptr, *mixed_heads = nullptr;
     // recurrences
     void *mixed = nullptr, *chunks = nullptr;
     float *steps = nullptr, *units = nullptr;
@@ -169,11 +182,13 @@ __global__ void compact_rows_kernel(int32_t* __restrict__ row, int32_t* __restri
 // A rotation whose frequencies may be stretched.
 bool rope_ok(const b200_layer_config& c, int widest) {
     return c.rotary_dim >= 0 && c.rotary_dim % 2 == 0 && c.rotary_dim <= widest && (c.rotary_dim == 0 || c.rope_base > 0.0) &&
-           (c.rope_factor == 0.0 || (c.rope_factor > 0.0 && c.rope_low > 0.0 && c.rope_high > c.rope_low && c.rope_original > 0.0));
+           (c.rope_factor == 0.0 || (c.rope_factor > 0.0 && c.rope_original == 0.0) ||
+            (c.rope_factor > 0.0 && c.rope_low > 0.0 && c.rope_high > c.rope_low && c.rope_original > 0.0));
 }
 bool same_rope(const b200_layer_config& a, const b200_layer_config& b) {
     if (a.rotary_dim != b.rotary_dim || a.rope_base != b.rope_base || a.rope_factor != b.rope_factor) return false;
-    return a.rope_factor == 0.0 || (a.rope_low == b.rope_low && a.rope_high == b.rope_high && a.rope_original == b.rope_original);
+    if (a.rope_factor == 0.0 || a.rope_original != b.rope_original) return a.rope_factor == 0.0;
+    return a.rope_original == 0.0 || (a.rope_low == b.rope_low && a.rope_high == b.rope_high);
 }
 
 int check_mixer(const b200_layer_config& c, int l) {
@@ -189,14 +204,22 @@ int check_mixer(const b200_layer_config& c, int l) {
         B200_CHECK_ARG(c.gate >= B200_GATE_NONE && c.gate <= B200_GATE_HEAD, "layer %d: unknown gate", l);
         B200_CHECK_ARG(rope_ok(c, c.head_dim), "layer %d: bad rotation", l);
         B200_CHECK_ARG(c.value_dim <= 1024 && c.head_dim <= 2048, "layer %d: heads are too wide", l);
+        B200_CHECK_ARG(c.head_norm >= B200_HEAD_NORM_NONE && c.head_norm <= B200_HEAD_NORM_UNIT, "layer %d: unknown head norm", l);
+        B200_CHECK_ARG(!(c.head_mix || c.value_rotary) || (!c.sink && c.heads <= 128), "layer %d: mixing heads take no sinks, and at most 128 heads", l);
+        B200_CHECK_ARG(!c.value_rotary || (c.value_dim % 2 == 0 && c.rope_base > 0.0 && !c.value_mix),
+                       "layer %d: bad value rotation", l);
+        B200_CHECK_ARG(c.kv_from < 0 || (!c.value_mix && !c.qkv_bias), "layer %d: no projections of its own to mix or bias", l);
     } else if (c.mixer == B200_MIXER_LINEAR_ATTENTION) {
         B200_CHECK_ARG(c.decay_rank > 0 && c.decay_tau > 0.f, "layer %d: bad decay", l);
         B200_CHECK_ARG(linear_attention_supported(pad_width(c.value_dim), pad_width(c.head_dim)),
                        "layer %d: heads are too wide", l);
     } else if (is_recurrence(c.mixer)) {
         B200_CHECK_ARG(c.kv_heads > 0 && c.heads % c.kv_heads == 0, "layer %d: %d heads over %d key heads", l, c.heads, c.kv_heads);
-        B200_CHECK_ARG(recurrence_supported(pad_width(c.value_dim), pad_width(c.head_dim), c.conv_taps),
+        const bool conv = c.mixer == B200_MIXER_STATE_SPACE || c.mixer == B200_MIXER_DELTA_RULE;
+        B200_CHECK_ARG(recurrence_supported(pad_width(c.value_dim), pad_width(c.head_dim), conv ? c.conv_taps : 1),
                        "layer %d: heads or convolution too wide", l);
+        B200_CHECK_ARG(conv || c.kv_heads == c.heads, "layer %d: every head has its own key head here", l);
+        B200_CHECK_ARG(c.mixer != B200_MIXER_MATRIX_MEMORY || c.gate_cap > 0.f, "layer %d: bad gate cap", l);
         B200_CHECK_ARG(c.mixer == B200_MIXER_DELTA_RULE || (c.norm_groups > 0 && c.heads * c.value_dim % c.norm_groups == 0),
                        "layer %d: bad norm groups", l);
     } else {
@@ -211,35 +234,39 @@ int check_layer(const b200_layer_config& c, int l) {
     if (c.mlp == B200_MLP_NONE) return B200_OK;
     B200_CHECK_ARG(c.intermediate > 0, "layer %d: feed-forward size must be positive", l);
     B200_CHECK_ARG(c.epilogue > B200_EPILOGUE_NONE && c.epilogue <= B200_EPILOGUE_CLAMPED_SWIGLU, "layer %d: unknown activation", l);
+    const int outputs = c.num_experts + (c.mlp == B200_MLP_SCORED_MOE ? c.identity_experts : 0);
     if (c.mlp != B200_MLP_DENSE)
-        B200_CHECK_ARG(c.num_experts > 0 && c.num_experts <= kMaxTableExperts && c.experts_per_tok > 0 &&
-                           c.experts_per_tok <= c.num_experts,
-                       "layer %d: %d of %d experts (at most %d)", l, c.experts_per_tok, c.num_experts, kMaxTableExperts);
-    if (c.mlp == B200_MLP_SCORED_MOE)
-        B200_CHECK_ARG(c.router_groups > 0 && c.num_experts % c.router_groups == 0 && c.router_keep > 0 &&
+        B200_CHECK_ARG(c.num_experts > 0 && outputs >= c.num_experts && outputs <= kMaxTableExperts && c.experts_per_tok > 0 &&
+                           c.experts_per_tok <= outputs,
+                       "layer %d: %d of %d experts (at most %d)", l, c.experts_per_tok, outputs, kMaxTableExperts);
+    if (c.mlp == B200_MLP_SCORED_MOE) {
+        B200_CHECK_ARG(c.router_groups > 0 && outputs % c.router_groups == 0 && c.router_keep > 0 &&
                            c.router_keep <= c.router_groups &&
-                           c.experts_per_tok <= c.num_experts / c.router_groups * c.router_keep && c.shared_intermediate >= 0,
+                           c.experts_per_tok <= outputs / c.router_groups * c.router_keep && c.shared_intermediate >= 0,
                        "layer %d: bad expert groups", l);
+        B200_CHECK_ARG(c.score == B200_SCORE_SOFTMAX || (c.score == B200_SCORE_SIGMOID && c.identity_experts == 0),
+                       "layer %d: identity experts come with softmax scores", l);
+        B200_CHECK_ARG(c.identity_experts == 0 || c.shared_intermediate == 0, "layer %d: identity experts beside a shared one", l);
+    }
     return B200_OK;
 }
 
 // Sizes of the activation buffers: the widest of any layer, in elements per token (workspaces: bytes).
 struct Widths {
     int64_t joint = 0, cq = 0, q = 0, attn = 0, h = 0, pairs = 0, latent = 0, xk = 0, xv = 0, xc = 0, ws = 0, first = 0,
-            experts = 0, router = 0, top = 0, shared = 0, mixed = 0, steps = 0, units = 0, chunks = 0;
+            experts = 0, router = 0, top = 0, shared = 0, mixed_heads = 0, mixed = 0, steps = 0, units = 0, chunks = 0;
     bool normed_pair = false;
     bool scored = false, any_expand = false;
     static void widest(int64_t& a, int64_t b) { if (b > a) a = b; }
 };
 
 // cos / sin of position * frequency, computed in double on the host; layers with the same rotation share a table.
-int rope_table(b200_engine* e, StackLayer& L) {
+int rope_table(b200_engine* e, const b200_layer_config& c, float*& cos_t, float*& sin_t) {
     LayerStack* S = e->stack;
-    const b200_layer_config& c = L.c;
     for (const LayerStack::RopeTable& t : S->ropes)
         if (same_rope(t.c, c)) {
-            L.cos_t = t.cos_t;
-            L.sin_t = t.sin_t;
+            cos_t = t.cos_t;
+            sin_t = t.sin_t;
             return B200_OK;
         }
     constexpr double kTwoPi = 6.283185307179586476925286766559;
@@ -248,7 +275,9 @@ int rope_table(b200_engine* e, StackLayer& L) {
     std::vector<float> cs(n), sn(n);
     for (int i = 0; i < half; ++i) {
         double f = pow(c.rope_base, -2.0 * i / c.rotary_dim);
-        if (c.rope_factor > 0.0) {
+        if (c.rope_factor > 0.0 && c.rope_original == 0.0) {
+            f /= c.rope_factor;
+        } else if (c.rope_factor > 0.0) {
             const double wave = kTwoPi / f;
             const double s = (c.rope_original / wave - c.rope_low) / (c.rope_high - c.rope_low);
             if (wave > c.rope_original / c.rope_low)
@@ -263,13 +292,13 @@ int rope_table(b200_engine* e, StackLayer& L) {
     }
     void* p = nullptr;
     S_TRY(dev_alloc(e, &p, n * 4, true));
-    L.cos_t = static_cast<float*>(p);
+    cos_t = static_cast<float*>(p);
     S_TRY(dev_alloc(e, &p, n * 4, true));
-    L.sin_t = static_cast<float*>(p);
-    S->ropes.push_back({c, L.cos_t, L.sin_t});
+    sin_t = static_cast<float*>(p);
+    S->ropes.push_back({c, cos_t, sin_t});
     if (n == 0) return B200_OK;
-    B200_CHECK_CUDA(cudaMemcpy(L.cos_t, cs.data(), n * 4, cudaMemcpyHostToDevice));
-    B200_CHECK_CUDA(cudaMemcpy(L.sin_t, sn.data(), n * 4, cudaMemcpyHostToDevice));
+    B200_CHECK_CUDA(cudaMemcpy(cos_t, cs.data(), n * 4, cudaMemcpyHostToDevice));
+    B200_CHECK_CUDA(cudaMemcpy(sin_t, sn.data(), n * 4, cudaMemcpyHostToDevice));
     return B200_OK;
 }
 
@@ -293,7 +322,7 @@ int alloc_latent(b200_engine* e, StackLayer& L, int l, const std::string& sfx, W
     S_TRY(named_bytes(e, &L.down_qkv, "down_qkv" + sfx, (qp + (own ? rp : 0)) * hp * z));
     S_TRY(named_bytes(e, &L.q_norm, "q_latent_norm" + sfx, qp * z));
     if (own) S_TRY(named_bytes(e, &L.kv_norm, "kv_latent_norm" + sfx, rp * z));
-    S_TRY(rope_table(e, L));
+    S_TRY(rope_table(e, c, L.cos_t, L.sin_t));
     S_TRY(named_bytes(e, &L.uq, "uq" + sfx, H * dp * qp * z));
     S_TRY(named_bytes(e, &L.uk_absorb, "uk_absorb" + sfx, H * rp * dp * z));
     S_TRY(named_bytes(e, &L.uv, "uv" + sfx, H * vp * op * z));
@@ -321,8 +350,9 @@ int64_t joint_width(const StackLayer& L) {
     const int64_t H = c.heads, G = c.kv_heads, dp = L.dp, vp = L.vp;
     if (c.mixer == B200_MIXER_LINEAR_ATTENTION) return 2 * H * (dp + vp) + pad_width(c.decay_rank);
     if (c.mixer == B200_MIXER_WINDOW_ATTENTION)
-        return (H + G) * dp + G * vp + (c.gate == B200_GATE_ELEMENT ? H * vp : c.gate == B200_GATE_HEAD ? pad_width(c.heads) : 0);
-    return 2 * H * vp + 2 * G * dp + pad_width(c.mixer == B200_MIXER_DELTA_RULE ? 2 * c.heads : c.heads);
+        return H * dp + (c.kv_from < 0 ? G * (dp + vp) : 0) + (c.gate == B200_GATE_ELEMENT ? H * vp : c.gate == B200_GATE_HEAD ? pad_width(c.heads) : 0);
+    const int steps = c.mixer == B200_MIXER_LIGHTNING ? 0 : c.mixer == B200_MIXER_STATE_SPACE ? 1 : 2;   // per head
+    return 2 * H * vp + 2 * G * dp + pad_width(steps * c.heads);
 }
 
 // (names of a mixer's tensors start with `pre`)
@@ -330,14 +360,37 @@ int alloc_window(b200_engine* e, StackLayer& L, int l, const std::string& pre, c
     LayerStack* S = e->stack;
     const b200_layer_config& c = L.c;
     const int64_t z = S->esz, G = c.kv_heads, dp = L.dp, vp = L.vp;
-    if (c.head_norm) {
+    if (c.head_norm == B200_HEAD_NORM_WEIGHTED) {
         S_TRY(named_bytes(e, &L.q_head_norm, pre + "q_head_norm" + sfx, dp * z));
         S_TRY(named_bytes(e, &L.k_head_norm, pre + "k_head_norm" + sfx, dp * z));
     }
-    S_TRY(named_bytes(e, &L.k_cache, pre + "k_cache" + sfx, e->num_slots * G * dp * z));
-    S_TRY(named_bytes(e, &L.v_cache, pre + "v_cache" + sfx, e->num_slots * G * vp * z));
-    S_TRY(rope_table(e, L));
+    if (c.kv_from < 0) {
+        S_TRY(named_bytes(e, &L.k_cache, pre + "k_cache" + sfx, e->num_slots * G * dp * z));
+        S_TRY(named_bytes(e, &L.v_cache, pre + "v_cache" + sfx, e->num_slots * G * vp * z));
+    } else {
+        B200_CHECK_ARG(pre.empty() && c.kv_from < l && S->layers[c.kv_from].c.mixer == B200_MIXER_WINDOW_ATTENTION &&
+                           S->layers[c.kv_from].c.kv_from < 0, "layer %d: layer %d has no keys and values of its own", l, c.kv_from);
+        const StackLayer& from = S->layers[c.kv_from];
+        B200_CHECK_ARG(from.c.kv_heads == c.kv_heads && from.c.head_dim == c.head_dim && from.c.value_dim == c.value_dim &&
+                           from.c.head_norm == c.head_norm && from.c.value_rotary == c.value_rotary && same_rope(from.c, c),
+                       "layer %d: its keys and values are not those of layer %d", l, c.kv_from);
+        L.k_cache = from.k_cache;
+        L.v_cache = from.v_cache;
+    }
+    S_TRY(rope_table(e, c, L.cos_t, L.sin_t));
     void* p = nullptr;
+    if (c.value_rotary) {
+        b200_layer_config whole = c;
+        whole.rotary_dim = c.value_dim;
+        whole.rope_factor = 0.0;
+        S_TRY(rope_table(e, whole, L.value_cos, L.value_sin));
+    }
+    if (c.head_mix || c.value_rotary) {
+        S_TRY(named_bytes(e, &p, pre + "head_mix" + sfx, static_cast<int64_t>(c.heads) * c.heads * 4));
+        L.head_mix = static_cast<float*>(p);
+        Widths::widest(w.mixed_heads, static_cast<int64_t>(c.heads) * G * vp);
+        if (talking_decode_supported(c.heads, c.kv_heads)) Widths::widest(w.ws, head_mix_workspace_bytes(e->max_batch, c.heads, c.kv_heads));
+    }
     if (c.sink) {
         S_TRY(named_bytes(e, &p, pre + "sinks" + sfx, c.heads * 4ll));
         L.sinks = static_cast<float*>(p);
@@ -380,7 +433,8 @@ int alloc_linear(b200_engine* e, StackLayer& L, const std::string& pre, const st
 int alloc_recurrence(b200_engine* e, StackLayer& L, const std::string& pre, const std::string& sfx, Widths& w) {
     LayerStack* S = e->stack;
     const b200_layer_config& c = L.c;
-    const bool delta = c.mixer == B200_MIXER_DELTA_RULE;
+    const bool delta = c.mixer == B200_MIXER_DELTA_RULE, conv = delta || c.mixer == B200_MIXER_STATE_SPACE,
+               memory = c.mixer == B200_MIXER_MATRIX_MEMORY;
     const int64_t z = S->esz, H = c.heads, dp = L.dp, vp = L.vp, channels = H * vp + 2 * c.kv_heads * dp;
     void* p = nullptr;
     auto floats = [&](float*& to, const char* name, int64_t n) -> int {
@@ -388,15 +442,18 @@ int alloc_recurrence(b200_engine* e, StackLayer& L, const std::string& pre, cons
         to = static_cast<float*>(p);
         return B200_OK;
     };
-    S_TRY(floats(L.conv, "conv", c.conv_taps * channels));
-    S_TRY(floats(L.conv_bias, "conv_bias", channels));
-    S_TRY(floats(L.decay_log, "decay_log", H));
-    S_TRY(floats(L.step_bias, "step_bias", H));
-    if (!delta) S_TRY(floats(L.skip, "skip", H));
+    if (conv) {
+        S_TRY(floats(L.conv, "conv", c.conv_taps * channels));
+        S_TRY(floats(L.conv_bias, "conv_bias", channels));
+        S_TRY(named_bytes(e, &L.conv_state, pre + "conv_state" + sfx, static_cast<int64_t>(e->pt_rows) * c.conv_taps * channels * z));
+    }
+    if (!memory) S_TRY(floats(L.decay_log, "decay_log", H));
+    if (conv || memory) S_TRY(floats(L.step_bias, "step_bias", memory ? 2 * H : H));
+    if (c.mixer == B200_MIXER_STATE_SPACE) S_TRY(floats(L.skip, "skip", H));
     S_TRY(named_bytes(e, &L.head_norm, pre + "head_norm" + sfx, (delta ? vp : H * vp) * z));
     S_TRY(floats(L.state, "state", static_cast<int64_t>(e->pt_rows) * H * dp * vp));
-    S_TRY(named_bytes(e, &L.conv_state, pre + "conv_state" + sfx, static_cast<int64_t>(e->pt_rows) * c.conv_taps * channels * z));
-    const RecurrenceScratch need = recurrence_scratch(delta ? B200_RULE_DELTA : B200_RULE_STATE_SPACE, e->max_tokens, e->max_batch,
+    if (memory) S_TRY(floats(L.memory, "memory", e->pt_rows * H * recurrence_memory_floats(L.dp, L.vp)));
+    const RecurrenceScratch need = recurrence_scratch(rule_of(c.mixer), e->max_tokens, e->max_batch,
                                                       c.heads, c.kv_heads, L.dp, L.vp, S->dtype);
     Widths::widest(w.mixed, need.mixed);
     Widths::widest(w.steps, need.steps);
@@ -463,6 +520,13 @@ int alloc_layer_mixer(b200_engine* e, StackLayer& L, int l, const std::string& s
     return B200_OK;
 }
 
+int norm_of(b200_engine* e, const char* name, const std::string& sfx, void*& weight, void*& bias) {
+    const LayerStack* S = e->stack;
+    const int64_t bytes = static_cast<int64_t>(S->hp) * S->esz;
+    S_TRY(named_bytes(e, &weight, name + sfx, bytes));
+    return S->layer_norm ? named_bytes(e, &bias, std::string(name) + "_bias" + sfx, bytes) : B200_OK;
+}
+
 int alloc_feed_forward(b200_engine* e, StackLayer& L, const std::string& sfx, Widths& w) {
     LayerStack* S = e->stack;
     const b200_layer_config& c = L.c;
@@ -470,8 +534,8 @@ int alloc_feed_forward(b200_engine* e, StackLayer& L, const std::string& sfx, Wi
     L.ip = pad_width(c.intermediate);
     const int64_t n_up = (epilogue_is_gated(c.epilogue) ? 2 : 1) * static_cast<int64_t>(L.ip);
     const int64_t E = c.mlp == B200_MLP_DENSE ? 1 : c.num_experts;
-    S_TRY(named_bytes(e, &L.norm2, "norm2" + sfx, hp * z));
-    if (S->norm_input && S->norm_output) S_TRY(named_bytes(e, &L.norm2_out, "norm2_out" + sfx, hp * z));
+    S_TRY(norm_of(e, "norm2", sfx, L.norm2, L.norm2_bias));
+    if (S->norm_input && S->norm_output) S_TRY(norm_of(e, "norm2_out", sfx, L.norm2_out, L.norm2_out_bias));
     S_TRY(named_bytes(e, &L.up, "mlp_up" + sfx, E * n_up * hp * z));
     S_TRY(named_bytes(e, &L.down, "mlp_down" + sfx, E * hp * L.ip * z));
     if (c.mlp == B200_MLP_DENSE) {
@@ -484,9 +548,14 @@ int alloc_feed_forward(b200_engine* e, StackLayer& L, const std::string& sfx, Wi
     void* p = nullptr;
     if (c.mlp == B200_MLP_SCORED_MOE) {
         w.scored = true;
-        S_TRY(named_bytes(e, &L.router, "router" + sfx, static_cast<int64_t>(pad_width(c.num_experts)) * hp * z));
+        const int outputs = pad_width(c.num_experts + c.identity_experts);
+        S_TRY(named_bytes(e, &L.router, "router" + sfx, outputs * hp * z));
+        if (c.score == B200_SCORE_SOFTMAX) {
+            S_TRY(named_bytes(e, &p, "router_correction" + sfx, (c.num_experts + c.identity_experts) * 4ll));
+            L.correction = static_cast<float*>(p);
+        }
         Widths::widest(w.experts, E);
-        Widths::widest(w.router, pad_width(c.num_experts));
+        Widths::widest(w.router, outputs);
         Widths::widest(w.top, top);
         if (c.shared_intermediate > 0) {
             L.isp = pad_width(c.shared_intermediate);
@@ -523,6 +592,10 @@ int layer_stack_create(b200_engine* e, const b200_stack_config* sc) {
     B200_CHECK_ARG(sc->num_beside >= 0 && (sc->num_beside == 0 || sc->beside), "layer stack: no mixers to run beside others");
     S->norm_input = sc->norm_output != B200_NORM_OUTPUT;
     S->norm_output = sc->norm_output != B200_NORM_INPUT;
+    B200_CHECK_ARG(sc->norm_kind == B200_NORM_RMS || sc->norm_kind == B200_NORM_LAYER, "layer stack: unknown norm");
+    S->layer_norm = sc->norm_kind == B200_NORM_LAYER;
+    B200_CHECK_ARG(!S->layer_norm || (sc->norm_offset == 0.f && sc->logit_scale == 1.f), "layer stack: layer norms take no offset or scale");
+    S->embed_scale = sc->embed_scale == 0.f ? 1.f : sc->embed_scale;
     S->hp = pad_width(e->m.hidden_size);
     S->vocab_p = pad_width(e->m.vocab_size);
     if (const char* v = getenv("B200_LATENT_EXPAND_MIN")) S->expand_min = atoi(v);
@@ -534,7 +607,7 @@ int layer_stack_create(b200_engine* e, const b200_stack_config* sc) {
     } else {
         S_TRY(named_bytes(e, &S->head, "lm_head", S->vocab_p * hp * z));
     }
-    S_TRY(named_bytes(e, &S->final_norm, "final_norm", hp * z));
+    S_TRY(norm_of(e, "final_norm", "", S->final_norm, S->final_norm_bias));
 
     Widths w;
     S->latent_rows = e->max_batch > 1024 ? e->max_batch : 1024;
@@ -547,11 +620,14 @@ int layer_stack_create(b200_engine* e, const b200_stack_config* sc) {
         L.c = sc->layers[l];
         const b200_layer_config& c = L.c;
         S_TRY(check_layer(c, l));
-        B200_CHECK_ARG(!(S->norm_output && c.mlp == B200_MLP_TABLE_MOE),
-                       "layer %d: experts by token id take the norm on their input", l);
+        B200_CHECK_ARG(!((S->norm_output || S->layer_norm) && c.mlp == B200_MLP_TABLE_MOE),
+                       "layer %d: experts by token id take the RMS norm on their input", l);
+        B200_CHECK_ARG(c.mlp != B200_MLP_SCORED_MOE || c.identity_experts == 0 || S->layer_norm,
+                       "layer %d: identity experts come with layer norms", l);
+        B200_CHECK_ARG(!S->layer_norm || c.beside < 0 || c.join == B200_JOIN_SUM, "layer %d: layer norms do not join mixers", l);
         const std::string sfx = "." + std::to_string(l);
-        S_TRY(named_bytes(e, &L.norm1, "norm1" + sfx, hp * z));
-        if (S->norm_input && S->norm_output) S_TRY(named_bytes(e, &L.norm1_out, "norm1_out" + sfx, hp * z));
+        S_TRY(norm_of(e, "norm1", sfx, L.norm1, L.norm1_bias));
+        if (S->norm_input && S->norm_output) S_TRY(norm_of(e, "norm1_out", sfx, L.norm1_out, L.norm1_out_bias));
         B200_CHECK_ARG(c.beside < sc->num_beside, "layer %d: no mixer %d to run beside", l, c.beside);
         if (c.beside >= 0) L.beside = &S->besides[c.beside];
         S_TRY(alloc_layer_mixer(e, L, l, sfx, w));
@@ -581,7 +657,7 @@ int layer_stack_create(b200_engine* e, const b200_stack_config* sc) {
     S->compact_row = static_cast<int32_t*>(p);
     S_TRY(dev_alloc(e, &p, Tm * 4, true));
     S->compact_len = static_cast<int32_t*>(p);
-    if (w.mixed > 0) {
+    if (w.steps > 0) {
         S_TRY(dev_alloc(e, &S->mixed, w.mixed, true));
         S_TRY(dev_alloc(e, &p, w.steps, true));
         S->steps = static_cast<float*>(p);
@@ -590,6 +666,7 @@ int layer_stack_create(b200_engine* e, const b200_stack_config* sc) {
         S_TRY(dev_alloc(e, &S->chunks, w.chunks, true));
     }
     if (w.normed_pair) S_TRY(dev_alloc(e, &S->y2, Tm * hp * z, true));
+    if (w.mixed_heads > 0) S_TRY(dev_alloc(e, &S->mixed_heads, Tm * w.mixed_heads * z, true));
     if (w.first > 0) S_TRY(dev_alloc(e, &S->first_values, Tm * w.first * z, true));
     if (w.scored) {
         S_TRY(dev_alloc(e, &p, Tm * w.router * 4, true));
@@ -823,10 +900,14 @@ int window_prepare(b200_engine* e, const StackLayer& L, int T) {
     a.ld = L.joint_ld;
     a.tokens = T;
     a.heads = c.heads;
-    a.kv_heads = c.kv_heads;
+    a.kv_heads = c.kv_from < 0 ? c.kv_heads : 0;   // (another layer has prepared its keys and values)
     a.dim = c.head_dim;
     a.dp = L.dp;
     a.vp = L.vp;
+    a.unit_norm = c.head_norm == B200_HEAD_NORM_UNIT;
+    a.value_rotary = c.value_rotary ? c.value_dim : 0;
+    a.value_cos = L.value_cos;
+    a.value_sin = L.value_sin;
     a.q_weight = L.q_head_norm;
     a.k_weight = L.k_head_norm;
     a.eps = e->m.rms_norm_eps;
@@ -878,13 +959,24 @@ int window_attend(b200_engine* e, const StackLayer& L, int phase, int Bp, int T)
     a.window.chunk = c.chunk;
     a.window.sinks = L.sinks;
     if (c.gate != B200_GATE_NONE) {
-        a.window.gate = joint_of(S, L) +
-                        (static_cast<int64_t>(c.heads + c.kv_heads) * L.dp + static_cast<int64_t>(c.kv_heads) * L.vp) * S->esz;
+        const int64_t own = c.kv_from < 0 ? static_cast<int64_t>(c.kv_heads) * (L.dp + L.vp) : 0;
+        a.window.gate = joint_of(S, L) + (static_cast<int64_t>(c.heads) * L.dp + own) * S->esz;
         a.window.gate_st = a.q_st;
         a.window.gate_per_head = c.gate == B200_GATE_HEAD;
     }
     a.window.out_scale = c.out_scale;
     a.window.out_st = L.out_ld;
+    if (L.head_mix != nullptr) {
+        a.mix.weights = L.head_mix;
+        a.mix.rotary = c.value_rotary ? c.value_dim : 0;
+        a.mix.max_pos = e->pt_cols;
+        a.mix.cos_t = L.value_cos;
+        a.mix.sin_t = L.value_sin;
+        a.mix.positions = e->positions;
+        // vectors of root mean square 1, a little longer for having been rounded
+        a.mix.score_bound = c.head_norm == B200_HEAD_NORM_UNIT ? 1.02f * static_cast<float>(c.head_dim) : 0.f;
+        a.mix.scratch = S->mixed_heads;
+    }
     a.workspace = S->ws;
     a.workspace_bytes = S->ws_bytes;
     a.status = e->status;
@@ -929,7 +1021,9 @@ int recurrence_mixer(b200_engine* e, const StackLayer& L, int phase, int Bp, int
     a.out_ld = L.out_ld;
     a.joint = joint_of(S, L);
     a.joint_ld = L.joint_ld;
-    a.rule = c.mixer == B200_MIXER_DELTA_RULE ? B200_RULE_DELTA : B200_RULE_STATE_SPACE;
+    a.rule = rule_of(c.mixer);
+    a.gate_cap = c.gate_cap;
+    a.memory = L.memory;
     a.tokens = T;
     a.batch = Bp;
     a.max_extend = S->max_extend;
@@ -1019,7 +1113,7 @@ int feed_forward(b200_engine* e, const StackLayer& L, int T) {
         S_TRY(project(e, S->h, S->x, L.up, T, gated * L.ip, hp, c.epilogue, c.act_limit));
         return project(e, S->y, S->h, L.down, T, hp, L.ip, B200_EPILOGUE_NONE);
     }
-    const int ep = pad_width(c.num_experts);
+    const int ep = pad_width(c.num_experts + c.identity_experts);
     S_TRY(project(e, S->router_logits, S->x, L.router, T, ep, hp,
                   S->dtype == B200_DTYPE_F32 ? B200_EPILOGUE_NONE : B200_EPILOGUE_F32));
     ScoreRoute r;
@@ -1031,6 +1125,9 @@ int feed_forward(b200_engine* e, const StackLayer& L, int T) {
     r.groups = c.router_groups;
     r.keep = c.router_keep;
     r.scale = c.router_scale;
+    r.score = c.score;
+    r.identity = c.identity_experts;
+    r.correction = L.correction;
     r.ids = S->route_ids;
     r.weights = S->route_weights;
     r.counts = S->route_counts;
@@ -1052,6 +1149,7 @@ void take_block(LayerStack* S, const StackLayer* experts, const StackLayer* pair
     rn.src_weights = experts ? S->route_weights : nullptr;
     rn.src_top = experts ? experts->c.experts_per_tok : 1;
     rn.src_count = static_cast<int64_t>(T) * rn.src_top;
+    rn.self = S->x;    // of identity experts
     rn.src2 = pair ? S->y2 : experts && experts->isp > 0 ? S->shared_y : nullptr;
     rn.pair_weight = pair ? pair->side_norm : nullptr;
     rn.pair_weight2 = pair ? pair->beside->side_norm : nullptr;
@@ -1094,6 +1192,8 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
     post.src = S->embed;
     post.src_rows = e->input_ids;
     post.src_count = e->m.vocab_size;
+    post.layer = S->layer_norm;
+    post.src_scale = rn.src_scale = S->embed_scale;
     post.init = true;
     post.weight_offset = S->norm_offset;
     post.tokens = T;
@@ -1102,7 +1202,7 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
     post.eps = e->m.rms_norm_eps;
     const StackLayer* scored = nullptr;   // the last block was this layer's scored experts
     const StackLayer* pair = nullptr;     // the last block was this layer's two mixers, normalised each
-    const void* own_norm = nullptr;       // norm_output: the norm of the last block's output
+    const void *own_norm = nullptr, *own_bias = nullptr;   // norm_output: the norm of the last block's output
     auto add_plain = [&]() {
         rn.src = S->y;
         rn.src_rows = nullptr;
@@ -1113,11 +1213,11 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
         scored = pair = nullptr;
     };
     // Adds the last block and leaves what the next one reads: normalised with `weight`, or as it is.
-    auto advance = [&](const void* weight, void* out, const int32_t* rows, int top, float out_scale,
+    auto advance = [&](const void* weight, const void* bias, void* out, const int32_t* rows, int top, float out_scale,
                        const StackLayer* next_scored) -> int {
         post.clear = next_scored ? S->route_counts : nullptr;
         post.clear_count = next_scored ? 2 * next_scored->c.num_experts : 0;
-        if (!S->norm_output && scored == nullptr && pair == nullptr && next_scored == nullptr) {
+        if (!S->norm_output && !S->layer_norm && scored == nullptr && pair == nullptr && next_scored == nullptr) {
             rn.weight = weight;
             rn.out = out;
             rn.out_rows = rows;
@@ -1127,7 +1227,9 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
         }
         if (!rn.init) take_block(S, scored, pair, T, post);
         post.add_weight = own_norm;
+        post.add_bias = own_bias;
         post.out_weight = weight;
+        post.out_bias = bias;
         post.out_scale = out_scale;
         return launch_residual_post_norm(post, S->dtype, e->status, s);
     };
@@ -1143,17 +1245,20 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
         const b200_layer_config& c = L.c;
         // The first norm is launched as an ordinary dependent of what prepares the step, so that every
         // kernel after it finds positions, slots and lengths complete even ahead of its own wait.
-        S_TRY(advance(S->norm_input ? L.norm1 : nullptr, S->x, nullptr, 1, 1.f, nullptr));
+        S_TRY(advance(S->norm_input ? L.norm1 : nullptr, L.norm1_bias, S->x, nullptr, 1, 1.f, nullptr));
         if (l == 0) set_pdl_launches(pdl);
         S_TRY(traced(l));
         S_TRY(mix(e, l, phase, Bp, T));
         add_plain();
         if (L.side_norm != nullptr) pair = &L;
-        if (S->norm_output) own_norm = S->norm_input ? L.norm1_out : L.norm1;
+        if (S->norm_output) {
+            own_norm = S->norm_input ? L.norm1_out : L.norm1;
+            own_bias = S->norm_input ? L.norm1_out_bias : L.norm1_bias;
+        }
         if (c.mlp == B200_MLP_NONE) continue;
         if (c.mlp == B200_MLP_TABLE_MOE) {
             const int n_up = (epilogue_is_gated(c.epilogue) ? 2 : 1) * L.ip;
-            S_TRY(advance(L.norm2, S->xp, L.rows, c.experts_per_tok, 1.f, nullptr));
+            S_TRY(advance(L.norm2, nullptr, S->xp, L.rows, c.experts_per_tok, 1.f, nullptr));
             S_TRY(project_experts(e, S->h, S->xp, L.up, L, L.counts, L.offsets, T, n_up, hp, c.epilogue));
             S_TRY(project_experts(e, S->ye, S->h, L.down, L, L.counts, L.offsets, T, hp, L.ip, B200_EPILOGUE_NONE));
             pair = nullptr;
@@ -1165,13 +1270,16 @@ int layer_stack_enqueue(b200_engine* e, int phase, int Bp, int T, bool pdl) {
             rn.init = false;
             continue;
         }
-        S_TRY(advance(S->norm_input ? L.norm2 : nullptr, S->x, nullptr, 1, 1.f, c.mlp == B200_MLP_SCORED_MOE ? &L : nullptr));
+        S_TRY(advance(S->norm_input ? L.norm2 : nullptr, L.norm2_bias, S->x, nullptr, 1, 1.f, c.mlp == B200_MLP_SCORED_MOE ? &L : nullptr));
         S_TRY(feed_forward(e, L, T));
         add_plain();
         if (c.mlp == B200_MLP_SCORED_MOE) scored = &L;
-        if (S->norm_output) own_norm = S->norm_input ? L.norm2_out : L.norm2;
+        if (S->norm_output) {
+            own_norm = S->norm_input ? L.norm2_out : L.norm2;
+            own_bias = S->norm_input ? L.norm2_out_bias : L.norm2_bias;
+        }
     }
-    S_TRY(advance(S->final_norm, S->x, nullptr, 1, S->logit_scale, nullptr));
+    S_TRY(advance(S->final_norm, S->final_norm_bias, S->x, nullptr, 1, S->logit_scale, nullptr));
     return traced(num_layers);
 }
 

@@ -231,7 +231,9 @@ struct ScoreRouteArgs {
     int32_t* ids;            // [tokens, top]
     float* weights;          // [tokens, top]
     int32_t* counts;         // [experts], zero before
-    int smem_floats;         // per warp: scores | group scores | chosen scores
+    int smem_floats;         // per warp: scores | group scores | chosen scores (| softmax scores)
+    int identity;            // outputs behind those of the experts
+    const float* correction;
 };
 
 __device__ __forceinline__ void warp_argmax(float& best, int& at) {
@@ -258,7 +260,10 @@ score_route_kernel(const ScoreRouteArgs a) {
     float* score = s_route + static_cast<int64_t>(warp) * a.smem_floats;
     float* group = score + a.experts;
     float* chosen = group + a.groups;
-    for (int e = lane; e < a.experts; e += 32) score[e] = 1.f / (1.f + expf(-a.logits[t * a.ld + e]));
+    for (int e = lane; e < a.experts; e += 32) {
+        const float s = 1.f / (1.f + expf(-a.logits[t * a.ld + e]));
+        score[e] = s == s ? s : 0.f;   // NaN logits: a token's experts are valid and differ all the same
+    }
     __syncwarp();
     if (a.keep < a.groups) {
         const int size = a.experts / a.groups;
@@ -302,10 +307,6 @@ score_route_kernel(const ScoreRouteArgs a) {
                 at = e;
             }
         warp_argmax(best, at);
-        if (at >= a.experts) {   // NaN logits: a valid expert all the same
-            at = 0;
-            best = 0.f;
-        }
         sum += best;
         if (lane == 0) {
             score[at] = kTaken;
@@ -316,6 +317,83 @@ score_route_kernel(const ScoreRouteArgs a) {
         __syncwarp();
     }
     for (int k = lane; k < a.top; k += 32) a.weights[t * a.top + k] = chosen[k] / (sum + 1e-20f) * a.scale;
+}
+
+// The same with softmax scores over experts and identity experts.  Groups and choice go by score + correction, which may
+// be negative; a group counts for its best.
+__global__ void __launch_bounds__(128)
+softmax_route_kernel(const ScoreRouteArgs a) {
+    extern __shared__ float s_route[];
+    pdl_launch_dependents();
+    pdl_wait_prior();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, outputs = a.experts + a.identity;
+    const int64_t t = static_cast<int64_t>(blockIdx.x) * (blockDim.x >> 5) + warp;
+    if (t >= a.tokens) return;
+    float* choice = s_route + static_cast<int64_t>(warp) * a.smem_floats;
+    float* group = choice + outputs;
+    float* score = group + a.groups;
+    const float* z = a.logits + t * a.ld;
+    float top = -INFINITY, sum = 0.f;
+    for (int e = lane; e < outputs; e += 32) top = fmaxf(top, z[e]);
+    top = warp_max(top);
+    for (int e = lane; e < outputs; e += 32) {
+        score[e] = expf(z[e] - top);
+        sum += score[e];
+    }
+    sum = warp_sum(sum);
+    for (int e = lane; e < outputs; e += 32) {
+        const float s = score[e] / sum, c = s + (a.correction != nullptr ? a.correction[e] : 0.f);
+        score[e] = s == s ? s : 0.f;   // NaN logits: a token's experts are valid and differ all the same
+        choice[e] = c == c ? c : 0.f;
+    }
+    __syncwarp();
+    const int size = outputs / a.groups;
+    // the best of n numbers, lowest index first; n when all of them are out
+    auto best_of = [&](const float* x, int n) {
+        float best = -INFINITY;
+        int at = n;
+        for (int i = lane; i < n; i += 32)
+            if (x[i] > best) {
+                best = x[i];
+                at = i;
+            }
+        warp_argmax(best, at);
+        return at;
+    };
+    if (a.keep < a.groups) {
+        for (int g = lane; g < a.groups; g += 32) {
+            float best = -INFINITY;
+            for (int i = 0; i < size; ++i) best = fmaxf(best, choice[g * size + i]);
+            group[g] = best;
+        }
+        __syncwarp();
+        constexpr float kKept = INFINITY;
+        for (int k = 0; k < a.keep; ++k) {
+            float best = -INFINITY;
+            int at = a.groups;
+            for (int g = lane; g < a.groups; g += 32)
+                if (group[g] != kKept && group[g] > best) {
+                    best = group[g];
+                    at = g;
+                }
+            warp_argmax(best, at);
+            if (lane == 0 && at < a.groups) group[at] = kKept;
+            __syncwarp();
+        }
+        for (int e = lane; e < outputs; e += 32)
+            if (group[e / size] != kKept) choice[e] = -INFINITY;
+        __syncwarp();
+    }
+    for (int k = 0; k < a.top; ++k) {
+        const int at = best_of(choice, outputs);
+        if (lane == 0 && at < outputs) {
+            choice[at] = -INFINITY;
+            a.ids[t * a.top + k] = at;
+            a.weights[t * a.top + k] = score[at] * a.scale;
+            if (at < a.experts) atomicAdd(&a.counts[at], 1);
+        }
+        __syncwarp();
+    }
 }
 
 // A row among its expert's for every choice of a token, and the token's activations copied there.  The first
@@ -331,6 +409,10 @@ score_place_kernel(uint4* __restrict__ xp, const uint4* __restrict__ x, int32_t*
     const int64_t t = blockIdx.x;
     for (int k = warp; k < top; k += warps) {
         const int e = ids[t * top + k];
+        if (e >= experts) {   // an identity expert: the token keeps its row where it is
+            if (lane == 0) s_place[k] = rows[t * top + k] = -1;
+            continue;
+        }
         int before = 0;
         for (int i = lane; i < e; i += 32) before += counts[i];
 #pragma unroll
@@ -360,7 +442,8 @@ score_place_kernel(uint4* __restrict__ xp, const uint4* __restrict__ x, int32_t*
     __syncthreads();
     for (int v = threadIdx.x; v < vec_per_row; v += blockDim.x) {
         const uint4 u = x[t * vec_per_row + v];
-        for (int k = 0; k < top; ++k) xp[static_cast<int64_t>(s_place[k]) * vec_per_row + v] = u;
+        for (int k = 0; k < top; ++k)
+            if (s_place[k] >= 0) xp[static_cast<int64_t>(s_place[k]) * vec_per_row + v] = u;
     }
 }
 
@@ -421,10 +504,14 @@ int launch_score_route(const ScoreRoute& r, cudaStream_t stream) {
     a.ids = r.ids;
     a.weights = r.weights;
     a.counts = r.counts;
-    a.smem_floats = r.experts + r.groups + r.top;
+    a.identity = r.identity;
+    a.correction = r.correction;
+    const bool softmax = r.score == B200_SCORE_SOFTMAX;
+    const int outputs = r.experts + r.identity;
+    a.smem_floats = softmax ? 2 * outputs + r.groups : r.experts + r.groups + r.top;
     // few tokens: one warp per CTA, spread over the SMs
-    const int warps = r.tokens >= 1024 && r.experts <= 1024 ? 4 : 1;
-    B200_CHECK_CUDA(launch_kernel(score_route_kernel, dim3(div_ceil(r.tokens, warps)), dim3(32 * warps),
+    const int warps = r.tokens >= 1024 && outputs <= 1024 ? 4 : 1;
+    B200_CHECK_CUDA(launch_kernel(softmax ? softmax_route_kernel : score_route_kernel, dim3(div_ceil(r.tokens, warps)), dim3(32 * warps),
                                   static_cast<size_t>(warps) * a.smem_floats * 4, stream, dim3(1, 1, 1), a));
     return B200_OK;
 }
@@ -535,11 +622,15 @@ int b200_table_route(int32_t* rows, int32_t* counts, int32_t* offsets, const int
 
 int b200_score_route(int32_t* ids, float* weights, int32_t* rows, int32_t* counts, int32_t* offsets, void* xp,
                      const void* x, int row_bytes, const float* logits, int64_t logits_ld, int tokens, int experts,
-                     int top, int groups, int keep_groups, float scale, b200_stream_t stream) {
-    B200_CHECK_ARG(tokens >= 0 && experts > 0 && experts <= b200::kMaxTableExperts && top > 0 && groups > 0 &&
-                       experts % groups == 0 && keep_groups > 0 && keep_groups <= groups &&
-                       top <= experts / groups * keep_groups, "score_route: bad shape");
-    B200_CHECK_ARG(row_bytes > 0 && row_bytes % 16 == 0 && logits_ld >= experts, "score_route: bad row size");
+                     int top, int groups, int keep_groups, float scale, int score, int identity_experts,
+                     const float* correction, b200_stream_t stream) {
+    const int outputs = experts + identity_experts;
+    B200_CHECK_ARG(tokens >= 0 && experts > 0 && identity_experts >= 0 && outputs <= b200::kMaxTableExperts && top > 0 && groups > 0 &&
+                       outputs % groups == 0 && keep_groups > 0 && keep_groups <= groups &&
+                       top <= outputs / groups * keep_groups, "score_route: bad shape");
+    B200_CHECK_ARG(score == B200_SCORE_SOFTMAX || (score == B200_SCORE_SIGMOID && identity_experts == 0 && !correction),
+                   "score_route: identity experts and corrections come with softmax scores");
+    B200_CHECK_ARG(row_bytes > 0 && row_bytes % 16 == 0 && logits_ld >= outputs, "score_route: bad row size");
     if (tokens == 0) return B200_OK;
     B200_CHECK_ARG(ids && weights && rows && counts && offsets && xp && x && logits, "score_route: NULL tensor");
     cudaStream_t s = static_cast<cudaStream_t>(stream);
@@ -553,6 +644,9 @@ int b200_score_route(int32_t* ids, float* weights, int32_t* rows, int32_t* count
     r.groups = groups;
     r.keep = keep_groups;
     r.scale = scale;
+    r.score = score;
+    r.identity = identity_experts;
+    r.correction = correction;
     r.ids = ids;
     r.weights = weights;
     r.counts = counts;

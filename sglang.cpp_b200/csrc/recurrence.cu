@@ -1,7 +1,12 @@
-// Recurrences with one decay per head and step, behind a short causal convolution: a scalar-decay state space
+// Recurrences with one decay per head and step.  Behind a short causal convolution, a scalar-decay state space
 //     S <- g S + dt k v^T,                    o = S^T q + skip v
 // and the gated delta rule (k and q unit vectors)
 //     S <- g S,  u = beta (v - S^T k),  S <- S + k u^T,    o = S^T q.
+// Without one, lightning attention, whose decay is constant (k, q, v behind a silu)
+//     S <- g S + k v^T,                       o = S^T q
+// and the matrix memory, whose exponential gates (logarithms i and f) refer to a running maximum
+//     m' = max(f + m, i),  S <- exp(f + m - m') S + exp(i - m') k v^T,  n likewise with k alone
+//     o = S^T q / (max(|n . q|, exp(-m')) + 1e-6).
 // The matrix state is fp32 and lives in a slot per page-table row, as do the convolution's last inputs (a ring: the
 // input of position p is at p mod taps, so that a step writes a place that nobody reads in the same step).
 //
@@ -16,6 +21,10 @@
 //         U = (I + A)^-1 diag(beta) (V - diag(G) K S)     (state space: U = diag(dt) V)
 //         O = diag(G) Q S + P U
 //         S <- G_n S + K^T diag(exp(B_n - B_s)) U
+//     (lightning: dt = 1).  The matrix memory, with m the maximum before the chunk and c_t = max_{s <= t} (i_s - B_s):
+//         P_ts = exp(i_s - B_s - c_t) q_t . k_s  (s <= t),           m_t = B_t + max(m, c_t)
+//         O = diag(exp(m - max(m, c))) Q S + diag(exp(c - max(m, c))) P V,   the same for n with 1 in the place of V
+//         S <- exp(m - max(m, c_n)) S + K^T diag(exp(i_s - B_s - max(m, c_n))) V
 //     No exponent is positive, however steep the decay.  P and the inverse do not depend on the state: prepare_kernel
 //     makes them for all chunks at once (the inverse by substitution in fp32) and stores them in the order in which
 //     chunk_kernel's threads hold MMA operands.  chunk_kernel walks a request's chunks, one CTA per head and 64
@@ -52,18 +61,53 @@ template <typename T>
 __device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
 template <>
 __device__ __forceinline__ float silu<__nv_bfloat16>(float x) { return x * sigmoid_f(x); }
+template <typename T>
+__device__ __forceinline__ float sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
+template <>
+__device__ __forceinline__ float sigmoid<__nv_bfloat16>(float x) { return sigmoid_f(x); }
 
 constexpr float kLog2e = 1.4426950408889634f;
-constexpr float kUnitEps = 1e-6f;
+constexpr float kUnitEps = 1e-6f, kMemoryEps = 1e-6f;
+constexpr int kStepThreads = 512;
+constexpr int kMaxAhead = 8;   // state rows per thread of the step kernel, in registers
 constexpr int kMaxTaps = 16;
-constexpr int kStateSpace = B200_RULE_STATE_SPACE, kDelta = B200_RULE_DELTA;
+constexpr int kStateSpace = B200_RULE_STATE_SPACE, kDelta = B200_RULE_DELTA, kLightning = B200_RULE_LIGHTNING,
+              kMemory = B200_RULE_MATRIX_MEMORY;
+constexpr bool has_convolution(int rule) { return rule == kStateSpace || rule == kDelta; }
 
 // Channel c of [v | k | q] is column values() + c of a row of the joint projection.
 __device__ __forceinline__ int64_t values(const Recurrence& a) { return static_cast<int64_t>(a.heads) * a.padded_value_dim; }
 __device__ __forceinline__ int64_t channels(const Recurrence& a) { return values(a) + 2ll * a.kv_heads * a.padded_dim; }
 
-// log2 of a step's decay and the weight of what it writes, from a head's columns of the joint projection.
-__device__ __forceinline__ float2 make_step(int rule, float za, float zb, float step_bias, float decay_log) {
+// What the recurrence reads channels from: what mix_kernel has left, or (matrix memory) the projection itself.
+template <typename T>
+__device__ __forceinline__ const T* mixed_rows(const Recurrence& a) {
+    return a.rule == kMemory ? static_cast<const T*>(a.joint) + values(a) : static_cast<const T*>(a.mixed);
+}
+__device__ __forceinline__ int64_t mixed_ld(const Recurrence& a) { return a.rule == kMemory ? a.joint_ld : channels(a); }
+
+// The matrix memory keeps n and m once per this many value columns: what one CTA writes no other one reads.
+__host__ __device__ inline int memory_columns(int padded_dim) {
+    const int most = kMaxAhead * kStepThreads / padded_dim;   // groups of four columns that a step CTA has room for
+    int cols = 64;
+    while (cols > 4 && cols > 4 * most) cols /= 2;
+    return cols;
+}
+__host__ __device__ inline int memory_copies(int padded_dim, int padded_value_dim) { return padded_value_dim / memory_columns(padded_dim); }
+__host__ __device__ inline int memory_width(int padded_dim) { return padded_dim + 4; }   // n, then m in units of log 2
+__device__ __forceinline__ float* memory_of(const Recurrence& a, int64_t row, int h, int col0) {
+    const int copy = col0 / memory_columns(a.padded_dim);
+    return a.memory + ((row * a.heads + h) * memory_copies(a.padded_dim, a.padded_value_dim) + copy) * memory_width(a.padded_dim);
+}
+
+// log2 of a step's decay and the weight of what it writes (matrix memory: log2 of that), from a head's columns of the
+// joint projection.
+__device__ __forceinline__ float2 make_step(int rule, float za, float zb, float step_bias, float decay_log, float cap) {
+    if (rule == kLightning) return make_float2(decay_log * kLog2e, 1.f);
+    if (rule == kMemory) {
+        const float f = cap * tanhf((zb + decay_log) / cap);
+        return make_float2((fminf(f, 0.f) - log1pf(expf(-fabsf(f)))) * kLog2e, cap * tanhf((za + step_bias) / cap) * kLog2e);
+    }
     const float x = za + step_bias, dt = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
     return make_float2(-expf(decay_log) * dt * kLog2e, rule == kStateSpace ? dt : 1.f / (1.f + expf(-zb)));
 }
@@ -118,8 +162,11 @@ mix_kernel(const Recurrence a, int v_blocks, int heads_per_block) {
         for (int i = threadIdx.x; i < n * a.heads; i += kMixThreads) {
             const int t = t0 + i / a.heads, h = i % a.heads;
             const T* tail = joint + t * a.joint_ld + values(a) + channels(a) + h;
+            const bool pair = a.rule == kDelta || a.rule == kMemory;
             reinterpret_cast<float2*>(a.steps)[static_cast<int64_t>(begin + t) * a.heads + h] =
-                make_step(a.rule, to_f32(tail[0]), a.rule == kDelta ? to_f32(tail[a.heads]) : 0.f, a.step_bias[h], a.decay_log[h]);
+                make_step(a.rule, a.rule == kLightning ? 0.f : to_f32(tail[0]), pair ? to_f32(tail[a.heads]) : 0.f,
+                          a.rule == kLightning ? 0.f : a.step_bias[h], a.rule == kMemory ? a.step_bias[a.heads + h] : a.decay_log[h],
+                          a.gate_cap);
         }
         return;
     }
@@ -156,7 +203,8 @@ mix_kernel(const Recurrence a, int v_blocks, int heads_per_block) {
         if (TAPS > 0) {
 #pragma unroll
             for (int i = 0; i < kWindow; ++i) {
-                w[i] = load8(a.conv + i * nc + c);
+                if (a.conv != nullptr) w[i] = load8(a.conv + i * nc + c);
+                else for (int j = 0; j < 8; ++j) w[i].v[j] = 1.f;
                 if (i + 1 < kWindow) x[i + 1] = input(t0 - (kWindow - 1) + i);
             }
         }
@@ -206,7 +254,7 @@ mix_kernel(const Recurrence a, int v_blocks, int heads_per_block) {
             }
         }
         // (a request's first block is the only one that reads the ring)
-        if (blockIdx.x == 0)
+        if (blockIdx.x == 0 && a.conv != nullptr)
             for (int r = max(0, ext - (taps - 1)); r < ext; ++r) store8(ring + (cached + r) % taps * nc, load8(in + r * a.joint_ld));
     }
     if (!heads || a.rule != kDelta) return;
@@ -224,8 +272,6 @@ mix_kernel(const Recurrence a, int v_blocks, int heads_per_block) {
 
 // ---- token by token: decode, and prompts that the chunked kernels do not take ------------
 
-constexpr int kStepThreads = 512;
-constexpr int kMaxAhead = 8;   // state rows per thread, in registers
 constexpr int kTapsAhead = 3;   // earlier inputs of a channel fetched together
 
 // Grid: heads, requests, blocks of 4 << log_cols value columns (at most kStepThreads).
@@ -233,11 +279,12 @@ template <typename T, int RULE, bool DECODE, int AHEAD>
 __global__ void __launch_bounds__(kStepThreads, 2)
 step_kernel(const Recurrence a, int log_cols, bool finish) {
     extern __shared__ __align__(16) float smem[];
-    __shared__ float s_ss[kStepThreads / 32];
+    __shared__ float s_ss[kStepThreads / 32], s_den[kStepThreads / 32];
     __shared__ float2 s_step;
+    constexpr bool CONV = has_convolution(RULE);
     const int dk = a.padded_dim, vp = a.padded_value_dim;
     const int nv4 = 1 << log_cols, cols = nv4 * 4, groups = kStepThreads >> log_cols;
-    float *s_v = smem, *s_k = s_v + cols, *s_q = s_k + dk, *s_red = s_q + dk;
+    float *s_v = smem, *s_k = s_v + cols, *s_q = s_k + dk, *s_red = s_q + dk, *s_n = s_red + kStepThreads * 4;   // s_n: kMemory
     const int h = blockIdx.x, b = blockIdx.y, col0 = blockIdx.z * cols;
     const int kvh = h / (a.heads / a.kv_heads);
     const int group = threadIdx.x >> log_cols, col = (threadIdx.x & (nv4 - 1)) * 4;
@@ -263,11 +310,21 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
         return nv + (i < dk ? static_cast<int64_t>(kvh) * dk + i : static_cast<int64_t>(a.kv_heads + kvh) * dk + i - dk);
     };
     auto place = [&](int i) -> float& { return i < own_v ? s_v[i] : s_k[i - own_v]; };   // (s_q follows s_k)
-    T* ring = static_cast<T*>(a.conv_state) + row_state * a.taps * nc;
-    const int now = DECODE ? cached % a.taps : 0;
+    T* ring = CONV ? static_cast<T*>(a.conv_state) + row_state * a.taps * nc : nullptr;
+    const int now = DECODE && CONV ? cached % a.taps : 0;
     const bool steps = threadIdx.x == kStepThreads - 1;   // this thread works out the step
-    float step_bias = 0.f, decay = 0.f, norm = 0.f;
-    if (DECODE) {
+    float step_bias = 0.f, decay = 0.f, norm = 0.f, top = 0.f;   // top: the running maximum of kMemory
+    if (RULE == kMemory) {   // (a thread works on the same elements of n all the way)
+        const float* memory = memory_of(a, row_state, h, col0);
+        for (int i = threadIdx.x; i < dk; i += kStepThreads) s_n[i] = cached > 0 ? memory[i] : 0.f;
+        if (cached > 0) top = memory[dk];
+    }
+    if (DECODE && !CONV) {
+        if (steps && RULE == kMemory) step_bias = a.step_bias[h], decay = a.step_bias[a.heads + h];
+        if (steps && RULE == kLightning) decay = a.decay_log[h];
+        if (finish && threadIdx.x < own_v) norm = to_f32(static_cast<const T*>(a.norm)[static_cast<int64_t>(h) * vp + threadIdx.x]);
+    }
+    if constexpr (DECODE && CONV) {
         // what the inputs before this one add to the channels, two of them at a time
         for (int i0 = threadIdx.x; i0 < own; i0 += 2 * kStepThreads) {
             float y[2] = {0.f, 0.f}, w[2][kTapsAhead], in[2][kTapsAhead];
@@ -313,40 +370,62 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
             const T* tail = row + nv + nc;
             float za = 0.f, zb = 0.f;
             if (steps) {
-                za = to_f32(tail[h]);
-                if (RULE == kDelta) zb = to_f32(tail[a.heads + h]);
+                if (RULE != kLightning) za = to_f32(tail[h]);
+                if (RULE == kDelta || RULE == kMemory) zb = to_f32(tail[a.heads + h]);
             }
             if (finish && threadIdx.x < own_v) gate = to_f32(row[static_cast<int64_t>(h) * vp + threadIdx.x]);
-            T* keep = ring + static_cast<int64_t>(now) * nc;
+            T* keep = CONV ? ring + static_cast<int64_t>(now) * nc : nullptr;
             const bool keeps = h % (a.heads / a.kv_heads) == 0 && blockIdx.z == 0;   // k and q are shared
-            for (int i0 = threadIdx.x; i0 < own; i0 += 2 * kStepThreads) {
-                T in[2];
-                float w[2];
-#pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const int i = i0 + e * kStepThreads;
-                    const int64_t c = channel(i < own ? i : 0);
-                    in[e] = row[nv + c];
-                    w[e] = a.conv[(a.taps - 1) * nc + c];
+            if constexpr (!CONV) {
+                for (int i = threadIdx.x; i < own; i += kStepThreads) {
+                    const float x = to_f32(row[nv + channel(i)]);
+                    place(i) = RULE == kLightning ? to_f32(from_f32<T>(silu<T>(x))) : x;
                 }
-#pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const int i = i0 + e * kStepThreads;
-                    if (i >= own) continue;
-                    place(i) = to_f32(from_f32<T>(silu<T>(fmaf(w[e], to_f32(in[e]), place(i)))));
-                    if (i < own_v || keeps) keep[channel(i)] = in[e];
+            } else {
+                for (int i0 = threadIdx.x; i0 < own; i0 += 2 * kStepThreads) {
+                    T in[2];
+                    float w[2];
+    #pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        const int i = i0 + e * kStepThreads;
+                        const int64_t c = channel(i < own ? i : 0);
+                        in[e] = row[nv + c];
+                        w[e] = a.conv[(a.taps - 1) * nc + c];
+                    }
+    #pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        const int i = i0 + e * kStepThreads;
+                        if (i >= own) continue;
+                        place(i) = to_f32(from_f32<T>(silu<T>(fmaf(w[e], to_f32(in[e]), place(i)))));
+                        if (i < own_v || keeps) keep[channel(i)] = in[e];
+                    }
                 }
             }
-            if (steps) s_step = make_step(RULE, za, zb, step_bias, decay);
+            if (steps) s_step = make_step(RULE, za, zb, step_bias, decay, a.gate_cap);
         } else {
-            const T* mixed = static_cast<const T*>(a.mixed) + t * nc;
+            const T* mixed = mixed_rows<T>(a) + t * mixed_ld(a);
             for (int i = threadIdx.x; i < own; i += kStepThreads) place(i) = to_f32(mixed[channel(i)]);
             step = reinterpret_cast<const float2*>(a.steps)[t * a.heads + h];
         }
         __syncthreads();
         if (DECODE) step = s_step;
         float kf = step.y, qf = 1.f;   // factors of k and q
-        const float g = exp2f(step.x);
+        float g = exp2f(step.x);
+        if (RULE == kMemory) {
+            const float next = fmaxf(step.x + top, step.y);
+            g = exp2f(step.x + top - next);
+            kf = exp2f(step.y - next);
+            qf = rsqrtf(static_cast<float>(a.dim));
+            top = next;
+            float den = 0.f;
+            for (int i = threadIdx.x; i < dk; i += kStepThreads) {
+                const float n = fmaf(kf, s_k[i], g * s_n[i]);
+                s_n[i] = n;
+                den = fmaf(n, s_q[i], den);
+            }
+            den = warp_sum(den);
+            if ((threadIdx.x & 31) == 0) s_den[threadIdx.x >> 5] = den;   // (published by the barrier below)
+        }
         if (RULE == kDelta) {
             if (DECODE) {
                 const int lane = threadIdx.x & 31;
@@ -413,19 +492,33 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
         if (c < own_v) {
             for (int i = 0; i < groups; ++i) y += s_red[i * cols + c];
             y *= qf;
+            if (RULE == kMemory) {
+                float den = 0.f;
+#pragma unroll
+                for (int i = 0; i < kStepThreads / 32; ++i) den += s_den[i];
+                y /= fmaxf(fabsf(den * qf), exp2f(-top)) + kMemoryEps;
+            }
             if (RULE == kStateSpace) y = fmaf(skip, s_v[c], y);
             if (!finish) out[c] = from_f32<T>(y);
         }
-        if (DECODE && RULE == kDelta && finish) {   // the whole head is here: norm and gate
+        if (DECODE && (RULE == kDelta || RULE == kMemory) && finish) {   // the whole head is here: norm and gate
             const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
             float ss = warp_sum(y * y);
             if (lane == 0) s_ss[warp] = ss;
             __syncthreads();
             ss = warp_sum(lane < kStepThreads / 32 ? s_ss[lane] : 0.f);
             const float scale = rsqrtf(ss / static_cast<float>(a.value_dim) + a.eps) * a.out_scale;
-            if (c < own_v) out[c] = from_f32<T>(y * scale * norm * silu<T>(gate));
+            if (c < own_v) out[c] = from_f32<T>(y * scale * norm * (RULE == kMemory ? sigmoid<T>(gate) : silu<T>(gate)));
         }
         if (!DECODE) __syncthreads();   // everything in shared memory has been used
+    }
+    if (RULE == kMemory && begin < end) {
+        const int each = memory_columns(dk);
+        for (int at = col0; at < min(col0 + cols, vp); at += each) {
+            float* memory = memory_of(a, row_state, h, at);
+            for (int i = threadIdx.x; i < dk; i += kStepThreads) memory[i] = s_n[i];
+            if (threadIdx.x == 0) memory[dk] = top;
+        }
     }
     if (DECODE || !active || begin >= end) return;
 #pragma unroll
@@ -471,7 +564,8 @@ finish_heads_kernel(const Recurrence a) {
     for (int c = c0 + 128; c < vp; c += 128) emit(c, load4(out + c), load4(gate + c), load4(norm + c));
 }
 
-// State space: one CTA per (token, part of the norm).  A part is a run of the concatenated heads without their
+// The others: one CTA per (token, part of the norm); the state space's gate comes before the norm, the others' behind it.
+// A part is a run of the concatenated heads without their
 // padding, so it may begin and end inside one; VEC elements at a time.
 constexpr int kPartThreads = 128;
 constexpr int kPartKeep = 4;   // pieces of VEC elements a thread keeps in registers
@@ -487,14 +581,20 @@ finish_parts_kernel(const Recurrence a) {
     T* out = static_cast<T*>(a.out) + t * a.out_ld;
     const T* gate = static_cast<const T*>(a.joint) + t * a.joint_ld;
     const T* norm = static_cast<const T*>(a.norm);
+    const bool before = a.rule == kStateSpace;
     auto place = [&](int i) { return (from + i) / a.value_dim * a.padded_value_dim + (from + i) % a.value_dim; };
     auto gated = [&](int at, float (&y)[VEC]) {
         if (VEC == 8) {
-            const Vec8 o = load8(out + at), z = load8(gate + at);
+            const Vec8 o = load8(out + at);
 #pragma unroll
-            for (int j = 0; j < VEC; ++j) y[j] = o.v[j & 7] * silu<T>(z.v[j & 7]);
+            for (int j = 0; j < VEC; ++j) y[j] = o.v[j & 7];
+            if (!before) return;
+            const Vec8 z = load8(gate + at);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) y[j] *= silu<T>(z.v[j & 7]);
         } else {
-            y[0] = to_f32(out[at]) * silu<T>(to_f32(gate[at]));
+            y[0] = to_f32(out[at]);
+            if (before) y[0] *= silu<T>(to_f32(gate[at]));
         }
     };
     float kept[kPartKeep][VEC], ss = 0.f;
@@ -524,9 +624,14 @@ finish_parts_kernel(const Recurrence a) {
             Vec8 o;
 #pragma unroll
             for (int j = 0; j < 8; ++j) o.v[j] = y[j % VEC] * scale * w.v[j];
+            if (!before) {
+                const Vec8 z = load8(gate + at);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) o.v[j] *= sigmoid<T>(z.v[j]);
+            }
             store8(out + at, o);
         } else {
-            out[at] = from_f32<T>(y[0] * scale * to_f32(norm[at]));
+            out[at] = from_f32<T>(y[0] * scale * to_f32(norm[at]) * (before ? 1.f : sigmoid<T>(to_f32(gate[at]))));
         }
     };
 #pragma unroll
@@ -591,6 +696,23 @@ struct PrepareSmem {
     };
     float sum[2][kChunk], weight[2][kChunk], kf[kChunk], qf[kChunk];
 };
+
+// Running maxima of a chunk's numbers, held like running_sums.
+__device__ __forceinline__ float2 running_maxima(float2 x) {
+    const int lane = threadIdx.x & 31;
+    float s = fmaxf(x.x, x.y);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const float up = __shfl_up_sync(0xffffffffu, s, o);
+        if (lane >= o) s = fmaxf(s, up);
+    }
+    const float before = __shfl_up_sync(0xffffffffu, s, 1);
+    return make_float2(lane > 0 ? fmaxf(before, x.x) : x.x, s);
+}
+// A token that is not there writes nothing.
+template <int RULE>
+__device__ __forceinline__ float2 no_step() { return make_float2(0.f, RULE == kMemory ? -INFINITY : 0.f); }
+
 
 // Barrier of the two warps that work on one head.
 __device__ __forceinline__ void pair_sync() {
@@ -689,8 +811,8 @@ prepare_kernel(const Recurrence a, int parts) {
     const int s0 = blockIdx.x * kChunk;
     if (s0 >= ext) return;
     const int n = min(kChunk, ext - s0);
-    const int64_t nc = channels(a), first = begin + s0;
-    const __nv_bfloat16* k0 = static_cast<const __nv_bfloat16*>(a.mixed) + first * nc + values(a) + static_cast<int64_t>(kvh) * a.padded_dim;
+    const int64_t nc = mixed_ld(a), first = begin + s0;
+    const __nv_bfloat16* k0 = mixed_rows<__nv_bfloat16>(a) + first * nc + values(a) + static_cast<int64_t>(kvh) * a.padded_dim;
     const int64_t to_q = static_cast<int64_t>(a.kv_heads) * a.padded_dim;
     if (threadIdx.x < kChunk) {
         float kf = 1.f, qf = 1.f;
@@ -741,11 +863,18 @@ prepare_kernel(const Recurrence a, int parts) {
         if ((warp & 1) == 0 && h0 + (warp >> 1) < to) {
             const int h = kvh * group + h0 + (warp >> 1);
             const float2* steps = reinterpret_cast<const float2*>(a.steps) + first * a.heads + h;
-            const float2 none = make_float2(0.f, 0.f);
+            const float2 none = no_step<RULE>();
             const float2 x = 2 * lane < n ? steps[static_cast<int64_t>(2 * lane) * a.heads] : none;
             const float2 y = 2 * lane + 1 < n ? steps[static_cast<int64_t>(2 * lane + 1) * a.heads] : none;
-            *reinterpret_cast<float2*>(&S.sum[warp >> 1][2 * lane]) = running_sums(make_float2(x.x, y.x));
-            *reinterpret_cast<float2*>(&S.weight[warp >> 1][2 * lane]) = make_float2(x.y, y.y);
+            const float2 B = running_sums(make_float2(x.x, y.x));
+            if (RULE == kMemory) {   // the exponent of P_ts is weight_s - sum_t: sum holds the maxima here
+                const float2 e = make_float2(x.y - B.x, y.y - B.y);
+                *reinterpret_cast<float2*>(&S.sum[warp >> 1][2 * lane]) = running_maxima(e);
+                *reinterpret_cast<float2*>(&S.weight[warp >> 1][2 * lane]) = e;
+            } else {
+                *reinterpret_cast<float2*>(&S.sum[warp >> 1][2 * lane]) = B;
+                *reinterpret_cast<float2*>(&S.weight[warp >> 1][2 * lane]) = make_float2(x.y, y.y);
+            }
         }
         __syncthreads();
 #pragma unroll
@@ -754,7 +883,8 @@ prepare_kernel(const Recurrence a, int parts) {
             uint4* out = chunks + (static_cast<int64_t>(kvh * group + h0 + hp) * kMatrices) * kMatrixVecs + lane;
             const int t0 = warp * 16 + g;
             const float sum_t[2] = {S.sum[hp][t0], S.sum[hp][t0 + 8]};
-            float q_t[2] = {1.f, 1.f}, k_t[2] = {0.f, 0.f};
+            float q_t[2] = {1.f, 1.f}, k_t[2] = {0.f, 0.f}, row_sum[2] = {0.f, 0.f};
+            if (RULE == kMemory) q_t[0] = q_t[1] = rsqrtf(static_cast<float>(a.dim));
             if (RULE == kDelta) {
                 q_t[0] = S.qf[t0];
                 q_t[1] = S.qf[t0 + 8];
@@ -775,8 +905,15 @@ prepare_kernel(const Recurrence a, int parts) {
 #pragma unroll
                     for (int half = 0; half < 2; ++half) {   // rows g, g + 8
                         const int t = t0 + half * 8, tile = 2 * kt + side;
-                        const float rx = (s <= t ? ex2(sum_t[half] - sum_s.x) : 0.f) * f_s.x;
-                        const float ry = (s + 1 <= t ? ex2(sum_t[half] - sum_s.y) : 0.f) * f_s.y;
+                        float rx, ry;
+                        if (RULE == kMemory) {
+                            rx = s <= t ? ex2(f_s.x - sum_t[half]) : 0.f;
+                            ry = s + 1 <= t ? ex2(f_s.y - sum_t[half]) : 0.f;
+                            row_sum[half] += qk[tile][2 * half] * (rx * q_t[half]) + qk[tile][2 * half + 1] * (ry * q_t[half]);
+                        } else {
+                            rx = (s <= t ? ex2(sum_t[half] - sum_s.x) : 0.f) * f_s.x;
+                            ry = (s + 1 <= t ? ex2(sum_t[half] - sum_s.y) : 0.f) * f_s.y;
+                        }
                         split2(qk[tile][2 * half] * (rx * q_t[half]), qk[tile][2 * half + 1] * (ry * q_t[half]), hi[2 * side + half],
                                lo[2 * side + half]);
                         am[half] = make_float2(s < t ? kk[tile][2 * half] * (rx * k_t[half]) : 0.f,
@@ -790,6 +927,15 @@ prepare_kernel(const Recurrence a, int parts) {
                 const int tile = warp * (warp + 1) / 2 + kt;
                 out[tile * 64] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
                 out[tile * 64 + 32] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            }
+            if (RULE == kMemory) {
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    float r = row_sum[half];
+                    r += __shfl_xor_sync(0xffffffffu, r, 1);
+                    r += __shfl_xor_sync(0xffffffffu, r, 2);
+                    if (tq == 0 && t0 + half * 8 < n) a.units[(first + t0 + half * 8) * a.heads + kvh * group + h0 + hp] = r;
+                }
             }
         }
         if (RULE != kDelta) continue;
@@ -843,6 +989,9 @@ struct WalkSmem {
     float beta[2][kChunk], read[2][kChunk];   // beta_t; beta_t G_t times k's factor
     float write[2][kChunk];    // exp(B_n - B_t) times k's factor (or times dt)
     float keep[2];             // G_n
+    // matrix memory: factors of P V, exp(-m_t), what the chunk's tokens add to n . q; n; one over the denominator
+    float own[RULE == kMemory ? 2 : 1][kChunk], floor[RULE == kMemory ? 2 : 1][kChunk], row_sum[RULE == kMemory ? 2 : 1][kChunk];
+    float n[RULE == kMemory ? DK : 4], over[RULE == kMemory ? kChunk : 4];
 };
 
 // Grid: slices of 64 value columns, heads, requests.  All products are formed transposed, 16 value columns by tokens (or
@@ -866,8 +1015,8 @@ chunk_kernel(const Recurrence a) {
     pdl_wait_prior();
     const int begin = a.qo_indptr[req], ext = a.qo_indptr[req + 1] - begin;
     if (ext <= 0) return;
-    const int64_t nc = channels(a);
-    const __nv_bfloat16* mixed = static_cast<const __nv_bfloat16*>(a.mixed) + begin * nc;
+    const int64_t nc = mixed_ld(a);
+    const __nv_bfloat16* mixed = mixed_rows<__nv_bfloat16>(a) + begin * nc;
     const int64_t at_k = values(a) + static_cast<int64_t>(kvh) * DK, to_q = static_cast<int64_t>(a.kv_heads) * DK;
     const int64_t at_v = static_cast<int64_t>(h) * vp + v0;
 
@@ -889,8 +1038,9 @@ chunk_kernel(const Recurrence a) {
     auto fetch_factors = [&](int s0) {
         const int n = min(kChunk, ext - s0);
         const float2* steps = reinterpret_cast<const float2*>(a.steps) + static_cast<int64_t>(begin + s0) * a.heads + h;
-        st0 = st1 = make_float2(0.f, 0.f);
+        st0 = st1 = no_step<RULE>();
         un0 = un1 = make_float2(1.f, 1.f);
+        auto sum_of = [&](int t) { return make_float2(a.units[static_cast<int64_t>(begin + s0 + t) * a.heads + h], 0.f); };
         auto unit = [&](int t) {
             const float* u = a.units + static_cast<int64_t>(begin + s0 + t) * 2 * a.kv_heads + kvh;
             return make_float2(u[0], u[a.kv_heads]);
@@ -898,15 +1048,32 @@ chunk_kernel(const Recurrence a) {
         if (2 * lane < n) {
             st0 = steps[static_cast<int64_t>(2 * lane) * a.heads];
             if (RULE == kDelta) un0 = unit(2 * lane);
+            if (RULE == kMemory) un0 = sum_of(2 * lane);
         }
         if (2 * lane + 1 < n) {
             st1 = steps[static_cast<int64_t>(2 * lane + 1) * a.heads];
             if (RULE == kDelta) un1 = unit(2 * lane + 1);
+            if (RULE == kMemory) un1 = sum_of(2 * lane + 1);
         }
     };
+    float top = 0.f;   // the matrix memory's running maximum (first warp)
     auto put_factors = [&](int buf) {
         const float2 B = running_sums(make_float2(st0.x, st1.x));
         const float last = __shfl_sync(0xffffffffu, B.y, 31);
+        if constexpr (RULE == kMemory) {
+            const float2 e = make_float2(st0.y - B.x, st1.y - B.y), c = running_maxima(e);
+            const float c_n = __shfl_sync(0xffffffffu, c.y, 31), qf = rsqrtf(static_cast<float>(a.dim));
+            const float r0 = fmaxf(top, c.x), r1 = fmaxf(top, c.y), r = fmaxf(top, c_n);
+            auto put = [&](float* to, float x, float y) { *reinterpret_cast<float2*>(to + 2 * lane) = make_float2(x, y); };
+            put(S.out[buf], ex2(top - r0) * qf, ex2(top - r1) * qf);
+            put(S.own[buf], ex2(c.x - r0), ex2(c.y - r1));
+            put(S.floor[buf], ex2(-(B.x + r0)), ex2(-(B.y + r1)));
+            put(S.row_sum[buf], un0.x, un1.x);
+            put(S.write[buf], ex2(e.x - r), ex2(e.y - r));
+            if (lane == 0) S.keep[buf] = ex2(top - r);
+            top = last + r;
+            return;
+        }
         const float g0 = ex2(B.x), g1 = ex2(B.y), w0 = ex2(last - B.x), w1 = ex2(last - B.y);
         *reinterpret_cast<float2*>(&S.out[buf][2 * lane]) = make_float2(g0 * un0.y, g1 * un1.y);
         if (RULE == kDelta) {
@@ -934,6 +1101,11 @@ chunk_kernel(const Recurrence a) {
     for (int j = 0; j < kRows / 8; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) st[j][e] = fresh ? 0.f : state[static_cast<int64_t>(8 * j + 2 * tq + (e & 1)) * vp + (e >> 1) * 8];
+    if constexpr (RULE == kMemory) {
+        const float* memory = memory_of(a, a.table_idx[req], h, v0);
+        for (int i = threadIdx.x; i < DK; i += kWalkThreads) S.n[i] = fresh ? 0.f : memory[i];
+        if (!fresh) top = memory[DK];
+    }
     if (warp == 0) {
         fetch_factors(0);
         put_factors(0);
@@ -997,6 +1169,31 @@ chunk_kernel(const Recurrence a) {
             if (warp == 0) fetch_factors(s0 + kChunk);
         }
         const __nv_bfloat16 *K = S.k[buf], *Q = S.q[buf], *V = S.v[buf];
+        if constexpr (RULE == kMemory) {
+            // denominators of the chunk's tokens, four threads each; then n moves on, kParts threads per element
+            constexpr int kEach = DK / 4;
+            const int t = threadIdx.x >> 2, d0 = (threadIdx.x & 3) * kEach;
+            float dot = 0.f;
+#pragma unroll
+            for (int d = 0; d < kEach; d += 8) {
+                const Vec8 x = load8(Q + t * ROW + d0 + d);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) dot = fmaf(x.v[j], S.n[d0 + d + j], dot);
+            }
+            dot += __shfl_xor_sync(0xffffffffu, dot, 1);
+            dot += __shfl_xor_sync(0xffffffffu, dot, 2);
+            if ((threadIdx.x & 3) == 0)
+                S.over[t] = 1.f / (fmaxf(fabsf(fmaf(S.out[buf][t], dot, S.own[buf][t] * S.row_sum[buf][t])), S.floor[buf][t]) + kMemoryEps);
+            __syncthreads();
+            constexpr int kParts = kWalkThreads / DK;
+            const int i = threadIdx.x / kParts, part = threadIdx.x % kParts;
+            float sum = 0.f;
+#pragma unroll 8
+            for (int s = part; s < kChunk; s += kParts) sum = fmaf(S.write[buf][s], __bfloat162float(K[s * ROW + i]), sum);
+#pragma unroll
+            for (int o = 1; o < kParts; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            if (part == 0) S.n[i] = fmaf(S.keep[buf], S.n[i], sum);
+        }
         // ---- S^T Q^T and S^T K^T ----
         float o[2][2][4], u[2][2][4];
         {
@@ -1126,7 +1323,24 @@ chunk_kernel(const Recurrence a) {
 #pragma unroll
             for (int kt = 0; kt < 4; ++kt) take(1, kt, xh[kt], xl[kt]);
         }
-        multiply(o, xh, RULE == kDelta ? xl : nullptr, S.m[buf]);
+        if constexpr (RULE == kMemory) {
+            float pv[2][2][4] = {};
+            multiply(pv, xh, nullptr, S.m[buf]);
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int side = 0; side < 2; ++side) {
+                    const int t = own[i] * 16 + side * 8 + 2 * tq;
+                    const float2 f = *reinterpret_cast<const float2*>(&S.own[buf][t]), z = *reinterpret_cast<const float2*>(&S.over[t]);
+                    float *c = o[i][side], *x = pv[i][side];
+                    c[0] = fmaf(f.x, x[0], c[0]) * z.x;
+                    c[1] = fmaf(f.y, x[1], c[1]) * z.y;
+                    c[2] = fmaf(f.x, x[2], c[2]) * z.x;
+                    c[3] = fmaf(f.y, x[3], c[3]) * z.y;
+                }
+        } else {
+            multiply(o, xh, RULE == kDelta ? xl : nullptr, S.m[buf]);
+        }
         {
             __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + static_cast<int64_t>(begin + s0) * a.out_ld + at_v + col0 + 2 * tq;
 #pragma unroll
@@ -1176,6 +1390,14 @@ chunk_kernel(const Recurrence a) {
         }
         if (more && warp == 0) put_factors(buf ^ 1);
     }
+    if constexpr (RULE == kMemory) {
+        __syncthreads();
+        for (int at = v0; at < v0 + kSlice; at += memory_columns(DK)) {
+            float* memory = memory_of(a, a.table_idx[req], h, at);
+            for (int i = threadIdx.x; i < DK; i += kWalkThreads) memory[i] = S.n[i];
+            if (threadIdx.x == 0) memory[DK] = top;
+        }
+    }
 #pragma unroll
     for (int j = 0; j < kRows / 8; ++j)
 #pragma unroll
@@ -1193,10 +1415,12 @@ int max_smem(const void* kernel, size_t bytes) {
 
 template <typename T>
 int launch_mix(const Recurrence& a, cudaStream_t stream) {
-    auto kernel = a.taps == 2 ? mix_kernel<T, 2> : a.taps == 3 ? mix_kernel<T, 3> : a.taps == 4 ? mix_kernel<T, 4> : mix_kernel<T, 0>;
+    auto kernel = a.conv == nullptr ? mix_kernel<T, 1> : a.taps == 2 ? mix_kernel<T, 2> : a.taps == 3 ? mix_kernel<T, 3> : a.taps == 4 ? mix_kernel<T, 4> : mix_kernel<T, 0>;
     const int v_blocks = div_ceil(a.heads * a.padded_value_dim, kMixThreads * 8);
     const int per_block = kMixThreads / (a.padded_dim / 8);
-    const dim3 grid(div_ceil(a.max_extend, kMixTokens), v_blocks + div_ceil(2 * a.kv_heads, per_block) + 1, a.batch);
+    // (of the matrix memory's channels nothing is made: the steps alone)
+    const int blocks = a.rule == kMemory ? 1 : v_blocks + div_ceil(2 * a.kv_heads, per_block) + 1;
+    const dim3 grid(div_ceil(a.max_extend, kMixTokens), blocks, a.batch);
     B200_CHECK_CUDA(launch_kernel(kernel, grid, dim3(kMixThreads), 0, stream, dim3(1, 1, 1), a, v_blocks, per_block));
     return B200_OK;
 }
@@ -1220,7 +1444,7 @@ int launch_chunked(const Recurrence& a, cudaStream_t stream) {
 
 template <typename T, int RULE>
 int launch_steps(const Recurrence& a, int log_cols, int slices, bool finish, cudaStream_t stream) {
-    const size_t smem = ((4ull << log_cols) + 2ull * a.padded_dim + kStepThreads * 4) * 4;
+    const size_t smem = ((4ull << log_cols) + (RULE == kMemory ? 3ull : 2ull) * a.padded_dim + kStepThreads * 4) * 4;
     const bool few = div_ceil(a.padded_dim, kStepThreads >> log_cols) <= 4;
     auto kernel = a.decode ? (few ? step_kernel<T, RULE, true, 4> : step_kernel<T, RULE, true, kMaxAhead>)
                            : (few ? step_kernel<T, RULE, false, 4> : step_kernel<T, RULE, false, kMaxAhead>);
@@ -1237,16 +1461,20 @@ int run(const Recurrence& a, int dtype, cudaStream_t stream) {
     if (err != B200_OK) return err;
     bool finished = false;
     if (!a.decode && chunked_supported(a, dtype)) {
-        err = delta ? launch_chunked<kDelta>(a, stream) : launch_chunked<kStateSpace>(a, stream);
+        err = delta ? launch_chunked<kDelta>(a, stream)
+              : a.rule == kStateSpace ? launch_chunked<kStateSpace>(a, stream)
+              : a.rule == kLightning ? launch_chunked<kLightning>(a, stream) : launch_chunked<kMemory>(a, stream);
     } else {
         // groups of four columns per CTA: a thread has room for kMaxAhead rows, and one output column
         const int most = kMaxAhead * kStepThreads / a.padded_dim;
         int log_cols = 0;
         while ((4 << log_cols) < a.padded_value_dim && (2 << log_cols) <= most && (8 << log_cols) <= kStepThreads) ++log_cols;
         const int slices = div_ceil(a.padded_value_dim, 4 << log_cols);
-        finished = a.decode && delta && slices == 1;
+        finished = a.decode && slices == 1 && (delta || (a.rule == kMemory && a.norm_groups == a.heads));
         err = delta ? launch_steps<T, kDelta>(a, log_cols, slices, finished, stream)
-                    : launch_steps<T, kStateSpace>(a, log_cols, slices, finished, stream);
+              : a.rule == kStateSpace ? launch_steps<T, kStateSpace>(a, log_cols, slices, finished, stream)
+              : a.rule == kLightning ? launch_steps<T, kLightning>(a, log_cols, slices, finished, stream)
+                                     : launch_steps<T, kMemory>(a, log_cols, slices, finished, stream);
     }
     if (err != B200_OK || finished) return err;
     if (delta) {
@@ -1274,11 +1502,16 @@ RecurrenceScratch recurrence_scratch(int rule, int max_tokens, int max_batch, in
     const int64_t T = max_tokens, esz = dtype == B200_DTYPE_F32 ? 4 : 2;
     s.mixed = T * (static_cast<int64_t>(heads) * padded_value_dim + 2ll * kv_heads * padded_dim) * esz;
     s.steps = T * heads * 8;
-    s.units = rule == kDelta ? T * kv_heads * 8 : 0;
+    s.units = rule == kDelta ? T * kv_heads * 8 : rule == kMemory ? T * heads * 4 : 0;
+    if (rule == kMemory) s.mixed = 0;
     s.chunks = dtype == B200_DTYPE_F32 || padded_dim > 128
                    ? 0
                    : (T / kChunk + max_batch + 1) * heads * (rule == kDelta ? 2 : 1) * kMatrixVecs * 16;
     return s;
+}
+
+int64_t recurrence_memory_floats(int padded_dim, int padded_value_dim) {
+    return static_cast<int64_t>(memory_copies(padded_dim, padded_value_dim)) * memory_width(padded_dim);
 }
 
 int launch_recurrence(const Recurrence& a, int dtype, cudaStream_t stream) {
@@ -1303,15 +1536,25 @@ int b200_recurrence_scratch(int rule, int max_tokens, int max_batch, int heads, 
     return B200_OK;
 }
 
+int64_t b200_recurrence_memory_bytes(int padded_dim, int padded_value_dim) {
+    if (padded_dim <= 0 || padded_dim % 64 != 0 || padded_value_dim <= 0 || padded_value_dim % 64 != 0 ||
+        !b200::recurrence_supported(padded_value_dim, padded_dim, 1))
+        return -1;
+    return b200::recurrence_memory_floats(padded_dim, padded_value_dim) * 4;
+}
+
 int b200_recurrence(const b200_recurrence_args* p, int dtype, b200_stream_t stream) {
     B200_CHECK_ARG(p, "recurrence: NULL argument");
     B200_CHECK_ARG(dtype == B200_DTYPE_BF16 || dtype == B200_DTYPE_F32, "recurrence: unknown dtype");
-    B200_CHECK_ARG(p->rule == B200_RULE_STATE_SPACE || p->rule == B200_RULE_DELTA, "recurrence: unknown rule");
+    B200_CHECK_ARG(p->rule >= B200_RULE_STATE_SPACE && p->rule <= B200_RULE_MATRIX_MEMORY, "recurrence: unknown rule");
+    const bool conv = b200::has_convolution(p->rule), memory = p->rule == B200_RULE_MATRIX_MEMORY;
+    B200_CHECK_ARG(conv || (p->kv_heads == p->heads && !p->conv && !p->conv_bias), "recurrence: no convolution with this rule");
+    B200_CHECK_ARG(!memory || p->gate_cap > 0.f, "recurrence: bad gate cap");
     B200_CHECK_ARG(p->tokens >= 0 && p->batch >= 0 && p->batch <= 65535 && p->heads > 0 && p->heads <= 65535 && p->kv_heads > 0 &&
                        p->heads % p->kv_heads == 0, "recurrence: bad sizes");
     B200_CHECK_ARG(p->dim > 0 && p->padded_dim >= p->dim && p->padded_dim % 64 == 0 && p->value_dim > 0 &&
                        p->padded_value_dim >= p->value_dim && p->padded_value_dim % 64 == 0 &&
-                       b200::recurrence_supported(p->padded_value_dim, p->padded_dim, p->taps), "recurrence: bad head sizes");
+                       b200::recurrence_supported(p->padded_value_dim, p->padded_dim, conv ? p->taps : 1), "recurrence: bad head sizes");
     B200_CHECK_ARG(p->joint_ld % 8 == 0 && p->out_ld % 8 == 0 && p->out_ld >= static_cast<int64_t>(p->heads) * p->padded_value_dim,
                    "recurrence: bad strides");
     B200_CHECK_ARG(p->rule == B200_RULE_DELTA || (p->norm_groups > 0 && p->heads * p->value_dim % p->norm_groups == 0),
@@ -1319,10 +1562,13 @@ int b200_recurrence(const b200_recurrence_args* p, int dtype, b200_stream_t stre
     B200_CHECK_ARG(static_cast<int64_t>(p->tokens) * p->heads < (1ll << 31), "recurrence: too many tokens");
     B200_CHECK_ARG(!p->decode || p->tokens == p->batch, "recurrence: a decode step brings one token per request");
     if (p->tokens == 0 || p->batch == 0) return B200_OK;
-    B200_CHECK_ARG(p->out && p->joint && p->table_idx && p->cached && p->state && p->conv_state && p->conv && p->decay_log &&
-                       p->step_bias && p->norm && (p->rule == B200_RULE_DELTA || p->skip), "recurrence: NULL tensor");
-    B200_CHECK_ARG(p->decode || (p->qo_indptr && p->mixed && p->steps && (p->units || p->rule != B200_RULE_DELTA) && p->chunks &&
-                                 p->max_extend > 0), "recurrence: NULL scratch");
+    B200_CHECK_ARG(p->out && p->joint && p->table_idx && p->cached && p->state && p->norm &&
+                       (!conv || (p->conv_state && p->conv && p->step_bias)) && (memory || p->decay_log) &&
+                       (p->rule != B200_RULE_STATE_SPACE || p->skip) && (!memory || (p->step_bias && p->memory)),
+                   "recurrence: NULL tensor");
+    B200_CHECK_ARG(p->decode || (p->qo_indptr && (p->mixed || memory) && p->steps &&
+                                 (p->units || (p->rule != B200_RULE_DELTA && !memory)) && p->chunks && p->max_extend > 0),
+                   "recurrence: NULL scratch");
     return b200::launch_recurrence(*p, dtype, static_cast<cudaStream_t>(stream));
 }
 

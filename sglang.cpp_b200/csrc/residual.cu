@@ -4,7 +4,7 @@
 // rows that the next block's grouped GEMM reads.  One CTA per token, the row in registers.
 //
 // Wirings: the norm on what the next block reads (residual_norm_kernel), or on what the previous block
-// returned, before it is added, or both (residual_post_norm_kernel).
+// returned, before it is added, or both (residual_post_norm_kernel, which also has layer norms).
 #include "common.cuh"
 #include "kernels.h"
 
@@ -168,16 +168,20 @@ struct PostArgs {
     int32_t* clear;
     int clear_count;
     int* status;
+    const void *add_bias, *out_bias, *self;   // KIND kLayer
+    float src_scale;                          // (kRms as well)
 };
+enum { kRms = 0, kPair = 1, kLayer = 2 };
 
 // What is added is a token's row of the source, or the weighted rows src_rows names, plus its row of a second
-// source (PAIR: both normalised by themselves first, the sum scaled); it is RMS-normalised when there is a weight
-// for it.  The sum goes to the residual and, rounded (or
-// normalised once more, before the output head), to `out`.
-template <typename T, int VEC, bool PAIR>
+// source (kPair: both normalised by themselves first, the sum scaled); it is normalised when there is a weight
+// for it.  The sum goes to the residual and, rounded (or normalised once more), to `out`.  kLayer: the norms are
+// layer norms, and a source row of -1 stands for the token's row of `self`.
+template <typename T, int VEC, int KIND>
 __global__ void __launch_bounds__(256)
 residual_post_norm_kernel(const PostArgs a) {
-    __shared__ float red[PAIR ? 4 : 2][8];
+    constexpr bool PAIR = KIND == kPair, LAYER = KIND == kLayer;
+    __shared__ float red[KIND == kRms ? 2 : 4][8];
     __shared__ int s_row[kRows];
     __shared__ float s_weight[kRows];
     pdl_launch_dependents();
@@ -225,6 +229,12 @@ residual_post_norm_kernel(const PostArgs a) {
             for (int k = 0; k < a.src_top; ++k) {
                 const int64_t row = k < kRows ? s_row[k] : a.src_rows[t * a.src_top + k];
                 const float g = k < kRows ? s_weight[k] : a.src_weights != nullptr ? a.src_weights[t * a.src_top + k] : 1.f;
+                if (LAYER && row == -1 && a.self != nullptr) {
+                    const Vec8 x = load8(static_cast<const T*>(a.self) + t * a.padded + v * 8);
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) y.v[j] += g * x.v[j];
+                    continue;
+                }
                 if (row < 0 || row >= a.src_count) {   // adds nothing and is reported
                     if (v == 0) atomicExch(&a.status[kStatusBadIndex], static_cast<int>(row) + 1);
                     continue;
@@ -234,6 +244,8 @@ residual_post_norm_kernel(const PostArgs a) {
                 for (int j = 0; j < 8; ++j) y.v[j] += g * x.v[j];
             }
         }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) y.v[j] *= a.src_scale;
         if (src2 != nullptr) {
             const Vec8 x = load8(src2 + t * a.padded + v * 8);
 #pragma unroll
@@ -273,27 +285,56 @@ residual_post_norm_kernel(const PostArgs a) {
             add[i] = addend(v);
         }
 #pragma unroll
-        for (int j = 0; j < 8; ++j) ss += add[i].v[j] * add[i].v[j];
+        for (int j = 0; j < 8; ++j) ss += LAYER ? add[i].v[j] : add[i].v[j] * add[i].v[j];
     }
+    // layer norms: the sum of a piece's squared deviations (the padding deviates from nothing)
+    auto deviation = [&](const Vec8& x, int v, float mean) {
+        float d = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+            if (v * 8 + j < a.width) d += (x.v[j] - mean) * (x.v[j] - mean);
+        return d;
+    };
+    const T* add_bias = static_cast<const T*>(a.add_bias);
+    const T* out_bias = static_cast<const T*>(a.out_bias);
+    float mean = 0.f;
     const int wide0 = threadIdx.x + VEC * static_cast<int>(blockDim.x);   // rows wider than the registers
     float scale = 1.f;
     if (add_weight != nullptr) {
         for (int v = wide0; v < nvec; v += blockDim.x) {
             const Vec8 y = addend(v);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) ss += y.v[j] * y.v[j];
+            for (int j = 0; j < 8; ++j) ss += LAYER ? y.v[j] : y.v[j] * y.v[j];
         }
-        scale = rsqrtf(block_sum(ss, red[0]) / static_cast<float>(a.width) + a.eps);
+        ss = block_sum(ss, red[0]);
+        if (LAYER) {
+            mean = ss / static_cast<float>(a.width);
+            ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) ss += deviation(add[i], threadIdx.x + i * blockDim.x, mean);
+            for (int v = wide0; v < nvec; v += blockDim.x) ss += deviation(addend(v), v, mean);
+            ss = block_sum(ss, red[LAYER ? 2 : 0]);
+        }
+        scale = rsqrtf(ss / static_cast<float>(a.width) + a.eps);
     }
     float ss2 = 0.f;
 #pragma unroll
     for (int i = 0; i < VEC; ++i) {
         const int v = threadIdx.x + i * blockDim.x;
         if (v >= nvec) continue;
+        Vec8 shift;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) shift.v[j] = 0.f;
+        if (LAYER && add_weight != nullptr) shift = load8(add_bias + v * 8);
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-            val[i].v[j] += add_weight != nullptr ? add[i].v[j] * scale * (w[i].v[j] + a.weight_offset) : add[i].v[j];
-            ss2 += val[i].v[j] * val[i].v[j];
+            if (LAYER) {
+                val[i].v[j] += add_weight != nullptr ? fmaf((add[i].v[j] - mean) * scale, w[i].v[j], shift.v[j]) : add[i].v[j];
+                ss2 += val[i].v[j];
+            } else {
+                val[i].v[j] += add_weight != nullptr ? add[i].v[j] * scale * (w[i].v[j] + a.weight_offset) : add[i].v[j];
+                ss2 += val[i].v[j] * val[i].v[j];
+            }
         }
         store8(res + v * 8, val[i]);
     }
@@ -307,22 +348,50 @@ residual_post_norm_kernel(const PostArgs a) {
         }
         if (!a.init) x = load8(static_cast<const float*>(res) + v * 8);
         if (add_weight != nullptr) g = load8(add_weight + v * 8);
+        if constexpr (LAYER) {
+            Vec8 shift;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            x.v[j] += y.v[j] * scale * (g.v[j] + a.weight_offset);
-            ss2 += x.v[j] * x.v[j];
+            for (int j = 0; j < 8; ++j) shift.v[j] = 0.f;
+            if (add_weight != nullptr) shift = load8(add_bias + v * 8);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                x.v[j] += add_weight != nullptr ? fmaf((y.v[j] - mean) * scale, g.v[j], shift.v[j]) : y.v[j];
+                ss2 += x.v[j];
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                x.v[j] += y.v[j] * scale * (g.v[j] + a.weight_offset);
+                ss2 += x.v[j] * x.v[j];
+            }
         }
         store8(res + v * 8, x);
     }
     float out_scale = 1.f;
-    if (out_weight != nullptr)
-        out_scale = rsqrtf(block_sum(ss2, red[1]) / static_cast<float>(a.width) + a.eps) * a.out_scale;
+    if (out_weight != nullptr) {
+        ss2 = block_sum(ss2, red[1]);
+        if (LAYER) {
+            mean = ss2 / static_cast<float>(a.width);
+            ss2 = 0.f;
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) ss2 += deviation(val[i], threadIdx.x + i * blockDim.x, mean);
+            for (int v = wide0; v < nvec; v += blockDim.x) ss2 += deviation(load8(static_cast<const float*>(res) + v * 8), v, mean);
+            ss2 = block_sum(ss2, red[LAYER ? 3 : 1]);
+        }
+        out_scale = rsqrtf(ss2 / static_cast<float>(a.width) + a.eps) * (LAYER ? 1.f : a.out_scale);
+    }
     T* out = static_cast<T*>(a.out) + t * a.padded;
     auto emit = [&](int v, Vec8 x) {
         if (out_weight != nullptr) {
             const Vec8 g = load8(out_weight + v * 8);
+            if (LAYER) {
+                const Vec8 shift = load8(out_bias + v * 8);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) x.v[j] *= out_scale * (g.v[j] + a.weight_offset);
+                for (int j = 0; j < 8; ++j) x.v[j] = fmaf((x.v[j] - mean) * out_scale, g.v[j], shift.v[j]);
+            } else {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) x.v[j] *= out_scale * (g.v[j] + a.weight_offset);
+            }
         }
         store8(out + v * 8, x);
     };
@@ -334,10 +403,15 @@ residual_post_norm_kernel(const PostArgs a) {
     for (int v = wide0; v < nvec; v += blockDim.x) emit(v, load8(static_cast<const float*>(res) + v * 8));
 }
 
-template <typename T, bool PAIR>
+template <typename T, int KIND>
 auto post_kernel_for(int pieces) {
-    return pieces <= 1 ? residual_post_norm_kernel<T, 1, PAIR>
-                       : pieces <= 2 ? residual_post_norm_kernel<T, 2, PAIR> : residual_post_norm_kernel<T, 4, PAIR>;
+    return pieces <= 1 ? residual_post_norm_kernel<T, 1, KIND>
+                       : pieces <= 2 ? residual_post_norm_kernel<T, 2, KIND> : residual_post_norm_kernel<T, 4, KIND>;
+}
+template <typename T>
+auto post_kernel_for(const ResidualPostNorm& r, int pieces) {
+    return r.layer ? post_kernel_for<T, kLayer>(pieces)
+                   : r.pair_weight != nullptr ? post_kernel_for<T, kPair>(pieces) : post_kernel_for<T, kRms>(pieces);
 }
 
 }  // namespace
@@ -370,10 +444,11 @@ int launch_residual_post_norm(const ResidualPostNorm& r, int dtype, int* status,
     int threads = 32;
     while (threads < 256 && threads * 8 < r.padded) threads *= 2;
     const int pieces = div_ceil(r.padded, threads * 8);
-    const bool f32 = dtype == B200_DTYPE_F32;
-    auto kernel = r.pair_weight != nullptr
-                      ? (f32 ? post_kernel_for<float, true>(pieces) : post_kernel_for<__nv_bfloat16, true>(pieces))
-                      : (f32 ? post_kernel_for<float, false>(pieces) : post_kernel_for<__nv_bfloat16, false>(pieces));
+    a.add_bias = r.add_bias;
+    a.out_bias = r.out_bias;
+    a.self = r.self;
+    a.src_scale = r.init ? r.src_scale : 1.f;
+    auto kernel = dtype == B200_DTYPE_F32 ? post_kernel_for<float>(r, pieces) : post_kernel_for<__nv_bfloat16>(r, pieces);
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(r.tokens), dim3(threads), 0, stream, dim3(1, 1, 1), a));
     return B200_OK;
 }
@@ -467,6 +542,43 @@ int b200_residual_post_norm(void* out, float* residual, const void* src, const i
     r.init = init != 0;
     r.add_weight = add_weight;
     r.out_weight = out_weight;
+    r.tokens = tokens;
+    r.width = width;
+    r.padded = padded;
+    r.eps = eps;
+    return b200::launch_residual_post_norm(r, dtype, status, static_cast<cudaStream_t>(stream));
+}
+
+int b200_residual_layer_norm(void* out, float* residual, const void* src, const int32_t* src_rows,
+                             const float* src_weights, int src_top, int64_t src_count, const void* self, float src_scale,
+                             int init, const void* add_weight, const void* add_bias, const void* out_weight,
+                             const void* out_bias, int tokens, int width, int padded, float eps, int dtype,
+                             b200_stream_t stream) {
+    B200_CHECK_ARG(tokens >= 0 && width > 0 && padded >= width && padded % 64 == 0, "residual_layer_norm: bad shape");
+    B200_CHECK_ARG(dtype == B200_DTYPE_BF16 || dtype == B200_DTYPE_F32, "residual_layer_norm: unknown dtype");
+    B200_CHECK_ARG(src_top >= 1, "residual_layer_norm: bad row count");
+    if (tokens == 0) return B200_OK;
+    B200_CHECK_ARG(out && residual && src && (!add_weight || add_bias) && (!out_weight || out_bias),
+                   "residual_layer_norm: NULL tensor");
+    int err = B200_OK;
+    int* status = b200::device_status_words(&err);
+    if (err != B200_OK) return err;
+    b200::ResidualPostNorm r;
+    r.layer = true;
+    r.out = out;
+    r.residual = residual;
+    r.src = src;
+    r.src_rows = src_rows;
+    r.src_weights = src_weights;
+    r.src_top = src_top;
+    r.src_count = src_count;
+    r.self = self;
+    r.src_scale = src_scale;
+    r.init = init != 0;
+    r.add_weight = add_weight;
+    r.add_bias = add_bias;
+    r.out_weight = out_weight;
+    r.out_bias = out_bias;
     r.tokens = tokens;
     r.width = width;
     r.padded = padded;

@@ -5,6 +5,7 @@
 //   * head_prepare_kernel: between the joint projection and the attention.  One warp per (token, head) row of
 //     the joint output [q heads | k heads | v heads | gate]: queries are normalised and rotated in place, keys
 //     and values go straight into the pools.
+//   * heads that mix their weights run in talking_heads.cu.
 //   * the attention itself: bf16 heads padded to 128 run on the paged kernels of the grouped-query models
 //     (attention_prefill_tc2.cu, attention_decode.cu) with their window; everything else (fp32, wider heads,
 //     head counts those do not take) on the plain kernel below, one CTA per (token, query head).
@@ -35,6 +36,14 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
 }
 
+// A token's position, inside the tables; one outside is reported by the threads with `report`.
+__device__ __forceinline__ int position(const HeadPrepare& a, int64_t t, bool report) {
+    const int pos = a.positions[t];
+    if (pos >= 0 && pos < a.max_pos) return pos;
+    if (report) atomicExch(&a.status[kStatusBadIndex], pos + 1);
+    return min(max(pos, 0), a.max_pos - 1);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kPrepareWarps * 32)
 head_prepare_kernel(const HeadPrepare a) {
@@ -62,6 +71,18 @@ head_prepare_kernel(const HeadPrepare a) {
         T* first = static_cast<T*>(a.first_values) + (t * a.kv_heads + h) * a.vp;
         T* dst = static_cast<T*>(a.v_cache) + (slot * a.kv_heads + h) * a.vp;
         const float lambda = a.mix == HeadPrepare::kMix ? *a.lambda : 0.f;
+        if (a.value_rotary > 0) {
+            const int half = a.value_rotary >> 1, pos = position(a, t, lane == 0);
+            const float* c = a.value_cos + static_cast<int64_t>(pos) * half;
+            const float* s = a.value_sin + static_cast<int64_t>(pos) * half;
+            for (int i = lane; i < half; i += 32) {
+                const float x = to_f32(src[i]), y = to_f32(src[i + half]);
+                dst[i] = from_f32<T>(x * c[i] - y * s[i]);
+                dst[i + half] = from_f32<T>(y * c[i] + x * s[i]);
+            }
+            for (int i = a.value_rotary + lane; i < a.vp; i += 32) dst[i] = src[i];
+            return;
+        }
         for (int i = lane * 4; i < a.vp; i += 128) {
             float4 v = load4(src + i);
             if (a.mix == HeadPrepare::kSave) store4(first + i, v);
@@ -87,7 +108,13 @@ head_prepare_kernel(const HeadPrepare a) {
         ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
         *reinterpret_cast<float4*>(buf + i) = v;
     }
-    if (weight != nullptr) {
+    if (a.unit_norm) {
+        const float scale = rsqrtf(warp_sum(ss) / static_cast<float>(a.dim) + a.eps);
+        for (int i = lane * 4; i < a.dp; i += 128) {
+            const float4 v = *reinterpret_cast<float4*>(buf + i);
+            *reinterpret_cast<float4*>(buf + i) = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
+        }
+    } else if (weight != nullptr) {
         const float scale = rsqrtf(warp_sum(ss) / static_cast<float>(a.dim) + a.eps);
         for (int i = lane * 4; i < a.dp; i += 128) {
             const float4 v = *reinterpret_cast<float4*>(buf + i), w = load4(weight + i);
@@ -96,11 +123,7 @@ head_prepare_kernel(const HeadPrepare a) {
         }
     }
     __syncwarp();
-    int pos = a.positions[t];
-    if (pos < 0 || pos >= a.max_pos) {
-        if (lane == 0) atomicExch(&a.status[kStatusBadIndex], pos + 1);
-        pos = min(max(pos, 0), a.max_pos - 1);
-    }
+    const int pos = position(a, t, lane == 0);
     const int half = a.rotary_dim >> 1;
     const float* c = a.cos_t + static_cast<int64_t>(pos) * half;
     const float* s = a.sin_t + static_cast<int64_t>(pos) * half;
@@ -136,19 +159,26 @@ head_prepare_128_kernel(const HeadPrepare a) {
     const bool turns = e0 < a.rotary_dim;
     const int pair = !turns ? lane : e0 < half ? lane + half / 4 : lane - half / 4;
     const int64_t slot = a.out_loc[t];
-    int pos = a.positions[t];
+    const int pos = position(a, t, threadIdx.x == 0);
     const bool slot_ok = slot >= 0 && slot < a.num_slots;
     if (threadIdx.x == 0 && !slot_ok) atomicExch(&a.status[kStatusBadIndex], static_cast<int>(slot) + 1);
-    if (pos < 0 || pos >= a.max_pos) {
-        if (threadIdx.x == 0) atomicExch(&a.status[kStatusBadIndex], pos + 1);
-        pos = min(max(pos, 0), a.max_pos - 1);
-    }
     float4 c = make_float4(1.f, 1.f, 1.f, 1.f), s = make_float4(0.f, 0.f, 0.f, 0.f);
     if (turns) {
         const int64_t at = static_cast<int64_t>(pos) * half + (e0 < half ? e0 : e0 - half);
         c = load4(a.cos_t + at);
         s = load4(a.sin_t + at);
         if (e0 < half) s = make_float4(-s.x, -s.y, -s.z, -s.w);
+    }
+    // the same for values
+    const int vhalf = a.value_rotary >> 1;
+    const bool vturns = e0 < a.value_rotary;
+    const int vpair = !vturns ? lane : e0 < vhalf ? lane + vhalf / 4 : lane - vhalf / 4;
+    float4 vc = make_float4(1.f, 1.f, 1.f, 1.f), vs = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (vturns) {
+        const int64_t at = static_cast<int64_t>(pos) * vhalf + (e0 < vhalf ? e0 : e0 - vhalf);
+        vc = load4(a.value_cos + at);
+        vs = load4(a.value_sin + at);
+        if (e0 < vhalf) vs = make_float4(-vs.x, -vs.y, -vs.z, -vs.w);
     }
     const float4 one = make_float4(1.f, 1.f, 1.f, 1.f);
     const float4 wq = a.q_weight != nullptr ? load4(static_cast<const T*>(a.q_weight) + e0) : one;
@@ -179,10 +209,18 @@ head_prepare_128_kernel(const HeadPrepare a) {
                     v.z = (1.f - lambda) * v.z + lambda * f.z;
                     v.w = (1.f - lambda) * v.w + lambda * f.w;
                 }
+                if (a.value_rotary > 0) {   // (the whole warp has this row)
+                    float4 o;
+                    o.x = __shfl_sync(0xffffffffu, v.x, vpair);
+                    o.y = __shfl_sync(0xffffffffu, v.y, vpair);
+                    o.z = __shfl_sync(0xffffffffu, v.z, vpair);
+                    o.w = __shfl_sync(0xffffffffu, v.w, vpair);
+                    v = make_float4(v.x * vc.x + o.x * vs.x, v.y * vc.y + o.y * vs.y, v.z * vc.z + o.z * vs.z, v.w * vc.w + o.w * vs.w);
+                }
                 if (slot_ok) store4(static_cast<T*>(a.v_cache) + (slot * a.kv_heads + h) * 128 + e0, v);
                 continue;
             }
-            if ((is_q ? a.q_weight : a.k_weight) != nullptr) {
+            if (a.unit_norm || (is_q ? a.q_weight : a.k_weight) != nullptr) {
                 const float scale =
                     rsqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / static_cast<float>(a.dim) + a.eps);
                 const float4 w = is_q ? wq : wk;
@@ -206,7 +244,8 @@ constexpr int kPlainThreads = 128;
 constexpr int kPlainKeys = 128;     // keys per round
 constexpr int kPlainMaxVec = 8;     // value elements per thread: heads of up to 1024 values
 
-template <typename T>
+// ALL: over the values of all key / value heads, 1024 columns per CTA; the averages themselves go to a.mix.scratch.
+template <typename T, bool ALL>
 __global__ void __launch_bounds__(kPlainThreads)
 window_attention_plain_kernel(const WindowAttention a) {
     extern __shared__ float s_q[];      // the query, dp floats
@@ -225,6 +264,9 @@ window_attention_plain_kernel(const WindowAttention a) {
     const int oldest = len > 0 ? a.window.oldest(len - 1) : 0;
     const int kept = min(a.window.keep_first, oldest);
     const int count = kept + len - oldest;             // keys it sees: [0, kept) and [oldest, len)
+    // this CTA's columns of a slot's row of values
+    const int col0 = ALL ? static_cast<int>(blockIdx.z) * kPlainMaxVec * kPlainThreads : 0;
+    const int cols = ALL ? min(a.kv_heads * a.vp - col0, kPlainMaxVec * kPlainThreads) : a.vp;
     float acc[kPlainMaxVec];
 #pragma unroll
     for (int i = 0; i < kPlainMaxVec; ++i) acc[i] = 0.f;
@@ -274,14 +316,24 @@ window_attention_plain_kernel(const WindowAttention a) {
 #pragma unroll
         for (int i = 0; i < kPlainMaxVec; ++i) acc[i] *= keep;
         for (int j = 0; j < n; ++j) {
-            const T* v = static_cast<const T*>(a.v_cache) + (static_cast<int64_t>(s_slot[j]) * a.kv_heads + g) * a.vp;
+            const T* v = static_cast<const T*>(a.v_cache) + (static_cast<int64_t>(s_slot[j]) * a.kv_heads + (ALL ? 0 : g)) * a.vp + col0;
             const float w = s_p[j];
 #pragma unroll
             for (int i = 0; i < kPlainMaxVec; ++i) {
                 const int c = threadIdx.x + i * kPlainThreads;
-                if (c < a.vp) acc[i] += w * to_f32(v[c]);
+                if (c < cols) acc[i] += w * to_f32(v[c]);
             }
         }
+    }
+    if (ALL) {
+        T* raw = static_cast<T*>(a.mix.scratch) + (t * a.heads + h) * a.kv_heads * a.vp + col0;
+        const float over = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+        for (int i = 0; i < kPlainMaxVec; ++i) {
+            const int c = threadIdx.x + i * kPlainThreads;
+            if (c < cols) raw[c] = from_f32<T>(acc[i] * over);
+        }
+        return;
     }
     T* out = static_cast<T*>(a.out) + t * a.window.out_st + static_cast<int64_t>(h) * a.vp;
     const T* gate = a.window.gate == nullptr ? nullptr : static_cast<const T*>(a.window.gate) + t * a.window.gate_st;
@@ -307,7 +359,7 @@ window_attention_plain_kernel(const WindowAttention a) {
 int launch_head_prepare(const HeadPrepare& a, int dtype, cudaStream_t stream) {
     if (a.tokens == 0) return B200_OK;
     const int64_t rows = static_cast<int64_t>(a.tokens) * (a.heads + 2 * a.kv_heads);
-    if (a.dp == 128 && a.vp == 128 && a.rotary_dim % 8 == 0 && rows >= 4096) {
+    if (a.dp == 128 && a.vp == 128 && a.rotary_dim % 8 == 0 && a.value_rotary % 8 == 0 && rows >= 4096) {
         auto fast = dtype == B200_DTYPE_F32 ? head_prepare_128_kernel<float> : head_prepare_128_kernel<__nv_bfloat16>;
         B200_CHECK_CUDA(launch_kernel(fast, dim3(a.tokens), dim3(kPrepareWarps * 32), 0, stream, dim3(1, 1, 1), a));
         return B200_OK;
@@ -327,8 +379,16 @@ bool window_attention_tc_supported(const WindowAttention& a, int dtype) {
     return (group & (group - 1)) == 0;
 }
 
+int launch_plain_all_values(const WindowAttention& a, int dtype, cudaStream_t stream) {
+    auto kernel = dtype == B200_DTYPE_F32 ? window_attention_plain_kernel<float, true> : window_attention_plain_kernel<__nv_bfloat16, true>;
+    const dim3 grid(a.tokens, a.heads, div_ceil(a.kv_heads * a.vp, kPlainMaxVec * kPlainThreads));
+    B200_CHECK_CUDA(launch_kernel(kernel, grid, dim3(kPlainThreads), static_cast<size_t>(a.dp) * 4, stream, dim3(1, 1, 1), a));
+    return B200_OK;
+}
+
 int launch_window_attention(const WindowAttention& a, int dtype, cudaStream_t stream) {
     if (a.tokens == 0) return B200_OK;
+    if (a.mix.weights != nullptr) return launch_talking_heads(a, dtype, stream);
     if (window_attention_tc_supported(a, dtype)) {
         if (!a.decode)
             return launch_attention_prefill_tc2(a.out, a.q, a.q_st, a.dp, a.k_cache, a.v_cache, a.num_slots, a.page_table,
@@ -345,7 +405,7 @@ int launch_window_attention(const WindowAttention& a, int dtype, cudaStream_t st
     }
     WindowAttention plain = a;
     if (plain.window.out_st == 0) plain.window.out_st = static_cast<int64_t>(a.heads) * a.vp;
-    auto kernel = dtype == B200_DTYPE_F32 ? window_attention_plain_kernel<float> : window_attention_plain_kernel<__nv_bfloat16>;
+    auto kernel = dtype == B200_DTYPE_F32 ? window_attention_plain_kernel<float, false> : window_attention_plain_kernel<__nv_bfloat16, false>;
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(a.tokens, a.heads), dim3(kPlainThreads), static_cast<size_t>(a.dp) * 4, stream,
                                   dim3(1, 1, 1), plain));
     return B200_OK;
@@ -364,6 +424,8 @@ int b200_head_prepare(const b200_head_prepare_args* p, int dtype, b200_stream_t 
     B200_CHECK_ARG(p->rotary_dim >= 0 && p->rotary_dim % 2 == 0 && p->rotary_dim <= p->dim, "head_prepare: bad rotary_dim");
     B200_CHECK_ARG(p->mix >= 0 && p->mix <= 2 && (p->mix == 0 || p->first_values) && (p->mix != 2 || p->lambda),
                    "head_prepare: bad value mixing");
+    B200_CHECK_ARG(p->value_rotary >= 0 && p->value_rotary % 2 == 0 && p->value_rotary <= p->padded_value_dim &&
+                       (p->value_rotary == 0 || (p->mix == 0 && p->value_cos && p->value_sin)), "head_prepare: bad value rotation");
     if (p->tokens == 0) return B200_OK;
     B200_CHECK_ARG(p->joint && p->positions && p->out_loc && p->k_cache && p->v_cache && p->cos_table && p->sin_table,
                    "head_prepare: NULL tensor");
@@ -394,6 +456,10 @@ int b200_head_prepare(const b200_head_prepare_args* p, int dtype, b200_stream_t 
     a.mix = p->mix;
     a.lambda = p->lambda;
     a.first_values = p->first_values;
+    a.unit_norm = p->unit_norm != 0;
+    a.value_rotary = p->value_rotary;
+    a.value_cos = p->value_cos;
+    a.value_sin = p->value_sin;
     return b200::launch_head_prepare(a, dtype, static_cast<cudaStream_t>(stream));
 }
 
@@ -451,6 +517,20 @@ int b200_window_attention(const b200_window_attention_args* p, int dtype, b200_s
     a.window.out_st = p->out_stride;
     a.workspace = p->workspace;
     a.workspace_bytes = p->workspace_bytes;
+    if (p->head_mix != nullptr) {
+        B200_CHECK_ARG(p->mix_scratch && !p->sinks && p->value_rotary >= 0 && p->value_rotary % 2 == 0 &&
+                           p->value_rotary <= p->padded_value_dim, "window_attention: bad head mixing");
+        B200_CHECK_ARG(p->value_rotary == 0 || (p->value_cos && p->value_sin && p->positions && p->max_pos > 0),
+                       "window_attention: NULL rotation");
+        a.mix.weights = p->head_mix;
+        a.mix.rotary = p->value_rotary;
+        a.mix.max_pos = p->max_pos;
+        a.mix.cos_t = p->value_cos;
+        a.mix.sin_t = p->value_sin;
+        a.mix.positions = p->positions;
+        a.mix.score_bound = p->score_bound;
+        a.mix.scratch = p->mix_scratch;
+    }
     return b200::launch_window_attention(a, dtype, static_cast<cudaStream_t>(stream));
 }
 

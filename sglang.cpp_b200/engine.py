@@ -115,7 +115,7 @@ class Engine:
         st = _lib.StackConfigStruct(len(model_config.layers), layers,
                                     _lib.DTYPE_F32 if self.dtype == torch.float32 else _lib.DTYPE_BF16,
                                     model_config.norm_offset, model_config.logit_scale, int(model_config.norm_output),
-                                    len(pairs), beside)
+                                    len(pairs), beside, int(model_config.norm_kind), model_config.embed_scale)
         call("b200_engine_create_stack", ctypes.byref(m), ctypes.byref(st), ctypes.byref(c), ctypes.byref(self._h))
 
     def close(self) -> None:

@@ -5,7 +5,7 @@
 
 * ``ModelConfig``: one layer repeated (Llama, Qwen2, Qwen3, Qwen3-MoE; the fields of
   include/sglang/models/config.h:15-42);
-* ``StackConfig``: layers listed one by one (Rapizen, Dilalix, Saluzen).  Each is a ``LayerSpec`` that names its mixer and
+* ``StackConfig``: layers listed one by one (Rapizen, Dilalix, Saluzen, Retotar).  Each is a ``LayerSpec`` that names its mixer and
   its feed-forward with their sizes; another design made of the same parts needs a reader here (and a
   packing in ``weights.py`` where its tensors are named differently).
 
@@ -84,22 +84,30 @@ class LayerSpec:
     act_limit: float = 0.0
     shared_act_limit: float = 0.0
     # window attention
-    head_norm: bool = True
+    head_norm: int = _lib.HEAD_NORM_WEIGHTED
     gate: int = _lib.GATE_ELEMENT
     qkv_bias: bool = False
     sink: bool = False            # a score per head in the softmax's denominator ...
     sink_learned: bool = True     # ... from the checkpoint, or 0
     chunk: int = 0                # keys of the query's own chunk, instead of a window
-    # rotations whose long wavelengths are stretched; latent attention counts its rotary_dim rotated dimensions in
+    # rotations whose long wavelengths are stretched (or, with rope_original 0, all of them); latent attention counts its rotary_dim rotated dimensions in
     # head_dim
     rope_factor: float = 0.0
     rope_low: float = 1.0
     rope_high: float = 1.0
     rope_original: float = 0.0
-    kv_from: int = -1             # latent attention: the layer whose latents are read
+    kv_from: int = -1             # latent and window attention: the layer whose cache is read
     # recurrences: head_dim state rows, kv_heads heads of k and q
     conv_taps: int = 1
     norm_groups: int = 1
+    # window attention: cached values turn with their position, the output turns back; heads mix their weights
+    value_rotary: bool = False
+    head_mix: bool = False
+    gate_cap: float = 0.0         # matrix memory
+    # scored experts: by sigmoid or softmax scores; experts that return their input
+    score: int = _lib.SCORE_SIGMOID
+    identity_experts: int = 0
+    decays: tuple = ()            # lightning: one per head
     # a second mixer on the same input, and how the results meet
     beside: Optional["LayerSpec"] = None
     join: int = _lib.JOIN_SUM
@@ -107,7 +115,7 @@ class LayerSpec:
 
     def as_struct(self) -> _lib.LayerConfigStruct:
         """(``beside`` becomes an index once the whole stack is known: Engine.)"""
-        values = {f.name: getattr(self, f.name) for f in fields(self) if f.name not in ("beside", "sink_learned")}
+        values = {f.name: getattr(self, f.name) for f in fields(self) if f.name not in ("beside", "sink_learned", "decays")}
         return _lib.LayerConfigStruct(beside=-1, **{k: int(v) if isinstance(v, bool) else v for k, v in values.items()})
 
 
@@ -122,6 +130,8 @@ class StackConfig:
     norm_output: int = _lib.NORM_INPUT   # norms on what the blocks read, on what they return, or on both
     tie_word_embeddings: bool = False
     torch_dtype: torch.dtype = torch.bfloat16
+    norm_kind: int = _lib.NORM_RMS       # RMS norms, or layer norms with biases
+    embed_scale: float = 1.0
 
     @property
     def num_layers(self) -> int:
@@ -129,7 +139,8 @@ class StackConfig:
 
     @property
     def carries_state(self) -> bool:
-        kinds = (_lib.MIXER_LINEAR_ATTENTION, _lib.MIXER_STATE_SPACE, _lib.MIXER_DELTA_RULE)
+        kinds = (_lib.MIXER_LINEAR_ATTENTION, _lib.MIXER_STATE_SPACE, _lib.MIXER_DELTA_RULE, _lib.MIXER_LIGHTNING,
+                 _lib.MIXER_MATRIX_MEMORY)
         return any(m is not None and m.mixer in kinds for c in self.layers for m in (c, c.beside))
 
     def expands_keys(self, c: LayerSpec) -> bool:
@@ -220,7 +231,7 @@ def _set_rotation(spec: LayerSpec, rot: dict) -> None:
 def _biased_attention(m: dict) -> LayerSpec:
     """Grouped-query attention with projection biases and a sink, without norms on queries and keys."""
     spec = LayerSpec(m["heads"], m["dim"], m["vdim"], score_scale=float(m["scale"]), mixer=_lib.MIXER_WINDOW_ATTENTION,
-                     kv_heads=m["kv_heads"], head_norm=False, qkv_bias=True, sink=True)
+                     kv_heads=m["kv_heads"], head_norm=_lib.HEAD_NORM_NONE, qkv_bias=True, sink=True)
     _set_rotation(spec, m["rot"])
     return spec
 
@@ -264,6 +275,49 @@ def read_saluzen(c: dict, shapes: Optional[dict] = None) -> StackConfig:
     return StackConfig(c["width"], c["vocab"], float(c["norm"]["eps"]), layers, norm_output=_lib.NORM_BOTH)
 
 
+def _talking_attention(m: dict) -> LayerSpec:
+    rot, mask = m.get("rot") or {}, m.get("mask") or {}
+    spec = LayerSpec(m["heads"], m["dim"], m["vdim"], score_scale=float(m["scale"]), mixer=_lib.MIXER_WINDOW_ATTENTION,
+                     kv_heads=m["kv_heads"], head_norm=_lib.HEAD_NORM_UNIT, value_rotary=True, head_mix=True)
+    spec.window = min(mask.get("size", NO_WINDOW), NO_WINDOW)
+    spec.rotary_dim, spec.rope_base = rot.get("dims", 0), float(rot.get("base", 1.0))
+    if rot.get("scaling"):
+        spec.rope_factor = float(rot["scaling"]["factor"])
+    if m.get("kv_from") is not None:
+        spec.kv_from = m["kv_from"]
+    return spec
+
+
+def read_retotar(c: dict, shapes: Optional[dict] = None) -> StackConfig:
+    layers = []
+    for i, entry in enumerate(c["layers"]):
+        m = entry["mixer"]
+        if entry["type"] == "attention":
+            spec = _talking_attention(m)
+        elif entry["type"] == "lightning":
+            if len(m["decay"]) != m["heads"]:
+                raise ValueError(f"layer {i}: {len(m['decay'])} decays for {m['heads']} heads")
+            spec = LayerSpec(m["heads"], m["dim"], m["vdim"], mixer=_lib.MIXER_LIGHTNING, kv_heads=m["heads"], norm_groups=1,
+                             decays=tuple(map(float, m["decay"])))
+        elif entry["type"] == "mlstm":
+            spec = LayerSpec(m["heads"], m["dim"], m["vdim"], mixer=_lib.MIXER_MATRIX_MEMORY, kv_heads=m["heads"],
+                             norm_groups=m["heads"], gate_cap=float(m["gate_cap"]))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {entry['type']!r}")
+        ff = entry.get("mlp")
+        if ff is not None:
+            if ff["kind"] != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward {ff['kind']!r}")
+            r, groups = ff["router"], ff["router"].get("groups") or {}
+            spec.mlp, spec.intermediate, spec.epilogue = _lib.MLP_SCORED_MOE, ff["expert"]["ff"], _lib.EPILOGUE_SWIGLU
+            spec.score, spec.num_experts, spec.identity_experts = _lib.SCORE_SOFTMAX, r["experts"], r.get("identity", 0)
+            spec.experts_per_tok = r["top"]
+            spec.router_groups, spec.router_keep = groups.get("count", 1), groups.get("keep", groups.get("count", 1))
+        layers.append(spec)
+    return StackConfig(c["width"], c["vocab"], float(c["norm"]["eps"]), layers, norm_output=_lib.NORM_BOTH,
+                       norm_kind=_lib.NORM_LAYER, embed_scale=float((c.get("embedding") or {}).get("scale", 1.0)))
+
+
 REGISTRY: dict[str, Callable] = {
     "LlamaForCausalLM": _uniform(qk_norm=False, fused_residual=False),
     "Qwen2ForCausalLM": _uniform(qk_norm=False, fused_residual=False, attention_bias=True),
@@ -272,6 +326,7 @@ REGISTRY: dict[str, Callable] = {
     "Rapizen": read_rapizen,
     "Dilalix": read_dilalix,
     "Saluzen": read_saluzen,
+    "Retotar": read_retotar,
 }
 
 

@@ -15,6 +15,7 @@ Models whose layers are listed one by one (``models.StackConfig``) have a packin
 from __future__ import annotations
 
 import json
+import math
 import re
 import struct
 from pathlib import Path
@@ -170,9 +171,9 @@ def unpack_checkpoint(cfg, w: dict) -> dict:
 def pack_layer_stack(cfg, tensors: dict) -> dict:
     """Parameter names of the layer-stack designs -> the padded layouts of ``b200_engine_create_stack``, in
     the dtype the model runs in.  Every tensor is checked against the shape its layer's description asks for."""
-    from ._lib import (GATE_ELEMENT, GATE_HEAD, JOIN_NORMED, MIXER_DELTA_RULE, MIXER_LATENT_ATTENTION, MIXER_LINEAR_ATTENTION,
-                       MIXER_STATE_SPACE, MIXER_WINDOW_ATTENTION, MLP_DENSE, MLP_NONE, MLP_SCORED_MOE, NORM_BOTH,
-                       epilogue_is_gated, load)
+    from ._lib import (GATE_ELEMENT, GATE_HEAD, HEAD_NORM_WEIGHTED, JOIN_NORMED, MIXER_DELTA_RULE, MIXER_LATENT_ATTENTION,
+                       MIXER_LIGHTNING, MIXER_LINEAR_ATTENTION, MIXER_MATRIX_MEMORY, MIXER_STATE_SPACE, MIXER_WINDOW_ATTENTION,
+                       MLP_DENSE, MLP_NONE, MLP_SCORED_MOE, NORM_BOTH, NORM_LAYER, SCORE_SOFTMAX, epilogue_is_gated, load)
 
     lib = load()
     width, head, latent = lib.b200_pad_width, lib.b200_pad_head_dim, lib.b200_pad_latent
@@ -192,7 +193,14 @@ def pack_layer_stack(cfg, tensors: dict) -> dict:
         out[tuple(slice(0, n) for n in t.shape)] = t
         return out
 
-    w = {"embed": pad(need("embed", V, D), width(V), hp), "final_norm": pad(need("final.norm", D), hp), "layers": []}
+    def norm(name, to):
+        """A norm's weight, and under layer norms its bias."""
+        out = {to: pad(need(name, D), hp)}
+        if cfg.norm_kind == NORM_LAYER:
+            out[to + "_bias"] = pad(need(name + ".b", D), hp)
+        return out
+
+    w = {"embed": pad(need("embed", V, D), width(V), hp), **norm("final.norm", "final_norm"), "layers": []}
     if not cfg.tie_word_embeddings:
         w["lm_head"] = pad(need("head", V, D), width(V), hp)
     def rows(name, n, to, k=D, kp=hp):
@@ -229,7 +237,7 @@ def pack_layer_stack(cfg, tensors: dict) -> dict:
     def window_attention(m, c):
         H, G, d, dv = c.heads, c.kv_heads, c.head_dim, c.value_dim
         dp, vp = head(d), head(dv)
-        parts = [("q", H, d, dp), ("k", G, d, dp), ("v", G, dv, vp)]
+        parts = [("q", H, d, dp), ("k", G, d, dp), ("v", G, dv, vp)][:3 if c.kv_from < 0 else 1]
         joint = [head_rows(m + name, n, k, kp) for name, n, k, kp in parts]
         if c.gate == GATE_ELEMENT:
             joint.append(head_rows(m + "g", H, dv, vp))
@@ -239,8 +247,10 @@ def pack_layer_stack(cfg, tensors: dict) -> dict:
         if c.qkv_bias:
             bias = torch.cat([pad(need(f"{m}{name}.b", n * k).view(n, k), n, kp).flatten() for name, n, k, kp in parts])
             bias = pad(bias, len(joint))
-        if c.head_norm:
+        if c.head_norm == HEAD_NORM_WEIGHTED:
             L.update(q_head_norm=pad(need(m + "q.norm", d), dp), k_head_norm=pad(need(m + "k.norm", d), dp))
+        if c.head_mix or c.value_rotary:
+            L["head_mix"] = need(m + "talk", H, H, dtype=torch.float32) if c.head_mix else torch.eye(H)
         if c.value_mix:
             L["value_mix"] = need(m + "vmix", dtype=torch.float32).reshape(1)
         if c.sink:
@@ -289,13 +299,32 @@ def pack_layer_stack(cfg, tensors: dict) -> dict:
              "step_bias": need(m + "dt_bias", H, **f32), "head_norm": pad(need(m + "norm", dv), vp)}
         return joint, None, L, vp
 
+    def head_channels(m, c, vp):
+        """Gate, values, keys and queries of a recurrence whose heads all have their own."""
+        H, d, dv, dp = c.heads, c.head_dim, c.value_dim, width(c.head_dim)
+        return [head_rows(m + name, H, n, to) for name, n, to in (("g", dv, vp), ("v", dv, vp), ("k", d, dp), ("q", d, dp))]
+
+    def lightning(m, c):
+        H, dv, vp = c.heads, c.value_dim, width(c.value_dim)
+        # (a decay of 0 as one that leaves nothing in fp32)
+        decay = torch.tensor([max(math.log(g), -250.0) if g > 0 else -250.0 for g in c.decays])
+        L = {"decay_log": decay, "head_norm": by_head(need(m + "norm", H * dv), H, dv, vp)}
+        return torch.cat(head_channels(m, c, vp)), None, L, vp
+
+    def matrix_memory(m, c):
+        H, dv, vp = c.heads, c.value_dim, width(c.value_dim)
+        gates = torch.cat([need(m + "i", H, D), need(m + "f", H, D)])
+        L = {"step_bias": torch.cat([need(m + name, H, dtype=torch.float32) for name in ("i.b", "f.b")]),
+             "head_norm": by_head(need(m + "norm", H * dv), H, dv, vp)}
+        return torch.cat(head_channels(m, c, vp) + [pad(gates, width(2 * H), hp)]), None, L, vp
+
     def output(m, c, vp):
         return pad(need(m + "o", D, c.heads * c.value_dim).view(D, c.heads, c.value_dim), hp, c.heads, vp)
 
     joint_names = {MIXER_WINDOW_ATTENTION: "qkvg", MIXER_LINEAR_ATTENTION: "qkvga", MIXER_STATE_SPACE: "recurrence",
-                   MIXER_DELTA_RULE: "recurrence"}
+                   MIXER_DELTA_RULE: "recurrence", MIXER_LIGHTNING: "recurrence", MIXER_MATRIX_MEMORY: "recurrence"}
     mixers = {MIXER_WINDOW_ATTENTION: window_attention, MIXER_LINEAR_ATTENTION: linear_attention, MIXER_STATE_SPACE: state_space,
-              MIXER_DELTA_RULE: delta_rule}
+              MIXER_DELTA_RULE: delta_rule, MIXER_LIGHTNING: lightning, MIXER_MATRIX_MEMORY: matrix_memory}
 
     def one_mixer(m, c):
         if c.mixer == MIXER_LATENT_ATTENTION:
@@ -333,7 +362,10 @@ def pack_layer_stack(cfg, tensors: dict) -> dict:
         L = {"mlp_up": torch.stack([up_matrix(e, I, ip, gated) for e in experts]),
              "mlp_down": torch.stack([rows(e + "down", D, hp, I, ip) for e in experts])}
         if c.mlp == MLP_SCORED_MOE:
-            L["router"] = rows(f + "router", c.num_experts, width(c.num_experts))
+            outputs = c.num_experts + c.identity_experts
+            L["router"] = rows(f + "router", outputs, width(outputs))
+            if c.score == SCORE_SOFTMAX:
+                L["router_correction"] = need(f + "correction", outputs, dtype=torch.float32)
             if c.shared_intermediate:
                 n, np_ = c.shared_intermediate, width(c.shared_intermediate)
                 L["shared_up"] = up_matrix(f + "shared.", n, np_, gated)
@@ -348,13 +380,13 @@ def pack_layer_stack(cfg, tensors: dict) -> dict:
     for i, c in enumerate(cfg.layers):
         p = f"l{i}."
         L = one_mixer(p + "mix.", c) if c.beside is None else two_mixers(p + "mix.", c)
-        L["norm1"] = pad(need(p + "norm1", D), hp)
+        L.update(norm(p + "norm1", "norm1"))
         if cfg.norm_output == NORM_BOTH:
-            L["norm1_out"] = pad(need(p + "norm1b", D), hp)
+            L.update(norm(p + "norm1b", "norm1_out"))
         if c.mlp != MLP_NONE:
-            L["norm2"] = pad(need(p + "norm2", D), hp)
+            L.update(norm(p + "norm2", "norm2"))
             if cfg.norm_output == NORM_BOTH:
-                L["norm2_out"] = pad(need(p + "norm2b", D), hp)
+                L.update(norm(p + "norm2b", "norm2_out"))
             L.update(feed_forward(p + "mlp.", c))
         w["layers"].append(L)
     return w

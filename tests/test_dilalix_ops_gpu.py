@@ -409,7 +409,7 @@ def test_scored_routing(call, tokens, experts, top, groups, keep):
     weights, counts, off = torch.zeros(tokens, top, device="cuda"), torch.zeros(2 * experts, **i32), torch.zeros(experts + 1, **i32)
     xp = torch.zeros(tokens * top, 64, dtype=torch.bfloat16, device="cuda")
     call("b200_score_route", ids.data_ptr(), weights.data_ptr(), rows.data_ptr(), counts.data_ptr(), off.data_ptr(), xp.data_ptr(),
-         x.data_ptr(), 128, logits.data_ptr(), ld, tokens, experts, top, groups, keep, 1.7, stream())
+         x.data_ptr(), 128, logits.data_ptr(), ld, tokens, experts, top, groups, keep, 1.7, 0, 0, None, stream())
     torch.cuda.synchronize()
     want_ids, want_w = O.choose_experts(torch.sigmoid(logits[:, :experts].cpu().double()), top, groups, keep, 1.7)
     order, want_order = ids.cpu().long().sort(1), want_ids.sort(1)
