@@ -27,7 +27,7 @@ of 4096 tokens prefilled in chunks, alternating with sampled decode steps of 56 
 prefill tokens/s, decode ms/step, fraction of the tensor-pipe rate); --workload c4 is Llama-3-8B under tensor parallelism and
 --workload c5 Qwen3-30B-A3B under expert parallelism + attention TP over the N ranks (strong
 scaling, weights drawn on the device); --workload rapizen is prefill and decode of the layer-stack
-design Rapizen at three sizes beside Qwen3-MoE of the same sizes, --workload dilalix that of Dilalix, --workload saluzen that of Saluzen beside Qwen3; --eager / --profile-region / --profile-prefill shape a run
+design Rapizen at three sizes beside Qwen3-MoE of the same sizes, --workload dilalix that of Dilalix, --workload saluzen that of Saluzen beside Qwen3, --workload retotar that of Retotar beside Qwen3-MoE; --eager / --profile-region / --profile-prefill shape a run
 for a profiler's launch list.
 """
 from __future__ import annotations
@@ -1051,6 +1051,100 @@ def run_gpu_saluzen(args):
         "sizes": sizes}))
 
 
+# name -> (width, layers, heads, KV heads, experts, top, expert width, window, batch, context); layers in turn: attention whose
+# heads mix (every other one on the keys and values of the one before it), lightning attention, matrix memory
+RETOTAR_SIZES = {
+    "1k": (1024, 12, 8, 2, 32, 2, 1024, 1024, 64, 2048),
+    "2k": (2048, 12, 16, 4, 64, 4, 1024, 1024, 64, 2048),
+    "4k": (4096, 9, 32, 8, 32, 2, 2048, 1024, 64, 2048),
+}
+
+
+def retotar_pair(size: str):
+    """A Retotar model (a quarter as many identity experts as experts) and a Qwen3-MoE model of the same width, depth,
+    heads and experts."""
+    from oracle import token_loop_oracle as O
+    from sglang_cpp_b200 import _lib
+    from sglang_cpp_b200.models import LayerSpec, StackConfig
+
+    D, L, H, G, E, top, ff, window, _, _ = RETOTAR_SIZES[size]
+    layers = []
+    for i in range(L):
+        if i % 3 == 0:
+            s = LayerSpec(H, 128, 128, score_scale=128 ** -0.5, mixer=_lib.MIXER_WINDOW_ATTENTION, kv_heads=G, window=window,
+                          rotary_dim=64, rope_base=1e6, rope_factor=4.0, head_norm=_lib.HEAD_NORM_UNIT, value_rotary=True,
+                          head_mix=True, kv_from=i - 3 if i % 6 == 3 else -1)
+        elif i % 3 == 1:
+            s = LayerSpec(H, 128, 128, mixer=_lib.MIXER_LIGHTNING, kv_heads=H,
+                          decays=tuple(1 - 2.0 ** (-1 - 9 * h / H) for h in range(H)))
+        else:
+            s = LayerSpec(H, 128, 128, mixer=_lib.MIXER_MATRIX_MEMORY, kv_heads=H, norm_groups=H, gate_cap=15.0)
+        s.mlp, s.intermediate, s.epilogue = _lib.MLP_SCORED_MOE, ff, _lib.EPILOGUE_SWIGLU
+        s.score, s.num_experts, s.identity_experts, s.experts_per_tok = _lib.SCORE_SOFTMAX, E, E // 4, top
+        s.router_groups, s.router_keep = 5, 4
+        layers.append(s)
+    new = StackConfig(D, RAPIZEN_VOCAB, 1e-6, layers, norm_output=_lib.NORM_BOTH, norm_kind=_lib.NORM_LAYER, embed_scale=0.5)
+    like = O.ModelConfig(L, D, H, G, 128, 4 * D, RAPIZEN_VOCAB, 1e-6, 1e6, 8192, False, True, True, "silu", E, top, ff, True)
+    return new, like
+
+
+def retotar_work(size: str, new: bool) -> dict:
+    D, L, H, G, E, top, ff, window, B, ctx = RETOTAR_SIZES[size]
+    outputs = E + (E // 4 if new else 0)
+    hit, used = E * (1 - (1 - top / outputs) ** B), top * E / outputs     # experts a step reads, and a token uses
+    kv_tok, attn_w = 2 * G * 128 * 2, D * (H + 2 * G) * 128 + H * 128 * D
+    experts = lambda n: L * (n * 3 * ff * D + D * outputs)
+    if not new:
+        return {"batch": B, "context": ctx, "vocab": RAPIZEN_VOCAB, "layers": L,
+                "step_bytes": lambda keys: 2 * (L * attn_w + experts(hit) + RAPIZEN_VOCAB * D) + L * B * keys * kv_tok,
+                "attention_bytes": lambda keys: B * keys * kv_tok,
+                "flops_tok": 2 * (L * attn_w + experts(used)) + L * 4 * H * 128 * ctx / 2,
+                "attention_flops_req": 4 * H * 128 * ctx * ctx / 2}
+    n_attn, n_rec = sum(i % 3 == 0 for i in range(L)), sum(i % 3 > 0 for i in range(L))
+    n_shared = sum(i % 6 == 3 for i in range(L))
+    matrices = n_attn * (attn_w + D * H * 128) - n_shared * D * 2 * G * 128 + n_rec * 5 * D * H * 128
+    state = 2 * H * 128 * 128 * 4                                    # read and written per token decoded
+    seen = lambda keys: min(keys, window)
+    pairs = window * ctx - window * window / 2                       # (query, key) pairs of a prompt
+    return {"batch": B, "context": ctx, "vocab": RAPIZEN_VOCAB, "layers": L,
+            "step_bytes": lambda keys: 2 * (matrices + experts(hit) + RAPIZEN_VOCAB * D) + B * (n_attn * seen(keys) * kv_tok + n_rec * state),
+            "attention_bytes": lambda keys: B * seen(keys) * kv_tok,
+            # attention: scores, mixed weights, values; recurrences: scores and state of chunks of 64
+            "flops_tok": 2 * (matrices + experts(used)) + n_attn * (4 * 128 + 2 * H) * H * pairs / ctx
+            + n_rec * H * (4 * 128 * 128 + 4 * 128 * 32),
+            "attention_flops_req": 4 * H * 128 * pairs}
+
+
+def run_gpu_retotar(args):
+    """Workload "retotar": prefill and decode of the Retotar design at sizes that resemble a real model's layers, beside
+    Qwen3-MoE of the same size.  (attention_us covers the attention layers only; its floating-point operations are those of
+    scores and values, as if heads did not mix.)"""
+    import __graft_entry__ as entry
+
+    torch.cuda.set_device(0)
+    pkg = entry.load_package()
+    pkg.load_library()
+    sampler = ClockSampler(0)
+    sampler.start()
+    sizes = {}
+    for size in (args.size.split(",") if args.size else RETOTAR_SIZES):
+        new, like = retotar_pair(size)
+        sizes[size] = {"retotar": stack_arm(pkg, new, retotar_work(size, True), args.steps, args.warmup)}
+        if not args.new_only:
+            sizes[size]["qwen3-moe"] = stack_arm(pkg, like, retotar_work(size, False), args.steps, args.warmup)
+    clocks = sampler.stop()
+    first = next(iter(sizes))
+    print(json.dumps({
+        "metric": "decode tokens/s (Retotar layer stack, %s)" % first, "value": sizes[first]["retotar"]["decode_tokens_s"],
+        "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+        "ms_per_step": sizes[first]["retotar"]["decode_ms"], "higher_is_better": True, "scaling": "strong",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "clocks": clocks,
+        "config": {"workload": "retotar: batch 64, context 2048, page 64; weights and caches larger than L2",
+                   "sizes": {k: dict(zip(("width", "layers", "heads", "kv_heads", "experts", "top", "expert_width", "window", "batch",
+                                          "context"), RETOTAR_SIZES[k])) for k in sizes}},
+        "sizes": sizes}))
+
+
 def run_gpu_dilalix(args):
     """Workload "dilalix": prefill and decode of the Dilalix design at sizes that resemble a real model's
     layers, beside Qwen3-MoE of the same size.  (attention_us covers the window attention layers only.)"""
@@ -1199,15 +1293,15 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--chunk-tokens", type=int, default=2048, help="c3: tokens a prompt advances per prefill batch")
-    ap.add_argument("--workload", default="c2", choices=["c2", "c3", "c4", "c5", "rapizen", "dilalix", "saluzen"],
+    ap.add_argument("--workload", default="c2", choices=["c2", "c3", "c4", "c5", "rapizen", "dilalix", "saluzen", "retotar"],
                     help="c2 (default, the headline metric): Qwen3-0.6B decode, replicas when N > 1; "
                          "c3: Qwen3-0.6B chunked prefill alternating with sampled decode, one GPU; "
                          "c4: Llama-3-8B decode, tensor parallel over the N ranks; "
                          "c5: Qwen3-30B-A3B decode, experts and attention heads split over the N ranks")
     ap.add_argument("--context", type=int, default=0,
                     help="c2 only: give every prompt this length instead of U[512,2048]")
-    ap.add_argument("--size", default="", help="rapizen, dilalix, saluzen: sizes to run, with commas between them (default: all)")
-    ap.add_argument("--new-only", action="store_true", help="dilalix, saluzen: without the model it is measured beside")
+    ap.add_argument("--size", default="", help="rapizen, dilalix, saluzen, retotar: sizes to run, with commas between them (default: all)")
+    ap.add_argument("--new-only", action="store_true", help="dilalix, saluzen, retotar: without the model it is measured beside")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-tp-record", action="store_true",
                     help="c2 only: do not run the tensor-parallel workload after the headline")
@@ -1235,6 +1329,10 @@ def main():
         if args.gpus != 1:
             raise SystemExit("workload dilalix runs on one GPU")
         run_gpu_dilalix(args)
+    elif args.workload == "retotar":
+        if args.gpus != 1:
+            raise SystemExit("workload retotar runs on one GPU")
+        run_gpu_retotar(args)
     elif args.workload == "saluzen":
         if args.gpus != 1:
             raise SystemExit("workload saluzen runs on one GPU")

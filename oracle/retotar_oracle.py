@@ -200,3 +200,106 @@ def forward(config, weights, tokens, dtype=torch.float64, keep_layers=False):
         trail.append(x)
     logits = norm(x, "final.norm") @ w["head"].T
     return (logits, trail) if keep_layers else logits
+
+
+# ---- random models -------------------------------------------------------------------
+ROUTER_GAIN = 4.0
+
+
+def _clear_choice(codes, correction, r, gap=0.02):
+    """Of which codes [n, outputs] is no choice of this router close, however much the norm in front of it shrinks them?"""
+    outputs, groups = r["experts"] + r.get("identity", 0), r.get("groups") or {"count": 1, "keep": 1}
+    count, keep, top = groups["count"], groups["keep"], r["top"]
+    shrink = torch.linspace(0.2, 1.0, 17)[:, None, None]
+    s = torch.softmax(ROUTER_GAIN * shrink * codes[:, :outputs], -1) + correction
+    parts = s.view(*s.shape[:2], count, -1)
+    best = parts.max(-1).values.sort(descending=True)
+    clear = torch.ones(s.shape[:2], dtype=torch.bool)
+    if keep < count:
+        clear &= best.values[..., keep - 1] - best.values[..., keep] >= gap
+    kept = best.indices[..., :keep, None].expand(*s.shape[:2], keep, parts.shape[-1])
+    left = parts.gather(2, kept).flatten(2).sort(descending=True).values
+    if top < left.shape[-1]:
+        clear &= left[..., top - 1] - left[..., top] >= gap
+    return clear.all(0)
+
+
+def random_model(config, seed=0, coded_router=True):
+    """bf16 weights of the shapes `config` describes, scaled so that every mechanism contributes to the logits.
+
+    With `coded_router` the first columns of the residual stream hold a code of the token that the blocks hardly
+    touch, and the routers read mostly that: no choice of experts is close, so runs in different precisions choose
+    alike.  Without it the routers are random matrices."""
+    g = torch.Generator().manual_seed(seed)
+    V, D = config["vocab"], config["width"]
+    w = {}
+
+    def mat(name, n, k, gain=1.0):
+        w[name] = (torch.randn(n, k, generator=g) * gain / math.sqrt(k)).to(torch.bfloat16)
+
+    def vec(name, n, centre=1.0, spread=0.2):
+        w[name] = (centre + spread * torch.randn(n, generator=g)).to(torch.bfloat16)
+
+    def norm(name, code, code_gain=1.0):
+        vec(name, D)
+        vec(name + ".b", D, 0.0, 0.2)
+        w[name][:code], w[name + ".b"][:code] = code_gain, 0.0
+
+    routers = [(i, l["mlp"]["router"]) for i, l in enumerate(config["layers"]) if l.get("mlp")]
+    for i, r in routers:
+        outputs = r["experts"] + r.get("identity", 0)
+        vec(f"l{i}.mlp.correction", outputs, -0.5, 0.3 / outputs)       # (choice scores below zero)
+    code = max([r["experts"] + r.get("identity", 0) for _, r in routers], default=0) if coded_router else 0
+    assert code <= D
+    embed = torch.randn(V, D, generator=g)
+    found = torch.zeros(0, code)
+    while code and len(found) < V:
+        codes = torch.linspace(-2.0, 2.0, code)[torch.rand(4096, code, generator=g).argsort(-1)] + 0.2 * torch.randn(4096, code, generator=g)
+        for i, r in routers:
+            codes = codes[_clear_choice(codes, w[f"l{i}.mlp.correction"].float(), r)]
+        found = torch.cat([found, codes])
+    if code:
+        embed[:, :code] = found[:V]
+    w["embed"] = (embed / config["embedding"]["scale"]).to(torch.bfloat16)
+    for i, layer in enumerate(config["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        for name in ("norm1", "norm1b", "norm2", "norm2b")[:4 if layer.get("mlp") else 2]:
+            norm(p + name, code, 0.002 if name.endswith("b") else 1.0)
+        p += "mix."
+        mat(p + "q", H * d, D)
+        mat(p + "g", H * dv, D, 1.5)
+        mat(p + "o", D, H * dv)
+        kv = m["kv_heads"] if layer["type"] == "attention" else H
+        if m.get("kv_from") is None:
+            mat(p + "k", kv * d, D)
+            mat(p + "v", kv * dv, D)
+        if layer["type"] == "attention":
+            w[p + "talk"] = (torch.eye(H) + 0.4 * torch.randn(H, H, generator=g)).to(torch.bfloat16)
+        else:
+            vec(p + "norm", H * dv)
+        if layer["type"] == "mlstm":
+            # Queries mostly on the side of all keys: what a head reads out is normalised, so that a sum which happens to
+            # cancel would turn any rounding into a result of its own.
+            q = 0.7 * w[p + "k"].float() + 0.5 * w[p + "q"].float()
+            w[p + "q"] = q.to(torch.bfloat16)
+            w[f"l{i}.norm1.b"][code:] *= 5.0
+            for name, centre in (("i", 0.0), ("f", 3.0)):
+                mat(p + name, H, D, 2.0)
+                vec(f"{p}{name}.b", H, centre, 2.0)
+        ff = layer.get("mlp")
+        if ff is None:
+            continue
+        p, r = f"l{i}.mlp.", ff["router"]
+        for e in range(r["experts"]):
+            n = ff["expert"]["ff"]
+            mat(f"{p}e{e}.gate", n, D, 1.5)
+            mat(f"{p}e{e}.up", n, D, 1.5)
+            mat(f"{p}e{e}.down", D, n)
+        outputs = r["experts"] + r.get("identity", 0)
+        mat(p + "router", outputs, D, 2.0)
+        if code:
+            w[p + "router"] = (0.002 * torch.randn(outputs, D, generator=g) + ROUTER_GAIN * torch.eye(outputs, D)).to(torch.bfloat16)
+    norm("final.norm", 0)
+    mat("head", V, D)
+    return w

@@ -418,7 +418,7 @@ extern "C" {
 int b200_head_prepare(const b200_head_prepare_args* p, int dtype, b200_stream_t stream) {
     B200_CHECK_ARG(p, "head_prepare: NULL argument");
     B200_CHECK_ARG(dtype == B200_DTYPE_BF16 || dtype == B200_DTYPE_F32, "head_prepare: unknown dtype");
-    B200_CHECK_ARG(p->tokens >= 0 && p->heads > 0 && p->kv_heads > 0 && p->dim > 0 && p->padded_dim >= p->dim &&
+    B200_CHECK_ARG(p->tokens >= 0 && p->heads > 0 && p->kv_heads >= 0 && p->dim > 0 && p->padded_dim >= p->dim &&
                        p->padded_dim % 64 == 0 && p->padded_value_dim > 0 && p->padded_value_dim % 64 == 0,
                    "head_prepare: bad shape");
     B200_CHECK_ARG(p->rotary_dim >= 0 && p->rotary_dim % 2 == 0 && p->rotary_dim <= p->dim, "head_prepare: bad rotary_dim");

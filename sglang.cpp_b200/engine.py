@@ -246,7 +246,9 @@ class Engine:
                 # (with an offset, the layer norms hold gain - 1: zero as allocated)
                 for name in norms if cfg.norm_offset else norms + ("norm1", "norm2", "norm1_out", "norm2_out"):
                     fill(name, l, 0, ones=True)
-                for name in ("conv", "beside_conv"):      # (fp32; decays, biases and skips stay zero)
+                if spec.decays:
+                    self.load("decay_log", l, torch.tensor(spec.decays).log())
+                for name in ("conv", "beside_conv", "head_mix"):      # (fp32; other decays, biases and skips stay zero)
                     try:
                         ptr, n = self.tensor_info(name, l)
                     except B200Error:
