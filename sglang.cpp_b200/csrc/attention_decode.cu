@@ -743,6 +743,7 @@ decode_mix_kernel(const DecodeParams p, const MixOutput a, int attn_grid) {
 #pragma unroll
     for (int i = 0; i < HC; ++i) u[i] = v[i] = make_float2(0.f, 0.f);
     pdl_wait_prior();
+    const Turn turn = turn_of(a, b, m < pairs ? m : 0);
     for (int g = warp; g < H; g += kMixWarps) {
         float l = 0.f;
         for (int i = lane; i < items * KG; i += 32) l += __ldcg(p.ws_l + (item0 * KG + i) * H + g);
@@ -783,8 +784,8 @@ decode_mix_kernel(const DecodeParams p, const MixOutput a, int attn_grid) {
                 s.x += x.x, s.y += x.y, s.z += x.z, s.w += x.w;
             }
             const int head = c * group + h0 + i;
-            if (m < pairs) finish_mixed<__nv_bfloat16>(a, b, head, m, make_float2(s.x, s.y), make_float2(s.z, s.w));
-            clear_padding<__nv_bfloat16>(a, b, head);
+            if (m < pairs) finish_mixed<__nv_bfloat16>(a, b, head, m, make_float2(s.x, s.y), make_float2(s.z, s.w), turn);
+            clear_padding<__nv_bfloat16>(a, b, head, 32);
         }
     }
 }

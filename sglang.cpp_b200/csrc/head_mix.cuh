@@ -65,27 +65,49 @@ __device__ __forceinline__ void store_pair(__nv_bfloat16* p, float2 x, bool even
     if (even) *reinterpret_cast<uint32_t*>(p) = pack_bf16(x.x, x.y);
     else p[0] = __float2bfloat16_rn(x.x), p[1] = __float2bfloat16_rn(x.y);
 }
+// Four neighbouring elements, 8 or 16 bytes at once where `vec`; of the others the first n.
+__device__ __forceinline__ float4 load_quad(const float* p, bool vec, int n) {
+    if (vec) return *reinterpret_cast<const float4*>(p);
+    return make_float4(n > 0 ? p[0] : 0.f, n > 1 ? p[1] : 0.f, n > 2 ? p[2] : 0.f, n > 3 ? p[3] : 0.f);
+}
+__device__ __forceinline__ float4 load_quad(const __nv_bfloat16* p, bool vec, int n) {
+    if (vec) {
+        const uint2 u = *reinterpret_cast<const uint2*>(p);
+        return make_float4(bf16_lo(u.x), bf16_hi(u.x), bf16_lo(u.y), bf16_hi(u.y));
+    }
+    auto at = [&](int i) { return n > i ? __bfloat162float(p[i]) : 0.f; };
+    return make_float4(at(0), at(1), at(2), at(3));
+}
 __device__ __forceinline__ float exact_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 
+// Cosines and sines of what elements m, m + 1 of token t turn back by (1 and 0 without a rotation).
+struct Turn {
+    float2 c, s;
+};
+__device__ __forceinline__ Turn turn_of(const MixOutput& a, int64_t t, int m) {
+    Turn r = {make_float2(1.f, 1.f), make_float2(0.f, 0.f)};
+    if (a.rotary == 0) return r;
+    int pos = __ldg(a.positions + t);
+    if (pos < 0 || pos >= a.max_pos) {
+        atomicExch(&a.status[kStatusBadIndex], pos + 1);
+        pos = min(max(pos, 0), a.max_pos - 1);
+    }
+    const int pairs = a.pairs();
+    const int64_t at = static_cast<int64_t>(pos) * pairs + m;
+    r.c.x = __ldg(a.cos_t + at), r.s.x = __ldg(a.sin_t + at);
+    if (m + 1 < pairs) r.c.y = __ldg(a.cos_t + at + 1), r.s.y = __ldg(a.sin_t + at + 1);
+    return r;
+}
+
 // Elements m, m + 1 (u) and m + pairs, m + pairs + 1 (v) of head h's mixed values for token t.  With an odd number of
-// pairs the last m stands alone: the second elements are neither turned nor stored.
+// pairs the last m stands alone: the second elements are not stored.
 template <typename T>
-__device__ __forceinline__ void finish_mixed(const MixOutput& a, int64_t t, int h, int m, float2 u, float2 v) {
+__device__ __forceinline__ void finish_mixed(const MixOutput& a, int64_t t, int h, int m, float2 u, float2 v, const Turn& r) {
     const int pairs = a.pairs();
     const bool even = (pairs & 1) == 0, two = m + 1 < pairs;
-    if (a.rotary > 0) {
-        int pos = a.positions[t];
-        if (pos < 0 || pos >= a.max_pos) {
-            atomicExch(&a.status[kStatusBadIndex], pos + 1);
-            pos = min(max(pos, 0), a.max_pos - 1);
-        }
-        const int64_t at = static_cast<int64_t>(pos) * pairs + m;
-        float2 c = make_float2(a.cos_t[at], 1.f), s = make_float2(a.sin_t[at], 0.f);
-        if (two) c.y = a.cos_t[at + 1], s.y = a.sin_t[at + 1];
-        const float2 x = u;
-        u = make_float2(x.x * c.x + v.x * s.x, x.y * c.y + v.y * s.y);
-        v = make_float2(v.x * c.x - x.x * s.x, v.y * c.y - x.y * s.y);
-    }
+    const float2 x = u;
+    u = make_float2(x.x * r.c.x + v.x * r.s.x, x.y * r.c.y + v.y * r.s.y);
+    v = make_float2(v.x * r.c.x - x.x * r.s.x, v.y * r.c.y - x.y * r.s.y);
     float2 fu = make_float2(a.out_scale, a.out_scale), fv = fu;
     const T* gate = static_cast<const T*>(a.gate);
     if (gate != nullptr) {
@@ -111,11 +133,11 @@ __device__ __forceinline__ void finish_mixed(const MixOutput& a, int64_t t, int 
     }
 }
 
-// The padding behind a rotated head is zero.  Called by a whole warp.
+// The padding behind a rotated head is zero.  Called by `lanes` neighbouring threads.
 template <typename T>
-__device__ __forceinline__ void clear_padding(const MixOutput& a, int64_t t, int h) {
+__device__ __forceinline__ void clear_padding(const MixOutput& a, int64_t t, int h, int lanes) {
     T* out = static_cast<T*>(a.out) + t * a.out_st + static_cast<int64_t>(h) * a.vp;
-    for (int i = 2 * a.pairs() + (threadIdx.x & 31); i < a.vp; i += 32) out[i] = static_cast<T>(0.f);
+    for (int i = 2 * a.pairs() + (threadIdx.x & (lanes - 1)); i < a.vp; i += lanes) out[i] = static_cast<T>(0.f);
 }
 #endif
 

@@ -528,7 +528,8 @@ step_kernel(const Recurrence a, int log_cols, bool finish) {
 
 // ---- norm and gate of raw outputs, in place ------------------------------------------------
 
-// Delta rule: one warp per (token, head), four elements per lane in registers (more, for wide heads, read again).
+// Delta rule, and matrix memory normed by head: one warp per (token, head), four elements per lane in registers (more, for
+// wide heads, read again).  The first has one norm for all heads, the second one of all heads' size.
 constexpr int kFinishWarps = 8;
 
 template <typename T>
@@ -543,7 +544,8 @@ finish_heads_kernel(const Recurrence a) {
     const int h = static_cast<int>(row - t * a.heads), c0 = lane * 4;
     T* out = static_cast<T*>(a.out) + t * a.out_ld + static_cast<int64_t>(h) * vp;
     const T* gate = static_cast<const T*>(a.joint) + t * a.joint_ld + static_cast<int64_t>(h) * vp;
-    const T* norm = static_cast<const T*>(a.norm);
+    const bool memory = a.rule == kMemory;
+    const T* norm = static_cast<const T*>(a.norm) + (memory ? static_cast<int64_t>(h) * vp : 0);
     float4 o = make_float4(0.f, 0.f, 0.f, 0.f), g = o, w = o;
     if (c0 < vp) {
         o = load4(out + c0);
@@ -557,8 +559,9 @@ finish_heads_kernel(const Recurrence a) {
     }
     const float scale = rsqrtf(warp_sum(ss) / static_cast<float>(a.value_dim) + a.eps) * a.out_scale;
     auto emit = [&](int c, const float4& y, const float4& z, const float4& n) {
-        store4(out + c, make_float4(y.x * scale * n.x * silu<T>(z.x), y.y * scale * n.y * silu<T>(z.y),
-                                    y.z * scale * n.z * silu<T>(z.z), y.w * scale * n.w * silu<T>(z.w)));
+        auto open = [&](float x) { return memory ? sigmoid<T>(x) : silu<T>(x); };
+        store4(out + c, make_float4(y.x * scale * n.x * open(z.x), y.y * scale * n.y * open(z.y), y.z * scale * n.z * open(z.z),
+                                    y.w * scale * n.w * open(z.w)));
     };
     if (c0 < vp) emit(c0, o, g, w);
     for (int c = c0 + 128; c < vp; c += 128) emit(c, load4(out + c), load4(gate + c), load4(norm + c));
@@ -1477,7 +1480,7 @@ int run(const Recurrence& a, int dtype, cudaStream_t stream) {
                                      : launch_steps<T, kMemory>(a, log_cols, slices, finished, stream);
     }
     if (err != B200_OK || finished) return err;
-    if (delta) {
+    if (delta || (a.rule == kMemory && a.norm_groups == a.heads)) {
         const int64_t rows = static_cast<int64_t>(a.tokens) * a.heads;
         B200_CHECK_CUDA(launch_kernel(finish_heads_kernel<T>, dim3(static_cast<unsigned>(div_ceil64(rows, kFinishWarps))),
                                       dim3(kFinishWarps * 32), 0, stream, dim3(1, 1, 1), a));

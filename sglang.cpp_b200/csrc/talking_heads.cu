@@ -6,7 +6,7 @@
 //     head in the group) pair, against the window's keys.  Per K/V tile of 128 keys
 //         S = Q K^T                  accumulator in TMEM, two of them in turn
 //         P = exp(S)                 written back into TMEM as bf16, over the columns of S that have been read
-//         O_c += P V_c               for both value heads, accumulators in TMEM for the whole row
+//         O_c += P V_c               for both value heads in one product, accumulators in TMEM for the whole row
 //     Queries and keys are bounded (they are unit vectors up to a factor), so the exponentials need no running maximum:
 //     nothing is rescaled, and the two groups of softmax warps take K/V tiles in turn without waiting for one another.
 //     Warp 0 loads tiles through a ring of six TMA buffers, warp 1 issues the products.
@@ -98,9 +98,10 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
         mbar_init(smem_u32(&all_done), 1);
         fence_mbar_init();
     }
-    // Clear the ring once so that rows no copy ever wrote cannot hold NaN patterns.  (Only the last tile has such rows;
-    // every buffer may come to hold it.)
-    if (kv_end % kTile != 0) {
+    // Rows that no copy ever wrote must not hold NaN patterns: only the last tile has such rows, and only in buffers that
+    // no tile before it has filled.
+    const bool clear = kv_end % kTile != 0 && (ntiles - 1) * parts < kSlots;
+    if (clear) {
         uint4* z = reinterpret_cast<uint4*>(smem_gen + kRingOff);
         for (uint32_t i = threadIdx.x; i < kSlots * kSlotBytes / 16; i += kThreads) z[i] = make_uint4(0, 0, 0, 0);
     }
@@ -122,19 +123,15 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
             asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(a), "r"(v.x), "r"(v.y), "r"(v.z), "r"(v.w) : "memory");
         }
     }
-    fence_proxy_async_smem();
-    tc_fence_before();
-    __syncthreads();
-    tc_fence_after();
-    const uint32_t tmem_base = tmem_base_slot;
-
-    if (warp == 0) {
-        // ================= producer =================
+    // The producer warp fills the ring before anybody else is ready, unless the ring is being cleared.
+    bool producer_failed = false;
+    int produced = 0, next_tile = 0;   // buffers filled, tiles begun
+    auto produce = [&](int tiles) {
         const int32_t* pt_row = p.page_table + static_cast<int64_t>(p.table_idx[b]) * p.pt_stride;
         const uint32_t copy_bytes = static_cast<uint32_t>(p.kpc) * 128u;
-        bool failed = false;
-        int n = 0;   // buffers filled so far
-        for (int kt = 0; kt < ntiles && !failed; ++kt) {
+        bool failed = producer_failed;
+        int n = produced;
+        for (int& kt = next_tile; kt < tiles && !failed; ++kt) {
             const int k0 = first_key(kt), valid = min(kTile, kv_end - k0);
             const int ncopies = (valid + p.kpc - 1) / p.kpc;
             int sl[4] = {0, 0, 0, 0};
@@ -186,21 +183,33 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
                 }
             }
         }
+        producer_failed = failed;
+        produced = n;
+    };
+    if (warp == 0 && !clear) {
+        __syncwarp();   // (thread 0 has set up the barriers)
+        produce(min(ntiles, kSlots / parts));
+    }
+    fence_proxy_async_smem();
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem_base = tmem_base_slot;
+
+    if (warp == 0) {
+        // ================= producer =================
+        produce(ntiles);
     } else if (warp == 1) {
         // ================= MMA issuer =================
         if (elect_one()) {
-            const uint32_t idesc_s = idesc_bf16_128x128(false), idesc_pv = idesc_bf16_128x128(true);
-            bool failed = false;
+            const uint32_t idesc_s = idesc_bf16_128x128(false), idesc_pv = idesc_bf16_128xn(nv * 128, true);
             auto buffer = [&](int n) { return smem_base + kRingOff + static_cast<uint32_t>(n % kSlots) * kSlotBytes; };
             auto filled = [&](int n) {
                 return mbar_wait_bounded(smem_u32(&full[n % kSlots]), static_cast<uint32_t>(n / kSlots) & 1u, p.status, 342);
             };
             auto issue_s = [&](int kt) {
                 const int n = kt * parts;
-                if (!filled(n)) {
-                    failed = true;
-                    return;
-                }
+                if (!filled(n)) return false;
                 tc_fence_after();
                 const uint32_t d = tmem_base + kColS + static_cast<uint32_t>(kt & 1) * 128u;
 #pragma unroll
@@ -211,36 +220,29 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
                 }
                 tc_commit(smem_u32(&s_full[kt & 1]));
                 tc_commit(smem_u32(&empty[n % kSlots]));
+                return true;
             };
-            issue_s(0);
-            if (!failed && ntiles > 1) issue_s(1);
-            for (int kt = 0; kt < ntiles && !failed; ++kt) {
+            const bool begun = issue_s(0) && (ntiles == 1 || issue_s(1));
+            for (int kt = 0; kt < ntiles && begun; ++kt) {
                 const uint32_t i = kt & 1, turn = static_cast<uint32_t>(kt >> 1) & 1u;
                 if (!mbar_wait_bounded(smem_u32(&p_full[i]), turn, p.status, 343)) break;
                 tc_fence_after();
-                for (int j = 0; j < nv && !failed; ++j) {
-                    const int n = kt * parts + 1 + j;
-                    if (!filled(n)) {
-                        failed = true;
-                        break;
-                    }
-                    tc_fence_after();
-                    const uint32_t d = tmem_base + kColO + static_cast<uint32_t>(j) * 128u;
+                // (a K/V tile's two value buffers are neighbours in the ring: one operand of 256 columns)
+                const int n = kt * parts + 1;
+                if (!filled(n) || (nv == 2 && !filled(n + 1))) break;
+                tc_fence_after();
 #pragma unroll
-                    for (int ks = 0; ks < 8; ++ks) {
-                        // keys ks*16 .. +15: eight packed columns; keys 64-127 start at column 64
-                        const uint32_t a = tmem_base + kColS + i * 128u + static_cast<uint32_t>((ks >> 2) * 64 + (ks & 3) * 8);
-                        tc_mma_bf16_ts(d, a, mnmajor_sw128_desc(buffer(n) + ks * 2048), idesc_pv, (kt > 0 || ks > 0) ? 1u : 0u);
-                    }
-                    tc_commit(smem_u32(&empty[n % kSlots]));
+                for (int ks = 0; ks < 8; ++ks) {
+                    // keys ks*16 .. +15: eight packed columns; keys 64-127 start at column 64
+                    const uint32_t a = tmem_base + kColS + i * 128u + static_cast<uint32_t>((ks >> 2) * 64 + (ks & 3) * 8);
+                    tc_mma_bf16_ts(tmem_base + kColO, a, mnmajor_sw128_desc(buffer(n) + ks * 2048), idesc_pv, (kt > 0 || ks > 0) ? 1u : 0u);
                 }
-                if (failed) break;
+                for (int j = 0; j < nv; ++j) tc_commit(smem_u32(&empty[(n + j) % kSlots]));
                 tc_commit(smem_u32(&pv_done[i]));
                 if (kt + 1 == ntiles) tc_commit(smem_u32(&all_done));
                 if (kt + 2 >= ntiles) continue;
                 // the next S overwrites the columns these products read P from
-                if (!mbar_wait_bounded(smem_u32(&pv_done[i]), turn, p.status, 344)) break;
-                issue_s(kt + 2);
+                if (!mbar_wait_bounded(smem_u32(&pv_done[i]), turn, p.status, 344) || !issue_s(kt + 2)) break;
             }
         }
     } else {
@@ -253,7 +255,11 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
         const int tok = t0 + r / G;
         const int limit = min(pos0 + tok, len - 1);   // last visible key of this row
         const int oldest = p.w.oldest(limit);         // keys before it are seen below keep_first only
-        auto sees = [&](int k) { return k <= limit && (k >= oldest || k < p.w.keep_first); };
+        // which of the 32 keys from `first` on this row sees, as bits
+        auto below = [](int n) { return n <= 0 ? 0u : n >= 32 ? 0xffffffffu : (1u << n) - 1u; };
+        auto seen = [&](int first) {
+            return below(limit + 1 - first) & (~below(oldest - first) | below(p.w.keep_first - first));
+        };
         const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(qtr * 32) << 16);
         const uint32_t s_addr = lane_addr + kColS + static_cast<uint32_t>(turn) * 128u + static_cast<uint32_t>(half * 64);
         const float sc = p.scale_log2;
@@ -271,14 +277,16 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
             tmem_ld_wait();
 #pragma unroll
             for (int c = 0; c < 2; ++c) {
+                if (need_mask) {   // (an exponent of -inf: no weight)
+                    const uint32_t bits = seen(k0 + c * 32);
+#pragma unroll
+                    for (int i = 0; i < 32; ++i)
+                        if ((bits & (1u << i)) == 0) sv[c][i] = 0xff800000u;
+                }
                 uint32_t packed[16];
 #pragma unroll
                 for (int i = 0; i < 32; i += 2) {
-                    float p0 = ex2(__uint_as_float(sv[c][i]) * sc), p1 = ex2(__uint_as_float(sv[c][i + 1]) * sc);
-                    if (need_mask) {
-                        if (!sees(k0 + c * 32 + i)) p0 = 0.f;
-                        if (!sees(k0 + c * 32 + i + 1)) p1 = 0.f;
-                    }
+                    const float p0 = ex2(__uint_as_float(sv[c][i]) * sc), p1 = ex2(__uint_as_float(sv[c][i + 1]) * sc);
                     sum0 += p0;
                     sum1 += p1;
                     packed[i >> 1] = pack_bf16(p0, p1);
@@ -325,52 +333,72 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
     if (warp == 1) tmem_dealloc(tmem_base, 512);
 }
 
-// One warp per (token, key / value head), HC output heads at a time.
-constexpr int kMixWarps = 4;
+// Half a warp per (token, key / value head), HC output heads and 64 pairs of elements at a time, four pairs per thread.
+constexpr int kMixWarps = 4, kMixLanes = 16, kMixItems = kMixWarps * 32 / kMixLanes;
 
 template <typename T, int HC>
-__global__ void __launch_bounds__(kMixWarps * 32)
+__global__ void __launch_bounds__(kMixWarps * 32, 5)
 mix_kernel(const MixOutput a, const T* __restrict__ raw, int tokens) {
-    extern __shared__ float s_mix[];   // transposed: [from head][to head]
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int H = a.heads, group = H / a.kv_heads, pairs = a.pairs();
+    extern __shared__ __align__(16) float s_mix[];   // transposed, rows of a multiple of HC: [from head][to head]
+    const int lane = threadIdx.x & (kMixLanes - 1);
+    const int H = a.heads, group = H / a.kv_heads, steps = (group + HC - 1) / HC, row = a.kv_heads * steps * HC, pairs = a.pairs();
     pdl_launch_dependents();
-    for (int i = threadIdx.x; i < H * H; i += kMixWarps * 32) s_mix[(i % H) * H + i / H] = a.weights[i];
+    for (int i = threadIdx.x; i < H * row; i += kMixWarps * 32) {
+        const int g = i / row, c = i % row / (steps * HC), j = i % (steps * HC);
+        s_mix[i] = j < group ? a.weights[(c * group + j) * H + g] : 0.f;
+    }
     __syncthreads();
     pdl_wait_prior();
-    const bool even = (pairs & 1) == 0;
+    const bool vec = (pairs & 3) == 0;
     const int64_t items = static_cast<int64_t>(tokens) * a.kv_heads, from = static_cast<int64_t>(a.kv_heads) * a.vp;
-    for (int64_t item = static_cast<int64_t>(blockIdx.x) * kMixWarps + warp; item < items; item += static_cast<int64_t>(gridDim.x) * kMixWarps) {
+    for (int64_t item = static_cast<int64_t>(blockIdx.x) * kMixItems + threadIdx.x / kMixLanes; item < items;
+         item += static_cast<int64_t>(gridDim.x) * kMixItems) {
         const int64_t t = item / a.kv_heads;
         const int c = static_cast<int>(item - t * a.kv_heads);
         const T* src = raw + t * H * from + static_cast<int64_t>(c) * a.vp;
         for (int h0 = 0; h0 < group; h0 += HC) {
-            for (int m = 2 * lane; m < pairs; m += 64) {
-                const bool two = m + 1 < pairs;
-                float2 u[HC], v[HC];
+            for (int m = 4 * lane; m < pairs; m += 4 * kMixLanes) {
+                float4 u[HC], v[HC];
 #pragma unroll
-                for (int i = 0; i < HC; ++i) u[i] = v[i] = make_float2(0.f, 0.f);
-                const float* w = s_mix + c * group + h0;
+                for (int i = 0; i < HC; ++i) u[i] = v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                const float* w = s_mix + c * steps * HC + h0;
 #pragma unroll 4
-                for (int g = 0; g < H; ++g, w += H) {
+                for (int g = 0; g < H; ++g, w += row) {
                     const T* o = src + g * from + m;
-                    const float2 x = load_pair(o, even), y = two ? load_pair(o + pairs, even) : make_float2(static_cast<float>(o[pairs]), 0.f);
+                    const float4 x = load_quad(o, vec, pairs - m), y = load_quad(o + pairs, vec, pairs - m);
+                    float f[HC];
+                    if (HC % 4 == 0) {
+#pragma unroll
+                        for (int i = 0; i < HC; i += 4) *reinterpret_cast<float4*>(f + i) = *reinterpret_cast<const float4*>(w + i);
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < HC; ++i) f[i] = w[i];
+                    }
 #pragma unroll
                     for (int i = 0; i < HC; ++i) {
-                        const float f = w[i];   // (beyond the group: another head's, not stored)
-                        u[i].x = fmaf(f, x.x, u[i].x);
-                        u[i].y = fmaf(f, x.y, u[i].y);
-                        v[i].x = fmaf(f, y.x, v[i].x);
-                        v[i].y = fmaf(f, y.y, v[i].y);
+                        u[i].x = fmaf(f[i], x.x, u[i].x);
+                        u[i].y = fmaf(f[i], x.y, u[i].y);
+                        u[i].z = fmaf(f[i], x.z, u[i].z);
+                        u[i].w = fmaf(f[i], x.w, u[i].w);
+                        v[i].x = fmaf(f[i], y.x, v[i].x);
+                        v[i].y = fmaf(f[i], y.y, v[i].y);
+                        v[i].z = fmaf(f[i], y.z, v[i].z);
+                        v[i].w = fmaf(f[i], y.w, v[i].w);
                     }
                 }
+                const bool more = m + 2 < pairs;
+                const Turn r = turn_of(a, t, m), r2 = more ? turn_of(a, t, m + 2) : r;
 #pragma unroll
-                for (int i = 0; i < HC; ++i)
-                    if (h0 + i < group) finish_mixed<T>(a, t, c * group + h0 + i, m, u[i], v[i]);
+                for (int i = 0; i < HC; ++i) {
+                    if (h0 + i >= group) break;
+                    const int h = c * group + h0 + i;
+                    finish_mixed<T>(a, t, h, m, make_float2(u[i].x, u[i].y), make_float2(v[i].x, v[i].y), r);
+                    if (more) finish_mixed<T>(a, t, h, m + 2, make_float2(u[i].z, u[i].w), make_float2(v[i].z, v[i].w), r2);
+                }
             }
         }
         if (2 * pairs < a.vp)
-            for (int i = 0; i < group; ++i) clear_padding<T>(a, t, c * group + i);
+            for (int i = 0; i < group; ++i) clear_padding<T>(a, t, c * group + i, kMixLanes);
     }
 }
 
@@ -378,10 +406,11 @@ template <typename T>
 int launch_mix(const WindowAttention& a, cudaStream_t stream) {
     const MixOutput m = mix_output(a);
     const int group = a.heads / a.kv_heads;
-    auto kernel = group <= 1 ? mix_kernel<T, 1> : group <= 2 ? mix_kernel<T, 2> : group <= 4 ? mix_kernel<T, 4> : mix_kernel<T, 8>;
-    const size_t smem = (static_cast<size_t>(a.heads) * a.heads + 8) * 4;
+    auto kernel = group <= 1 ? mix_kernel<T, 1> : group <= 2 ? mix_kernel<T, 2> : mix_kernel<T, 4>;
+    const int each = group <= 2 ? group : div_ceil(group, 4) * 4;   // (columns of a group in shared memory)
+    const size_t smem = static_cast<size_t>(a.heads) * a.kv_heads * each * 4;
     B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
-    const int64_t ctas = div_ceil64(static_cast<int64_t>(a.tokens) * a.kv_heads, kMixWarps);
+    const int64_t ctas = div_ceil64(static_cast<int64_t>(a.tokens) * a.kv_heads, kMixItems);
     const int most = sm_count() * 12;
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(static_cast<unsigned>(ctas < most ? ctas : most)), dim3(kMixWarps * 32), smem, stream,
                                   dim3(1, 1, 1), m, static_cast<const T*>(a.mix.scratch), a.tokens));

@@ -112,8 +112,8 @@ __device__ __forceinline__ uint32_t idesc_bf16(int m, int n) {
 __device__ __forceinline__ uint32_t idesc_bf16_m128(int n) { return idesc_bf16(128, n); }
 
 // MN-major operand under the 128-byte swizzle (V as the B operand of P V: rows are keys, 64 head-dim
-// elements per 128-byte row): 8-key groups 1024 bytes apart along K, the second 64 head-dim elements one
-// atom (16 KB) further.
+// elements per 128-byte row): 8-key groups 1024 bytes apart along K, every further 64 head-dim elements one
+// atom (16 KB) on.
 __device__ __forceinline__ uint64_t mnmajor_sw128_desc(uint32_t smem_addr) {
     uint64_t d = 0;
     d |= static_cast<uint64_t>((smem_addr >> 4) & 0x3FFFu);
@@ -123,10 +123,11 @@ __device__ __forceinline__ uint64_t mnmajor_sw128_desc(uint32_t smem_addr) {
     d |= static_cast<uint64_t>(2) << 61;
     return d;
 }
-__device__ __forceinline__ uint32_t idesc_bf16_128x128(bool b_mn_major) {
+__device__ __forceinline__ uint32_t idesc_bf16_128xn(int n, bool b_mn_major) {
     return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn_major ? (1u << 16) : 0u) |
-           (static_cast<uint32_t>(128 >> 3) << 17) | (static_cast<uint32_t>(128 >> 4) << 24);
+           (static_cast<uint32_t>(n >> 3) << 17) | (static_cast<uint32_t>(128 >> 4) << 24);
 }
+__device__ __forceinline__ uint32_t idesc_bf16_128x128(bool b_mn_major) { return idesc_bf16_128xn(128, b_mn_major); }
 // D[tmem] (+)= A[tmem] * B[smem]
 __device__ __forceinline__ void tc_mma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc,
                                                uint32_t accumulate) {

@@ -149,7 +149,7 @@ def test_pages_and_states_that_held_something_else(pkg, name, dtype):
     each time."""
     e, hb = engine_of(name, dtype, pages=3, live=1)
     for k, n in enumerate((192, 70, 129, 1, 65, 192)):
-        ids = C.prompt(C.CONFIGS[name], n, 40 + k)
+        ids = C.prompt(C.CONFIGS[name], n, 240 + k)
         a = hb.open_request(192)
         got = run(e, hb, a, ids, [n - 3, 1, 2] if n > 3 else [n])
         assert C.error(got, oracle(name, ids)) < limit(name, dtype)
