@@ -336,7 +336,8 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
 // Half a warp per (token, key / value head), HC output heads and 64 pairs of elements at a time, four pairs per thread.
 constexpr int kMixWarps = 4, kMixLanes = 16, kMixItems = kMixWarps * 32 / kMixLanes;
 
-template <typename T, int HC>
+// VEC: the number of pairs is a multiple of four.
+template <typename T, int HC, bool VEC>
 __global__ void __launch_bounds__(kMixWarps * 32, 5)
 mix_kernel(const MixOutput a, const T* __restrict__ raw, int tokens) {
     extern __shared__ __align__(16) float s_mix[];   // transposed, rows of a multiple of HC: [from head][to head]
@@ -349,7 +350,6 @@ mix_kernel(const MixOutput a, const T* __restrict__ raw, int tokens) {
     }
     __syncthreads();
     pdl_wait_prior();
-    const bool vec = (pairs & 3) == 0;
     const int64_t items = static_cast<int64_t>(tokens) * a.kv_heads, from = static_cast<int64_t>(a.kv_heads) * a.vp;
     for (int64_t item = static_cast<int64_t>(blockIdx.x) * kMixItems + threadIdx.x / kMixLanes; item < items;
          item += static_cast<int64_t>(gridDim.x) * kMixItems) {
@@ -362,10 +362,10 @@ mix_kernel(const MixOutput a, const T* __restrict__ raw, int tokens) {
 #pragma unroll
                 for (int i = 0; i < HC; ++i) u[i] = v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
                 const float* w = s_mix + c * steps * HC + h0;
-#pragma unroll 4
+#pragma unroll 8
                 for (int g = 0; g < H; ++g, w += row) {
                     const T* o = src + g * from + m;
-                    const float4 x = load_quad(o, vec, pairs - m), y = load_quad(o + pairs, vec, pairs - m);
+                    const float4 x = load_quad(o, VEC, pairs - m), y = load_quad(o + pairs, VEC, pairs - m);
                     float f[HC];
                     if (HC % 4 == 0) {
 #pragma unroll
@@ -402,11 +402,16 @@ mix_kernel(const MixOutput a, const T* __restrict__ raw, int tokens) {
     }
 }
 
+template <typename T, bool VEC>
+auto mix_kernel_for(int group) {
+    return group <= 1 ? mix_kernel<T, 1, VEC> : group <= 2 ? mix_kernel<T, 2, VEC> : mix_kernel<T, 4, VEC>;
+}
+
 template <typename T>
 int launch_mix(const WindowAttention& a, cudaStream_t stream) {
     const MixOutput m = mix_output(a);
     const int group = a.heads / a.kv_heads;
-    auto kernel = group <= 1 ? mix_kernel<T, 1> : group <= 2 ? mix_kernel<T, 2> : mix_kernel<T, 4>;
+    auto kernel = m.pairs() % 4 == 0 ? mix_kernel_for<T, true>(group) : mix_kernel_for<T, false>(group);
     const int each = group <= 2 ? group : div_ceil(group, 4) * 4;   // (columns of a group in shared memory)
     const size_t smem = static_cast<size_t>(a.heads) * a.kv_heads * each * 4;
     B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
