@@ -714,22 +714,22 @@ attention_decode_merge_kernel(const DecodeParams p, int attn_grid) {
     *reinterpret_cast<uint2*>(p.out + (WINDOW ? b * p.w.out_st : static_cast<int64_t>(b) * Hq * kD) + head * kD + lane * 4) = packed;
 }
 
-// Mixing heads: the partials of a request added up, mixed and finished.  One CTA per (request, key / value head); its warps
-// share the heads that are summed over.  HC: room for the heads of a group.
-constexpr int kMixThreads = 256, kMixWarps = kMixThreads / 32;
+// Mixing heads: the partials of a request added up, mixed and finished.  One CTA per (request, key / value head); half
+// warps share the heads that are summed over.  HC: room for the heads of a group; VEC: as in finish_mixed.
+constexpr int kMixThreads = 256, kMixLanes = 16, kMixParts = kMixThreads / kMixLanes;   // (four pairs of elements per lane)
 
-template <int HC>
+template <int HC, bool VEC>
 __global__ void __launch_bounds__(kMixThreads)
 decode_mix_kernel(const DecodeParams p, const MixOutput a, int attn_grid) {
     __shared__ int3 s_split;
-    constexpr int kOnce = HC < 8 ? HC : 8;   // heads added up at a time
-    __shared__ float4 s_part[kMixWarps][kOnce][32];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    constexpr int kOnce = HC < 4 ? HC : 4;   // heads added up at a time
+    __shared__ float4 s_part[kMixParts][kOnce][2][kMixLanes];
+    const int part = threadIdx.x / kMixLanes, lane = threadIdx.x % kMixLanes;
     const int b = blockIdx.x, c = blockIdx.y, H = a.heads, group = p.group, pairs = a.pairs();
     pdl_launch_dependents();
-    if (warp == 0) {
+    if (threadIdx.x < 32) {
         const int3 r = request_stages<true>(p, b);
-        if (lane == 0) s_split = r;
+        if (threadIdx.x == 0) s_split = r;
     }
     __syncthreads();
     const int first = s_split.x, st = s_split.y;
@@ -737,57 +737,73 @@ decode_mix_kernel(const DecodeParams p, const MixOutput a, int attn_grid) {
     const int items = st > 0 ? (first + st - 1) / per - c0 + 1 : 0;
     const int KG = kConsumerWarps / p.kv_heads;
     const int64_t item0 = b + c0;
-    const bool even = (pairs & 1) == 0;
-    const int m = 2 * lane;
-    float2 u[HC], v[HC];
+    const int m = 4 * lane;
+    const bool there = m < pairs;
+    float4 u[HC], v[HC];
 #pragma unroll
-    for (int i = 0; i < HC; ++i) u[i] = v[i] = make_float2(0.f, 0.f);
+    for (int i = 0; i < HC; ++i) u[i] = v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    auto add = [](float4& to, const float4& x) { to.x += x.x, to.y += x.y, to.z += x.z, to.w += x.w; };
+    auto weigh = [](float4& to, float f, const float4& x) {
+        to.x = fmaf(f, x.x, to.x);
+        to.y = fmaf(f, x.y, to.y);
+        to.z = fmaf(f, x.z, to.z);
+        to.w = fmaf(f, x.w, to.w);
+    };
     pdl_wait_prior();
-    const Turn turn = turn_of(a, b, m < pairs ? m : 0);
-    for (int g = warp; g < H; g += kMixWarps) {
+    const Turn turn = turn_of<VEC>(a, b, there ? m : 0);
+    // (H need not be a multiple of the parts: every thread takes every round, for the shuffles)
+    for (int g0 = 0; g0 < H; g0 += kMixParts) {
+        const int g = min(g0 + part, H - 1);
         float l = 0.f;
-        for (int i = lane; i < items * KG; i += 32) l += __ldcg(p.ws_l + (item0 * KG + i) * H + g);
-        l = warp_sum(l);
-        float2 x = make_float2(0.f, 0.f), y = x;
-        if (m < pairs) {
+        for (int i = lane; i < items * KG; i += kMixLanes) l += __ldcg(p.ws_l + (item0 * KG + i) * H + g);
+#pragma unroll
+        for (int o = kMixLanes / 2; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
+        if (there) {
             const float* o = p.ws_o + ((item0 * H + g) * p.kv_heads + c) * kD + m;
             const int64_t step = static_cast<int64_t>(H) * p.kv_heads * kD;
 #pragma unroll 4
             for (int i = 0; i < items; ++i, o += step) {
-                const float2 d = load_pair(o, true);
-                const float2 e = m + 1 < pairs ? load_pair(o + pairs, even) : make_float2(o[pairs], 0.f);
-                x.x += d.x, x.y += d.y, y.x += e.x, y.y += e.y;
+                add(x, load_quad<VEC>(o, pairs - m));
+                add(y, load_quad<VEC>(o + pairs, pairs - m));
             }
         }
-        const float inv = l > 0.f ? 1.f / l : 0.f;
+        const float inv = g0 + part < H && l > 0.f ? 1.f / l : 0.f;
 #pragma unroll
         for (int i = 0; i < HC; ++i) {
             if (i >= group) break;
             const float f = a.weights[static_cast<int64_t>(c * group + i) * H + g] * inv;
-            u[i].x = fmaf(f, x.x, u[i].x);
-            u[i].y = fmaf(f, x.y, u[i].y);
-            v[i].x = fmaf(f, y.x, v[i].x);
-            v[i].y = fmaf(f, y.y, v[i].y);
+            weigh(u[i], f, x);
+            weigh(v[i], f, y);
         }
     }
 #pragma unroll
     for (int h0 = 0; h0 < HC; h0 += kOnce) {
         if (h0 > 0) __syncthreads();
 #pragma unroll
-        for (int i = 0; i < kOnce; ++i) s_part[warp][i][lane] = make_float4(u[h0 + i].x, u[h0 + i].y, v[h0 + i].x, v[h0 + i].y);
+        for (int i = 0; i < kOnce; ++i) {
+            s_part[part][i][0][lane] = u[h0 + i];
+            s_part[part][i][1][lane] = v[h0 + i];
+        }
         __syncthreads();
-        for (int i = warp; i < min(kOnce, group - h0); i += kMixWarps) {
-            float4 s = s_part[0][i][lane];
+        if (part < kOnce && h0 + part < group) {
+            float4 x = s_part[0][part][0][lane], y = s_part[0][part][1][lane];
 #pragma unroll
-            for (int w = 1; w < kMixWarps; ++w) {
-                const float4 x = s_part[w][i][lane];
-                s.x += x.x, s.y += x.y, s.z += x.z, s.w += x.w;
+            for (int w = 1; w < kMixParts; ++w) {
+                add(x, s_part[w][part][0][lane]);
+                add(y, s_part[w][part][1][lane]);
             }
-            const int head = c * group + h0 + i;
-            if (m < pairs) finish_mixed<__nv_bfloat16>(a, b, head, m, make_float2(s.x, s.y), make_float2(s.z, s.w), turn);
-            clear_padding<__nv_bfloat16>(a, b, head, 32);
+            const int head = c * group + h0 + part;
+            if (there) finish_mixed<__nv_bfloat16, VEC>(a, b, head, m, x, y, turn);
+            clear_padding<__nv_bfloat16>(a, b, head, kMixLanes);
         }
     }
+}
+
+template <bool VEC>
+auto decode_mix_for(int group) {
+    return group <= 1 ? decode_mix_kernel<1, VEC> : group <= 2 ? decode_mix_kernel<2, VEC> : group <= 4 ? decode_mix_kernel<4, VEC>
+           : group <= 8 ? decode_mix_kernel<8, VEC> : decode_mix_kernel<16, VEC>;
 }
 
 // The attention kernel of mixing heads for these counts, or NULL.
@@ -850,10 +866,9 @@ int launch_talking_decode(const WindowAttention& a, cudaStream_t stream) {
     const int smem = kStages * kStageBytes + 1024;
     B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     B200_CHECK_CUDA(launch_kernel(kernel, dim3(grid), dim3(kThreads), smem, stream, dim3(1, 1, 1), tk, tv, p));
-    const int g = p.group;
-    auto mix = g <= 1 ? decode_mix_kernel<1> : g <= 2 ? decode_mix_kernel<2> : g <= 4 ? decode_mix_kernel<4>
-               : g <= 8 ? decode_mix_kernel<8> : decode_mix_kernel<16>;
-    B200_CHECK_CUDA(launch_kernel(mix, dim3(a.batch, a.kv_heads), dim3(kMixThreads), 0, stream, dim3(1, 1, 1), p, mix_output(a), grid));
+    const MixOutput m = mix_output(a);
+    auto mix = m.pairs() % 4 == 0 ? decode_mix_for<true>(p.group) : decode_mix_for<false>(p.group);
+    B200_CHECK_CUDA(launch_kernel(mix, dim3(a.batch, a.kv_heads), dim3(kMixThreads), 0, stream, dim3(1, 1, 1), p, m, grid));
     return B200_OK;
 }
 

@@ -49,88 +49,95 @@ inline MixOutput mix_output(const WindowAttention& a) {
 }
 
 #ifdef __CUDACC__
-__device__ __forceinline__ float2 load_pair(const float* p, bool even) {
-    return even ? *reinterpret_cast<const float2*>(p) : make_float2(p[0], p[1]);
+// Elements m .. m + 3 of a row whose elements up to m + n are there; 8 or 16 bytes at once under VEC (all four are).
+template <bool VEC>
+__device__ __forceinline__ float4 load_quad(const float* p, int n) {
+    if (VEC) return *reinterpret_cast<const float4*>(p);
+    auto at = [&](int i) { return n > i ? p[i] : 0.f; };
+    return make_float4(at(0), at(1), at(2), at(3));
 }
-__device__ __forceinline__ float2 load_pair(const __nv_bfloat16* p, bool even) {
-    if (!even) return make_float2(__bfloat162float(p[0]), __bfloat162float(p[1]));
-    const uint32_t u = *reinterpret_cast<const uint32_t*>(p);
-    return make_float2(bf16_lo(u), bf16_hi(u));
-}
-__device__ __forceinline__ void store_pair(float* p, float2 x, bool even) {
-    if (even) *reinterpret_cast<float2*>(p) = x;
-    else p[0] = x.x, p[1] = x.y;
-}
-__device__ __forceinline__ void store_pair(__nv_bfloat16* p, float2 x, bool even) {
-    if (even) *reinterpret_cast<uint32_t*>(p) = pack_bf16(x.x, x.y);
-    else p[0] = __float2bfloat16_rn(x.x), p[1] = __float2bfloat16_rn(x.y);
-}
-// Four neighbouring elements, 8 or 16 bytes at once where `vec`; of the others the first n.
-__device__ __forceinline__ float4 load_quad(const float* p, bool vec, int n) {
-    if (vec) return *reinterpret_cast<const float4*>(p);
-    return make_float4(n > 0 ? p[0] : 0.f, n > 1 ? p[1] : 0.f, n > 2 ? p[2] : 0.f, n > 3 ? p[3] : 0.f);
-}
-__device__ __forceinline__ float4 load_quad(const __nv_bfloat16* p, bool vec, int n) {
-    if (vec) {
+template <bool VEC>
+__device__ __forceinline__ float4 load_quad(const __nv_bfloat16* p, int n) {
+    if (VEC) {
         const uint2 u = *reinterpret_cast<const uint2*>(p);
         return make_float4(bf16_lo(u.x), bf16_hi(u.x), bf16_lo(u.y), bf16_hi(u.y));
     }
     auto at = [&](int i) { return n > i ? __bfloat162float(p[i]) : 0.f; };
     return make_float4(at(0), at(1), at(2), at(3));
 }
-__device__ __forceinline__ float exact_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
+template <bool VEC>
+__device__ __forceinline__ void store_quad(float* p, const float4& x, int n) {
+    if (VEC) {
+        *reinterpret_cast<float4*>(p) = x;
+        return;
+    }
+    const float v[4] = {x.x, x.y, x.z, x.w};
+    for (int i = 0; i < 4; ++i)
+        if (n > i) p[i] = v[i];
+}
+template <bool VEC>
+__device__ __forceinline__ void store_quad(__nv_bfloat16* p, const float4& x, int n) {
+    if (VEC) {
+        *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(x.x, x.y), pack_bf16(x.z, x.w));
+        return;
+    }
+    const float v[4] = {x.x, x.y, x.z, x.w};
+    for (int i = 0; i < 4; ++i)
+        if (n > i) p[i] = __float2bfloat16_rn(v[i]);
+}
+template <typename T>
+__device__ __forceinline__ float open_gate(float x) { return 1.f / (1.f + expf(-x)); }
+template <>
+__device__ __forceinline__ float open_gate<__nv_bfloat16>(float x) { return sigmoid_f(x); }
 
-// Cosines and sines of what elements m, m + 1 of token t turn back by (1 and 0 without a rotation).
+// Cosines and sines of what elements m .. m + 3 of token t turn back by (1 and 0 without a rotation).
 struct Turn {
-    float2 c, s;
+    float4 c, s;
 };
+template <bool VEC>
 __device__ __forceinline__ Turn turn_of(const MixOutput& a, int64_t t, int m) {
-    Turn r = {make_float2(1.f, 1.f), make_float2(0.f, 0.f)};
+    Turn r = {make_float4(1.f, 1.f, 1.f, 1.f), make_float4(0.f, 0.f, 0.f, 0.f)};
     if (a.rotary == 0) return r;
-    int pos = __ldg(a.positions + t);
+    int pos = a.positions[t];
     if (pos < 0 || pos >= a.max_pos) {
         atomicExch(&a.status[kStatusBadIndex], pos + 1);
         pos = min(max(pos, 0), a.max_pos - 1);
     }
-    const int pairs = a.pairs();
-    const int64_t at = static_cast<int64_t>(pos) * pairs + m;
-    r.c.x = __ldg(a.cos_t + at), r.s.x = __ldg(a.sin_t + at);
-    if (m + 1 < pairs) r.c.y = __ldg(a.cos_t + at + 1), r.s.y = __ldg(a.sin_t + at + 1);
+    const int64_t at = static_cast<int64_t>(pos) * a.pairs() + m;
+    r.c = load_quad<VEC>(a.cos_t + at, a.pairs() - m);
+    r.s = load_quad<VEC>(a.sin_t + at, a.pairs() - m);
     return r;
 }
 
-// Elements m, m + 1 (u) and m + pairs, m + pairs + 1 (v) of head h's mixed values for token t.  With an odd number of
-// pairs the last m stands alone: the second elements are not stored.
-template <typename T>
-__device__ __forceinline__ void finish_mixed(const MixOutput& a, int64_t t, int h, int m, float2 u, float2 v, const Turn& r) {
-    const int pairs = a.pairs();
-    const bool even = (pairs & 1) == 0, two = m + 1 < pairs;
-    const float2 x = u;
-    u = make_float2(x.x * r.c.x + v.x * r.s.x, x.y * r.c.y + v.y * r.s.y);
-    v = make_float2(v.x * r.c.x - x.x * r.s.x, v.y * r.c.y - x.y * r.s.y);
-    float2 fu = make_float2(a.out_scale, a.out_scale), fv = fu;
+// Elements m .. m + 3 (u) and those a.pairs() further (v) of head h's mixed values for token t.  VEC: the number of pairs is
+// a multiple of four.
+template <typename T, bool VEC>
+__device__ __forceinline__ void finish_mixed(const MixOutput& a, int64_t t, int h, int m, const float4& u, const float4& v, const Turn& r) {
+    const int pairs = a.pairs(), n = pairs - m;
+    float4 x = make_float4(u.x * r.c.x + v.x * r.s.x, u.y * r.c.y + v.y * r.s.y, u.z * r.c.z + v.z * r.s.z, u.w * r.c.w + v.w * r.s.w);
+    float4 y = make_float4(v.x * r.c.x - u.x * r.s.x, v.y * r.c.y - u.y * r.s.y, v.z * r.c.z - u.z * r.s.z, v.w * r.c.w - u.w * r.s.w);
+    auto scale = [](float4& z, float f) { z.x *= f, z.y *= f, z.z *= f, z.w *= f; };
+    float factor = a.out_scale;
     const T* gate = static_cast<const T*>(a.gate);
     if (gate != nullptr) {
         gate += t * a.gate_st;
         if (a.gate_per_head) {
-            const float g = exact_sigmoid(static_cast<float>(gate[h]));
-            fu.x *= g, fu.y *= g, fv.x *= g, fv.y *= g;
+            factor *= open_gate<T>(static_cast<float>(gate[h]));
         } else {
             gate += static_cast<int64_t>(h) * a.vp + m;
-            const float2 gu = load_pair(gate, even && two), gv = two ? load_pair(gate + pairs, even) : make_float2(static_cast<float>(gate[pairs]), 0.f);
-            fu.x *= exact_sigmoid(gu.x), fu.y *= exact_sigmoid(gu.y);
-            fv.x *= exact_sigmoid(gv.x), fv.y *= exact_sigmoid(gv.y);
+            const float4 gx = load_quad<VEC>(gate, n), gy = load_quad<VEC>(gate + pairs, n);
+            auto open = [](float4& z, const float4& g) {
+                z.x *= open_gate<T>(g.x), z.y *= open_gate<T>(g.y), z.z *= open_gate<T>(g.z), z.w *= open_gate<T>(g.w);
+            };
+            open(x, gx);
+            open(y, gy);
         }
     }
-    u.x *= fu.x, u.y *= fu.y, v.x *= fv.x, v.y *= fv.y;
-    T* out = static_cast<T*>(a.out) + t * a.out_st + static_cast<int64_t>(h) * a.vp;
-    if (two) {
-        store_pair(out + m, u, even);
-        store_pair(out + m + pairs, v, even);
-    } else {
-        out[m] = static_cast<T>(u.x);
-        out[m + pairs] = static_cast<T>(v.x);
-    }
+    scale(x, factor);
+    scale(y, factor);
+    T* out = static_cast<T*>(a.out) + t * a.out_st + static_cast<int64_t>(h) * a.vp + m;
+    store_quad<VEC>(out, x, n);
+    store_quad<VEC>(out + pairs, y, n);
 }
 
 // The padding behind a rotated head is zero.  Called by `lanes` neighbouring threads.

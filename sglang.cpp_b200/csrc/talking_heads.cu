@@ -4,12 +4,13 @@
 //   * prefill_kernel leaves O_gc, what the weights of head g make of the values of key / value head c, for all pairs.
 //     One CTA owns (request, key head, 128 / group query tokens, two value heads): a tile of 128 rows, each a (token,
 //     head in the group) pair, against the window's keys.  Per K/V tile of 128 keys
-//         S = Q K^T                  accumulator in TMEM, two of them in turn
-//         P = exp(S)                 written back into TMEM as bf16, over the columns of S that have been read
+//         S = Q K^T                  accumulator in TMEM
+//         P = exp(S)                 as bf16 in TMEM, in two places in turn; S is free once its threads have read it
 //         O_c += P V_c               for both value heads in one product, accumulators in TMEM for the whole row
 //     Queries and keys are bounded (they are unit vectors up to a factor), so the exponentials need no running maximum:
 //     nothing is rescaled, and the two groups of softmax warps take K/V tiles in turn without waiting for one another.
-//     Warp 0 loads tiles through a ring of six TMA buffers, warp 1 issues the products.
+//     No product waits for the one before it: S of the next tile runs ahead of P V of this one.  Warp 0 loads tiles
+//     through rings of two TMA buffers, keys a tile ahead of values; warp 1 issues the products.
 //   * mix_kernel sums O_gc over the heads.
 //   * fp32, other head sizes and counts, unbounded scores: the plain attention kernel in place of the first one.
 #include "common.cuh"
@@ -26,10 +27,11 @@ constexpr int kTile = 128;                  // keys per K/V tile and rows per qu
 constexpr int kSoftmaxThreads = 2 * 256;
 constexpr int kThreads = 64 + kSoftmaxThreads;
 constexpr uint32_t kAtomBytes = 128 * 128;  // 128 rows x 64 bf16: one swizzle atom column
-constexpr uint32_t kQOff = 0, kRingOff = 2 * kAtomBytes, kSlotBytes = 2 * kAtomBytes;
-constexpr int kSlots = 6;                   // K, then the value heads, of one K/V tile after another
-constexpr uint32_t kSmemBytes = kRingOff + kSlots * kSlotBytes;
-constexpr uint32_t kColS = 0, kColO = 256;  // TMEM columns: S of even and odd tiles, O of the two value heads
+constexpr int kStages = 2;
+constexpr uint32_t kQOff = 0, kKOff = 2 * kAtomBytes, kKBytes = 2 * kAtomBytes;   // per stage: keys 64 columns wide each
+constexpr uint32_t kVOff = kKOff + kStages * kKBytes, kVBytes = 4 * kAtomBytes;   // per stage: both value heads
+constexpr uint32_t kSmemBytes = kVOff + kStages * kVBytes;
+constexpr uint32_t kColS = 0, kColP = 128, kColO = 256;   // TMEM columns: S; P of even and odd tiles (64 each); O of the value heads
 constexpr float kMaxExponent = 100.f;       // log2 of the largest exponential
 
 struct PrefillParams {
@@ -59,8 +61,8 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
                const __grid_constant__ CUtensorMap tmap_k_tile, const __grid_constant__ CUtensorMap tmap_v_tile,
                const PrefillParams p) {
     extern __shared__ uint8_t smem_raw[];
-    __shared__ __align__(8) uint64_t full[kSlots], empty[kSlots];
-    __shared__ __align__(8) uint64_t s_full[2], p_full[2], pv_done[2];   // per tile parity
+    __shared__ __align__(8) uint64_t k_full[kStages], k_empty[kStages], v_full[kStages], v_empty[kStages];
+    __shared__ __align__(8) uint64_t s_full[2], s_free[2], p_full[2], pv_done[2];   // per tile parity
     __shared__ __align__(8) uint64_t all_done;   // (of its own: a group that skips phases of pv_done cannot wait for a later one)
     __shared__ uint32_t tmem_base_slot;
 
@@ -69,12 +71,12 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
     uint8_t* smem_gen = smem_raw + (smem_base - smem_u32(smem_raw));
     const int G = p.group, QB = kTile / G;
     const int b = blockIdx.z, h = blockIdx.y / p.value_pairs, c0 = blockIdx.y % p.value_pairs * 2;
-    const int nv = min(2, p.kv_heads - c0), parts = 1 + nv;   // buffers per K/V tile
+    const int nv = min(2, p.kv_heads - c0);
 
     pdl_launch_dependents();
     pdl_wait_prior();
 
-    const int q_begin = p.qo_indptr[b], ext = p.qo_indptr[b + 1] - q_begin, len = p.seq_lens[b];
+    const int q_begin = p.qo_indptr[b], ext = p.qo_indptr[b + 1] - q_begin, len = p.seq_lens[b], table = p.table_idx[b];
     const int nqb = (ext + QB - 1) / QB;
     const int qb = nqb - 1 - static_cast<int>(blockIdx.x);   // heaviest blocks first
     if (qb < 0 || ext <= 0 || len <= 0) return;              // whole CTA, before any barrier or TMEM use
@@ -86,12 +88,15 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
     auto first_key = [&](int kt) { return (kt >= head_tiles ? kt + skip : kt) * kTile; };
 
     if (threadIdx.x == 0) {
-        for (int s = 0; s < kSlots; ++s) {
-            mbar_init(smem_u32(&full[s]), 1);
-            mbar_init(smem_u32(&empty[s]), 1);
+        for (int s = 0; s < kStages; ++s) {
+            mbar_init(smem_u32(&k_full[s]), 1);
+            mbar_init(smem_u32(&k_empty[s]), 1);
+            mbar_init(smem_u32(&v_full[s]), 1);
+            mbar_init(smem_u32(&v_empty[s]), 1);
         }
         for (int i = 0; i < 2; ++i) {
             mbar_init(smem_u32(&s_full[i]), 1);
+            mbar_init(smem_u32(&s_free[i]), 8);   // likewise
             mbar_init(smem_u32(&p_full[i]), 8);   // one arrival per softmax warp of the tile
             mbar_init(smem_u32(&pv_done[i]), 1);
         }
@@ -100,10 +105,10 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
     }
     // Rows that no copy ever wrote must not hold NaN patterns: only the last tile has such rows, and only in buffers that
     // no tile before it has filled.
-    const bool clear = kv_end % kTile != 0 && (ntiles - 1) * parts < kSlots;
+    const bool clear = kv_end % kTile != 0 && ntiles <= kStages;
     if (clear) {
-        uint4* z = reinterpret_cast<uint4*>(smem_gen + kRingOff);
-        for (uint32_t i = threadIdx.x; i < kSlots * kSlotBytes / 16; i += kThreads) z[i] = make_uint4(0, 0, 0, 0);
+        uint4* z = reinterpret_cast<uint4*>(smem_gen + kKOff);
+        for (uint32_t i = threadIdx.x; i < (kSmemBytes - kKOff) / 16; i += kThreads) z[i] = make_uint4(0, 0, 0, 0);
     }
     if (warp == 1) {
         tmem_alloc(smem_u32(&tmem_base_slot), 512);
@@ -123,31 +128,49 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
             asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(a), "r"(v.x), "r"(v.y), "r"(v.z), "r"(v.w) : "memory");
         }
     }
-    // The producer warp fills the ring before anybody else is ready, unless the ring is being cleared.
-    bool producer_failed = false;
-    int produced = 0, next_tile = 0;   // buffers filled, tiles begun
-    auto produce = [&](int tiles) {
-        const int32_t* pt_row = p.page_table + static_cast<int64_t>(p.table_idx[b]) * p.pt_stride;
+    fence_proxy_async_smem();
+    tc_fence_before();
+    // The producer does not wait for the others, unless they are clearing its buffers.
+    if (warp == 0 && !clear)
+        asm volatile("bar.arrive 2, %0;" ::"n"(kThreads) : "memory");
+    else
+        asm volatile("bar.sync 2, %0;" ::"n"(kThreads) : "memory");
+    tc_fence_after();
+
+    if (warp == 0) {
+        // ================= producer =================
+        __syncwarp();   // (one of its threads has set up the barriers)
+        const int32_t* pt_row = p.page_table + static_cast<int64_t>(table) * p.pt_stride;
         const uint32_t copy_bytes = static_cast<uint32_t>(p.kpc) * 128u;
-        bool failed = producer_failed;
-        int n = produced;
-        for (int& kt = next_tile; kt < tiles && !failed; ++kt) {
-            const int k0 = first_key(kt), valid = min(kTile, kv_end - k0);
-            const int ncopies = (valid + p.kpc - 1) / p.kpc;
-            int sl[4] = {0, 0, 0, 0};
+        // the first slots of a tile's pages, fetched a tile ahead of their use
+        struct Pages {
+            int at[4];
+        };
+        auto pages_of = [&](int kt) {
+            Pages s = {{0, 0, 0, 0}};
+            if (kt >= ntiles) return s;
+            const int k0 = first_key(kt), ncopies = (min(kTile, kv_end - k0) + p.kpc - 1) / p.kpc;
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+                if (i * 32 + lane < ncopies) s.at[i] = pt_row[k0 + (i * 32 + lane) * p.kpc];
+            return s;
+        };
+        auto load = [&](int kt, const Pages& pages, bool values) {
+            const int stage = kt % kStages, valid = min(kTile, kv_end - first_key(kt)), ncopies = (valid + p.kpc - 1) / p.kpc;
+            const uint32_t bar = smem_u32(values ? &v_full[stage] : &k_full[stage]);
+            if (kt >= kStages && !mbar_wait_bounded(smem_u32(values ? &v_empty[stage] : &k_empty[stage]),
+                                                    static_cast<uint32_t>(kt / kStages - 1) & 1u, p.status, 341))
+                return false;
+            int sl[4];
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-                const int copy = i * 32 + lane;
-                if (copy < ncopies) {
-                    int64_t v = pt_row[k0 + copy * p.kpc];
-                    if (v < 0 || v + p.kpc > p.num_slots) {
-                        atomicExch(&p.status[kStatusBadIndex], static_cast<int>(v) + 1);
-                        v = 0;
-                    }
-                    sl[i] = static_cast<int>(v);
+                sl[i] = pages.at[i];
+                if (sl[i] < 0 || static_cast<int64_t>(sl[i]) + p.kpc > p.num_slots) {
+                    atomicExch(&p.status[kStatusBadIndex], sl[i] + 1);
+                    sl[i] = 0;
                 }
             }
-            // A tile whose pages are consecutive slots is fetched with two 128-key boxes.
+            // A tile whose pages are consecutive slots is fetched with two 128-key boxes per head.
             bool mine = true;
             const int first = __shfl_sync(0xffffffffu, sl[0], 0);
 #pragma unroll
@@ -156,93 +179,76 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
                 if (copy < ncopies && sl[i] != first + copy * p.kpc) mine = false;
             }
             const bool whole = __all_sync(0xffffffffu, mine) && valid == kTile && p.whole_tile_boxes;
-            for (int part = 0; part < parts; ++part, ++n) {
-                const uint32_t slot = n % kSlots;
-                if (n >= kSlots &&
-                    !mbar_wait_bounded(smem_u32(&empty[slot]), static_cast<uint32_t>(n / kSlots - 1) & 1u, p.status, 341)) {
-                    failed = true;
-                    break;
-                }
-                const uint32_t bar = smem_u32(&full[slot]), dst0 = smem_base + kRingOff + slot * kSlotBytes;
-                const int head = part == 0 ? h : c0 + part - 1;
-                if (lane == 0) mbar_arrive_expect_tx(bar, static_cast<uint32_t>(ncopies) * 2u * copy_bytes);
-                __syncwarp();
-                if (whole) {
-                    if (lane < 2)
-                        tma_load_3d(dst0 + lane * kAtomBytes, part == 0 ? &tmap_k_tile : &tmap_v_tile, lane * 64, head, first, bar);
-                    continue;
-                }
+            const int heads = values ? nv : 1;
+            const uint32_t dst0 = smem_base + (values ? kVOff + stage * kVBytes : kKOff + stage * kKBytes);
+            if (lane == 0) mbar_arrive_expect_tx(bar, static_cast<uint32_t>(heads * ncopies) * 2u * copy_bytes);
+            __syncwarp();
+            if (whole) {
+                if (lane < 2 * heads)
+                    tma_load_3d(dst0 + lane * kAtomBytes, values ? &tmap_v_tile : &tmap_k_tile, (lane & 1) * 64,
+                                values ? c0 + (lane >> 1) : h, first, bar);
+                return true;
+            }
+            for (int j = 0; j < heads; ++j) {
+                const int head = values ? c0 + j : h;
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
                     const int copy = i * 32 + lane;
                     if (copy < ncopies) {
-                        const uint32_t dst = dst0 + copy * copy_bytes;
-                        tma_load_3d(dst, part == 0 ? &tmap_k : &tmap_v, 0, head, sl[i], bar);
-                        tma_load_3d(dst + kAtomBytes, part == 0 ? &tmap_k : &tmap_v, 64, head, sl[i], bar);
+                        const uint32_t dst = dst0 + j * 2 * kAtomBytes + copy * copy_bytes;
+                        tma_load_3d(dst, values ? &tmap_v : &tmap_k, 0, head, sl[i], bar);
+                        tma_load_3d(dst + kAtomBytes, values ? &tmap_v : &tmap_k, 64, head, sl[i], bar);
                     }
                 }
             }
+            return true;
+        };
+        Pages now = pages_of(0), next = pages_of(1);
+        bool going = load(0, now, false);
+        for (int kt = 0; kt < ntiles && going; ++kt) {
+            const Pages after = pages_of(kt + 2);
+            going = (kt + 1 >= ntiles || load(kt + 1, next, false)) && load(kt, now, true);
+            now = next;
+            next = after;
         }
-        producer_failed = failed;
-        produced = n;
-    };
-    if (warp == 0 && !clear) {
-        __syncwarp();   // (thread 0 has set up the barriers)
-        produce(min(ntiles, kSlots / parts));
-    }
-    fence_proxy_async_smem();
-    tc_fence_before();
-    __syncthreads();
-    tc_fence_after();
-    const uint32_t tmem_base = tmem_base_slot;
-
-    if (warp == 0) {
-        // ================= producer =================
-        produce(ntiles);
     } else if (warp == 1) {
         // ================= MMA issuer =================
         if (elect_one()) {
+            const uint32_t tmem_base = tmem_base_slot;
             const uint32_t idesc_s = idesc_bf16_128x128(false), idesc_pv = idesc_bf16_128xn(nv * 128, true);
-            auto buffer = [&](int n) { return smem_base + kRingOff + static_cast<uint32_t>(n % kSlots) * kSlotBytes; };
-            auto filled = [&](int n) {
-                return mbar_wait_bounded(smem_u32(&full[n % kSlots]), static_cast<uint32_t>(n / kSlots) & 1u, p.status, 342);
-            };
             auto issue_s = [&](int kt) {
-                const int n = kt * parts;
-                if (!filled(n)) return false;
+                const int stage = kt % kStages;
+                const uint32_t keys = smem_base + kKOff + stage * kKBytes;
+                if (!mbar_wait_bounded(smem_u32(&k_full[stage]), static_cast<uint32_t>(kt / kStages) & 1u, p.status, 342)) return false;
                 tc_fence_after();
-                const uint32_t d = tmem_base + kColS + static_cast<uint32_t>(kt & 1) * 128u;
 #pragma unroll
                 for (int ks = 0; ks < 8; ++ks) {
                     const uint32_t off = (ks >> 2) * kAtomBytes + (ks & 3) * 32;
-                    tc_mma_bf16(d, kmajor_sw128_desc(smem_base + kQOff + off), kmajor_sw128_desc(buffer(n) + off), idesc_s,
+                    tc_mma_bf16(tmem_base + kColS, kmajor_sw128_desc(smem_base + kQOff + off), kmajor_sw128_desc(keys + off), idesc_s,
                                 ks > 0 ? 1u : 0u);
                 }
                 tc_commit(smem_u32(&s_full[kt & 1]));
-                tc_commit(smem_u32(&empty[n % kSlots]));
+                tc_commit(smem_u32(&k_empty[stage]));
                 return true;
             };
-            const bool begun = issue_s(0) && (ntiles == 1 || issue_s(1));
+            const bool begun = issue_s(0);
             for (int kt = 0; kt < ntiles && begun; ++kt) {
                 const uint32_t i = kt & 1, turn = static_cast<uint32_t>(kt >> 1) & 1u;
-                if (!mbar_wait_bounded(smem_u32(&p_full[i]), turn, p.status, 343)) break;
+                const int stage = kt % kStages;
+                // S of the next tile as soon as this one's has been read
+                if (kt + 1 < ntiles && (!mbar_wait_bounded(smem_u32(&s_free[i]), turn, p.status, 344) || !issue_s(kt + 1))) break;
+                if (!mbar_wait_bounded(smem_u32(&v_full[stage]), static_cast<uint32_t>(kt / kStages) & 1u, p.status, 347) ||
+                    !mbar_wait_bounded(smem_u32(&p_full[i]), turn, p.status, 343))
+                    break;
                 tc_fence_after();
-                // (a K/V tile's two value buffers are neighbours in the ring: one operand of 256 columns)
-                const int n = kt * parts + 1;
-                if (!filled(n) || (nv == 2 && !filled(n + 1))) break;
-                tc_fence_after();
+                const uint32_t values = smem_base + kVOff + stage * kVBytes;
 #pragma unroll
-                for (int ks = 0; ks < 8; ++ks) {
-                    // keys ks*16 .. +15: eight packed columns; keys 64-127 start at column 64
-                    const uint32_t a = tmem_base + kColS + i * 128u + static_cast<uint32_t>((ks >> 2) * 64 + (ks & 3) * 8);
-                    tc_mma_bf16_ts(tmem_base + kColO, a, mnmajor_sw128_desc(buffer(n) + ks * 2048), idesc_pv, (kt > 0 || ks > 0) ? 1u : 0u);
-                }
-                for (int j = 0; j < nv; ++j) tc_commit(smem_u32(&empty[(n + j) % kSlots]));
+                for (int ks = 0; ks < 8; ++ks)   // keys ks*16 .. +15: eight packed columns of P; both value heads' columns
+                    tc_mma_bf16_ts(tmem_base + kColO, tmem_base + kColP + i * 64u + ks * 8u, mnmajor_sw128_desc(values + ks * 2048),
+                                   idesc_pv, (kt > 0 || ks > 0) ? 1u : 0u);
+                tc_commit(smem_u32(&v_empty[stage]));
                 tc_commit(smem_u32(&pv_done[i]));
                 if (kt + 1 == ntiles) tc_commit(smem_u32(&all_done));
-                if (kt + 2 >= ntiles) continue;
-                // the next S overwrites the columns these products read P from
-                if (!mbar_wait_bounded(smem_u32(&pv_done[i]), turn, p.status, 344) || !issue_s(kt + 2)) break;
             }
         }
     } else {
@@ -260,8 +266,9 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
         auto seen = [&](int first) {
             return below(limit + 1 - first) & (~below(oldest - first) | below(p.w.keep_first - first));
         };
-        const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(qtr * 32) << 16);
-        const uint32_t s_addr = lane_addr + kColS + static_cast<uint32_t>(turn) * 128u + static_cast<uint32_t>(half * 64);
+        const uint32_t lane_addr = tmem_base_slot + (static_cast<uint32_t>(qtr * 32) << 16);
+        const uint32_t s_addr = lane_addr + kColS + static_cast<uint32_t>(half * 64);
+        const uint32_t p_addr = lane_addr + kColP + static_cast<uint32_t>(turn * 64 + half * 32);
         const float sc = p.scale_log2;
         float sum0 = 0.f, sum1 = 0.f;
         bool failed = false;
@@ -275,6 +282,9 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
             tmem_ld_32x32b_x32(s_addr, sv[0]);
             tmem_ld_32x32b_x32(s_addr + 32, sv[1]);
             tmem_ld_wait();
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(smem_u32(&s_free[turn]));
 #pragma unroll
             for (int c = 0; c < 2; ++c) {
                 if (need_mask) {   // (an exponent of -inf: no weight)
@@ -291,7 +301,12 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
                     sum1 += p1;
                     packed[i >> 1] = pack_bf16(p0, p1);
                 }
-                tmem_st_32x32b_x16(s_addr + c * 16, packed);
+                if (c == 0 && kt >= 2) {   // P of this group's last tile has been read
+                    if (!failed && !mbar_wait_bounded(smem_u32(&pv_done[turn]), static_cast<uint32_t>((kt >> 1) - 1) & 1u, p.status, 348))
+                        failed = true;
+                    tc_fence_after();
+                }
+                tmem_st_32x32b_x16(p_addr + c * 16, packed);
             }
             tmem_st_wait();
             tc_fence_before();
@@ -330,7 +345,7 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant
     __syncwarp();
     tc_fence_before();
     __syncthreads();
-    if (warp == 1) tmem_dealloc(tmem_base, 512);
+    if (warp == 1) tmem_dealloc(tmem_base_slot, 512);
 }
 
 // Half a warp per (token, key / value head), HC output heads and 64 pairs of elements at a time, four pairs per thread.
@@ -362,10 +377,10 @@ mix_kernel(const MixOutput a, const T* __restrict__ raw, int tokens) {
 #pragma unroll
                 for (int i = 0; i < HC; ++i) u[i] = v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
                 const float* w = s_mix + c * steps * HC + h0;
-#pragma unroll 8
+#pragma unroll 4
                 for (int g = 0; g < H; ++g, w += row) {
                     const T* o = src + g * from + m;
-                    const float4 x = load_quad(o, VEC, pairs - m), y = load_quad(o + pairs, VEC, pairs - m);
+                    const float4 x = load_quad<VEC>(o, pairs - m), y = load_quad<VEC>(o + pairs, pairs - m);
                     float f[HC];
                     if (HC % 4 == 0) {
 #pragma unroll
@@ -386,14 +401,11 @@ mix_kernel(const MixOutput a, const T* __restrict__ raw, int tokens) {
                         v[i].w = fmaf(f[i], y.w, v[i].w);
                     }
                 }
-                const bool more = m + 2 < pairs;
-                const Turn r = turn_of(a, t, m), r2 = more ? turn_of(a, t, m + 2) : r;
+                const Turn r = turn_of<VEC>(a, t, m);
 #pragma unroll
                 for (int i = 0; i < HC; ++i) {
                     if (h0 + i >= group) break;
-                    const int h = c * group + h0 + i;
-                    finish_mixed<T>(a, t, h, m, make_float2(u[i].x, u[i].y), make_float2(v[i].x, v[i].y), r);
-                    if (more) finish_mixed<T>(a, t, h, m + 2, make_float2(u[i].z, u[i].w), make_float2(v[i].z, v[i].w), r2);
+                    finish_mixed<T, VEC>(a, t, c * group + h0 + i, m, u[i], v[i], r);
                 }
             }
         }
