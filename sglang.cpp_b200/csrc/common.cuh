@@ -212,7 +212,10 @@ constexpr uint64_t kWaitLimitNs = 2000000000ull;  // 2 s
 // time limit ran out; the caller must then stop issuing work and unwind.
 __device__ __forceinline__ bool mbar_wait_bounded(uint32_t bar, uint32_t parity, int* status,
                                                   int site) {
-    if (mbar_try_wait(bar, parity)) return true;
+    // (reading the timer takes longer than most waits)
+#pragma unroll 1
+    for (int i = 0; i < 32; ++i)
+        if (mbar_try_wait(bar, parity)) return true;
     const uint64_t t0 = global_timer_ns();
     uint32_t spins = 0;
     while (!mbar_try_wait(bar, parity)) {

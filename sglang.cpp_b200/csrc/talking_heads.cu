@@ -35,12 +35,20 @@ constexpr uint32_t kTileBytes = kVOff + kStages * kVBytes;
 constexpr uint32_t kColS = 0, kColP = 128, kColO = 256;   // TMEM columns: S; P of even and odd tiles (64 each); O of the value heads
 constexpr float kMaxExponent = 100.f;       // log2 of the largest exponential
 
+// A work item.
+struct PrefillItem {
+    int q_begin, t0, t_end, pos0, len, table, h, c0;
+    int kv_end, head_tiles, skip, ntiles;    // ntiles 0: nothing to do; handed to the other roles, the end
+    __device__ __forceinline__ int first_key(int kt) const { return (kt >= head_tiles ? kt + skip : kt) * kTile; }
+};
 // Behind the tiles in shared memory.  Barriers in pairs: per stage, or for even and odd tiles.
 struct PrefillSync {
     float sum[4][kTile];                    // a row's weights, added up by the four threads that share it
     uint64_t k_full[kStages], k_empty[kStages], v_full[kStages], v_empty[kStages];
     uint64_t s_full[2], s_free[2], p_full[2], pv_done[2];
     uint64_t q_full, q_free, o_full, o_free;   // once per item
+    uint64_t item_seen;
+    PrefillItem item[2];                    // in place with q_full
     uint32_t tmem;
 };
 constexpr uint32_t kMaxSmem = 227 * 1024;   // (tiles start on a multiple of 1024, as the array itself should)
@@ -80,12 +88,20 @@ __device__ __forceinline__ void store_32b(void* p, const uint32_t (&v)[8]) {
                  : "memory");
 }
 
-// A work item; every role of a CTA goes through the same ones.
-struct PrefillItem {
-    int q_begin, t0, t_end, pos0, len, table, h, c0;
-    int kv_end, head_tiles, skip, ntiles;    // ntiles 0: nothing to do
-    __device__ __forceinline__ int first_key(int kt) const { return (kt >= head_tiles ? kt + skip : kt) * kTile; }
-};
+// Whether any of the softmax threads says so; all of them meet here.
+__device__ __forceinline__ bool softmax_any(bool mine) {
+    int any;
+    asm volatile(
+        "{\n\t.reg .pred p, q;\n\t"
+        "setp.ne.b32 p, %1, 0;\n\t"
+        "bar.red.or.pred q, 1, %2, p;\n\t"
+        "selp.b32 %0, 1, 0, q;\n\t}"
+        : "=r"(any)
+        : "r"(static_cast<int>(mine)), "n"(kSoftmaxThreads)
+        : "memory");
+    return any != 0;
+}
+
 __device__ __forceinline__ PrefillItem item_of(const PrefillParams& p, int index) {
     PrefillItem it = {};
     if (index >= p.items) return it;
@@ -138,6 +154,7 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant
         mbar_init(smem_u32(&S.q_full), 1);
         mbar_init(smem_u32(&S.q_free), 1);
         mbar_init(smem_u32(&S.o_full), 1);
+        mbar_init(smem_u32(&S.item_seen), 1);
         mbar_init(smem_u32(&S.o_free), kSoftmaxThreads / 32);
         fence_mbar_init();
     }
@@ -169,8 +186,9 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant
         for (int index = blockIdx.x; index < p.items && going; index += step) {
             const PrefillItem next = item_of(p, index + step);
             if (it.ntiles > 0) {
-                if (items > 0 && !wait(S.q_free, items - 1, 340)) break;
+                if (items > 0 && !(wait(S.q_free, items - 1, 340) && wait(S.item_seen, items - 1, 354))) break;
                 if (lane == 0) {
+                    S.item[items & 1] = it;
                     mbar_arrive_expect_tx(smem_u32(&S.q_full), 2 * kAtomBytes);
                     tma_load_4d(smem_base + kQOff, &tmap_q, 0, it.h * G, it.q_begin + it.t0, 0, smem_u32(&S.q_full));
                 }
@@ -236,15 +254,20 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant
             }
             it = next;
         }
+        if (going && (items == 0 || (wait(S.q_free, items - 1, 352) && wait(S.item_seen, items - 1, 355))) && lane == 0) {
+            S.item[items & 1].ntiles = 0;
+            mbar_arrive(smem_u32(&S.q_full));
+        }
     } else if (warp == 1) {
         // ================= MMA issuer =================
         if (elect_one()) {
             const uint32_t tmem = S.tmem, idesc_s = idesc_bf16_128x128(false), idesc_pv = idesc_bf16_128xn(heads_per_box * 128, true);
             int n = 0, items = 0;
             bool going = true;
-            PrefillItem it = item_of(p, blockIdx.x);
-            for (int index = blockIdx.x; index < p.items && going; index += step) {
-                const PrefillItem next = item_of(p, index + step);
+            while (going) {
+                if (!mbar_wait_bounded(smem_u32(&S.q_full), static_cast<uint32_t>(items) & 1u, p.status, 345)) break;
+                const int ntiles = S.item[items & 1].ntiles;
+                if (ntiles == 0) break;
                 auto issue_s = [&](int kt) {
                     const int g = n + kt, stage = g % kStages;
                     const uint32_t keys = smem_base + kKOff + stage * kKBytes;
@@ -261,34 +284,31 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant
                     }
                     tc_commit(smem_u32(&S.s_full[g & 1]));
                     tc_commit(smem_u32(&S.k_empty[stage]));
-                    if (kt + 1 == it.ntiles) tc_commit(smem_u32(&S.q_free));
+                    if (kt + 1 == ntiles) tc_commit(smem_u32(&S.q_free));
                     return true;
                 };
-                if (it.ntiles > 0) {
-                    going = mbar_wait_bounded(smem_u32(&S.q_full), static_cast<uint32_t>(items) & 1u, p.status, 345) && issue_s(0);
-                    for (int kt = 0; kt < it.ntiles && going; ++kt) {
-                        const int g = n + kt, stage = g % kStages;
-                        going = (kt + 1 >= it.ntiles || issue_s(kt + 1)) &&
-                                mbar_wait_bounded(smem_u32(&S.v_full[stage]), static_cast<uint32_t>(g / kStages) & 1u, p.status, 347) &&
-                                mbar_wait_bounded(smem_u32(&S.p_full[g & 1]), static_cast<uint32_t>(g >> 1) & 1u, p.status, 343) &&
-                                // O of the item before has been read
-                                (kt > 0 || items == 0 ||
-                                 mbar_wait_bounded(smem_u32(&S.o_free), static_cast<uint32_t>(items - 1) & 1u, p.status, 350));
-                        if (!going) break;
-                        tc_fence_after();
-                        const uint32_t values = smem_base + kVOff + stage * kVBytes;
+                going = issue_s(0);
+                for (int kt = 0; kt < ntiles && going; ++kt) {
+                    const int g = n + kt, stage = g % kStages;
+                    going = (kt + 1 >= ntiles || issue_s(kt + 1)) &&
+                            mbar_wait_bounded(smem_u32(&S.v_full[stage]), static_cast<uint32_t>(g / kStages) & 1u, p.status, 347) &&
+                            // O of the item before has been read
+                            (kt > 0 || items == 0 ||
+                             mbar_wait_bounded(smem_u32(&S.o_free), static_cast<uint32_t>(items - 1) & 1u, p.status, 350)) &&
+                            mbar_wait_bounded(smem_u32(&S.p_full[g & 1]), static_cast<uint32_t>(g >> 1) & 1u, p.status, 343);
+                    if (!going) break;
+                    tc_fence_after();
+                    const uint32_t values = smem_base + kVOff + stage * kVBytes;
 #pragma unroll
-                        for (int ks = 0; ks < 8; ++ks)   // keys ks*16 .. +15: eight packed columns of P; both heads' columns
-                            tc_mma_bf16_ts(tmem + kColO, tmem + kColP + (g & 1) * 64u + ks * 8u, mnmajor_sw128_desc(values + ks * 2048),
-                                           idesc_pv, (kt > 0 || ks > 0) ? 1u : 0u);
-                        tc_commit(smem_u32(&S.v_empty[stage]));
-                        tc_commit(smem_u32(&S.pv_done[g & 1]));
-                    }
-                    if (going) tc_commit(smem_u32(&S.o_full));
-                    n += it.ntiles;
-                    ++items;
+                    for (int ks = 0; ks < 8; ++ks)   // keys ks*16 .. +15: eight packed columns of P; both heads' columns
+                        tc_mma_bf16_ts(tmem + kColO, tmem + kColP + (g & 1) * 64u + ks * 8u, mnmajor_sw128_desc(values + ks * 2048),
+                                       idesc_pv, (kt > 0 || ks > 0) ? 1u : 0u);
+                    tc_commit(smem_u32(&S.v_empty[stage]));
+                    tc_commit(smem_u32(&S.pv_done[g & 1]));
+                    if (kt + 1 == ntiles) tc_commit(smem_u32(&S.o_full));
                 }
-                it = next;
+                n += ntiles;
+                ++items;
             }
         }
     } else {
@@ -309,85 +329,102 @@ prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant
             if (!failed && !mbar_wait_bounded(smem_u32(&bar), static_cast<uint32_t>(phase) & 1u, p.status, site)) failed = true;
             tc_fence_after();
         };
-        PrefillItem it = item_of(p, blockIdx.x);
-        for (int index = blockIdx.x; index < p.items; index += step) {
-            const PrefillItem next = item_of(p, index + step);
-            if (it.ntiles > 0) {
-                const int tok = it.t0 + r / G;
-                const int limit = min(it.pos0 + tok, it.len - 1);   // last visible key of this row
-                const int oldest = p.w.oldest(limit);               // keys before it are seen below keep_first only
-                // which of the 32 keys from `first` on this row sees, as bits
-                auto below = [](int m) { return m <= 0 ? 0u : m >= 32 ? 0xffffffffu : (1u << m) - 1u; };
-                auto seen = [&](int first) {
-                    return below(limit + 1 - first) & (~below(oldest - first) | below(p.w.keep_first - first));
-                };
-                float sum0 = 0.f, sum1 = 0.f;
-                for (int kt = (n & 1) ^ turn; kt < it.ntiles; kt += 2, ++mine) {
-                    wait(S.s_full[turn], mine, 346);
-                    const int k0 = it.first_key(kt) + half * 64;    // first key of this thread's columns
-                    const bool need_mask = __any_sync(0xffffffffu, k0 + 63 > limit || (k0 < oldest && k0 + 63 >= p.w.keep_first));
-                    uint32_t sv[2][32];
-                    tmem_ld_32x32b_x32(s_addr, sv[0]);
-                    tmem_ld_32x32b_x32(s_addr + 32, sv[1]);
-                    tmem_ld_wait();
-                    tc_fence_before();
-                    __syncwarp();
-                    if (lane == 0) mbar_arrive(smem_u32(&S.s_free[turn]));
-                    if (mine > 0) wait(S.pv_done[turn], mine - 1, 348);   // P of this group's last tile has been read
-#pragma unroll
-                    for (int c = 0; c < 2; ++c) {
-                        if (need_mask) {   // (an exponent of -inf: no weight)
-                            const uint32_t bits = seen(k0 + c * 32);
-#pragma unroll
-                            for (int i = 0; i < 32; ++i)
-                                if ((bits & (1u << i)) == 0) sv[c][i] = 0xff800000u;
-                        }
-                        uint32_t packed[16];
-#pragma unroll
-                        for (int i = 0; i < 32; i += 2) {
-                            const float p0 = ex2(__uint_as_float(sv[c][i]) * sc), p1 = ex2(__uint_as_float(sv[c][i + 1]) * sc);
-                            sum0 += p0;
-                            sum1 += p1;
-                            packed[i >> 1] = pack_bf16(p0, p1);
-                        }
-                        tmem_st_32x32b_x16(p_addr + c * 16, packed);
-                    }
-                    tmem_st_wait();
-                    tc_fence_before();
-                    __syncwarp();
-                    if (lane == 0) mbar_arrive(smem_u32(&S.p_full[turn]));
-                }
-                // O over the sum of the row's four partial sums (once everybody has read the last item's)
-                asm volatile("bar.sync 1, %0;" ::"n"(kSoftmaxThreads) : "memory");
-                S.sum[turn * 2 + half][r] = sum0 + sum1;
-                asm volatile("bar.sync 1, %0;" ::"n"(kSoftmaxThreads) : "memory");
-                const float l = (S.sum[0][r] + S.sum[1][r]) + (S.sum[2][r] + S.sum[3][r]);
-                wait(S.o_full, items, 351);
-                uint32_t ov[2][32];
-                tmem_ld_32x32b_x32(o_addr, ov[0]);
-                tmem_ld_32x32b_x32(o_addr + 32, ov[1]);
+        while (true) {
+            wait(S.q_full, items, 353);
+            const PrefillItem it = S.item[items & 1];
+            if (softmax_any(failed || it.ntiles == 0)) break;   // (everybody has read the last item's sums as well)
+            if (threadIdx.x == 64) mbar_arrive(smem_u32(&S.item_seen));
+            const int tok = it.t0 + r / G;
+            const int limit = min(it.pos0 + tok, it.len - 1);   // last visible key of this row
+            const int oldest = p.w.oldest(limit);               // keys before it are seen below keep_first only
+            // which of the 32 keys from `first` on this row sees, as bits
+            auto below = [](int m) { return m <= 0 ? 0u : m >= 32 ? 0xffffffffu : (1u << m) - 1u; };
+            auto seen = [&](int first) {
+                return below(limit + 1 - first) & (~below(oldest - first) | below(p.w.keep_first - first));
+            };
+            float sum0 = 0.f, sum1 = 0.f;
+            for (int kt = (n & 1) ^ turn; kt < it.ntiles; kt += 2, ++mine) {
+                wait(S.s_full[turn], mine, 346);
+                const int k0 = it.first_key(kt) + half * 64;    // first key of this thread's columns
+                const bool need_mask = __any_sync(0xffffffffu, k0 + 63 > limit || (k0 < oldest && k0 + 63 >= p.w.keep_first));
+                uint32_t sv[2][32];
+                tmem_ld_32x32b_x32(s_addr, sv[0]);
+                tmem_ld_32x32b_x32(s_addr + 32, sv[1]);
                 tmem_ld_wait();
                 tc_fence_before();
                 __syncwarp();
-                if (lane == 0) mbar_arrive(smem_u32(&S.o_free));   // (the sums have been read as well)
-                if (it.c0 + turn < p.kv_heads && tok < it.t_end && !failed) {
-                    const float inv = l > 0.f ? 1.f / l : 0.f;
-                    const int64_t row = (static_cast<int64_t>(it.q_begin + tok) * p.q_heads + it.h * G + r % G) * p.kv_heads + it.c0 + turn;
-                    __nv_bfloat16* dst = p.raw + row * kD + half * 64;
+                if (lane == 0) mbar_arrive(smem_u32(&S.s_free[turn]));
+                if (mine > 0) wait(S.pv_done[turn], mine - 1, 348);   // P of this group's last tile has been read
+#pragma unroll
+                for (int c = 0; c < 2; ++c) {
+                    if (need_mask) {   // (an exponent of -inf: no weight)
+                        const uint32_t bits = seen(k0 + c * 32);
+#pragma unroll
+                        for (int i = 0; i < 32; ++i)
+                            if ((bits & (1u << i)) == 0) sv[c][i] = 0xff800000u;
+                    }
+                    uint32_t packed[16];
+#pragma unroll
+                    for (int i = 0; i < 32; i += 2) {
+                        const float p0 = ex2(__uint_as_float(sv[c][i]) * sc), p1 = ex2(__uint_as_float(sv[c][i + 1]) * sc);
+                        sum0 += p0;
+                        sum1 += p1;
+                        packed[i >> 1] = pack_bf16(p0, p1);
+                    }
+                    tmem_st_32x32b_x16(p_addr + c * 16, packed);
+                }
+                tmem_st_wait();
+                tc_fence_before();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(smem_u32(&S.p_full[turn]));
+            }
+            // O over the sum of the row's four partial sums
+            S.sum[turn * 2 + half][r] = sum0 + sum1;
+            asm volatile("bar.sync 1, %0;" ::"n"(kSoftmaxThreads) : "memory");
+            const float l = (S.sum[0][r] + S.sum[1][r]) + (S.sum[2][r] + S.sum[3][r]);
+            wait(S.o_full, items, 351);
+            uint32_t ov[2][32];
+            tmem_ld_32x32b_x32(o_addr, ov[0]);
+            tmem_ld_32x32b_x32(o_addr + 32, ov[1]);
+            tmem_ld_wait();
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(smem_u32(&S.o_free));   // (the sums have been read as well)
+            if (it.c0 + turn < p.kv_heads) {
+                // Four neighbouring threads exchange quarters of their rows (16 columns, 32 bytes), so that they store
+                // whole ones: of the row of thread `row` of the four, this thread gets its own quarter.
+                const float inv = l > 0.f ? 1.f / l : 0.f;
+                const int me = lane & 3;
+                uint32_t w[4][8];   // [quarter]
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+#pragma unroll
+                    for (int j = 0; j < 8; ++j)
+                        w[c][j] = pack_bf16(__uint_as_float(ov[c >> 1][(c & 1) * 16 + 2 * j]) * inv,
+                                            __uint_as_float(ov[c >> 1][(c & 1) * 16 + 2 * j + 1]) * inv);
+#pragma unroll
+                for (int bit = 1; bit < 4; bit <<= 1)   // rows and quarters trade places, a bit of their numbers at a time
 #pragma unroll
                     for (int c = 0; c < 4; ++c) {
-                        uint32_t w[8];
+                        if (c & bit) continue;
 #pragma unroll
-                        for (int j = 0; j < 8; ++j)
-                            w[j] = pack_bf16(__uint_as_float(ov[c >> 1][(c & 1) * 16 + 2 * j]) * inv,
-                                             __uint_as_float(ov[c >> 1][(c & 1) * 16 + 2 * j + 1]) * inv);
-                        store_32b(dst + c * 16, w);
+                        for (int j = 0; j < 8; ++j) {
+                            const bool upper = (me & bit) != 0;
+                            const uint32_t give = upper ? w[c][j] : w[c | bit][j];
+                            const uint32_t got = __shfl_xor_sync(0xffffffffu, give, bit);
+                            if (upper) w[c][j] = got;
+                            else w[c | bit][j] = got;
+                        }
                     }
+#pragma unroll
+                for (int c = 0; c < 4; ++c) {
+                    const int row = (r & ~3) + c, tok_c = it.t0 + row / G;
+                    const int64_t at = (static_cast<int64_t>(it.q_begin + tok_c) * p.q_heads + it.h * G + row % G) * p.kv_heads + it.c0 + turn;
+                    if (tok_c < it.t_end && !failed) store_32b(p.raw + at * kD + half * 64 + me * 16, w[c]);
                 }
-                n += it.ntiles;
-                ++items;
             }
-            it = next;
+            n += it.ntiles;
+            ++items;
         }
     }
     __syncwarp();
