@@ -112,9 +112,14 @@ __device__ __forceinline__ void consumer_bar() {
     asm volatile("bar.sync 1, %0;" ::"n"(kConsumerThreads) : "memory");
 }
 
+// Mixing heads: the producer is one warp of a warpgroup that leaves its registers to the consumers; 384 x 168 are launched.
+constexpr int kMixingThreads = kConsumerThreads + 128;
+constexpr int kProducerRegs = 72, kConsumerRegs = 216;
+static_assert(128 * kProducerRegs + kConsumerThreads * kConsumerRegs <= kMixingThreads * 168, "");
+
 // KEY_GROUPS: 16-key groups per stage (8 / kv_heads), with MT only.
 template <bool WINDOW, int MT, int KEY_GROUPS>
-__global__ void __launch_bounds__(kThreads, 1)
+__global__ void __launch_bounds__(MT > 0 ? kMixingThreads : kThreads, 1)
 attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
                         const __grid_constant__ CUtensorMap tmap_v, const DecodeParams p) {
     extern __shared__ uint8_t smem_raw[];
@@ -139,7 +144,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
         fence_mbar_init();
     }
     if (MT > 0)
-        for (int i = threadIdx.x; i < 2 * MT * 16 * kPRow; i += kThreads) s_p[0][i] = __float2bfloat16_rn(0.f);
+        for (int i = threadIdx.x; i < 2 * MT * 16 * kPRow; i += kMixingThreads) s_p[0][i] = __float2bfloat16_rn(0.f);
     if (warp == kConsumerWarps && lane == 0) {
         tma_prefetch_desc(&tmap_k);
         tma_prefetch_desc(&tmap_v);
@@ -220,6 +225,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
     bool failed = false;
     uint32_t it_count = 0;  // stages consumed / produced so far by this CTA
 
+    if (MT > 0 && warp >= kConsumerWarps) asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(kProducerRegs));
+    if (MT > 0 && warp > kConsumerWarps) return;
     if (warp == kConsumerWarps) {
         // ================= producer warp =================
         const uint32_t copy_bytes = static_cast<uint32_t>(p.kpc) * Hkv * 128u;  // one half-tile box
@@ -287,6 +294,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
     }
 
     // ================= consumer warps =================
+    if (MT > 0) asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(kConsumerRegs));
     const int h = warp % Hkv;       // KV head of this warp
     const int kg = warp / Hkv;      // 16-key group inside a stage
     const int G = p.group;
@@ -294,11 +302,12 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
     const int mi = lane >> 3, r8 = lane & 7;
 
     // Query fragments: rows of the A operand are the G heads of this KV group.
+    constexpr bool kManyRows = MT == 0 || 2 * MT * KEY_GROUPS > 8;   // groups of more than 8 heads are possible
     uint32_t qa[8][4];
     auto load_q = [&](int b) {
         const __nv_bfloat16* q0 = p.q + b * p.q_st + static_cast<int64_t>(h * G + g) * p.q_sh;
         const __nv_bfloat16* q1 = q0 + 8 * p.q_sh;
-        const bool r0 = g < G, r1 = (g + 8) < G;
+        const bool r0 = g < G, r1 = kManyRows && (g + 8) < G;
 #pragma unroll
         for (int ks = 0; ks < 8; ++ks) {
             const int d0 = ks * 16 + 2 * t;
@@ -356,7 +365,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
 #pragma unroll
                     for (int e = 0; e < 8; ++e) {
                         const int key = (e >> 2) * 8 + 2 * t + (e & 1);
-                        const bool sees = key < nvalid && (key0 + key >= oldest || key0 + key < p.w.keep_first);
+                        const bool sees = (kManyRows || (e & 2) == 0) && key < nvalid && (key0 + key >= oldest || key0 + key < p.w.keep_first);
                         x[e] = sees ? exp2f((e < 4 ? s0[e] : s1[e - 4]) * p.scale_log2) : 0.f;
                     }
                     l0 += (x[0] + x[1]) + (x[4] + x[5]);
@@ -371,7 +380,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
                     uint32_t* row = reinterpret_cast<uint32_t*>(P + (h * G + g) * kPRow + kg * 16 + 2 * t);
                     if (g < G) row[0] = w[0], row[4] = w[2];
                     row += 8 * (kPRow / 2);
-                    if (g + 8 < G) row[0] = w[1], row[4] = w[3];
+                    if (kManyRows && g + 8 < G) row[0] = w[1], row[4] = w[3];
                 }
                 consumer_bar();   // (the other buffer's readers are through: they have been at this barrier)
                 // ---- all heads' weights times this warp's columns of its head's values ----
@@ -405,7 +414,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap tmap_k,
             l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
             float* l = p.ws_l + (static_cast<int64_t>(it.item) * KG + kg) * Hq + h * G + g;
             if (t == 0 && g < G) l[0] = l0;
-            if (t == 0 && g + 8 < G) l[8] = l1;
+            if (kManyRows && t == 0 && g + 8 < G) l[8] = l1;
 #pragma unroll
             for (int i = 0; i < MT; ++i)
 #pragma unroll
@@ -865,7 +874,7 @@ int launch_talking_decode(const WindowAttention& a, cudaStream_t stream) {
     auto kernel = talking_kernel(a.heads, a.kv_heads);
     const int smem = kStages * kStageBytes + 1024;
     B200_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-    B200_CHECK_CUDA(launch_kernel(kernel, dim3(grid), dim3(kThreads), smem, stream, dim3(1, 1, 1), tk, tv, p));
+    B200_CHECK_CUDA(launch_kernel(kernel, dim3(grid), dim3(kMixingThreads), smem, stream, dim3(1, 1, 1), tk, tv, p));
     const MixOutput m = mix_output(a);
     auto mix = m.pairs() % 4 == 0 ? decode_mix_for<true>(p.group) : decode_mix_for<false>(p.group);
     B200_CHECK_CUDA(launch_kernel(mix, dim3(a.batch, a.kv_heads), dim3(kMixThreads), 0, stream, dim3(1, 1, 1), p, m, grid));
